@@ -6,8 +6,10 @@ silent Python fallback: if a library is missing, the first use raises and names 
 """
 from __future__ import annotations
 
+import contextlib
 import ctypes
 import os
+import sys
 from pathlib import Path
 
 _LIB_DIR = Path(__file__).resolve().parent / "_lib"
@@ -19,8 +21,25 @@ class NativeLibraryMissing(RuntimeError):
     pass
 
 
+_subset = None
+
+
+def use_subset(name: str) -> None:
+    """Before the first native call: a library that is not built yet is built (and loaded) as the subset ``build.SUBSETS[name]`` instead of
+    in full.  A full library that is there is used."""
+    global _subset
+    from . import build as _build
+    if name not in _build.SUBSETS:
+        raise ValueError(f"unknown library subset {name!r}")
+    _subset = name
+
+
 def _load(name: str):
     path = _LIB_DIR / name
+    if _subset is not None and not path.exists() and name in ("libgb_cuda.so", "libgb_host.so"):
+        from . import build as _build
+        with contextlib.redirect_stdout(sys.stderr):
+            path = _build.build_subset(_subset, host=name == "libgb_host.so")
     if not path.exists():
         if os.environ.get("GEMM_B200_AUTOBUILD", "1") != "0":
             from . import build as _build

@@ -85,6 +85,31 @@ def _build_lib(name, sources, compiler_cmd, link_cmd, hdr_time, force, verbose, 
 SHARED_HEADER = CSRC / "kernels" / "geometry.cuh"      # inline code the host library compiles too (host/geometry_host.cc)
 
 
+# Parts of the two libraries that suffice for one model family: a program that serves nothing else compiles no more than this.
+# name -> (CUDA sources, extra nvcc flags, host sources)
+SUBSETS = {
+    "layered": (["runtime", "elementwise", "gemm_tc", "gemm_f32", "flash_attn", "attn_any", "stream_ops", "lightning", "sampler"],
+                ["-DGB_GEMM_BF16_ONLY"], ["common", "runtime", "safetensors"]),
+}
+
+
+def build_subset(name: str, host: bool, force=False, verbose=False) -> Path:
+    """``_lib/libgb_cuda_<name>.so`` or ``_lib/libgb_host_<name>.so``: the part of the library listed in ``SUBSETS``."""
+    cu, flags, cc = SUBSETS[name]
+    tag = "_" + name
+    if host:
+        cxx = os.environ.get("CXX", "g++")
+        return _build_lib(f"libgb_host_{name}.so", [CSRC / "host" / (s + ".cc") for s in cc], [cxx] + CXX_FLAGS + ["-I", str(CSRC / "host")],
+                          [cxx, "-shared", "-pthread"], _newest_header([CSRC / "host"]), force, verbose, tag=tag)
+    nvcc = _nvcc()
+    if nvcc is None:
+        raise RuntimeError("nvcc not found; cannot build the sm_100a kernels")
+    inc = ["-I", str(CSRC / "kernels"), "-I", str(CSRC / "fabric")]
+    return _build_lib(f"libgb_cuda_{name}.so", [CSRC / "kernels" / (s + ".cu") for s in cu], [nvcc] + NVCC_FLAGS + flags + inc,
+                      [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a"], _newest_header([CSRC / "kernels", CSRC / "fabric"]), force, verbose,
+                      tag=tag)
+
+
 def build_host(force=False, verbose=False) -> Path:
     srcs = sorted((CSRC / "host").glob("*.cc"))
     hdr = max(_newest_header([CSRC / "host"]), SHARED_HEADER.stat().st_mtime)

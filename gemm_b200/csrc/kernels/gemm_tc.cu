@@ -10,7 +10,7 @@
 //   MODE 0  bf16 x bf16  (kind::f16)
 //   MODE 1  MXFP8: e4m3 x e4m3 with one E8M0 scale per 32 K-elements on both operands
 //           (kind::mxf8f6f4.block_scale; scale factors copied smem -> TMEM with tcgen05.cp)
-//   DUAL    two weight tiles (gate rows, up rows) share one token tile; epilogue = SiLU(gate) * up
+//   DUAL    two weight tiles (gate rows, up rows) share one token tile; epilogue = SiLU(gate) * up (or GELU(gate) * up)
 //   grouped (run time)  one weight matrix per group (expert); every group owns a row segment of X
 //           described by device arrays, so no host synchronisation is needed after routing.
 // Epilogues: bf16 / f32 store with optional bias, per-row scale and row scatter; or MXFP8
@@ -83,6 +83,7 @@ struct GemmArgs {
   int early_weights;  // != 0: a plain decode-sized launch requests its first weight tiles before the dependency wait
   int dual_raw;  // DUAL without the activation: the second accumulator is the row block up_row_offset further down the same matrix
   int w_tiled;
+  int act;       // activation of the gate half of a DUAL launch: 0 = SiLU, 1 = the tanh form of GELU
 };
 
 // k-steps whose MXFP8 scale atoms are fetched by one bulk copy (2 for the widest tile, whose stages are short of room)
@@ -128,6 +129,11 @@ struct TileCursor {
 };
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
+// Gate activation.  The tanh form of GELU, x (1 + tanh u) / 2 with u = sqrt(2 / pi) (x + 0.044715 x^3), is x / (1 + exp(-2 u)).
+__device__ __forceinline__ float gate_act(float x, int act) {
+  const float z = act == 1 ? 1.5957691216057308f * (x + 0.044715f * x * x * x) : x;
+  return x / (1.0f + __expf(-z));
+}
 
 // E8M0 exponent for a block whose absolute maximum is `amax`: the smallest power of two s with
 // amax / s <= 448 (largest e4m3 magnitude), so quantisation never saturates.
@@ -400,7 +406,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         for (int j = 0; j < 16; ++j) {
           const int xr = c + j;
           float v = __uint_as_float(r0[j]);
-          if (DUAL) v = silu_f(v) * __uint_as_float(r1[j]);
+          if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
           v += bias;
           const bool live = xr < t.valid;
           const int x_row = t.x_row0 + xr;
@@ -604,7 +610,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               float v = __uint_as_float(r0[j]);
-              if (DUAL) v = silu_f(v) * __uint_as_float(r1[j]);
+              if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
               v += bias;
               if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
               else o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v);
@@ -613,7 +619,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               float v = __uint_as_float(r0[j]);
-              if (DUAL) v = silu_f(v) * __uint_as_float(r1[j]);
+              if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
               v += bias;
               if (c + j < t.valid) {
                 if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
@@ -731,7 +737,7 @@ struct GemmExtras {
 };
 
 // Flags of gb_gemm.
-enum { GEMM_MX = 1, GEMM_DUAL = 2, GEMM_QUANT_OUT = 4, GEMM_OUT_F32 = 8, GEMM_W_TILED = 16, GEMM_DUAL_RAW = 32 };
+enum { GEMM_MX = 1, GEMM_DUAL = 2, GEMM_QUANT_OUT = 4, GEMM_OUT_F32 = 8, GEMM_W_TILED = 16, GEMM_DUAL_RAW = 32, GEMM_GELU = 64 };
 
 // Linear layer on tensor cores.
 //   w        [w_rows, k] row-major (bf16, or e4m3 bytes when GEMM_MX), w_rows = groups * w_rows_per_group
@@ -785,6 +791,7 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
     a.early_weights = early;
   }
   a.dual_raw = (flags & GEMM_DUAL_RAW) ? 1 : 0;
+  a.act = (flags & GEMM_GELU) ? 1 : 0;
   if (a.dual_raw && (!dual || qo)) return fail("gemm: GEMM_DUAL_RAW needs GEMM_DUAL without GEMM_QUANT_OUT%s");
   a.out_sf = (uint8_t*)out_sf; a.bias = bias; a.row_map = row_map; a.row_scale = row_scale; a.status = (KernelStatus*)status;
   if (ex != nullptr) {
@@ -821,6 +828,14 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
   a.m_tok_hint = num_groups == 0 ? m_tok : (tn <= 32 ? tn : 1 << 20);
   if (num_groups == 0 && m_tok <= 0) return 0;
 
+#ifdef GB_GEMM_BF16_ONLY
+  // build without the MXFP8 variants: the library subset of models whose weights are bf16 or f32
+#define GB_DISPATCH(TNV)                                                                                      \
+  if (tn == TNV) {                                                                                            \
+    if (!mx && !dual && !qo) return launch_gemm<TNV, 0, false, false>(tmW, tmX, a, max_tiles, stream);        \
+    if (!mx && dual && !qo) return launch_gemm<TNV, 0, true, false>(tmW, tmX, a, max_tiles, stream);          \
+  }
+#else
 #define GB_DISPATCH(TNV)                                                                                      \
   if (tn == TNV) {                                                                                            \
     if (!mx && !dual && !qo) return launch_gemm<TNV, 0, false, false>(tmW, tmX, a, max_tiles, stream);        \
@@ -830,12 +845,15 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
     if (mx && dual && !qo) return launch_gemm<TNV, 1, true, false>(tmW, tmX, a, max_tiles, stream);           \
     if (!mx && dual && qo) return launch_gemm<TNV, 0, true, true>(tmW, tmX, a, max_tiles, stream);            \
   }
+#endif
   GB_DISPATCH(16)
   GB_DISPATCH(32)
   GB_DISPATCH(64)
   GB_DISPATCH(128)
   if (tn == 256 && !mx && !dual && !qo) return launch_gemm<256, 0, false, false>(tmW, tmX, a, max_tiles, stream);
+#ifndef GB_GEMM_BF16_ONLY
   if (tn == 256 && mx && !dual && !qo) return launch_gemm<256, 1, false, false>(tmW, tmX, a, max_tiles, stream);
+#endif
 #undef GB_DISPATCH
   return fail("gemm: unsupported variant%s (tn=%ld flags=%ld)", "", (long)tn, (long)flags);
 }

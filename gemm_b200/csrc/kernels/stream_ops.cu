@@ -1,0 +1,383 @@
+// Token-wise kernels of models that keep their residual stream in 32-bit floats (models described layer by layer):
+//   embed_f32           rows of a bf16 / f32 embedding table -> f32 stream
+//   stream_norm         stream += pending update (bf16, f32, or K-split fp32 partial sums of a projection) [+ a vector added to
+//                       every row], then RMSNorm of the row with an f32 weight -> bf16 or f32 rows for the next projection
+//   qk_unit_store       fused Q | K | V rows -> Q / K divided by their root mean square per head (no weight), K / V into their
+//                       cache slots, Q scaled and laid out for the attention kernels
+//   gated_norm          RMSNorm over all heads' outputs together, times sigmoid(gate): the tail of a linear-attention mixer
+//   act_mul             act(gate) * up of f32 rows (the 32-bit path; the bf16 path has it in the GEMM epilogue)
+// One pass over HBM each; sizes are arbitrary (vector paths when they divide).  Output rows may be wider than the data (padding to
+// the 16-byte row pitch the TMA descriptors of the next GEMM need); the padding is written as zero.
+//
+// The bf16-stream counterparts are in elementwise.cu (reference: common/transformer.h:593-637, :1281-1315).
+#include "sm100.cuh"
+#include "host_common.h"
+#include <algorithm>
+
+namespace gb {
+
+__device__ __forceinline__ float ld_f(const float* p) { return *p; }
+__device__ __forceinline__ float ld_f(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void st_f(float* p, float v) { *p = v; }
+__device__ __forceinline__ void st_f(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
+
+// four consecutive elements (aligned)
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 ld4(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+__device__ __forceinline__ void st4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void st4(__nv_bfloat16* p, float4 v) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v.x, v.y), pack_bf16x2(v.z, v.w));
+}
+
+// Sum over the block (256 threads); every thread gets it.
+__device__ __forceinline__ float block_sum_256(float v, float* red) {
+  v = warp_sum(v);
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float s = 0.f;
+#pragma unroll
+  for (int i = 0; i < 8; ++i) s += red[i];
+  return s;
+}
+
+// ------------------------------------------------------------------------------------------ embed
+template <typename T>
+__global__ void embed_f32_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out, int width, int vocab) {
+  pdl_wait();
+  pdl_trigger();
+  const int t = blockIdx.x;
+  int id = ids[t];
+  if (id < 0 || id >= vocab) id = 0;
+  for (int i = threadIdx.x; i < width; i += blockDim.x) out[(size_t)t * width + i] = ld_f(table + (size_t)id * width + i);
+}
+
+// ------------------------------------------------------------------------------------------ stream norm
+struct StreamNormArgs {
+  float* x;                     // stream [rows, width]
+  const void* delta;            // pending update: f32 / bf16 [n_part][rows, ld_delta]; null = none
+  int n_part; long part_stride; // K-split partial sums: slabs `part_stride` elements apart, added in order
+  int ld_delta;
+  const float* add;             // vector added to every row after the update; null = none
+  const float* weight;          // f32 [width]
+  const long long* rows;        // output row r comes from stream row rows[r] (then the stream is not written); null = all rows in place
+  void* out; int ld_out;        // normalised rows, ld_out >= width, the columns behind `width` are zeroed; null = only update the stream
+  int width; float eps;
+};
+
+template <typename TD, typename TO, int VPT>       // VPT float4 per thread, width <= 1024 * VPT and width % 4 == 0
+__global__ void __launch_bounds__(256)
+stream_norm_vec_kernel(const StreamNormArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[8];
+  const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
+  float* x = a.x + src * a.width;
+  const TD* d = a.delta != nullptr ? (const TD*)a.delta + src * a.ld_delta : nullptr;
+  const int nv = a.width >> 2;
+  float4 v[VPT];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * 256;
+    if (c >= nv) continue;
+    v[i] = ld4(x + c * 4);
+    if (d != nullptr) {
+      float4 s = ld4(d + c * 4);
+      for (int p = 1; p < a.n_part; ++p) {
+        const float4 q = ld4(d + (size_t)p * a.part_stride + c * 4);
+        s.x += q.x; s.y += q.y; s.z += q.z; s.w += q.w;
+      }
+      v[i].x += s.x; v[i].y += s.y; v[i].z += s.z; v[i].w += s.w;
+    }
+    if (a.add != nullptr) {
+      const float4 q = ld4(a.add + c * 4);
+      v[i].x += q.x; v[i].y += q.y; v[i].z += q.z; v[i].w += q.w;
+    }
+    if (a.rows == nullptr && (d != nullptr || a.add != nullptr)) st4(x + c * 4, v[i]);
+    ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+  }
+  if (a.out == nullptr) return;
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.width + a.eps);
+  TO* o = (TO*)a.out + r * a.ld_out;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * 256;
+    if (c >= nv) continue;
+    const float4 w = ld4(a.weight + c * 4);
+    st4(o + c * 4, make_float4(v[i].x * inv * w.x, v[i].y * inv * w.y, v[i].z * inv * w.z, v[i].w * inv * w.w));
+  }
+  for (int c = a.width + threadIdx.x; c < a.ld_out; c += 256) st_f(o + c, 0.f);
+}
+
+template <typename TD, typename TO>                // any width
+__global__ void __launch_bounds__(256)
+stream_norm_any_kernel(const StreamNormArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[8];
+  const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
+  float* x = a.x + src * a.width;
+  const TD* d = a.delta != nullptr ? (const TD*)a.delta + src * a.ld_delta : nullptr;
+  auto value = [&](int c) {
+    float v = x[c];
+    if (d != nullptr) {
+      float s = ld_f(d + c);
+      for (int p = 1; p < a.n_part; ++p) s += ld_f(d + (size_t)p * a.part_stride + c);
+      v += s;
+    }
+    if (a.add != nullptr) v += a.add[c];
+    return v;
+  };
+  const bool in_place = a.rows == nullptr;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < a.width; c += 256) {
+    const float v = value(c);
+    if (in_place) x[c] = v;
+    ss += v * v;
+  }
+  if (a.out == nullptr) return;
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.width + a.eps);
+  TO* o = (TO*)a.out + r * a.ld_out;
+  for (int c = threadIdx.x; c < a.width; c += 256) st_f(o + c, (in_place ? x[c] : value(c)) * inv * a.weight[c]);
+  for (int c = a.width + threadIdx.x; c < a.ld_out; c += 256) st_f(o + c, 0.f);
+}
+
+// ------------------------------------------------------------------------------------------ Q / K unit norm + cache store
+struct QkUnitArgs {
+  const void* qkv;              // [n_part][tokens, ld]: rows [Q heads | K heads | V heads]
+  int n_part; long part_stride; int ld;
+  const int* slots;             // [tokens] cache slot (-1 = not stored)
+  void* q_out;                  // [tokens, hq, dkp]
+  void* k_cache; void* v_cache; // [slots, hkv, dkp] / [slots, hkv, dvp]
+  long num_slots;
+  int hq, hkv, dk, dv, dkp, dvp;
+  float eps, q_scale;
+  int unit;                     // 0: no normalisation
+};
+
+// One warp per (token, head): heads 0 .. hq-1 are queries, then hkv keys, then hkv values.
+template <typename TI, typename TC>
+__global__ void __launch_bounds__(256)
+qk_unit_store_kernel(const QkUnitArgs a, long n_items) {
+  pdl_wait();
+  pdl_trigger();
+  const long w = ((long)blockIdx.x * 256 + threadIdx.x) >> 5;
+  if (w >= n_items) return;
+  const int lane = threadIdx.x & 31;
+  const int per = a.hq + 2 * a.hkv;
+  const long t = w / per;
+  const int h = (int)(w - t * per);
+  const bool is_q = h < a.hq, is_k = !is_q && h < a.hq + a.hkv;
+  const int d = (is_q || is_k) ? a.dk : a.dv, dp = (is_q || is_k) ? a.dkp : a.dvp;
+  const int col = is_q ? h * a.dk : is_k ? a.hq * a.dk + (h - a.hq) * a.dk : (a.hq + a.hkv) * a.dk + (h - a.hq - a.hkv) * a.dv;
+  const TI* src = (const TI*)a.qkv + (size_t)t * a.ld + col;
+  TC* dst;
+  if (is_q) dst = (TC*)a.q_out + ((size_t)t * a.hq + h) * a.dkp;
+  else {
+    const int slot = a.slots[t];
+    if (slot < 0 || slot >= a.num_slots) return;
+    dst = is_k ? (TC*)a.k_cache + ((size_t)slot * a.hkv + (h - a.hq)) * a.dkp
+               : (TC*)a.v_cache + ((size_t)slot * a.hkv + (h - a.hq - a.hkv)) * a.dvp;
+  }
+  auto value = [&](int c) {
+    float s = ld_f(src + c);
+    for (int p = 1; p < a.n_part; ++p) s += ld_f(src + (size_t)p * a.part_stride + c);
+    return s;
+  };
+  const bool norm = a.unit && (is_q || is_k);
+  if (d <= 128) {               // the head's values stay in registers
+    float v[4];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { const int c = lane + 32 * i; v[i] = c < d ? value(c) : 0.f; ss += v[i] * v[i]; }
+    float sc = 1.0f;
+    if (norm) sc = 1.0f / sqrtf(warp_sum(ss) / (float)d + a.eps);
+    if (is_q) sc *= a.q_scale;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { const int c = lane + 32 * i; if (c < dp) st_f(dst + c, v[i] * sc); }
+    return;
+  }
+  float sc = 1.0f;
+  if (norm) {
+    float ss = 0.f;
+    for (int c = lane; c < d; c += 32) { const float v = value(c); ss += v * v; }
+    sc = 1.0f / sqrtf(warp_sum(ss) / (float)d + a.eps);
+  }
+  if (is_q) sc *= a.q_scale;
+  for (int c = lane; c < dp; c += 32) st_f(dst + c, c < d ? value(c) * sc : 0.f);
+}
+
+// ------------------------------------------------------------------------------------------ gated norm
+struct GatedNormArgs {
+  const float* o; int ld_o;     // [rows, n] f32
+  const void* gate; int n_part; long part_stride; int ld_gate;     // gate pre-activations (columns of the mixer's input projection)
+  const float* weight;          // f32 [n]
+  void* out; int ld_out; int n; float eps;
+};
+
+template <typename TG, typename TO, int VPT>       // n % 4 == 0 and n <= 1024 * VPT
+__global__ void __launch_bounds__(256)
+gated_norm_vec_kernel(const GatedNormArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[8];
+  const size_t r = blockIdx.x;
+  const float* o = a.o + r * a.ld_o;
+  const TG* g = (const TG*)a.gate + r * a.ld_gate;
+  const int nv = a.n >> 2;
+  float4 v[VPT], gv[VPT];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * 256;
+    if (c >= nv) continue;
+    v[i] = ld4(o + c * 4);
+    gv[i] = ld4(g + c * 4);
+    for (int p = 1; p < a.n_part; ++p) {
+      const float4 q = ld4(g + (size_t)p * a.part_stride + c * 4);
+      gv[i].x += q.x; gv[i].y += q.y; gv[i].z += q.z; gv[i].w += q.w;
+    }
+    ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+  }
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.n + a.eps);
+  TO* out = (TO*)a.out + r * a.ld_out;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * 256;
+    if (c >= nv) continue;
+    const float4 w = ld4(a.weight + c * 4);
+    st4(out + c * 4, make_float4(v[i].x * inv * w.x / (1.0f + expf(-gv[i].x)), v[i].y * inv * w.y / (1.0f + expf(-gv[i].y)),
+                                 v[i].z * inv * w.z / (1.0f + expf(-gv[i].z)), v[i].w * inv * w.w / (1.0f + expf(-gv[i].w))));
+  }
+  for (int c = a.n + threadIdx.x; c < a.ld_out; c += 256) st_f(out + c, 0.f);
+}
+
+template <typename TG, typename TO>
+__global__ void __launch_bounds__(256)
+gated_norm_any_kernel(const GatedNormArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[8];
+  const size_t r = blockIdx.x;
+  const float* o = a.o + r * a.ld_o;
+  const TG* g = (const TG*)a.gate + r * a.ld_gate;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < a.n; c += 256) { const float v = o[c]; ss += v * v; }
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.n + a.eps);
+  TO* out = (TO*)a.out + r * a.ld_out;
+  for (int c = threadIdx.x; c < a.n; c += 256) {
+    float gv = ld_f(g + c);
+    for (int p = 1; p < a.n_part; ++p) gv += ld_f(g + (size_t)p * a.part_stride + c);
+    st_f(out + c, o[c] * inv * a.weight[c] / (1.0f + expf(-gv)));
+  }
+  for (int c = a.n + threadIdx.x; c < a.ld_out; c += 256) st_f(out + c, 0.f);
+}
+
+// ------------------------------------------------------------------------------------------ act(gate) * up, f32
+__global__ void act_mul_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, long n, int inter, int ld, int act) {
+  pdl_wait();
+  pdl_trigger();
+  const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const long r = i / inter;
+  const int c = (int)(i - r * inter);
+  const float g = gu[r * ld + c], u = gu[r * ld + inter + c];
+  const float y = act == 1 ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g / (1.0f + expf(-g));
+  out[r * inter + c] = y * u;
+}
+
+}  // namespace gb
+
+using namespace gb;
+
+GB_API int gb_embed_f32(const int* ids, const void* table, int table_f32, float* out, int n_tok, int width, int vocab, cudaStream_t stream) {
+  if (n_tok <= 0) return 0;
+  if (table_f32) launch_k(embed_f32_kernel<float>, (unsigned)n_tok, 256, 0, stream, ids, (const float*)table, out, width, vocab);
+  else launch_k(embed_f32_kernel<__nv_bfloat16>, (unsigned)n_tok, 256, 0, stream, ids, (const __nv_bfloat16*)table, out, width, vocab);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+template <typename TD, typename TO>
+static int stream_norm_launch(const StreamNormArgs& a, int n_rows, cudaStream_t stream) {
+  const size_t ed = sizeof(TD) * 4, eo = sizeof(TO) * 4;
+  const bool vec = a.width % 4 == 0 && a.width <= 16384 && (a.delta == nullptr || (a.ld_delta % 4 == 0 && a.part_stride % 4 == 0 && (uintptr_t)a.delta % ed == 0)) &&
+                   (a.out == nullptr || (a.ld_out % 4 == 0 && (uintptr_t)a.out % eo == 0)) && (uintptr_t)a.x % 16 == 0 && (uintptr_t)a.weight % 16 == 0 &&
+                   (uintptr_t)a.add % 16 == 0;
+  if (!vec) launch_k(stream_norm_any_kernel<TD, TO>, (unsigned)n_rows, 256, 0, stream, a);
+  else if (a.width <= 1024) launch_k(stream_norm_vec_kernel<TD, TO, 1>, (unsigned)n_rows, 256, 0, stream, a);
+  else if (a.width <= 4096) launch_k(stream_norm_vec_kernel<TD, TO, 4>, (unsigned)n_rows, 256, 0, stream, a);
+  else launch_k(stream_norm_vec_kernel<TD, TO, 16>, (unsigned)n_rows, 256, 0, stream, a);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// See StreamNormArgs.  delta_f32 / out_f32 give the element types; `rows` (int64, device) selects stream rows.
+GB_API int gb_stream_norm(float* x, const void* delta, int delta_f32, int n_part, long part_stride, int ld_delta, const float* add, const float* weight,
+                          const long long* rows, void* out, int out_f32, int ld_out, int n_rows, int width, float eps, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (width <= 0 || (out != nullptr && (ld_out < width || weight == nullptr)) || (delta != nullptr && (ld_delta < width || n_part < 1)))
+    return fail("stream_norm: bad widths%s");
+  StreamNormArgs a;
+  a.x = x; a.delta = delta; a.n_part = n_part; a.part_stride = part_stride; a.ld_delta = ld_delta; a.add = add; a.weight = weight; a.rows = rows;
+  a.out = out; a.ld_out = ld_out; a.width = width; a.eps = eps;
+  if (delta_f32) return out_f32 ? stream_norm_launch<float, float>(a, n_rows, stream) : stream_norm_launch<float, __nv_bfloat16>(a, n_rows, stream);
+  return out_f32 ? stream_norm_launch<__nv_bfloat16, float>(a, n_rows, stream) : stream_norm_launch<__nv_bfloat16, __nv_bfloat16>(a, n_rows, stream);
+}
+
+// See QkUnitArgs.  in_f32: element type of qkv; cache_f32: element type of q_out and the caches.
+GB_API int gb_qk_unit_store(const void* qkv, int in_f32, int n_part, long part_stride, int ld, const int* slots, void* q_out, void* k_cache, void* v_cache,
+                            int cache_f32, long num_slots, int tokens, int hq, int hkv, int dk, int dv, int dkp, int dvp, float eps, float q_scale,
+                            int unit, cudaStream_t stream) {
+  if (tokens <= 0) return 0;
+  if (hq < 1 || hkv < 1 || hq % hkv || dk < 1 || dv < 1 || dkp < dk || dvp < dv || n_part < 1) return fail("qk_unit_store: bad sizes%s");
+  if ((dk <= 128 && dkp > 128) || (dv <= 128 && dvp > 128)) return fail("qk_unit_store: padding beyond 128%s");
+  QkUnitArgs a;
+  a.qkv = qkv; a.n_part = n_part; a.part_stride = part_stride; a.ld = ld; a.slots = slots; a.q_out = q_out; a.k_cache = k_cache; a.v_cache = v_cache;
+  a.num_slots = num_slots; a.hq = hq; a.hkv = hkv; a.dk = dk; a.dv = dv; a.dkp = dkp; a.dvp = dvp; a.eps = eps; a.q_scale = q_scale; a.unit = unit;
+  const long n = (long)tokens * (hq + 2 * hkv);
+  const unsigned grid = (unsigned)((n + 7) / 8);
+  if (in_f32 && cache_f32) launch_k(qk_unit_store_kernel<float, float>, grid, 256, 0, stream, a, n);
+  else if (in_f32) launch_k(qk_unit_store_kernel<float, __nv_bfloat16>, grid, 256, 0, stream, a, n);
+  else if (cache_f32) return fail("qk_unit_store: a 32-bit cache takes 32-bit rows%s");
+  else launch_k(qk_unit_store_kernel<__nv_bfloat16, __nv_bfloat16>, grid, 256, 0, stream, a, n);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+template <typename TG, typename TO>
+static int gated_norm_launch(const GatedNormArgs& a, int rows, cudaStream_t stream) {
+  const size_t eg = sizeof(TG) * 4, eo = sizeof(TO) * 4;
+  const bool vec = a.n % 4 == 0 && a.n <= 16384 && a.ld_o % 4 == 0 && a.ld_gate % 4 == 0 && a.part_stride % 4 == 0 && a.ld_out % 4 == 0 &&
+                   (uintptr_t)a.o % 16 == 0 && (uintptr_t)a.gate % eg == 0 && (uintptr_t)a.out % eo == 0 && (uintptr_t)a.weight % 16 == 0;
+  if (!vec) launch_k(gated_norm_any_kernel<TG, TO>, (unsigned)rows, 256, 0, stream, a);
+  else if (a.n <= 1024) launch_k(gated_norm_vec_kernel<TG, TO, 1>, (unsigned)rows, 256, 0, stream, a);
+  else if (a.n <= 4096) launch_k(gated_norm_vec_kernel<TG, TO, 4>, (unsigned)rows, 256, 0, stream, a);
+  else launch_k(gated_norm_vec_kernel<TG, TO, 16>, (unsigned)rows, 256, 0, stream, a);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+GB_API int gb_gated_norm(const float* o, int ld_o, const void* gate, int gate_f32, int n_part, long part_stride, int ld_gate, const float* weight,
+                         void* out, int out_f32, int ld_out, int rows, int n, float eps, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (n < 1 || ld_o < n || ld_out < n || n_part < 1) return fail("gated_norm: bad sizes%s");
+  GatedNormArgs a;
+  a.o = o; a.ld_o = ld_o; a.gate = gate; a.n_part = n_part; a.part_stride = part_stride; a.ld_gate = ld_gate; a.weight = weight; a.out = out;
+  a.ld_out = ld_out; a.n = n; a.eps = eps;
+  if (gate_f32) return out_f32 ? gated_norm_launch<float, float>(a, rows, stream) : gated_norm_launch<float, __nv_bfloat16>(a, rows, stream);
+  return out_f32 ? gated_norm_launch<__nv_bfloat16, float>(a, rows, stream) : gated_norm_launch<__nv_bfloat16, __nv_bfloat16>(a, rows, stream);
+}
+
+// act(gate) * up over f32 rows [gate | up]; act 0 = SiLU, 1 = the tanh form of GELU.
+GB_API int gb_act_mul_f32(const float* gate_up, float* out, long rows, int inter, int ld, int act, cudaStream_t stream) {
+  const long n = rows * inter;
+  if (n <= 0) return 0;
+  launch_k(act_mul_f32_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, gate_up, out, n, inter, ld, act);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}

@@ -12,7 +12,59 @@ from __future__ import annotations
 from dataclasses import asdict, dataclass, field, replace
 from typing import Dict, List, Optional
 
+# Architectures described layer by layer (``ModelConfig.layer_specs``): name in config.json -> arch
+LAYERED_ARCHS = {"Zogavik": "zogavik"}
+
 ARCHS = ("qwen2", "qwen2vl", "qwen3", "qwen3vl", "qwen3moe", "qwen3vlmoe", "qwen35", "qwen35moe")
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a model described layer by layer: its mixer with the mixer's own sizes, and its feed-forward."""
+    mixer: str                              # "attention" | "lightning"
+    n_heads: int
+    head_dim: int                           # query / key size per head
+    v_dim: int                              # value size per head
+    n_kv_heads: int = 0                     # attention only
+    # attention
+    scale: float = 0.0                      # factor of q . k (0 = 1 / sqrt(head_dim))
+    qkv_bias: bool = False
+    qk_unit: bool = False                   # q and k divided by their root mean square per head (no weight)
+    window: int = 0                         # position i sees j with i - j < window ... (0 = all)
+    keep_first: int = 0                     # ... or j < keep_first
+    rel_buckets: int = 0                    # rows of the learned distance-bias table (0 = none)
+    rel_max: float = 0                      # distance from which the last bucket holds
+    # lightning attention
+    decay: Optional[List[float]] = None     # per head
+    # feed-forward: act(gate) * up -> down; 0 = none
+    ffn: int = 0
+    act: str = "silu"                       # or "gelu_tanh"
+
+    @property
+    def q_dim(self) -> int:
+        return self.n_heads * self.head_dim
+
+    @property
+    def span(self) -> int:
+        """Most keys a position sees (0 = no limit)."""
+        return self.window + self.keep_first if self.window > 0 else 0
+
+
+@dataclass
+class LoopSpec:
+    """Layers ``start .. stop - 1`` run ``times`` times in a row with the same weights; every pass has its own cache or state, and
+    a learned vector is added to the stream in front of each pass."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class LayerRun:
+    """One execution of a layer: ``layer`` is its index in the weights, ``step`` the row of the step-vector table added in front of it
+    (-1 = none).  The position of the run in ``ModelConfig.layer_runs`` is the index of its cache."""
+    layer: int
+    step: int = -1
 
 
 @dataclass
@@ -51,6 +103,39 @@ class ModelConfig:
     # M-RoPE (Qwen2-VL / Qwen3-VL): sections of rotary pairs assigned to t / h / w
     mrope_sections: Optional[List[int]] = None
     n_deepstack_layers: int = 0
+    # models described layer by layer (the residual stream is then kept in 32-bit floats)
+    layer_specs: Optional[List[LayerSpec]] = None
+    loop: Optional[LoopSpec] = None
+    norm_offset: float = 0.0                # stored norm weights are added to this (1 = stored around zero)
+    logit_scale: float = 1.0
+
+    def __post_init__(self):
+        if self.layer_specs is not None:
+            self.layer_specs = [x if isinstance(x, LayerSpec) else LayerSpec(**x) for x in self.layer_specs]
+            self.n_layers = len(self.layer_specs)
+        if self.loop is not None and not isinstance(self.loop, LoopSpec):
+            self.loop = LoopSpec(**self.loop)
+
+    @property
+    def is_layered(self) -> bool:
+        return self.layer_specs is not None
+
+    def layer_runs(self) -> List[LayerRun]:
+        """The layers in the order of execution (looped layers appear once per pass)."""
+        n, lp = self.n_layers, self.loop
+        if lp is None:
+            return [LayerRun(i) for i in range(n)]
+        if not 0 <= lp.start < lp.stop <= n or lp.times < 1:
+            raise ValueError(f"bad layer loop {lp} for {n} layers")
+        runs = [LayerRun(i) for i in range(lp.start)]
+        for t in range(lp.times):
+            runs += [LayerRun(i, t if i == lp.start else -1) for i in range(lp.start, lp.stop)]
+        return runs + [LayerRun(i) for i in range(lp.stop, n)]
+
+    @property
+    def has_recurrent_state(self) -> bool:
+        """Whether a sequence carries state that cannot drop positions (Delta-Net or lightning layers)."""
+        return self.is_hybrid or (self.is_layered and any(x.mixer == "lightning" for x in self.layer_specs))
 
     @property
     def is_moe(self) -> bool:
@@ -82,6 +167,15 @@ class ModelConfig:
         return (layer + 1) % self.full_attention_interval != 0
 
     def param_count(self) -> int:
+        if self.is_layered:
+            tot = self.vocab * self.hidden
+            for x in self.layer_specs:
+                if x.mixer == "lightning":
+                    tot += self.hidden * (2 * x.q_dim + 3 * x.n_heads * x.v_dim)
+                else:
+                    tot += self.hidden * (x.q_dim + x.n_kv_heads * (x.head_dim + x.v_dim) + x.n_heads * x.v_dim)
+                tot += 3 * self.hidden * x.ffn
+            return tot
         per_layer = self.hidden * (self.q_dim + 2 * self.kv_dim) + self.q_dim * self.hidden
         if self.is_moe:
             per_layer += self.n_experts * 3 * self.hidden * self.expert_ffn + self.n_experts * self.hidden
@@ -124,6 +218,29 @@ PRESETS: Dict[str, ModelConfig] = {
     "tiny-qwen2": ModelConfig(arch="qwen2", n_layers=2, hidden=256, n_heads=4, n_kv_heads=2, head_dim=128, ffn=512, vocab=512,
                               qk_norm=False, qkv_bias=True, tie_embeddings=True),
 }
+
+
+def _zogavik(pattern: str, hidden: int, heads: int, kv_heads: int, dim: int, ffn: int, vocab: int, window: int, keep: int, rel_max: int, loop=None,
+             v_dim: int = 0, lin_heads: int = 0, lin_dim: int = 0, lin_v: int = 0, rel_buckets: int = 32) -> ModelConfig:
+    """``pattern``: one letter per layer, L = lightning, A = attention."""
+    lh = lin_heads or heads
+    specs = []
+    for c in pattern:
+        if c == "L":
+            specs.append(LayerSpec("lightning", lh, lin_dim or dim, lin_v or dim, decay=[1.0 - 2.0 ** -(1.0 + 7.0 * i / lh) for i in range(lh)],
+                                   ffn=ffn, act="gelu_tanh"))
+        else:
+            specs.append(LayerSpec("attention", heads, dim, v_dim or dim, n_kv_heads=kv_heads, scale=dim ** -0.5, qkv_bias=True, qk_unit=True,
+                                   window=window, keep_first=keep, rel_buckets=rel_buckets, rel_max=rel_max, ffn=ffn, act="gelu_tanh"))
+    return ModelConfig(arch="zogavik", layer_specs=specs, hidden=hidden, n_heads=heads, n_kv_heads=kv_heads, head_dim=dim, ffn=ffn, vocab=vocab,
+                       tie_embeddings=True, loop=loop, norm_offset=1.0, logit_scale=1.0, qk_norm=False, qkv_bias=True)
+
+
+PRESETS["tiny-zogavik"] = _zogavik("ALLA", 192, 4, 2, 40, 320, 500, 48, 8, 100, LoopSpec(0, 2, 3), v_dim=56, lin_heads=3, lin_dim=24, lin_v=40)
+# layers of the sizes of an 8-billion-parameter dense model, three lightning layers to one of windowed attention
+PRESETS["zogavik-8b"] = _zogavik("LLLA" * 9, 4096, 32, 8, 128, 12288, 151936, 4096, 128, 4096)
+# the same layers with the middle ones looped: a smaller model of the same depth
+PRESETS["zogavik-4b-loop2"] = _zogavik("LLLA" * 5, 4096, 32, 8, 128, 12288, 151936, 4096, 128, 4096, LoopSpec(2, 18, 2))
 
 
 def get_config(name: str) -> ModelConfig:

@@ -18,7 +18,7 @@ import torch
 
 from .. import _native
 from ..utils import gguf as G
-from .config import ARCHS, ModelConfig
+from .config import ARCHS, LAYERED_ARCHS, LayerSpec, LoopSpec, ModelConfig
 from .weights import ModelWeights, RandomSource, build_weights
 
 
@@ -519,9 +519,79 @@ def _qwen35_config_from_hf(c: dict) -> ModelConfig:
         norm_topk=True)
 
 
+class LayeredSource(SafetensorsSource):
+    """Checkpoints of models described layer by layer: tensors ``l<i>.norm1``, ``l<i>.mix.*``, ``l<i>.norm2``, ``l<i>.mlp.*``, ``embed``,
+    ``final.norm``, ``loop.step``, served under the names the model builder asks for."""
+
+    _LAYER = {"attn_norm.weight": "norm1", "ffn_norm.weight": "norm2", "attn_q.weight": "mix.q", "attn_k.weight": "mix.k", "attn_v.weight": "mix.v",
+              "attn_q.bias": "mix.q.b", "attn_k.bias": "mix.k.b", "attn_v.bias": "mix.v.b", "attn_output.weight": "mix.o", "attn_rel.weight": "mix.rel",
+              "lin_q.weight": "mix.q", "lin_k.weight": "mix.k", "lin_v.weight": "mix.v", "lin_gate.weight": "mix.g", "lin_norm.weight": "mix.norm",
+              "lin_out.weight": "mix.o", "ffn_gate.weight": "mlp.gate", "ffn_up.weight": "mlp.up", "ffn_down.weight": "mlp.down"}
+    _TOP = {"token_embd.weight": "embed", "output_norm.weight": "final.norm", "loop_step.weight": "loop.step", "output.weight": "head"}
+
+    @classmethod
+    def file_name(cls, name: str) -> str:
+        if name in cls._TOP:
+            return cls._TOP[name]
+        _, li, rest = name.split(".", 2)
+        return f"l{li}.{cls._LAYER[rest]}"
+
+    def has(self, name: str) -> bool:
+        return self.file_name(name) in self.where
+
+    def shape(self, name: str):
+        key = self.file_name(name)
+        return self.where[key].info[key][2]
+
+    def get(self, name: str, shape) -> torch.Tensor:
+        key = self.file_name(name)
+        if key not in self.where:
+            raise ValueError(f"the checkpoint has no tensor {key!r}")
+        t = self._raw(key)
+        if tuple(t.shape) != tuple(shape):
+            raise ValueError(f"{key}: checkpoint has shape {tuple(t.shape)}, model wants {tuple(shape)}")
+        return t
+
+
+def _layered_config(c: dict, path: str) -> ModelConfig:
+    """config.json of a model described layer by layer: ``layers`` (each with its mixer's type and sizes and its feed-forward), ``loop``,
+    ``norm``, ``vocab``, ``width``, ``logit_scale``."""
+    src = LayeredSource(path)
+    specs = []
+    for li, e in enumerate(c["layers"]):
+        m, mlp = e["mixer"], e.get("mlp")
+        ff = 0
+        if mlp is not None:
+            if mlp.get("kind", "dense") != "dense":
+                raise ValueError(f"layer {li}: feed-forward kind {mlp['kind']!r} is not supported")
+            ff = int(mlp["ff"])
+        if e["type"] == "lightning":
+            decay = m["decay"] if isinstance(m["decay"], list) else [m["decay"]] * int(m["heads"])
+            if len(decay) != int(m["heads"]):
+                raise ValueError(f"layer {li}: {len(decay)} decays for {m['heads']} heads")
+            specs.append(LayerSpec("lightning", int(m["heads"]), int(m["dim"]), int(m["vdim"]), decay=[float(x) for x in decay], ffn=ff, act="gelu_tanh"))
+        elif e["type"] == "attention":
+            mask = m.get("mask") or {}
+            specs.append(LayerSpec("attention", int(m["heads"]), int(m["dim"]), int(m["vdim"]), n_kv_heads=int(m["kv_heads"]), scale=float(m["scale"]),
+                                   qkv_bias=True, qk_unit=True, window=int(mask.get("size") or 0), keep_first=int(mask.get("keep_first") or 0),
+                                   rel_buckets=int(src.shape(f"blk.{li}.attn_rel.weight")[0]), rel_max=float(m["bias_max"]), ffn=ff, act="gelu_tanh"))
+        else:
+            raise ValueError(f"layer {li}: mixer {e['type']!r} is not supported")
+    lp = c.get("loop")
+    att = next((s for s in specs if s.mixer == "attention"), specs[0])
+    return ModelConfig(arch=LAYERED_ARCHS[c["architecture"]], layer_specs=specs, hidden=int(c["width"]), vocab=int(c["vocab"]), n_heads=att.n_heads,
+                       n_kv_heads=max(1, att.n_kv_heads), head_dim=att.head_dim, ffn=max(s.ffn for s in specs), rms_eps=float(c["norm"]["eps"]),
+                       tie_embeddings=True, qk_norm=False, qkv_bias=True, norm_offset=1.0, logit_scale=float(c.get("logit_scale", 1.0)),
+                       loop=LoopSpec(int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else None)
+
+
 def config_from_hf(path: str) -> ModelConfig:
     with open(os.path.join(path, "config.json")) as fh:
         c = json.load(fh)
+    if c.get("architecture") in LAYERED_ARCHS:
+        return _layered_config(c, path)
+    if "architecture" in c and "layers" in c:
+        raise ValueError(f"unsupported architecture {c['architecture']!r} (described layer by layer: {sorted(LAYERED_ARCHS)})")
     mt = c.get("model_type", "qwen3")
     if mt.startswith("qwen3_5"):
         return _qwen35_config_from_hf(c)
@@ -554,7 +624,7 @@ def config_from_hf(path: str) -> ModelConfig:
 def load_safetensors(path: str, fmt: str = "bf16", device="cuda", cfg: Optional[ModelConfig] = None, **shard) -> ModelWeights:
     """Load an HF checkpoint directory (config.json + *.safetensors)."""
     cfg = cfg or config_from_hf(path)
-    src = HFQwen35Source(path, cfg) if cfg.is_hybrid else SafetensorsSource(path)
+    src = LayeredSource(path) if cfg.is_layered else HFQwen35Source(path, cfg) if cfg.is_hybrid else SafetensorsSource(path)
     return build_weights(cfg, src, fmt, device, **shard)
 
 
@@ -563,6 +633,8 @@ def save_hf_checkpoint(cfg: ModelConfig, src, path: str, mxfp8: bool = False) ->
     as F8_E4M3 + ``_scale_inv`` E8M0 the way MXFP8 checkpoints do."""
     from ..ops import mxfp8 as MX
     os.makedirs(path, exist_ok=True)
+    if cfg.is_layered:
+        return _save_layered(cfg, src, path)
     out: Dict[str, torch.Tensor] = {}
     h, d = cfg.hidden, cfg.head_dim
 
@@ -609,3 +681,42 @@ def save_hf_checkpoint(cfg: ModelConfig, src, path: str, mxfp8: bool = False) ->
                    "rope_theta": cfg.rope_theta, "tie_word_embeddings": cfg.tie_embeddings, "max_position_embeddings": cfg.max_seq_len,
                    "num_experts": cfg.n_experts, "num_experts_per_tok": cfg.n_experts_used, "moe_intermediate_size": cfg.expert_ffn,
                    "norm_topk_prob": cfg.norm_topk}, fh)
+
+
+def _save_layered(cfg: ModelConfig, src, path: str) -> None:
+    """Write a model described layer by layer as config.json + model.safetensors (bf16), the layout ``LayeredSource`` reads."""
+    out: Dict[str, torch.Tensor] = {}
+    h = cfg.hidden
+
+    def put(name, shape):
+        out[LayeredSource.file_name(name)] = src.get(name, shape).to(torch.bfloat16)
+
+    put("token_embd.weight", (cfg.vocab, h))
+    put("output_norm.weight", (h,))
+    if cfg.loop is not None:
+        put("loop_step.weight", (cfg.loop.times, h))
+    layers = []
+    for li, sp in enumerate(cfg.layer_specs):
+        p, nv = f"blk.{li}.", sp.n_heads * sp.v_dim
+        put(p + "attn_norm.weight", (h,))
+        if sp.mixer == "lightning":
+            for nm, shp in (("lin_q", (sp.q_dim, h)), ("lin_k", (sp.q_dim, h)), ("lin_v", (nv, h)), ("lin_gate", (nv, h)), ("lin_norm", (nv,)), ("lin_out", (h, nv))):
+                put(p + nm + ".weight", shp)
+            m = {"heads": sp.n_heads, "dim": sp.head_dim, "vdim": sp.v_dim, "decay": list(sp.decay)}
+        else:
+            for c, n in (("q", sp.q_dim), ("k", sp.n_kv_heads * sp.head_dim), ("v", sp.n_kv_heads * sp.v_dim)):
+                put(p + f"attn_{c}.weight", (n, h))
+                put(p + f"attn_{c}.bias", (n,))
+            put(p + "attn_rel.weight", (sp.rel_buckets, sp.n_heads))
+            put(p + "attn_output.weight", (h, nv))
+            m = {"heads": sp.n_heads, "kv_heads": sp.n_kv_heads, "dim": sp.head_dim, "vdim": sp.v_dim, "scale": sp.scale, "bias_max": sp.rel_max,
+                 "mask": {"size": sp.window, "keep_first": sp.keep_first} if sp.window else None}
+        if sp.ffn:
+            put(p + "ffn_norm.weight", (h,))
+            put(p + "ffn_gate.weight", (sp.ffn, h)); put(p + "ffn_up.weight", (sp.ffn, h)); put(p + "ffn_down.weight", (h, sp.ffn))
+        layers.append({"type": sp.mixer, "mixer": m, "mlp": {"kind": "dense", "ff": sp.ffn} if sp.ffn else None})
+    save_safetensors(out, os.path.join(path, "model.safetensors"))
+    name = {v: k for k, v in LAYERED_ARCHS.items()}[cfg.arch]
+    with open(os.path.join(path, "config.json"), "w") as fh:
+        json.dump({"architecture": name, "layers": layers, "vocab": cfg.vocab, "width": h, "norm": {"eps": cfg.rms_eps}, "logit_scale": cfg.logit_scale,
+                   "loop": {"start": cfg.loop.start, "stop": cfg.loop.stop, "times": cfg.loop.times} if cfg.loop else None}, fh)

@@ -11,6 +11,10 @@ Layer recipe (reference: common/transformer.h:3550-4174):
   h = RMSNorm(x); dense: x += (SiLU(h Wg^T) * h Wu^T) Wd^T  [TP all-reduce]
                   MoE  : softmax router -> top-k -> renormalise; x += sum_k w_k FFN_k(h)  [EP dispatch / combine]
   logits = RMSNorm(x) Whead^T on the last token of every sequence.
+
+Models described layer by layer (``ModelConfig.layer_specs``) run through the same loop: every layer names its mixer (windowed
+attention with kept first tokens and a distance bias, or lightning attention) with sizes of its own, layers may be looped (every
+run has its own cache: ``KvCache`` is indexed by run), and the residual stream is f32.
 """
 from __future__ import annotations
 
@@ -25,9 +29,9 @@ from .. import _native
 from ..ops import attention as att
 from ..ops import elementwise as ew
 from ..ops import deltanet as dn
-from ..ops import gemm, moe, qlinear, sampling
+from ..ops import gemm, lightning, moe, qlinear, sampling, stream
 from ..ops.mxfp8 import MxTensor
-from .config import ModelConfig
+from .config import LayerRun, LayerSpec, ModelConfig
 from .weights import LinearWeight, ModelWeights
 from ..utils import profiler
 
@@ -67,6 +71,8 @@ class KvCache:
         shape = (num_pages * page_size, hkv, cfg.head_dim)
         ssm = [cfg.is_ssm_layer(first_layer + i) for i in range(nl)]
         none = (0, hkv, cfg.head_dim)
+        if cfg.is_layered:
+            return KvCache._allocate_layered(cfg, num_pages, page_size, device, n_seq_slots, kv_dtype)
         if kv_dtype == "int8":
             if any(ssm) or cfg.head_dim != 128:
                 raise ValueError("the INT8 KV cache is built for attention-only models with head_dim 128")
@@ -90,15 +96,40 @@ class KvCache:
                       if ssm[i] else None for i in range(nl)]
         return kv
 
+    @staticmethod
+    def _allocate_layered(cfg: ModelConfig, num_pages: int, page_size: int, device, n_seq_slots: int, kv_dtype: str) -> "KvCache":
+        """One entry per layer RUN: K / V pages with the layer's own head sizes (attention), or ``rec`` f32 ``[slots, heads, dim, vdim]``
+        (lightning attention)."""
+        dtypes = {"bf16": torch.bfloat16, "f32": torch.float32}
+        if kv_dtype not in dtypes:
+            raise ValueError(f"models described layer by layer keep a bf16 or f32 KV cache, not {kv_dtype!r}")
+        dt = dtypes[kv_dtype]
+        kv = KvCache([], [], page_size, num_pages)
+        kv.rec = []
+        for run in cfg.layer_runs():
+            sp = cfg.layer_specs[run.layer]
+            lin = sp.mixer == "lightning"
+            dkp, dvp = att.cache_head_dims(sp.head_dim, sp.v_dim, dt)
+            rows, heads = (0, 1) if lin else (num_pages * page_size, sp.n_kv_heads)
+            kv.k.append(torch.zeros(rows, heads, dkp, dtype=dt, device=device))
+            kv.v.append(torch.zeros(rows, heads, dvp, dtype=dt, device=device))
+            kv.rec.append(torch.zeros(n_seq_slots, sp.n_heads, sp.head_dim, sp.v_dim, dtype=torch.float32, device=device) if lin else None)
+        if not any(r is not None for r in kv.rec):
+            kv.rec = None
+        return kv
+
+    def recurrent(self, li: int) -> List[torch.Tensor]:
+        """The per-slot state tensors of entry ``li`` (empty for attention layers)."""
+        return [t[li] for t in (self.conv, self.rec) if t is not None and t[li] is not None]
+
     def reset_slots(self, slots) -> None:
         """Zero the recurrent state of the given sequence slots (a new sequence starts from an empty state)."""
-        if self.conv is None:
+        if self.rec is None:
             return
         idx = torch.as_tensor(list(slots), dtype=torch.long, device=self.k[0].device)
-        for c, r in zip(self.conv, self.rec):
-            if c is not None:
-                c[idx] = 0
-                r[idx] = 0
+        for li in range(len(self.k)):
+            for t in self.recurrent(li):
+                t[idx] = 0
 
     def copy_pages(self, pairs) -> None:
         """``page dst <- page src`` for every ``(src, dst)`` of ``pairs`` in every layer's K and V: the copy-on-write step of a
@@ -131,10 +162,8 @@ class KvCache:
         if self.quantized:
             return sum(t.numel() * t.element_size() for t in list(self.kq) + list(self.vq) + list(self.ks) + list(self.vs)) + \
                 2 * self.k[0].numel() * 2
-        tot = sum(t.numel() * 2 for t in self.k) * 2
-        if self.conv is not None:
-            tot += sum(c.numel() * 4 + r.numel() * 4 for c, r in zip(self.conv, self.rec) if c is not None)
-        return tot
+        tot = sum(t.numel() * t.element_size() for t in list(self.k) + list(self.v))
+        return tot + sum(t.numel() * 4 for li in range(len(self.k)) for t in self.recurrent(li))
 
 
 @dataclass
@@ -157,6 +186,10 @@ class ForwardBatch:
     # INT8 KV cache: where a step's new K / V rows sit in the bf16 staging buffer, and (prefill) the block table of the staged sequences
     stage_slots: Optional[torch.Tensor] = None # int32 [T]
     stage_bt: Optional[torch.Tensor] = None    # int32 [B, pages]
+    # attention work lists by head shape (models whose layers differ in it): (query heads, KV heads, span) -> (work, KV splits)
+    plans: Optional[dict] = None
+    q_lens: Optional[List[int]] = None             # host copies of the chunk and sequence lengths, from which a missing plan is made
+    kv_lens: Optional[List[int]] = None
     # context-parallel prefill: the cache slots whose K / V rows this rank contributes to the per-layer all-gather (staging order)
     cp_send_slots: Optional[torch.Tensor] = None   # int64 [p_local * page_size]
 
@@ -197,7 +230,7 @@ class ForwardBatch:
                 for s in range(b):
                     st_bt[s, : pages[s]] = torch.arange(first[s], first[s] + pages[s], dtype=torch.int32)
                 st_bt = st_bt.to(device)
-        return ForwardBatch(stage_slots=st_slots, stage_bt=st_bt,
+        return ForwardBatch(stage_slots=st_slots, stage_bt=st_bt, plans={}, q_lens=list(q_lens), kv_lens=[c + q for c, q in zip(ctx_lens, q_lens)],
                             ids=ids_t, positions=torch.tensor(pos, **i32), slots=torch.tensor(slots, **i32),
                             cu_q=torch.tensor(cu, **i32), kv_len=torch.tensor([c + q for c, q in zip(ctx_lens, q_lens)], **i32),
                             block_table=block_table.to(device=device, dtype=torch.int32),
@@ -205,6 +238,13 @@ class ForwardBatch:
                             logit_rows=torch.tensor(rows, dtype=torch.int64, device=device), num_splits=num_splits, n_tokens=t,
                             seq_slots=torch.tensor(list(seq_slots) if seq_slots is not None else list(range(b)), **i32),
                             is_decode=(b > 0 and all(q == 1 for q in q_lens)))
+
+
+def attention_plan(q_lens: Sequence[int], max_kv: int, hq: int, hkv: int, span: int, device, decode: bool):
+    """(work list on the device, KV splits) of the tcgen05 attention kernels for one head shape; ``span`` is the most keys a position
+    sees (0 = no limit)."""
+    splits = att.pick_splits(len(q_lens), hkv, min(max_kv, span + 128) if span else max_kv) if decode and torch.device(device).type == "cuda" else 1
+    return att.build_work(q_lens, hq, hkv, splits).to(device), splits
 
 
 # K-split partial sums for decode-sized row projections (GB_SPLIT_PROJ=0 switches them off)
@@ -281,6 +321,24 @@ def apply_linear_split(lw: LinearWeight, x: torch.Tensor, x_mx: Optional[MxTenso
     return apply_linear(lw, x, x_mx)
 
 
+def apply_linear_stream(lw: LinearWeight, x: torch.Tensor):
+    """A projection whose result joins an f32 stream or an f32 computation: f32, or K-split partial sums for the consumer to add."""
+    if lw.fmt == "f32":
+        return gemm.linear_f32(x, lw.w, bias=lw.bias)
+    sp = gemm.pick_partials(lw.n, x.shape[0], (lw.k + 63) // 64 * 64, False) if SPLIT_PROJ and x.is_cuda else 1
+    if sp > 1:
+        return gemm.linear_partials(x, lw.w, sp, bias=lw.bias, w_tiled=lw.tiled)
+    return gemm.linear(x, lw.w, bias=lw.bias, out_dtype=torch.float32, w_tiled=lw.tiled)
+
+
+def apply_linear_mixer(lw: LinearWeight, x: torch.Tensor):
+    """The input projection of a mixer: as ``apply_linear_stream`` for decode-sized batches (the mixer's kernels add the partial sums), bf16
+    rows for prefill-sized ones."""
+    if lw.fmt == "f32" or x.shape[0] <= 64:
+        return apply_linear_stream(lw, x)
+    return gemm.linear(x, lw.w, bias=lw.bias, w_tiled=lw.tiled)
+
+
 def expert_gate_up_mx(x_q: torch.Tensor, x_sf: torch.Tensor, w13: LinearWeight, n_w_groups: int, seg_start: torch.Tensor,
                       seg_count: torch.Tensor, tn: int, hq: torch.Tensor, hsf: torch.Tensor, row_valid: Optional[torch.Tensor] = None,
                       extras=None, w_groups: Optional[int] = None, scratch: Optional[torch.Tensor] = None) -> None:
@@ -313,12 +371,16 @@ class Transformer:
         self.hkv_local = max(1, cfg.n_kv_heads // weights.tp_size)
         self.q_scale = ew.softmax_scale_log2(cfg.head_dim)
         self.mx = weights.fmt == "mxfp8"
+        self.runs = cfg.layer_runs() if cfg.is_layered else [LayerRun(i) for i in range(len(weights.layers))]
+        # models described layer by layer: f32 stream, activations in the weights' own width
+        self.stream_f32 = cfg.is_layered
+        self.act_dtype = torch.float32 if weights.fmt == "f32" else torch.bfloat16
         rd = cfg.rope_dim or cfg.head_dim
         if cfg.mrope_sections and sum(cfg.mrope_sections) > 0:
             rd = 2 * sum(cfg.mrope_sections)           # the rotary width under M-RoPE (common/transformer.h:1229-1232)
         self.rope_dim = rd
         self.rope_table = ew.rope_table(min(max(cfg.max_seq_len, 4096), 65536), rd, cfg.rope_theta, weights.embed.device) \
-            if weights.embed.is_cuda else None
+            if weights.embed.is_cuda and not cfg.is_layered else None
         self.snapshots = {}            # layer -> hidden rows captured after that layer (debug / DeepStack)
         self.snapshot_layers: Sequence[int] = ()
 
@@ -415,6 +477,49 @@ class Transformer:
                           cfg.ssm_n_heads_v, cfg.ssm_head_dim, cfg.rms_eps)
         return self.par.row_linear(ssm.w_out, out)
 
+    def attention_plans(self, q_lens: Sequence[int], max_kv: int, device, decode: bool) -> dict:
+        """Work lists for every head shape of the model (made up front where nothing may be allocated later: a captured decode step)."""
+        plans = {}
+        for sp in (self.cfg.layer_specs or ()):
+            if sp.mixer == "attention" and (sp.n_heads, sp.n_kv_heads, sp.span) not in plans:
+                plans[(sp.n_heads, sp.n_kv_heads, sp.span)] = attention_plan(q_lens, max_kv, sp.n_heads, sp.n_kv_heads, sp.span, device, decode)
+        return plans
+
+    def masked_attention_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
+        """Attention of a layer described by ``LayerSpec``: biased projection -> Q / K unit norm + cache store -> windowed attention with
+        kept first tokens and distance bias -> output projection.  ``li`` is the run, which has its own cache."""
+        kc, vc = self.kv.k[li], self.kv.v[li]
+        qkv = apply_linear_mixer(lw.wqkv, h)
+        q = stream.qk_unit(qkv, fb.slots, kc, vc, sp.n_heads, sp.n_kv_heads, sp.head_dim, sp.v_dim, self.cfg.rms_eps,
+                           (sp.scale or sp.head_dim ** -0.5) * att.LOG2E, unit=sp.qk_unit)
+        key = (sp.n_heads, sp.n_kv_heads, sp.span)
+        if fb.plans is None:
+            fb.plans = {}
+        if key not in fb.plans and q.is_cuda:
+            fb.plans[key] = attention_plan(fb.q_lens, max(fb.kv_lens), *key, q.device, fb.is_decode)
+        a = att.attention_masked(q, kc, vc, fb.cu_q, fb.kv_len, fb.block_table, self.kv.page_size, window=sp.window, keep_first=sp.keep_first,
+                                 bias=lw.rel_bias, plan=fb.plans.get(key), decode=fb.is_decode)
+        return apply_linear_stream(lw.wo, a.reshape(a.shape[0], -1))
+
+    def lightning_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
+        """Lightning attention: projection -> SiLU + decayed recurrence -> RMSNorm over all heads * sigmoid(gate) -> output projection."""
+        proj = apply_linear_mixer(lw.lin.w_in, h)
+        o = lightning.lightning(proj, lw.lin.decay, self.kv.rec[li], fb.cu_q, fb.seq_slots, sp.n_heads, sp.head_dim, sp.v_dim)
+        y = stream.gated_norm(o, proj, 2 * sp.q_dim + sp.n_heads * sp.v_dim, lw.lin.norm, self.cfg.rms_eps, self.act_dtype)
+        return apply_linear_stream(lw.lin.w_out, y)
+
+    def stream_ffn(self, lw, sp: LayerSpec, h: torch.Tensor):
+        gu = lw.w_gate_up
+        if gu.fmt == "f32":
+            return apply_linear_stream(lw.w_down, stream.act_mul(gemm.linear_f32(h, gu.w), sp.act))
+        inter = gu.n // 2
+        split = gemm.pick_partials_dual(inter, h.shape[0], (gu.k + 63) // 64 * 64, False) if SPLIT_PROJ and h.is_cuda else 1
+        if split > 1:
+            act = ew.silu_mul_partials(gemm.swiglu_partials(h, gu.w, split, w_tiled=gu.tiled), act=sp.act)
+        else:
+            act = gemm.linear_swiglu(h, gu.w, w_tiled=gu.tiled, act=sp.act)
+        return apply_linear_stream(lw.w_down, act)
+
     def shared_expert(self, lw, h: torch.Tensor) -> torch.Tensor:
         """Always-on expert of the qwen35moe layers, scaled by sigmoid(h . g) (cuda/llm/cuda_llm_runner.c:11879-11897)."""
         if lw.sh_gate_up.fmt == "bf16":
@@ -492,8 +597,10 @@ class Transformer:
                        x: Optional[torch.Tensor] = None) -> torch.Tensor:
         """Residual stream after layers ``[first_layer, last_layer)`` (pipeline stages pass ``x`` in)."""
         cfg, w = self.cfg, self.w
-        last_layer = len(w.layers) if last_layer is None else last_layer
-        if x is None:
+        last_layer = len(self.runs) if last_layer is None else last_layer
+        if x is None and self.stream_f32:
+            x = stream.embed(fb.ids, w.embed) if fb.embeds is None else fb.embeds.float()
+        elif x is None:
             x = fb.embeds if fb.embeds is not None else ew.embed(fb.ids, w.embed)
         delta = None
         if hasattr(self.par, "_sp_ok"):
@@ -501,8 +608,20 @@ class Transformer:
             # plain dense stacks (nothing reads the whole stream or the normalised rows outside a GEMM in between)
             self.par._sp_ok = not (cfg.is_moe or cfg.attn_output_gate or fb.deepstack is not None or self.snapshot_layers or
                                    any(l.ssm is not None for l in w.layers[first_layer:last_layer]))
-        for li in range(first_layer, last_layer):
-            lw = w.layers[li]
+        for li in range(first_layer, last_layer):           # li: the layer RUN, index of its cache (looped layers run several times)
+            lw = w.layers[self.runs[li].layer]
+            if self.stream_f32:
+                sp, step = cfg.layer_specs[self.runs[li].layer], self.runs[li].step
+                h = stream.norm(x, lw.attn_norm, cfg.rms_eps, delta, add=w.loop_step[step] if step >= 0 else None, out_dtype=self.act_dtype)
+                with profiler.region(sp.mixer, "block", "attention", li):
+                    delta = self.lightning_block(li, lw, sp, h, fb) if sp.mixer == "lightning" else self.masked_attention_block(li, lw, sp, h, fb)
+                if sp.ffn:
+                    h = stream.norm(x, lw.ffn_norm, cfg.rms_eps, delta, out_dtype=self.act_dtype)
+                    with profiler.region("ffn", "block", "ffn", li):
+                        delta = self.stream_ffn(lw, sp, h)
+                if li in self.snapshot_layers:
+                    self.snapshots[li] = x + stream.whole(delta)
+                continue
             lay = 32 if x.shape[0] <= 32 else 128
             par = self.par
             is_ssm = lw.ssm is not None
@@ -538,6 +657,9 @@ class Transformer:
         # the last delta stays pending: the head (or the next pipeline stage) folds it into the stream
         if hasattr(self.par, "finish_residual"):
             self.par.finish_residual(x, delta)
+        if self.stream_f32:
+            self._last_delta = delta
+            return x
         self._last_delta = self.par.materialize(delta) if delta is not None else None
         return x
 
@@ -550,6 +672,8 @@ class Transformer:
         cfg, w = self.cfg, self.w
         delta = self._last_delta
         rows = fb.logit_rows
+        if self.stream_f32:
+            return stream.norm(x, w.final_norm, cfg.rms_eps, delta, rows=rows.long(), out_dtype=self.act_dtype)
         xr = x[rows]
         if delta is not None:
             xr = (xr.float() + delta[rows].float()).to(torch.bfloat16)
@@ -558,13 +682,15 @@ class Transformer:
     def head(self, x: torch.Tensor, fb: ForwardBatch) -> torch.Tensor:
         if self.w.lm_head.is_quant:
             return qlinear.linear(self._head_input(x, fb), self.w.lm_head.q, out_dtype=torch.float32)
+        if self.w.lm_head.fmt == "f32":
+            return gemm.linear_f32(self._head_input(x, fb), self.w.lm_head.w)
         return gemm.linear(self._head_input(x, fb), self.w.lm_head.w, out_dtype=torch.float32, w_tiled=self.w.lm_head.tiled)
 
     def forward_greedy(self, fb: ForwardBatch, want_value: bool = False):
         """Greedy next tokens ``int32 [len(logit_rows)]``: the arg-max runs in the LM-head GEMM's epilogue, no logits are stored."""
         x = self.forward_hidden(fb)
-        if self.w.lm_head.is_quant:
-            logits = qlinear.linear(self._head_input(x, fb), self.w.lm_head.q, out_dtype=torch.float32)
+        if self.w.lm_head.is_quant or self.w.lm_head.fmt == "f32":
+            logits = self.head(x, fb)
             return sampling.argmax(logits, idx_offset=self.w.vocab_start, want_value=want_value)
         return gemm.linear_argmax(self._head_input(x, fb), self.w.lm_head.w, idx_offset=self.w.vocab_start, want_value=want_value,
                                   w_tiled=self.w.lm_head.tiled)
@@ -573,6 +699,8 @@ class Transformer:
         """Residual stream with the pending delta folded in (what a pipeline stage hands to the next)."""
         if self._last_delta is None:
             return x
+        if self.stream_f32:
+            return x + stream.whole(self._last_delta)
         return (x.float() + self._last_delta.float()).to(torch.bfloat16)
 
 

@@ -4,6 +4,7 @@ A ``LinearWeight`` keeps one projection in the format the kernels consume:
 
 * ``bf16``   row-major ``[N, K]``
 * ``mxfp8``  e4m3 bytes + E8M0 scale atoms (``ops.mxfp8.MxTensor``)
+* ``f32``    row-major ``[N, K]`` in 32-bit floats (models described layer by layer: the exact path the 16-bit one is checked against)
 
 Grouped (expert) weights use the same class with ``groups > 0`` and rows stacked expert after expert.
 Tensor-parallel and expert-parallel shards are cut when the weights are made or loaded, never at run
@@ -22,13 +23,15 @@ import torch
 
 from ..ops import elementwise as ew
 from ..ops import mxfp8
+from ..ops.attention import cache_head_dims, distance_bias_table
+from ..ops.stream import row_width
 from ..ops.mxfp8 import MxTensor
 from .config import ModelConfig
 
 
 @dataclass
 class LinearWeight:
-    fmt: str                                  # "bf16" | "mxfp8" | "q4_k" | "q8_0" (ggml blocks kept quantised in HBM)
+    fmt: str                                  # "bf16" | "mxfp8" | "f32" | "q4_k" | "q8_0" (ggml blocks kept quantised in HBM)
     n: int                                    # output features (per group)
     k: int
     w: Optional[torch.Tensor] = None          # bf16 [rows, K]
@@ -47,11 +50,11 @@ class LinearWeight:
     def is_tiled(self) -> bool:
         if self.is_quant:
             return True
-        return self.tiled if self.fmt == "bf16" else self.mx.tiled
+        return self.tiled if self.fmt in ("bf16", "f32") else self.mx.tiled
 
     def tile_(self) -> "LinearWeight":
         """Re-lay the matrix in place into the GEMM kernel's tiled weight layout (``ops.mxfp8.tile_weight``)."""
-        if self.is_quant:
+        if self.is_quant or self.fmt == "f32":
             return self                       # ggml blocks are stored in their own tile order from the start
         t = self.w if self.fmt == "bf16" else self.mx.data
         if self.is_tiled or not mxfp8.can_tile(t) or (self.groups and self.rows_per_group % 128):
@@ -65,6 +68,8 @@ class LinearWeight:
 
     def untiled_data(self) -> torch.Tensor:
         """Row-major copy of the stored matrix (bf16 values or e4m3 bytes)."""
+        if self.fmt == "f32":
+            return self.w
         t = self.w if self.fmt == "bf16" else self.mx.data
         return mxfp8.untile_weight(t) if self.is_tiled else t
 
@@ -78,15 +83,15 @@ class LinearWeight:
         """fp32 copy of the full matrix (tests and CPU reference paths)."""
         if self.is_quant:
             return self.q.dequantize()
-        if self.fmt == "bf16":
+        if self.fmt in ("bf16", "f32"):
             return self.untiled_data().float()
         return mxfp8.dequantize(self.mx)
 
     def nbytes(self) -> int:
         if self.is_quant:
             return self.q.nbytes()
-        if self.fmt == "bf16":
-            return self.w.numel() * 2
+        if self.fmt in ("bf16", "f32"):
+            return self.w.numel() * self.w.element_size()
         return self.mx.data.numel() + self.mx.sf.numel()
 
     def to(self, device) -> "LinearWeight":
@@ -182,6 +187,8 @@ def make_linear(w_f, fmt: str, bias: Optional[torch.Tensor] = None, groups: int 
     n = rpg if groups else rows
     if fmt == "bf16":
         return LinearWeight("bf16", n, k, w=w_f.to(torch.bfloat16).contiguous(), bias=bias, groups=groups, rows_per_group=rpg)
+    if fmt == "f32":
+        return LinearWeight("f32", n, k, w=w_f.to(torch.float32).contiguous(), bias=bias, groups=groups, rows_per_group=rpg)
     if fmt == "mxfp8":
         if w_f.is_cuda:
             mx = ew.mx_quantize(w_f.to(torch.bfloat16).contiguous())
@@ -208,6 +215,18 @@ class SsmWeights:
 
 
 @dataclass
+class LightningWeights:
+    """A lightning-attention mixer."""
+    w_in: LinearWeight            # rows [q ; k ; v ; gate]
+    decay: torch.Tensor           # f32 [heads]
+    norm: torch.Tensor            # f32 [heads * v_dim]
+    w_out: LinearWeight           # [H, heads * v_dim]
+
+    def to(self, device) -> "LightningWeights":
+        return LightningWeights(self.w_in.to(device), self.decay.to(device), self.norm.to(device), self.w_out.to(device))
+
+
+@dataclass
 class LayerWeights:
     attn_norm: torch.Tensor
     wqkv: Optional[LinearWeight]                  # rows [Q ; K ; V] (+ [gate] after V when the attention output is gated); None in SSM layers
@@ -225,6 +244,16 @@ class LayerWeights:
     sh_gate_up: Optional[LinearWeight] = None     # shared expert [gate ; up]
     sh_down: Optional[LinearWeight] = None
     sh_gate: Optional[torch.Tensor] = None        # bf16 [1, H]: sigmoid gate of the shared expert (absent = ungated)
+    lin: Optional[LightningWeights] = None        # lightning-attention layer (then wqkv / wo are None)
+    rel_bias: Optional[torch.Tensor] = None       # f32 [heads, N + 1] distance bias (ops.attention.distance_bias_table)
+
+    def linears(self) -> List[LinearWeight]:
+        """Every projection matrix of the layer."""
+        own = [self.wqkv, self.wo, self.w_gate_up, self.w_down, self.w13, self.w2, self.sh_gate_up, self.sh_down]
+        for part in (self.ssm, self.lin):
+            if part is not None:
+                own += [part.w_in, part.w_out]
+        return [lw for lw in own if lw is not None]
 
 
 @dataclass
@@ -240,6 +269,12 @@ class ModelWeights:
     ep_rank: int = 0
     ep_size: int = 1
     vocab_start: int = 0                          # first vocabulary id of the LM-head shard
+    loop_step: Optional[torch.Tensor] = None      # f32 [times, H]: vectors added in front of the passes of a layer loop
+
+    @property
+    def kv_dtype(self) -> str:
+        """The KV cache format that goes with the weights."""
+        return "f32" if self.fmt == "f32" else "bf16"
 
     def to(self, device) -> "ModelWeights":
         def mv(x):
@@ -247,18 +282,17 @@ class ModelWeights:
         layers = [LayerWeights(attn_norm=mv(l.attn_norm), wqkv=mv(l.wqkv), wo=mv(l.wo), ffn_norm=mv(l.ffn_norm), q_norm=mv(l.q_norm),
                                k_norm=mv(l.k_norm), w_gate_up=mv(l.w_gate_up), w_down=mv(l.w_down), router=mv(l.router),
                                router_bias=mv(l.router_bias), w13=mv(l.w13), w2=mv(l.w2), ssm=mv(l.ssm), sh_gate_up=mv(l.sh_gate_up),
-                               sh_down=mv(l.sh_down), sh_gate=mv(l.sh_gate)) for l in self.layers]
+                               sh_down=mv(l.sh_down), sh_gate=mv(l.sh_gate), lin=mv(l.lin), rel_bias=mv(l.rel_bias)) for l in self.layers]
         return ModelWeights(cfg=self.cfg, embed=mv(self.embed), layers=layers, final_norm=mv(self.final_norm), lm_head=mv(self.lm_head),
                             fmt=self.fmt, tp_rank=self.tp_rank, tp_size=self.tp_size, ep_rank=self.ep_rank, ep_size=self.ep_size,
-                            vocab_start=self.vocab_start)
+                            vocab_start=self.vocab_start, loop_step=mv(self.loop_step))
 
     def tile_(self) -> "ModelWeights":
         """Put every projection matrix into the tiled weight layout (in place).  An LM head that shares its storage with
         the embedding table (tied embeddings) stays row-major: the embedding lookup reads rows."""
         for l in self.layers:
-            for lw in (l.wqkv, l.wo, l.w_gate_up, l.w_down, l.w13, l.w2, l.sh_gate_up, l.sh_down) + ((l.ssm.w_in, l.ssm.w_out) if l.ssm else ()):
-                if lw is not None:
-                    lw.tile_()
+            for lw in l.linears():
+                lw.tile_()
         if self.lm_head.w is not None and self.lm_head.w.data_ptr() != self.embed.data_ptr():
             self.lm_head.tile_()
         return self
@@ -266,9 +300,8 @@ class ModelWeights:
     def nbytes(self) -> int:
         tot = self.embed.numel() * 2 + self.lm_head.nbytes()
         for l in self.layers:
-            for lw in (l.wqkv, l.wo, l.w_gate_up, l.w_down, l.w13, l.w2, l.sh_gate_up, l.sh_down) + ((l.ssm.w_in, l.ssm.w_out) if l.ssm else ()):
-                if lw is not None:
-                    tot += lw.nbytes()
+            for lw in l.linears():
+                tot += lw.nbytes()
         return tot
 
 
@@ -307,6 +340,8 @@ class RandomSource:
         return True
 
     def get(self, name: str, shape) -> torch.Tensor:
+        if name.endswith("norm.weight") and not name.endswith("lin_norm.weight") and self.cfg.norm_offset:
+            return torch.full(tuple(shape), 1.0 - self.cfg.norm_offset, dtype=torch.bfloat16, device=self.device)
         if name.endswith("norm.weight"):
             return torch.ones(tuple(shape), dtype=torch.bfloat16, device=self.device)
         if name.endswith("ssm_a"):                       # fixed decay constants are negative
@@ -374,6 +409,10 @@ def build_weights(cfg: ModelConfig, src, fmt: str = "bf16", device="cuda", tp_ra
 
     TP shards attention and the dense FFN Megatron style (q/k/v/gate/up by rows, o/down by columns; KV heads are
     replicated when ``n_kv_heads < tp_size``), EP keeps the experts ``[ep_rank * E/ep_size, (ep_rank+1) * E/ep_size)``."""
+    if cfg.is_layered:
+        if tp_size > 1 or ep_size > 1 or layer_range is not None or n_layers is not None:
+            raise NotImplementedError("models described layer by layer run unsharded")
+        return _build_layered(cfg, src, fmt, torch.device(device), tile)
     h, d = cfg.hidden, cfg.head_dim
     dev = torch.device(device)
     assert cfg.n_heads % tp_size == 0, "n_heads must divide by the TP size"
@@ -458,6 +497,71 @@ def build_weights(cfg: ModelConfig, src, fmt: str = "bf16", device="cuda", tp_ra
     mw = ModelWeights(cfg=cfg, embed=embed, layers=layers, final_norm=mv(src.get("output_norm.weight", (h,)).to(torch.bfloat16)),
                       lm_head=lm_head, fmt=fmt, tp_rank=tp_rank, tp_size=tp_size, ep_rank=ep_rank, ep_size=ep_size, vocab_start=v0)
     if tile if tile is not None else dev.type == "cuda":
+        mw.tile_()
+    return mw
+
+
+def _padded_linear(t: torch.Tensor, fmt: str, dev, rows: int = 0, bias: Optional[torch.Tensor] = None) -> LinearWeight:
+    """A projection whose input rows are padded the way ``ops.stream`` pads them (``row_width``); ``rows`` pads the output features too.
+    The padding is zero."""
+    k = row_width(t.shape[1], torch.float32 if fmt == "f32" else torch.bfloat16)
+    rows = rows or t.shape[0]
+    if (rows, k) != tuple(t.shape):
+        t = torch.nn.functional.pad(t, (0, k - t.shape[1], 0, rows - t.shape[0]))
+    return make_linear(t.to(dev), fmt, bias=bias)
+
+
+def _build_layered(cfg: ModelConfig, src, fmt: str, dev, tile: Optional[bool]) -> ModelWeights:
+    """Weights of a model described layer by layer.  Norm weights become f32 ``offset + w``; the factor of the logits is folded into the
+    final norm's weight."""
+    if fmt not in ("bf16", "f32"):
+        raise ValueError(f"models described layer by layer run in bf16 or f32, not {fmt!r}")
+    h = cfg.hidden
+    exact = fmt == "f32"
+
+    def norm_w(name, n, offset):
+        return (src.get(name, (n,)).float() + offset).contiguous().to(dev)
+
+    layers: List[LayerWeights] = []
+    for li, sp in enumerate(cfg.layer_specs):
+        pre = f"blk.{li}."
+        lw = LayerWeights(attn_norm=norm_w(pre + "attn_norm.weight", h, cfg.norm_offset), wqkv=None, wo=None,
+                          ffn_norm=norm_w(pre + "ffn_norm.weight", h, cfg.norm_offset) if sp.ffn else None)
+        nv = sp.n_heads * sp.v_dim
+        if sp.mixer == "lightning":
+            w_in = torch.cat([src.get(pre + "lin_q.weight", (sp.q_dim, h)), src.get(pre + "lin_k.weight", (sp.q_dim, h)),
+                              src.get(pre + "lin_v.weight", (nv, h)), src.get(pre + "lin_gate.weight", (nv, h))])
+            lw.lin = LightningWeights(w_in=_padded_linear(w_in, fmt, dev), decay=torch.tensor(sp.decay, dtype=torch.float32, device=dev),
+                                      norm=norm_w(pre + "lin_norm.weight", nv, 0.0),
+                                      w_out=_padded_linear(src.get(pre + "lin_out.weight", (h, nv)), fmt, dev))
+        else:
+            nk, nkv = sp.n_kv_heads * sp.head_dim, sp.n_kv_heads * sp.v_dim
+            w = torch.cat([src.get(pre + "attn_q.weight", (sp.q_dim, h)), src.get(pre + "attn_k.weight", (nk, h)), src.get(pre + "attn_v.weight", (nkv, h))])
+            bias = None
+            if sp.qkv_bias:
+                bias = torch.cat([src.get(pre + f"attn_{c}.bias", (n,)).float() for c, n in (("q", sp.q_dim), ("k", nk), ("v", nkv))]).contiguous().to(dev)
+            lw.wqkv = _padded_linear(w, fmt, dev, bias=bias)
+            # the attention kernels emit heads of the cache's (padded) value width: the output projection has zero columns there
+            wo = src.get(pre + "attn_output.weight", (h, nv))
+            dvp = cache_head_dims(sp.head_dim, sp.v_dim, torch.float32 if exact else torch.bfloat16)[1]
+            wo = torch.nn.functional.pad(wo.reshape(h, sp.n_heads, sp.v_dim), (0, dvp - sp.v_dim)).reshape(h, sp.n_heads * dvp)
+            lw.wo = _padded_linear(wo, fmt, dev)
+            if sp.rel_buckets:
+                lw.rel_bias = distance_bias_table(src.get(pre + "attn_rel.weight", (sp.rel_buckets, sp.n_heads)).float().cpu(), sp.rel_max).to(dev)
+        if sp.ffn:
+            wg, wu = src.get(pre + "ffn_gate.weight", (sp.ffn, h)), src.get(pre + "ffn_up.weight", (sp.ffn, h))
+            wd = src.get(pre + "ffn_down.weight", (h, sp.ffn))
+            fp = sp.ffn if exact else (sp.ffn + 127) // 128 * 128       # the gate / up GEMM works on whole 128-row tiles
+            pad = torch.nn.functional.pad
+            lw.w_gate_up = _padded_linear(torch.cat([pad(wg, (0, 0, 0, fp - sp.ffn)), pad(wu, (0, 0, 0, fp - sp.ffn))]), fmt, dev)
+            lw.w_down = _padded_linear(pad(wd, (0, fp - sp.ffn)), fmt, dev)
+        layers.append(lw)
+    embed = src.get("token_embd.weight", (cfg.vocab, h)).to(torch.float32 if exact else torch.bfloat16).contiguous().to(dev)
+    head = embed if (cfg.tie_embeddings or not src.has("output.weight")) else src.get("output.weight", (cfg.vocab, h))
+    step = src.get("loop_step.weight", (cfg.loop.times, h)).float().contiguous().to(dev) if cfg.loop is not None else None
+    mw = ModelWeights(cfg=cfg, embed=embed, layers=layers, final_norm=norm_w("output_norm.weight", h, cfg.norm_offset) * cfg.logit_scale,
+                      lm_head=_padded_linear(head, fmt, dev), fmt=fmt, loop_step=step)
+    if (tile if tile is not None else dev.type == "cuda") and not exact:
         mw.tile_()
     return mw
 

@@ -307,3 +307,101 @@ def attention_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, cau
         p = torch.softmax(sc, dim=-1)
         out[q0:q1] = torch.einsum("hqk,khd->qhd", p, v)
     return out.to(torch.bfloat16)
+
+
+# ------------------------------------------------------------------------------------------ masks, distance bias, any head size
+LOG2E = math.log2(math.e)
+
+
+def distance_bucket(n: int, buckets: int, max_distance: float) -> int:
+    """Bucket of a query-key distance ``n >= 0``: one bucket per distance below ``buckets // 2``, then logarithmically wider ones up to
+    ``max_distance``; everything beyond falls into the last."""
+    half = buckets // 2
+    if n < half:
+        return n
+    if half == 0:
+        return buckets - 1
+    if max_distance <= half:
+        return buckets - 1
+    x = math.log(n / half) / math.log(max_distance / half) * (buckets - half)
+    near = round(x)
+    x = near if abs(x - near) < 1e-9 * max(1.0, abs(x)) else x        # an exact power hits its bucket's edge: rounding must not miss it
+    return min(buckets - 1, half + math.floor(x))
+
+
+def distance_bias_table(rel: torch.Tensor, max_distance: float) -> torch.Tensor:
+    """``rel [buckets, heads]`` -> f32 ``[heads, N + 1]``: the bias of every distance 0 .. N - 1 times log2(e) (larger distances equal the
+    last of them), and in column N the largest bias of the head (an upper bound the flash kernels use as part of their reference
+    maximum)."""
+    buckets, heads = rel.shape
+    idx, n = [], 0
+    while True:
+        b = distance_bucket(n, buckets, max_distance)
+        idx.append(b)
+        if b == buckets - 1:
+            break
+        n += 1
+    t = rel.double()[torch.tensor(idx)].t() * LOG2E                   # [heads, N]
+    return torch.cat([t, t.max(dim=1, keepdim=True).values], dim=1).float().contiguous()
+
+
+def flash_head_dims(dk: int, dv: int):
+    """Padded (key, value) widths of a head in the caches of the tcgen05 kernels (64 or 128 columns), or None if it is too wide."""
+    if dk > 128 or dv > 128:
+        return None
+    return (64 if dk <= 64 else 128), (64 if dv <= 64 else 128)
+
+
+def cache_head_dims(dk: int, dv: int, dtype: torch.dtype):
+    """Widths a head's keys and values take in the KV cache: padded for the tcgen05 kernels, else as they are (bf16: to 8 elements)."""
+    if dtype == torch.float32:
+        return dk, dv
+    return flash_head_dims(dk, dv) or ((dk + 7) // 8 * 8, (dv + 7) // 8 * 8)
+
+
+def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window=0, keep_first=0, bias=None) -> torch.Tensor:
+    t, hq, d = q.shape
+    g = hq // k_cache.shape[1]
+    out = torch.zeros(t, hq, v_cache.shape[2], dtype=torch.float32)
+    cu = cu_q.tolist()
+    for s in range(len(cu) - 1):
+        q0, q1 = cu[s], cu[s + 1]
+        ql, kl = q1 - q0, int(kv_len[s])
+        if ql == 0:
+            continue
+        n_pages = (kl + page_size - 1) // page_size
+        slots = (block_table[s, :n_pages].long().unsqueeze(1) * page_size + torch.arange(page_size)).reshape(-1)[:kl]
+        k = k_cache[slots].float().repeat_interleave(g, dim=1)
+        v = v_cache[slots].float().repeat_interleave(g, dim=1)
+        sc = torch.einsum("qhd,khd->hqk", q[q0:q1].float(), k)
+        dist = torch.arange(kl - ql, kl).unsqueeze(1) - torch.arange(kl).unsqueeze(0)
+        if bias is not None:
+            n = bias.shape[1] - 1
+            sc = sc + bias[:, dist.clamp(0, n - 1)]
+        see = dist >= 0
+        if window > 0:
+            see &= (dist < window) | (torch.arange(kl).unsqueeze(0) < keep_first)
+        p = torch.softmax((sc * math.log(2.0)).masked_fill(~see.unsqueeze(0), float("-inf")), dim=-1)
+        out[q0:q1] = torch.einsum("hqk,khd->qhd", p, v)
+    return out.to(k_cache.dtype)
+
+
+def attention_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
+                     block_table: torch.Tensor, page_size: int, window: int = 0, keep_first: int = 0, bias: Optional[torch.Tensor] = None,
+                     plan=None, decode: bool = False) -> torch.Tensor:
+    """Causal attention in which position i sees j <= i with ``i - j < window`` (0: no limit) or ``j < keep_first``, with an optional distance
+    bias (``distance_bias_table``) added to the scores.  Key and value widths may differ (``k_cache [slots, Hkv, dk]``, ``v_cache [slots, Hkv,
+    dv]``, ``q [T, Hq, dk]`` times scale * log2(e)).  Returns ``[T, Hq, dv]`` in the cache's dtype.  ``plan``: ``(work list, KV splits)`` for
+    the tcgen05 kernels; without one, or for an f32 cache or wider heads, the any-size kernel runs."""
+    t, hq, dk = q.shape
+    hkv, dv = k_cache.shape[1], v_cache.shape[2]
+    if not q.is_cuda:
+        return attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window, keep_first, bias)
+    out = torch.empty(t, hq, dv, dtype=k_cache.dtype, device=q.device)
+    n_bias, ld_bias = (bias.shape[1] - 1, bias.stride(0)) if bias is not None else (0, 0)
+    stream = _c(torch.cuda.current_stream().cuda_stream)
+    rc = _native.cuda().gb_attn_any(_p(q), _p(k_cache), _p(v_cache), _p(out), _i(int(k_cache.dtype == torch.float32)), _p(cu_q), _p(kv_len),
+                                    _p(block_table), _i(block_table.shape[1]), _i(page_size), _i(cu_q.numel() - 1), _l(k_cache.shape[0]), _i(t), _i(hq),
+                                    _i(hkv), _i(dk), _i(dv), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), stream)
+    _native.check(rc, "gb_attn_any")
+    return out

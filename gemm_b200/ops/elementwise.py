@@ -266,14 +266,15 @@ def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def silu_mul_partials(pend, quantize: bool = False, sf_layout: int = 128):
-    """SiLU(gate) * up from the K-split partial sums of ``ops.gemm.swiglu_partials`` (``pend.buf`` f32 ``[S, M, 2I]``): bf16 ``[M, I]``, or
-    an ``MxTensor`` when ``quantize``."""
+def silu_mul_partials(pend, quantize: bool = False, sf_layout: int = 128, act: str = "silu"):
+    """act(gate) * up (SiLU, or the tanh form of GELU) from the K-split partial sums of ``ops.gemm.swiglu_partials`` (``pend.buf`` f32
+    ``[S, M, 2I]``): bf16 ``[M, I]``, or an ``MxTensor`` when ``quantize``."""
     s_, m, two_i = pend.buf.shape
     inter = two_i // 2
     if not pend.buf.is_cuda:
         y = pend.buf.sum(0)
-        h = torch.nn.functional.silu(y[:, :inter]) * y[:, inter:]
+        from .gemm import gate_act_ref
+        h = gate_act_ref(y[:, :inter], act) * y[:, inter:]
         return mxfp8.quantize(h, sf_layout=sf_layout) if quantize else h.to(torch.bfloat16)
     dev = pend.buf.device
     out = q = sf = None
@@ -284,7 +285,7 @@ def silu_mul_partials(pend, quantize: bool = False, sf_layout: int = 128):
     else:
         out = torch.empty(m, inter, dtype=torch.bfloat16, device=dev)
     rc = _native.cuda().gb_silu_mul_partials(_p(pend.buf), _i(s_), _l(m * two_i), _p(out), _p(q), _p(sf), _l(m), _i(inter),
-                                             _i(1 if sf_layout == 32 else 0), _s())
+                                             _i(1 if sf_layout == 32 else 0), _i(1 if act == "gelu_tanh" else 0), _s())
     _native.check(rc, "gb_silu_mul_partials")
     return MxTensor(q, sf, m, inter, sf_layout) if quantize else out
 

@@ -16,7 +16,8 @@ from .. import _native
 from . import mxfp8
 from .mxfp8 import MxTensor
 
-GEMM_MX, GEMM_DUAL, GEMM_QUANT_OUT, GEMM_OUT_F32, GEMM_W_TILED, GEMM_DUAL_RAW = 1, 2, 4, 8, 16, 32
+GEMM_MX, GEMM_DUAL, GEMM_QUANT_OUT, GEMM_OUT_F32, GEMM_W_TILED, GEMM_DUAL_RAW, GEMM_GELU = 1, 2, 4, 8, 16, 32, 64
+GATE_ACTS = ("silu", "gelu_tanh")         # activations of a gated feed-forward, by the code the kernels use
 
 
 class GemmExtras(ctypes.Structure):
@@ -173,18 +174,38 @@ def linear_argmax(x: torch.Tensor, w: torch.Tensor, idx_offset: int = 0, want_va
     return (out, val) if want_value else out
 
 
+def gate_act_ref(g: torch.Tensor, act: str) -> torch.Tensor:
+    if act == "gelu_tanh":
+        return torch.nn.functional.gelu(g, approximate="tanh")
+    return torch.nn.functional.silu(g)
+
+
+def linear_f32(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``x [M, K] @ w [N, K]^T (+ bias)`` with f32 operands and f32 FMAs (csrc/kernels/gemm_f32.cu): the "f32" weight format."""
+    m, k = x.shape
+    n = w.shape[0]
+    assert x.dtype == torch.float32 and w.dtype == torch.float32 and x.stride(1) == 1 and w.stride(1) == 1 and w.shape[1] == k
+    if not x.is_cuda:
+        y = x @ w.t()
+        return y + bias if bias is not None else y
+    out = torch.empty(m, n, dtype=torch.float32, device=x.device)
+    rc = _native.cuda().gb_gemm_f32(_p(x), _p(w), _p(bias), _p(out), _i(m), _i(n), _i(k), _i(x.stride(0)), _i(w.stride(0)), _i(n), _stream())
+    _native.check(rc, "gb_gemm_f32")
+    return out
+
+
 def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: Optional[torch.Tensor] = None,
-                  tn: Optional[int] = None, w_tiled: bool = False) -> torch.Tensor:
-    """``silu(x @ Wg^T) * (x @ Wu^T)`` with ``w_gate_up = [Wg; Wu]`` stacked along rows ([2I, K])."""
+                  tn: Optional[int] = None, w_tiled: bool = False, act: str = "silu") -> torch.Tensor:
+    """``act(x @ Wg^T) * (x @ Wu^T)`` with ``w_gate_up = [Wg; Wu]`` stacked along rows ([2I, K]); ``act`` is one of ``GATE_ACTS``."""
     m, k = x.shape
     inter = w_gate_up.shape[0] // 2
     if not x.is_cuda:
         y = x.float() @ (mxfp8.untile_weight(w_gate_up) if w_tiled else w_gate_up).float().t()
-        return (torch.nn.functional.silu(y[:, :inter]) * y[:, inter:]).to(torch.bfloat16)
+        return (gate_act_ref(y[:, :inter], act) * y[:, inter:]).to(torch.bfloat16)
     if out is None:
         out = torch.empty(m, inter, dtype=torch.bfloat16, device=x.device)
-    _launch(w_gate_up, x, out, inter, k, m, w_gate_up.stride(0), x.stride(0), out.stride(0), GEMM_DUAL | (GEMM_W_TILED if w_tiled else 0),
-            tn or pick_tn(m, dual=True), up_row_offset=inter)
+    _launch(w_gate_up, x, out, inter, k, m, w_gate_up.stride(0), x.stride(0), out.stride(0),
+            GEMM_DUAL | (GEMM_W_TILED if w_tiled else 0) | (GEMM_GELU if act == "gelu_tanh" else 0), tn or pick_tn(m, dual=True), up_row_offset=inter)
     return out
 
 

@@ -56,8 +56,9 @@ class PageAllocator:
 
 class Engine:
     def __init__(self, weights: ModelWeights, max_batch: int, max_seq_len: int, page_size: int = 128, par=None,
-                 max_prefill_tokens: int = 16384, num_pages: Optional[int] = None, kv_dtype: str = "bf16"):
+                 max_prefill_tokens: int = 16384, num_pages: Optional[int] = None, kv_dtype: Optional[str] = None):
         self.w = weights
+        kv_dtype = kv_dtype or weights.kv_dtype
         self.cfg: ModelConfig = weights.cfg
         if weights.embed.is_cuda and "GB_PDL" not in os.environ:
             # Programmatic dependent launch (every kernel starts its prologue under the tail of the one before): chosen by what was
@@ -236,6 +237,7 @@ class Engine:
         st["block_table"] = bt
         st["cu_q"] = torch.arange(b + 1, dtype=torch.int32, device=self.device)
         st["work"] = att.build_work([1] * b, self.hq_local, self.hkv_local, splits).to(self.device)
+        st["plans"] = self.model.attention_plans([1] * b, max_kv, self.device, True)
         st["rows"] = torch.arange(b, dtype=torch.int64, device=self.device)
         st["tokens"] = torch.zeros(b, dtype=torch.int32, device=self.device)
         st["seq_slots"] = torch.arange(b, dtype=torch.int32, device=self.device)
@@ -272,7 +274,8 @@ class Engine:
         st = self._static
         fb = ForwardBatch(ids=st["ids"], positions=st["positions"], slots=st["slots"], cu_q=st["cu_q"], kv_len=st["kv_len"],
                           block_table=st["block_table"], work=st["work"], logit_rows=st["rows"], num_splits=self._splits,
-                          n_tokens=st["ids"].numel(), seq_slots=st["seq_slots"], is_decode=True, stage_slots=st["stage_slots"])
+                          n_tokens=st["ids"].numel(), seq_slots=st["seq_slots"], is_decode=True, stage_slots=st["stage_slots"],
+                          plans=st["plans"])
         if self._sp.temperature <= 0 and not hasattr(self.par, "merge_sampled"):
             tok = self.model.forward_greedy(fb)
         else:

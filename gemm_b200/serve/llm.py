@@ -47,7 +47,8 @@ class LLM:
         self.page_size = page_size
         self.num_pages = num_pages
         hkv_local = max(1, self.cfg.n_kv_heads // weights.tp_size)
-        self.kv = KvCache.allocate(self.cfg, num_pages, page_size, self.device, hkv_local, n_layers=len(weights.layers), n_seq_slots=max_running)
+        self.kv = KvCache.allocate(self.cfg, num_pages, page_size, self.device, hkv_local, n_layers=len(weights.layers), n_seq_slots=max_running,
+                                   kv_dtype=weights.kv_dtype)
         self._free_slots = list(range(max_running))       # recurrent-state slots of the hybrid models, one per running request
         self._slot_of: Dict[int, int] = {}
         self.blocks = KvBlockManager(num_pages, page_size)
@@ -100,10 +101,28 @@ class LLM:
         """Speculative decoding inside continuous batching: decode items of greedy requests carry up to ``drafter.gamma`` draft
         tokens (``drafter.propose(tokens)``, e.g. ``serve.speculative.NgramDrafter``), verified in the same step; the scheduler
         reserves the extra positions and counts them against the token budget.  ``None`` switches it off."""
-        if drafter is not None and self.cfg.is_hybrid:
+        if drafter is not None and self.cfg.has_recurrent_state:
             raise ValueError("speculative decoding needs a cache that can drop rejected positions: recurrent layers cannot")
         self.drafter = drafter
         self.sched.set_lookahead(drafter.gamma if drafter is not None else 0)
+
+    def build_batch(self, seqs: Sequence[int], slots: Sequence[int], q_lens: Sequence[int], ctx: Sequence[int], ids: Sequence[int],
+                    rows: Optional[Sequence[int]] = None) -> ForwardBatch:
+        """One engine step over the block manager's sequences ``seqs`` (state slots ``slots``): sequence i brings ``q_lens[i]`` tokens on top of
+        ``ctx[i]`` cached positions.  ``rows``: the places among the step's tokens whose logits are wanted (default: each sequence's last)."""
+        pages = [self.blocks.pages(s) for s in seqs]
+        bt = torch.zeros(len(seqs), max(len(p) for p in pages), dtype=torch.int32)
+        for i, p in enumerate(pages):
+            bt[i, : len(p)] = torch.tensor(p, dtype=torch.int32)
+        # a sequence starts (or restarts after a recompute-preemption) from an empty recurrent state: unlike K/V, which the prefill
+        # overwrites, the state that an earlier user of the slot (or the first pass) left would otherwise leak into it
+        fresh = [sl for sl, c in zip(slots, ctx) if c == 0]
+        if fresh:
+            self.kv.reset_slots(fresh)
+        fb = ForwardBatch.build(q_lens, ctx, ids, bt, self.page_size, self.model.hq_local, self.model.hkv_local, self.device, seq_slots=slots)
+        if rows is not None:
+            fb.logit_rows = torch.tensor(list(rows), dtype=torch.int64, device=self.device)
+        return fb
 
     def has_work(self) -> bool:
         return self.sched.num_waiting > 0 or self.sched.num_running > 0
@@ -126,8 +145,6 @@ class LLM:
             return {}
         self._idle_steps = 0
         q_lens, ctx, ids, drafts = [], [], [], []
-        max_pages = max(len(self.blocks.pages(it.seq)) for it in plan)
-        bt = torch.zeros(len(plan), max_pages, dtype=torch.int32)
         draft_of: Dict[int, List[int]] = {}
         if self.drafter is not None:                        # drafts for the decode items of greedy requests, batched if the drafter can
             cand = [(it, self._reqs[it.req_id]) for it in plan if not it.is_prefill and self._reqs[it.req_id].sp.temperature <= 0]
@@ -138,10 +155,8 @@ class LLM:
                 ds = [self.drafter.propose(r.tokens) if room > 0 else [] for (_, r), room in zip(cand, rooms)]
             for (it, _), d, room in zip(cand, ds, rooms):
                 draft_of[it.req_id] = [int(t) for t in d][:room]
-        for i, it in enumerate(plan):
+        for it in plan:
             r = self._reqs[it.req_id]
-            pages = self.blocks.pages(it.seq)
-            bt[i, : len(pages)] = torch.tensor(pages, dtype=torch.int32)
             draft = draft_of.get(it.req_id, [])
             drafts.append(draft)
             q_lens.append(it.q_len + len(draft))
@@ -149,12 +164,13 @@ class LLM:
             ids.extend(r.tokens[it.ctx_len: it.ctx_len + it.q_len] + draft)
             if it.req_id not in self._slot_of:              # first chunk of this request: take a state slot
                 self._slot_of[it.req_id] = self._free_slots.pop()
-            if it.is_prefill and it.ctx_len == 0:
-                # a sequence starts (or restarts after a recompute-preemption) from an empty recurrent state: unlike K/V, which the
-                # re-prefill overwrites, the conv / Delta-Net state of the first pass would otherwise leak into the second
-                self.kv.reset_slots([self._slot_of[it.req_id]])
-        fb = ForwardBatch.build(q_lens, ctx, ids, bt, self.page_size, self.model.hq_local, self.model.hkv_local, self.device,
-                                seq_slots=[self._slot_of[it.req_id] for it in plan])
+        # logits: one row per plan item (its last token); an item with draft tokens gets a row for each of its positions
+        row0, rows, p0 = [], [], 0
+        for q, d in zip(q_lens, drafts):
+            row0.append(len(rows))
+            rows.extend(range(p0 + q - 1 - len(d), p0 + q))
+            p0 += q
+        fb = self.build_batch([it.seq for it in plan], [self._slot_of[it.req_id] for it in plan], q_lens, ctx, ids, rows)
         if any(self._reqs[it.req_id].embeds is not None and it.ctx_len < self._reqs[it.req_id].prompt_len for it in plan):
             # a prefill chunk of a multimodal prompt is in the batch: every row of the step enters as an embedding
             rows_in = ew.embed(fb.ids, self.w.embed).clone()
@@ -170,14 +186,6 @@ class LLM:
                         ds_in[:, p0: p0 + hi - lo] = r.deepstack[:, lo:hi].to(self.device, torch.bfloat16)
                 p0 += q
             fb.embeds, fb.deepstack = rows_in, ds_in
-        # logits: one row per plan item (its last token); an item with draft tokens gets a row for each of its positions
-        row0, rows, p0 = [], [], 0
-        for q, d in zip(q_lens, drafts):
-            row0.append(len(rows))
-            rows.extend(range(p0 + q - 1 - len(d), p0 + q))
-            p0 += q
-        if any(drafts):
-            fb.logit_rows = torch.tensor(rows, dtype=torch.int64, device=self.device)
         logits = self.model.forward(fb)
         greedy_rows = sampling.argmax(logits).cpu().tolist() if any(drafts) else None     # one device read for all drafted items
         produced: Dict[int, int] = {}

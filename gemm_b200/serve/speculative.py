@@ -60,7 +60,7 @@ class ModelDrafter:
     the target's does: positions beyond the common prefix of what it was fed and what was kept are overwritten."""
 
     def __init__(self, model: Transformer, kv: KvCache, page_size: int, num_pages: int, gamma: int = 4):
-        if model.cfg.is_hybrid:
+        if model.cfg.has_recurrent_state:
             raise ValueError("a draft model with recurrent layers cannot drop rejected positions")
         self.model, self.kv, self.page, self.gamma = model, kv, page_size, gamma
         self.blocks = KvBlockManager(num_pages, page_size)
@@ -153,7 +153,7 @@ class SpeculativeDecoder:
     """Greedy generation for a fixed group of prompts over a ``Transformer`` and its paged cache (CPU or GPU tensors)."""
 
     def __init__(self, model: Transformer, kv: KvCache, page_size: int, num_pages: int, drafter=None):
-        if model.cfg.is_hybrid:
+        if model.cfg.has_recurrent_state:
             raise ValueError("speculative decoding needs a cache that can drop rejected positions: recurrent layers cannot")
         if model.w.tp_size > 1 and model.w.lm_head.w.shape[0] != model.cfg.vocab:
             raise ValueError("speculative decoding takes the arg-max of the local logits: it needs an unsharded LM head")

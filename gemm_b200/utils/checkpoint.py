@@ -23,7 +23,7 @@ MAGIC = b"GBKV1\n"
 
 def _geometry(engine) -> Dict:
     cfg = engine.cfg
-    return {"arch": cfg.arch, "n_layers": len(engine.w.layers), "hidden": cfg.hidden, "n_kv_heads_local": _kv_rows(engine)[0],
+    return {"arch": cfg.arch, "n_layers": len(engine.kv.k), "hidden": cfg.hidden, "n_kv_heads_local": _kv_rows(engine)[0],
             "head_dim": cfg.head_dim, "vocab": cfg.vocab, "tp_size": engine.w.tp_size, "tp_rank": engine.w.tp_rank,
             "ep_size": engine.w.ep_size, "ep_rank": engine.w.ep_rank, "fmt": engine.w.fmt,
             "ssm_layers": [i for i in range(len(engine.kv.k)) if engine.kv.k[i].shape[0] == 0]}
@@ -60,7 +60,7 @@ def save_state(engine, path: str, next_tokens=None, kv_format: str = "bf16") -> 
         for li in range(len(engine.kv.k)):
             if engine.kv.k[li].shape[0] == 0:
                 # recurrent layer: the state slots of the live sequences (slot s belongs to sequence s in a static-batch engine)
-                for t in (engine.kv.conv[li], engine.kv.rec[li]):
+                for t in engine.kv.recurrent(li):
                     f.write(t[:n_seq].contiguous().cpu().numpy().tobytes())
                 continue
             for t in (engine.kv.k[li], engine.kv.v[li]):
@@ -107,12 +107,10 @@ def load_state(engine, path: str) -> torch.Tensor:
             pages = engine.seq_pages[s]
             slots.extend(pages[p // ps] * ps + p % ps for p in range(n))
         idx = torch.tensor(slots, dtype=torch.long, device=engine.device)
-        hk, hd = _kv_rows(engine)
-        row = hk * hd * 2
         n_seq = len(header["seq_len"])
         for li in range(len(engine.kv.k)):
             if engine.kv.k[li].shape[0] == 0:
-                for t in (engine.kv.conv[li], engine.kv.rec[li]):
+                for t in engine.kv.recurrent(li):
                     nb = n_seq * t[0].numel() * 4
                     buf = f.read(nb)
                     if len(buf) != nb:
@@ -120,8 +118,9 @@ def load_state(engine, path: str) -> torch.Tensor:
                     t[:n_seq] = torch.frombuffer(bytearray(buf), dtype=torch.float32).reshape(n_seq, *t.shape[1:]).to(engine.device)
                 continue
             for t in (engine.kv.k[li], engine.kv.v[li]):
+                row = t.shape[1] * t.shape[2] * t.element_size()
                 if kv_format == "q8":
-                    nq, ns = len(slots) * (row // 2), len(slots) * t.shape[1] * 4
+                    nq, ns = len(slots) * t.shape[1] * t.shape[2], len(slots) * t.shape[1] * 4
                     buf, sbuf = f.read(nq), f.read(ns)
                     if len(buf) != nq or len(sbuf) != ns:
                         raise ValueError("truncated KV state file")
@@ -132,6 +131,6 @@ def load_state(engine, path: str) -> torch.Tensor:
                 buf = f.read(len(slots) * row)
                 if len(buf) != len(slots) * row:
                     raise ValueError("truncated KV state file")
-                vals = torch.frombuffer(bytearray(buf), dtype=torch.uint8).view(torch.bfloat16).reshape(len(slots), t.shape[1], t.shape[2])
+                vals = torch.frombuffer(bytearray(buf), dtype=torch.uint8).view(t.dtype).reshape(len(slots), t.shape[1], t.shape[2])
                 t[idx] = vals.to(engine.device)
     return torch.tensor(header["next_tokens"], dtype=torch.int32)
