@@ -90,7 +90,7 @@ def _load_llm(args):
 
 def _add_model_args(p):
     p.add_argument("--model", required=True, help="GGUF file, HF safetensors directory, or synthetic:<preset>")
-    p.add_argument("--format", default="bf16", choices=["bf16", "mxfp8"], help="run-time weight format")
+    p.add_argument("--format", default="bf16", choices=["bf16", "mxfp8", "f32"], help="run-time weight format (f32: models described layer by layer)")
     p.add_argument("--device", default="cuda")
     p.add_argument("--tokenizer", default="", help="GGUF file to take the tokenizer from (safetensors checkpoints)")
     p.add_argument("--max-running", type=int, default=64)
@@ -472,7 +472,7 @@ def main(argv=None):
     cp.set_defaults(fn=cmd_compare)
     dp = sub.add_parser("dump", help="per-layer hidden states as .npy")
     dp.add_argument("--model", required=True, help="GGUF file, HF safetensors directory, or synthetic:<preset>")
-    dp.add_argument("--format", default="bf16", choices=["bf16", "mxfp8"])
+    dp.add_argument("--format", default="bf16", choices=["bf16", "mxfp8", "f32"])
     dp.add_argument("--device", default="cuda")
     dp.add_argument("--ids", required=True, help="prompt as token ids")
     dp.add_argument("--out", required=True)

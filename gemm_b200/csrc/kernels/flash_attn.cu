@@ -49,7 +49,26 @@ struct FaArgs {
   uint8_t* out_q;
   uint8_t* out_sf;
   int out_sf32;             // scale-atom layout: one atom per 32 rows (1) or per 128 rows (0)
+  // masked form only (EXT)
+  int keep_first;           // positions below this stay visible behind the window
+  const float* bias;        // [hq][ld_bias]: n_bias scores added at distances 0, 1, ... (the last one beyond), times log2 e; then, per
+  int n_bias, ld_bias;      // distance n, the largest of the 128 from n on.  null = none
 };
+
+// KV blocks of a query tile or decode token, in order: with a window and kept first positions, the blocks of the kept positions that lie
+// in front of the window, then the window's own.
+struct FaBlocks {
+  int n_keep, lo, n;        // n blocks: 0 .. n_keep - 1, then lo, lo + 1, ...
+  __device__ __forceinline__ int at(int i) const { return i < n_keep ? i : lo + (i - n_keep); }
+};
+
+__device__ __forceinline__ FaBlocks fa_blocks(const FaArgs& a, int first_pos, int last_pos) {
+  FaBlocks b;
+  b.lo = first_pos / 128;
+  b.n_keep = min((a.keep_first + 127) / 128, b.lo);
+  b.n = b.n_keep + max(0, last_pos / 128 + 1 - b.lo);
+  return b;
+}
 
 __device__ __forceinline__ float fast_exp2(float x) {
   float y;
@@ -57,7 +76,19 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
+// Barrier over the 128 softmax threads (named barrier 1) that also ANDs a predicate: every thread learns whether all of them
+// got through their bounded wait, so they leave the loop together and nobody is left standing at a barrier.
+__device__ __forceinline__ bool softmax_bar_and(bool pred) {
+  uint32_t r;
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 q, %1, 0;\n\tbar.red.and.pred p, 1, 128, q;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+               : "=r"(r) : "r"((uint32_t)pred) : "memory");
+  return r != 0;
+}
+
 constexpr int kFaSmem = 32768 * 3 + 256 + 1024;
+
+// DK / DV: width of a key / value head in the cache (64 or 128 columns).  EXT: kept first positions and a distance bias.
+template <int DK, int DV, bool EXT>
 
 __global__ void __launch_bounds__(kFaThreads, 2)
 flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
@@ -111,10 +142,12 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   int last_pos = a.causal ? (pos0 + n_tok - 1) : (kv_len - 1);
   int first_pos = 0;
   if (a.window > 0) first_pos = max(0, pos0 - a.window + 1);
-  int blk_lo = first_pos / kBN, blk_hi = last_pos / kBN + 1;     // [lo, hi)
+  FaBlocks blocks = {0, first_pos / kBN, last_pos / kBN + 1 - first_pos / kBN};
+  if constexpr (EXT) blocks = fa_blocks(a, first_pos, last_pos);
+  int blk_lo = 0, blk_hi = blocks.n;                             // [lo, hi) of them
   if (a.num_splits > 1) {
-    const int nb = blk_hi - blk_lo, per = (nb + a.num_splits - 1) / a.num_splits;
-    blk_lo = blk_lo + split * per;
+    const int per = (blocks.n + a.num_splits - 1) / a.num_splits;
+    blk_lo = split * per;
     blk_hi = min(blk_hi, blk_lo + per);
   }
   int n_blk = max(0, blk_hi - blk_lo);
@@ -129,9 +162,9 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
   if (warp == 0) {
     if (lane == 0 && n_blk > 0) {
       // Q tile: box (64 d, G heads, tpt tokens), two d-halves
-      mbar_expect_tx(q_full, (uint32_t)(2 * 128 * G * tpt));
+      mbar_expect_tx(q_full, (uint32_t)(2 * DK * G * tpt));
       tma_load_3d(sQ, &tmQ, q_full, 0, kvh * G, q_begin + q_tok0);
-      tma_load_3d(sQ + 16384, &tmQ, q_full, 64, kvh * G, q_begin + q_tok0);
+      if constexpr (DK > 64) tma_load_3d(sQ + 16384, &tmQ, q_full, 64, kvh * G, q_begin + q_tok0);
       const int ppb = kBN / a.page_size;               // pages per KV block
       const uint32_t page_bytes = (uint32_t)a.page_size * 128;
       const int* bt = a.block_table + (size_t)seq * a.max_pages;
@@ -139,32 +172,32 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       bool ok = true;
       for (int j = 0; j < n_blk && ok; ++j) {
         const uint32_t ph = j & 1;
-        const int blk = blk_lo + j;
+        const int blk = blocks.at(blk_lo + j);
         // Pages past the end of the sequence are replaced by its last page: the tile is always filled with
         // finite cache contents (their scores are masked, and 0 * finite stays 0 in P V).
         // K_j may land as soon as S_{j-1} has been computed, V_j as soon as P_{j-1} V_{j-1} has: both long before they are needed.
         if (!mbar_wait(k_empty, ph ^ 1, abort_flag, a.status, 400, j)) { ok = false; break; }
-        mbar_expect_tx(k_full, 32768u);
+        mbar_expect_tx(k_full, 256u * DK);
         for (int p = 0; p < ppb; ++p) {
           const int page = bt[min(blk * ppb + p, last_page)];
           uint8_t* dst = sK + p * page_bytes;
           tma_load_3d(dst, &tmK, k_full, 0, kvh, page * a.page_size);
-          tma_load_3d(dst + 16384, &tmK, k_full, 64, kvh, page * a.page_size);
+          if constexpr (DK > 64) tma_load_3d(dst + 16384, &tmK, k_full, 64, kvh, page * a.page_size);
         }
         if (!mbar_wait(v_empty, ph ^ 1, abort_flag, a.status, 401, j)) { ok = false; break; }
-        mbar_expect_tx(v_full, 32768u);
+        mbar_expect_tx(v_full, 256u * DV);
         for (int p = 0; p < ppb; ++p) {
           const int page = bt[min(blk * ppb + p, last_page)];
           uint8_t* dst = sV + p * page_bytes;
           tma_load_3d(dst, &tmV, v_full, 0, kvh, page * a.page_size);
-          tma_load_3d(dst + 16384, &tmV, v_full, 64, kvh, page * a.page_size);
+          if constexpr (DV > 64) tma_load_3d(dst + 16384, &tmV, v_full, 64, kvh, page * a.page_size);
         }
       }
     }
   } else if (warp == 1) {
     if (lane == 0 && n_blk > 0) {
       constexpr uint32_t idesc_s = make_idesc(128, 128, 1, 1, 0, 0);
-      constexpr uint32_t idesc_o = make_idesc(128, 128, 1, 1, 0, 1);     // B (= V) is MN-major
+      constexpr uint32_t idesc_o = make_idesc(128, DV, 1, 1, 0, 1);     // B (= V) is MN-major
       const uint32_t q_addr = smem_u32(sQ), k_addr = smem_u32(sK), v_addr = smem_u32(sV);
       bool ok = mbar_wait(q_full, 0, abort_flag, a.status, 500);
       for (int j = 0; j < n_blk && ok; ++j) {
@@ -174,7 +207,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         if (!mbar_wait(k_full, ph, abort_flag, a.status, 501, j)) { ok = false; break; }
         tc_fence_after();
 #pragma unroll
-        for (int ks = 0; ks < 8; ++ks) {
+        for (int ks = 0; ks < DK / 16; ++ks) {
           const uint32_t off = (ks >> 2) * 16384 + (ks & 3) * 32;
           mma_f16_ss(tmem_base, make_sdesc_sw128(q_addr + off), make_sdesc_sw128(k_addr + off), idesc_s, ks > 0 ? 1u : 0u);
         }
@@ -204,15 +237,32 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     constexpr float kTau = 8.0f;
     float m = -INFINITY, l = 0.f;
     bool ok = true;
+    const float* bias_row = EXT && a.bias != nullptr ? a.bias + (size_t)(bad_item ? 0 : kvh * G) * a.ld_bias : nullptr;   // the group's first head
+    float* s_bias = reinterpret_cast<float*>(smem + 32768 * 3 + 256);      // EXT: two windows of G x bias_w scores, by block parity
+    const int bias_w = 127 + tpt;
     for (int j = 0; j < n_blk && ok; ++j) {
-      if (!mbar_wait(s_full, j & 1, abort_flag, a.status, 600, j)) { ok = false; break; }
+      const int kv0 = blocks.at(blk_lo + j) * kBN;
+      // distance of the tile's first token to the block's last key: a row's distances are dmin + t_local + 127 - (column)
+      const int dmin = pos0 - kv0 - (kBN - 1);
+      const bool near = EXT && bias_row != nullptr && dmin < a.n_bias - 1;       // else one score for the whole block
+      float* win = s_bias + (size_t)(j & 1) * G * bias_w;
+      bool got = true;
+      if constexpr (EXT) {
+        if (near)
+          for (int h = 0; h < G; ++h)
+            for (int x = q * 32 + lane; x < bias_w; x += 128)
+              win[h * bias_w + x] = bias_row[(size_t)h * a.ld_bias + max(0, min(dmin + x, a.n_bias - 1))];
+      }
+      got = mbar_wait(s_full, j & 1, abort_flag, a.status, 600, j);
+      if constexpr (EXT) got = softmax_bar_and(got);            // the window is complete; all 128 threads leave together
+      if (!got) { ok = false; break; }
       tc_fence_after();
-      const int kv0 = (blk_lo + j) * kBN;
       int hi = kv_len - 1;
       if (a.causal) hi = min(hi, qpos);
       int lo = 0;
       if (a.window > 0) lo = max(0, qpos - a.window + 1);
-      const bool edge = (kv0 + kBN - 1 > hi || kv0 < lo);
+      const int keep = EXT ? a.keep_first : 0;
+      const bool edge = (kv0 + kBN - 1 > hi || (kv0 < lo && !(EXT && kv0 + kBN <= keep)));
       // pass 1: row maximum (the scores are read again in pass 2 instead of being kept in 128 registers)
       float mx = -INFINITY;
 #pragma unroll
@@ -222,10 +272,19 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         tc_wait_ld();
         if (edge) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i) { const int kp = kv0 + c * 32 + i; if (kp > hi || kp < lo) sv[i] = -INFINITY; }
+          for (int i = 0; i < 32; ++i) { const int kp = kv0 + c * 32 + i; if (kp > hi || (kp < lo && !(EXT && kp < keep))) sv[i] = -INFINITY; }
         }
 #pragma unroll
         for (int i = 0; i < 32; ++i) mx = fmaxf(mx, sv[i]);
+      }
+      // with a bias the reference is an upper bound: the largest raw score plus the largest bias of the row's 128 distances
+      float bfar = 0.f;
+      if constexpr (EXT) {
+        if (bias_row != nullptr) {
+          const float* br = bias_row + (size_t)h_local * a.ld_bias + max(0, min(qpos - kv0 - (kBN - 1), a.n_bias - 1));
+          bfar = *br;
+          mx += br[a.n_bias];
+        }
       }
       float alpha = 1.0f;
       const bool grow = mx > m + kTau || (m == -INFINITY && mx > -INFINITY);
@@ -234,7 +293,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       // O holds all products up to block j - 1 (see the MMA thread): rescale it now if some row of this warp moved its reference
       if (j > 0 && __any_sync(0xffffffffu, grow)) {
 #pragma unroll
-        for (int c = 0; c < 4; ++c) {
+        for (int c = 0; c < DV / 32; ++c) {
           uint32_t o[32];
           tmem_ld_x32(tmem_o + lane_off + c * 32, o);
           tc_wait_ld();
@@ -246,6 +305,8 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       // pass 2: P = exp2(S - m) as packed bf16 over the first half of the S columns (chunk c lands on columns that
       // chunks <= c have already been read from)
       float rs = 0.f;
+      const float m_far = EXT && !near ? m_use - bfar : m_use;
+      const float* wrow = EXT ? win + h_local * bias_w + min(t_local, tpt - 1) + 127 : nullptr;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         float sv[32];
@@ -253,12 +314,18 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         tc_wait_ld();
         if (edge) {
 #pragma unroll
-          for (int i = 0; i < 32; ++i) { const int kp = kv0 + c * 32 + i; if (kp > hi || kp < lo) sv[i] = -INFINITY; }
+          for (int i = 0; i < 32; ++i) { const int kp = kv0 + c * 32 + i; if (kp > hi || (kp < lo && !(EXT && kp < keep))) sv[i] = -INFINITY; }
+        }
+        if constexpr (EXT) {
+          if (near) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) sv[i] += wrow[-(c * 32 + i)];
+          }
         }
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float p0 = fast_exp2(sv[2 * i] - m_use), p1 = fast_exp2(sv[2 * i + 1] - m_use);
+          const float p0 = fast_exp2(sv[2 * i] - m_far), p1 = fast_exp2(sv[2 * i + 1] - m_far);
           rs += p0 + p1;
           pk[i] = pack_bf16x2(p0, p1);
         }
@@ -277,7 +344,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       const float inv_l = (l > 0.f) ? 1.0f / l : 0.f;
       uint32_t sf_word = 0;                  // the row's four E8M0 scales (MXFP8 output)
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
+      for (int c = 0; c < DV / 32; ++c) {
         uint32_t o[32];
         if (n_blk > 0) { tmem_ld_x32(tmem_o + lane_off + c * 32, o); tc_wait_ld(); }
         else {
@@ -296,7 +363,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
             e = amax == 0.0f ? 127 : max(1, min(e, 254));
             const float inv = __uint_as_float((uint32_t)(254 - e) << 23) * inv_l;
             sf_word |= (uint32_t)e << (8 * c);
-            uint4* dst = reinterpret_cast<uint4*>(a.out_q + ((size_t)tok * a.hq + head) * kD + c * 32);
+            uint4* dst = reinterpret_cast<uint4*>(a.out_q + ((size_t)tok * a.hq + head) * DV + c * 32);
 #pragma unroll
             for (int v = 0; v < 2; ++v) {
               uint32_t w4[4];
@@ -309,7 +376,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
               dst[v] = make_uint4(w4[0], w4[1], w4[2], w4[3]);
             }
           } else if (a.part_o == nullptr) {
-            uint4* dst = reinterpret_cast<uint4*>(a.out + ((size_t)tok * a.hq + head) * kD + c * 32);
+            uint4* dst = reinterpret_cast<uint4*>(a.out + ((size_t)tok * a.hq + head) * DV + c * 32);
 #pragma unroll
             for (int v = 0; v < 4; ++v) {
               uint4 w;
@@ -320,7 +387,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
               dst[v] = w;
             }
           } else {
-            float4* dst = reinterpret_cast<float4*>(a.part_o + (((size_t)split * a.total_tokens + tok) * a.hq + head) * kD + c * 32);
+            float4* dst = reinterpret_cast<float4*>(a.part_o + (((size_t)split * a.total_tokens + tok) * a.hq + head) * DV + c * 32);
 #pragma unroll
             for (int v = 0; v < 8; ++v)
               dst[v] = make_float4(__uint_as_float(o[v * 4]) * inv_l, __uint_as_float(o[v * 4 + 1]) * inv_l,
@@ -384,15 +451,7 @@ __device__ __forceinline__ float warp_reduce16_sum(const float* v, int lane) {
   return d[0] + __shfl_xor_sync(0xffffffffu, d[0], 1);
 }
 
-// Barrier over the 128 softmax threads (named barrier 1) that also ANDs a predicate: every thread learns whether all of them
-// got through their bounded wait, so they leave the loop together and nobody is left standing at a barrier.
-__device__ __forceinline__ bool softmax_bar_and(bool pred) {
-  uint32_t r;
-  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 q, %1, 0;\n\tbar.red.and.pred p, 1, 128, q;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-               : "=r"(r) : "r"((uint32_t)pred) : "memory");
-  return r != 0;
-}
-
+template <int DK, int DV, bool EXT>
 __global__ void __launch_bounds__(kFdThreads, 2)
 flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const FaArgs a) {
@@ -447,10 +506,12 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   const int qpos = kv_len - 1;
   int first_pos = 0;
   if (a.window > 0) first_pos = max(0, qpos - a.window + 1);
-  int blk_lo = first_pos / kBN, blk_hi = (kv_len > 0) ? (kv_len - 1) / kBN + 1 : 0;
+  FaBlocks blocks = {0, first_pos / kBN, (kv_len > 0) ? (kv_len - 1) / kBN + 1 - first_pos / kBN : 0};
+  if constexpr (EXT) { if (kv_len > 0) blocks = fa_blocks(a, first_pos, qpos); }
+  int blk_lo = 0, blk_hi = blocks.n;
   if (a.num_splits > 1) {
-    const int nb = blk_hi - blk_lo, per = (nb + a.num_splits - 1) / a.num_splits;
-    blk_lo = blk_lo + split * per;
+    const int per = (blocks.n + a.num_splits - 1) / a.num_splits;
+    blk_lo = split * per;
     blk_hi = min(blk_hi, blk_lo + per);
   }
   int n_blk = max(0, blk_hi - blk_lo);
@@ -462,9 +523,9 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 
   if (warp == 0) {
     if (lane == 0 && n_blk > 0) {
-      mbar_expect_tx(q_full, (uint32_t)(2 * 128 * G));
+      mbar_expect_tx(q_full, (uint32_t)(2 * DK * G));
       tma_load_3d(sQ, &tmQ, q_full, 0, kvh * G, tok);
-      tma_load_3d(sQ + 2048, &tmQ, q_full, 64, kvh * G, tok);
+      if constexpr (DK > 64) tma_load_3d(sQ + 2048, &tmQ, q_full, 64, kvh * G, tok);
       const int ppb = kBN / a.page_size;
       const uint32_t page_bytes = (uint32_t)a.page_size * 128;
       const int* bt = a.block_table + (size_t)seq * a.max_pages;
@@ -472,15 +533,15 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       bool ok = true;
       for (int t = 0; t < 2 * n_blk && ok; ++t) {
         const int slot = t % 3; const uint32_t ph = (uint32_t)(t / 3) & 1;
-        const int blk = blk_lo + (t >> 1);
+        const int blk = blocks.at(blk_lo + (t >> 1));
         const CUtensorMap* tm = (t & 1) ? &tmV : &tmK;
         if (!mbar_wait(&t_empty[slot], ph ^ 1, abort_flag, a.status, 410, t)) { ok = false; break; }
-        mbar_expect_tx(&t_full[slot], 32768u);
+        mbar_expect_tx(&t_full[slot], 256u * ((t & 1) ? DV : DK));
         for (int p = 0; p < ppb; ++p) {
           const int page = bt[min(blk * ppb + p, last_page)];
           uint8_t* dst = ring + slot * 32768 + p * page_bytes;
           tma_load_3d(dst, tm, &t_full[slot], 0, kvh, page * a.page_size);
-          tma_load_3d(dst + 16384, tm, &t_full[slot], 64, kvh, page * a.page_size);
+          if (((t & 1) ? DV : DK) > 64) tma_load_3d(dst + 16384, tm, &t_full[slot], 64, kvh, page * a.page_size);
         }
       }
     }
@@ -497,7 +558,7 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         tc_fence_after();
         const uint32_t k_addr = smem_u32(ring + slot * 32768);
 #pragma unroll
-        for (int ks = 0; ks < 8; ++ks)
+        for (int ks = 0; ks < DK / 16; ++ks)
           mma_f16_ss(tmem_base + s * kFdN, make_sdesc_sw128(k_addr + (ks >> 2) * 16384 + (ks & 3) * 32),
                      make_sdesc_sw128(q_addr + (ks >> 2) * 2048 + (ks & 3) * 32), idesc_s, ks > 0 ? 1u : 0u);
         tc_commit(&s_full[s]);
@@ -514,7 +575,7 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         const uint32_t v_addr = smem_u32(ring + vslot * 32768);
         const uint32_t pj = p_addr + (j & 1) * 4096;
 #pragma unroll
-        for (int ks = 0; ks < 8; ++ks)
+        for (int ks = 0; ks < 8; ++ks)                        // DV = 64: rows 64 .. 127 of O are products of whatever the tile's second half holds
           mma_f16_ss(tmem_o, make_sdesc_sw128_mn(v_addr + ks * 2048, 16384), make_sdesc_sw128(pj + (ks >> 2) * 2048 + (ks & 3) * 32),
                      idesc_o, (j > 0 || ks > 0) ? 1u : 0u);
         tc_commit(&o_ready[j & 1]);
@@ -534,16 +595,30 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     bool ok = true, fail_o = false;  // fail_o: a wait for the second MMA ran out; it is put to the vote at the next barrier
     for (int j = 0; j < n_blk && ok; ++j) {
       const int s = j & 1;
+      const int kp = blocks.at(blk_lo + j) * kBN + r;
+      float bv[kFdN];                                    // the position's distance bias, requested before the wait for the scores
+      if constexpr (EXT) {
+        if (a.bias != nullptr && !bad_item) {
+          const float* br = a.bias + (size_t)kvh * G * a.ld_bias + max(0, min(qpos - kp, a.n_bias - 1));
+#pragma unroll
+          for (int h = 0; h < kFdN; ++h) bv[h] = h < G ? br[(size_t)h * a.ld_bias] : 0.f;
+        } else {
+#pragma unroll
+          for (int h = 0; h < kFdN; ++h) bv[h] = 0.f;
+        }
+      }
       const bool got_s = mbar_wait(&s_full[s], (j >> 1) & 1, abort_flag, a.status, 610, j);
       tc_fence_after();
       float sv[kFdN];
       tmem_ld_x16(tmem_base + s * kFdN + lane_off, reinterpret_cast<uint32_t*>(sv));
       tc_wait_ld();
-      const int kp = (blk_lo + j) * kBN + r;
-      const bool live = kp <= qpos && kp >= first_pos;
+      const bool live = kp <= qpos && (kp >= first_pos || (EXT && kp < a.keep_first));
       float* rm = red_max + (j & 1) * 4 * kFdN;
 #pragma unroll
-      for (int h = 0; h < kFdN; ++h) if (!live || h >= G) sv[h] = -INFINITY;
+      for (int h = 0; h < kFdN; ++h) {
+        if constexpr (EXT) sv[h] += bv[h];
+        if (!live || h >= G) sv[h] = -INFINITY;
+      }
       {
         const float v = warp_reduce16_max(sv, lane);            // lane L ends with head L >> 1
         if ((lane & 1) == 0) rm[q * kFdN + (lane >> 1)] = v;
@@ -619,7 +694,7 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       }
 #pragma unroll
       for (int h = 0; h < kFdN; ++h) {
-        if (h >= G) continue;
+        if (h >= G || (DV < 128 && r >= DV)) continue;
         const float inv_l = (l[h] > 0.f) ? 1.0f / l[h] : 0.f;
         const int head = kvh * G + h;
         const float val = __uint_as_float(o[h]) * inv_l;
@@ -632,15 +707,15 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
           e = amax == 0.0f ? 127 : max(1, min(e, 254));
           const float inv = __uint_as_float((uint32_t)(254 - e) << 23);
           __nv_fp8_e4m3 f8(val * inv);
-          a.out_q[(size_t)tok * a.hq * kD + (size_t)head * kD + r] = *reinterpret_cast<uint8_t*>(&f8);
+          a.out_q[(size_t)tok * a.hq * DV + (size_t)head * DV + r] = *reinterpret_cast<uint8_t*>(&f8);
           if (lane == 0) {
             const int blk = head * 4 + q, k_atoms = a.hq;       // 128 features per head = one atom column block per head
             const size_t off = a.out_sf32 ? ((size_t)(tok >> 5) * k_atoms + (blk >> 2)) * 512 + (tok & 31) * 16 + (blk & 3)
                                           : ((size_t)(tok >> 7) * k_atoms + (blk >> 2)) * 512 + (tok & 31) * 16 + ((tok >> 5) & 3) * 4 + (blk & 3);
             a.out_sf[off] = (uint8_t)e;
           }
-        } else if (a.part_o == nullptr) a.out[((size_t)tok * a.hq + head) * kD + r] = __float2bfloat16(val);
-        else a.part_o[(((size_t)split * a.total_tokens + tok) * a.hq + head) * kD + r] = val;
+        } else if (a.part_o == nullptr) a.out[((size_t)tok * a.hq + head) * DV + r] = __float2bfloat16(val);
+        else a.part_o[(((size_t)split * a.total_tokens + tok) * a.hq + head) * DV + r] = val;
         if (a.part_o != nullptr && r == 0)
           a.part_lse[((size_t)split * a.total_tokens + tok) * a.hq + head] = (l[h] > 0.f) ? (m[h] + log2f(l[h])) : -INFINITY;
       }
@@ -658,10 +733,10 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 }
 
 // Merge of split-KV partials: out = sum_s 2^(lse_s - lse_max) O_s / sum_s 2^(lse_s - lse_max).
-// One warp per (token, head); D = 128 -> 4 floats per lane.
+// One warp per (token, head); 4 floats per lane of the d <= 128 features (a multiple of 4; 128 with MXFP8 output).
 __global__ void fa_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse, __nv_bfloat16* __restrict__ out,
                                   float* __restrict__ out_lse, int splits, long rows, uint8_t* __restrict__ out_q, uint8_t* __restrict__ out_sf,
-                                  int out_sf32, int hq) {
+                                  int out_sf32, int hq, int d) {
   pdl_wait();
   pdl_trigger();
   const long w = ((long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
@@ -675,7 +750,7 @@ __global__ void fa_combine_kernel(const float* __restrict__ part_o, const float*
     const float ls = part_lse[(size_t)s * rows + w];
     if (ls == -INFINITY) continue;
     const float wgt = exp2f(ls - mx);
-    const float4 v = *reinterpret_cast<const float4*>(part_o + ((size_t)s * rows + w) * kD + lane * 4);
+    const float4 v = lane * 4 < d ? *reinterpret_cast<const float4*>(part_o + ((size_t)s * rows + w) * d + lane * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
     acc[0] += wgt * v.x; acc[1] += wgt * v.y; acc[2] += wgt * v.z; acc[3] += wgt * v.w;
     den += wgt;
   }
@@ -706,7 +781,7 @@ __global__ void fa_combine_kernel(const float* __restrict__ part_o, const float*
   uint2 o;
   o.x = pack_bf16x2(acc[0] * inv, acc[1] * inv);
   o.y = pack_bf16x2(acc[2] * inv, acc[3] * inv);
-  *reinterpret_cast<uint2*>(out + (size_t)w * kD + lane * 4) = o;
+  if (lane * 4 < d) *reinterpret_cast<uint2*>(out + (size_t)w * d + lane * 4) = o;
   if (out_lse != nullptr && lane == 0) out_lse[w] = den > 0.f ? mx + log2f(den) : -INFINITY;
 }
 
@@ -754,10 +829,10 @@ static int flash_attn_impl(const void* q, const void* k_cache, const void* v_cac
   const int smem = kFaSmem;
   static bool attr_set = false;
   if (!attr_set) {
-    GB_CUDA_OK(cudaFuncSetAttribute(flash_attn_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    GB_CUDA_OK(cudaFuncSetAttribute(flash_attn_kernel<128, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     attr_set = true;
   }
-  launch_k(flash_attn_kernel, n_work, kFaThreads, smem, stream, tmQ, tmK, tmV, a);
+  launch_k(flash_attn_kernel<128, 128, false>, n_work, kFaThreads, smem, stream, tmQ, tmK, tmV, a);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -814,10 +889,10 @@ static int flash_decode_impl(const void* q, const void* k_cache, const void* v_c
   a.out_q = out_q; a.out_sf = out_sf; a.out_sf32 = out_sf32;
   static bool attr_set = false;
   if (!attr_set) {
-    GB_CUDA_OK(cudaFuncSetAttribute(flash_decode_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kFdSmem));
+    GB_CUDA_OK(cudaFuncSetAttribute(flash_decode_kernel<128, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFdSmem));
     attr_set = true;
   }
-  launch_k(flash_decode_kernel, n_work, kFdThreads, kFdSmem, stream, tmQ, tmK, tmV, a);
+  launch_k(flash_decode_kernel<128, 128, false>, n_work, kFdThreads, kFdSmem, stream, tmQ, tmK, tmV, a);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -842,7 +917,7 @@ GB_API int gb_flash_decode_mx(const void* q, const void* k_cache, const void* v_
 GB_API int gb_fa_combine(const float* part_o, const float* part_lse, void* out, float* out_lse, int splits, long rows, cudaStream_t stream) {
   if (rows <= 0) return 0;
   launch_k(fa_combine_kernel, (unsigned)((rows * 32 + 255) / 256), 256, 0, stream, part_o, part_lse, (__nv_bfloat16*)out, out_lse, splits, rows,
-           (uint8_t*)nullptr, (uint8_t*)nullptr, 0, 1);
+           (uint8_t*)nullptr, (uint8_t*)nullptr, 0, 1, kD);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -853,7 +928,82 @@ GB_API int gb_fa_combine_mx(const float* part_o, const float* part_lse, void* ou
   if (rows <= 0) return 0;
   if (hq < 1 || rows % hq) return fail("fa_combine_mx: rows must be tokens * heads%s");
   launch_k(fa_combine_kernel, (unsigned)((rows * 32 + 255) / 256), 256, 0, stream, part_o, part_lse, (__nv_bfloat16*)nullptr, (float*)nullptr, splits,
-           rows, (uint8_t*)out_q, (uint8_t*)out_sf, sf32, hq);
+           rows, (uint8_t*)out_q, (uint8_t*)out_sf, sf32, hq, kD);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// ------------------------------------------------------------------------------------------ masks, distance bias, 64- and 128-wide heads
+template <int DK, int DV>
+static int flash_masked_launch(const void* q, const void* k_cache, const void* v_cache, const FaArgs& a, int n_work, long num_slots, int decode, cudaStream_t stream) {
+  const int G = a.hq / a.hkv, tpt = 128 / G;
+  CUtensorMap tmQ, tmK, tmV;
+  {
+    uint64_t dims[3] = {DK, (uint64_t)a.hq, (uint64_t)a.total_tokens};
+    uint64_t strides[2] = {DK * 2, (uint64_t)a.hq * DK * 2};
+    uint32_t box[3] = {64, (uint32_t)G, decode ? 1u : (uint32_t)tpt};
+    if (make_tmap(&tmQ, q, TM_BF16, 3, dims, strides, box, TM_SW_128)) return -1;
+  }
+  {
+    uint64_t dk[3] = {DK, (uint64_t)a.hkv, (uint64_t)num_slots}, dv[3] = {DV, (uint64_t)a.hkv, (uint64_t)num_slots};
+    uint64_t sk[2] = {DK * 2, (uint64_t)a.hkv * DK * 2}, sv[2] = {DV * 2, (uint64_t)a.hkv * DV * 2};
+    uint32_t box[3] = {64, 1, (uint32_t)a.page_size};
+    if (make_tmap(&tmK, k_cache, TM_BF16, 3, dk, sk, box, TM_SW_128)) return -1;
+    if (make_tmap(&tmV, v_cache, TM_BF16, 3, dv, sv, box, TM_SW_128)) return -1;
+  }
+  if (decode) {
+    static bool attr_set = false;
+    if (!attr_set) {
+      GB_CUDA_OK(cudaFuncSetAttribute(flash_decode_kernel<DK, DV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFdSmem));
+      attr_set = true;
+    }
+    launch_k(flash_decode_kernel<DK, DV, true>, n_work, kFdThreads, kFdSmem, stream, tmQ, tmK, tmV, a);
+  } else {
+    const int smem = kFaSmem + (a.bias != nullptr ? 2 * G * (127 + tpt) * 4 : 0);
+    static int attr_max = 0;
+    if (smem > 227 * 1024) return fail("flash_masked: the bias windows of this group size do not fit shared memory%s");
+    if (smem > attr_max) {
+      GB_CUDA_OK(cudaFuncSetAttribute(flash_attn_kernel<DK, DV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+      attr_max = smem;
+    }
+    launch_k(flash_attn_kernel<DK, DV, true>, n_work, kFaThreads, smem, stream, tmQ, tmK, tmV, a);
+  }
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// gb_flash_attn / gb_flash_decode (decode != 0: one query token per sequence, Hq / Hkv <= 16) with keys of dk and values of dv columns (64 or
+// 128 each), a window that keeps the first `keep_first` positions, and a distance bias (see FaArgs).  q is [T, Hq, dk], out [T, Hq, dv].
+GB_API int gb_flash_masked(const void* q, const void* k_cache, const void* v_cache, void* out, float* part_o, float* part_lse, const int* work, int n_work,
+                           const int* cu_q, const int* kv_len, const int* block_table, int max_pages, int page_size, long num_slots, int total_tokens,
+                           int hq, int hkv, int dk, int dv, int num_splits, int window, int keep_first, const float* bias, int n_bias, int ld_bias,
+                           int decode, void* status, cudaStream_t stream) {
+  if ((dk != 64 && dk != 128) || (dv != 64 && dv != 128)) return fail("flash_masked: heads of 64 or 128 columns%s");
+  if (hq < 1 || hkv < 1 || hq % hkv || hq / hkv > (decode ? kFdN : 128)) return fail("flash_masked: bad head counts%s");
+  if (page_size < 8 || page_size > 128 || (128 % page_size) || (page_size % 8)) return fail("flash_masked: page_size must be 8..128, a multiple of 8 dividing 128%s");
+  if (bias != nullptr && (n_bias < 1 || ld_bias < 2 * n_bias)) return fail("flash_masked: bad bias table%s");
+  if (window < 0 || keep_first < 0 || num_splits < 1) return fail("flash_masked: bad mask%s");
+  if (n_work <= 0) return 0;
+  if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return fail("flash_masked: num_splits > 1 needs partial buffers%s");
+  if (part_o == nullptr && out == nullptr) return fail("flash_masked: no output buffer%s");
+  FaArgs a;
+  memset(&a, 0, sizeof(a));
+  a.work = work; a.cu_q = cu_q; a.kv_len = kv_len; a.block_table = block_table; a.max_pages = max_pages; a.page_size = page_size;
+  a.hq = hq; a.hkv = hkv; a.num_splits = num_splits; a.causal = 1; a.window = window; a.keep_first = window > 0 ? keep_first : 0; a.out = (__nv_bfloat16*)out;
+  a.part_o = part_o; a.part_lse = part_lse; a.total_tokens = total_tokens; a.status = (KernelStatus*)status;
+  a.bias = bias; a.n_bias = n_bias; a.ld_bias = ld_bias;
+  if (dk == 64) return dv == 64 ? flash_masked_launch<64, 64>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream)
+                                : flash_masked_launch<64, 128>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream);
+  return dv == 64 ? flash_masked_launch<128, 64>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream)
+                  : flash_masked_launch<128, 128>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream);
+}
+
+// gb_fa_combine for heads of `head_dim` (64 or 128) features.
+GB_API int gb_fa_combine_dim(const float* part_o, const float* part_lse, void* out, int splits, long rows, int head_dim, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (head_dim < 4 || head_dim > 128 || head_dim % 4) return fail("fa_combine_dim: head_dim must be a multiple of 4 up to 128%s");
+  launch_k(fa_combine_kernel, (unsigned)((rows * 32 + 255) / 256), 256, 0, stream, part_o, part_lse, (__nv_bfloat16*)out, (float*)nullptr, splits, rows,
+           (uint8_t*)nullptr, (uint8_t*)nullptr, 0, 1, head_dim);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }

@@ -84,6 +84,7 @@ struct GemmArgs {
   int dual_raw;  // DUAL without the activation: the second accumulator is the row block up_row_offset further down the same matrix
   int w_tiled;
   int act;       // activation of the gate half of a DUAL launch: 0 = SiLU, 1 = the tanh form of GELU
+  int silu_rows; // plain launches: SiLU on the output features below this (the q / k / v part of a linear-attention projection)
 };
 
 // k-steps whose MXFP8 scale atoms are fetched by one bulk copy (2 for the widest tile, whose stages are short of room)
@@ -399,6 +400,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       const uint32_t tacc = tmem_base + acc * ACC_COLS + ((uint32_t)(q * 32) << 16);
       const int n = t.n0 + row;
       const bool n_ok = n < args.n_out;
+      const bool row_act = !DUAL && n < args.silu_rows;
       const float bias = (args.bias != nullptr && n_ok && (args.partial_stride == 0 || t.ks == 0)) ? args.bias[n] : 0.0f;
       // Everything after the accumulators are in registers: activation, bias, then one of the store forms.
       auto finish_chunk = [&](int c, const uint32_t* r0, const uint32_t* r1) {
@@ -408,6 +410,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           float v = __uint_as_float(r0[j]);
           if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
           v += bias;
+          if (row_act) v = silu_f(v);
           const bool live = xr < t.valid;
           const int x_row = t.x_row0 + xr;
           if (QUANT_OUT) {
@@ -542,7 +545,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         __nv_bfloat16* o16 = (__nv_bfloat16*)obase + part_off + orow0 * args.ldo + n;
         float* o32 = (float*)obase + part_off + orow0 * args.ldo + n;
         if constexpr (NACC == 1 && !DUAL) {
-          if (!args.out_f32) {
+          if (!args.out_f32 && args.silu_rows == 0) {
             // One accumulator buffer (the widest tile with its scale columns fills TMEM): pull the whole row into registers
             // as packed bf16, hand the buffer back to the MMA thread, and only then store, so that the stores overlap the
             // next tile's MMAs.
@@ -612,6 +615,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               float v = __uint_as_float(r0[j]);
               if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
               v += bias;
+              if (row_act) v = silu_f(v);
               if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
               else o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v);
             }
@@ -621,6 +625,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               float v = __uint_as_float(r0[j]);
               if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
               v += bias;
+              if (row_act) v = silu_f(v);
               if (c + j < t.valid) {
                 if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
                 else o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v);
@@ -734,6 +739,7 @@ struct GemmExtras {
   int epoch_self_tick;
   size_t sfa_bytes, sfb_bytes, out_bytes, out_sf_bytes;
   long partial_stride;       // > 0 with splits > 1: every K split stores its fp32 partial into its own slab of `out` (the consumer sums them)
+  int silu_rows;             // SiLU on the output features below this (launches that are neither DUAL nor K-split)
 };
 
 // Flags of gb_gemm.
@@ -800,6 +806,8 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
     a.peer_region_rows = ex->peer_region_rows; a.peer_rank = ex->peer_rank; a.signal_n = ex->signal_n; a.done_ctr = ex->done_ctr;
     a.amax_val = ex->amax_val; a.amax_idx = ex->amax_idx; a.peer_bcast = ex->peer_bcast; a.epoch_self_tick = ex->epoch_self_tick;
     a.sfa_bytes = ex->sfa_bytes; a.sfb_bytes = ex->sfb_bytes; a.out_bytes = ex->out_bytes; a.out_sf_bytes = ex->out_sf_bytes;
+    if (ex->silu_rows > 0 && (dual || ex->splits > 1)) return fail("gemm: silu_rows needs a plain launch%s");
+    a.silu_rows = ex->silu_rows;
     if (ex->splits > 1 && num_groups == 0 && ex->partial_stride > 0) {
       if (!(flags & GEMM_OUT_F32) || qo) return fail("gemm: split-K partials need a plain fp32 output%s");
       const int kb_elems = mx ? 128 : 64;

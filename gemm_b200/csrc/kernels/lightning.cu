@@ -10,7 +10,7 @@
 namespace gb {
 
 struct LightningArgs {
-  const void* proj;             // [n_part][tokens, ld]: columns [q heads x dim | k heads x dim | v heads x vdim | ...], pre-activation
+  const void* proj;             // [n_part][tokens, ld]: columns [q heads x dim | k heads x dim | v heads x vdim | ...]
   int n_part; long part_stride; int ld;
   const float* decay;           // [heads]
   float* state;                 // [slots, heads, dim, vdim]
@@ -18,6 +18,7 @@ struct LightningArgs {
   const int* cu_q; const int* seq_slots;
   float* out; int ld_out;       // [tokens, heads * vdim] f32
   int heads, dim, vdim;
+  int raw;                      // != 0: the columns are pre-activations (one bf16 slab of activated columns otherwise)
 };
 
 __device__ __forceinline__ float silu_exact(float x) { return x / (1.0f + expf(-x)); }
@@ -29,7 +30,7 @@ __device__ __forceinline__ float proj_silu(const LightningArgs& a, size_t tok, i
   const TI* p = (const TI*)a.proj + tok * a.ld + col;
   float s = ldp(p);
   for (int i = 1; i < a.n_part; ++i) s += ldp(p + (size_t)i * a.part_stride);
-  return silu_exact(s);
+  return a.raw ? silu_exact(s) : s;
 }
 
 template <typename TI, int VEC, int R>             // dim <= 8 * R
@@ -129,14 +130,15 @@ static int lightning_step_launch(const LightningArgs& a, int n_seqs, cudaStream_
 
 using namespace gb;
 
-GB_API int gb_lightning_step(const void* proj, int proj_f32, int n_part, long part_stride, int ld, const float* decay, float* state, int n_slots,
+// raw != 0: SiLU is applied here; else the columns carry it already.
+GB_API int gb_lightning_step(const void* proj, int proj_f32, int raw, int n_part, long part_stride, int ld, const float* decay, float* state, int n_slots,
                              const int* cu_q, const int* seq_slots, float* out, int ld_out, int heads, int dim, int vdim, int n_seqs, cudaStream_t stream) {
   if (n_seqs <= 0) return 0;
   if (heads < 1 || dim < 1 || vdim < 1 || n_part < 1 || ld < 2 * heads * dim + heads * vdim || ld_out < heads * vdim) return fail("lightning: bad sizes%s");
   if (dim > 512) return fail("lightning: a key dimension of at most 512%s");
   if (n_seqs > 65535) return fail("lightning: too many sequences%s");
   LightningArgs a;
-  a.proj = proj; a.n_part = n_part; a.part_stride = part_stride; a.ld = ld; a.decay = decay; a.state = state; a.n_slots = n_slots; a.cu_q = cu_q;
+  a.raw = raw; a.proj = proj; a.n_part = n_part; a.part_stride = part_stride; a.ld = ld; a.decay = decay; a.state = state; a.n_slots = n_slots; a.cu_q = cu_q;
   a.seq_slots = seq_slots; a.out = out; a.ld_out = ld_out; a.heads = heads; a.dim = dim; a.vdim = vdim;
   return proj_f32 ? lightning_step_launch<float>(a, n_seqs, stream) : lightning_step_launch<__nv_bfloat16>(a, n_seqs, stream);
 }

@@ -331,12 +331,12 @@ def apply_linear_stream(lw: LinearWeight, x: torch.Tensor):
     return gemm.linear(x, lw.w, bias=lw.bias, out_dtype=torch.float32, w_tiled=lw.tiled)
 
 
-def apply_linear_mixer(lw: LinearWeight, x: torch.Tensor):
+def apply_linear_mixer(lw: LinearWeight, x: torch.Tensor, silu_rows: int = 0):
     """The input projection of a mixer: as ``apply_linear_stream`` for decode-sized batches (the mixer's kernels add the partial sums), bf16
-    rows for prefill-sized ones."""
+    rows for prefill-sized ones, with SiLU on the first ``silu_rows`` features.  Returns ``(result, whether SiLU was applied)``."""
     if lw.fmt == "f32" or x.shape[0] <= 64:
-        return apply_linear_stream(lw, x)
-    return gemm.linear(x, lw.w, bias=lw.bias, w_tiled=lw.tiled)
+        return apply_linear_stream(lw, x), False
+    return gemm.linear(x, lw.w, bias=lw.bias, w_tiled=lw.tiled, silu_rows=silu_rows), silu_rows > 0
 
 
 def expert_gate_up_mx(x_q: torch.Tensor, x_sf: torch.Tensor, w13: LinearWeight, n_w_groups: int, seg_start: torch.Tensor,
@@ -489,7 +489,7 @@ class Transformer:
         """Attention of a layer described by ``LayerSpec``: biased projection -> Q / K unit norm + cache store -> windowed attention with
         kept first tokens and distance bias -> output projection.  ``li`` is the run, which has its own cache."""
         kc, vc = self.kv.k[li], self.kv.v[li]
-        qkv = apply_linear_mixer(lw.wqkv, h)
+        qkv, _ = apply_linear_mixer(lw.wqkv, h)
         q = stream.qk_unit(qkv, fb.slots, kc, vc, sp.n_heads, sp.n_kv_heads, sp.head_dim, sp.v_dim, self.cfg.rms_eps,
                            (sp.scale or sp.head_dim ** -0.5) * att.LOG2E, unit=sp.qk_unit)
         key = (sp.n_heads, sp.n_kv_heads, sp.span)
@@ -503,8 +503,9 @@ class Transformer:
 
     def lightning_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
         """Lightning attention: projection -> SiLU + decayed recurrence -> RMSNorm over all heads * sigmoid(gate) -> output projection."""
-        proj = apply_linear_mixer(lw.lin.w_in, h)
-        o = lightning.lightning(proj, lw.lin.decay, self.kv.rec[li], fb.cu_q, fb.seq_slots, sp.n_heads, sp.head_dim, sp.v_dim)
+        proj, activated = apply_linear_mixer(lw.lin.w_in, h, silu_rows=2 * sp.q_dim + sp.n_heads * sp.v_dim)
+        o = lightning.lightning(proj, lw.lin.decay, self.kv.rec[li], fb.cu_q, fb.seq_slots, sp.n_heads, sp.head_dim, sp.v_dim, activated,
+                                max(fb.q_lens) if fb.q_lens else 1)
         y = stream.gated_norm(o, proj, 2 * sp.q_dim + sp.n_heads * sp.v_dim, lw.lin.norm, self.cfg.rms_eps, self.act_dtype)
         return apply_linear_stream(lw.lin.w_out, y)
 

@@ -245,7 +245,7 @@ class LayerWeights:
     sh_down: Optional[LinearWeight] = None
     sh_gate: Optional[torch.Tensor] = None        # bf16 [1, H]: sigmoid gate of the shared expert (absent = ungated)
     lin: Optional[LightningWeights] = None        # lightning-attention layer (then wqkv / wo are None)
-    rel_bias: Optional[torch.Tensor] = None       # f32 [heads, N + 1] distance bias (ops.attention.distance_bias_table)
+    rel_bias: Optional[torch.Tensor] = None       # f32 [heads, 2 N] distance bias (ops.attention.distance_bias_table)
 
     def linears(self) -> List[LinearWeight]:
         """Every projection matrix of the layer."""

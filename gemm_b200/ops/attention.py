@@ -330,9 +330,8 @@ def distance_bucket(n: int, buckets: int, max_distance: float) -> int:
 
 
 def distance_bias_table(rel: torch.Tensor, max_distance: float) -> torch.Tensor:
-    """``rel [buckets, heads]`` -> f32 ``[heads, N + 1]``: the bias of every distance 0 .. N - 1 times log2(e) (larger distances equal the
-    last of them), and in column N the largest bias of the head (an upper bound the flash kernels use as part of their reference
-    maximum)."""
+    """``rel [buckets, heads]`` -> f32 ``[heads, 2 N]``: the bias of every distance 0 .. N - 1 times log2(e) (larger distances equal the last
+    of them), then, per distance n, the largest bias of the distances n .. n + 127 (the flash kernels' bound on a block's biases)."""
     buckets, heads = rel.shape
     idx, n = [], 0
     while True:
@@ -341,8 +340,9 @@ def distance_bias_table(rel: torch.Tensor, max_distance: float) -> torch.Tensor:
         if b == buckets - 1:
             break
         n += 1
-    t = rel.double()[torch.tensor(idx)].t() * LOG2E                   # [heads, N]
-    return torch.cat([t, t.max(dim=1, keepdim=True).values], dim=1).float().contiguous()
+    t = (rel.double()[torch.tensor(idx)].t() * LOG2E).float()         # [heads, N]
+    ahead = torch.cat([t, t[:, -1:].expand(heads, 127)], dim=1)
+    return torch.cat([t, ahead.unfold(1, 128, 1).max(dim=2).values], dim=1).contiguous()
 
 
 def flash_head_dims(dk: int, dv: int):
@@ -376,7 +376,7 @@ def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_si
         sc = torch.einsum("qhd,khd->hqk", q[q0:q1].float(), k)
         dist = torch.arange(kl - ql, kl).unsqueeze(1) - torch.arange(kl).unsqueeze(0)
         if bias is not None:
-            n = bias.shape[1] - 1
+            n = bias.shape[1] // 2
             sc = sc + bias[:, dist.clamp(0, n - 1)]
         see = dist >= 0
         if window > 0:
@@ -398,10 +398,25 @@ def attention_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     if not q.is_cuda:
         return attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window, keep_first, bias)
     out = torch.empty(t, hq, dv, dtype=k_cache.dtype, device=q.device)
-    n_bias, ld_bias = (bias.shape[1] - 1, bias.stride(0)) if bias is not None else (0, 0)
-    stream = _c(torch.cuda.current_stream().cuda_stream)
-    rc = _native.cuda().gb_attn_any(_p(q), _p(k_cache), _p(v_cache), _p(out), _i(int(k_cache.dtype == torch.float32)), _p(cu_q), _p(kv_len),
-                                    _p(block_table), _i(block_table.shape[1]), _i(page_size), _i(cu_q.numel() - 1), _l(k_cache.shape[0]), _i(t), _i(hq),
-                                    _i(hkv), _i(dk), _i(dv), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), stream)
+    n_bias, ld_bias = (bias.shape[1] // 2, bias.stride(0)) if bias is not None else (0, 0)
+    lib, stream = _native.cuda(), _c(torch.cuda.current_stream().cuda_stream)
+    if plan is not None and k_cache.dtype == torch.bfloat16 and dk in (64, 128) and dv in (64, 128) and page_size % 8 == 0 and 128 % page_size == 0 \
+            and hq // hkv <= 128:
+        work, splits = plan
+        part_o = part_lse = None
+        if splits > 1:
+            part_o = torch.empty(splits, t, hq, dv, dtype=torch.float32, device=q.device)
+            part_lse = torch.empty(splits, t, hq, dtype=torch.float32, device=q.device)
+        rc = lib.gb_flash_masked(_p(q), _p(k_cache), _p(v_cache), _p(out), _p(part_o), _p(part_lse), _p(work), _i(work.shape[0]), _p(cu_q), _p(kv_len),
+                                 _p(block_table), _i(block_table.shape[1]), _i(page_size), _l(k_cache.shape[0]), _i(t), _i(hq), _i(hkv), _i(dk), _i(dv),
+                                 _i(splits), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), _i(int(decode and hq // hkv <= 16)),
+                                 _c(_native.status_ptr()), stream)
+        _native.check(rc, "gb_flash_masked")
+        if splits > 1:
+            _native.check(lib.gb_fa_combine_dim(_p(part_o), _p(part_lse), _p(out), _i(splits), _l(t * hq), _i(dv), stream), "gb_fa_combine_dim")
+        return out
+    rc = lib.gb_attn_any(_p(q), _p(k_cache), _p(v_cache), _p(out), _i(int(k_cache.dtype == torch.float32)), _p(cu_q), _p(kv_len),
+                         _p(block_table), _i(block_table.shape[1]), _i(page_size), _i(cu_q.numel() - 1), _l(k_cache.shape[0]), _i(t), _i(hq),
+                         _i(hkv), _i(dk), _i(dv), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), stream)
     _native.check(rc, "gb_attn_any")
     return out

@@ -29,7 +29,7 @@ class GemmExtras(ctypes.Structure):
                 ("sk_ws", ctypes.c_void_p), ("sk_ctr", ctypes.c_void_p), ("amax_val", ctypes.c_void_p), ("amax_idx", ctypes.c_void_p),
                 ("sk_ws_bytes", ctypes.c_long), ("sk_ctr_count", ctypes.c_long), ("peer_bcast", ctypes.c_int), ("epoch_self_tick", ctypes.c_int),
                 ("sfa_bytes", ctypes.c_size_t), ("sfb_bytes", ctypes.c_size_t), ("out_bytes", ctypes.c_size_t), ("out_sf_bytes", ctypes.c_size_t),
-                ("partial_stride", ctypes.c_long)]
+                ("partial_stride", ctypes.c_long), ("silu_rows", ctypes.c_int)]
 
 
 _SK_WS_BYTES = 64 << 20
@@ -132,22 +132,28 @@ def _launch(w, x, out, n_out, k, m_tok, ldw, ldx, ldo, flags, tn, num_groups=0, 
 
 # --------------------------------------------------------------------------------------------- bf16
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
-           out_dtype=torch.bfloat16, tn: Optional[int] = None, split_k: bool = False, w_tiled: bool = False) -> torch.Tensor:
-    """``x [M, K] @ w[N, K]^T`` (bf16 operands, fp32 accumulate).  ``w_tiled``: ``w`` is in ``mxfp8.tile_weight`` layout."""
+           out_dtype=torch.bfloat16, tn: Optional[int] = None, split_k: bool = False, w_tiled: bool = False,
+           silu_rows: int = 0) -> torch.Tensor:
+    """``x [M, K] @ w[N, K]^T`` (bf16 operands, fp32 accumulate).  ``w_tiled``: ``w`` is in ``mxfp8.tile_weight`` layout.  ``silu_rows``: SiLU on
+    that many leading output features, in the epilogue."""
     m, k = x.shape
     n = w.shape[0]
     if not x.is_cuda:
         y = x.float() @ (mxfp8.untile_weight(w) if w_tiled else w).float().t()
         if bias is not None:
             y = y + bias.float()
+        if silu_rows:
+            y = torch.cat([torch.nn.functional.silu(y[:, :silu_rows]), y[:, silu_rows:]], dim=1)
         return y.to(out_dtype)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.stride(1) == 1 and w.stride(1) == 1
     if out is None:
         out = torch.empty(m, n, dtype=out_dtype, device=x.device)
     flags = (GEMM_OUT_F32 if out.dtype == torch.float32 else 0) | (GEMM_W_TILED if w_tiled else 0)
     tn = tn or pick_tn(m)
-    _launch(w, x, out, n, k, m, w.stride(0), x.stride(0), out.stride(0), flags, tn, bias=bias,
-            extras=_splitk_extras(n, m, k, tn, False, x.device, split_k))
+    ex = _splitk_extras(n, m, k, tn, False, x.device, split_k) if not silu_rows else GemmExtras()
+    if silu_rows:
+        ex.silu_rows = silu_rows
+    _launch(w, x, out, n, k, m, w.stride(0), x.stride(0), out.stride(0), flags, tn, bias=bias, extras=ex)
     return out
 
 

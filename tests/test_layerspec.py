@@ -1,0 +1,294 @@
+"""Models described layer by layer, end to end: checkpoint -> loader -> paged cache and state slots -> engine step, against the plain
+reference of ``layerspec_oracle`` (float64).  Every test runs on the CPU references of the ops and, on a GPU box, on the kernels."""
+import os
+import subprocess
+import sys
+
+import numpy as np
+import pytest
+import torch
+
+from . import layerspec_cases as C
+from . import layerspec_oracle as O
+from gemm_b200.models import loader
+from gemm_b200.models.config import LayerSpec, LoopSpec, ModelConfig
+from gemm_b200.serve.engine import Engine, SamplingParams
+from gemm_b200.serve.llm import LLM
+from gemm_b200.serve.replay import Replay
+
+DEVICES = ["cpu", pytest.param("cuda", marks=pytest.mark.gpu)]
+FORMATS = ["f32", "bf16"]
+TOL = {"f32": 5e-5, "bf16": 4e-2}
+PAGE = 64
+_models, _logits = {}, {}
+
+
+@pytest.fixture(scope="module")
+def folder(tmp_path_factory):
+    return tmp_path_factory.mktemp("layerspec")
+
+
+def get_model(name):
+    if name not in _models:
+        _models[name] = C.make_model(name)
+    return _models[name]
+
+
+def want(name, n, seed):
+    """Tokens and the reference's logits of a sequence (computed once)."""
+    key = (name, n, seed)
+    if key not in _logits:
+        toks = C.tokens(get_model(name), n, seed)
+        _logits[key] = (toks, O.forward(get_model(name), toks))
+    return _logits[key]
+
+
+def weights(folder, name, fmt, device):
+    path = os.path.join(str(folder), name)
+    if not os.path.exists(path):
+        C.save_model(get_model(name), path)
+    return loader.load_safetensors(path, fmt, device)
+
+
+def make_llm(folder, name, fmt, device, pages=12, slots=4, page=PAGE, **kw):
+    return LLM(weights(folder, name, fmt, device), None, max_running=slots, num_pages=pages, page_size=page, **kw)
+
+
+def check_ok(device):
+    if device == "cuda":
+        from gemm_b200 import _native
+        _native.assert_status_ok()
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("fmt", FORMATS)
+@pytest.mark.parametrize("name", sorted(C.CASES))
+def test_whole_prompt(folder, name, fmt, device):
+    toks, ref = want(name, 203, 0)
+    got = C.replay_one(Replay(make_llm(folder, name, fmt, device)), toks, [203])
+    check_ok(device)
+    assert C.err(got, ref).max() < TOL[fmt]
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("fmt", FORMATS)
+@pytest.mark.parametrize("sizes", [[2], [64], [65, 1, 63, 2, 3], [130, 7]])
+def test_portions(folder, sizes, fmt, device):
+    for name in ("mixed", "wide"):
+        toks, ref = want(name, 203, 0)
+        got = C.replay_one(Replay(make_llm(folder, name, fmt, device)), toks, C.cuts(203, sizes))
+        check_ok(device)
+        assert C.err(got, ref).max() < TOL[fmt]
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("fmt", FORMATS)
+@pytest.mark.parametrize("name", sorted(C.CASES))
+def test_token_by_token(folder, name, fmt, device):
+    """Prefill and decoding agree; decoding goes on past every window and across pages."""
+    toks, ref = want(name, 203, 0)
+    rep = Replay(make_llm(folder, name, fmt, device))
+    got = C.replay_one(rep, toks, [20] + [1] * 183)
+    check_ok(device)
+    assert C.err(got, ref).max() < TOL[fmt]
+    first = C.replay_one(rep, toks[:9], [1] * 9)                     # the first tokens of a sequence, one by one
+    assert C.err(first, ref[:9]).max() < TOL[fmt]
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("fmt", FORMATS)
+@pytest.mark.parametrize("name", ["mixed", "wide", "odd"])
+def test_batches_of_unequal_requests(folder, name, fmt, device):
+    """Requests of unequal lengths in one batch, portions beside single tokens, one left out for some steps; the pool holds little more than
+    what is live, so pages and slots are used again by later requests."""
+    lens = {"a": 150, "b": 70, "c": 1, "d": 203, "e": 97, "f": 130}
+    seq = {k: want(name, n, 0 if n == 203 else i + 1) for i, (k, n) in enumerate(lens.items())}
+    llm = make_llm(folder, name, fmt, device, pages=10)
+    rep = Replay(llm)
+    at = {k: 0 for k in lens}
+    got = {k: [] for k in lens}
+
+    def step(**portions):
+        entries, end = [], []
+        for k, n in portions.items():
+            n = min(n, lens[k] - at[k])
+            entries.append({"id": k, "tokens": seq[k][0][at[k]: at[k] + n], "want": list(range(n))})
+        out = rep.step(entries, [k for k, n in portions.items() if at[k] + n >= lens[k]])
+        p = 0
+        for e in entries:
+            n = len(e["tokens"])
+            got[e["id"]].append(out[p: p + n])
+            at[e["id"]] += n
+            p += n
+
+    step(a=90, b=3)
+    step(a=1, b=40, c=1)                       # c comes and goes
+    for _ in range(5):
+        step(a=1, b=1, d=2)
+    step(a=30, d=100)                          # b is left out
+    step(b=70, d=1)
+    step(a=200, d=1)                           # a ends: its pages and slot go to e and f
+    step(d=60, e=50, f=1)
+    for _ in range(12):
+        step(d=1, e=1, f=2)
+    step(d=200, e=200, f=105)
+    assert llm.blocks.num_free == 10 and sorted(llm._free_slots) == [0, 1, 2, 3] and not rep.live
+    check_ok(device)
+    for k in lens:
+        assert at[k] == lens[k]
+        assert C.err(torch.cat(got[k]), seq[k][1]).max() < TOL[fmt], k
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("name", ["mixed", "wide"])
+def test_page_sizes_do_not_matter(folder, name, device):
+    toks, ref = want(name, 203, 0)
+    for page in (16, 128, 24):                 # 24 is no page size of the flash kernels
+        got = C.replay_one(Replay(make_llm(folder, name, "bf16", device, pages=30, page=page)), toks, [101, 1, 1, 100])
+        assert C.err(got, ref).max() < TOL["bf16"]
+    check_ok(device)
+
+
+@pytest.mark.parametrize("device", DEVICES)
+def test_stream_after_every_layer_run(folder, device):
+    toks = C.tokens(get_model("mixed"), 75, 5)
+    cap = []
+    O.forward(get_model("mixed"), toks, capture=cap)
+    llm = make_llm(folder, "mixed", "f32", device)
+    llm.model.snapshot_layers = range(len(cap))
+    assert len(llm.model.runs) == len(cap) == 2 * 3 + 2
+    Replay(llm).step([{"id": "x", "tokens": toks, "want": [74]}])
+    for li, x in enumerate(cap):
+        d = llm.model.snapshots[li].double().cpu() - x
+        assert d.abs().max() < 1e-4 * x.abs().max(), li
+
+
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("fmt", FORMATS)
+@pytest.mark.parametrize("name", ["mixed", "wide"])
+def test_greedy_generation_through_the_scheduler(folder, name, fmt, device):
+    """``LLM.generate`` (continuous batching, chunked prompts, a pool too small for all at once) and the static-batch engine (CUDA graph on a
+    GPU): each token is the reference's best, or within rounding of it."""
+    model = get_model(name)
+    prompts = [C.tokens(model, n, 20 + n) for n in (5, 90, 131)]
+    new = 12
+    llm = make_llm(folder, name, fmt, device, pages=6, slots=3, max_batch_tokens=48)
+    outs = llm.generate(prompts, SamplingParams(max_new_tokens=new))
+    eng = Engine(weights(folder, name, fmt, device), max_batch=3, max_seq_len=256, page_size=PAGE, max_prefill_tokens=100)
+    outs2 = eng.generate(prompts, SamplingParams(max_new_tokens=new))
+    check_ok(device)
+    for res in (outs, outs2):
+        for p, o in zip(prompts, res):
+            assert len(o) == new
+            ref = O.forward(model, p + o)[len(p) - 1: -1]
+            scale = (ref - ref.mean(-1, keepdim=True)).pow(2).mean().sqrt()
+            gap = ref.max(-1).values - ref[torch.arange(new), torch.tensor(o)]
+            assert (gap / scale).max() < 3 * TOL[fmt]
+    assert llm.blocks.num_free == 6
+
+
+@pytest.mark.parametrize("device", DEVICES)
+def test_sampling_is_served(folder, device):
+    llm = make_llm(folder, "mixed", "bf16", device)
+    sp = SamplingParams(max_new_tokens=6, temperature=0.8, top_k=20, top_p=0.9, seed=3)
+    a = llm.generate([C.tokens(get_model("mixed"), 30, 9)], sp)
+    assert len(a[0]) == 6 and all(0 <= t < 211 for t in a[0])
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("fmt,dtype", [("bf16", "bfloat16"), ("f32", "float32")])
+def test_trace_program(folder, tmp_path, fmt, dtype):
+    """``bin/trace_run``: steps on standard input, one answer line each, the wanted logits in files."""
+    import json
+    weights(folder, "wide", fmt, "cpu")
+    toks, ref = want("wide", 203, 0)
+    steps, at = [], 0
+    for i, n in enumerate([100, 2, 1, 100]):
+        steps.append({"step": i, "entries": [{"id": "q", "tokens": toks[at: at + n], "want": [] if i == 1 else [0, n - 1]}], "end": ["q"] if i == 3 else []})
+        at += n
+    prog = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "bin", "trace_run")
+    r = subprocess.run([sys.executable, prog, "--model", os.path.join(str(folder), "wide"), "--dtype", dtype, "--out", str(tmp_path), "--max-tokens", "256"],
+                       input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr
+    assert [x for x in r.stdout.splitlines() if x.startswith("done")] == [f"done {i}" for i in range(4)]
+    assert not os.path.exists(tmp_path / "1.f32")
+    for i, rows in ((0, [0, 99]), (2, [102, 102]), (3, [103, 202])):
+        got = torch.from_numpy(np.fromfile(tmp_path / f"{i}.f32", dtype="<f4")).reshape(2, -1)
+        assert C.err(got, ref[rows]).max() < TOL[fmt]
+
+
+# ------------------------------------------------------------------------------------------ configuration, loading, command line
+def test_config_reads_every_size(folder):
+    w = weights(folder, "mixed", "f32", "cpu")
+    cfg = w.cfg
+    assert cfg.arch == "zogavik" and cfg.vocab == 211 and cfg.hidden == 136 and cfg.loop == LoopSpec(1, 3, 3) and cfg.logit_scale == 0.7
+    att, lin = cfg.layer_specs[1], cfg.layer_specs[2]
+    assert (att.mixer, att.n_heads, att.n_kv_heads, att.head_dim, att.v_dim, att.window, att.keep_first, att.rel_buckets, att.rel_max, att.ffn) == \
+        ("attention", 4, 2, 40, 56, 33, 5, 12, 90, 144)
+    assert (lin.mixer, lin.n_heads, lin.head_dim, lin.v_dim, lin.ffn, lin.decay) == ("lightning", 2, 72, 24, 0, [0.9, 0.5])
+    assert [r.layer for r in cfg.layer_runs()] == [0, 1, 2, 1, 2, 1, 2, 3] and [r.step for r in cfg.layer_runs()] == [-1, 0, -1, 1, -1, 2, -1, -1]
+    assert ModelConfig(**{**cfg.__dict__}).layer_specs == cfg.layer_specs
+
+
+def test_saved_checkpoints_load_again(tmp_path):
+    from gemm_b200.models.config import get_config
+    from gemm_b200.models.weights import RandomSource, build_weights
+    cfg = get_config("tiny-zogavik")
+    loader.save_hf_checkpoint(cfg, RandomSource(cfg, seed=4, device="cpu"), str(tmp_path))
+    a, b = loader.load_safetensors(str(tmp_path), "bf16", "cpu"), build_weights(cfg, RandomSource(cfg, seed=4, device="cpu"), "bf16", "cpu")
+    assert a.cfg.layer_specs == b.cfg.layer_specs and a.cfg.loop == b.cfg.loop
+    assert torch.equal(a.embed, b.embed) and torch.equal(a.loop_step, b.loop_step)
+    for x, y in zip(a.layers, b.layers):
+        assert all(torch.equal(p.w, q.w) for p, q in zip(x.linears(), y.linears()))
+
+
+@pytest.mark.parametrize("change,word", [
+    (lambda c: c["layers"][0].update(type="spiral"), "spiral"),
+    (lambda c: c["layers"][0]["mlp"].update(kind="experts"), "experts"),
+    (lambda c: c.update(architecture="Unheard"), "Unheard"),
+    (lambda c: c["layers"][0]["mixer"].update(decay=[0.5]), "decay"),
+    (lambda c: c["loop"].update(stop=9), "loop"),
+])
+def test_unknown_parts_are_refused(tmp_path, change, word):
+    import copy
+    m = copy.deepcopy(get_model("mixed"))
+    change(m["config"])
+    C.save_model(m, str(tmp_path))
+    with pytest.raises(ValueError, match=word):
+        loader.load_safetensors(str(tmp_path), "f32", "cpu").cfg.layer_runs()
+
+
+def test_a_missing_or_misshapen_tensor_is_named(tmp_path):
+    m = C.make_model("mixed")
+    del m["t"]["l2.mix.g"]
+    C.save_model(m, str(tmp_path / "a"))
+    with pytest.raises(ValueError, match="l2.mix.g"):
+        loader.load_safetensors(str(tmp_path / "a"), "f32", "cpu")
+    m = C.make_model("mixed")
+    m["t"]["l1.mlp.up"] = m["t"]["l1.mlp.up"][:-1]
+    C.save_model(m, str(tmp_path / "b"))
+    with pytest.raises(ValueError, match="l1.mlp.up"):
+        loader.load_safetensors(str(tmp_path / "b"), "f32", "cpu")
+
+
+@pytest.mark.parametrize("device", DEVICES)
+def test_command_line(folder, device):
+    model = get_model("mixed")
+    weights(folder, "mixed", "f32", "cpu")
+    p = C.tokens(model, 40, 2)
+    r = subprocess.run([sys.executable, "-m", "gemm_b200", "generate", "--model", os.path.join(str(folder), "mixed"), "--format", "f32", "--device", device,
+                        "--ids", "--prompt", " ".join(map(str, p)), "--max-new-tokens", "4", "--pages", "8", "--page-size", "64"],
+                       capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr
+    out = [int(x) for x in r.stdout.replace(",", " ").replace("[", " ").replace("]", " ").split() if x.isdigit()][-4:]
+    ids = list(p)
+    for t in out:
+        assert int(O.forward(model, ids)[-1].argmax()) == t
+        ids.append(t)
+
+
+def test_recurrent_models_refuse_speculation(folder):
+    from gemm_b200.serve.speculative import NgramDrafter
+    with pytest.raises(ValueError, match="recurrent"):
+        make_llm(folder, "mixed", "f32", "cpu").set_drafter(NgramDrafter(gamma=2))
+    assert LayerSpec("attention", 1, 8, 8, window=5, keep_first=2).span == 7
