@@ -53,6 +53,9 @@ def parse_args():
                          "batch replicated (dense models); tp+ep = attention sharded by heads and experts spread over the same ranks, "
                          "batch replicated (the layout of the largest MoE models, e.g. --model qwen3-235b-a22b); auto picks by model")
     ap.add_argument("--moe-path", default="fused", choices=["fused", "nccl"], help="multi-GPU expert exchange: fused peer-memory kernels or the NCCL baseline")
+    ap.add_argument("--design", default="", choices=["", "zogavik"],
+                    help="instead of the default workload: prefill and decode throughput of a model described layer by layer, at several sizes, beside the "
+                         "closest other model at equal size (random weights, bf16, one GPU); one JSON line per measurement")
     return ap.parse_args()
 
 
@@ -282,12 +285,83 @@ def baseline_arm(args):
     return 0
 
 
+def design_arm(args):
+    """Prefill and decode throughput of the design's presets and of a Qwen3.5 hybrid (three Delta-Net layers to one of gated attention) of the
+    same width, depth, heads and feed-forward.  Weights and activations exceed L2 in every timed region."""
+    import gc
+    import torch
+    from gemm_b200 import _native
+    from gemm_b200.models.config import ModelConfig, get_config
+    from gemm_b200.models.weights import synthetic_weights
+    from gemm_b200.serve.engine import Engine, SamplingParams
+    torch.cuda.set_device(0)
+    dev = torch.device("cuda", 0)
+
+    def hybrid(layers):
+        return ModelConfig(arch="qwen35", n_layers=layers, hidden=4096, n_heads=32, n_kv_heads=8, head_dim=128, ffn=12288, vocab=151936, rope_dim=64,
+                           full_attention_interval=4, ssm_d_conv=4, ssm_n_heads_k=32, ssm_n_heads_v=32, ssm_head_dim=128, attn_output_gate=True)
+
+    models = [("zogavik-8b", get_config("zogavik-8b")), ("qwen35-hybrid, 36 layers of the same sizes", hybrid(36)), ("zogavik-4b-loop2", get_config("zogavik-4b-loop2"))]
+    sampler = ClockSampler(0)
+    sampler.start()
+    sampler.mark()
+    g = torch.Generator().manual_seed(0)
+    for name, cfg in models:
+        w = synthetic_weights(cfg, "bf16", device=dev, seed=0)
+        torch.cuda.synchronize()
+
+        def emit(metric, tokens, ms, n0, **kw):
+            print(json.dumps({"metric": metric, "value": round(tokens / ms * 1e3, 1), "unit": "tokens/s", "ms": round(ms, 3), "model": name, "params": cfg.param_count(),
+                              "dtype": "bf16", "data": "synthetic, random weights", "gpu_launches": _native.launch_count() - n0, **kw}), flush=True)
+
+        def timed(fn, n):
+            torch.cuda.synchronize()
+            a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+            a.record()
+            for _ in range(n):
+                fn()
+            b.record()
+            torch.cuda.synchronize()
+            return a.elapsed_time(b) / n
+
+        for b, n in ((1, 1024), (1, 8192), (8, 2048)):
+            prompts = [torch.randint(0, cfg.vocab, (n,), generator=g, dtype=torch.int32).to(dev) for _ in range(b)]
+            eng = Engine(w, max_batch=b, max_seq_len=n + 128, page_size=128, max_prefill_tokens=16384, num_pages=b * ((n + 127) // 128 + 1))
+
+            def run():
+                eng.reset()
+                eng.prefill(prompts)
+
+            for _ in range(3):
+                run()
+            n0 = _native.launch_count()
+            emit("prefill", b * n, timed(run, 5), n0, batch=b, prompt_len=n)
+            del eng
+        for b, ctx in ((1, 2048), (16, 2048), (64, 2048), (16, 8192)):
+            eng = Engine(w, max_batch=b, max_seq_len=ctx + 128, page_size=128, max_prefill_tokens=16384, num_pages=b * ((ctx + 127) // 128 + 1))
+            first = eng.prefill([torch.randint(0, cfg.vocab, (ctx,), generator=g, dtype=torch.int32).to(dev) for _ in range(b)], reserve=100).argmax(-1)
+            eng.begin_decode(first, SamplingParams(), 80)
+            for _ in range(8):
+                eng.decode_step()
+            emit("decode", b, timed(eng.decode_step, 50), _native.launch_count() - eng.kernels_per_step * 50, batch=b, context=ctx, kernels_per_step=eng.kernels_per_step)
+            del eng
+        _native.assert_status_ok()
+        del w
+        gc.collect()
+        torch.cuda.empty_cache()
+    clocks = sampler.stop()
+    print(json.dumps({"clocks": clocks}), flush=True)
+    return 0
+
+
 def main():
     args = parse_args()
     if args.impl == "reference":
         return reference_arm(args)
     if args.impl == "baseline":
         return baseline_arm(args)
+    if args.design:
+        return design_arm(args)
 
     import torch
     import torch.distributed as dist

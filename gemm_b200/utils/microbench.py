@@ -17,6 +17,9 @@ Cases
                1 and 4 tokens, fused dequant-GEMM for 8, 64 and 4096 tokens
   small        the kernels around them: RMSNorm + residual + MXFP8 copy, QK-norm + RoPE + cache write (64 and 16384 tokens), the
                one-launch MoE front end, sampler and arg-max over 64 x 151936 logits, the Delta-Net recurrence (decode, prefill)
+  layered      the kernels of models described layer by layer beside the like kernels of the other models at equal size: lightning
+               attention (decode, prefill) and the Delta-Net recurrence; windowed attention with kept tokens and distance bias and the
+               plain causal kernels; the f32-stream norm, Q / K unit norm and gated norm and their bf16-stream counterparts
   spec_verify  whole-model step over 1, 2, 3 and 5 positions per sequence (speculative verification against plain decode);
                builds the full Qwen3-30B-A3B shape, not part of ``all``
 
@@ -339,9 +342,88 @@ def case_small(args):
              2 * st.numel() * 4 + qkv.numel() * 2 + 2 * z.numel() * 2, args)
 
 
+def case_layered(args):
+    from ..ops import deltanet as dn
+    from ..ops import lightning, stream
+    dev, h, hd, d = "cuda", 4096, 32, 128
+    # recurrent layers, 32 heads of 128 x 128
+    for name, lens in (("decode_1", [1]), ("decode_64", [1] * 64), ("prefill_1x8192", [8192]), ("prefill_8x2048", [2048] * 8)):
+        t = sum(lens)
+        cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        sl = torch.arange(len(lens), dtype=torch.int32, device=dev)
+        st = torch.randn(len(lens), hd, d, d, device=dev) * 0.1
+        proj = (torch.randn(t, 4 * hd * d, device=dev) * 0.5).bfloat16()
+        decay = torch.rand(hd, device=dev) * 0.5 + 0.499
+        dec = t == len(lens)
+        src = proj.float() if dec else proj
+        _run(f"lightning_{name}", lambda: lightning.lightning(src, decay, st, cu, sl, hd, d, d, activated=not dec, max_tokens=max(lens)), 4.0 * t * hd * d * d,
+             2 * st.numel() * 4 + t * 3 * hd * d * src.element_size() + t * hd * d * 4, args)
+        o = torch.randn(t, hd * d, device=dev)
+        nw = torch.ones(hd * d, device=dev)
+        _run(f"gated_norm_{name}", lambda: stream.gated_norm(o, src, 3 * hd * d, nw, 1e-6), 0.0, t * hd * d * (4 + src.element_size() + 2), args)
+        z = torch.randn(t, hd * d, device=dev).bfloat16()
+        ab = torch.randn(t, 2 * hd, device=dev)
+        a, bias, nwd = -(torch.rand(hd, device=dev) * 2 + 0.1), torch.randn(hd, device=dev) * 0.5, torch.rand(d, device=dev) + 0.5
+        _run(f"deltanet_{name}", lambda: dn.deltanet(proj[:, : 3 * hd * d], z, ab, a, bias, nwd, st, cu, sl, hd, hd, d, 1e-6), 4.0 * t * hd * d * d,
+             2 * st.numel() * 4 + t * 5 * hd * d * 2, args)
+    # attention, 32 query heads over 8 key / value heads
+    hq, hkv, page = 32, 8, 128
+    for name, b, q_len, ctx, window, keep in (("decode_1x32768", 1, 1, 32767, 4096, 128), ("decode_64x2048", 64, 1, 2047, 4096, 128), ("decode_64x8192", 64, 1, 8191, 4096, 128),
+                                              ("prefill_1x8192", 1, 8192, 0, 4096, 128), ("prefill_8x2048", 8, 2048, 0, 4096, 128)):
+        kv = ctx + q_len
+        pages = (kv + page - 1) // page
+        k = (torch.randn((b * pages + 1) * page, hkv, d, device=dev) * 0.5).bfloat16()
+        v = torch.randn_like(k)
+        bt = torch.arange(b * pages, device=dev, dtype=torch.int32).reshape(b, pages) + 1
+        q = (torch.randn(b * q_len, hq, d, device=dev) * 0.5 * ew.softmax_scale_log2(d)).bfloat16()
+        cu = torch.tensor([i * q_len for i in range(b + 1)], device=dev, dtype=torch.int32)
+        kvl = torch.full((b,), kv, device=dev, dtype=torch.int32)
+        table = att.distance_bias_table(torch.randn(32, hq), 4096).to(dev)
+        dec = q_len == 1
+        seen = [min(i + 1, window + keep) for i in range(ctx, kv)]
+        kv_bytes = b * min(kv, window + keep + q_len) * hkv * d * 4 + b * q_len * hq * d * 4
+        splits = att.pick_splits(b, hkv, min(kv, window + keep + 128)) if dec else 1
+        plan = (att.build_work([q_len] * b, hq, hkv, splits).to(dev), splits)
+        _run(f"attn_masked_{name}", lambda: att.attention_masked(q, k, v, cu, kvl, bt, page, window, keep, table, plan, dec), 4.0 * b * hq * d * sum(seen), kv_bytes, args,
+             splits=splits)
+        _run(f"attn_window_{name}", lambda: att.attention(q, k, v, cu, kvl, bt, page, plan[0], num_splits=splits, window=window, decode=dec),
+             4.0 * b * hq * d * sum(min(i + 1, window) for i in range(ctx, kv)), kv_bytes, args, splits=splits)
+        del k, v
+    for t in (1, 64, 8192):
+        x, w = torch.randn(t, h, device=dev), torch.ones(h, device=dev)
+        up = torch.randn(t, h, device=dev)
+        _run(f"stream_norm_{t}x{h}", lambda: stream.norm(x, w, 1e-6, up), 0.0, t * h * (4 + 4 + 4 + 2), args)
+        xb, wb = x.bfloat16(), w.bfloat16()
+        _run(f"rmsnorm_add_{t}x{h}", lambda: ew.rmsnorm(xb, wb, 1e-6, residual=xb), 0.0, t * h * 8, args)
+        qkv = torch.randn(t, (hq + 2 * hkv) * d, device=dev)
+        qkvb = qkv.bfloat16()
+        src = qkv if t <= 64 else qkvb
+        slots = torch.randperm(t, device=dev).to(torch.int32)
+        pos = torch.arange(t, device=dev, dtype=torch.int32) % 4096
+        kc, vc = torch.empty(t, hkv, d, device=dev, dtype=torch.bfloat16), torch.empty(t, hkv, d, device=dev, dtype=torch.bfloat16)
+        _run(f"qk_unit_{t}", lambda: stream.qk_unit(src, slots, kc, vc, hq, hkv, d, d, 1e-6, 0.1), 0.0, t * (hq + 2 * hkv) * d * (src.element_size() + 2), args)
+        qw = torch.ones(d, device=dev, dtype=torch.bfloat16)
+        tab = ew.rope_table(4096, d, 1e6, dev)
+        _run(f"qk_norm_rope_{t}", lambda: ew.qk_norm_rope(qkvb, pos, slots, qw, qw, kc, vc, hq, hkv, d, 1e6, 1e-6, 1.0, table=tab), 0.0, t * (hq + 2 * hkv) * d * 4, args)
+        xb = (torch.randn(t, h, device=dev) * 0.5).bfloat16()
+        for nm, n, kk in (("in", 16384, 4096), ("out", 4096, 4096), ("down", 4096, 12288)):
+            wt = mxfp8.tile_weight((torch.randn(n, kk, device=dev) * 0.02).bfloat16())
+            xk = xb if kk == 4096 else xb.repeat(1, 3)
+            _run(f"gemm_{nm}_bf16_{t}", lambda: gemm.linear(xk, wt, w_tiled=True), 2.0 * t * n * kk, n * kk * 2 + t * kk * 2 + t * n * 2, args)
+            if nm == "in":
+                _run(f"gemm_{nm}_silu_{t}", lambda: gemm.linear(xk, wt, w_tiled=True, silu_rows=12288), 2.0 * t * n * kk, n * kk * 2 + t * kk * 2 + t * n * 2, args)
+            else:
+                _run(f"gemm_{nm}_f32_{t}", lambda: gemm.linear(xk, wt, w_tiled=True, out_dtype=torch.float32), 2.0 * t * n * kk, n * kk * 2 + t * kk * 2 + t * n * 4, args)
+            del wt
+        wg = mxfp8.tile_weight((torch.randn(24576, h, device=dev) * 0.02).bfloat16())
+        for act in ("silu", "gelu_tanh"):
+            _run(f"gate_up_{act}_{t}", lambda: gemm.linear_swiglu(xb, wg, w_tiled=True, act=act), 2.0 * t * 24576 * h, 24576 * h * 2 + t * h * 2 + t * 12288 * 2, args)
+        del wg
+
+
 MODEL_CASES = {"spec_verify": case_spec_verify}      # build the whole benchmark model: not part of --case all
 CASES = {"gemm": case_gemm, "moe_decode": case_moe_decode, "moe_prefill": case_moe_prefill, "attn_decode": case_attn_decode,
-         "attn_prefill": case_attn_prefill, "lm_head": case_lm_head, "quant": case_quant, "small": case_small}
+         "attn_prefill": case_attn_prefill, "lm_head": case_lm_head, "quant": case_quant, "small": case_small, "layered": case_layered}
 
 
 def main(argv=None):
