@@ -76,15 +76,6 @@ __device__ __forceinline__ float fast_exp2(float x) {
   return y;
 }
 
-// Barrier over the 128 softmax threads (named barrier 1) that also ANDs a predicate: every thread learns whether all of them
-// got through their bounded wait, so they leave the loop together and nobody is left standing at a barrier.
-__device__ __forceinline__ bool softmax_bar_and(bool pred) {
-  uint32_t r;
-  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 q, %1, 0;\n\tbar.red.and.pred p, 1, 128, q;\n\tselp.u32 %0, 1, 0, p;\n\t}"
-               : "=r"(r) : "r"((uint32_t)pred) : "memory");
-  return r != 0;
-}
-
 constexpr int kFaSmem = 32768 * 3 + 256 + 1024;
 
 // DK / DV: width of a key / value head in the cache (64 or 128 columns).  EXT: kept first positions and a distance bias.
@@ -94,7 +85,7 @@ __global__ void __launch_bounds__(kFaThreads, 2)
 flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, const FaArgs a) {
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);      // an offset, so that accesses stay shared-memory ones
   uint8_t* sQ = smem;                       // 2 x [128 rows x 128 B]  (d halves)
   uint8_t* sK = smem + 32768;               // one block: 2 x [128 positions x 128 B]
   uint8_t* sV = smem + 32768 * 2;           // one block
@@ -254,7 +245,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
               win[h * bias_w + x] = bias_row[(size_t)h * a.ld_bias + max(0, min(dmin + x, a.n_bias - 1))];
       }
       got = mbar_wait(s_full, j & 1, abort_flag, a.status, 600, j);
-      if constexpr (EXT) got = softmax_bar_and(got);            // the window is complete; all 128 threads leave together
+      if constexpr (EXT) got = bar128_and(got);            // the window is complete; all 128 threads leave together
       if (!got) { ok = false; break; }
       tc_fence_after();
       int hi = kv_len - 1;
@@ -456,7 +447,7 @@ __global__ void __launch_bounds__(kFdThreads, 2)
 flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const FaArgs a) {
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);      // an offset, so that accesses stay shared-memory ones
   uint8_t* sQ = smem;                          // 2 d-halves x [16 heads x 128 B]
   uint8_t* ring = smem + 4096;                 // 3 slots x 32 KB; tile t = 2j is K of block j, t = 2j + 1 is V of block j, slot = t % 3
   uint8_t* sP = ring + 3 * 32768;              // 2 buffers x 2 position-halves x [16 heads x 128 B] (bf16, 128B swizzle)
@@ -623,7 +614,7 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         const float v = warp_reduce16_max(sv, lane);            // lane L ends with head L >> 1
         if ((lane & 1) == 0) rm[q * kFdN + (lane >> 1)] = v;
       }
-      if (!softmax_bar_and(got_s && !fail_o)) { ok = false; break; }   // maxima of all four warps are in rm; all 128 threads leave together
+      if (!bar128_and(got_s && !fail_o)) { ok = false; break; }   // maxima of all four warps are in rm; all 128 threads leave together
       float bm[kFdN];
       bool need = false;
 #pragma unroll
@@ -680,7 +671,7 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     {
       const float v = warp_reduce16_sum(l, lane);
       if ((lane & 1) == 0) red_sum[q * kFdN + (lane >> 1)] = v;
-      ok = softmax_bar_and(ok && !fail_o);       // every softmax thread gets here exactly once, whatever happened in the loop
+      ok = bar128_and(ok && !fail_o);       // every softmax thread gets here exactly once, whatever happened in the loop
 #pragma unroll
       for (int h = 0; h < kFdN; ++h) l[h] = red_sum[h] + red_sum[kFdN + h] + red_sum[2 * kFdN + h] + red_sum[3 * kFdN + h];
     }

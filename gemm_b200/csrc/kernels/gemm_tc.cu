@@ -410,7 +410,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           float v = __uint_as_float(r0[j]);
           if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
           v += bias;
-          if (row_act) v = silu_f(v);
+          if (row_act) v = __fdividef(v, 1.0f + __expf(-v));
           const bool live = xr < t.valid;
           const int x_row = t.x_row0 + xr;
           if (QUANT_OUT) {
@@ -615,7 +615,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               float v = __uint_as_float(r0[j]);
               if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
               v += bias;
-              if (row_act) v = silu_f(v);
+              if (row_act) v = __fdividef(v, 1.0f + __expf(-v));
               if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
               else o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v);
             }
@@ -625,7 +625,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               float v = __uint_as_float(r0[j]);
               if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
               v += bias;
-              if (row_act) v = silu_f(v);
+              if (row_act) v = __fdividef(v, 1.0f + __expf(-v));
               if (c + j < t.valid) {
                 if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
                 else o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v);

@@ -7,7 +7,7 @@
 // with the activation applied (the projection's GEMM does it), fetched by TMA; the state is f32 in registers, one key row per thread.
 //   TMA warp    : Q, K, V of chunk j + 1 land while chunk j is computed
 //   MMA thread  : S1 = Q K^T;  dS = K^T (w V);  O1 = Q S;  O2 = P V         (A of O2 is P in TMEM; S and w V are written to smem)
-//   P warps     : S1 row -> times g^(i-j), lower triangle -> P in TMEM;  g^(i+1) O1 + O2 -> global f32
+//   P warps     : S1 row -> times g^(i-j), lower triangle -> P in TMEM;  g^(i+1) O1 + O2 -> global f32 (TMA)
 //   state warps : V -> w V in smem;  S <- g^n S + dS;  S -> smem for the next chunk's O1
 // Every f32 factor that goes through the tensor cores (P, w V, S) is the sum of two bf16 operands (hi + lo, 16 bits of mantissa), so
 // decays and state keep 32-bit accuracy; only q, k and v themselves are bf16.
@@ -48,33 +48,35 @@ __device__ __forceinline__ bool warp_wait(uint64_t* bar, uint32_t parity, volati
 template <int DP>                          // key size padded: 64 or 128
 __global__ void __launch_bounds__(kLcThreads, 1)
 lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                       const LightningChunkArgs a) {
+                       const __grid_constant__ CUtensorMap tmO, const LightningChunkArgs a) {
   extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = (uint8_t*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
+  uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);      // an offset, so that accesses stay shared-memory ones
   // stage b at b * kLcStage: Q, K, V
   uint8_t* sWV = smem + 2 * kLcStage;                       // hi, lo
   uint8_t* sS = sWV + 2 * kLcVt;                            // hi, lo
   uint64_t* bars = (uint64_t*)(sS + 2 * kLcVt);
   uint64_t* qk_full = bars;          // 2
   uint64_t* v_full = bars + 2;       // 2
-  uint64_t* t_empty = bars + 4;      // 2
+  uint64_t* t_empty = bars + 4;      // 2: the chunk's last MMA, and the output tile (staged over Q) has been read
   uint64_t* s1_full = bars + 6;
   uint64_t* p_ready = bars + 7;      // 128 arrivals
   uint64_t* wv_ready = bars + 8;     // 128
   uint64_t* s_ready = bars + 9;      // 128
   uint64_t* ds_full = bars + 10;
   uint64_t* o_full = bars + 11;
-  uint32_t* tmem_slot = (uint32_t*)(bars + 12);
+  uint64_t* o_free = bars + 12;      // 128
+  uint64_t* o1_done = bars + 13;
+  uint32_t* tmem_slot = (uint32_t*)(bars + 14);
   volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
   float* pz = (float*)(bars + 32);                          // 128 zeros, then g^0 .. g^128
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < 2; ++i) { mbar_init(&qk_full[i], 1); mbar_init(&v_full[i], 1); mbar_init(&t_empty[i], 1); }
-    mbar_init(s1_full, 1); mbar_init(p_ready, 128); mbar_init(wv_ready, 128); mbar_init(s_ready, 128); mbar_init(ds_full, 1); mbar_init(o_full, 1);
+    for (int i = 0; i < 2; ++i) { mbar_init(&qk_full[i], 1); mbar_init(&v_full[i], 1); mbar_init(&t_empty[i], 2); }
+    mbar_init(s1_full, 1); mbar_init(p_ready, 128); mbar_init(wv_ready, 128); mbar_init(s_ready, 128); mbar_init(ds_full, 1); mbar_init(o_full, 1); mbar_init(o_free, 128); mbar_init(o1_done, 1);
     *abort_flag = 0;
     fence_barrier_init();
-    tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
+    tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV); tma_prefetch_desc(&tmO);
   }
   if (warp == 1) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
   pdl_wait();
@@ -137,8 +139,7 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
                        (part > 0 || ks > 0) ? 1u : 0u);
         tc_commit(ds_full);
         if (!mbar_wait(s_ready, ph, abort_flag, a.status, 712, j)) break;
-        if (!mbar_wait(p_ready, ph, abort_flag, a.status, 713, j)) break;
-        if (!mbar_wait(&v_full[b], ph2, abort_flag, a.status, 714, j)) break;
+        if (j > 0 && !mbar_wait(o_free, ph ^ 1, abort_flag, a.status, 715, j)) break;
         tc_fence_after();
 #pragma unroll
         for (int part = 0; part < 2; ++part)
@@ -146,6 +147,10 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
           for (int ks = 0; ks < DP / 16; ++ks)
             mma_f16_ss(t_o1, make_sdesc_sw128(q_addr + (ks >> 2) * 16384 + (ks & 3) * 32), make_sdesc_sw128_mn(sst + part * kLcVt + ks * 2048, 16384), id_o,
                        (part > 0 || ks > 0) ? 1u : 0u);
+        tc_commit(o1_done);
+        if (!mbar_wait(p_ready, ph, abort_flag, a.status, 713, j)) break;
+        if (!mbar_wait(&v_full[b], ph2, abort_flag, a.status, 714, j)) break;
+        tc_fence_after();
 #pragma unroll
         for (int part = 0; part < 2; ++part)
 #pragma unroll
@@ -161,54 +166,76 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     const float* pw = pz + 128;
     const float gi = pw[i + 1];
+    bool staged = false;                    // the output tile of the previous chunk is on its way out of stage (j - 1) & 1
     for (int j = 0; j < n_chunks; ++j) {
       const uint32_t ph = j & 1;
-      const int t0 = t_begin + j * kLcC;
-      if (!warp_wait(s1_full, ph, abort_flag, a.status, 720, j)) break;
+      const int b = j & 1, t0 = t_begin + j * kLcC;
+      bool ok = warp_wait(s1_full, ph, abort_flag, a.status, 720, j);
       tc_fence_after();
+      if (ok) {
 #pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        uint32_t hi[16], lo[16];
-        if (c <= q) {                       // columns up to the warp's own rows; the rest of P is zero
-          float s[32];
-          tmem_ld_x32(t_s1 + lane_off + c * 32, reinterpret_cast<uint32_t*>(s));
-          tc_wait_ld();
-          const float* w = pw + (i - c * 32);
+        for (int c = 0; c < 4; ++c) {
+          uint32_t hi[16], lo[16];
+          if (c <= q) {                     // columns up to the warp's own rows; the rest of P is zero
+            float s[32];
+            tmem_ld_x32(t_s1 + lane_off + c * 32, reinterpret_cast<uint32_t*>(s));
+            float w[32];                    // zero above the diagonal
 #pragma unroll
-          for (int x = 0; x < 16; ++x) {
-            const int c0 = c * 32 + 2 * x;
-            const float p0 = c0 <= i ? s[2 * x] * w[-(2 * x)] : 0.f, p1 = c0 + 1 <= i ? s[2 * x + 1] * w[-(2 * x + 1)] : 0.f;
-            split_bf16x2(p0, p1, hi[x], lo[x]);
+            for (int x = 0; x < 32; ++x) { w[x] = (pw + (i - c * 32))[-x]; asm volatile("" : "+f"(w[x])); }
+            tc_wait_ld();
+#pragma unroll
+            for (int x = 0; x < 32; ++x) s[x] *= w[x];
+            if (c == q) {
+#pragma unroll
+              for (int x = 0; x < 32; ++x) s[x] = x <= lane ? s[x] : 0.f;
+            }
+#pragma unroll
+            for (int x = 0; x < 16; ++x) split_bf16x2(s[2 * x], s[2 * x + 1], hi[x], lo[x]);
+          } else {
+#pragma unroll
+            for (int x = 0; x < 16; ++x) hi[x] = lo[x] = 0u;
           }
-        } else {
-#pragma unroll
-          for (int x = 0; x < 16; ++x) hi[x] = lo[x] = 0u;
+          tmem_st_x16(t_s1 + lane_off + c * 16, hi);        // over columns that are already read
+          tmem_st_x16(t_plo + lane_off + c * 16, lo);
         }
-        tmem_st_x16(t_s1 + lane_off + c * 16, hi);          // over columns that are already read
-        tmem_st_x16(t_plo + lane_off + c * 16, lo);
+        tc_wait_st();
+        tc_fence_before();
+        mbar_arrive(p_ready);
       }
-      tc_wait_st();
-      tc_fence_before();
-      mbar_arrive(p_ready);
-      if (!warp_wait(o_full, ph, abort_flag, a.status, 721, j)) break;
+      if (staged && threadIdx.x == 64) { tma_store_wait_read(); mbar_arrive(&t_empty[b ^ 1]); }
+      if (ok) ok = warp_wait(o_full, ph, abort_flag, a.status, 721, j);
       tc_fence_after();
+      const bool full = t0 + kLcC <= t_end;         // a whole tile leaves through shared memory (over the chunk's Q) and TMA
+      uint8_t* so = smem + b * kLcStage;
+      if (ok) {
 #pragma unroll
-      for (int c = 0; c < 2; ++c) {
-        float o1[32], o2[32];
-        tmem_ld_x32(t_o1 + lane_off + c * 32, reinterpret_cast<uint32_t*>(o1));
-        tmem_ld_x32(t_o2 + lane_off + c * 32, reinterpret_cast<uint32_t*>(o2));
-        tc_wait_ld();
-        if (t0 + i < t_end) {
+        for (int c = 0; c < 2; ++c) {
+          float o1[32], o2[32];
+          tmem_ld_x32(t_o1 + lane_off + c * 32, reinterpret_cast<uint32_t*>(o1));
+          tmem_ld_x32(t_o2 + lane_off + c * 32, reinterpret_cast<uint32_t*>(o2));
+          tc_wait_ld();
           float* dst = a.out + (size_t)(t0 + i) * a.ld_out + (size_t)h * a.vdim + e0 + c * 32;
 #pragma unroll
-          for (int x = 0; x < 8; ++x)
-            if (e0 + c * 32 + x * 4 < a.vdim)
-              *reinterpret_cast<float4*>(dst + x * 4) = make_float4(fmaf(gi, o1[4 * x], o2[4 * x]), fmaf(gi, o1[4 * x + 1], o2[4 * x + 1]),
-                                                                    fmaf(gi, o1[4 * x + 2], o2[4 * x + 2]), fmaf(gi, o1[4 * x + 3], o2[4 * x + 3]));
+          for (int x = 0; x < 8; ++x) {
+            const float4 v = make_float4(fmaf(gi, o1[4 * x], o2[4 * x]), fmaf(gi, o1[4 * x + 1], o2[4 * x + 1]), fmaf(gi, o1[4 * x + 2], o2[4 * x + 2]),
+                                         fmaf(gi, o1[4 * x + 3], o2[4 * x + 3]));
+            if (full) *reinterpret_cast<float4*>(so + c * 16384 + i * 128 + ((x ^ (i & 7)) << 4)) = v;
+            else if (t0 + i < t_end && e0 + c * 32 + x * 4 < a.vdim) *reinterpret_cast<float4*>(dst + x * 4) = v;
+          }
         }
+        tc_fence_before();
+        mbar_arrive(o_free);
+        fence_proxy_async_smem();
       }
-      tc_fence_before();                    // O1 / O2 are read before the next p_ready lets them be overwritten
+      if (!bar128_and(ok)) break;
+      staged = full;
+      if (full && threadIdx.x == 64) {
+        tma_store_3d(&tmO, so, e0, h, t0);
+        if (e0 + 32 < a.vdim) tma_store_3d(&tmO, so + 16384, e0 + 32, h, t0);
+        tma_store_commit();
+      }
     }
+    if (threadIdx.x == 64) tma_store_wait_read();
   } else {
     // ---------------------------------------------------------------- state: thread = key row d; for w V: thread = token row
     const int q = warp & 3, d = q * 32 + lane;
@@ -279,8 +306,8 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       }
       tc_fence_before();
       if (j + 1 < n_chunks) {
-        // the chunk's O1 has read the state in shared memory once o_full is there
-        if (!warp_wait(o_full, ph, abort_flag, a.status, 732, j)) { ok = false; break; }
+        // the chunk's O1 has read the state in shared memory
+        if (!warp_wait(o1_done, ph, abort_flag, a.status, 732, j)) { ok = false; break; }
         publish();
       }
     }
@@ -302,7 +329,7 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
 }
 
 template <int DP>
-static int lightning_chunk_launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const LightningChunkArgs& a, int n_seqs,
+static int lightning_chunk_launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CUtensorMap& tmO, const LightningChunkArgs& a, int n_seqs,
                                   cudaStream_t stream) {
   static bool attr_set = false;
   if (!attr_set) {
@@ -310,7 +337,7 @@ static int lightning_chunk_launch(const CUtensorMap& tmQ, const CUtensorMap& tmK
     attr_set = true;
   }
   const dim3 grid((unsigned)a.heads, (unsigned)((a.vdim + kLcV - 1) / kLcV), (unsigned)n_seqs);
-  launch_k(lightning_chunk_kernel<DP>, grid, kLcThreads, kLcSmem, stream, tmQ, tmK, tmV, a);
+  launch_k(lightning_chunk_kernel<DP>, grid, kLcThreads, kLcSmem, stream, tmQ, tmK, tmV, tmO, a);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -329,15 +356,18 @@ GB_API int gb_lightning_chunk(const void* proj, int ld, int tokens, const float*
   if (((uintptr_t)proj & 15) || ((uintptr_t)state & 15) || ((uintptr_t)out & 15)) return fail("lightning_chunk: misaligned rows%s");
   if (n_seqs > 65535 || (vdim + kLcV - 1) / kLcV > 65535) return fail("lightning_chunk: too many sequences%s");
   const __nv_bfloat16* p = (const __nv_bfloat16*)proj;
-  CUtensorMap tmQ, tmK, tmV;
+  CUtensorMap tmQ, tmK, tmV, tmO;
   uint32_t box[3] = {64, 1, (uint32_t)kLcC};
   uint64_t dk[3] = {(uint64_t)dim, (uint64_t)heads, (uint64_t)tokens}, dv[3] = {(uint64_t)vdim, (uint64_t)heads, (uint64_t)tokens};
   uint64_t sk[2] = {(uint64_t)dim * 2, (uint64_t)ld * 2}, sv[2] = {(uint64_t)vdim * 2, (uint64_t)ld * 2};
   if (make_tmap(&tmQ, p, TM_BF16, 3, dk, sk, box, TM_SW_128)) return -1;
   if (make_tmap(&tmK, p + (size_t)heads * dim, TM_BF16, 3, dk, sk, box, TM_SW_128)) return -1;
   if (make_tmap(&tmV, p + (size_t)2 * heads * dim, TM_BF16, 3, dv, sv, box, TM_SW_128)) return -1;
+  uint32_t obox[3] = {32, 1, (uint32_t)kLcC};
+  uint64_t so[2] = {(uint64_t)vdim * 4, (uint64_t)ld_out * 4};
+  if (make_tmap(&tmO, out, TM_F32, 3, dv, so, obox, TM_SW_128)) return -1;
   LightningChunkArgs a;
   a.decay = decay; a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out; a.ld_out = ld_out;
   a.heads = heads; a.dim = dim; a.vdim = vdim; a.status = (KernelStatus*)status;
-  return dim <= 64 ? lightning_chunk_launch<64>(tmQ, tmK, tmV, a, n_seqs, stream) : lightning_chunk_launch<128>(tmQ, tmK, tmV, a, n_seqs, stream);
+  return dim <= 64 ? lightning_chunk_launch<64>(tmQ, tmK, tmV, tmO, a, n_seqs, stream) : lightning_chunk_launch<128>(tmQ, tmK, tmV, tmO, a, n_seqs, stream);
 }

@@ -129,6 +129,15 @@ __device__ __forceinline__ bool mbar_wait(uint64_t* bar, uint32_t parity, volati
   }
 }
 
+// Barrier over 128 threads of the CTA (named barrier 1) that also ANDs a predicate: every thread learns whether all of them got through
+// their bounded waits, so they leave a loop together and nobody is left standing at a barrier.
+__device__ __forceinline__ bool bar128_and(bool pred) {
+  uint32_t r;
+  asm volatile("{\n\t.reg .pred p, q;\n\tsetp.ne.u32 q, %1, 0;\n\tbar.red.and.pred p, 1, 128, q;\n\tselp.u32 %0, 1, 0, p;\n\t}"
+               : "=r"(r) : "r"((uint32_t)pred) : "memory");
+  return r != 0;
+}
+
 // ---------------------------------------------------------------------------------------------
 // TMA (tiled bulk tensor copies, no multicast anywhere in this library)
 // ---------------------------------------------------------------------------------------------
@@ -148,6 +157,14 @@ __device__ __forceinline__ void tma_load_4d(void* smem_dst, const void* tmap, ui
   asm volatile("cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%3, %4, %5, %6}], [%2];"
                :: "r"(smem_u32(smem_dst)), "l"(tmap), "r"(smem_u32(bar)), "r"(x), "r"(y), "r"(z), "r"(w) : "memory");
 }
+// Shared memory -> global.  The writer makes its stores visible with fence_proxy_async_smem first; the source may be reused after
+// tma_store_wait_read.
+__device__ __forceinline__ void tma_store_3d(const void* tmap, const void* smem_src, int x, int y, int z) {
+  asm volatile("cp.async.bulk.tensor.3d.global.shared::cta.bulk_group [%0, {%2, %3, %4}], [%1];" :: "l"(tmap), "r"(smem_u32(smem_src)), "r"(x), "r"(y), "r"(z) : "memory");
+}
+__device__ __forceinline__ void tma_store_commit() { asm volatile("cp.async.bulk.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void tma_store_wait_read() { asm volatile("cp.async.bulk.wait_group.read 0;" ::: "memory"); }
+
 // Untiled bulk copy global -> shared (both 16-byte aligned, size multiple of 16).
 __device__ __forceinline__ void bulk_load(void* smem_dst, const void* gsrc, uint32_t bytes, uint64_t* bar) {
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
