@@ -387,8 +387,8 @@ def cmd_dump(args):
     ids = [int(x) for x in args.ids.replace(",", " ").split()]
     page = 16
     n_pages = len(ids) // page + 2
-    m = Transformer(w, KvCache.allocate(cfg, n_pages, page, dev))
-    m.snapshot_layers = tuple(range(len(w.layers)))
+    m = Transformer(w, KvCache.allocate(cfg, n_pages, page, dev, kv_dtype=w.kv_dtype))
+    m.snapshot_layers = tuple(range(len(m.runs)))
     bt = torch.arange(n_pages, dtype=torch.int32).unsqueeze(0)
     fb = ForwardBatch.build([len(ids)], [0], torch.tensor(ids), bt, page, cfg.n_heads, cfg.n_kv_heads, dev)
     fb.logit_rows = torch.arange(len(ids), device=fb.ids.device)
