@@ -83,8 +83,7 @@ struct GemmArgs {
   int early_weights;  // != 0: a plain decode-sized launch requests its first weight tiles before the dependency wait
   int dual_raw;  // DUAL without the activation: the second accumulator is the row block up_row_offset further down the same matrix
   int w_tiled;
-  int act;       // activation of the gate half of a DUAL launch: 0 = SiLU, 1 = the tanh form of GELU
-  int silu_rows; // plain launches: SiLU on the output features below this (the q / k / v part of a linear-attention projection)
+  int silu_rows; // plain launches with ACT = 1: SiLU on the output features below this (the q / k / v part of a linear-attention projection)
 };
 
 // k-steps whose MXFP8 scale atoms are fetched by one bulk copy (2 for the widest tile, whose stages are short of room)
@@ -130,10 +129,12 @@ struct TileCursor {
 };
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
-// Gate activation.  The tanh form of GELU, x (1 + tanh u) / 2 with u = sqrt(2 / pi) (x + 0.044715 x^3), is x / (1 + exp(-2 u)).
-__device__ __forceinline__ float gate_act(float x, int act) {
-  const float z = act == 1 ? 1.5957691216057308f * (x + 0.044715f * x * x * x) : x;
-  return x / (1.0f + __expf(-z));
+// Gate activation: 0 = SiLU, 1 = the tanh form of GELU, x (1 + tanh u) / 2 with u = sqrt(2 / pi) (x + 0.044715 x^3), which is
+// x / (1 + exp(-2 u)).
+template <int ACT>
+__device__ __forceinline__ float gate_act(float x) {
+  if constexpr (ACT == 0) return silu_f(x);
+  else return x / (1.0f + __expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
 }
 
 // E8M0 exponent for a block whose absolute maximum is `amax`: the smallest power of two s with
@@ -146,7 +147,8 @@ __device__ __forceinline__ int e8m0_from_amax(float amax) {
   return amax == 0.0f ? 127 : max(1, min(e, 254));   // an all-zero block gets scale 1
 }
 
-template <int TN, int MODE, bool DUAL, bool QUANT_OUT>
+// ACT, DUAL: the gate's activation (gate_act); plain: 1 = SiLU on the output features below args.silu_rows.
+template <int TN, int MODE, bool DUAL, bool QUANT_OUT, int ACT = 0>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, const GemmArgs args) {
   constexpr int NA = DUAL ? 2 : 1;
@@ -400,7 +402,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       const uint32_t tacc = tmem_base + acc * ACC_COLS + ((uint32_t)(q * 32) << 16);
       const int n = t.n0 + row;
       const bool n_ok = n < args.n_out;
-      const bool row_act = !DUAL && n < args.silu_rows;
+      const bool row_act = !DUAL && ACT == 1 && n < args.silu_rows;
       const float bias = (args.bias != nullptr && n_ok && (args.partial_stride == 0 || t.ks == 0)) ? args.bias[n] : 0.0f;
       // Everything after the accumulators are in registers: activation, bias, then one of the store forms.
       auto finish_chunk = [&](int c, const uint32_t* r0, const uint32_t* r1) {
@@ -408,9 +410,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         for (int j = 0; j < 16; ++j) {
           const int xr = c + j;
           float v = __uint_as_float(r0[j]);
-          if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
+          if (DUAL) v = gate_act<ACT>(v) * __uint_as_float(r1[j]);
           v += bias;
-          if (row_act) v = __fdividef(v, 1.0f + __expf(-v));
+          if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
           const bool live = xr < t.valid;
           const int x_row = t.x_row0 + xr;
           if (QUANT_OUT) {
@@ -544,8 +546,8 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         }
         __nv_bfloat16* o16 = (__nv_bfloat16*)obase + part_off + orow0 * args.ldo + n;
         float* o32 = (float*)obase + part_off + orow0 * args.ldo + n;
-        if constexpr (NACC == 1 && !DUAL) {
-          if (!args.out_f32 && args.silu_rows == 0) {
+        if constexpr (NACC == 1 && !DUAL && ACT == 0) {
+          if (!args.out_f32) {
             // One accumulator buffer (the widest tile with its scale columns fills TMEM): pull the whole row into registers
             // as packed bf16, hand the buffer back to the MMA thread, and only then store, so that the stores overlap the
             // next tile's MMAs.
@@ -613,9 +615,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               float v = __uint_as_float(r0[j]);
-              if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
+              if (DUAL) v = gate_act<ACT>(v) * __uint_as_float(r1[j]);
               v += bias;
-              if (row_act) v = __fdividef(v, 1.0f + __expf(-v));
+              if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
               if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
               else o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v);
             }
@@ -623,9 +625,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               float v = __uint_as_float(r0[j]);
-              if (DUAL) v = gate_act(v, args.act) * __uint_as_float(r1[j]);
+              if (DUAL) v = gate_act<ACT>(v) * __uint_as_float(r1[j]);
               v += bias;
-              if (row_act) v = __fdividef(v, 1.0f + __expf(-v));
+              if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
               if (c + j < t.valid) {
                 if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
                 else o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v);
@@ -672,7 +674,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
   }
 }
 
-template <int TN, int MODE, bool DUAL, bool QUANT_OUT>
+template <int TN, int MODE, bool DUAL, bool QUANT_OUT, int ACT = 0>
 static int launch_gemm(const CUtensorMap& tmW, const CUtensorMap& tmX, GemmArgs a, int max_tiles, cudaStream_t stream) {
   constexpr int NA = DUAL ? 2 : 1;
   constexpr int SFB_ATOMS = (TN + 127) / 128;
@@ -683,7 +685,7 @@ static int launch_gemm(const CUtensorMap& tmW, const CUtensorMap& tmX, GemmArgs 
   if (stages < 2) return fail("gemm: tile does not fit shared memory%s");
   a.stages = stages;
   const int smem = stages * STAGE_BYTES + tail + 1024;
-  auto kern = gemm_tc_kernel<TN, MODE, DUAL, QUANT_OUT>;
+  auto kern = gemm_tc_kernel<TN, MODE, DUAL, QUANT_OUT, ACT>;
   static bool attr_set = false;
   if (!attr_set) {
     GB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024));
@@ -797,7 +799,8 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
     a.early_weights = early;
   }
   a.dual_raw = (flags & GEMM_DUAL_RAW) ? 1 : 0;
-  a.act = (flags & GEMM_GELU) ? 1 : 0;
+  const bool gelu = flags & GEMM_GELU;
+  if (gelu && (!dual || mx || qo)) return fail("gemm: GEMM_GELU needs a bf16 GEMM_DUAL launch%s");
   if (a.dual_raw && (!dual || qo)) return fail("gemm: GEMM_DUAL_RAW needs GEMM_DUAL without GEMM_QUANT_OUT%s");
   a.out_sf = (uint8_t*)out_sf; a.bias = bias; a.row_map = row_map; a.row_scale = row_scale; a.status = (KernelStatus*)status;
   if (ex != nullptr) {
@@ -806,7 +809,7 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
     a.peer_region_rows = ex->peer_region_rows; a.peer_rank = ex->peer_rank; a.signal_n = ex->signal_n; a.done_ctr = ex->done_ctr;
     a.amax_val = ex->amax_val; a.amax_idx = ex->amax_idx; a.peer_bcast = ex->peer_bcast; a.epoch_self_tick = ex->epoch_self_tick;
     a.sfa_bytes = ex->sfa_bytes; a.sfb_bytes = ex->sfb_bytes; a.out_bytes = ex->out_bytes; a.out_sf_bytes = ex->out_sf_bytes;
-    if (ex->silu_rows > 0 && (dual || ex->splits > 1)) return fail("gemm: silu_rows needs a plain launch%s");
+    if (ex->silu_rows > 0 && (dual || mx || qo || ex->splits > 1 || tn < 128)) return fail("gemm: silu_rows needs a plain bf16 launch with a token tile of 128 or 256%s");
     a.silu_rows = ex->silu_rows;
     if (ex->splits > 1 && num_groups == 0 && ex->partial_stride > 0) {
       if (!(flags & GEMM_OUT_F32) || qo) return fail("gemm: split-K partials need a plain fp32 output%s");
@@ -836,17 +839,23 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
   a.m_tok_hint = num_groups == 0 ? m_tok : (tn <= 32 ? tn : 1 << 20);
   if (num_groups == 0 && m_tok <= 0) return 0;
 
+  if (a.silu_rows > 0) {
+    if (tn == 128) return launch_gemm<128, 0, false, false, 1>(tmW, tmX, a, max_tiles, stream);
+    if (tn == 256) return launch_gemm<256, 0, false, false, 1>(tmW, tmX, a, max_tiles, stream);
+  }
 #ifdef GB_GEMM_BF16_ONLY
   // build without the MXFP8 variants: the library subset of models whose weights are bf16 or f32
 #define GB_DISPATCH(TNV)                                                                                      \
   if (tn == TNV) {                                                                                            \
     if (!mx && !dual && !qo) return launch_gemm<TNV, 0, false, false>(tmW, tmX, a, max_tiles, stream);        \
+    if (gelu) return launch_gemm<TNV, 0, true, false, 1>(tmW, tmX, a, max_tiles, stream);                     \
     if (!mx && dual && !qo) return launch_gemm<TNV, 0, true, false>(tmW, tmX, a, max_tiles, stream);          \
   }
 #else
 #define GB_DISPATCH(TNV)                                                                                      \
   if (tn == TNV) {                                                                                            \
     if (!mx && !dual && !qo) return launch_gemm<TNV, 0, false, false>(tmW, tmX, a, max_tiles, stream);        \
+    if (gelu) return launch_gemm<TNV, 0, true, false, 1>(tmW, tmX, a, max_tiles, stream);                     \
     if (!mx && dual && !qo) return launch_gemm<TNV, 0, true, false>(tmW, tmX, a, max_tiles, stream);          \
     if (mx && !dual && !qo) return launch_gemm<TNV, 1, false, false>(tmW, tmX, a, max_tiles, stream);         \
     if (mx && dual && qo) return launch_gemm<TNV, 1, true, true>(tmW, tmX, a, max_tiles, stream);             \

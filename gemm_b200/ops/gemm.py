@@ -149,7 +149,7 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
     if out is None:
         out = torch.empty(m, n, dtype=out_dtype, device=x.device)
     flags = (GEMM_OUT_F32 if out.dtype == torch.float32 else 0) | (GEMM_W_TILED if w_tiled else 0)
-    tn = tn or pick_tn(m)
+    tn = tn or (max(128, pick_tn(m)) if silu_rows else pick_tn(m))
     ex = _splitk_extras(n, m, k, tn, False, x.device, split_k) if not silu_rows else GemmExtras()
     if silu_rows:
         ex.silu_rows = silu_rows
