@@ -134,7 +134,7 @@ __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)
 template <int ACT>
 __device__ __forceinline__ float gate_act(float x) {
   if constexpr (ACT == 0) return silu_f(x);
-  else return x / (1.0f + __expf(-1.5957691216057308f * (x + 0.044715f * x * x * x)));
+  else return __fdividef(x, 1.0f + __expf(x * fmaf(-0.07135481627f, x * x, -1.5957691216057308f)));       // -2 sqrt(2 / pi) (x + 0.044715 x^3)
 }
 
 // E8M0 exponent for a block whose absolute maximum is `amax`: the smallest power of two s with
