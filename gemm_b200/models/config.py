@@ -9,21 +9,66 @@ cuda/llm/cuda_llm_runner.c:11277-11310): ``<arch>.embedding_length``, ``attentio
 """
 from __future__ import annotations
 
+import math
 from dataclasses import asdict, dataclass, field, replace
 from typing import Dict, List, Optional
 
 # Architectures described layer by layer (``ModelConfig.layer_specs``): name in config.json -> arch
-LAYERED_ARCHS = {"Zogavik": "zogavik"}
+LAYERED_ARCHS = {"Zogavik": "zogavik", "Famepel": "famepel"}
 
 ARCHS = ("qwen2", "qwen2vl", "qwen3", "qwen3vl", "qwen3moe", "qwen3vlmoe", "qwen35", "qwen35moe")
 
 
 @dataclass
+class RotarySpec:
+    """Rotary positions of neighbouring pairs (2i, 2i + 1).  ``factor`` > 0: YaRN, with the pairs between ``fast`` and ``slow`` turns over
+    ``original`` positions blended from the plain to the divided frequency."""
+    dims: int
+    base: float
+    factor: float = 0.0
+    original: float = 0.0
+    fast: float = 0.0
+    slow: float = 0.0
+
+    def frequencies(self) -> List[float]:
+        f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        if self.factor <= 0:
+            return f
+
+        def pair_of(turns: float) -> float:         # the (fractional) pair that makes `turns` turns over the original length
+            return self.dims * math.log(self.original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.base))
+
+        lo = max(math.floor(pair_of(self.fast)), 0)
+        hi = min(math.ceil(pair_of(self.slow)), self.dims - 1)
+        ramp = [min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0) for i in range(len(f))]
+        return [x / self.factor * r + x * (1.0 - r) for x, r in zip(f, ramp)]
+
+    @property
+    def magnitude(self) -> float:
+        """Factor of cos and sin."""
+        return 0.1 * math.log(self.factor) + 1.0 if self.factor > 0 else 1.0
+
+
+@dataclass
+class MoeSpec:
+    """A mixture of experts: gated feed-forwards of width ``ffn``, ``top`` of ``n_experts`` per token.  ``groups`` > 1: the experts form groups of
+    neighbours, a group scores the sum of its two best experts, and only the best ``groups_kept`` groups can be chosen from."""
+    n_experts: int
+    top: int
+    ffn: int
+    router: str = "softmax"                 # or "sigmoid"
+    renorm: bool = True                     # the chosen scores are divided by their sum
+    scale: float = 1.0
+    groups: int = 1
+    groups_kept: int = 1
+
+
+@dataclass
 class LayerSpec:
     """One layer of a model described layer by layer: its mixer with the mixer's own sizes, and its feed-forward."""
-    mixer: str                              # "attention" | "lightning"
+    mixer: str                              # "attention" | "lightning" | "mamba2" | "hgrn2" | "latent"
     n_heads: int
-    head_dim: int                           # query / key size per head
+    head_dim: int                           # query / key size per head (mamba2: the state size; latent: without the rotated part)
     v_dim: int                              # value size per head
     n_kv_heads: int = 0                     # attention only
     # attention
@@ -36,13 +81,45 @@ class LayerSpec:
     rel_max: float = 0                      # distance from which the last bucket holds
     # lightning attention
     decay: Optional[List[float]] = None     # per head
+    # mamba2
+    state_groups: int = 1                   # heads share B and C by groups
+    conv_taps: int = 0                      # causal convolution in front of the recurrence
+    norm_parts: int = 1                     # the output norm's equal parts
+    # latent attention: keys and values are projections of a cached latent, next to one rotated key part for all heads
+    kv_rank: int = 0
+    q_rank: int = 0
+    rot_dim: int = 0
+    rotary: Optional[RotarySpec] = None
+    sink: bool = False                      # a learned score per head joins the softmax's sum
+    kv_from: int = -1                       # layer whose cache this one reads (-1: its own)
     # feed-forward: act(gate) * up -> down; 0 = none
     ffn: int = 0
     act: str = "silu"                       # or "gelu_tanh"
+    moe: Optional[MoeSpec] = None           # in place of the dense feed-forward
+
+    def __post_init__(self):
+        if isinstance(self.rotary, dict):
+            self.rotary = RotarySpec(**self.rotary)
+        if isinstance(self.moe, dict):
+            self.moe = MoeSpec(**self.moe)
 
     @property
     def q_dim(self) -> int:
         return self.n_heads * self.head_dim
+
+    @property
+    def has_ffn(self) -> bool:
+        return self.ffn > 0 or self.moe is not None
+
+    @property
+    def has_state(self) -> bool:
+        """Whether the mixer carries recurrent state (in place of cache pages)."""
+        return self.mixer in ("lightning", "mamba2", "hgrn2")
+
+    @property
+    def conv_channels(self) -> int:
+        """Channels of the convolution: [x heads x v_dim | B groups x head_dim | C groups x head_dim]."""
+        return self.n_heads * self.v_dim + 2 * self.state_groups * self.head_dim
 
     @property
     def span(self) -> int:
@@ -108,6 +185,9 @@ class ModelConfig:
     loop: Optional[LoopSpec] = None
     norm_offset: float = 0.0                # stored norm weights are added to this (1 = stored around zero)
     logit_scale: float = 1.0
+    norm_kind: str = "rms"                  # or "dyt": tanh(alpha x) w + b
+    post_norm: bool = False                 # every sublayer's result passes a norm of its own and a per-channel scale
+    embed_scale: float = 1.0
 
     def __post_init__(self):
         if self.layer_specs is not None:
@@ -134,8 +214,8 @@ class ModelConfig:
 
     @property
     def has_recurrent_state(self) -> bool:
-        """Whether a sequence carries state that cannot drop positions (Delta-Net or lightning layers)."""
-        return self.is_hybrid or (self.is_layered and any(x.mixer == "lightning" for x in self.layer_specs))
+        """Whether a sequence carries state that cannot drop positions (Delta-Net, lightning, Mamba-2 or HGRN2 layers)."""
+        return self.is_hybrid or (self.is_layered and any(x.has_state for x in self.layer_specs))
 
     @property
     def is_moe(self) -> bool:
@@ -168,10 +248,20 @@ class ModelConfig:
 
     def param_count(self) -> int:
         if self.is_layered:
-            tot = self.vocab * self.hidden
+            tot = self.vocab * self.hidden * (1 if self.tie_embeddings else 2)
             for x in self.layer_specs:
+                nv = x.n_heads * x.v_dim
+                if x.moe is not None:
+                    tot += x.moe.n_experts * self.hidden * (3 * x.moe.ffn + 1)
                 if x.mixer == "lightning":
-                    tot += self.hidden * (2 * x.q_dim + 3 * x.n_heads * x.v_dim)
+                    tot += self.hidden * (2 * x.q_dim + 3 * nv)
+                elif x.mixer == "hgrn2":
+                    tot += self.hidden * (2 * x.q_dim + 2 * nv)
+                elif x.mixer == "mamba2":
+                    tot += self.hidden * (2 * nv + x.conv_channels + x.n_heads) + x.conv_channels * x.conv_taps
+                elif x.mixer == "latent":
+                    own = 0 if x.kv_from >= 0 else x.kv_rank + x.rot_dim
+                    tot += self.hidden * (x.q_rank + own + nv) + x.q_rank * x.n_heads * (x.head_dim + x.rot_dim) + x.kv_rank * (x.q_dim + nv)
                 else:
                     tot += self.hidden * (x.q_dim + x.n_kv_heads * (x.head_dim + x.v_dim) + x.n_heads * x.v_dim)
                 tot += 3 * self.hidden * x.ffn
@@ -241,6 +331,34 @@ PRESETS["tiny-zogavik"] = _zogavik("ALLA", 192, 4, 2, 40, 320, 500, 48, 8, 100, 
 PRESETS["zogavik-8b"] = _zogavik("LLLA" * 9, 4096, 32, 8, 128, 12288, 151936, 4096, 128, 4096)
 # the same layers with the middle ones looped: a smaller model of the same depth
 PRESETS["zogavik-4b-loop2"] = _zogavik("LLLA" * 5, 4096, 32, 8, 128, 12288, 151936, 4096, 128, 4096, LoopSpec(2, 18, 2))
+
+
+def _famepel(pattern: str, hidden: int, vocab: int, moe: MoeSpec, hgrn, mamba, latent, rotary: RotarySpec) -> ModelConfig:
+    """``pattern``: one letter per layer, H = HGRN2, M = Mamba-2, L = latent attention, S = latent attention over the cache of the nearest L in
+    front of it.  ``hgrn`` (heads, dim, vdim), ``mamba`` (heads, state, vdim, groups, taps, norm parts), ``latent`` (heads, dim, rot_dim, vdim,
+    kv_rank, q_rank)."""
+    specs: List[LayerSpec] = []
+    own = -1
+    for i, c in enumerate(pattern):
+        if c == "H":
+            specs.append(LayerSpec("hgrn2", *hgrn, moe=moe))
+        elif c == "M":
+            heads, n, v, groups, taps, parts = mamba
+            specs.append(LayerSpec("mamba2", heads, n, v, state_groups=groups, conv_taps=taps, norm_parts=parts, moe=moe))
+        else:
+            heads, d, r, v, kvr, qr = latent
+            own = i if c == "L" else own
+            specs.append(LayerSpec("latent", heads, d, v, n_kv_heads=1, scale=(d + r) ** -0.5, kv_rank=kvr, q_rank=qr, rot_dim=r, rotary=rotary, sink=True,
+                                   kv_from=own if c == "S" else -1, moe=moe))
+    return ModelConfig(arch="famepel", layer_specs=specs, hidden=hidden, n_heads=latent[0], n_kv_heads=1, head_dim=latent[1], ffn=moe.ffn, vocab=vocab,
+                       rms_eps=1e-5, norm_kind="dyt", post_norm=True, embed_scale=hidden ** 0.5, qk_norm=False)
+
+
+PRESETS["tiny-famepel"] = _famepel("MHLMS", 192, 300, MoeSpec(10, 3, 48, "sigmoid", True, 1.7, 5, 2), (3, 24, 40), (4, 40, 24, 2, 4, 2), (3, 24, 16, 40, 72, 56),
+                                   RotarySpec(16, 10000.0, 4.0, 64, 32.0, 1.0))
+# layers of the sizes of a 30-billion-parameter mixture of experts (128 experts, 8 per token)
+PRESETS["famepel-30b-a3b"] = _famepel("HMLHMMHMS" * 5, 2048, 151936, MoeSpec(128, 8, 768, "sigmoid", True, 2.5, 8, 4), (16, 128, 128), (64, 128, 64, 8, 4, 8),
+                                      (32, 128, 64, 128, 512, 1536), RotarySpec(64, 500000.0, 8.0, 4096, 32.0, 1.0))
 
 
 def get_config(name: str) -> ModelConfig:

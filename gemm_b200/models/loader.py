@@ -18,7 +18,7 @@ import torch
 
 from .. import _native
 from ..utils import gguf as G
-from .config import ARCHS, LAYERED_ARCHS, LayerSpec, LoopSpec, ModelConfig
+from .config import ARCHS, LAYERED_ARCHS, LayerSpec, LoopSpec, ModelConfig, MoeSpec, RotarySpec
 from .weights import ModelWeights, RandomSource, build_weights
 
 
@@ -523,18 +523,40 @@ class LayeredSource(SafetensorsSource):
     """Checkpoints of models described layer by layer: tensors ``l<i>.norm1``, ``l<i>.mix.*``, ``l<i>.norm2``, ``l<i>.mlp.*``, ``embed``,
     ``final.norm``, ``loop.step``, served under the names the model builder asks for."""
 
-    _LAYER = {"attn_norm.weight": "norm1", "ffn_norm.weight": "norm2", "attn_q.weight": "mix.q", "attn_k.weight": "mix.k", "attn_v.weight": "mix.v",
+    _LAYER = {"attn_q.weight": "mix.q", "attn_k.weight": "mix.k", "attn_v.weight": "mix.v",
               "attn_q.bias": "mix.q.b", "attn_k.bias": "mix.k.b", "attn_v.bias": "mix.v.b", "attn_output.weight": "mix.o", "attn_rel.weight": "mix.rel",
               "lin_q.weight": "mix.q", "lin_k.weight": "mix.k", "lin_v.weight": "mix.v", "lin_gate.weight": "mix.g", "lin_norm.weight": "mix.norm",
-              "lin_out.weight": "mix.o", "ffn_gate.weight": "mlp.gate", "ffn_up.weight": "mlp.up", "ffn_down.weight": "mlp.down"}
-    _TOP = {"token_embd.weight": "embed", "output_norm.weight": "final.norm", "loop_step.weight": "loop.step", "output.weight": "head"}
+              "lin_out.weight": "mix.o", "ffn_gate.weight": "mlp.gate", "ffn_up.weight": "mlp.up", "ffn_down.weight": "mlp.down",
+              "attn_post_scale.weight": "ls1", "ffn_post_scale.weight": "ls2", "ffn_gate_inp.weight": "mlp.router",
+              "ssm_in.weight": "mix.in", "ssm_conv1d.weight": "mix.conv", "ssm_conv1d.bias": "mix.conv.b", "ssm_dt.bias": "mix.dt_bias", "ssm_a_log": "mix.A_log",
+              "ssm_d": "mix.D", "ssm_norm.weight": "mix.norm", "ssm_out.weight": "mix.o",
+              "gla_q.weight": "mix.q", "gla_f.weight": "mix.f", "gla_f.bias": "mix.f.b", "gla_lower": "mix.lower", "gla_v.weight": "mix.v", "gla_norm.weight": "mix.norm",
+              "gla_out.weight": "mix.o",
+              "attn_q_a.weight": "mix.dq", "attn_q_a_norm.weight": "mix.dq.norm", "attn_q_b.weight": "mix.uq", "attn_kv_a.weight": "mix.dkv",
+              "attn_kv_a_norm.weight": "mix.dkv.norm", "attn_k_b.weight": "mix.uk", "attn_v_b.weight": "mix.uv", "attn_sink": "mix.sink"}
+    _NORM = {"attn_norm": "norm1", "attn_post_norm": "norm1b", "ffn_norm": "norm2", "ffn_post_norm": "norm2b", "output_norm": "final.norm"}
+    _PART = {"weight": "", "bias": ".b", "alpha": ".alpha"}
+    _EXPERT = {"ffn_gate_exps.weight": "gate", "ffn_up_exps.weight": "up", "ffn_down_exps.weight": "down"}
+    _TOP = {"token_embd.weight": "embed", "loop_step.weight": "loop.step", "output.weight": "head"}
 
     @classmethod
     def file_name(cls, name: str) -> str:
         if name in cls._TOP:
             return cls._TOP[name]
-        _, li, rest = name.split(".", 2)
-        return f"l{li}.{cls._LAYER[rest]}"
+        pre, rest = "", name
+        if name.startswith("blk."):
+            _, li, rest = name.split(".", 2)
+            pre = f"l{li}."
+        head, _, part = rest.partition(".")
+        if head in cls._NORM:
+            return pre + cls._NORM[head] + cls._PART[part]
+        if rest.partition("#")[0] in cls._EXPERT:              # "<name>#<expert>"
+            rest, _, e = rest.partition("#")
+            return f"{pre}mlp.e{e}.{cls._EXPERT[rest]}"
+        return pre + cls._LAYER[rest]
+
+    def get_expert(self, name: str, e: int, shape) -> torch.Tensor:
+        return self.get(f"{name}#{e}", shape)
 
     def has(self, name: str) -> bool:
         return self.file_name(name) in self.where
@@ -553,7 +575,63 @@ class LayeredSource(SafetensorsSource):
         return t
 
 
+def _moe_spec(mlp: dict) -> MoeSpec:
+    r, g = mlp["router"], mlp["router"].get("groups") or {"count": 1, "keep": 1}
+    spec = MoeSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), router="sigmoid", renorm=True, scale=float(r["scale"]), groups=int(g["count"]),
+                   groups_kept=int(g["keep"]))
+    if spec.groups < 1 or spec.n_experts % spec.groups or not 1 <= spec.groups_kept <= spec.groups:
+        raise ValueError(f"router groups: {spec.n_experts} experts in {spec.groups} groups, {spec.groups_kept} kept")
+    if not 1 <= spec.top <= spec.n_experts // spec.groups * spec.groups_kept:
+        raise ValueError(f"router: {spec.top} experts per token of {spec.n_experts // spec.groups * spec.groups_kept} that can be chosen")
+    return spec
+
+
+def _famepel_layer(li: int, e: dict, layers: list) -> LayerSpec:
+    m, mlp = e["mixer"], e.get("mlp")
+    if mlp is not None and mlp.get("kind") != "moe":
+        raise ValueError(f"layer {li}: feed-forward kind {mlp.get('kind')!r} is not supported")
+    moe = _moe_spec(mlp) if mlp is not None else None
+    heads, v = int(m["heads"]), int(m["vdim"])
+    if e["type"] == "hgrn2":
+        return LayerSpec("hgrn2", heads, int(m["dim"]), v, moe=moe)
+    if e["type"] == "mamba2":
+        g, parts = int(m["groups"]), int(m["norm_groups"])
+        if heads % g or (heads * v) % parts:
+            raise ValueError(f"layer {li}: {heads} heads in {g} groups, norm over {parts} parts of {heads * v}")
+        return LayerSpec("mamba2", heads, int(m["state"]), v, state_groups=g, conv_taps=int(m["conv"]), norm_parts=parts, moe=moe)
+    if e["type"] == "latent_attention":
+        r = m["rot"]
+        sc = r.get("scaling")
+        rot = RotarySpec(int(r["dims"]), float(r["base"]), *((float(sc[k]) for k in ("factor", "original", "fast", "slow")) if sc else ()))
+        if rot.dims != int(m["rot_dim"]):
+            raise ValueError(f"layer {li}: rotation over {rot.dims} of {m['rot_dim']} dimensions is not supported")
+        src = m.get("kv_from")
+        if src is not None:
+            o = layers[src] if 0 <= src < li else None
+            if o is None or o["type"] != "latent_attention" or o["mixer"].get("kv_from") is not None or \
+                    any(o["mixer"][k] != m[k] for k in ("kv_rank", "rot_dim")):
+                raise ValueError(f"layer {li}: kv_from {src} is not an earlier latent-attention layer with a cache of the same sizes")
+        return LayerSpec("latent", heads, int(m["dim"]), v, n_kv_heads=1, scale=float(m["scale"]), kv_rank=int(m["kv_rank"]), q_rank=int(m["q_rank"]),
+                         rot_dim=int(m["rot_dim"]), rotary=rot, sink=True, kv_from=-1 if src is None else int(src), moe=moe)
+    raise ValueError(f"layer {li}: mixer {e['type']!r} is not supported")
+
+
+def _famepel_config(c: dict) -> ModelConfig:
+    """config.json of Famepel: HGRN2, Mamba-2 and latent-attention mixers, grouped mixtures of experts, Dynamic-Tanh norms around every sublayer."""
+    specs = [_famepel_layer(li, e, c["layers"]) for li, e in enumerate(c["layers"])]
+    att = next((s for s in specs if s.mixer == "latent"), specs[0])
+    return ModelConfig(arch=LAYERED_ARCHS[c["architecture"]], layer_specs=specs, hidden=int(c["width"]), vocab=int(c["vocab"]), n_heads=att.n_heads, n_kv_heads=1,
+                       head_dim=att.head_dim, ffn=max((s.moe.ffn for s in specs if s.moe), default=0), rms_eps=float(c["norm"]["eps"]), qk_norm=False,
+                       norm_kind="dyt", post_norm=True, embed_scale=float(c["embedding"]["scale"]))
+
+
 def _layered_config(c: dict, path: str) -> ModelConfig:
+    if c["architecture"] == "Famepel":
+        return _famepel_config(c)
+    return _zogavik_config(c, path)
+
+
+def _zogavik_config(c: dict, path: str) -> ModelConfig:
     """config.json of a model described layer by layer: ``layers`` (each with its mixer's type and sizes and its feed-forward), ``loop``,
     ``norm``, ``vocab``, ``width``, ``logit_scale``."""
     src = LayeredSource(path)
@@ -691,32 +769,96 @@ def _save_layered(cfg: ModelConfig, src, path: str) -> None:
     def put(name, shape):
         out[LayeredSource.file_name(name)] = src.get(name, shape).to(torch.bfloat16)
 
+    def put_norm(name):
+        put(name + ".weight", (h,))
+        if cfg.norm_kind == "dyt":
+            put(name + ".bias", (h,))
+            put(name + ".alpha", ())
+
     put("token_embd.weight", (cfg.vocab, h))
-    put("output_norm.weight", (h,))
+    put_norm("output_norm")
+    if not cfg.tie_embeddings:
+        put("output.weight", (cfg.vocab, h))
     if cfg.loop is not None:
         put("loop_step.weight", (cfg.loop.times, h))
     layers = []
     for li, sp in enumerate(cfg.layer_specs):
-        p, nv = f"blk.{li}.", sp.n_heads * sp.v_dim
-        put(p + "attn_norm.weight", (h,))
-        if sp.mixer == "lightning":
-            for nm, shp in (("lin_q", (sp.q_dim, h)), ("lin_k", (sp.q_dim, h)), ("lin_v", (nv, h)), ("lin_gate", (nv, h)), ("lin_norm", (nv,)), ("lin_out", (h, nv))):
-                put(p + nm + ".weight", shp)
-            m = {"heads": sp.n_heads, "dim": sp.head_dim, "vdim": sp.v_dim, "decay": list(sp.decay)}
-        else:
-            for c, n in (("q", sp.q_dim), ("k", sp.n_kv_heads * sp.head_dim), ("v", sp.n_kv_heads * sp.v_dim)):
-                put(p + f"attn_{c}.weight", (n, h))
-                put(p + f"attn_{c}.bias", (n,))
-            put(p + "attn_rel.weight", (sp.rel_buckets, sp.n_heads))
-            put(p + "attn_output.weight", (h, nv))
-            m = {"heads": sp.n_heads, "kv_heads": sp.n_kv_heads, "dim": sp.head_dim, "vdim": sp.v_dim, "scale": sp.scale, "bias_max": sp.rel_max,
-                 "mask": {"size": sp.window, "keep_first": sp.keep_first} if sp.window else None}
+        p = f"blk.{li}."
+        for nm, present in (("attn", True), ("ffn", sp.has_ffn)):
+            if present:
+                put_norm(p + nm + "_norm")
+                if cfg.post_norm:
+                    put_norm(p + nm + "_post_norm")
+                    put(p + nm + "_post_scale.weight", (h,))
+        for nm, shp in mixer_tensors(sp, h):
+            put(p + nm, shp)
         if sp.ffn:
-            put(p + "ffn_norm.weight", (h,))
             put(p + "ffn_gate.weight", (sp.ffn, h)); put(p + "ffn_up.weight", (sp.ffn, h)); put(p + "ffn_down.weight", (h, sp.ffn))
-        layers.append({"type": sp.mixer, "mixer": m, "mlp": {"kind": "dense", "ff": sp.ffn} if sp.ffn else None})
+        if sp.moe is not None:
+            put(p + "ffn_gate_inp.weight", (sp.moe.n_experts, h))
+            for e in range(sp.moe.n_experts):
+                for nm, shp in (("gate", (sp.moe.ffn, h)), ("up", (sp.moe.ffn, h)), ("down", (h, sp.moe.ffn))):
+                    name = f"ffn_{nm}_exps.weight"
+                    out[LayeredSource.file_name(f"{p}{name}#{e}")] = src.get_expert(p + name, e, shp).to(torch.bfloat16)
+        layers.append({"type": {"latent": "latent_attention"}.get(sp.mixer, sp.mixer), "mixer": _mixer_config(sp), "mlp": _ffn_config(sp)})
     save_safetensors(out, os.path.join(path, "model.safetensors"))
     name = {v: k for k, v in LAYERED_ARCHS.items()}[cfg.arch]
+    c = {"architecture": name, "layers": layers, "vocab": cfg.vocab, "width": h, "norm": {"eps": cfg.rms_eps}}
+    if cfg.arch == "famepel":
+        c["embedding"] = {"scale": cfg.embed_scale}
+    else:
+        c["logit_scale"] = cfg.logit_scale
+        c["loop"] = {"start": cfg.loop.start, "stop": cfg.loop.stop, "times": cfg.loop.times} if cfg.loop else None
     with open(os.path.join(path, "config.json"), "w") as fh:
-        json.dump({"architecture": name, "layers": layers, "vocab": cfg.vocab, "width": h, "norm": {"eps": cfg.rms_eps}, "logit_scale": cfg.logit_scale,
-                   "loop": {"start": cfg.loop.start, "stop": cfg.loop.stop, "times": cfg.loop.times} if cfg.loop else None}, fh)
+        json.dump(c, fh)
+
+
+def mixer_tensors(sp: LayerSpec, h: int):
+    """(builder's name, shape) of a mixer's tensors."""
+    nq, nv = sp.q_dim, sp.n_heads * sp.v_dim
+    if sp.mixer == "lightning":
+        return [("lin_q.weight", (nq, h)), ("lin_k.weight", (nq, h)), ("lin_v.weight", (nv, h)), ("lin_gate.weight", (nv, h)), ("lin_norm.weight", (nv,)),
+                ("lin_out.weight", (h, nv))]
+    if sp.mixer == "hgrn2":
+        return [("gla_q.weight", (nq, h)), ("gla_f.weight", (nq, h)), ("gla_f.bias", (nq,)), ("gla_lower", (nq,)), ("gla_v.weight", (nv, h)),
+                ("gla_norm.weight", (sp.v_dim,)), ("gla_out.weight", (h, nv))]
+    if sp.mixer == "mamba2":
+        ch, hd = sp.conv_channels, (sp.n_heads,)
+        return [("ssm_in.weight", (nv + ch + sp.n_heads, h)), ("ssm_conv1d.weight", (ch, sp.conv_taps)), ("ssm_conv1d.bias", (ch,)), ("ssm_dt.bias", hd),
+                ("ssm_a_log", hd), ("ssm_d", hd), ("ssm_norm.weight", (nv,)), ("ssm_out.weight", (h, nv))]
+    if sp.mixer == "latent":
+        own = [] if sp.kv_from >= 0 else [("attn_kv_a.weight", (sp.kv_rank + sp.rot_dim, h)), ("attn_kv_a_norm.weight", (sp.kv_rank,))]
+        return own + [("attn_q_a.weight", (sp.q_rank, h)), ("attn_q_a_norm.weight", (sp.q_rank,)),
+                      ("attn_q_b.weight", (sp.n_heads * (sp.head_dim + sp.rot_dim), sp.q_rank)), ("attn_k_b.weight", (nq, sp.kv_rank)),
+                      ("attn_v_b.weight", (nv, sp.kv_rank)), ("attn_sink", (sp.n_heads,)), ("attn_output.weight", (h, nv))]
+    own = []
+    for c, n in (("q", nq), ("k", sp.n_kv_heads * sp.head_dim), ("v", sp.n_kv_heads * sp.v_dim)):
+        own += [(f"attn_{c}.weight", (n, h)), (f"attn_{c}.bias", (n,))]
+    return own + [("attn_rel.weight", (sp.rel_buckets, sp.n_heads)), ("attn_output.weight", (h, nv))]
+
+
+def _mixer_config(sp: LayerSpec) -> dict:
+    m = {"heads": sp.n_heads, "vdim": sp.v_dim}
+    if sp.mixer == "lightning":
+        return {**m, "dim": sp.head_dim, "decay": list(sp.decay)}
+    if sp.mixer == "hgrn2":
+        return {**m, "dim": sp.head_dim}
+    if sp.mixer == "mamba2":
+        return {**m, "state": sp.head_dim, "groups": sp.state_groups, "conv": sp.conv_taps, "norm_groups": sp.norm_parts}
+    if sp.mixer == "latent":
+        r = sp.rotary
+        rot = {"dims": r.dims, "base": r.base}
+        if r.factor > 0:
+            rot["scaling"] = {"factor": r.factor, "original": r.original, "fast": r.fast, "slow": r.slow}
+        m = {**m, "dim": sp.head_dim, "rot_dim": sp.rot_dim, "kv_rank": sp.kv_rank, "q_rank": sp.q_rank, "scale": sp.scale, "rot": rot}
+        return {**m, "kv_from": sp.kv_from} if sp.kv_from >= 0 else m
+    return {**m, "kv_heads": sp.n_kv_heads, "dim": sp.head_dim, "scale": sp.scale, "bias_max": sp.rel_max,
+            "mask": {"size": sp.window, "keep_first": sp.keep_first} if sp.window else None}
+
+
+def _ffn_config(sp: LayerSpec):
+    if sp.moe is not None:
+        r = sp.moe
+        return {"kind": "moe", "expert": {"ff": r.ffn}, "router": {"experts": r.n_experts, "top": r.top, "scale": r.scale,
+                                                                  "groups": {"count": r.groups, "keep": r.groups_kept}}}
+    return {"kind": "dense", "ff": sp.ffn} if sp.ffn else None
