@@ -2,9 +2,12 @@
 //   embed_f32           rows of a bf16 / f32 embedding table -> f32 stream
 //   stream_norm         stream += pending update (bf16, f32, or K-split fp32 partial sums of a projection) [+ a vector added to
 //                       every row], then RMSNorm of the row with an f32 weight -> bf16 or f32 rows for the next projection
+//   stream_dyt          the same with Dynamic Tanh, tanh(alpha x) w + b, in place of the norm, and one of its own over the update, which
+//                       may also be the router-weighted sum of expert outputs (formed here)
 //   qk_unit_store       fused Q | K | V rows -> Q / K divided by their root mean square per head (no weight), K / V into their
 //                       cache slots, Q scaled and laid out for the attention kernels
 //   gated_norm          RMSNorm over all heads' outputs together, times sigmoid(gate): the tail of a linear-attention mixer
+//   part_norm           RMSNorm of equal parts of a row, after SiLU(gate) if there is one: the tail of Mamba-2 and HGRN2 mixers
 //   act_mul             act(gate) * up of f32 rows (the 32-bit path; the bf16 path has it in the GEMM epilogue)
 // One pass over HBM each; sizes are arbitrary (vector paths when they divide).  Output rows may be wider than the data (padding to
 // the 16-byte row pitch the TMA descriptors of the next GEMM need); the padding is written as zero.
@@ -46,13 +49,13 @@ __device__ __forceinline__ float block_sum_256(float v, float* red) {
 
 // ------------------------------------------------------------------------------------------ embed
 template <typename T>
-__global__ void embed_f32_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out, int width, int vocab) {
+__global__ void embed_f32_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out, int width, int vocab, float scale) {
   pdl_wait();
   pdl_trigger();
   const int t = blockIdx.x;
   int id = ids[t];
   if (id < 0 || id >= vocab) id = 0;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) out[(size_t)t * width + i] = ld_f(table + (size_t)id * width + i);
+  for (int i = threadIdx.x; i < width; i += blockDim.x) out[(size_t)t * width + i] = ld_f(table + (size_t)id * width + i) * scale;
 }
 
 // ------------------------------------------------------------------------------------------ stream norm
@@ -144,6 +147,92 @@ stream_norm_any_kernel(const StreamNormArgs a) {
   TO* o = (TO*)a.out + r * a.ld_out;
   for (int c = threadIdx.x; c < a.width; c += 256) st_f(o + c, (in_place ? x[c] : value(c)) * inv * a.weight[c]);
   for (int c = a.width + threadIdx.x; c < a.ld_out; c += 256) st_f(o + c, 0.f);
+}
+
+// ------------------------------------------------------------------------------------------ stream with Dynamic Tanh
+struct DytArgs {
+  float* x;                     // stream [rows, width]
+  const void* delta;            // update: f32 / bf16 [n_part][rows, ld_delta], or expert outputs [*, ld_delta] when pair_row is set; null = none
+  int n_part; long part_stride; int ld_delta;
+  const int* pair_row; const float* weights; int k;      // update of row r = sum_j weights[r k + j] * delta[pair_row[r k + j]] (negative row: nothing)
+  float post_alpha; const float* post_w; const float* post_b;   // the update passes tanh(alpha u) w + b before it is added; null = it does not
+  float alpha; const float* w; const float* b;
+  const long long* rows;        // as in StreamNormArgs
+  void* out; int ld_out;        // null = only update the stream
+  int width;
+};
+
+__device__ __forceinline__ float dyt(float x, float alpha, float w, float b) { return fmaf(tanhf(alpha * x), w, b); }
+
+// One thread per V neighbouring columns of a row (nothing is reduced over a row).
+template <typename TD, typename TO, int V>
+__global__ void __launch_bounds__(256)
+stream_dyt_kernel(const DytArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
+  const int c = (blockIdx.y * 256 + threadIdx.x) * V;
+  const int end = a.out != nullptr ? a.ld_out : a.width;
+  if (c >= end) return;
+  if (c >= a.width) {                              // padding (width % V == 0)
+#pragma unroll
+    for (int i = 0; i < V; ++i) if (c + i < end) st_f((TO*)a.out + r * a.ld_out + c + i, 0.f);
+    return;
+  }
+  float x[V];
+  auto load = [&](const auto* p, float* v) {
+    if constexpr (V == 4) { const float4 q = ld4(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+    else v[0] = ld_f(p);
+  };
+  load(a.x + src * a.width + c, x);
+  if (a.delta != nullptr) {
+    float u[V];
+    if (a.pair_row != nullptr) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) u[i] = 0.f;
+      const int* pr = a.pair_row + src * a.k;
+      for (int j = 0; j < a.k; ++j) {
+        const int row = pr[j];
+        if (row < 0) continue;
+        const float w = a.weights[src * a.k + j];
+        float q[V];
+        load((const TD*)a.delta + (size_t)row * a.ld_delta + c, q);
+#pragma unroll
+        for (int i = 0; i < V; ++i) u[i] = fmaf(w, q[i], u[i]);
+      }
+    } else {
+      const TD* d = (const TD*)a.delta + src * a.ld_delta + c;
+      load(d, u);
+      for (int p = 1; p < a.n_part; ++p) {
+        float q[V];
+        load(d + (size_t)p * a.part_stride, q);
+#pragma unroll
+        for (int i = 0; i < V; ++i) u[i] += q[i];
+      }
+    }
+    if (a.post_w != nullptr) {
+      float w[V], b[V];
+      load(a.post_w + c, w);
+      load(a.post_b + c, b);
+#pragma unroll
+      for (int i = 0; i < V; ++i) u[i] = dyt(u[i], a.post_alpha, w[i], b[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) x[i] += u[i];
+    if (a.rows == nullptr) {
+      if constexpr (V == 4) st4(a.x + src * a.width + c, make_float4(x[0], x[1], x[2], x[3]));
+      else a.x[src * a.width + c] = x[0];
+    }
+  }
+  if (a.out == nullptr) return;
+  float w[V], b[V];
+  load(a.w + c, w);
+  load(a.b + c, b);
+  TO* o = (TO*)a.out + r * a.ld_out + c;
+#pragma unroll
+  for (int i = 0; i < V; ++i) x[i] = dyt(x[i], a.alpha, w[i], b[i]);
+  if constexpr (V == 4) st4(o, make_float4(x[0], x[1], x[2], x[3]));
+  else st_f(o, x[0]);
 }
 
 // ------------------------------------------------------------------------------------------ Q / K unit norm + cache store
@@ -277,6 +366,58 @@ gated_norm_any_kernel(const GatedNormArgs a) {
   for (int c = a.n + threadIdx.x; c < a.ld_out; c += 256) st_f(out + c, 0.f);
 }
 
+// ------------------------------------------------------------------------------------------ norm of equal parts
+struct PartNormArgs {
+  const float* o; int ld_o;     // [rows, n] f32
+  const void* gate; int n_part; long part_stride; int ld_gate;     // gate pre-activations (null = none)
+  const float* weight; int n_weight;   // f32, column c uses weight[c % n_weight]
+  void* out; int ld_out; int n, parts; float eps; long items;
+};
+
+// G threads (a warp or a CTA) per (row, part).
+template <typename TG, typename TO, int G>
+__global__ void __launch_bounds__(256)
+part_norm_kernel(const PartNormArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[8];
+  constexpr int kKeep = 8;                         // values per thread kept in registers
+  const long item = (long)blockIdx.x * (256 / G) + threadIdx.x / G;
+  const bool live = item < a.items;
+  const long r = live ? item / a.parts : 0;
+  const int part = live ? (int)(item - r * a.parts) : 0, lane = threadIdx.x % G;
+  const int len = a.n / a.parts, c0 = part * len;
+  const float* o = a.o + (size_t)r * a.ld_o + c0;
+  const TG* g = a.gate != nullptr ? (const TG*)a.gate + (size_t)r * a.ld_gate + c0 : nullptr;
+  auto value = [&](int c) {
+    float v = o[c];
+    if (g != nullptr) {
+      float z = ld_f(g + c);
+      for (int p = 1; p < a.n_part; ++p) z += ld_f(g + (size_t)p * a.part_stride + c);
+      v *= z / (1.0f + expf(-z));
+    }
+    return v;
+  };
+  float keep[kKeep];
+  float ss = 0.f;
+  if (live) {
+#pragma unroll
+    for (int i = 0; i < kKeep; ++i) { const int c = lane + i * G; if (c < len) { keep[i] = value(c); ss += keep[i] * keep[i]; } }
+    for (int c = lane + kKeep * G; c < len; c += G) { const float v = value(c); ss += v * v; }
+  }
+  if constexpr (G == 32) ss = warp_sum(ss);
+  else ss = block_sum_256(ss, red);
+  if (!live) return;
+  const float inv = 1.0f / sqrtf(ss / (float)len + a.eps);
+  TO* out = (TO*)a.out + (size_t)r * a.ld_out;
+  auto w = [&](int c) { return a.weight[(c0 + c) % a.n_weight]; };
+#pragma unroll
+  for (int i = 0; i < kKeep; ++i) { const int c = lane + i * G; if (c < len) st_f(out + c0 + c, keep[i] * inv * w(c)); }
+  for (int c = lane + kKeep * G; c < len; c += G) st_f(out + c0 + c, value(c) * inv * w(c));
+  if (part == a.parts - 1)
+    for (int c = a.n + lane; c < a.ld_out; c += G) st_f(out + c, 0.f);
+}
+
 // ------------------------------------------------------------------------------------------ act(gate) * up, f32
 __global__ void act_mul_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, long n, int inter, int ld, int act) {
   pdl_wait();
@@ -294,10 +435,11 @@ __global__ void act_mul_f32_kernel(const float* __restrict__ gu, float* __restri
 
 using namespace gb;
 
-GB_API int gb_embed_f32(const int* ids, const void* table, int table_f32, float* out, int n_tok, int width, int vocab, cudaStream_t stream) {
+GB_API int gb_embed_f32(const int* ids, const void* table, int table_f32, float* out, int n_tok, int width, int vocab, float scale,
+                        cudaStream_t stream) {
   if (n_tok <= 0) return 0;
-  if (table_f32) launch_k(embed_f32_kernel<float>, (unsigned)n_tok, 256, 0, stream, ids, (const float*)table, out, width, vocab);
-  else launch_k(embed_f32_kernel<__nv_bfloat16>, (unsigned)n_tok, 256, 0, stream, ids, (const __nv_bfloat16*)table, out, width, vocab);
+  if (table_f32) launch_k(embed_f32_kernel<float>, (unsigned)n_tok, 256, 0, stream, ids, (const float*)table, out, width, vocab, scale);
+  else launch_k(embed_f32_kernel<__nv_bfloat16>, (unsigned)n_tok, 256, 0, stream, ids, (const __nv_bfloat16*)table, out, width, vocab, scale);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -327,6 +469,53 @@ GB_API int gb_stream_norm(float* x, const void* delta, int delta_f32, int n_part
   a.out = out; a.ld_out = ld_out; a.width = width; a.eps = eps;
   if (delta_f32) return out_f32 ? stream_norm_launch<float, float>(a, n_rows, stream) : stream_norm_launch<float, __nv_bfloat16>(a, n_rows, stream);
   return out_f32 ? stream_norm_launch<__nv_bfloat16, float>(a, n_rows, stream) : stream_norm_launch<__nv_bfloat16, __nv_bfloat16>(a, n_rows, stream);
+}
+
+template <typename TD, typename TO>
+static int stream_dyt_launch(const DytArgs& a, int n_rows, cudaStream_t stream) {
+  const size_t ed = sizeof(TD) * 4, eo = sizeof(TO) * 4;
+  const auto ok16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  const bool vec = a.width % 4 == 0 && (a.delta == nullptr || (a.ld_delta % 4 == 0 && a.part_stride % 4 == 0 && (uintptr_t)a.delta % ed == 0)) &&
+                   (a.out == nullptr || (a.ld_out % 4 == 0 && (uintptr_t)a.out % eo == 0)) && ok16(a.x) && ok16(a.w) && ok16(a.b) && ok16(a.post_w) && ok16(a.post_b);
+  const int cols = a.out != nullptr ? a.ld_out : a.width;
+  if (vec) launch_k(stream_dyt_kernel<TD, TO, 4>, dim3((unsigned)n_rows, (unsigned)((cols + 1023) / 1024)), 256, 0, stream, a);
+  else launch_k(stream_dyt_kernel<TD, TO, 1>, dim3((unsigned)n_rows, (unsigned)((cols + 255) / 256)), 256, 0, stream, a);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// See DytArgs.
+GB_API int gb_stream_dyt(float* x, const void* delta, int delta_f32, int n_part, long part_stride, int ld_delta, const int* pair_row, const float* weights, int k,
+                         float post_alpha, const float* post_w, const float* post_b, float alpha, const float* w, const float* b, const long long* rows, void* out,
+                         int out_f32, int ld_out, int n_rows, int width, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (width <= 0 || (out != nullptr && (ld_out < width || w == nullptr || b == nullptr)) || (delta != nullptr && (ld_delta < width || n_part < 1)) ||
+      (pair_row != nullptr && (weights == nullptr || k < 1)) || (post_w != nullptr && post_b == nullptr))
+    return fail("stream_dyt: bad arguments%s");
+  DytArgs a;
+  a.x = x; a.delta = delta; a.n_part = n_part; a.part_stride = part_stride; a.ld_delta = ld_delta; a.pair_row = pair_row; a.weights = weights; a.k = k;
+  a.post_alpha = post_alpha; a.post_w = post_w; a.post_b = post_b; a.alpha = alpha; a.w = w; a.b = b; a.rows = rows; a.out = out; a.ld_out = ld_out; a.width = width;
+  if (delta_f32) return out_f32 ? stream_dyt_launch<float, float>(a, n_rows, stream) : stream_dyt_launch<float, __nv_bfloat16>(a, n_rows, stream);
+  return out_f32 ? stream_dyt_launch<__nv_bfloat16, float>(a, n_rows, stream) : stream_dyt_launch<__nv_bfloat16, __nv_bfloat16>(a, n_rows, stream);
+}
+
+template <typename TG, typename TO>
+static int part_norm_launch(const PartNormArgs& a, cudaStream_t stream) {
+  if (a.n / a.parts <= 512) launch_k(part_norm_kernel<TG, TO, 32>, (unsigned)((a.items + 7) / 8), 256, 0, stream, a);
+  else launch_k(part_norm_kernel<TG, TO, 256>, (unsigned)a.items, 256, 0, stream, a);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+GB_API int gb_part_norm(const float* o, int ld_o, const void* gate, int gate_f32, int n_part, long part_stride, int ld_gate, const float* weight, int n_weight,
+                        void* out, int out_f32, int ld_out, int rows, int n, int parts, float eps, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (n < 1 || parts < 1 || n % parts || n_weight < 1 || n % n_weight || ld_o < n || ld_out < n || n_part < 1) return fail("part_norm: bad sizes%s");
+  PartNormArgs a;
+  a.o = o; a.ld_o = ld_o; a.gate = gate; a.n_part = n_part; a.part_stride = part_stride; a.ld_gate = ld_gate; a.weight = weight; a.n_weight = n_weight;
+  a.out = out; a.ld_out = ld_out; a.n = n; a.parts = parts; a.eps = eps; a.items = (long)rows * parts;
+  if (gate_f32) return out_f32 ? part_norm_launch<float, float>(a, stream) : part_norm_launch<float, __nv_bfloat16>(a, stream);
+  return out_f32 ? part_norm_launch<__nv_bfloat16, float>(a, stream) : part_norm_launch<__nv_bfloat16, __nv_bfloat16>(a, stream);
 }
 
 // See QkUnitArgs.  in_f32: element type of qkv; cache_f32: element type of q_out and the caches.

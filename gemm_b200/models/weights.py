@@ -23,8 +23,8 @@ import torch
 
 from ..ops import elementwise as ew
 from ..ops import mxfp8
-from ..ops.attention import cache_head_dims, distance_bias_table
-from ..ops.stream import row_width
+from ..ops.attention import LOG2E, cache_head_dims, distance_bias_table
+from ..ops.stream import DynTanh, row_width
 from ..ops.mxfp8 import MxTensor
 from .config import ModelConfig
 
@@ -65,6 +65,11 @@ class LinearWeight:
         else:
             self.mx.tiled = True
         return self
+
+    def rows(self, a: int, b: int) -> "LinearWeight":
+        """The features ``a .. b - 1`` as a projection of their own (a view; of a tiled matrix ``a`` and ``b`` are multiples of 128, or ``b`` is its end)."""
+        assert self.fmt in ("bf16", "f32") and not self.groups and (not self.tiled or (a % 128 == 0 and (b % 128 == 0 or b == self.n)))
+        return LinearWeight(self.fmt, b - a, self.k, w=self.w[a:b], bias=self.bias[a:b] if self.bias is not None else None, tiled=self.tiled)
 
     def untiled_data(self) -> torch.Tensor:
         """Row-major copy of the stored matrix (bf16 values or e4m3 bytes)."""
@@ -227,8 +232,61 @@ class LightningWeights:
 
 
 @dataclass
+class Mamba2Weights:
+    """A Mamba-2 mixer.  ``w_in`` rows: [z | x | B | C], padding up to ``dt_row`` (a multiple of 128), [dt]."""
+    w_in: LinearWeight
+    dt_row: int
+    conv_w: torch.Tensor          # f32 [channels, taps]
+    conv_b: torch.Tensor          # f32 [channels]
+    dt_bias: torch.Tensor         # f32 [heads]
+    a: torch.Tensor               # f32 [heads]: the state decays by exp(a dt)
+    d: torch.Tensor               # f32 [heads]
+    norm: torch.Tensor            # f32 [heads * v_dim]
+    w_out: LinearWeight
+
+    def to(self, device) -> "Mamba2Weights":
+        return Mamba2Weights(self.w_in.to(device), self.dt_row, *(t.to(device) for t in (self.conv_w, self.conv_b, self.dt_bias, self.a, self.d, self.norm)),
+                             self.w_out.to(device))
+
+
+@dataclass
+class GlaWeights:
+    """A linear-attention mixer with a forget gate per key channel (HGRN2).  ``w_in`` rows: [q | v], padding up to ``f_row`` (a multiple of 128),
+    [f]."""
+    w_in: LinearWeight
+    f_row: int
+    f_bias: torch.Tensor          # f32 [heads * dim]
+    lower: torch.Tensor           # f32 [heads * dim]
+    norm: torch.Tensor            # f32 [v_dim]
+    w_out: LinearWeight
+
+    def to(self, device) -> "GlaWeights":
+        return GlaWeights(self.w_in.to(device), self.f_row, self.f_bias.to(device), self.lower.to(device), self.norm.to(device), self.w_out.to(device))
+
+
+@dataclass
+class LatentWeights:
+    """A latent-attention mixer.  ``w_kv`` expands cached latents to all heads' keys and values (prompts); ``w_uk`` / ``w_uv`` are the same matrices
+    head by head, for attention over the latents themselves (decoding)."""
+    w_a: LinearWeight             # rows [q latent | kv latent | rotated key part], or [q latent] alone
+    q_norm: torch.Tensor          # f32 [q_rank]
+    kv_norm: Optional[torch.Tensor]   # f32 [kv_rank]
+    w_qb: LinearWeight            # [heads * (dim + rot_dim), q_rank]
+    w_kv: Optional[LinearWeight]  # rows [heads * dim ; heads * v_dim], each head padded to 8 rows (bf16 only)
+    w_uk: LinearWeight            # per head [rank, dim]
+    w_uv: LinearWeight            # per head [v_dim, rank]
+    sink: torch.Tensor            # f32 [heads], times log2 e
+    freq: torch.Tensor            # f64 [rot_dim / 2] rotary frequencies
+
+    def to(self, device) -> "LatentWeights":
+        mv = lambda t: t.to(device) if t is not None else None
+        return LatentWeights(self.w_a.to(device), mv(self.q_norm), mv(self.kv_norm), self.w_qb.to(device), mv(self.w_kv), self.w_uk.to(device), self.w_uv.to(device),
+                             mv(self.sink), mv(self.freq))
+
+
+@dataclass
 class LayerWeights:
-    attn_norm: torch.Tensor
+    attn_norm: torch.Tensor                       # or DynTanh
     wqkv: Optional[LinearWeight]                  # rows [Q ; K ; V] (+ [gate] after V when the attention output is gated); None in SSM layers
     wo: Optional[LinearWeight]
     ffn_norm: torch.Tensor
@@ -246,13 +304,20 @@ class LayerWeights:
     sh_gate: Optional[torch.Tensor] = None        # bf16 [1, H]: sigmoid gate of the shared expert (absent = ungated)
     lin: Optional[LightningWeights] = None        # lightning-attention layer (then wqkv / wo are None)
     rel_bias: Optional[torch.Tensor] = None       # f32 [heads, 2 N] distance bias (ops.attention.distance_bias_table)
+    attn_post: Optional[DynTanh] = None           # norm of the mixer's / feed-forward's result, with its per-channel scale folded in
+    ffn_post: Optional[DynTanh] = None
+    mamba: Optional[Mamba2Weights] = None
+    gla: Optional[GlaWeights] = None
+    latent: Optional[LatentWeights] = None        # (the output projection is wo)
 
     def linears(self) -> List[LinearWeight]:
         """Every projection matrix of the layer."""
         own = [self.wqkv, self.wo, self.w_gate_up, self.w_down, self.w13, self.w2, self.sh_gate_up, self.sh_down]
-        for part in (self.ssm, self.lin):
+        for part in (self.ssm, self.lin, self.mamba, self.gla):
             if part is not None:
                 own += [part.w_in, part.w_out]
+        if self.latent is not None:
+            own += [self.latent.w_a, self.latent.w_qb, self.latent.w_kv, self.latent.w_uk, self.latent.w_uv]
         return [lw for lw in own if lw is not None]
 
 
@@ -282,7 +347,8 @@ class ModelWeights:
         layers = [LayerWeights(attn_norm=mv(l.attn_norm), wqkv=mv(l.wqkv), wo=mv(l.wo), ffn_norm=mv(l.ffn_norm), q_norm=mv(l.q_norm),
                                k_norm=mv(l.k_norm), w_gate_up=mv(l.w_gate_up), w_down=mv(l.w_down), router=mv(l.router),
                                router_bias=mv(l.router_bias), w13=mv(l.w13), w2=mv(l.w2), ssm=mv(l.ssm), sh_gate_up=mv(l.sh_gate_up),
-                               sh_down=mv(l.sh_down), sh_gate=mv(l.sh_gate), lin=mv(l.lin), rel_bias=mv(l.rel_bias)) for l in self.layers]
+                               sh_down=mv(l.sh_down), sh_gate=mv(l.sh_gate), lin=mv(l.lin), rel_bias=mv(l.rel_bias), attn_post=mv(l.attn_post),
+                               ffn_post=mv(l.ffn_post), mamba=mv(l.mamba), gla=mv(l.gla), latent=mv(l.latent)) for l in self.layers]
         return ModelWeights(cfg=self.cfg, embed=mv(self.embed), layers=layers, final_norm=mv(self.final_norm), lm_head=mv(self.lm_head),
                             fmt=self.fmt, tp_rank=self.tp_rank, tp_size=self.tp_size, ep_rank=self.ep_rank, ep_size=self.ep_size,
                             vocab_start=self.vocab_start, loop_step=mv(self.loop_step))
@@ -340,6 +406,16 @@ class RandomSource:
         return True
 
     def get(self, name: str, shape) -> torch.Tensor:
+        if name.endswith(".alpha"):
+            return torch.full(tuple(shape), 0.75, dtype=torch.bfloat16, device=self.device)
+        if name.endswith("post_scale.weight"):
+            return torch.full(tuple(shape), 0.25, dtype=torch.bfloat16, device=self.device)
+        if name.endswith("ssm_a_log"):                   # decay rates 1 .. 16 over the heads
+            return torch.linspace(0.0, 2.75, shape[0], device=self.device).to(torch.bfloat16)
+        if self.cfg.is_layered and name.endswith("ssm_dt.bias"):
+            return (self._randn(name, shape).float() * 25 - 3.0).to(torch.bfloat16)
+        if name.endswith("gla_lower"):
+            return (self._randn(name, shape).float() * 5 + 0.5).clamp(0.0, 0.95).to(torch.bfloat16)
         if name.endswith("norm.weight") and not name.endswith("lin_norm.weight") and self.cfg.norm_offset:
             return torch.full(tuple(shape), 1.0 - self.cfg.norm_offset, dtype=torch.bfloat16, device=self.device)
         if name.endswith("norm.weight"):
@@ -501,67 +577,170 @@ def build_weights(cfg: ModelConfig, src, fmt: str = "bf16", device="cuda", tp_ra
     return mw
 
 
-def _padded_linear(t: torch.Tensor, fmt: str, dev, rows: int = 0, bias: Optional[torch.Tensor] = None) -> LinearWeight:
-    """A projection whose input rows are padded the way ``ops.stream`` pads them (``row_width``); ``rows`` pads the output features too.
-    The padding is zero."""
+def _padded_linear(t: torch.Tensor, fmt: str, dev, bias: Optional[torch.Tensor] = None, groups: int = 0) -> LinearWeight:
+    """A projection whose input rows are padded with zeros the way ``ops.stream`` pads them (``row_width``).  ``groups``: ``t`` is stacked group by
+    group."""
     k = row_width(t.shape[1], torch.float32 if fmt == "f32" else torch.bfloat16)
-    rows = rows or t.shape[0]
-    if (rows, k) != tuple(t.shape):
-        t = torch.nn.functional.pad(t, (0, k - t.shape[1], 0, rows - t.shape[0]))
-    return make_linear(t.to(dev), fmt, bias=bias)
+    if k != t.shape[1]:
+        t = torch.nn.functional.pad(t, (0, k - t.shape[1]))
+    return make_linear(t.to(dev), fmt, bias=bias, groups=groups)
+
+
+def _stack_at_128(a: torch.Tensor, b: torch.Tensor):
+    """Rows of ``b`` behind those of ``a``, starting at a multiple of 128 (so that either part is a projection of its own in the tiled layout), the
+    whole padded to a multiple of 128.  Returns (stack, first row of b)."""
+    at = (a.shape[0] + 127) // 128 * 128
+    out = torch.zeros((at + b.shape[0] + 127) // 128 * 128, a.shape[1], dtype=a.dtype, device=a.device)
+    out[: a.shape[0]] = a
+    out[at: at + b.shape[0]] = b
+    return out, at
+
+
+class _LayeredBuilder:
+    """Weights of a model described layer by layer.  Norm weights become f32 ``offset + w``; the factor of the logits is folded into the
+    final norm's weight, the per-channel scale behind a post norm into that norm."""
+
+    def __init__(self, cfg: ModelConfig, src, fmt: str, dev):
+        self.cfg, self.src, self.fmt, self.dev, self.exact = cfg, src, fmt, dev, fmt == "f32"
+        self.h = cfg.hidden
+
+    def get(self, name, *shape):
+        return self.src.get(name, shape)
+
+    def f32(self, name, *shape):
+        return self.get(name, *shape).float().contiguous().to(self.dev)
+
+    def linear(self, t, **kw) -> LinearWeight:
+        return _padded_linear(t, self.fmt, self.dev, **kw)
+
+    def norm(self, name, scale=None):
+        """A norm over the stream; ``scale``: name of a per-channel factor of its result."""
+        w = (self.get(name + ".weight", self.h).float() + self.cfg.norm_offset).contiguous().to(self.dev)
+        if self.cfg.norm_kind == "rms":
+            return w
+        b = self.f32(name + ".bias", self.h)
+        if scale is not None:
+            s = self.f32(scale, self.h)
+            w, b = w * s, b * s                      # products of bf16 values: exact in f32
+        return DynTanh(float(self.get(name + ".alpha").float()), w, b)
+
+    def lightning(self, pre, sp, lw):
+        h, nv = self.h, sp.n_heads * sp.v_dim
+        w_in = torch.cat([self.get(pre + "lin_q.weight", sp.q_dim, h), self.get(pre + "lin_k.weight", sp.q_dim, h),
+                          self.get(pre + "lin_v.weight", nv, h), self.get(pre + "lin_gate.weight", nv, h)])
+        lw.lin = LightningWeights(w_in=self.linear(w_in), decay=torch.tensor(sp.decay, dtype=torch.float32, device=self.dev),
+                                  norm=self.f32(pre + "lin_norm.weight", nv), w_out=self.linear(self.get(pre + "lin_out.weight", h, nv)))
+
+    def mamba2(self, pre, sp, lw):
+        h, nv, ch = self.h, sp.n_heads * sp.v_dim, sp.conv_channels
+        w = self.get(pre + "ssm_in.weight", nv + ch + sp.n_heads, h)
+        w_in, at = _stack_at_128(w[: nv + ch], w[nv + ch:])
+        a = -torch.exp(self.get(pre + "ssm_a_log", sp.n_heads).double()).float().contiguous().to(self.dev)
+        lw.mamba = Mamba2Weights(w_in=self.linear(w_in), dt_row=at, conv_w=self.f32(pre + "ssm_conv1d.weight", ch, sp.conv_taps), conv_b=self.f32(pre + "ssm_conv1d.bias", ch),
+                                 dt_bias=self.f32(pre + "ssm_dt.bias", sp.n_heads), a=a, d=self.f32(pre + "ssm_d", sp.n_heads), norm=self.f32(pre + "ssm_norm.weight", nv),
+                                 w_out=self.linear(self.get(pre + "ssm_out.weight", h, nv)))
+
+    def hgrn2(self, pre, sp, lw):
+        h, nv = self.h, sp.n_heads * sp.v_dim
+        w_in, at = _stack_at_128(torch.cat([self.get(pre + "gla_q.weight", sp.q_dim, h), self.get(pre + "gla_v.weight", nv, h)]), self.get(pre + "gla_f.weight", sp.q_dim, h))
+        lw.gla = GlaWeights(w_in=self.linear(w_in), f_row=at, f_bias=self.f32(pre + "gla_f.bias", sp.q_dim), lower=self.f32(pre + "gla_lower", sp.q_dim),
+                            norm=self.f32(pre + "gla_norm.weight", sp.v_dim), w_out=self.linear(self.get(pre + "gla_out.weight", h, nv)))
+
+    def latent(self, pre, sp, lw):
+        h, hd, d, v, r, qr = self.h, sp.n_heads, sp.head_dim, sp.v_dim, sp.kv_rank, sp.q_rank
+        w_a = self.get(pre + "attn_q_a.weight", qr, h)
+        kv_norm = None
+        if sp.kv_from < 0:
+            w_a = torch.cat([w_a, self.get(pre + "attn_kv_a.weight", r + sp.rot_dim, h)])
+            kv_norm = self.f32(pre + "attn_kv_a_norm.weight", r)
+        uk, uv = self.get(pre + "attn_k_b.weight", hd * d, r).reshape(hd, d, r), self.get(pre + "attn_v_b.weight", hd * v, r).reshape(hd, v, r)
+        w_kv, pad = None, torch.nn.functional.pad
+        rows_k, v8 = r, v
+        if not self.exact:
+            d8, v8 = row_width(d, torch.bfloat16), row_width(v, torch.bfloat16)      # heads are padded; the output projection has zero columns there
+            uv = pad(uv, (0, 0, 0, v8 - v))
+            w_kv = self.linear(torch.cat([pad(uk, (0, 0, 0, d8 - d)).reshape(hd * d8, r), uv.reshape(hd * v8, r)]))
+            rows_k = (r + 127) // 128 * 128          # whole 128-row tiles per head
+        lw.latent = LatentWeights(
+            w_a=self.linear(w_a), q_norm=self.f32(pre + "attn_q_a_norm.weight", qr), kv_norm=kv_norm,
+            w_qb=self.linear(self.get(pre + "attn_q_b.weight", hd * (d + sp.rot_dim), qr)), w_kv=w_kv,
+            w_uk=self.linear(pad(uk.transpose(1, 2), (0, 0, 0, rows_k - r)).reshape(hd * rows_k, d), groups=hd),
+            w_uv=self.linear(uv.reshape(hd * v8, r), groups=hd),
+            sink=(self.get(pre + "attn_sink", hd).double() * LOG2E).float().contiguous().to(self.dev) if sp.sink else None,
+            freq=torch.tensor(sp.rotary.frequencies(), dtype=torch.float64, device=self.dev))
+        lw.wo = self.linear(pad(self.get(pre + "attn_output.weight", h, hd * v).reshape(h, hd, v), (0, v8 - v)).reshape(h, hd * v8))
+
+    def attention(self, pre, sp, lw):
+        h, nv = self.h, sp.n_heads * sp.v_dim
+        nk, nkv = sp.n_kv_heads * sp.head_dim, sp.n_kv_heads * sp.v_dim
+        w = torch.cat([self.get(pre + "attn_q.weight", sp.q_dim, h), self.get(pre + "attn_k.weight", nk, h), self.get(pre + "attn_v.weight", nkv, h)])
+        bias = None
+        if sp.qkv_bias:
+            bias = torch.cat([self.get(pre + f"attn_{c}.bias", n).float() for c, n in (("q", sp.q_dim), ("k", nk), ("v", nkv))]).contiguous().to(self.dev)
+        lw.wqkv = self.linear(w, bias=bias)
+        # the attention kernels emit heads of the cache's (padded) value width: the output projection has zero columns there
+        wo = self.get(pre + "attn_output.weight", h, nv)
+        dvp = cache_head_dims(sp.head_dim, sp.v_dim, torch.float32 if self.exact else torch.bfloat16)[1]
+        wo = torch.nn.functional.pad(wo.reshape(h, sp.n_heads, sp.v_dim), (0, dvp - sp.v_dim)).reshape(h, sp.n_heads * dvp)
+        lw.wo = self.linear(wo)
+        if sp.rel_buckets:
+            lw.rel_bias = distance_bias_table(self.get(pre + "attn_rel.weight", sp.rel_buckets, sp.n_heads).float().cpu(), sp.rel_max).to(self.dev)
+
+    def dense_ffn(self, pre, sp, lw):
+        h = self.h
+        wg, wu = self.get(pre + "ffn_gate.weight", sp.ffn, h), self.get(pre + "ffn_up.weight", sp.ffn, h)
+        wd = self.get(pre + "ffn_down.weight", h, sp.ffn)
+        fp = sp.ffn if self.exact else (sp.ffn + 127) // 128 * 128       # the gate / up GEMM works on whole 128-row tiles
+        pad = torch.nn.functional.pad
+        lw.w_gate_up = self.linear(torch.cat([pad(wg, (0, 0, 0, fp - sp.ffn)), pad(wu, (0, 0, 0, fp - sp.ffn))]))
+        lw.w_down = self.linear(pad(wd, (0, fp - sp.ffn)))
+
+    def moe_ffn(self, pre, sp, lw):
+        """Expert weights with the expert width and, per expert, the rows of the down projection padded to whole 128-row tiles (bf16)."""
+        h, m = self.h, sp.moe
+        dt = torch.float32 if self.exact else torch.bfloat16
+        up = lambda n: n if self.exact else (n + 127) // 128 * 128
+        k, ip, hp = row_width(h, dt), up(m.ffn), up(h)
+        lw.router = torch.nn.functional.pad(self.get(pre + "ffn_gate_inp.weight", m.n_experts, h).to(dt), (0, k - h)).contiguous().to(self.dev)
+        w13 = torch.zeros(m.n_experts, 2, ip, k, dtype=dt, device=self.dev)
+        w2 = torch.zeros(m.n_experts, hp, ip, dtype=dt, device=self.dev)
+        for e in range(m.n_experts):
+            w13[e, 0, : m.ffn, :h] = self.src.get_expert(pre + "ffn_gate_exps.weight", e, (m.ffn, h)).to(self.dev)
+            w13[e, 1, : m.ffn, :h] = self.src.get_expert(pre + "ffn_up_exps.weight", e, (m.ffn, h)).to(self.dev)
+            w2[e, :h, : m.ffn] = self.src.get_expert(pre + "ffn_down_exps.weight", e, (h, m.ffn)).to(self.dev)
+        lw.w13 = make_linear(w13.reshape(-1, k), self.fmt, groups=m.n_experts)
+        lw.w2 = make_linear(w2.reshape(-1, ip), self.fmt, groups=m.n_experts)
+
+    def layer(self, li: int, sp) -> LayerWeights:
+        pre, post = f"blk.{li}.", self.cfg.post_norm
+        lw = LayerWeights(attn_norm=self.norm(pre + "attn_norm"), wqkv=None, wo=None, ffn_norm=self.norm(pre + "ffn_norm") if sp.has_ffn else None)
+        if post:
+            lw.attn_post = self.norm(pre + "attn_post_norm", pre + "attn_post_scale.weight")
+            lw.ffn_post = self.norm(pre + "ffn_post_norm", pre + "ffn_post_scale.weight") if sp.has_ffn else None
+        getattr(self, sp.mixer)(pre, sp, lw)
+        if sp.ffn:
+            self.dense_ffn(pre, sp, lw)
+        elif sp.moe is not None:
+            self.moe_ffn(pre, sp, lw)
+        return lw
+
+    def model(self) -> ModelWeights:
+        cfg, h, src = self.cfg, self.h, self.src
+        layers = [self.layer(li, sp) for li, sp in enumerate(cfg.layer_specs)]
+        embed = self.get("token_embd.weight", cfg.vocab, h).to(torch.float32 if self.exact else torch.bfloat16).contiguous().to(self.dev)
+        head = embed if (cfg.tie_embeddings or not src.has("output.weight")) else self.get("output.weight", cfg.vocab, h)
+        step = self.f32("loop_step.weight", cfg.loop.times, h) if cfg.loop is not None else None
+        final = self.norm("output_norm")
+        if cfg.norm_kind == "rms":
+            final = final * cfg.logit_scale
+        return ModelWeights(cfg=cfg, embed=embed, layers=layers, final_norm=final, lm_head=self.linear(head), fmt=self.fmt, loop_step=step)
 
 
 def _build_layered(cfg: ModelConfig, src, fmt: str, dev, tile: Optional[bool]) -> ModelWeights:
-    """Weights of a model described layer by layer.  Norm weights become f32 ``offset + w``; the factor of the logits is folded into the
-    final norm's weight."""
     if fmt not in ("bf16", "f32"):
         raise ValueError(f"models described layer by layer run in bf16 or f32, not {fmt!r}")
-    h = cfg.hidden
-    exact = fmt == "f32"
-
-    def norm_w(name, n, offset):
-        return (src.get(name, (n,)).float() + offset).contiguous().to(dev)
-
-    layers: List[LayerWeights] = []
-    for li, sp in enumerate(cfg.layer_specs):
-        pre = f"blk.{li}."
-        lw = LayerWeights(attn_norm=norm_w(pre + "attn_norm.weight", h, cfg.norm_offset), wqkv=None, wo=None,
-                          ffn_norm=norm_w(pre + "ffn_norm.weight", h, cfg.norm_offset) if sp.ffn else None)
-        nv = sp.n_heads * sp.v_dim
-        if sp.mixer == "lightning":
-            w_in = torch.cat([src.get(pre + "lin_q.weight", (sp.q_dim, h)), src.get(pre + "lin_k.weight", (sp.q_dim, h)),
-                              src.get(pre + "lin_v.weight", (nv, h)), src.get(pre + "lin_gate.weight", (nv, h))])
-            lw.lin = LightningWeights(w_in=_padded_linear(w_in, fmt, dev), decay=torch.tensor(sp.decay, dtype=torch.float32, device=dev),
-                                      norm=norm_w(pre + "lin_norm.weight", nv, 0.0),
-                                      w_out=_padded_linear(src.get(pre + "lin_out.weight", (h, nv)), fmt, dev))
-        else:
-            nk, nkv = sp.n_kv_heads * sp.head_dim, sp.n_kv_heads * sp.v_dim
-            w = torch.cat([src.get(pre + "attn_q.weight", (sp.q_dim, h)), src.get(pre + "attn_k.weight", (nk, h)), src.get(pre + "attn_v.weight", (nkv, h))])
-            bias = None
-            if sp.qkv_bias:
-                bias = torch.cat([src.get(pre + f"attn_{c}.bias", (n,)).float() for c, n in (("q", sp.q_dim), ("k", nk), ("v", nkv))]).contiguous().to(dev)
-            lw.wqkv = _padded_linear(w, fmt, dev, bias=bias)
-            # the attention kernels emit heads of the cache's (padded) value width: the output projection has zero columns there
-            wo = src.get(pre + "attn_output.weight", (h, nv))
-            dvp = cache_head_dims(sp.head_dim, sp.v_dim, torch.float32 if exact else torch.bfloat16)[1]
-            wo = torch.nn.functional.pad(wo.reshape(h, sp.n_heads, sp.v_dim), (0, dvp - sp.v_dim)).reshape(h, sp.n_heads * dvp)
-            lw.wo = _padded_linear(wo, fmt, dev)
-            if sp.rel_buckets:
-                lw.rel_bias = distance_bias_table(src.get(pre + "attn_rel.weight", (sp.rel_buckets, sp.n_heads)).float().cpu(), sp.rel_max).to(dev)
-        if sp.ffn:
-            wg, wu = src.get(pre + "ffn_gate.weight", (sp.ffn, h)), src.get(pre + "ffn_up.weight", (sp.ffn, h))
-            wd = src.get(pre + "ffn_down.weight", (h, sp.ffn))
-            fp = sp.ffn if exact else (sp.ffn + 127) // 128 * 128       # the gate / up GEMM works on whole 128-row tiles
-            pad = torch.nn.functional.pad
-            lw.w_gate_up = _padded_linear(torch.cat([pad(wg, (0, 0, 0, fp - sp.ffn)), pad(wu, (0, 0, 0, fp - sp.ffn))]), fmt, dev)
-            lw.w_down = _padded_linear(pad(wd, (0, fp - sp.ffn)), fmt, dev)
-        layers.append(lw)
-    embed = src.get("token_embd.weight", (cfg.vocab, h)).to(torch.float32 if exact else torch.bfloat16).contiguous().to(dev)
-    head = embed if (cfg.tie_embeddings or not src.has("output.weight")) else src.get("output.weight", (cfg.vocab, h))
-    step = src.get("loop_step.weight", (cfg.loop.times, h)).float().contiguous().to(dev) if cfg.loop is not None else None
-    mw = ModelWeights(cfg=cfg, embed=embed, layers=layers, final_norm=norm_w("output_norm.weight", h, cfg.norm_offset) * cfg.logit_scale,
-                      lm_head=_padded_linear(head, fmt, dev), fmt=fmt, loop_step=step)
-    if (tile if tile is not None else dev.type == "cuda") and not exact:
+    mw = _LayeredBuilder(cfg, src, fmt, dev).model()
+    if (tile if tile is not None else dev.type == "cuda") and fmt != "f32":
         mw.tile_()
     return mw
 
