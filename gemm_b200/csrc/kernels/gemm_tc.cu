@@ -769,7 +769,8 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
   // (128-row layout, second half at column 2) is kept to a single token block.
   if (mx && tn == 64 && (num_groups > 0 || m_tok > tn)) return fail("gemm: MXFP8 with tn = 64 needs a single token block%s");
   if (!mx && (k % 8 != 0)) return fail("gemm: bf16 needs k %% 8 == 0%s");
-  if ((mx || num_groups > 0 || dual) && (n_out % 128 != 0)) return fail("gemm: n_out must be a multiple of 128 for MX / grouped / dual%s");
+  if ((mx || dual) && (n_out % 128 != 0)) return fail("gemm: n_out must be a multiple of 128 for MX / dual%s");
+  if (num_groups > 0 && n_out > w_rows_per_group) return fail("gemm: a group has fewer rows than features are asked for%s");
   const int esz = mx ? 1 : 2;
   const int w_groups = (ex != nullptr && ex->w_group_mod > 0) ? ex->w_group_mod : num_groups;
   const long w_rows = (num_groups > 0) ? (long)w_groups * w_rows_per_group : (dual ? (long)up_row_offset + n_out : (long)n_out);

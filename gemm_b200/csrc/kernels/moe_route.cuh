@@ -10,11 +10,15 @@ namespace gb {
 
 constexpr int kMaxTopK = 16;
 
+constexpr int kMaxExpertGroups = 128;
+
 // Routing of token `w` by one warp (E <= 512): lane j < k ends with the j-th pick.  Returns the (possibly local) expert id.
+// groups > 1 (at most kMaxExpertGroups, dividing the experts): a group of neighbouring experts scores the sum of its two best, and only
+// experts of the `keep` best groups can be picked (ties: lower group).  renorm: 1 = weights over max(sum, 1e-20), 2 = over sum + 1e-20.
 template <int MAXV>
 __device__ __forceinline__ int route_row(const float* row, const float* __restrict__ bias, int* __restrict__ ids_row,
                                          float* __restrict__ weights_row, int lane, int n_exp, int k, int mode, int renorm,
-                                         float routed_scale, int id_shift, int n_local) {
+                                         float routed_scale, int groups, int keep, int id_shift, int n_local) {
   float p[MAXV], sel[MAXV];
   float mx = -FLT_MAX;
 #pragma unroll
@@ -40,6 +44,55 @@ __device__ __forceinline__ int route_row(const float* row, const float* __restri
       const int e = lane + 32 * i;
       p[i] = (e < n_exp) ? 1.0f / (1.0f + expf(-p[i])) : 0.f;
       sel[i] = (e < n_exp) ? p[i] + (bias != nullptr ? bias[e] : 0.f) : -FLT_MAX;
+    }
+  }
+  if (groups > 1 && keep < groups) {
+    const int size = n_exp / groups;
+    float gs[kMaxExpertGroups / 32];
+    unsigned kept[kMaxExpertGroups / 32];
+#pragma unroll
+    for (int i = 0; i < kMaxExpertGroups / 32; ++i) {
+      const int g = lane + 32 * i;
+      kept[i] = 0u;
+      gs[i] = -FLT_MAX;
+      if (g >= groups) continue;
+      float b1 = -FLT_MAX, b2 = -FLT_MAX;           // the group's scores, as above
+      for (int x = 0; x < size; ++x) {
+        float v = row[g * size + x];
+        if (!(v == v)) v = -FLT_MAX;
+        v = mode == 0 ? expf(v - mx) : 1.0f / (1.0f + expf(-v)) + (bias != nullptr ? bias[g * size + x] : 0.f);
+        if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) b2 = v;
+      }
+      gs[i] = size > 1 ? b1 + b2 : b1;
+    }
+    for (int j = 0; j < keep; ++j) {
+      float best = -FLT_MAX; int bi = 0x7fffffff;
+#pragma unroll
+      for (int i = 0; i < kMaxExpertGroups / 32; ++i) {
+        const int g = lane + 32 * i;
+        if (g < groups && (gs[i] > best || (gs[i] == best && g < bi))) { best = gs[i]; bi = g; }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        const float ob = __shfl_xor_sync(0xffffffffu, best, o);
+        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+        if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
+      }
+#pragma unroll
+      for (int i = 0; i < kMaxExpertGroups / 32; ++i) {
+        if (lane + 32 * i == bi) gs[i] = -FLT_MAX;
+        if (bi < groups && (bi >> 5) == i) kept[i] |= 1u << (bi & 31);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < MAXV; ++i) {
+      const int e = lane + 32 * i;
+      if (e >= n_exp) continue;
+      const int g = e / size;
+      unsigned m = 0u;
+#pragma unroll
+      for (int x = 0; x < kMaxExpertGroups / 32; ++x) if ((g >> 5) == x) m = kept[x];
+      if (!((m >> (g & 31)) & 1u)) sel[i] = -FLT_MAX;
     }
   }
   float wsum = 0.f;
@@ -68,7 +121,7 @@ __device__ __forceinline__ int route_row(const float* row, const float* __restri
   int out_id = -1;
   if (lane < k) {
     float wv = my_w;
-    if (renorm) wv = wv / fmaxf(wsum, 1e-20f);
+    if (renorm) wv = wv / (renorm == 2 ? wsum + 1e-20f : fmaxf(wsum, 1e-20f));
     // expert-parallel ranks that see every token keep only their own experts: ids become local, the others -1
     const int lid = my_id - id_shift;
     out_id = (n_local > 0 && (lid < 0 || lid >= n_local)) ? -1 : lid;

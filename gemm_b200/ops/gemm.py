@@ -200,6 +200,37 @@ def linear_f32(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = 
     return out
 
 
+def batched_linear_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``out[b] = x[b] @ w[b]^T`` in f32: ``x [B, M, K]``, ``w [B, N, K]``, ``out [B, M, N]``, views with unit stride in the last dimension."""
+    b, m, k = x.shape
+    n = w.shape[1]
+    if not x.is_cuda:
+        out.copy_(torch.bmm(x, w.transpose(1, 2)))
+        return out
+    assert x.dtype == w.dtype == out.dtype == torch.float32 and x.stride(2) == w.stride(2) == out.stride(2) == 1
+    rc = _native.cuda().gb_gemm_f32_batched(_p(x), _p(w), _p(out), _i(b), _i(m), _i(n), _i(k), _i(x.stride(1)), _i(w.stride(1)), _i(out.stride(1)),
+                                            ctypes.c_long(x.stride(0)), ctypes.c_long(w.stride(0)), ctypes.c_long(out.stride(0)), _stream())
+    _native.check(rc, "gb_gemm_f32_batched")
+    return out
+
+
+def grouped_linear_f32(x: torch.Tensor, w: torch.Tensor, seg_start: torch.Tensor, seg_count: torch.Tensor, rows: int,
+                       row_src: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``grouped_linear`` in f32: rows ``seg_start[g] ...`` (multiples of 64) times ``w[g] [N, K]^T`` -> ``[rows, N]``; row r is ``x[row_src[r]]``, or
+    ``x[r]``.  Rows of no segment are undefined."""
+    g, n, k = w.shape
+    if not x.is_cuda:
+        out = torch.zeros(rows, n)
+        for gi in range(g):
+            s, c = int(seg_start[gi]), int(seg_count[gi])
+            out[s: s + c] = (x[row_src[s: s + c].long()] if row_src is not None else x[s: s + c]) @ w[gi].t()
+        return out
+    out = torch.empty(rows, n, dtype=torch.float32, device=x.device)
+    rc = _native.cuda().gb_gemm_f32_grouped(_p(x), _p(w), _p(out), _p(seg_start), _p(seg_count), _i(g), _i(rows), _i(n), _i(k), _i(x.stride(0)), _p(row_src), _stream())
+    _native.check(rc, "gb_gemm_f32_grouped")
+    return out
+
+
 def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: Optional[torch.Tensor] = None,
                   tn: Optional[int] = None, w_tiled: bool = False, act: str = "silu") -> torch.Tensor:
     """``act(x @ Wg^T) * (x @ Wu^T)`` with ``w_gate_up = [Wg; Wu]`` stacked along rows ([2I, K]); ``act`` is one of ``GATE_ACTS``."""
@@ -350,7 +381,7 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, seg_start: torch.Tensor, se
                    out: Optional[torch.Tensor] = None, dual: bool = False, row_map: Optional[torch.Tensor] = None,
                    row_scale: Optional[torch.Tensor] = None, sfa=None, sfb=None, quant_out: bool = False,
                    out_sf: Optional[torch.Tensor] = None, extras=None, w_groups: Optional[int] = None,
-                   w_tiled: bool = False, pair_rows: bool = False) -> torch.Tensor:
+                   w_tiled: bool = False, pair_rows: bool = False, n_out: Optional[int] = None) -> torch.Tensor:
     """One GEMM per group over row segments of ``x``.
 
     ``w`` is ``[G, R, K]`` (R = 2I stacked gate/up rows when ``dual``); group g multiplies the rows
@@ -364,12 +395,12 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, seg_start: torch.Tensor, se
     # ``pair_rows``: a tile takes row blocks n and R/2 + n of the SAME projection (two accumulators, plain stores): half the tiles
     # and token-tile loads for projections with a short K, such as the expert down projection of a decode step
     pair = bool(pair_rows and not dual and not quant_out and row_map is None and row_scale is None and x.is_cuda and r % 256 == 0)
-    n_out = r // 2 if (dual or pair) else r
+    n_out = r // 2 if (dual or pair) else n_out or r          # ``n_out``: leading features of each group (bf16, plain)
     mx = sfa is not None
     if not x.is_cuda:
         if w_tiled:
             w = mxfp8.untile_weight(w.reshape(-1, k)).reshape(w.shape)
-        return _grouped_reference(x, w, seg_start, seg_count, dual, row_map, row_scale, sfa, sfb, quant_out, out, out_sf)
+        return _grouped_reference(x, w if dual else w[:, :n_out], seg_start, seg_count, dual, row_map, row_scale, sfa, sfb, quant_out, out, out_sf)
     flags = (GEMM_MX if mx else 0) | (GEMM_DUAL if dual else 0) | (GEMM_QUANT_OUT if quant_out else 0) | (GEMM_W_TILED if w_tiled else 0)
     if pair:
         flags |= GEMM_DUAL | GEMM_DUAL_RAW
@@ -419,6 +450,9 @@ def _grouped_reference(x, w, seg_start, seg_count, dual, row_map, row_scale, sfa
     if row_map is not None:
         assert out is not None
         keep = row_map >= 0
-        out[row_map[keep].long()] = res[keep].to(out.dtype)
+        out[row_map[keep].long(), :n_out] = res[keep].to(out.dtype)
+        return out
+    if out is not None:
+        out[: res.shape[0], :n_out] = res.to(out.dtype)
         return out
     return res.to(torch.bfloat16)
