@@ -13,6 +13,7 @@
 // decays and state keep 32-bit accuracy; only q, k and v themselves are bf16.
 #include "sm100.cuh"
 #include "host_common.h"
+#include "recurrent.cuh"
 
 namespace gb {
 
@@ -32,18 +33,6 @@ struct LightningChunkArgs {
   int heads, dim, vdim;
   KernelStatus* status;
 };
-
-// x = hi + lo in bf16, for two neighbours
-__device__ __forceinline__ void split_bf16x2(float a, float b, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(a, b);
-  const float2 h = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&hi));
-  lo = pack_bf16x2(a - h.x, b - h.y);
-}
-
-// Bounded wait of a whole warp: its lanes leave a failed wait together (the tcgen05 loads that follow need all of them).
-__device__ __forceinline__ bool warp_wait(uint64_t* bar, uint32_t parity, volatile int* abort_flag, KernelStatus* st, int where, int aux) {
-  return __all_sync(0xffffffffu, mbar_wait(bar, parity, abort_flag, st, where, aux));
-}
 
 template <int DP>                          // key size padded: 64 or 128
 __global__ void __launch_bounds__(kLcThreads, 1)

@@ -1,0 +1,291 @@
+// Recurrent mixers with input-dependent decay, token by token (decode steps, short portions, the 32-bit format):
+//   causal_conv   depthwise causal convolution with bias + SiLU over packed tokens, the last taps - 1 inputs carried per sequence
+//   ssd           Mamba-2:  S_t = exp(a dt_t) S_{t-1} + dt_t B_t x_t^T,  y_t = S_t^T C_t + D x_t, one scalar decay per head and token
+//   gla           HGRN2:    S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T,  o_t = S_t^T q_t, one decay per key channel
+// The state S [dim, vdim] is f32 and lives in a slot per sequence.  The chunked forms for prompts are in lightning_chunk.cu (Mamba-2) and
+// gla_chunk.cu (HGRN2).
+//
+// The step kernel has the layout of lightning.cu: one CTA per (sequence, head, slice of value columns); a lane owns VEC value columns, the eight
+// warps split the key rows, and a decode step is one pass over the state with all of a thread's loads in flight at once.
+#include "sm100.cuh"
+#include "host_common.h"
+#include "recurrent.cuh"
+
+namespace gb {
+
+// ------------------------------------------------------------------------------------------ convolution
+struct CausalConvArgs {
+  const void* x; int n_part; long part_stride; int ld_x;      // [n_part][tokens, ld_x], the channels are the first columns
+  const float* w; const float* b;                             // [channels, taps], [channels]
+  float* state; int n_slots;                                  // [slots, taps - 1, channels], oldest row first
+  const int* cu_q; const int* seq_slots;
+  void* out; int ld_out;                                      // activated channels
+  int channels, taps;
+};
+
+constexpr int kConvTile = 32;                                 // tokens per CTA, at least the longest history
+constexpr int kMaxTaps = 16;
+
+// V neighbouring channels per thread.  Only a sequence's first tile reads the old state (a tile is longer than the history), and the same
+// threads write the new one, so nothing races.
+template <typename TI, typename TO, int V, int MT>            // taps <= MT
+__global__ void __launch_bounds__(128)
+causal_conv_kernel(const CausalConvArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V, s = blockIdx.z;
+  const int t0 = a.cu_q[s], t1 = a.cu_q[s + 1];
+  const int tb = t0 + blockIdx.y * kConvTile, te = min(t1, tb + kConvTile);
+  const int slot = a.seq_slots[s];
+  if (c >= a.channels || tb >= t1 || slot < 0 || slot >= a.n_slots) return;
+  const int nh = a.taps - 1;
+  float* st = a.state + (size_t)slot * nh * a.channels + c;
+  float w[MT][V], b[V], win[MT][V];                           // win[i]: the input nh - i tokens in front of the current one
+  auto input = [&](int t, float* v) {
+    const TI* p = (const TI*)a.x + (size_t)t * a.ld_x + c;
+    load_cols<V>(p, v);
+    for (int q = 1; q < a.n_part; ++q) {
+      float y[V];
+      load_cols<V>(p + (size_t)q * a.part_stride, y);
+#pragma unroll
+      for (int i = 0; i < V; ++i) v[i] += y[i];
+    }
+  };
+#pragma unroll
+  for (int i = 0; i < V; ++i) b[i] = a.b[c + i];
+#pragma unroll
+  for (int k = 0; k < MT; ++k)
+#pragma unroll
+    for (int i = 0; i < V; ++i) { w[k][i] = k < a.taps ? a.w[(size_t)(c + i) * a.taps + k] : 0.f; win[k][i] = 0.f; }
+#pragma unroll
+  for (int k = 0; k < MT - 1; ++k)
+    if (k < nh) {
+      const int t = tb - nh + k;
+      if (t >= t0) input(t, win[k]);
+      else load_cols<V>(st + (size_t)(t - t0 + nh) * a.channels, win[k]);
+    }
+  if (blockIdx.y == 0) {                                      // the history behind the sequence's last token
+    float keep[MT][V];
+#pragma unroll
+    for (int k = 0; k < MT - 1; ++k)
+      if (k < nh) {
+        const int t = t1 - nh + k;
+        if (t >= t0) input(t, keep[k]);
+        else load_cols<V>(st + (size_t)(t - t0 + nh) * a.channels, keep[k]);
+      }
+#pragma unroll
+    for (int k = 0; k < MT - 1; ++k)
+      if (k < nh) store_cols<V>(st + (size_t)k * a.channels, keep[k]);
+  }
+  for (int t = tb; t < te; ++t) {
+    float cur[V], y[V];
+    input(t, cur);
+#pragma unroll
+    for (int i = 0; i < V; ++i) y[i] = b[i];
+#pragma unroll
+    for (int k = 0; k < MT; ++k) {
+      if (k < nh) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[i] = fmaf(w[k][i], win[k][i], y[i]);
+      } else if (k == nh) {
+#pragma unroll
+        for (int i = 0; i < V; ++i) y[i] = fmaf(w[k][i], cur[i], y[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) y[i] = y[i] / (1.0f + expf(-y[i]));
+    store_cols<V>((TO*)a.out + (size_t)t * a.ld_out + c, y);
+#pragma unroll
+    for (int k = 0; k < MT - 1; ++k)
+      if (k < nh)
+#pragma unroll
+        for (int i = 0; i < V; ++i) win[k][i] = k + 1 < nh ? win[k + 1][i] : cur[i];
+  }
+}
+
+// ------------------------------------------------------------------------------------------ recurrence
+struct RecurrentArgs {
+  // ssd: activated channels of the convolution [tokens, ld]: [x heads x vdim | B groups x dim | C groups x dim] (one slab)
+  // gla: input projection [n_part][tokens, ld]: q heads x dim from column 0, v heads x vdim behind it
+  const void* in; int n_part; long part_stride; int ld;
+  // the gate's pre-activations, [g_part][tokens, g_ld] f32: dt (heads columns) or f (heads x dim columns)
+  const float* gate; int g_part; long g_stride; int g_ld;
+  const float* gate_bias;       // ssd: dt_bias [heads]; gla: [heads * dim]
+  const float* par;             // ssd: a [heads], negative; gla: lower bound [heads * dim]
+  const float* d_skip;          // ssd: [heads]
+  float* state; int n_slots;    // [slots, heads, dim, vdim]
+  const int* cu_q; const int* seq_slots;
+  float* out; int ld_out;       // [tokens, heads * vdim]
+  int heads, groups, dim, vdim;
+  int q_raw;                    // gla: != 0: q has no SiLU yet
+};
+
+template <typename TI>
+__device__ __forceinline__ float in_col(const RecurrentArgs& a, size_t tok, int col) {
+  const TI* p = (const TI*)a.in + tok * a.ld + col;
+  float s = ldv(p);
+  for (int i = 1; i < a.n_part; ++i) s += ldv(p + (size_t)i * a.part_stride);
+  return s;
+}
+__device__ __forceinline__ float gate_col(const RecurrentArgs& a, size_t tok, int col) {
+  const float* p = a.gate + tok * a.g_ld + col;
+  float s = *p;
+  for (int i = 1; i < a.g_part; ++i) s += p[(size_t)i * a.g_stride];
+  return s;
+}
+
+template <typename TI, bool GLA, int VEC, int R>   // dim <= 8 * R
+__global__ void __launch_bounds__(256)
+recurrent_step_kernel(const RecurrentArgs a) {
+  __shared__ float sq[8 * R], sk[8 * R], sf[GLA ? 8 * R : 1];
+  __shared__ float red[8][32 * VEC];
+  __shared__ float s_dec;
+  pdl_wait();
+  pdl_trigger();
+  const int h = blockIdx.x, s = blockIdx.z, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int t0 = a.cu_q[s], t1 = a.cu_q[s + 1];
+  const int slot = a.seq_slots[s];
+  if (t1 <= t0 || slot < 0 || slot >= a.n_slots) return;
+  const int e0 = (blockIdx.y * 32 + lane) * VEC;
+  const bool live = e0 < a.vdim;                   // VEC > 1 only when vdim % VEC == 0
+  float* st = a.state + ((size_t)slot * a.heads + h) * a.dim * a.vdim + e0;
+  float S[R][VEC];
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+    const int d = warp + 8 * r;
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) S[r][j] = 0.f;
+    if (live && d < a.dim) load_cols<VEC>(st + (size_t)d * a.vdim, S[r]);
+  }
+  const int nv = a.heads * a.vdim, grp = h / (a.heads / a.groups);
+  const int q_col = GLA ? h * a.dim : nv + (a.groups + grp) * a.dim, k_col = nv + grp * a.dim;
+  const int v_col = (GLA ? a.heads * a.dim : 0) + h * a.vdim + e0;
+  const float a_h = GLA ? 0.f : a.par[h], bias_h = GLA ? 0.f : a.gate_bias[h], skip = GLA ? 0.f : a.d_skip[h];
+  for (int t = t0; t < t1; ++t) {
+    float dt = 0.f;
+    if constexpr (!GLA) {
+      dt = softplus_exact(gate_col(a, t, h) + bias_h);
+      if (threadIdx.x == 0) s_dec = expf(a_h * dt);
+    }
+    for (int i = threadIdx.x; i < 2 * a.dim; i += 256) {
+      const bool isk = i >= a.dim;
+      const int c = isk ? i - a.dim : i;
+      if constexpr (GLA) {
+        if (isk) {
+          const float z = gate_col(a, t, h * a.dim + c) + a.gate_bias[h * a.dim + c], low = a.par[h * a.dim + c];
+          sf[c] = forget_gate(z, low, sk[c]);
+        } else {
+          const float q = in_col<TI>(a, t, q_col + c);
+          sq[c] = a.q_raw ? q / (1.0f + expf(-q)) : q;
+        }
+      } else {
+        if (isk) sk[c] = in_col<TI>(a, t, k_col + c) * dt; else sq[c] = in_col<TI>(a, t, q_col + c);
+      }
+    }
+    float v[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) v[j] = live ? in_col<TI>(a, t, v_col + j) : 0.f;
+    __syncthreads();
+    float o[VEC];
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) o[j] = 0.f;
+    const float dec = GLA ? 0.f : s_dec;
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int d = warp + 8 * r;
+      if (d < a.dim) {
+        const float kd = sk[d], qd = sq[d], f = GLA ? sf[GLA ? d : 0] : dec;
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) { S[r][j] = fmaf(f, S[r][j], kd * v[j]); o[j] = fmaf(S[r][j], qd, o[j]); }
+      }
+    }
+    if (!GLA && warp == 0) {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) o[j] = fmaf(skip, v[j], o[j]);
+    }
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) red[warp][lane * VEC + j] = o[j];
+    __syncthreads();
+    if (threadIdx.x < 32 * VEC) {
+      float acc = 0.f;
+#pragma unroll
+      for (int w = 0; w < 8; ++w) acc += red[w][threadIdx.x];
+      const int e = blockIdx.y * 32 * VEC + threadIdx.x;
+      if (e < a.vdim) a.out[(size_t)t * a.ld_out + h * a.vdim + e] = acc;
+    }
+    // the shared rows are rewritten only after every thread has passed the second barrier; red is read before the next token's first barrier
+  }
+  if (live) {
+#pragma unroll
+    for (int r = 0; r < R; ++r) {
+      const int d = warp + 8 * r;
+      if (d < a.dim) store_cols<VEC>(st + (size_t)d * a.vdim, S[r]);
+    }
+  }
+}
+
+template <typename TI, bool GLA>
+static int recurrent_step_launch(const RecurrentArgs& a, int n_seqs, cudaStream_t stream) {
+  const bool vec = a.vdim % 4 == 0 && a.vdim > 32 && a.dim <= 256 && ((uintptr_t)a.state & 15) == 0;
+  const int cols = vec ? 128 : 32;
+  const dim3 grid((unsigned)a.heads, (unsigned)((a.vdim + cols - 1) / cols), (unsigned)n_seqs);
+#define GB_RS(VECV, RV) launch_k(recurrent_step_kernel<TI, GLA, VECV, RV>, grid, 256, 0, stream, a)
+  if (vec) {
+    if (a.dim <= 32) GB_RS(4, 4); else if (a.dim <= 64) GB_RS(4, 8); else if (a.dim <= 128) GB_RS(4, 16); else GB_RS(4, 32);
+  } else {
+    if (a.dim <= 64) GB_RS(1, 8); else if (a.dim <= 256) GB_RS(1, 32); else GB_RS(1, 64);
+  }
+#undef GB_RS
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+template <typename TI, typename TO>
+static int causal_conv_launch(const CausalConvArgs& a, int max_tokens, int n_seqs, cudaStream_t stream) {
+  const bool vec = a.taps <= 4 && a.channels % 4 == 0 && a.ld_x % 4 == 0 && a.part_stride % 4 == 0 && a.ld_out % 4 == 0 && (uintptr_t)a.x % (4 * sizeof(TI)) == 0 &&
+                   (uintptr_t)a.out % (4 * sizeof(TO)) == 0 && ((uintptr_t)a.state & 15) == 0;
+  const int cols = vec ? 512 : 128;
+  const dim3 grid((unsigned)((a.channels + cols - 1) / cols), (unsigned)((max_tokens + kConvTile - 1) / kConvTile), (unsigned)n_seqs);
+  if (vec) launch_k(causal_conv_kernel<TI, TO, 4, 4>, grid, 128, 0, stream, a);
+  else if (a.taps <= 4) launch_k(causal_conv_kernel<TI, TO, 1, 4>, grid, 128, 0, stream, a);
+  else launch_k(causal_conv_kernel<TI, TO, 1, kMaxTaps>, grid, 128, 0, stream, a);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+}  // namespace gb
+
+using namespace gb;
+
+// x: channels in the first columns of [n_part][tokens, ld_x]; out [tokens, ld_out] = SiLU(conv + bias); max_tokens: of the longest sequence.
+GB_API int gb_causal_conv(const void* x, int x_f32, int n_part, long part_stride, int ld_x, const float* w, const float* b, float* state, int n_slots,
+                          const int* cu_q, const int* seq_slots, void* out, int out_f32, int ld_out, int channels, int taps, int max_tokens, int n_seqs,
+                          cudaStream_t stream) {
+  if (n_seqs <= 0 || max_tokens <= 0) return 0;
+  if (channels < 1 || taps < 1 || taps > kMaxTaps || n_part < 1 || ld_x < channels || ld_out < channels) return fail("causal_conv: bad sizes (at most 16 taps)%s");
+  if (n_seqs > 65535 || (max_tokens + kConvTile - 1) / kConvTile > 65535) return fail("causal_conv: too many tokens%s");
+  CausalConvArgs a;
+  a.x = x; a.n_part = n_part; a.part_stride = part_stride; a.ld_x = ld_x; a.w = w; a.b = b; a.state = state; a.n_slots = n_slots; a.cu_q = cu_q;
+  a.seq_slots = seq_slots; a.out = out; a.ld_out = ld_out; a.channels = channels; a.taps = taps;
+  if (x_f32) return out_f32 ? causal_conv_launch<float, float>(a, max_tokens, n_seqs, stream) : causal_conv_launch<float, __nv_bfloat16>(a, max_tokens, n_seqs, stream);
+  if (out_f32) return fail("causal_conv: 32-bit results take 32-bit rows%s");
+  return causal_conv_launch<__nv_bfloat16, __nv_bfloat16>(a, max_tokens, n_seqs, stream);
+}
+
+// See RecurrentArgs.  gla != 0: HGRN2 (groups and d_skip are not used); else Mamba-2.
+GB_API int gb_recurrent_step(int gla, const void* in, int in_f32, int n_part, long part_stride, int ld, const float* gate, int g_part, long g_stride, int g_ld,
+                             const float* gate_bias, const float* par, const float* d_skip, float* state, int n_slots, const int* cu_q, const int* seq_slots,
+                             float* out, int ld_out, int heads, int groups, int dim, int vdim, int q_raw, int n_seqs, cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  if (heads < 1 || dim < 1 || vdim < 1 || n_part < 1 || g_part < 1 || groups < 1 || heads % groups || ld_out < heads * vdim) return fail("recurrent: bad sizes%s");
+  if (gla ? (ld < heads * (dim + vdim) || g_ld < heads * dim) : (ld < heads * vdim + 2 * groups * dim || g_ld < heads || n_part != 1 || d_skip == nullptr))
+    return fail("recurrent: rows are too short%s");
+  if (dim > 512) return fail("recurrent: a key dimension of at most 512%s");
+  if (n_seqs > 65535) return fail("recurrent: too many sequences%s");
+  RecurrentArgs a;
+  a.in = in; a.n_part = n_part; a.part_stride = part_stride; a.ld = ld; a.gate = gate; a.g_part = g_part; a.g_stride = g_stride; a.g_ld = g_ld;
+  a.gate_bias = gate_bias; a.par = par; a.d_skip = d_skip; a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out;
+  a.ld_out = ld_out; a.heads = heads; a.groups = groups; a.dim = dim; a.vdim = vdim; a.q_raw = q_raw;
+  if (gla) return in_f32 ? recurrent_step_launch<float, true>(a, n_seqs, stream) : recurrent_step_launch<__nv_bfloat16, true>(a, n_seqs, stream);
+  return in_f32 ? recurrent_step_launch<float, false>(a, n_seqs, stream) : recurrent_step_launch<__nv_bfloat16, false>(a, n_seqs, stream);
+}

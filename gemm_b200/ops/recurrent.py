@@ -1,0 +1,140 @@
+"""Recurrent mixers with input-dependent decay (csrc/kernels/recurrent.cu and its chunked forms) and their PyTorch references.
+
+``causal_conv``  depthwise causal convolution + SiLU, the last inputs carried per sequence (Mamba-2)
+``ssd``          Mamba-2:  S_t = exp(a dt_t) S_{t-1} + dt_t B_t x_t^T,  y_t = S_t^T C_t + D x_t
+``gla``          HGRN2:    S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T,  o_t = S_t^T q_t
+
+State tensors: ``conv_state`` f32 ``[slots, taps - 1, channels]`` (oldest row first), ``state`` f32 ``[slots, heads, dim, vdim]``; one slot per
+sequence, updated in place.
+"""
+from __future__ import annotations
+
+import ctypes
+import os
+
+import torch
+
+from .. import _native
+from .stream import row_width, split_rows, whole
+
+_c, _i, _f, _l = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_long
+F = torch.nn.functional
+
+
+def _p(t):
+    return _c(t.data_ptr()) if t is not None else _c(0)
+
+
+def _s():
+    return _c(torch.cuda.current_stream().cuda_stream)
+
+
+def _n_rows(y) -> int:
+    return y.rows if hasattr(y, "buf") else y.shape[0]
+
+
+def _at(base: torch.Tensor, col: int):
+    return _c(base.data_ptr() + col * base.element_size())
+
+
+def causal_conv_ref(x, w, b, state, cu_q, seq_slots, out_dtype):
+    t, ch = x.shape
+    out = torch.zeros(t, row_width(ch, out_dtype), dtype=out_dtype)
+    nh = w.shape[1] - 1
+    cu = cu_q.tolist()
+    for s in range(len(cu) - 1):
+        if cu[s + 1] == cu[s]:
+            continue
+        rows = torch.cat([state[int(seq_slots[s])], x[cu[s]: cu[s + 1]]])
+        y = sum(w[:, k] * rows[k: k + cu[s + 1] - cu[s]] for k in range(nh + 1)) + b
+        out[cu[s]: cu[s + 1], :ch] = F.silu(y).to(out_dtype)
+        state[int(seq_slots[s])] = rows[rows.shape[0] - nh:]
+    return out
+
+
+def causal_conv(proj, col: int, w: torch.Tensor, b: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, seq_slots: torch.Tensor, max_tokens: int,
+                out_dtype=torch.bfloat16) -> torch.Tensor:
+    """SiLU(conv + b) of the columns ``col ... col + channels - 1`` of the projection result ``proj`` -> rows ``[T, row_width(channels)]``."""
+    ch, taps = w.shape
+    base, f32, parts, stride, ld = split_rows(proj)
+    if not base.is_cuda:
+        return causal_conv_ref(whole(proj)[:, col: col + ch], w, b, state, cu_q, seq_slots, out_dtype)
+    t = _n_rows(proj)
+    assert state.is_contiguous() and state.dtype == torch.float32
+    out = torch.empty(t, row_width(ch, out_dtype), dtype=out_dtype, device=base.device)
+    rc = _native.cuda().gb_causal_conv(_at(base, col), _i(f32), _i(parts), _l(stride), _i(ld), _p(w), _p(b), _p(state), _i(state.shape[0]), _p(cu_q), _p(seq_slots),
+                                       _p(out), _i(int(out_dtype == torch.float32)), _i(out.shape[1]), _i(ch), _i(taps), _i(max_tokens), _i(cu_q.numel() - 1), _s())
+    _native.check(rc, "gb_causal_conv")
+    return out
+
+
+def ssd_ref(xbc, dt, dt_bias, a, d_skip, state, cu_q, seq_slots, heads, groups, dim, vdim):
+    t, nv = xbc.shape[0], heads * vdim
+    y = xbc.float()
+    x = y[:, :nv].reshape(t, heads, vdim)
+    bm = y[:, nv: nv + groups * dim].reshape(t, groups, dim).repeat_interleave(heads // groups, dim=1)
+    cm = y[:, nv + groups * dim: nv + 2 * groups * dim].reshape(t, groups, dim).repeat_interleave(heads // groups, dim=1)
+    dt = F.softplus(dt.float() + dt_bias, threshold=1e9)
+    dec = torch.exp(a * dt)
+    out = torch.zeros(t, nv)
+    cu = cu_q.tolist()
+    for s in range(len(cu) - 1):
+        st = state[int(seq_slots[s])] if cu[s + 1] > cu[s] else None
+        for i in range(cu[s], cu[s + 1]):
+            st.mul_(dec[i].reshape(heads, 1, 1)).add_((dt[i].unsqueeze(-1) * bm[i]).unsqueeze(-1) * x[i].unsqueeze(1))
+            out[i] = (torch.einsum("hde,hd->he", st, cm[i]) + d_skip.unsqueeze(-1) * x[i]).reshape(-1)
+    return out
+
+
+def ssd(xbc: torch.Tensor, dt, dt_col: int, dt_bias: torch.Tensor, a: torch.Tensor, d_skip: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor,
+        seq_slots: torch.Tensor, heads: int, groups: int, dim: int, vdim: int, max_tokens: int = 1) -> torch.Tensor:
+    """``xbc``: activated rows ``[x heads x vdim | B groups x dim | C groups x dim | ...]``; ``dt``: projection result (f32 or partial sums) whose
+    columns ``dt_col ...`` are the step sizes before bias and softplus.  ``max_tokens``: of the longest sequence.  Returns f32 ``[T, heads * vdim]``."""
+    base, f32, parts, stride, ld = split_rows(dt)
+    if not base.is_cuda:
+        return ssd_ref(xbc, whole(dt)[:, dt_col: dt_col + heads], dt_bias, a, d_skip, state, cu_q, seq_slots, heads, groups, dim, vdim)
+    t = xbc.shape[0]
+    assert f32 and state.is_contiguous() and state.dtype == torch.float32
+    out = torch.empty(t, heads * vdim, dtype=torch.float32, device=base.device)
+    rc = _native.cuda().gb_recurrent_step(_i(0), _p(xbc), _i(int(xbc.dtype == torch.float32)), _i(1), _l(0), _i(xbc.stride(0)), _at(base, dt_col), _i(parts), _l(stride),
+                                          _i(ld), _p(dt_bias), _p(a), _p(d_skip), _p(state), _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(heads * vdim),
+                                          _i(heads), _i(groups), _i(dim), _i(vdim), _i(0), _i(cu_q.numel() - 1), _s())
+    _native.check(rc, "gb_recurrent_step")
+    return out
+
+
+def gla_ref(q, v, z, lower, state, cu_q, seq_slots, heads, dim, vdim):
+    t = q.shape[0]
+    q, v = q.reshape(t, heads, dim), v.reshape(t, heads, vdim)
+    f = (lower + (1 - lower) * torch.sigmoid(z)).reshape(t, heads, dim)
+    k = ((1 - lower) * torch.sigmoid(-z)).reshape(t, heads, dim)
+    out = torch.zeros(t, heads * vdim)
+    cu = cu_q.tolist()
+    for s in range(len(cu) - 1):
+        st = state[int(seq_slots[s])] if cu[s + 1] > cu[s] else None
+        for i in range(cu[s], cu[s + 1]):
+            st.mul_(f[i].unsqueeze(-1)).add_(k[i].unsqueeze(-1) * v[i].unsqueeze(1))
+            out[i] = torch.einsum("hde,hd->he", st, q[i]).reshape(-1)
+    return out
+
+
+def gla(qv, gate, gate_col: int, f_bias: torch.Tensor, lower: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, seq_slots: torch.Tensor, heads: int, dim: int,
+        vdim: int, activated: bool = False, max_tokens: int = 1) -> torch.Tensor:
+    """``qv``: projection result with columns ``[q heads x dim | v heads x vdim | ...]``, q before its SiLU or (``activated``) after it; ``gate``:
+    projection result (f32 or partial sums) whose columns ``gate_col ...`` are the forget gates before bias and sigmoid.  Returns f32
+    ``[T, heads * vdim]``."""
+    gb, gf32, gparts, gstride, gld = split_rows(gate)
+    nq, nv = heads * dim, heads * vdim
+    if not gb.is_cuda:
+        y = whole(qv)
+        q = y[:, :nq] if activated else F.silu(y[:, :nq])
+        return gla_ref(q, y[:, nq: nq + nv], whole(gate)[:, gate_col: gate_col + nq] + f_bias, lower, state, cu_q, seq_slots, heads, dim, vdim)
+    base, f32, parts, stride, ld = split_rows(qv)
+    t = _n_rows(qv)
+    assert gf32 and state.is_contiguous() and state.dtype == torch.float32
+    out = torch.empty(t, nv, dtype=torch.float32, device=base.device)
+    rc = _native.cuda().gb_recurrent_step(_i(1), _p(base), _i(f32), _i(parts), _l(stride), _i(ld), _at(gb, gate_col), _i(gparts), _l(gstride), _i(gld), _p(f_bias), _p(lower),
+                                          _c(0), _p(state), _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(nv), _i(heads), _i(1), _i(dim), _i(vdim),
+                                          _i(int(not activated)), _i(cu_q.numel() - 1), _s())
+    _native.check(rc, "gb_recurrent_step")
+    return out
