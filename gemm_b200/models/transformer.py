@@ -13,8 +13,9 @@ Layer recipe (reference: common/transformer.h:3550-4174):
   logits = RMSNorm(x) Whead^T on the last token of every sequence.
 
 Models described layer by layer (``ModelConfig.layer_specs``) run through the same loop: every layer names its mixer (windowed
-attention with kept first tokens and a distance bias, or lightning attention) with sizes of its own, layers may be looped (every
-run has its own cache: ``KvCache`` is indexed by run), and the residual stream is f32.
+attention with kept first tokens and a distance bias, latent attention, lightning attention, HGRN2 or Mamba-2) and its feed-forward (dense or
+a mixture of experts) with sizes of its own, layers may be looped (every run has its own cache: ``KvCache`` is indexed by run), and the
+residual stream is f32.
 """
 from __future__ import annotations
 
@@ -29,9 +30,9 @@ from .. import _native
 from ..ops import attention as att
 from ..ops import elementwise as ew
 from ..ops import deltanet as dn
-from ..ops import gemm, lightning, moe, qlinear, sampling, stream
+from ..ops import gemm, latent, lightning, moe, qlinear, recurrent, sampling, stream
 from ..ops.mxfp8 import MxTensor
-from .config import LayerRun, LayerSpec, ModelConfig
+from .config import LayerRun, LayerSpec, ModelConfig, MoeSpec
 from .weights import LinearWeight, ModelWeights
 from ..utils import profiler
 
@@ -98,24 +99,30 @@ class KvCache:
 
     @staticmethod
     def _allocate_layered(cfg: ModelConfig, num_pages: int, page_size: int, device, n_seq_slots: int, kv_dtype: str) -> "KvCache":
-        """One entry per layer RUN: K / V pages with the layer's own head sizes (attention), or ``rec`` f32 ``[slots, heads, dim, vdim]``
-        (lightning attention)."""
+        """One entry per layer RUN: K / V pages with the layer's own head sizes (attention); pages of latents and rotated key parts in ``k`` (latent
+        attention; nothing for a layer that reads another's); or ``rec`` f32 ``[slots, heads, dim, vdim]``, for Mamba-2 also ``conv`` f32 ``[slots,
+        taps - 1, channels]`` (recurrent layers)."""
         dtypes = {"bf16": torch.bfloat16, "f32": torch.float32}
         if kv_dtype not in dtypes:
             raise ValueError(f"models described layer by layer keep a bf16 or f32 KV cache, not {kv_dtype!r}")
         dt = dtypes[kv_dtype]
         kv = KvCache([], [], page_size, num_pages)
-        kv.rec = []
+        kv.rec, kv.conv = [], []
         for run in cfg.layer_runs():
             sp = cfg.layer_specs[run.layer]
-            lin = sp.mixer == "lightning"
             dkp, dvp = att.cache_head_dims(sp.head_dim, sp.v_dim, dt)
-            rows, heads = (0, 1) if lin else (num_pages * page_size, sp.n_kv_heads)
+            rows, heads = (0, 1) if sp.has_state else (num_pages * page_size, sp.n_kv_heads)
+            if sp.mixer == "latent":
+                rows, dkp, dvp = (rows if sp.kv_from < 0 else 0), stream.row_width(sp.kv_rank + sp.rot_dim, dt), 0
             kv.k.append(torch.zeros(rows, heads, dkp, dtype=dt, device=device))
             kv.v.append(torch.zeros(rows, heads, dvp, dtype=dt, device=device))
-            kv.rec.append(torch.zeros(n_seq_slots, sp.n_heads, sp.head_dim, sp.v_dim, dtype=torch.float32, device=device) if lin else None)
+            f32 = dict(dtype=torch.float32, device=device)
+            kv.rec.append(torch.zeros(n_seq_slots, sp.n_heads, sp.head_dim, sp.v_dim, **f32) if sp.has_state else None)
+            kv.conv.append(torch.zeros(n_seq_slots, sp.conv_taps - 1, sp.conv_channels, **f32) if sp.mixer == "mamba2" else None)
         if not any(r is not None for r in kv.rec):
             kv.rec = None
+        if not any(r is not None for r in kv.conv):
+            kv.conv = None
         return kv
 
     def recurrent(self, li: int) -> List[torch.Tensor]:
@@ -146,7 +153,7 @@ class KvCache:
                 pg[dst.long()] = pg[src.long()]
             return
         for t in list(self.k) + list(self.v):
-            if t.shape[0] == 0:
+            if t.numel() == 0:
                 continue
             if not t.is_cuda:
                 pg = t.view(self.num_pages, self.page_size, *t.shape[1:])
@@ -331,6 +338,11 @@ def apply_linear_stream(lw: LinearWeight, x: torch.Tensor):
     return gemm.linear(x, lw.w, bias=lw.bias, out_dtype=torch.float32, w_tiled=lw.tiled)
 
 
+def apply_linear_rows(lw: LinearWeight, x: torch.Tensor):
+    """A projection for a token-wise kernel: f32 (or K-split partial sums) for decode-sized batches, bf16 rows for prefill-sized ones."""
+    return apply_linear_mixer(lw, x)[0]
+
+
 def apply_linear_mixer(lw: LinearWeight, x: torch.Tensor, silu_rows: int = 0):
     """The input projection of a mixer: as ``apply_linear_stream`` for decode-sized batches (the mixer's kernels add the partial sums), bf16
     rows for prefill-sized ones, with SiLU on the first ``silu_rows`` features.  Returns ``(result, whether SiLU was applied)``."""
@@ -381,6 +393,8 @@ class Transformer:
         self.rope_dim = rd
         self.rope_table = ew.rope_table(min(max(cfg.max_seq_len, 4096), 65536), rd, cfg.rope_theta, weights.embed.device) \
             if weights.embed.is_cuda and not cfg.is_layered else None
+        self.mixer_blocks = {"attention": self.masked_attention_block, "lightning": self.lightning_block, "mamba2": self.mamba2_block, "hgrn2": self.hgrn2_block,
+                             "latent": self.latent_block}
         self.snapshots = {}            # layer -> hidden rows captured after that layer (debug / DeepStack)
         self.snapshot_layers: Sequence[int] = ()
 
@@ -480,6 +494,8 @@ class Transformer:
     def attention_plans(self, q_lens: Sequence[int], max_kv: int, device, decode: bool) -> dict:
         """Work lists for every head shape of the model (made up front where nothing may be allocated later: a captured decode step)."""
         plans = {}
+        if any(sp.mixer == "latent" for sp in (self.cfg.layer_specs or ())):
+            plans["latent"] = self.latent_plan(q_lens, [max_kv] * len(q_lens), max_kv, device, decode)
         for sp in (self.cfg.layer_specs or ()):
             if sp.mixer == "attention" and (sp.n_heads, sp.n_kv_heads, sp.span) not in plans:
                 plans[(sp.n_heads, sp.n_kv_heads, sp.span)] = attention_plan(q_lens, max_kv, sp.n_heads, sp.n_kv_heads, sp.span, device, decode)
@@ -509,7 +525,91 @@ class Transformer:
         y = stream.gated_norm(o, proj, 2 * sp.q_dim + sp.n_heads * sp.v_dim, lw.lin.norm, self.cfg.rms_eps, self.act_dtype)
         return apply_linear_stream(lw.lin.w_out, y)
 
+    def mamba2_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
+        """Mamba-2: projection -> causal convolution + SiLU -> recurrence -> norm of y * SiLU(z) -> output projection.  The step sizes stay f32."""
+        w, nv, most = lw.mamba, sp.n_heads * sp.v_dim, max(fb.q_lens) if fb.q_lens else 1
+        proj, dt, dt_col = self._mixer_rows(w.w_in, h, w.dt_row)
+        xbc = recurrent.causal_conv(proj, nv, w.conv_w, w.conv_b, self.kv.conv[li], fb.cu_q, fb.seq_slots, most, self.act_dtype)
+        y = recurrent.ssd(xbc, dt, dt_col, w.dt_bias, w.a, w.d, self.kv.rec[li], fb.cu_q, fb.seq_slots, sp.n_heads, sp.state_groups, sp.head_dim, sp.v_dim, most)
+        return apply_linear_stream(w.w_out, stream.part_norm(y, w.norm, sp.norm_parts, self.cfg.rms_eps, proj, 0, self.act_dtype))
+
+    def hgrn2_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
+        """HGRN2: projection -> SiLU(q), recurrence with a forget gate per key channel (f32) -> RMSNorm per head -> output projection."""
+        w = lw.gla
+        qv, gate, col = self._mixer_rows(w.w_in, h, w.f_row, silu_rows=sp.q_dim)
+        o = recurrent.gla(qv, gate, col, w.f_bias, w.lower, self.kv.rec[li], fb.cu_q, fb.seq_slots, sp.n_heads, sp.head_dim, sp.v_dim, activated=qv is not gate,
+                          max_tokens=max(fb.q_lens) if fb.q_lens else 1)
+        return apply_linear_stream(w.w_out, stream.part_norm(o, w.norm, sp.n_heads, self.cfg.rms_eps, out_dtype=self.act_dtype))
+
+    @staticmethod
+    def _mixer_rows(w_in: LinearWeight, h: torch.Tensor, at: int, silu_rows: int = 0):
+        """Input projection whose features from ``at`` on feed a recurrence's gates and stay f32: (rows, result that holds the gates, their column).
+        One product for decode-sized batches; for prefill-sized ones bf16 rows (with SiLU on the first ``silu_rows``) and an f32 product."""
+        if w_in.fmt == "f32" or h.shape[0] <= 64:
+            proj = apply_linear_stream(w_in, h)
+            return proj, proj, at
+        main, gates = w_in.rows(0, at), w_in.rows(at, w_in.n)
+        return gemm.linear(h, main.w, w_tiled=main.tiled, silu_rows=silu_rows), gemm.linear(h, gates.w, out_dtype=torch.float32, w_tiled=gates.tiled), 0
+
+    def latent_plan(self, q_lens, kv_lens, max_kv: int, device, decode: bool) -> latent.LatentPlan:
+        specs = [sp for sp in self.cfg.layer_specs if sp.mixer == "latent"]
+        expand = torch.device(device).type == "cuda" and self.act_dtype == torch.bfloat16 and all(latent.can_expand(sp) for sp in specs)
+        return latent.make_plan(q_lens, kv_lens, max_kv, device, decode, expand, sorted({sp.n_heads for sp in specs}))
+
+    def latent_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
+        """Latent attention: q and kv latents -> norms, cache store -> query heads -> attention over the cached latents (absorbed) or over keys and values
+        expanded from them -> output projection.  A layer with ``kv_from`` reads the cache of that layer."""
+        w, dt, dev = lw.latent, self.act_dtype, h.device
+        hd, d, rd, r = sp.n_heads, sp.head_dim, sp.rot_dim, sp.kv_rank
+        cache = self.kv.k[li if sp.kv_from < 0 else sp.kv_from]
+        if fb.plans is None:
+            fb.plans = {}
+        plan = fb.plans.get("latent")
+        if plan is None:
+            plan = fb.plans["latent"] = self.latent_plan(fb.q_lens, fb.kv_lens, max(fb.kv_lens), dev, fb.is_decode)
+        mag = sp.rotary.magnitude
+        cq = latent.latent_store(apply_linear_rows(w.w_a, h), fb.positions, fb.slots, w.q_norm, w.kv_norm, w.freq, mag, cache, sp.q_rank, r, rd, self.cfg.rms_eps, dt)
+        q = apply_linear_rows(w.w_qb, cq)
+        dp, vp, rp = (stream.row_width(n, dt) for n in (d, sp.v_dim, rd))
+        a = torch.empty(h.shape[0], hd * vp, dtype=dt, device=dev)
+        qa = qn = en = er = None
+        if plan.n_abs:
+            qa, qn = torch.empty(hd, plan.m, cache.shape[2], dtype=dt, device=dev), torch.empty(hd, plan.m, dp, dtype=dt, device=dev)
+        if plan.n_exp:
+            en, er = torch.empty(plan.n_exp, hd, dp, dtype=dt, device=dev), torch.empty(plan.n_exp, hd, rp, dtype=dt, device=dev)
+        latent.latent_q(q, fb.positions, w.freq, mag, sp.scale * att.LOG2E, plan.dst, (qn.transpose(0, 1), qa[:, :, r:].transpose(0, 1)) if qa is not None else None,
+                        (en, er) if en is not None else None, hd, d, rd)
+        if qa is not None:
+            seg, cnt, rows = plan.groups(hd, dev)
+            if dt == torch.float32:
+                gemm.batched_linear_f32(qn, w.w_uk.w.view(hd, r, d), qa[:, :, :r])
+            else:
+                gemm.grouped_linear(qn.view(-1, dp), w.w_uk.w.view(hd, -1, dp), seg, cnt, plan.tile, out=qa.view(-1, cache.shape[2]), n_out=r, w_tiled=w.w_uk.tiled)
+            o = latent.attend_latents(qa, cache, r, r + rd, plan, fb, self.kv.page_size, w.sink)
+            if dt == torch.float32:
+                # nothing is expanded in f32: the absorbed rows are the tokens in order
+                gemm.batched_linear_f32(o[:, : plan.n_abs], w.w_uv.w.view(hd, vp, r), a.view(-1, hd, vp).transpose(0, 1))
+            else:
+                gemm.grouped_linear(o.view(-1, o.shape[2]), w.w_uv.w.view(hd, vp, -1), seg, cnt, plan.tile, out=a.view(-1, vp), row_map=rows, n_out=vp, w_tiled=w.w_uv.tiled)
+        if en is not None:
+            rows_kv = latent.gather_latents(cache, plan, fb.block_table, self.kv.page_size)
+            kvx = gemm.linear(rows_kv[:, : w.w_kv.k], w.w_kv.w, w_tiled=w.w_kv.tiled)
+            latent.attend_expanded(en, er, kvx, rows_kv, r, plan, w.sink, a.view(-1, hd, vp))
+        return apply_linear_stream(lw.wo, a)
+
+    def stream_moe(self, lw, m: MoeSpec, h: torch.Tensor):
+        """Mixture of experts of a layer described by ``LayerSpec``; the weighted sum stays pending for the stream's norm."""
+        rt = dict(mode=m.router, renorm=2 if m.renorm else 0, routed_scale=m.scale, groups=(m.groups, m.groups_kept))
+        if lw.w13.fmt != "f32":
+            return self.moe_local(lw, h, spec=m, rt=rt)
+        ids, wts, pl = moe.route_plan(gemm.linear_f32(h, lw.router), m.top, m.n_experts, 64, **rt)
+        gu = gemm.grouped_linear_f32(h, lw.w13.w.view(m.n_experts, -1, h.shape[1]), pl.seg_start, pl.seg_count, pl.capacity, pl.row_token)
+        y = gemm.grouped_linear_f32(stream.act_mul(gu, "silu"), lw.w2.w.view(m.n_experts, -1, lw.w2.k), pl.seg_start, pl.seg_count, pl.capacity)
+        return moe.PendingCombine(y, pl.pair_row, wts, h.shape[0], m.top)
+
     def stream_ffn(self, lw, sp: LayerSpec, h: torch.Tensor):
+        if sp.moe is not None:
+            return self.stream_moe(lw, sp.moe, h)
         gu = lw.w_gate_up
         if gu.fmt == "f32":
             return apply_linear_stream(lw.w_down, stream.act_mul(gemm.linear_f32(h, gu.w), sp.act))
@@ -554,14 +654,18 @@ class Transformer:
             act = gemm.linear_mx_swiglu_quant(xm, gu.mx)
         return self.par.row_linear(lw.w_down, None, act)
 
-    def moe_local(self, lw, h: torch.Tensor, h_mx: Optional[MxTensor] = None, local_range=None) -> torch.Tensor:
+    def moe_local(self, lw, h: torch.Tensor, h_mx: Optional[MxTensor] = None, local_range=None, spec: Optional[MoeSpec] = None, rt=None) -> torch.Tensor:
         """The experts held by this GPU over the rows ``h``: route -> plan -> (gather + quantise) -> gate/up -> down -> combine.
         ``local_range = (first expert, count)``: the weights are that slice of the experts; (token, expert) pairs routed
-        elsewhere are dropped from the plan and contribute nothing to the pending sum (the caller adds the ranks' sums)."""
+        elsewhere are dropped from the plan and contribute nothing to the pending sum (the caller adds the ranks' sums).
+        ``spec`` / ``rt``: sizes and routing rule of one layer (models described layer by layer) instead of the model's."""
         cfg = self.cfg
         t = h.shape[0]
         e, k, inter, hid = (local_range[1] if local_range else cfg.n_experts), cfg.n_experts_used, cfg.expert_ffn, cfg.hidden
-        rt = dict(mode=cfg.router, bias=lw.router_bias, renorm=cfg.norm_topk, routed_scale=cfg.routed_scale, local_range=local_range)
+        n_exp = cfg.n_experts
+        if spec is not None:
+            e, n_exp, k, inter, hid = spec.n_experts, spec.n_experts, spec.top, lw.w2.k, lw.w13.k
+        rt = rt or dict(mode=cfg.router, bias=lw.router_bias, renorm=cfg.norm_topk, routed_scale=cfg.routed_scale, local_range=local_range)
         if self.mx:
             # token tile (= scale-atom layout) by the expected rows per expert: 32 for decode-sized batches
             tn = 32 if (t * k) // cfg.n_experts <= 24 else 128
@@ -583,14 +687,14 @@ class Transformer:
                 y = gemm.grouped_linear(hq, lw.w2.mx.data.view(e, hid, inter), pl.seg_start, pl.seg_count, tn, sfa=lw.w2.mx.sf, sfb=hsf,
                                         w_tiled=lw.w2.mx.tiled, pair_rows=(tn == 32 and PAIR_DOWN))
         else:
-            tn = gemm.pick_tn(max(1, (t * k + cfg.n_experts - 1) // cfg.n_experts), dual=True)
+            tn = gemm.pick_tn(max(1, (t * k + n_exp - 1) // n_exp), dual=True)
             if moe.can_prep(h, lw.router, k):
                 ids, wts, pl, xs = moe.prep_hidden(h, lw.router, k, e, tn, quantize=False, **rt)
             else:
                 ids, wts, pl = moe.route_plan_hidden(h, lw.router, k, e, tn, **rt)
                 xs = moe.gather_rows(h, pl.row_token)
             act = gemm.grouped_linear(xs, lw.w13.w.view(e, 2 * inter, hid), pl.seg_start, pl.seg_count, tn, dual=True, w_tiled=lw.w13.tiled)
-            y = gemm.grouped_linear(act, lw.w2.w.view(e, hid, inter), pl.seg_start, pl.seg_count, tn, w_tiled=lw.w2.tiled)
+            y = gemm.grouped_linear(act, lw.w2.w.view(e, -1, inter), pl.seg_start, pl.seg_count, tn, w_tiled=lw.w2.tiled)
         return moe.PendingCombine(y, pl.pair_row, wts, t, k)
 
     # ------------------------------------------------------------------------------------------------
@@ -600,7 +704,7 @@ class Transformer:
         cfg, w = self.cfg, self.w
         last_layer = len(self.runs) if last_layer is None else last_layer
         if x is None and self.stream_f32:
-            x = stream.embed(fb.ids, w.embed) if fb.embeds is None else fb.embeds.float()
+            x = stream.embed(fb.ids, w.embed, cfg.embed_scale) if fb.embeds is None else fb.embeds.float()
         elif x is None:
             x = fb.embeds if fb.embeds is not None else ew.embed(fb.ids, w.embed)
         delta = None
@@ -615,13 +719,17 @@ class Transformer:
                 sp, step = cfg.layer_specs[self.runs[li].layer], self.runs[li].step
                 h = stream.norm(x, lw.attn_norm, cfg.rms_eps, delta, add=w.loop_step[step] if step >= 0 else None, out_dtype=self.act_dtype)
                 with profiler.region(sp.mixer, "block", "attention", li):
-                    delta = self.lightning_block(li, lw, sp, h, fb) if sp.mixer == "lightning" else self.masked_attention_block(li, lw, sp, h, fb)
-                if sp.ffn:
+                    delta = self.mixer_blocks[sp.mixer](li, lw, sp, h, fb)
+                if lw.attn_post is not None:
+                    delta = stream.PostNormed(delta, lw.attn_post)
+                if sp.has_ffn:
                     h = stream.norm(x, lw.ffn_norm, cfg.rms_eps, delta, out_dtype=self.act_dtype)
                     with profiler.region("ffn", "block", "ffn", li):
                         delta = self.stream_ffn(lw, sp, h)
+                    if lw.ffn_post is not None:
+                        delta = stream.PostNormed(delta, lw.ffn_post)
                 if li in self.snapshot_layers:
-                    self.snapshots[li] = x + stream.whole(delta)
+                    self.snapshots[li] = x + stream.whole(delta)[:, : x.shape[1]]
                 continue
             lay = 32 if x.shape[0] <= 32 else 128
             par = self.par
@@ -701,7 +809,7 @@ class Transformer:
         if self._last_delta is None:
             return x
         if self.stream_f32:
-            return x + stream.whole(self._last_delta)
+            return x + stream.whole(self._last_delta)[:, : x.shape[1]]
         return (x.float() + self._last_delta.float()).to(torch.bfloat16)
 
 
