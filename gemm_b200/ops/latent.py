@@ -213,7 +213,8 @@ def attend_latents(q: torch.Tensor, cache: torch.Tensor, rank: int, width: int, 
     heads, m, _ = q.shape
     if not q.is_cuda:
         return attend_latents_ref(q, cache, rank, width, plan, fb, page_size, sink)
-    out = torch.empty(heads, m, row_width(rank, cache.dtype), dtype=q.dtype, device=q.device)
+    wo = row_width(rank, cache.dtype)
+    out = (torch.empty if wo == rank else torch.zeros)(heads, m, wo, dtype=q.dtype, device=q.device)      # the padding meets zero weights: finite
     lib = _native.cuda()
     rc = lib.gb_attn_latent_any(_p(q), _l(q.stride(1)), _l(q.stride(0)), _p(cache), _i(cache.shape[2]), _p(out), _l(out.stride(1)), _l(out.stride(0)),
                                 _i(int(q.dtype == torch.float32)), _p(fb.cu_q), _p(fb.kv_len), _p(plan.abs_seq), _p(plan.abs_kv), _p(fb.block_table),

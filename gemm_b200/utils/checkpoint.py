@@ -64,6 +64,8 @@ def save_state(engine, path: str, next_tokens=None, kv_format: str = "bf16") -> 
                     f.write(t[:n_seq].contiguous().cpu().numpy().tobytes())
                 continue
             for t in (engine.kv.k[li], engine.kv.v[li]):
+                if t.shape[2] == 0:
+                    continue                     # latent attention keeps no values of their own
                 rows = t[idx].contiguous()
                 if kv_format == "q8":
                     q, sc = kvquant.quantize_q8(rows)
@@ -112,12 +114,16 @@ def load_state(engine, path: str) -> torch.Tensor:
             if engine.kv.k[li].shape[0] == 0:
                 for t in engine.kv.recurrent(li):
                     nb = n_seq * t[0].numel() * 4
+                    if nb == 0:
+                        continue
                     buf = f.read(nb)
                     if len(buf) != nb:
                         raise ValueError("truncated KV state file")
                     t[:n_seq] = torch.frombuffer(bytearray(buf), dtype=torch.float32).reshape(n_seq, *t.shape[1:]).to(engine.device)
                 continue
             for t in (engine.kv.k[li], engine.kv.v[li]):
+                if t.shape[2] == 0:
+                    continue                     # latent attention keeps no values of their own
                 row = t.shape[1] * t.shape[2] * t.element_size()
                 if kv_format == "q8":
                     nq, ns = len(slots) * t.shape[1] * t.shape[2], len(slots) * t.shape[1] * 4
