@@ -22,6 +22,7 @@
 // (common/transformer.h:1333-1530).
 #include "sm100.cuh"
 #include "host_common.h"
+#include "flash_common.cuh"
 
 namespace gb {
 
@@ -68,12 +69,6 @@ __device__ __forceinline__ FaBlocks fa_blocks(const FaArgs& a, int first_pos, in
   b.n_keep = min((a.keep_first + 127) / 128, b.lo);
   b.n = b.n_keep + max(0, last_pos / 128 + 1 - b.lo);
   return b;
-}
-
-__device__ __forceinline__ float fast_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
 }
 
 constexpr int kFaSmem = 32768 * 3 + 256 + 1024;
@@ -420,27 +415,6 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
 constexpr int kFdN = 16;                 // MMA N: query heads of one KV head, zero padded
 constexpr int kFdThreads = 192;
 constexpr int kFdSmem = 4096 + 3 * 32768 + 8192 + 2048 + 1024;   // Q, tile ring, P x2, barriers + reductions, alignment
-
-// Reduce 16 per-lane values over the 32 lanes of a warp with 16 shuffles (a reduce-scatter: 8 + 4 + 2 + 1 exchanges, then one
-// more between neighbours): lane L returns the result for index L >> 1.
-#define GB_RS_STEP(IN, OUT, N, BIT, OP)                                                       \
-  _Pragma("unroll") for (int i = 0; i < N; ++i) {                                            \
-    const bool up = (lane & BIT) != 0;                                                       \
-    const float send = up ? IN[i] : IN[N + i], keep = up ? IN[N + i] : IN[i];                 \
-    OUT[i] = OP(keep, __shfl_xor_sync(0xffffffffu, send, BIT));                               \
-  }
-__device__ __forceinline__ float rs_max(float a, float b) { return fmaxf(a, b); }
-__device__ __forceinline__ float rs_add(float a, float b) { return a + b; }
-__device__ __forceinline__ float warp_reduce16_max(const float* v, int lane) {
-  float a[8], b[4], c[2], d[1];
-  GB_RS_STEP(v, a, 8, 16, rs_max) GB_RS_STEP(a, b, 4, 8, rs_max) GB_RS_STEP(b, c, 2, 4, rs_max) GB_RS_STEP(c, d, 1, 2, rs_max)
-  return fmaxf(d[0], __shfl_xor_sync(0xffffffffu, d[0], 1));
-}
-__device__ __forceinline__ float warp_reduce16_sum(const float* v, int lane) {
-  float a[8], b[4], c[2], d[1];
-  GB_RS_STEP(v, a, 8, 16, rs_add) GB_RS_STEP(a, b, 4, 8, rs_add) GB_RS_STEP(b, c, 2, 4, rs_add) GB_RS_STEP(c, d, 1, 2, rs_add)
-  return d[0] + __shfl_xor_sync(0xffffffffu, d[0], 1);
-}
 
 template <int DK, int DV, bool EXT>
 __global__ void __launch_bounds__(kFdThreads, 2)

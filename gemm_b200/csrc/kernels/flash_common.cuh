@@ -1,0 +1,34 @@
+// Helpers shared by the attention kernels.
+#pragma once
+#include "sm100.cuh"
+
+namespace gb {
+
+__device__ __forceinline__ float fast_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// Reduce 16 per-lane values over the 32 lanes of a warp with 16 shuffles (a reduce-scatter: 8 + 4 + 2 + 1 exchanges, then one
+// more between neighbours): lane L returns the result for index L >> 1.
+#define GB_RS_STEP(IN, OUT, N, BIT, OP)                                                       \
+  _Pragma("unroll") for (int i = 0; i < N; ++i) {                                            \
+    const bool up = (lane & BIT) != 0;                                                       \
+    const float send = up ? IN[i] : IN[N + i], keep = up ? IN[N + i] : IN[i];                 \
+    OUT[i] = OP(keep, __shfl_xor_sync(0xffffffffu, send, BIT));                               \
+  }
+__device__ __forceinline__ float rs_max(float a, float b) { return fmaxf(a, b); }
+__device__ __forceinline__ float rs_add(float a, float b) { return a + b; }
+__device__ __forceinline__ float warp_reduce16_max(const float* v, int lane) {
+  float a[8], b[4], c[2], d[1];
+  GB_RS_STEP(v, a, 8, 16, rs_max) GB_RS_STEP(a, b, 4, 8, rs_max) GB_RS_STEP(b, c, 2, 4, rs_max) GB_RS_STEP(c, d, 1, 2, rs_max)
+  return fmaxf(d[0], __shfl_xor_sync(0xffffffffu, d[0], 1));
+}
+__device__ __forceinline__ float warp_reduce16_sum(const float* v, int lane) {
+  float a[8], b[4], c[2], d[1];
+  GB_RS_STEP(v, a, 8, 16, rs_add) GB_RS_STEP(a, b, 4, 8, rs_add) GB_RS_STEP(b, c, 2, 4, rs_add) GB_RS_STEP(c, d, 1, 2, rs_add)
+  return d[0] + __shfl_xor_sync(0xffffffffu, d[0], 1);
+}
+
+}  // namespace gb

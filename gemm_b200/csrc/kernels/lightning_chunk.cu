@@ -9,6 +9,9 @@
 //   MMA thread  : S1 = Q K^T;  dS = K^T (w V);  O1 = Q S;  O2 = P V         (A of O2 is P in TMEM; S and w V are written to smem)
 //   P warps     : S1 row -> times g^(i-j), lower triangle -> P in TMEM;  g^(i+1) O1 + O2 -> global f32 (TMA)
 //   state warps : V -> w V in smem;  S <- g^n S + dS;  S -> smem for the next chunk's O1
+// The SSD form (Mamba-2) is the same scan with a decay per token: with L_i the sum of a dt log2(e) up to token i of the chunk, g^(i-j) becomes
+// 2^(L_i - L_j) dt_j (one exponential of L_i - (L_j - log2 dt_j)), w of a token 2^(L_n-1 - L_j) dt_j, and D x_i joins P's diagonal.  q and k are C
+// and B of the head's group.  Every warp of the two groups sums the chunk's step sizes itself, so they need no exchange.
 // Every f32 factor that goes through the tensor cores (P, w V, S) is the sum of two bf16 operands (hi + lo, 16 bits of mantissa), so
 // decays and state keep 32-bit accuracy; only q, k and v themselves are bf16.
 #include "sm100.cuh"
@@ -32,9 +35,46 @@ struct LightningChunkArgs {
   float* out; int ld_out;       // [tokens, heads * vdim] f32
   int heads, dim, vdim;
   KernelStatus* status;
+  // SSD
+  const float* gate; int g_part; long g_stride; int g_ld;       // step sizes before bias and softplus, [g_part][tokens, g_ld], column = head
+  const float* gate_bias; const float* d_skip; int groups;      // `decay` holds a (negative)
 };
 
-template <int DP>                          // key size padded: 64 or 128
+__device__ __forceinline__ float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+
+// Step sizes of a chunk, of token 32 b + lane for b = 0 .. 3, before bias and softplus.
+__device__ __forceinline__ void ssd_load(const LightningChunkArgs& a, int t0, int n, int h, int lane, float* raw) {
+#pragma unroll
+  for (int b = 0; b < 4; ++b) {
+    raw[b] = 0.f;
+    if (32 * b + lane < n) {
+      const float* p = a.gate + (size_t)(t0 + 32 * b + lane) * a.g_ld + h;
+      for (int i = 0; i < a.g_part; ++i) raw[b] += p[(size_t)i * a.g_stride];
+    }
+  }
+}
+
+// Sum of the logarithmic decays (base 2) up to token 32 q + lane, the step size of that token, and the chunk's total; every warp gets the same sums.
+__device__ __forceinline__ void ssd_scan(const float* raw, int n, float bias, float a2, int q, int lane, float& L, float& dt, float& total) {
+  float base = 0.f, own = 0.f;
+  total = 0.f; dt = 0.f;
+#pragma unroll
+  for (int b = 0; b < 4; ++b) {
+    const float d = 32 * b + lane < n ? softplus_exact(raw[b] + bias) : 0.f;
+    const float l = a2 * d;
+    if (b == q) { dt = d; own = l; base = total; }
+    total += warp_sum(l);
+  }
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, own, o); if (lane >= o) own += v; }
+  L = base + own;
+}
+
+template <int DP, bool SSD>                // DP: key size padded, 64 or 128
 __global__ void __launch_bounds__(kLcThreads, 1)
 lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
                        const __grid_constant__ CUtensorMap tmO, const LightningChunkArgs a) {
@@ -71,7 +111,9 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   pdl_wait();
   const int h = blockIdx.x, e0 = blockIdx.y * kLcV, seq = blockIdx.z;
   const float g = a.decay[h];
-  for (int i = threadIdx.x; i < 257; i += kLcThreads) pz[i] = i < 128 ? 0.f : i == 128 ? 1.f : powf(g, (float)(i - 128));
+  if constexpr (!SSD) { for (int i = threadIdx.x; i < 257; i += kLcThreads) pz[i] = i < 128 ? 0.f : i == 128 ? 1.f : powf(g, (float)(i - 128)); }
+  const int hk = SSD ? h / (a.heads / a.groups) : h;            // head of q and k
+  const float a2 = SSD ? g * 1.4426950408889634f : 0.f, dt_bias = SSD ? a.gate_bias[h] : 0.f;
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -89,11 +131,11 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
         uint8_t* st = smem + b * kLcStage;
         if (!mbar_wait(&t_empty[b], ((uint32_t)(j >> 1) & 1) ^ 1, abort_flag, a.status, 700, j)) break;
         mbar_expect_tx(&qk_full[b], 4u * kLcC * DP);
-        tma_load_3d(st, &tmQ, &qk_full[b], 0, h, t0);
-        tma_load_3d(st + kLcQ, &tmK, &qk_full[b], 0, h, t0);
+        tma_load_3d(st, &tmQ, &qk_full[b], 0, hk, t0);
+        tma_load_3d(st + kLcQ, &tmK, &qk_full[b], 0, hk, t0);
         if constexpr (DP > 64) {
-          tma_load_3d(st + 16384, &tmQ, &qk_full[b], 64, h, t0);
-          tma_load_3d(st + kLcQ + 16384, &tmK, &qk_full[b], 64, h, t0);
+          tma_load_3d(st + 16384, &tmQ, &qk_full[b], 64, hk, t0);
+          tma_load_3d(st + kLcQ + 16384, &tmK, &qk_full[b], 64, hk, t0);
         }
         mbar_expect_tx(&v_full[b], 2u * kLcC * kLcV);
         tma_load_3d(st + 2 * kLcQ, &tmV, &v_full[b], e0, h, t0);
@@ -154,11 +196,23 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     const int q = warp & 3, i = q * 32 + lane;
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     const float* pw = pz + 128;
-    const float gi = pw[i + 1];
+    float gi = SSD ? 0.f : pw[i + 1];
+    const float skip = SSD ? a.d_skip[h] : 0.f;
+    float raw[4];
+    if (SSD && n_chunks > 0) ssd_load(a, t_begin, min(kLcC, t_end - t_begin), h, lane, raw);
     bool staged = false;                    // the output tile of the previous chunk is on its way out of stage (j - 1) & 1
     for (int j = 0; j < n_chunks; ++j) {
       const uint32_t ph = j & 1;
       const int b = j & 1, t0 = t_begin + j * kLcC;
+      float Li = 0.f;
+      if constexpr (SSD) {
+        float dt, total;
+        ssd_scan(raw, min(kLcC, t_end - t0), dt_bias, a2, q, lane, Li, dt, total);
+        pz[i] = Li - log2f(dt);             // (read by everyone below; the barrier at the end of the chunk lets the next one overwrite it)
+        gi = ex2(Li);
+        if (j + 1 < n_chunks) ssd_load(a, t0 + kLcC, min(kLcC, t_end - t0 - kLcC), h, lane, raw);
+        bar128_and(true);
+      }
       bool ok = warp_wait(s1_full, ph, abort_flag, a.status, 720, j);
       tc_fence_after();
       if (ok) {
@@ -170,13 +224,20 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
             tmem_ld_x32(t_s1 + lane_off + c * 32, reinterpret_cast<uint32_t*>(s));
             float w[32];                    // zero above the diagonal
 #pragma unroll
-            for (int x = 0; x < 32; ++x) { w[x] = (pw + (i - c * 32))[-x]; asm volatile("" : "+f"(w[x])); }
+            for (int x = 0; x < 32; ++x) {
+              if constexpr (SSD) w[x] = pz[c * 32 + x];
+              else { w[x] = (pw + (i - c * 32))[-x]; asm volatile("" : "+f"(w[x])); }
+            }
+            if constexpr (SSD) {
+#pragma unroll
+              for (int x = 0; x < 32; ++x) w[x] = ex2(Li - w[x]);       // above the diagonal anything, cleared below
+            }
             tc_wait_ld();
 #pragma unroll
             for (int x = 0; x < 32; ++x) s[x] *= w[x];
             if (c == q) {
 #pragma unroll
-              for (int x = 0; x < 32; ++x) s[x] = x <= lane ? s[x] : 0.f;
+              for (int x = 0; x < 32; ++x) s[x] = x < lane ? s[x] : x == lane ? (SSD ? s[x] + skip : s[x]) : 0.f;
             }
 #pragma unroll
             for (int x = 0; x < 16; ++x) split_bf16x2(s[2 * x], s[2 * x + 1], hi[x], lo[x]);
@@ -255,16 +316,23 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       mbar_arrive(s_ready);
     };
     bool ok = true;
+    float raw[4];
+    if (SSD && n_chunks > 0) ssd_load(a, t_begin, min(kLcC, t_end - t_begin), h, lane, raw);
     if (n_chunks > 0) publish();
     for (int j = 0; j < n_chunks; ++j) {
       const uint32_t ph = j & 1;
       const int b = j & 1, n = min(kLcC, t_end - (t_begin + j * kLcC));
+      float L = 0.f, dt = 0.f, total = 0.f;
+      if constexpr (SSD) {
+        ssd_scan(raw, n, dt_bias, a2, q, lane, L, dt, total);
+        if (j + 1 < n_chunks) ssd_load(a, t_begin + (j + 1) * kLcC, min(kLcC, t_end - t_begin - (j + 1) * kLcC), h, lane, raw);
+      }
       // w V: a token's values times what its contribution still decays by until the end of the chunk
       if (!warp_wait(&v_full[b], (uint32_t)(j >> 1) & 1, abort_flag, a.status, 730, j)) { ok = false; break; }
       {
         const uint8_t* sV = smem + b * kLcStage + 2 * kLcQ;
         const bool live = d < n;
-        const float w = live ? pw[n - 1 - d] : 0.f;
+        const float w = !live ? 0.f : SSD ? ex2(total - L) * dt : pw[n - 1 - d];
 #pragma unroll
         for (int c = 0; c < 8; ++c) {
           const int off = d * 128 + ((c ^ (d & 7)) << 4);
@@ -284,7 +352,7 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       }
       if (!warp_wait(ds_full, ph, abort_flag, a.status, 731, j)) { ok = false; break; }
       tc_fence_after();
-      const float gn = pw[n];
+      const float gn = SSD ? ex2(total) : pw[n];
 #pragma unroll
       for (int c = 0; c < 2; ++c) {
         float x[32];
@@ -317,16 +385,16 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
   if (warp == 1) { tc_fence_after(); tmem_dealloc(tmem_base, 512); }
 }
 
-template <int DP>
+template <int DP, bool SSD>
 static int lightning_chunk_launch(const CUtensorMap& tmQ, const CUtensorMap& tmK, const CUtensorMap& tmV, const CUtensorMap& tmO, const LightningChunkArgs& a, int n_seqs,
                                   cudaStream_t stream) {
   static bool attr_set = false;
   if (!attr_set) {
-    GB_CUDA_OK(cudaFuncSetAttribute(lightning_chunk_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLcSmem));
+    GB_CUDA_OK(cudaFuncSetAttribute(lightning_chunk_kernel<DP, SSD>, cudaFuncAttributeMaxDynamicSharedMemorySize, kLcSmem));
     attr_set = true;
   }
   const dim3 grid((unsigned)a.heads, (unsigned)((a.vdim + kLcV - 1) / kLcV), (unsigned)n_seqs);
-  launch_k(lightning_chunk_kernel<DP>, grid, kLcThreads, kLcSmem, stream, tmQ, tmK, tmV, tmO, a);
+  launch_k(lightning_chunk_kernel<DP, SSD>, grid, kLcThreads, kLcSmem, stream, tmQ, tmK, tmV, tmO, a);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -335,28 +403,53 @@ static int lightning_chunk_launch(const CUtensorMap& tmQ, const CUtensorMap& tmK
 
 using namespace gb;
 
+// Tensor maps and launch: q, k [tokens, qk_heads, dim] and v [tokens, heads, vdim] inside bf16 rows of pitch ld.
+template <bool SSD>
+static int chunk_launch(const void* q, const void* k, const void* v, int ld, int tokens, int qk_heads, LightningChunkArgs& a, int n_seqs, cudaStream_t stream) {
+  if (a.heads < 1 || a.dim < 8 || a.dim > 128 || a.dim % 8 || a.vdim < 8 || a.vdim % 8) return fail("lightning_chunk: dim <= 128, dim and vdim multiples of 8%s");
+  if (ld % 8 || a.ld_out < a.heads * a.vdim || a.ld_out % 4) return fail("lightning_chunk: bad row pitch%s");
+  if (((uintptr_t)q & 15) || ((uintptr_t)k & 15) || ((uintptr_t)v & 15) || ((uintptr_t)a.state & 15) || ((uintptr_t)a.out & 15)) return fail("lightning_chunk: misaligned rows%s");
+  if (n_seqs > 65535 || (a.vdim + kLcV - 1) / kLcV > 65535) return fail("lightning_chunk: too many sequences%s");
+  const int dim = a.dim, vdim = a.vdim;
+  CUtensorMap tmQ, tmK, tmV, tmO;
+  uint32_t box[3] = {64, 1, (uint32_t)kLcC};
+  uint64_t dk[3] = {(uint64_t)dim, (uint64_t)qk_heads, (uint64_t)tokens}, dv[3] = {(uint64_t)vdim, (uint64_t)a.heads, (uint64_t)tokens};
+  uint64_t sk[2] = {(uint64_t)dim * 2, (uint64_t)ld * 2}, sv[2] = {(uint64_t)vdim * 2, (uint64_t)ld * 2};
+  if (make_tmap(&tmQ, q, TM_BF16, 3, dk, sk, box, TM_SW_128)) return -1;
+  if (make_tmap(&tmK, k, TM_BF16, 3, dk, sk, box, TM_SW_128)) return -1;
+  if (make_tmap(&tmV, v, TM_BF16, 3, dv, sv, box, TM_SW_128)) return -1;
+  uint32_t obox[3] = {32, 1, (uint32_t)kLcC};
+  uint64_t so[2] = {(uint64_t)vdim * 4, (uint64_t)a.ld_out * 4};
+  if (make_tmap(&tmO, a.out, TM_F32, 3, dv, so, obox, TM_SW_128)) return -1;
+  return dim <= 64 ? lightning_chunk_launch<64, SSD>(tmQ, tmK, tmV, tmO, a, n_seqs, stream) : lightning_chunk_launch<128, SSD>(tmQ, tmK, tmV, tmO, a, n_seqs, stream);
+}
+
 // proj: bf16 rows [tokens, ld] with columns [q heads x dim | k heads x dim | v heads x vdim | ...], SiLU applied; dim <= 128, dim and vdim
 // multiples of 8.  state and out as in gb_lightning_step.
 GB_API int gb_lightning_chunk(const void* proj, int ld, int tokens, const float* decay, float* state, int n_slots, const int* cu_q, const int* seq_slots,
                               float* out, int ld_out, int heads, int dim, int vdim, int n_seqs, void* status, cudaStream_t stream) {
   if (n_seqs <= 0 || tokens <= 0) return 0;
-  if (heads < 1 || dim < 8 || dim > 128 || dim % 8 || vdim < 8 || vdim % 8) return fail("lightning_chunk: dim <= 128, dim and vdim multiples of 8%s");
-  if (ld % 8 || ld < 2 * heads * dim + heads * vdim || ld_out < heads * vdim || ld_out % 4) return fail("lightning_chunk: bad row pitch%s");
-  if (((uintptr_t)proj & 15) || ((uintptr_t)state & 15) || ((uintptr_t)out & 15)) return fail("lightning_chunk: misaligned rows%s");
-  if (n_seqs > 65535 || (vdim + kLcV - 1) / kLcV > 65535) return fail("lightning_chunk: too many sequences%s");
+  if (ld < 2 * heads * dim + heads * vdim) return fail("lightning_chunk: bad row pitch%s");
   const __nv_bfloat16* p = (const __nv_bfloat16*)proj;
-  CUtensorMap tmQ, tmK, tmV, tmO;
-  uint32_t box[3] = {64, 1, (uint32_t)kLcC};
-  uint64_t dk[3] = {(uint64_t)dim, (uint64_t)heads, (uint64_t)tokens}, dv[3] = {(uint64_t)vdim, (uint64_t)heads, (uint64_t)tokens};
-  uint64_t sk[2] = {(uint64_t)dim * 2, (uint64_t)ld * 2}, sv[2] = {(uint64_t)vdim * 2, (uint64_t)ld * 2};
-  if (make_tmap(&tmQ, p, TM_BF16, 3, dk, sk, box, TM_SW_128)) return -1;
-  if (make_tmap(&tmK, p + (size_t)heads * dim, TM_BF16, 3, dk, sk, box, TM_SW_128)) return -1;
-  if (make_tmap(&tmV, p + (size_t)2 * heads * dim, TM_BF16, 3, dv, sv, box, TM_SW_128)) return -1;
-  uint32_t obox[3] = {32, 1, (uint32_t)kLcC};
-  uint64_t so[2] = {(uint64_t)vdim * 4, (uint64_t)ld_out * 4};
-  if (make_tmap(&tmO, out, TM_F32, 3, dv, so, obox, TM_SW_128)) return -1;
   LightningChunkArgs a;
+  memset(&a, 0, sizeof(a));
   a.decay = decay; a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out; a.ld_out = ld_out;
   a.heads = heads; a.dim = dim; a.vdim = vdim; a.status = (KernelStatus*)status;
-  return dim <= 64 ? lightning_chunk_launch<64>(tmQ, tmK, tmV, tmO, a, n_seqs, stream) : lightning_chunk_launch<128>(tmQ, tmK, tmV, tmO, a, n_seqs, stream);
+  return chunk_launch<false>(p, p + (size_t)heads * dim, p + (size_t)2 * heads * dim, ld, tokens, heads, a, n_seqs, stream);
+}
+
+// xbc: bf16 rows [tokens, ld] with columns [x heads x vdim | B groups x dim | C groups x dim | ...]; the other arguments as in gb_recurrent_step.
+GB_API int gb_ssd_chunk(const void* xbc, int ld, int tokens, const float* gate, int g_part, long g_stride, int g_ld, const float* gate_bias, const float* par,
+                        const float* d_skip, float* state, int n_slots, const int* cu_q, const int* seq_slots, float* out, int ld_out, int heads, int groups, int dim,
+                        int vdim, int n_seqs, void* status, cudaStream_t stream) {
+  if (n_seqs <= 0 || tokens <= 0) return 0;
+  if (groups < 1 || heads % groups || g_part < 1 || g_ld < heads || ld < heads * vdim + 2 * groups * dim) return fail("ssd_chunk: bad sizes%s");
+  const __nv_bfloat16* p = (const __nv_bfloat16*)xbc;
+  LightningChunkArgs a;
+  memset(&a, 0, sizeof(a));
+  a.decay = par; a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out; a.ld_out = ld_out;
+  a.heads = heads; a.dim = dim; a.vdim = vdim; a.status = (KernelStatus*)status;
+  a.gate = gate; a.g_part = g_part; a.g_stride = g_stride; a.g_ld = g_ld; a.gate_bias = gate_bias; a.d_skip = d_skip; a.groups = groups;
+  const __nv_bfloat16* bm = p + (size_t)heads * vdim;
+  return chunk_launch<true>(bm + (size_t)groups * dim, bm, p, ld, tokens, groups, a, n_seqs, stream);
 }

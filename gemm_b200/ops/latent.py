@@ -216,6 +216,16 @@ def attend_latents(q: torch.Tensor, cache: torch.Tensor, rank: int, width: int, 
     wo = row_width(rank, cache.dtype)
     out = (torch.empty if wo == rank else torch.zeros)(heads, m, wo, dtype=q.dtype, device=q.device)      # the padding meets zero weights: finite
     lib = _native.cuda()
+    if q.dtype == torch.bfloat16 and lib.gb_latent_decode_heads(_i(heads), _i(width), _i(rank), _i(page_size)):
+        po = pl = None
+        if plan.splits > 1:
+            po = torch.empty(plan.splits, plan.n_abs, heads, rank, dtype=torch.float32, device=q.device)
+            pl = torch.empty(plan.splits, plan.n_abs, heads, dtype=torch.float32, device=q.device)
+        rc = lib.gb_latent_decode(_p(q), _p(cache), _i(cache.shape[2]), _l(cache.shape[0]), _p(plan.abs_seq), _p(plan.abs_kv), _p(fb.kv_len), _p(fb.block_table),
+                                  _i(fb.block_table.shape[1]), _i(page_size), _i(plan.n_abs), _i(heads), _i(width), _i(rank), _i(plan.splits), _p(out), _i(m), _i(wo),
+                                  _p(po), _p(pl), _p(sink), _c(_native.status_ptr()), _s())
+        _native.check(rc, "gb_latent_decode", n=1 if plan.splits == 1 else 2)
+        return out
     rc = lib.gb_attn_latent_any(_p(q), _l(q.stride(1)), _l(q.stride(0)), _p(cache), _i(cache.shape[2]), _p(out), _l(out.stride(1)), _l(out.stride(0)),
                                 _i(int(q.dtype == torch.float32)), _p(fb.cu_q), _p(fb.kv_len), _p(plan.abs_seq), _p(plan.abs_kv), _p(fb.block_table),
                                 _i(fb.block_table.shape[1]), _i(page_size), _i(fb.cu_q.numel() - 1), _l(cache.shape[0]), _i(plan.n_abs), _i(heads), _i(width),
@@ -226,5 +236,30 @@ def attend_latents(q: torch.Tensor, cache: torch.Tensor, rank: int, width: int, 
 
 # ------------------------------------------------------------------------------------------ expanded form
 def can_expand(sp) -> bool:
-    """Head sizes the expanded kernel is built for."""
-    return False
+    """Head sizes the expanded kernel is built for: at most 128 unrotated and 64 rotated key columns, at most 128 value columns."""
+    return sp.head_dim <= 128 and 0 < sp.rot_dim <= 64 and sp.v_dim <= 128 and sp.kv_rank % 8 == 0
+
+
+def attend_expanded(q_n: torch.Tensor, q_r: torch.Tensor, kv: torch.Tensor, cached: torch.Tensor, rank: int, plan: LatentPlan, sink, out: torch.Tensor) -> None:
+    """Causal attention of the plan's expanded rows: ``q_n [n_exp, heads, dn]`` and ``q_r [n_exp, heads, dr]`` (times scale * log2 e) against ``kv [n_kv,
+    heads x dn | heads x dv]`` and the rotated key parts (columns ``rank ...`` of the gathered cache rows ``cached``) -> ``out [T, heads, dv]`` at the
+    rows' tokens."""
+    n, heads, dn = q_n.shape
+    dr, dv = q_r.shape[2], out.shape[2]
+    if not q_n.is_cuda:
+        for i in range(plan.seqs.numel()):
+            a, b, k0, k1 = (int(x) for x in (plan.q0[i], plan.q0[i + 1], plan.kv0[i], plan.kv0[i + 1]))
+            k = torch.cat([kv[k0:k1, : heads * dn].float().reshape(-1, heads, dn), cached[k0:k1, rank: rank + dr].float().unsqueeze(1).expand(-1, heads, dr)], -1)
+            s = torch.einsum("qhd,khd->hqk", torch.cat([q_n[a:b], q_r[a:b]], -1).float(), k) * math.log(2.0)
+            see = torch.arange(k1 - k0).unsqueeze(0) <= torch.arange(k1 - k0 - (b - a), k1 - k0).unsqueeze(1)
+            s = s.masked_fill(~see, float("-inf"))
+            if sink is not None:
+                s = torch.cat([s, (sink * math.log(2.0)).reshape(heads, 1, 1).expand(heads, b - a, 1)], dim=2)
+            p = torch.softmax(s, dim=-1)[:, :, : k1 - k0]
+            out[plan.exp_tok[a:b].long()] = torch.einsum("hqk,khd->qhd", p, kv[k0:k1, heads * dn:].float().reshape(-1, heads, dv)).to(out.dtype)
+        return
+    e = kv.element_size()
+    rc = _native.cuda().gb_latent_prefill(_p(q_n), _p(q_r), _p(kv), _c(cached.data_ptr() + rank * e), _c(kv.data_ptr() + heads * dn * e), _i(kv.stride(0)),
+                                          _i(cached.stride(0)), _i(n), _i(kv.shape[0]), _p(plan.tiles), _i(plan.tiles.shape[0]), _p(plan.q0), _p(plan.kv0),
+                                          _p(plan.exp_tok), _p(out), _i(heads), _i(dn), _i(dr), _i(dv), _p(sink), _c(_native.status_ptr()), _s())
+    _native.check(rc, "gb_latent_prefill")

@@ -29,6 +29,16 @@ def _s():
     return _c(torch.cuda.current_stream().cuda_stream)
 
 
+# Launches whose longest sequence brings at least this many tokens take the chunked scans
+CHUNKED = os.environ.get("GB_RECURRENT_CHUNKED", "1") != "0"
+CHUNKED_MIN_TOKENS = 16
+
+
+def can_chunk(rows: torch.Tensor, dim: int, vdim: int) -> bool:
+    """Whether the chunked kernels take these rows: bf16 with a 16-byte pitch, key size up to 128."""
+    return bool(rows.is_cuda and rows.dtype == torch.bfloat16 and dim <= 128 and dim % 8 == 0 and vdim % 8 == 0 and rows.stride(0) % 8 == 0 and rows.data_ptr() % 16 == 0)
+
+
 def _n_rows(y) -> int:
     return y.rows if hasattr(y, "buf") else y.shape[0]
 
@@ -96,6 +106,12 @@ def ssd(xbc: torch.Tensor, dt, dt_col: int, dt_bias: torch.Tensor, a: torch.Tens
     t = xbc.shape[0]
     assert f32 and state.is_contiguous() and state.dtype == torch.float32
     out = torch.empty(t, heads * vdim, dtype=torch.float32, device=base.device)
+    if CHUNKED and max_tokens >= CHUNKED_MIN_TOKENS and can_chunk(xbc, dim, vdim):
+        rc = _native.cuda().gb_ssd_chunk(_p(xbc), _i(xbc.stride(0)), _i(t), _at(base, dt_col), _i(parts), _l(stride), _i(ld), _p(dt_bias), _p(a), _p(d_skip), _p(state),
+                                         _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(heads * vdim), _i(heads), _i(groups), _i(dim), _i(vdim),
+                                         _i(cu_q.numel() - 1), _c(_native.status_ptr()), _s())
+        _native.check(rc, "gb_ssd_chunk")
+        return out
     rc = _native.cuda().gb_recurrent_step(_i(0), _p(xbc), _i(int(xbc.dtype == torch.float32)), _i(1), _l(0), _i(xbc.stride(0)), _at(base, dt_col), _i(parts), _l(stride),
                                           _i(ld), _p(dt_bias), _p(a), _p(d_skip), _p(state), _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(heads * vdim),
                                           _i(heads), _i(groups), _i(dim), _i(vdim), _i(0), _i(cu_q.numel() - 1), _s())
