@@ -149,6 +149,15 @@ def gla(qv, gate, gate_col: int, f_bias: torch.Tensor, lower: torch.Tensor, stat
     t = _n_rows(qv)
     assert gf32 and state.is_contiguous() and state.dtype == torch.float32
     out = torch.empty(t, nv, dtype=torch.float32, device=base.device)
+    if CHUNKED and max_tokens >= CHUNKED_MIN_TOKENS and activated and not hasattr(qv, "buf") and can_chunk(base, dim, vdim):
+        lib, n_seqs = _native.cuda(), cu_q.numel() - 1
+        lib.gb_gla_chunk_workspace.restype = _l
+        nb = int(lib.gb_gla_chunk_workspace(_l(t), _i(n_seqs), _i(heads), _i(dim)))
+        ws = torch.empty(nb, dtype=torch.uint8, device=base.device)
+        rc = lib.gb_gla_chunk(_p(base), _i(ld), _i(t), _at(gb, gate_col), _i(gparts), _l(gstride), _i(gld), _p(f_bias), _p(lower), _p(state), _i(state.shape[0]), _p(cu_q),
+                              _p(seq_slots), _p(out), _i(nv), _i(heads), _i(dim), _i(vdim), _i(max_tokens), _i(n_seqs), _p(ws), _l(nb), _c(_native.status_ptr()), _s())
+        _native.check(rc, "gb_gla_chunk", n=2)
+        return out
     rc = _native.cuda().gb_recurrent_step(_i(1), _p(base), _i(f32), _i(parts), _l(stride), _i(ld), _at(gb, gate_col), _i(gparts), _l(gstride), _i(gld), _p(f_bias), _p(lower),
                                           _c(0), _p(state), _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(nv), _i(heads), _i(1), _i(dim), _i(vdim),
                                           _i(int(not activated)), _i(cu_q.numel() - 1), _s())
