@@ -53,7 +53,7 @@ def parse_args():
                          "batch replicated (dense models); tp+ep = attention sharded by heads and experts spread over the same ranks, "
                          "batch replicated (the layout of the largest MoE models, e.g. --model qwen3-235b-a22b); auto picks by model")
     ap.add_argument("--moe-path", default="fused", choices=["fused", "nccl"], help="multi-GPU expert exchange: fused peer-memory kernels or the NCCL baseline")
-    ap.add_argument("--design", default="", choices=["", "zogavik"],
+    ap.add_argument("--design", default="", choices=["", "zogavik", "famepel"],
                     help="instead of the default workload: prefill and decode throughput of a model described layer by layer, at several sizes, beside the "
                          "closest other model at equal size (random weights, bf16, one GPU); one JSON line per measurement")
     return ap.parse_args()
@@ -286,8 +286,8 @@ def baseline_arm(args):
 
 
 def design_arm(args):
-    """Prefill and decode throughput of the design's presets and of a Qwen3.5 hybrid (three Delta-Net layers to one of gated attention) of the
-    same width, depth, heads and feed-forward.  Weights and activations exceed L2 in every timed region."""
+    """Prefill and decode throughput of the design's presets and of a Qwen3.5 hybrid (Delta-Net layers and gated attention, dense or with a mixture of
+    experts) of the same width, depth, heads and feed-forward.  Weights and activations exceed L2 in every timed region."""
     import gc
     import torch
     from gemm_b200 import _native
@@ -301,7 +301,15 @@ def design_arm(args):
         return ModelConfig(arch="qwen35", n_layers=layers, hidden=4096, n_heads=32, n_kv_heads=8, head_dim=128, ffn=12288, vocab=151936, rope_dim=64,
                            full_attention_interval=4, ssm_d_conv=4, ssm_n_heads_k=32, ssm_n_heads_v=32, ssm_head_dim=128, attn_output_gate=True)
 
-    models = [("zogavik-8b", get_config("zogavik-8b")), ("qwen35-hybrid, 36 layers of the same sizes", hybrid(36)), ("zogavik-4b-loop2", get_config("zogavik-4b-loop2"))]
+    def hybrid_moe(layers):
+        return ModelConfig(arch="qwen35moe", n_layers=layers, hidden=2048, n_heads=32, n_kv_heads=4, head_dim=128, ffn=6144, vocab=151936, rope_dim=64,
+                           full_attention_interval=5, ssm_d_conv=4, ssm_n_heads_k=32, ssm_n_heads_v=32, ssm_head_dim=128, attn_output_gate=True, n_experts=128,
+                           n_experts_used=8, expert_ffn=768)
+
+    if args.design == "famepel":
+        models = [("famepel-30b-a3b", get_config("famepel-30b-a3b")), ("qwen35moe-hybrid, 45 layers of the same sizes", hybrid_moe(45))]
+    else:
+        models = [("zogavik-8b", get_config("zogavik-8b")), ("qwen35-hybrid, 36 layers of the same sizes", hybrid(36)), ("zogavik-4b-loop2", get_config("zogavik-4b-loop2"))]
     sampler = ClockSampler(0)
     sampler.start()
     sampler.mark()

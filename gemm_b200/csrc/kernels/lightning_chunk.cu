@@ -9,8 +9,8 @@
 //   MMA thread  : S1 = Q K^T;  dS = K^T (w V);  O1 = Q S;  O2 = P V         (A of O2 is P in TMEM; S and w V are written to smem)
 //   P warps     : S1 row -> times g^(i-j), lower triangle -> P in TMEM;  g^(i+1) O1 + O2 -> global f32 (TMA)
 //   state warps : V -> w V in smem;  S <- g^n S + dS;  S -> smem for the next chunk's O1
-// The SSD form (Mamba-2) is the same scan with a decay per token: with L_i the sum of a dt log2(e) up to token i of the chunk, g^(i-j) becomes
-// 2^(L_i - L_j) dt_j (one exponential of L_i - (L_j - log2 dt_j)), w of a token 2^(L_n-1 - L_j) dt_j, and D x_i joins P's diagonal.  q and k are C
+// The SSD form (Mamba-2) is the same scan with a decay per token: with L_i the sum of a dt log2(e) up to token i, g^(i-j) becomes
+// 2^(L_i - L_j) dt_j (one exponential of L_i - (L_j - log2 dt_j)), w of a token 2^(L_(n-1) - L_j) dt_j, and D x_i joins P's diagonal.  q and k are C
 // and B of the head's group.  Every warp of the two groups sums the chunk's step sizes itself, so they need no exchange.
 // Every f32 factor that goes through the tensor cores (P, w V, S) is the sum of two bf16 operands (hi + lo, 16 bits of mantissa), so
 // decays and state keep 32-bit accuracy; only q, k and v themselves are bf16.
@@ -58,20 +58,22 @@ __device__ __forceinline__ void ssd_load(const LightningChunkArgs& a, int t0, in
   }
 }
 
-// Sum of the logarithmic decays (base 2) up to token 32 q + lane, the step size of that token, and the chunk's total; every warp gets the same sums.
-__device__ __forceinline__ void ssd_scan(const float* raw, int n, float bias, float a2, int q, int lane, float& L, float& dt, float& total) {
-  float base = 0.f, own = 0.f;
-  total = 0.f; dt = 0.f;
+// Of the logarithmic decays (base 2): the sum L over block q of 32 tokens up to token 32 q + lane, the sums S of the four blocks, and the token's step
+// size.  Sums that go on over the whole chunk would lose the small decays between neighbours behind large ones; so a pair in one block takes the
+// difference of its L, and only pairs further apart add block sums.
+__device__ __forceinline__ void ssd_scan(const float* raw, int n, float bias, float a2, int q, int lane, float& L, float& dt, float* S) {
+  float own = 0.f;
+  dt = 0.f;
 #pragma unroll
   for (int b = 0; b < 4; ++b) {
     const float d = 32 * b + lane < n ? softplus_exact(raw[b] + bias) : 0.f;
     const float l = a2 * d;
-    if (b == q) { dt = d; own = l; base = total; }
-    total += warp_sum(l);
+    if (b == q) { dt = d; own = l; }
+    S[b] = warp_sum(l);
   }
 #pragma unroll
   for (int o = 1; o < 32; o <<= 1) { const float v = __shfl_up_sync(0xffffffffu, own, o); if (lane >= o) own += v; }
-  L = base + own;
+  L = own;
 }
 
 template <int DP, bool SSD>                // DP: key size padded, 64 or 128
@@ -204,12 +206,15 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     for (int j = 0; j < n_chunks; ++j) {
       const uint32_t ph = j & 1;
       const int b = j & 1, t0 = t_begin + j * kLcC;
-      float Li = 0.f;
+      float Li = 0.f, S[4] = {0.f, 0.f, 0.f, 0.f};
       if constexpr (SSD) {
-        float dt, total;
-        ssd_scan(raw, min(kLcC, t_end - t0), dt_bias, a2, q, lane, Li, dt, total);
+        float dt;
+        ssd_scan(raw, min(kLcC, t_end - t0), dt_bias, a2, q, lane, Li, dt, S);
         pz[i] = Li - log2f(dt);             // (read by everyone below; the barrier at the end of the chunk lets the next one overwrite it)
-        gi = ex2(Li);
+        gi = Li;
+#pragma unroll
+        for (int c = 2; c >= 0; --c) if (c < q) gi += S[c];
+        gi = ex2(gi);
         if (j + 1 < n_chunks) ssd_load(a, t0 + kLcC, min(kLcC, t_end - t0 - kLcC), h, lane, raw);
         bar128_and(true);
       }
@@ -229,8 +234,11 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
               else { w[x] = (pw + (i - c * 32))[-x]; asm volatile("" : "+f"(w[x])); }
             }
             if constexpr (SSD) {
+              float L = Li;                     // to the start of block c (its own sums count from there)
 #pragma unroll
-              for (int x = 0; x < 32; ++x) w[x] = ex2(Li - w[x]);       // above the diagonal anything, cleared below
+              for (int y = 2; y >= 0; --y) if (y < q && y >= c) L += S[y];
+#pragma unroll
+              for (int x = 0; x < 32; ++x) w[x] = ex2(L - w[x]);        // above the diagonal anything, cleared below
             }
             tc_wait_ld();
 #pragma unroll
@@ -322,9 +330,15 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
     for (int j = 0; j < n_chunks; ++j) {
       const uint32_t ph = j & 1;
       const int b = j & 1, n = min(kLcC, t_end - (t_begin + j * kLcC));
-      float L = 0.f, dt = 0.f, total = 0.f;
+      float after = 0.f, dt = 0.f, total = 0.f;
       if constexpr (SSD) {
-        ssd_scan(raw, n, dt_bias, a2, q, lane, L, dt, total);
+        float L, B[4];
+        ssd_scan(raw, n, dt_bias, a2, q, lane, L, dt, B);
+        total = ((B[0] + B[1]) + B[2]) + B[3];
+#pragma unroll
+        for (int c = 0; c < 4; ++c) if (c == q) after = B[c] - L;
+#pragma unroll
+        for (int c = 1; c < 4; ++c) if (c > q) after += B[c];
         if (j + 1 < n_chunks) ssd_load(a, t_begin + (j + 1) * kLcC, min(kLcC, t_end - t_begin - (j + 1) * kLcC), h, lane, raw);
       }
       // w V: a token's values times what its contribution still decays by until the end of the chunk
@@ -332,7 +346,7 @@ lightning_chunk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_con
       {
         const uint8_t* sV = smem + b * kLcStage + 2 * kLcQ;
         const bool live = d < n;
-        const float w = !live ? 0.f : SSD ? ex2(total - L) * dt : pw[n - 1 - d];
+        const float w = !live ? 0.f : SSD ? ex2(after) * dt : pw[n - 1 - d];
 #pragma unroll
         for (int c = 0; c < 8; ++c) {
           const int off = d * 128 + ((c ^ (d & 7)) << 4);

@@ -216,14 +216,15 @@ def batched_linear_f32(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> t
 
 def grouped_linear_f32(x: torch.Tensor, w: torch.Tensor, seg_start: torch.Tensor, seg_count: torch.Tensor, rows: int,
                        row_src: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``grouped_linear`` in f32: rows ``seg_start[g] ...`` (multiples of 64) times ``w[g] [N, K]^T`` -> ``[rows, N]``; row r is ``x[row_src[r]]``, or
-    ``x[r]``.  Rows of no segment are undefined."""
+    """``grouped_linear`` in f32: rows ``seg_start[g] ...`` (multiples of 64) times ``w[g] [N, K]^T`` -> ``[rows, N]``; row r is ``x[row_src[r]]``
+    (zeros where negative), or ``x[r]``.  Rows of no segment are undefined."""
     g, n, k = w.shape
     if not x.is_cuda:
         out = torch.zeros(rows, n)
         for gi in range(g):
             s, c = int(seg_start[gi]), int(seg_count[gi])
-            out[s: s + c] = (x[row_src[s: s + c].long()] if row_src is not None else x[s: s + c]) @ w[gi].t()
+            xs = x[s: s + c] if row_src is None else x[row_src[s: s + c].long().clamp_min(0)] * (row_src[s: s + c] >= 0).unsqueeze(1)
+            out[s: s + c] = xs @ w[gi].t()
         return out
     out = torch.empty(rows, n, dtype=torch.float32, device=x.device)
     rc = _native.cuda().gb_gemm_f32_grouped(_p(x), _p(w), _p(out), _p(seg_start), _p(seg_count), _i(g), _i(rows), _i(n), _i(k), _i(x.stride(0)), _p(row_src), _stream())

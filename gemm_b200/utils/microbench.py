@@ -20,6 +20,8 @@ Cases
   layered      the kernels of models described layer by layer beside the like kernels of the other models at equal size: lightning
                attention (decode, prefill) and the Delta-Net recurrence; windowed attention with kept tokens and distance bias and the
                plain causal kernels; the f32-stream norm, Q / K unit norm and gated norm and their bf16-stream counterparts
+  famepel      the kernels of Famepel at the sizes of ``famepel-30b-a3b`` beside the like kernels of the other models: Mamba-2 and HGRN2
+               scans and Delta-Net; latent attention and plain attention; Dynamic-Tanh stream and RMSNorm, part norm, convolution, routing
   spec_verify  whole-model step over 1, 2, 3 and 5 positions per sequence (speculative verification against plain decode);
                builds the full Qwen3-30B-A3B shape, not part of ``all``
 
@@ -422,9 +424,138 @@ def case_layered(args):
         del wg
 
 
+def case_famepel(args):
+    from ..models.config import get_config
+    from ..ops import deltanet as dn
+    from ..ops import latent, recurrent, stream
+    dev = "cuda"
+    cfg = get_config("famepel-30b-a3b")
+    spec = {sp.mixer: sp for sp in cfg.layer_specs}
+    m, hg, la, h = spec["mamba2"], spec["hgrn2"], spec["latent"], cfg.hidden
+    f32 = dict(device=dev, dtype=torch.float32)
+    for name, lens in (("decode_1", [1]), ("decode_64", [1] * 64), ("prefill_1x8192", [8192]), ("prefill_8x2048", [2048] * 8)):
+        t, b, dec = sum(lens), len(lens), len(lens) == sum(lens)
+        cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        sl = torch.arange(b, dtype=torch.int32, device=dev)
+        nv, ch = m.n_heads * m.v_dim, m.conv_channels
+        at = (nv + ch + 127) // 128 * 128
+        proj = torch.randn(t, at + 128, device=dev)
+        rows = proj if dec else proj.bfloat16()
+        es = rows.element_size()
+        cw, cb, cst = torch.randn(ch, m.conv_taps, device=dev), torch.randn(ch, device=dev), torch.zeros(b, m.conv_taps - 1, ch, **f32)
+        _run(f"causal_conv_{name}", lambda: recurrent.causal_conv(rows, nv, cw, cb, cst, cu, sl, max(lens)), 0.0, t * ch * (es + 2) + 2 * cst.numel() * 4, args)
+        x = (torch.randn(t, ch, device=dev) * 0.5).bfloat16()
+        if m.conv_taps <= 8:
+            _run(f"ssm_conv_{name}", lambda: dn.conv_silu(x, cw, cst, cu, sl), 0.0, t * ch * 4 + 2 * cst.numel() * 4, args)
+        st = torch.randn(b, m.n_heads, m.head_dim, m.v_dim, device=dev) * 0.1
+        hv = [torch.randn(m.n_heads, device=dev) for _ in range(2)] + [-torch.rand(m.n_heads, device=dev) - 0.1]
+        _run(f"ssd_{name}", lambda: recurrent.ssd(x, proj, at, hv[0], hv[2], hv[1], st, cu, sl, m.n_heads, m.state_groups, m.head_dim, m.v_dim, max(lens)),
+             4.0 * t * m.n_heads * m.head_dim * m.v_dim, 2 * st.numel() * 4 + t * (ch * 2 + nv * 4), args)
+        o, nw = torch.randn(t, nv, device=dev), torch.ones(nv, device=dev)
+        _run(f"part_norm_gated_{name}", lambda: stream.part_norm(o, nw, m.norm_parts, 1e-5, rows), 0.0, t * nv * (4 + es + 2), args)
+        _run(f"gated_norm_{name}", lambda: stream.gated_norm(o, rows, 0, nw, 1e-5), 0.0, t * nv * (4 + es + 2), args)
+        del o, st
+        nq, nv = hg.q_dim, hg.n_heads * hg.v_dim
+        qv, z = torch.randn(t, nq + nv, device=dev), torch.randn(t, nq, device=dev) + 2
+        qv = qv if dec else qv.bfloat16()
+        st = torch.randn(b, hg.n_heads, hg.head_dim, hg.v_dim, device=dev) * 0.1
+        fb, low = torch.zeros(nq, device=dev), torch.full((nq,), 0.3, device=dev)
+        _run(f"gla_{name}", lambda: recurrent.gla(qv, z, 0, fb, low, st, cu, sl, hg.n_heads, hg.head_dim, hg.v_dim, not dec, max(lens)),
+             4.0 * t * hg.n_heads * hg.head_dim * hg.v_dim, 2 * st.numel() * 4 + t * ((nq + nv) * qv.element_size() + nq * 4 + nv * 4), args)
+        # Delta-Net with states of the same sizes: 16 and 32 heads of 128 x 128
+        for hd in (16, 32):
+            ds = 128
+            qkv, zz, ab = torch.randn(t, 3 * hd * ds, device=dev).bfloat16(), torch.randn(t, hd * ds, device=dev).bfloat16(), torch.randn(t, 2 * hd, device=dev)
+            a, bias, nwd = -(torch.rand(hd, device=dev) * 2 + 0.1), torch.randn(hd, device=dev) * 0.5, torch.ones(ds, device=dev)
+            st = torch.randn(b, hd, ds, ds, device=dev) * 0.1
+            _run(f"deltanet_{hd}_{name}", lambda: dn.deltanet(qkv, zz, ab, a, bias, nwd, st, cu, sl, hd, hd, ds, 1e-6), 4.0 * t * hd * ds * ds,
+                 2 * st.numel() * 4 + t * 5 * hd * ds * 2, args)
+        del qv, z, proj, rows, x, qkv, zz, st
+    # latent attention: 32 heads, latents of 512 + 64 columns; plain attention with 32 heads over 4 key / value heads of 128
+    hd, d, rd, v, r, page = la.n_heads, la.head_dim, la.rot_dim, la.v_dim, la.kv_rank, 128
+    w = stream.row_width(r + rd, torch.bfloat16)
+
+    class Batch:
+        pass
+
+    for name, b, q_len, ctx in (("decode_1x32768", 1, 1, 32767), ("decode_16x8192", 16, 1, 8191), ("decode_64x2048", 64, 1, 2047), ("decode_64x8192", 64, 1, 8191),
+                                ("prefill_1x8192", 1, 8192, 0), ("prefill_8x2048", 8, 2048, 0)):
+        kv, dec = ctx + q_len, q_len == 1
+        pages = (kv + page - 1) // page
+        bt = torch.arange(b * pages, device=dev, dtype=torch.int32).reshape(b, pages)
+        cu, kvl = torch.tensor([i * q_len for i in range(b + 1)], device=dev, dtype=torch.int32), torch.full((b,), kv, device=dev, dtype=torch.int32)
+        batch = Batch()
+        batch.block_table, batch.kv_len, batch.cu_q = bt, kvl, cu
+        cache = torch.randn(b * pages * page, 1, w, device=dev).bfloat16()
+        sink = torch.zeros(hd, device=dev)
+        plan = latent.make_plan([q_len] * b, [kv] * b, kv, dev, dec, True, [hd])
+        seen = float(sum(range(ctx + 1, kv + 1)) * b)
+        if dec:
+            qa = (torch.randn(hd, plan.m, w, device=dev) * 0.1).bfloat16()
+            _run(f"latent_{name}", lambda: latent.attend_latents(qa, cache, r, r + rd, plan, batch, page, sink), 2.0 * seen * hd * (2 * r + rd),
+                 b * (kv * w * 2 + hd * (w + r) * 2), args, splits=plan.splits)
+            qn = torch.randn(hd * plan.m, d, device=dev).bfloat16()
+            uk, uv = torch.randn(hd, r, d, device=dev).bfloat16(), torch.randn(hd, v, r, device=dev).bfloat16()
+            seg, cnt, rows = plan.groups(hd, dev)
+            oo = torch.randn(hd * plan.m, r, device=dev).bfloat16()
+            out = torch.empty(b * hd, v, device=dev, dtype=torch.bfloat16)
+            _run(f"absorb_k_{name}", lambda: gemm.grouped_linear(qn, uk, seg, cnt, plan.tile, out=qa.view(-1, w), n_out=r), 2.0 * b * hd * d * r, hd * (d * r + b * (d + r)) * 2, args)
+            _run(f"absorb_v_{name}", lambda: gemm.grouped_linear(oo, uv, seg, cnt, plan.tile, out=out, row_map=rows, n_out=v), 2.0 * b * hd * v * r,
+                 hd * (v * r + b * (v + r)) * 2, args)
+        else:
+            en, er = torch.randn(b * q_len, hd, d, device=dev).bfloat16() * 0.1, torch.randn(b * q_len, hd, rd, device=dev).bfloat16() * 0.1
+            kvx = torch.randn(b * kv, hd * (d + v), device=dev).bfloat16()
+            out = torch.empty(b * q_len, hd, v, device=dev, dtype=torch.bfloat16)
+            rows = latent.gather_latents(cache, plan, bt, page)
+            _run(f"latent_{name}", lambda: latent.attend_expanded(en, er, kvx, rows, r, plan, sink, out), 2.0 * seen * hd * (d + rd + v),
+                 (kvx.numel() + out.numel() + en.numel() + er.numel() + rows.numel()) * 2, args)
+            _run(f"latent_gather_{name}", lambda: latent.gather_latents(cache, plan, bt, page), 0.0, b * kv * w * 4, args)
+            del kvx
+        hkv = 4
+        k, vv = (torch.randn(b * pages * page, hkv, 128, device=dev).bfloat16() for _ in range(2))
+        q = (torch.randn(b * q_len, hd, 128, device=dev) * 0.1).bfloat16()
+        splits = att.pick_splits(b, hkv, kv) if dec else 1
+        work = att.build_work([q_len] * b, hd, hkv, splits).to(dev)
+        _run(f"attn_{name}", lambda: att.attention(q, k, vv, cu, kvl, bt, page, work, num_splits=splits, decode=dec), 4.0 * seen * hd * 128, b * (kv * hkv * 512 + q_len * hd * 512),
+             args, splits=splits)
+        del k, vv, cache
+    for t in (1, 64, 8192):
+        x, u = torch.randn(t, h, device=dev), torch.randn(t, h, device=dev)
+        n1, n2 = (stream.DynTanh(0.5, torch.ones(h, device=dev), torch.zeros(h, device=dev)) for _ in range(2))
+        _run(f"stream_dyt_{t}x{h}", lambda: stream.norm(x, n1, 1e-5, stream.PostNormed(u, n2)), 0.0, t * h * 14, args)
+        _run(f"stream_norm_{t}x{h}", lambda: stream.norm(x, n1.weight, 1e-5, u), 0.0, t * h * 14, args)
+        k, e = 8, 128
+        y = torch.randn(t * k, h, device=dev).bfloat16()
+        pend = moe.PendingCombine(y, torch.randperm(t * k, device=dev).to(torch.int32), torch.rand(t, k, device=dev), t, k)
+        _run(f"stream_dyt_moe_{t}x{h}", lambda: stream.norm(x, n1, 1e-5, stream.PostNormed(pend, n2)), 0.0, t * h * (10 + 2 * k), args)
+        xb = x.bfloat16()
+        _run(f"rmsnorm_moe_{t}x{h}", lambda: ew.rmsnorm(pend, n1.weight.bfloat16(), 1e-5, residual=xb), 0.0, t * h * (6 + 2 * k), args)
+        z = torch.randn(t, e, device=dev)
+        for groups in ((1, 1), (8, 4)):
+            _run(f"route_{groups[0]}_groups_{t}", lambda: moe.route(z, k, "sigmoid", None, 2, 2.5, None, groups), 0.0, t * (e * 4 + k * 8), args)
+        nk = hd * (d + rd)
+        qf = torch.randn(t, nk, device=dev)
+        qf = qf if t <= 64 else qf.bfloat16()
+        pos = torch.arange(t, device=dev, dtype=torch.int32)
+        freq = torch.tensor(la.rotary.frequencies(), dtype=torch.float64, device=dev)
+        en, er = torch.empty(t, hd, d, device=dev, dtype=torch.bfloat16), torch.empty(t, hd, rd, device=dev, dtype=torch.bfloat16)
+        _run(f"latent_q_{t}", lambda: latent.latent_q(qf, pos, freq, 1.0, 0.1, None, (en, er), None, hd, d, rd), 0.0, t * nk * (qf.element_size() + 2), args)
+        a = torch.randn(t, la.q_rank + r + rd, device=dev)
+        a = a if t <= 64 else a.bfloat16()
+        cache = torch.empty(t, 1, w, device=dev, dtype=torch.bfloat16)
+        qn, kn = torch.ones(la.q_rank, device=dev), torch.ones(r, device=dev)
+        _run(f"latent_store_{t}", lambda: latent.latent_store(a, pos, pos, qn, kn, freq, 1.0, cache, la.q_rank, r, rd, 1e-5, torch.bfloat16), 0.0,
+             t * (la.q_rank + r + rd) * (a.element_size() + 2), args)
+        qkv = torch.randn(t, (hd + 8) * 128, device=dev).bfloat16()
+        kc, vc = (torch.empty(t, 4, 128, device=dev, dtype=torch.bfloat16) for _ in range(2))
+        tab, qw = ew.rope_table(8192, 128, 1e6, dev), torch.ones(128, device=dev, dtype=torch.bfloat16)
+        _run(f"qk_norm_rope_{t}", lambda: ew.qk_norm_rope(qkv, pos, pos, qw, qw, kc, vc, hd, 4, 128, 1e6, 1e-6, 1.0, table=tab), 0.0, t * (hd + 8) * 128 * 4, args)
+
+
 MODEL_CASES = {"spec_verify": case_spec_verify}      # build the whole benchmark model: not part of --case all
 CASES = {"gemm": case_gemm, "moe_decode": case_moe_decode, "moe_prefill": case_moe_prefill, "attn_decode": case_attn_decode,
-         "attn_prefill": case_attn_prefill, "lm_head": case_lm_head, "quant": case_quant, "small": case_small, "layered": case_layered}
+         "attn_prefill": case_attn_prefill, "lm_head": case_lm_head, "quant": case_quant, "small": case_small, "layered": case_layered,
+         "famepel": case_famepel}
 
 
 def main(argv=None):
