@@ -147,7 +147,7 @@ __device__ __forceinline__ int e8m0_from_amax(float amax) {
   return amax == 0.0f ? 127 : max(1, min(e, 254));   // an all-zero block gets scale 1
 }
 
-// ACT, DUAL: the gate's activation (gate_act); plain: 1 = SiLU on the output features below args.silu_rows.
+// ACT, DUAL: the gate's activation (gate_act); plain: 1 = SiLU on the output features below args.silu_rows, 2 = bf16 rows scattered by args.row_map.
 template <int TN, int MODE, bool DUAL, bool QUANT_OUT, int ACT = 0>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, const GemmArgs args) {
@@ -472,6 +472,28 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           }
         }
       };
+      if constexpr (!DUAL && ACT == 2) {
+        // rows scattered by row_map, nothing else to decide (grouped products whose results belong side by side, such as one per head)
+#pragma unroll 1
+        for (int c = 0; c < TN; c += 16) {
+          uint32_t r0[16];
+          tmem_ld_x16(tacc + c, r0);
+          tc_wait_ld();
+          if (c >= t.valid || !n_ok) continue;
+#pragma unroll
+          for (int j = 0; j < 16; ++j) {
+            if (c + j >= t.valid) continue;
+            const int orow = args.row_map[t.x_row0 + c + j];
+            const size_t off = (size_t)orow * args.ldo + n;
+            if (orow >= 0 && (args.out_bytes == 0 || off * 2 < args.out_bytes)) ((__nv_bfloat16*)args.out)[off] = __float2bfloat16(__uint_as_float(r0[j]) + bias);
+          }
+        }
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(&acce_bar[acc]);
+        if (NACC == 2) { if (++acc == 2) { acc = 0; acc_ph ^= 1; } } else { acc_ph ^= 1; }
+        continue;
+      }
       if (args.splits > 1 && args.partial_stride == 0) {
         // ---- split-K: park the partial, the last warp to arrive reduces
         float* ws = args.sk_ws + ((size_t)t.tile_id * args.splits) * (size_t)(NA * TN * 128);
@@ -843,6 +865,12 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
   if (a.silu_rows > 0) {
     if (tn == 128) return launch_gemm<128, 0, false, false, 1>(tmW, tmX, a, max_tiles, stream);
     if (tn == 256) return launch_gemm<256, 0, false, false, 1>(tmW, tmX, a, max_tiles, stream);
+  }
+  if (row_map != nullptr && !mx && !dual && !qo && row_scale == nullptr && a.amax_val == nullptr && !a.out_f32 && a.splits <= 1 && a.peer_bcast == 0 && a.peer_region_rows == 0) {
+    if (tn == 16) return launch_gemm<16, 0, false, false, 2>(tmW, tmX, a, max_tiles, stream);
+    if (tn == 32) return launch_gemm<32, 0, false, false, 2>(tmW, tmX, a, max_tiles, stream);
+    if (tn == 64) return launch_gemm<64, 0, false, false, 2>(tmW, tmX, a, max_tiles, stream);
+    if (tn == 128) return launch_gemm<128, 0, false, false, 2>(tmW, tmX, a, max_tiles, stream);
   }
 #ifdef GB_GEMM_BF16_ONLY
   // build without the MXFP8 variants: the library subset of models whose weights are bf16 or f32

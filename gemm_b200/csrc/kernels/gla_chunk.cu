@@ -199,14 +199,15 @@ gla_scan_kernel(const __grid_constant__ CUtensorMap tmV, const GlaArgs a) {
   } else if (warp == 1) {
     if (lane == 0) {
       constexpr uint32_t id_ds = make_idesc(128, DP, 1, 1, 1, 1), id_s = make_idesc(128, kGlB, 1, 1, 0, 0), id_p = make_idesc(128, kGlB, 1, 1, 1, 0);
+      const uint64_t d_k = make_sdesc_sw128(smem_u32(smem)), d_mn = make_sdesc_sw128_mn(smem_u32(smem), 2048);      // of stage 0's start
       // vdim <= 64: rows 64 .. 127 of the products come from whatever the second V tile holds; nobody reads them
       auto issue_ds = [&](int b) -> bool {
         const int st = b % kGlStages;
         if (!mbar_wait(&full[st], (uint32_t)(b / kGlStages) & 1, abort_flag, a.status, 910, b)) return false;
         tc_fence_after();
-        const uint32_t v = smem_u32(smem + st * kStage), k = v + 4096 + R::kK;
-        mma_f16_ss(t_ds, make_sdesc_sw128_mn(v, 2048), make_sdesc_sw128_mn(k, 2048), id_ds, 0u);
-        mma_f16_ss(t_ds, make_sdesc_sw128_mn(v, 2048), make_sdesc_sw128_mn(k + R::kTile, 2048), id_ds, 1u);
+        const uint64_t v = sdesc_at(d_mn, st * kStage), k = sdesc_at(v, 4096 + R::kK);
+        mma_f16_ss(t_ds, v, k, id_ds, 0u);
+        mma_f16_ss(t_ds, v, sdesc_at(k, R::kTile), id_ds, 1u);
         tc_commit(ds_full);
         return true;
       };
@@ -221,15 +222,15 @@ gla_scan_kernel(const __grid_constant__ CUtensorMap tmV, const GlaArgs a) {
         if (b >= 2 && !mbar_wait(&o_free[b & 1], ((uint32_t)(b >> 1) & 1) ^ 1, abort_flag, a.status, 913, b)) break;
         tc_fence_after();
         const int st = b % kGlStages;
-        const uint32_t v = smem_u32(smem + st * kStage), q = v + 4096 + R::kQ, p = v + 4096 + R::kP;
+        const uint64_t v = sdesc_at(d_mn, st * kStage), q = sdesc_at(d_k, st * kStage + 4096 + R::kQ), p = sdesc_at(d_k, st * kStage + 4096 + R::kP);
         const uint32_t s_hi = t_s + (b & 1) * 128, s_lo = s_hi + 64, o = t_o + (b & 1) * kGlB;
-        mma_f16_ss(o, make_sdesc_sw128_mn(v, 2048), make_sdesc_sw128(p), id_p, 0u);
-        mma_f16_ss(o, make_sdesc_sw128_mn(v, 2048), make_sdesc_sw128(p + 32), id_p, 1u);
+        mma_f16_ss(o, v, p, id_p, 0u);
+        mma_f16_ss(o, v, sdesc_at(p, 32), id_p, 1u);
 #pragma unroll
         for (int x = 0; x < 3; ++x)
 #pragma unroll
           for (int ks = 0; ks < DP / 16; ++ks)
-            mma_f16_ts(o, (x == 1 ? s_lo : s_hi) + ks * 8, make_sdesc_sw128(q + (x == 2 ? R::kTile : 0) + (ks >> 2) * 2048 + (ks & 3) * 32), id_s, 1u);
+            mma_f16_ts(o, (x == 1 ? s_lo : s_hi) + ks * 8, sdesc_at(q, (x == 2 ? R::kTile : 0) + (ks >> 2) * 2048 + (ks & 3) * 32), id_s, 1u);
         tc_commit(&o_full[b & 1]);
         tc_commit(&empty[st]);
       }

@@ -13,9 +13,9 @@ namespace gb {
 
 // cos and sin of position * freq, times mag
 __device__ __forceinline__ void rotation(int pos, double freq, float mag, float& c, float& s) {
-  const double turn = 6.283185307179586476925286766559;
+  const double turn = 6.283185307179586476925286766559, inv_turn = 0.15915494309189533576888376337251;
   double a = (double)pos * freq;
-  a -= turn * rint(a / turn);
+  a = fma(-turn, rint(a * inv_turn), a);
   sincosf((float)a, &s, &c);
   c *= mag; s *= mag;
 }
@@ -32,54 +32,77 @@ struct LatentStoreArgs {
 
 constexpr int kLatKeep = 8;                                    // values per thread kept in registers (ranks up to 256 * kLatKeep)
 
-template <typename TI, typename TO>
+template <typename TI, typename TO, int V>                     // V columns at a time
 __global__ void __launch_bounds__(256)
 latent_store_kernel(const LatentStoreArgs a) {
   pdl_wait();
   pdl_trigger();
   __shared__ float red[2][8];
+  constexpr int N = kLatKeep / V;
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5;
   const TI* src = (const TI*)a.a + (size_t)t * a.ld;
-  auto value = [&](int c) {
-    float v = ldv(src + c);
-    for (int p = 1; p < a.n_part; ++p) v += ldv(src + (size_t)p * a.part_stride + c);
-    return v;
+  auto values = [&](int c, float* v) {
+    load_cols<V>(src + c, v);
+    for (int p = 1; p < a.n_part; ++p) {
+      float y[V];
+      load_cols<V>(src + (size_t)p * a.part_stride + c, y);
+#pragma unroll
+      for (int x = 0; x < V; ++x) v[x] += y[x];
+    }
   };
   const int slot = a.kv_norm != nullptr ? a.slots[t] : -1;
   const bool kv = slot >= 0 && slot < a.num_slots;
-  float q[kLatKeep], k[kLatKeep], sq = 0.f, sk = 0.f;
+  float q[N][V], k[N][V], sq = 0.f, sk = 0.f;
 #pragma unroll
-  for (int i = 0; i < kLatKeep; ++i) {
-    const int c = tid + i * 256;
-    q[i] = c < a.q_rank ? value(c) : 0.f;
-    k[i] = kv && c < a.rank ? value(a.q_rank + c) : 0.f;
-    sq += q[i] * q[i]; sk += k[i] * k[i];
+  for (int i = 0; i < N; ++i) {
+    const int c = (tid + i * 256) * V;
+#pragma unroll
+    for (int x = 0; x < V; ++x) q[i][x] = k[i][x] = 0.f;
+    if (c < a.q_rank) values(c, q[i]);
+    if (kv && c < a.rank) values(a.q_rank + c, k[i]);
+#pragma unroll
+    for (int x = 0; x < V; ++x) { sq += q[i][x] * q[i][x]; sk += k[i][x] * k[i][x]; }
   }
   sq = warp_sum(sq); sk = warp_sum(sk);
   if ((tid & 31) == 0) { red[0][warp] = sq; red[1][warp] = sk; }
+  TO* co = (TO*)a.cache + (size_t)(kv ? slot : 0) * a.ld_c;
+  if (kv) {
+    for (int i = 255 - tid; i < a.rot_dim / 2; i += 256) {     // (the last warps: the first hold the ends of the ranks)
+      float c, s, u = 0.f, v = 0.f;
+      rotation(a.positions[t], a.freq[i], a.mag, c, s);
+      const TI* p0 = src + a.q_rank + a.rank + 2 * i;
+      for (int p = 0; p < a.n_part; ++p) { u += ldv(p0 + (size_t)p * a.part_stride); v += ldv(p0 + (size_t)p * a.part_stride + 1); }
+      stv(co + a.rank + 2 * i, u * c - v * s);
+      stv(co + a.rank + 2 * i + 1, v * c + u * s);
+    }
+    for (int c = a.rank + a.rot_dim + tid; c < a.ld_c; c += 256) stv(co + c, 0.f);
+  }
   __syncthreads();
   sq = sk = 0.f;
 #pragma unroll
   for (int i = 0; i < 8; ++i) { sq += red[0][i]; sk += red[1][i]; }
   const float iq = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps), ik = 1.0f / sqrtf(sk / (float)a.rank + a.eps);
   TO* qo = (TO*)a.q_out + (size_t)t * a.ld_q;
-  TO* co = (TO*)a.cache + (size_t)(kv ? slot : 0) * a.ld_c;
 #pragma unroll
-  for (int i = 0; i < kLatKeep; ++i) {
-    const int c = tid + i * 256;
-    if (c < a.q_rank) stv(qo + c, q[i] * iq * a.q_norm[c]);
-    else if (c < a.ld_q) stv(qo + c, 0.f);
-    if (kv && c < a.rank) stv(co + c, k[i] * ik * a.kv_norm[c]);
+  for (int i = 0; i < N; ++i) {
+    const int c = (tid + i * 256) * V;
+    if (c < a.ld_q) {                                          // zero behind q_rank
+      float w[V];
+#pragma unroll
+      for (int x = 0; x < V; ++x) w[x] = 0.f;
+      if (c < a.q_rank) load_cols<V>(a.q_norm + c, w);
+#pragma unroll
+      for (int x = 0; x < V; ++x) w[x] *= q[i][x] * iq;
+      store_cols<V>(qo + c, w);
+    }
+    if (kv && c < a.rank) {
+      float w[V];
+      load_cols<V>(a.kv_norm + c, w);
+#pragma unroll
+      for (int x = 0; x < V; ++x) w[x] *= k[i][x] * ik;
+      store_cols<V>(co + c, w);
+    }
   }
-  if (!kv) return;
-  for (int i = tid; i < a.rot_dim / 2; i += 256) {
-    float c, s;
-    rotation(a.positions[t], a.freq[i], a.mag, c, s);
-    const float u = value(a.q_rank + a.rank + 2 * i), v = value(a.q_rank + a.rank + 2 * i + 1);
-    stv(co + a.rank + 2 * i, u * c - v * s);
-    stv(co + a.rank + 2 * i + 1, v * c + u * s);
-  }
-  for (int c = a.rank + a.rot_dim + tid; c < a.ld_c; c += 256) stv(co + c, 0.f);
 }
 
 struct LatentQArgs {
@@ -93,43 +116,38 @@ struct LatentQArgs {
   int heads, dim, rot_dim;
 };
 
+// A CTA: one token, `per` heads; a warp per head, a lane per pair of columns.
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256)
-latent_q_kernel(const LatentQArgs a) {
+latent_q_kernel(const LatentQArgs a, int per) {
   pdl_wait();
   pdl_trigger();
   extern __shared__ float cs[];                                // cos, sin of the token's pairs
-  const int t = blockIdx.x, tid = threadIdx.x;
+  const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int half = a.rot_dim / 2;
   for (int i = tid; i < half; i += 256) rotation(a.positions[t], a.freq[i], a.mag * a.scale, cs[i], cs[half + i]);
   __syncthreads();
   const int d = a.dst != nullptr ? a.dst[t] : t;
   const bool ab = d >= 0;
   const size_t row = ab ? (size_t)d : (size_t)(-1 - d);
-  TO* on = (TO*)(ab ? a.a_n : a.m_n) + row * (ab ? a.an_ts : a.mn_ts);
-  TO* orr = (TO*)(ab ? a.a_r : a.m_r) + row * (ab ? a.ar_ts : a.mr_ts);
-  const long n_hs = ab ? a.an_hs : a.mn_hs, r_hs = ab ? a.ar_hs : a.mr_hs;
-  const int nw = ab ? a.an_w : a.mn_w, rw = ab ? a.ar_w : a.mr_w;
-  const TI* src = (const TI*)a.q + (size_t)t * a.ld;
-  auto value = [&](int c) {
-    float v = ldv(src + c);
-    for (int p = 1; p < a.n_part; ++p) v += ldv(src + (size_t)p * a.part_stride + c);
-    return v;
-  };
-  const int w = nw + rw, hd = a.dim + a.rot_dim;
-  for (int i = tid; i < a.heads * w; i += 256) {
-    const int h = i / w, c = i - h * w;
-    if (c < nw) stv(on + h * n_hs + c, c < a.dim ? value(h * hd + c) * a.scale : 0.f);
-    else {
-      const int x = c - nw;
-      float y = 0.f;
-      if (x < a.rot_dim) {
-        const int p = h * hd + a.dim + (x & ~1);
-        const float u = value(p), v = value(p + 1), co = cs[x >> 1], si = cs[half + (x >> 1)];
-        y = (x & 1) ? v * co + u * si : u * co - v * si;
-      }
-      stv(orr + h * r_hs + x, y);
+  const int nw = ab ? a.an_w : a.mn_w, rw = ab ? a.ar_w : a.mr_w, hd = a.dim + a.rot_dim;
+  const int h_end = min(a.heads, (int)(blockIdx.y + 1) * per);
+  for (int h = blockIdx.y * per + warp; h < h_end; h += 8) {
+    TO* on = (TO*)(ab ? a.a_n : a.m_n) + row * (ab ? a.an_ts : a.mn_ts) + h * (ab ? a.an_hs : a.mn_hs);
+    TO* orr = (TO*)(ab ? a.a_r : a.m_r) + row * (ab ? a.ar_ts : a.mr_ts) + h * (ab ? a.ar_hs : a.mr_hs);
+    const TI* src = (const TI*)a.q + (size_t)t * a.ld + h * hd;
+    auto value = [&](int c) {
+      float v = ldv(src + c);
+      for (int p = 1; p < a.n_part; ++p) v += ldv(src + (size_t)p * a.part_stride + c);
+      return v;
+    };
+    for (int c = lane; c < nw; c += 32) stv(on + c, c < a.dim ? value(c) * a.scale : 0.f);
+    for (int i = lane; i < half; i += 32) {
+      const float u = value(a.dim + 2 * i), v = value(a.dim + 2 * i + 1), co = cs[i], si = cs[half + i];
+      stv(orr + 2 * i, u * co - v * si);
+      stv(orr + 2 * i + 1, v * co + u * si);
     }
+    for (int c = a.rot_dim + lane; c < rw; c += 32) stv(orr + c, 0.f);
   }
 }
 
@@ -168,10 +186,16 @@ GB_API int gb_latent_store(const void* rows, int in_f32, int n_part, long part_s
   a.a = rows; a.n_part = n_part; a.part_stride = part_stride; a.ld = ld; a.positions = positions; a.slots = slots; a.q_norm = q_norm; a.kv_norm = kv_norm;
   a.freq = freq; a.mag = mag; a.q_out = q_out; a.ld_q = ld_q; a.cache = cache; a.num_slots = num_slots; a.ld_c = ld_c; a.q_rank = q_rank; a.rank = rank;
   a.rot_dim = rot_dim; a.eps = eps;
-  if (in_f32 && out_f32) launch_k(latent_store_kernel<float, float>, (unsigned)tokens, 256, 0, stream, a);
-  else if (in_f32) launch_k(latent_store_kernel<float, __nv_bfloat16>, (unsigned)tokens, 256, 0, stream, a);
-  else if (out_f32) return fail("latent_store: a 32-bit cache takes 32-bit rows%s");
-  else launch_k(latent_store_kernel<__nv_bfloat16, __nv_bfloat16>, (unsigned)tokens, 256, 0, stream, a);
+  const auto al = [](const void* p, size_t n) { return (uintptr_t)p % n == 0; };
+  const size_t ei = in_f32 ? 16 : 8, eo = out_f32 ? 16 : 8;
+  const bool vec = q_rank % 4 == 0 && rank % 4 == 0 && ld % 4 == 0 && part_stride % 4 == 0 && ld_q % 4 == 0 && ld_c % 4 == 0 && al(rows, ei) && al(q_out, eo) && al(cache, eo) &&
+                   al(q_norm, 16) && al(kv_norm, 16);
+  if (!in_f32 && out_f32) return fail("latent_store: a 32-bit cache takes 32-bit rows%s");
+#define GB_LAT(TI, TO) (vec ? launch_k(latent_store_kernel<TI, TO, 4>, (unsigned)tokens, 256, 0, stream, a) : launch_k(latent_store_kernel<TI, TO, 1>, (unsigned)tokens, 256, 0, stream, a))
+  if (in_f32 && out_f32) GB_LAT(float, float);
+  else if (in_f32) GB_LAT(float, __nv_bfloat16);
+  else GB_LAT(__nv_bfloat16, __nv_bfloat16);
+#undef GB_LAT
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -189,10 +213,12 @@ GB_API int gb_latent_q(const void* q, int in_f32, int n_part, long part_stride, 
   a.m_n = m_n; a.mn_ts = mn_ts; a.mn_hs = mn_hs; a.mn_w = mn_w; a.m_r = m_r; a.mr_ts = mr_ts; a.mr_hs = mr_hs; a.mr_w = mr_w;
   a.heads = heads; a.dim = dim; a.rot_dim = rot_dim;
   const size_t smem = (size_t)rot_dim * sizeof(float);
-  if (in_f32 && out_f32) launch_k(latent_q_kernel<float, float>, (unsigned)tokens, 256, smem, stream, a);
-  else if (in_f32) launch_k(latent_q_kernel<float, __nv_bfloat16>, (unsigned)tokens, 256, smem, stream, a);
+  const int per = tokens >= 1024 ? heads : 8;                  // small batches spread a token's heads over CTAs
+  const dim3 grid((unsigned)tokens, (unsigned)((heads + per - 1) / per));
+  if (in_f32 && out_f32) launch_k(latent_q_kernel<float, float>, grid, 256, smem, stream, a, per);
+  else if (in_f32) launch_k(latent_q_kernel<float, __nv_bfloat16>, grid, 256, smem, stream, a, per);
   else if (out_f32) return fail("latent_q: 32-bit results take 32-bit rows%s");
-  else launch_k(latent_q_kernel<__nv_bfloat16, __nv_bfloat16>, (unsigned)tokens, 256, smem, stream, a);
+  else launch_k(latent_q_kernel<__nv_bfloat16, __nv_bfloat16>, grid, 256, smem, stream, a, per);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }

@@ -2,10 +2,12 @@
 //
 // latent_decode_kernel (absorbed form): the cached rows [latent | rotated key part] are keys and values of all query heads at once.  A CTA owns one
 // token, a tile of NH heads and a range of its keys.  As in the decode kernel of flash_attn.cu the key POSITIONS are the MMA's M dimension:
-//   S^T[128 positions x NH] = C_j[128 x width] Q^T           (A = rows as they are cached, K-major; B = the heads' queries)
-//   O^T[128 columns x NH]  += C_j^T[128 x 128 positions] P_j  (A = the same rows, MN-major, one product per 128 latent columns; B = P^T in shared memory)
-// so that every cached byte is fetched once for both products.  A block of 128 positions is a row of boxes of 64 columns (16 KB), each with its own
-// barriers: S starts with the first box that lands, and O's products free the boxes pair by pair for the next block.
+//   S^T[positions x NH]   = C_j[positions x width] Q^T       (A = rows as they are cached, K-major; B = the heads' queries)
+//   O^T[128 columns x NH] += C_j^T[128 x positions] P_j      (A = the same rows, MN-major, one product per 128 latent columns; B = P^T in shared memory)
+// so that every cached byte is fetched once for both products.  A block of 64 positions is a row of boxes of 64 columns (8 KB), each with its own
+// barriers: S starts with the first box that lands, and O's products free the boxes pair by pair.  Two blocks of 512 + 64 columns fit beside the
+// queries of 32 heads (with 128 positions it would be one, and loads would stop while a block is computed: measured 2.4 times slower), so S of a
+// block has only half of an MMA's rows.
 //
 // latent_prefill_kernel (expanded form): keys [expanded part | rotated part shared by the heads] and values of one head.  A CTA owns one head and
 // two tiles of 128 tokens, which take turns: while one tile's softmax runs, the tensor core works for the other.  K is double-buffered.
@@ -19,8 +21,9 @@
 namespace gb {
 
 constexpr int kLdThreads = 192;
-constexpr int kLdBox = 16384;             // 128 positions x 64 columns
-constexpr int kLdMaxBoxes = 16;           // boxes in shared memory
+constexpr int kLdB = 64;                  // positions per block
+constexpr int kLdBox = 8192;              // 64 positions x 64 columns
+constexpr int kLdMaxPairs = 24;           // pairs of boxes in shared memory
 
 struct LatentDecodeArgs {
   const int* tok_seq; const int* tok_kv;  // per token: row of the block table, number of keys; null: token i is sequence i, kv_len[i] keys
@@ -28,7 +31,7 @@ struct LatentDecodeArgs {
   const int* block_table; int max_pages, page_size;
   int tokens, heads, head_tiles, splits;
   int width, rank;                        // key columns, of which the first `rank` are the values
-  int boxes, stages;                      // 64-column boxes per block (even), blocks in shared memory
+  int boxes, stages;                      // 64-column boxes per block, blocks in shared memory
   __nv_bfloat16* out; int m_rows, ld_out; // [heads][m_rows][ld_out]
   float* part_o; float* part_lse;         // [splits][tokens][heads][rank], [splits][tokens][heads] (splits > 1)
   const float* sink;
@@ -45,27 +48,28 @@ __global__ void __launch_bounds__(kLdThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmC, const LatentDecodeArgs a) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
-  constexpr int kQ = NH * 128;            // bytes of a 64-column box of queries
-  const int slots = a.boxes * a.stages;
+  constexpr int kQ = NH * 128;            // bytes of a 64-column box of queries, and of P^T
+  const int pairs = (a.boxes + 1) >> 1;
   uint8_t* sC = smem;
-  uint8_t* sQ = sC + slots * kLdBox;
-  uint8_t* sP = sQ + a.boxes * kQ;        // two halves of 64 positions x NH rows
-  uint64_t* bars = (uint64_t*)(sP + 2 * kQ);
+  uint8_t* sP = sC + a.boxes * a.stages * kLdBox;      // two buffers
+  uint8_t* sQ = sP + 2 * kQ;              // (behind the last box at least 8 KB are queries and P: an operand of 128 rows may start in it)
+  uint64_t* bars = (uint64_t*)(sQ + max(a.boxes, 2) * kQ);
   uint64_t* q_full = bars;
-  uint64_t* s_full = bars + 1;
-  uint64_t* p_ready = bars + 2;           // 128 arrivals
-  uint64_t* o_ready = bars + 3;
-  uint64_t* t_full = bars + 4;            // per box
-  uint64_t* t_empty = t_full + kLdMaxBoxes;
-  uint32_t* tmem_slot = (uint32_t*)(t_empty + kLdMaxBoxes);
+  uint64_t* s_full = bars + 1;            // 2, by block parity
+  uint64_t* p_ready = bars + 3;           // 2, 128 arrivals each (two for the reason given in flash_decode_kernel)
+  uint64_t* o_ready = bars + 5;           // 2
+  uint64_t* t_full = bars + 7;            // per box
+  uint64_t* t_empty = t_full + kLdMaxPairs;
+  uint32_t* tmem_slot = (uint32_t*)(t_empty + kLdMaxPairs);
   volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
-  float* red_max = (float*)(tmem_slot + 4);            // [2][4][NH]
-  float* red_sum = red_max + 2 * 4 * NH;               // [4][NH]
+  float* red_max = (float*)(((uintptr_t)(tmem_slot + 2) + 15) & ~(uintptr_t)15);       // [2 (block parity)][2 warps][NH]
+  float* red_sum = red_max + 4 * NH;                                                   // [2][NH]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    mbar_init(q_full, 1); mbar_init(s_full, 1); mbar_init(p_ready, 128); mbar_init(o_ready, 1);
-    for (int i = 0; i < slots; ++i) { mbar_init(&t_full[i], 1); mbar_init(&t_empty[i], 1); }
+    mbar_init(q_full, 1);
+    for (int i = 0; i < 2; ++i) { mbar_init(&s_full[i], 1); mbar_init(&p_ready[i], 128); mbar_init(&o_ready[i], 1); }
+    for (int i = 0; i < pairs * a.stages; ++i) { mbar_init(&t_full[i], 1); mbar_init(&t_empty[i], 1); }
     *abort_flag = 0;
     fence_barrier_init();
     tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmC);
@@ -74,14 +78,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + NH;
+  const uint32_t tmem_s = *tmem_slot, tmem_o = tmem_s + 2 * NH;
   pdl_wait();
 
   const int split = blockIdx.x % a.splits, ht = (blockIdx.x / a.splits) % a.head_tiles, tok = blockIdx.x / (a.splits * a.head_tiles);
   const int h0 = ht * NH, n_heads = min(NH, a.heads - h0);
   const int seq = a.tok_seq != nullptr ? a.tok_seq[tok] : tok;
   const int kv = a.tok_kv != nullptr ? a.tok_kv[tok] : a.kv_len[tok];
-  const int n_all = (kv + 127) >> 7, per = (n_all + a.splits - 1) / a.splits;
+  const int n_all = (kv + kLdB - 1) / kLdB, per = (n_all + a.splits - 1) / a.splits;
   const int blk0 = split * per, n_blk = max(0, min(n_all, blk0 + per) - blk0);
   const int m_tiles = (a.rank + 127) >> 7;
 
@@ -89,131 +93,186 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     if (lane == 0 && n_blk > 0) {
       mbar_expect_tx(q_full, (uint32_t)(a.boxes * kQ));
       for (int b = 0; b < a.boxes; ++b) tma_load_3d(sQ + b * kQ, &tmQ, q_full, b * 64, tok, h0);
-      const int ppb = 128 / a.page_size;
+      // page sizes are powers of two.  Pages behind the last one are replaced by it: finite rows, masked
+      const int shift = __ffs(a.page_size) - 1, last_page = (kv - 1) >> shift;
       const int* bt = a.block_table + (size_t)seq * a.max_pages;
-      const int last_page = (kv + a.page_size - 1) / a.page_size - 1;
+      auto cache_row = [&](int pos) { return (bt[min(pos >> shift, last_page)] << shift) + (pos & (a.page_size - 1)); };
       bool ok = true;
-      for (int j = 0; j < n_blk && ok; ++j) {
-        const int st = j % a.stages;
-        const uint32_t ph = (uint32_t)(j / a.stages) & 1;
-        for (int b = 0; b < a.boxes; ++b) {
-          const int s = st * a.boxes + b;
-          if (!mbar_wait(&t_empty[s], ph ^ 1, abort_flag, a.status, 800, j)) { ok = false; break; }
-          mbar_expect_tx(&t_full[s], kLdBox);
-          for (int p = 0; p < ppb; ++p) {        // pages behind the last one are replaced by it: finite rows, masked
-            const int page = bt[min((blk0 + j) * ppb + p, last_page)];
-            tma_load_2d(sC + s * kLdBox + p * a.page_size * 128, &tmC, &t_full[s], b * 64, page * a.page_size);
+      int st = 0; uint32_t ph = 1;
+      if (a.page_size >= kLdB) {                 // a block lies in one page; its row is looked up a block ahead
+        int next = cache_row(blk0 * kLdB);
+        for (int j = 0; j < n_blk && ok; ++j) {
+          const int row = next;
+          if (j + 1 < n_blk) next = cache_row((blk0 + j + 1) * kLdB);
+          uint8_t* dst = sC + st * a.boxes * kLdBox;
+          for (int b = 0; b < a.boxes; b += 2, dst += 2 * kLdBox) {
+            const int s = st * pairs + (b >> 1);
+            if (!mbar_wait(&t_empty[s], ph, abort_flag, a.status, 800, j)) { ok = false; break; }
+            const bool two = b + 1 < a.boxes;
+            mbar_expect_tx(&t_full[s], two ? 2 * kLdBox : kLdBox);
+            tma_load_2d(dst, &tmC, &t_full[s], b * 64, row);
+            if (two) tma_load_2d(dst + kLdBox, &tmC, &t_full[s], b * 64 + 64, row);
           }
+          if (++st == a.stages) { st = 0; ph ^= 1; }
+        }
+      } else {
+        for (int j = 0; j < n_blk && ok; ++j) {
+          for (int b = 0; b < a.boxes; b += 2) {
+            const int s = st * pairs + (b >> 1);
+            if (!mbar_wait(&t_empty[s], ph, abort_flag, a.status, 801, j)) { ok = false; break; }
+            const bool two = b + 1 < a.boxes;
+            mbar_expect_tx(&t_full[s], two ? 2 * kLdBox : kLdBox);
+            for (int x = 0; x < kLdB; x += a.page_size) {
+              const int row = cache_row((blk0 + j) * kLdB + x);
+              uint8_t* dst = sC + (st * a.boxes + b) * kLdBox + x * 128;
+              tma_load_2d(dst, &tmC, &t_full[s], b * 64, row);
+              if (two) tma_load_2d(dst + kLdBox, &tmC, &t_full[s], b * 64 + 64, row);
+            }
+          }
+          if (++st == a.stages) { st = 0; ph ^= 1; }
         }
       }
     }
   } else if (warp == 1) {
     if (lane == 0 && n_blk > 0) {
+      // S: the operand's rows 64 .. 127 are whatever lies behind the box; nobody reads their scores
       constexpr uint32_t id_s = make_idesc(128, NH, 1, 1, 0, 0);
       constexpr uint32_t id_o = make_idesc(128, NH, 1, 1, 1, 0);      // A (latents by position) is MN-major
-      const uint32_t q_addr = smem_u32(sQ), p_addr = smem_u32(sP), c_addr = smem_u32(sC);
+      const uint64_t d_q = make_sdesc_sw128(smem_u32(sQ)), d_p = make_sdesc_sw128(smem_u32(sP)), d_c = make_sdesc_sw128(smem_u32(sC));
+      const uint64_t d_v = make_sdesc_sw128_mn(smem_u32(sC), kLdBox);
       const int k_steps = (a.width + 15) >> 4;
       bool ok = mbar_wait(q_full, 0, abort_flag, a.status, 810);
-      for (int j = 0; j < n_blk && ok; ++j) {
-        const int s0 = (j % a.stages) * a.boxes;
-        const uint32_t ph = (uint32_t)(j / a.stages) & 1;
-        for (int b = 0; b < a.boxes; ++b) {
-          if (!mbar_wait(&t_full[s0 + b], ph, abort_flag, a.status, 811, j)) { ok = false; break; }
+      int st_s = 0, st_o = 0; uint32_t ph_s = 0;
+      auto issue_s = [&](int j) -> bool {
+        const uint32_t d = tmem_s + (j & 1) * NH;
+        uint64_t dc = sdesc_at(d_c, st_s * a.boxes * kLdBox), dq = d_q;
+        for (int b = 0; b < pairs; ++b) {
+          uint64_t* bar = &t_full[st_s * pairs + b];
+          if (!mbar_wait(bar, ph_s, abort_flag, a.status, 811, j)) return false;
           tc_fence_after();
-          for (int x = 0; x < 4; ++x)
-            if (b * 4 + x < k_steps)
-              mma_f16_ss(tmem_s, make_sdesc_sw128(c_addr + (s0 + b) * kLdBox + x * 32), make_sdesc_sw128(q_addr + b * kQ + x * 32), id_s, (b | x) ? 1u : 0u);
-          if (b >= 2 * m_tiles) tc_commit(&t_empty[s0 + b]);          // no values in this box
-        }
-        if (!ok) break;
-        tc_commit(s_full);                 // also: every product of the earlier blocks has landed in O
-        if (!mbar_wait(p_ready, j & 1, abort_flag, a.status, 812, j)) { ok = false; break; }
-        tc_fence_after();
-        for (int m = 0; m < m_tiles; ++m) {
-          const uint32_t base = c_addr + (s0 + 2 * m) * kLdBox;
+          const uint32_t acc = b > 0 ? 1u : 0u;
+          if (b * 8 + 8 <= k_steps) {
 #pragma unroll
-          for (int ks = 0; ks < 8; ++ks)
-            mma_f16_ss(tmem_o + m * NH, make_sdesc_sw128_mn(base + ks * 2048, kLdBox), make_sdesc_sw128(p_addr + (ks >> 2) * kQ + (ks & 3) * 32), id_o,
-                       (j > 0 || ks > 0) ? 1u : 0u);
-          tc_commit(&t_empty[s0 + 2 * m]);
-          tc_commit(&t_empty[s0 + 2 * m + 1]);
+            for (int x = 0; x < 8; ++x)
+              mma_f16_ss(d, sdesc_at(dc, (x >> 2) * kLdBox + (x & 3) * 32), sdesc_at(dq, (x >> 2) * kQ + (x & 3) * 32), id_s, x > 0 ? 1u : acc);
+          } else {
+            for (int x = 0; b * 8 + x < k_steps; ++x)
+              mma_f16_ss(d, sdesc_at(dc, (x >> 2) * kLdBox + (x & 3) * 32), sdesc_at(dq, (x >> 2) * kQ + (x & 3) * 32), id_s, x > 0 ? 1u : acc);
+          }
+          if (b >= m_tiles) tc_commit(&t_empty[st_s * pairs + b]);      // no values in these boxes
+          dc = sdesc_at(dc, 2 * kLdBox); dq = sdesc_at(dq, 2 * kQ);
         }
+        tc_commit(&s_full[j & 1]);
+        if (++st_s == a.stages) { st_s = 0; ph_s ^= 1; }
+        return true;
+      };
+      if (ok) ok = issue_s(0);
+      for (int j = 0; j < n_blk && ok; ++j) {
+        if (a.stages > 1 && j + 1 < n_blk && !issue_s(j + 1)) { ok = false; break; }
+        if (!mbar_wait(&p_ready[j & 1], (uint32_t)(j >> 1) & 1, abort_flag, a.status, 812, j)) { ok = false; break; }
+        tc_fence_after();
+        uint64_t dv = sdesc_at(d_v, st_o * a.boxes * kLdBox);
+        const uint64_t dp = sdesc_at(d_p, (j & 1) * kQ);
+        const uint32_t acc = j > 0 ? 1u : 0u;
+        for (int m = 0; m < m_tiles; ++m) {
+#pragma unroll
+          for (int ks = 0; ks < 4; ++ks) mma_f16_ss(tmem_o + m * NH, sdesc_at(dv, ks * 2048), sdesc_at(dp, ks * 32), id_o, ks > 0 ? 1u : acc);
+          tc_commit(&t_empty[st_o * pairs + m]);
+          dv = sdesc_at(dv, 2 * kLdBox);
+        }
+        tc_commit(&o_ready[j & 1]);
+        if (++st_o == a.stages) st_o = 0;
+        if (a.stages == 1 && j + 1 < n_blk && !issue_s(j + 1)) { ok = false; break; }
       }
-      if (ok) tc_commit(o_ready);
     }
   } else {
-    const int q = warp & 3, r = q * 32 + lane;           // position of the block, later column of O
+    // thread r: position r of the block (r < 64), column r of each tile of O
+    const int q = warp & 3, r = q * 32 + lane;
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     float m[NH], l[NH];                                  // reference maximum; this thread's share of the sums
 #pragma unroll
     for (int h = 0; h < NH; ++h) { m[h] = -INFINITY; l[h] = 0.f; }
     constexpr float kTau = 8.0f;                         // O and l are rescaled only when a maximum has grown by more than 2^kTau
-    bool ok = true;
+    bool ok = true, fail_o = false;                      // fail_o: a wait for O ran out; it is put to the vote at the next barrier
     for (int j = 0; j < n_blk && ok; ++j) {
-      const bool got = warp_wait(s_full, j & 1, abort_flag, a.status, 820, j);
+      const bool got = warp_wait(&s_full[j & 1], (uint32_t)(j >> 1) & 1, abort_flag, a.status, 820, j);
       tc_fence_after();
       float sv[NH];
-      tmem_ld_heads<NH>(tmem_s + lane_off, reinterpret_cast<uint32_t*>(sv));
-      tc_wait_ld();
-      const bool live = (blk0 + j) * 128 + r < kv;
+      float* rm = red_max + (j & 1) * 2 * NH;
+      if (q < 2) {
+        tmem_ld_heads<NH>(tmem_s + (j & 1) * NH + lane_off, reinterpret_cast<uint32_t*>(sv));
+        tc_wait_ld();
+        const bool live = (blk0 + j) * kLdB + r < kv;
 #pragma unroll
-      for (int h = 0; h < NH; ++h) if (!live || h >= n_heads) sv[h] = -INFINITY;
-      float* rm = red_max + (j & 1) * 4 * NH;
+        for (int h = 0; h < NH; ++h) if (!live || h >= n_heads) sv[h] = -INFINITY;
 #pragma unroll
-      for (int x = 0; x < NH; x += 16) {
-        const float v = warp_reduce16_max(sv + x, lane);
-        if ((lane & 1) == 0) rm[q * NH + x + (lane >> 1)] = v;
+        for (int x = 0; x < NH; x += 16) {
+          const float v = warp_reduce16_max(sv + x, lane);
+          if ((lane & 1) == 0) rm[q * NH + x + (lane >> 1)] = v;
+        }
       }
-      if (!bar128_and(got)) { ok = false; break; }       // all 128 threads leave together
+      if (!bar128_and(got && !fail_o)) { ok = false; break; }       // all 128 threads leave together
       bool need = false;
-      float bm[NH];
 #pragma unroll
-      for (int h = 0; h < NH; ++h) {
-        bm[h] = fmaxf(fmaxf(rm[h], rm[NH + h]), fmaxf(rm[2 * NH + h], rm[3 * NH + h]));
-        need |= (h < n_heads) && (bm[h] > m[h] + kTau);  // also the first finite maximum
+      for (int h = 0; h < NH; h += 4) {
+        const float4 x = *reinterpret_cast<const float4*>(rm + h), y = *reinterpret_cast<const float4*>(rm + NH + h);
+        need |= fmaxf(x.x, y.x) > m[h] + kTau || fmaxf(x.y, y.y) > m[h + 1] + kTau || fmaxf(x.z, y.z) > m[h + 2] + kTau || fmaxf(x.w, y.w) > m[h + 3] + kTau;
       }
-      if (need) {
-        // the same for all 128 threads.  Every earlier product is in O (see s_full)
+      bool got_o = true;
+      if (need) {                                        // the same for all 128 threads; also the first finite maximum
+        // every earlier product is in O before it is rescaled
+        if (j > 0) got_o = warp_wait(&o_ready[(j - 1) & 1], (uint32_t)((j - 1) >> 1) & 1, abort_flag, a.status, 821, j);
+        tc_fence_after();
+        float al[NH];
 #pragma unroll
         for (int h = 0; h < NH; ++h) {
-          const float mn = fmaxf(m[h], bm[h]);
-          const float al = mn == -INFINITY ? 1.0f : fast_exp2(m[h] - mn);
-          m[h] = mn; l[h] *= al; bm[h] = al;             // bm: factor from here on
+          const float mn = fmaxf(m[h], fmaxf(rm[h], rm[NH + h]));
+          al[h] = mn == -INFINITY ? 1.0f : fast_exp2(m[h] - mn);
+          m[h] = mn; l[h] *= al[h];
         }
-        if (j > 0)
+        if (j > 0 && got_o)
           for (int t = 0; t < m_tiles; ++t) {
             uint32_t o[NH];
             tmem_ld_heads<NH>(tmem_o + t * NH + lane_off, o);
             tc_wait_ld();
 #pragma unroll
-            for (int h = 0; h < NH; ++h) o[h] = __float_as_uint(__uint_as_float(o[h]) * bm[h]);
+            for (int h = 0; h < NH; ++h) o[h] = __float_as_uint(__uint_as_float(o[h]) * al[h]);
             tmem_st_heads<NH>(tmem_o + t * NH + lane_off, o);
             tc_wait_st();
           }
       }
-      const int half = r >> 6, chunk = (r & 63) >> 3;
-      uint8_t* pb = sP + half * kQ + (r & 7) * 2;
+      // the P buffer of this parity was read by the product of block j - 2
+      if (got_o && j >= 2) got_o = warp_wait(&o_ready[j & 1], (uint32_t)((j - 2) >> 1) & 1, abort_flag, a.status, 822, j);
+      if (got_o) {
+        if (q < 2) {
+          uint8_t* pb = sP + (j & 1) * kQ + (r & 7) * 2;
+          const int chunk = r >> 3;
 #pragma unroll
-      for (int h = 0; h < NH; ++h) {
-        const float p = m[h] == -INFINITY ? 0.f : fast_exp2(sv[h] - m[h]);
-        l[h] += p;
-        *reinterpret_cast<__nv_bfloat16*>(pb + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16(p);
+          for (int h = 0; h < NH; ++h) {
+            const float p = h < n_heads ? fast_exp2(sv[h] - m[h]) : 0.f;
+            l[h] += p;
+            *reinterpret_cast<__nv_bfloat16*>(pb + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16(p);
+          }
+          fence_proxy_async_smem();
+        }
+        tc_fence_before();
+        mbar_arrive(&p_ready[j & 1]);
       }
-      fence_proxy_async_smem();
-      tc_fence_before();
-      mbar_arrive(p_ready);
+      fail_o |= !got_o;
     }
-    if (ok && n_blk > 0) ok = warp_wait(o_ready, 0, abort_flag, a.status, 821, 0);
+    if (ok && !fail_o && n_blk > 0) ok = warp_wait(&o_ready[(n_blk - 1) & 1], (uint32_t)((n_blk - 1) >> 1) & 1, abort_flag, a.status, 823, 0);
+    if (q < 2) {
 #pragma unroll
-    for (int x = 0; x < NH; x += 16) {
-      const float v = warp_reduce16_sum(l + x, lane);
-      if ((lane & 1) == 0) red_sum[q * NH + x + (lane >> 1)] = v;
+      for (int x = 0; x < NH; x += 16) {
+        const float v = warp_reduce16_sum(l + x, lane);
+        if ((lane & 1) == 0) red_sum[q * NH + x + (lane >> 1)] = v;
+      }
     }
-    ok = bar128_and(ok);
+    ok = bar128_and(ok && !fail_o);
     if (ok) {
       tc_fence_after();
 #pragma unroll
-      for (int h = 0; h < NH; ++h) l[h] = red_sum[h] + red_sum[NH + h] + red_sum[2 * NH + h] + red_sum[3 * NH + h];
+      for (int h = 0; h < NH; ++h) l[h] = red_sum[h] + red_sum[NH + h];
       float inv[NH];
 #pragma unroll
       for (int h = 0; h < NH; ++h) {
@@ -373,15 +432,16 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
     if (lane == 0) {
       constexpr uint32_t id_s = make_idesc(128, 128, 1, 1, 0, 0);
       const uint32_t id_o = v2 ? make_idesc(128, 128, 1, 1, 0, 1) : make_idesc(128, 64, 1, 1, 0, 1);
-      const uint32_t q_addr = smem_u32(sQ), k_addr = smem_u32(sK), v_addr = smem_u32(sV);
+      const uint64_t d_q = make_sdesc_sw128(smem_u32(sQ)), d_k = make_sdesc_sw128(smem_u32(sK)), d_v = make_sdesc_sw128_mn(smem_u32(sV), 16384);
       const int kn = (a.dn + 15) >> 4, kr = (a.dr + 15) >> 4;
       auto issue_s = [&](int t, int j) {
-        const uint32_t q = q_addr + t * 49152, k = k_addr + (j & 1) * 49152, d = tmem + 128 * t;
+        const uint64_t q = sdesc_at(d_q, t * 49152), k = sdesc_at(d_k, (j & 1) * 49152);
+        const uint32_t d = tmem + 128 * t;
         for (int ks = 0; ks < kn; ++ks) {
           const uint32_t off = (ks >> 2) * 16384 + (ks & 3) * 32;
-          mma_f16_ss(d, make_sdesc_sw128(q + off), make_sdesc_sw128(k + off), id_s, ks > 0 ? 1u : 0u);
+          mma_f16_ss(d, sdesc_at(q, off), sdesc_at(k, off), id_s, ks > 0 ? 1u : 0u);
         }
-        for (int ks = 0; ks < kr; ++ks) mma_f16_ss(d, make_sdesc_sw128(q + 32768 + ks * 32), make_sdesc_sw128(k + 32768 + ks * 32), id_s, 1u);
+        for (int ks = 0; ks < kr; ++ks) mma_f16_ss(d, sdesc_at(q, 32768 + ks * 32), sdesc_at(k, 32768 + ks * 32), id_s, 1u);
         tc_commit(&s_full[t]);
       };
       bool ok = true;
@@ -401,7 +461,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
           tc_fence_after();
 #pragma unroll
           for (int ks = 0; ks < 8; ++ks)
-            mma_f16_ts(tmem + 256 + 128 * t, tmem + 128 * t + ks * 8, make_sdesc_sw128_mn(v_addr + ks * 2048, 16384), id_o, (j > 0 || ks > 0) ? 1u : 0u);
+            mma_f16_ts(tmem + 256 + 128 * t, tmem + 128 * t + ks * 8, sdesc_at(d_v, ks * 2048), id_o, (j > 0 || ks > 0) ? 1u : 0u);
           if (j + 1 < n_blk[t]) issue_s(t, j + 1);          // in order behind the product that reads P from the same columns
           else tc_commit(&o_ready[t]);
         }
@@ -513,15 +573,18 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
 }
 
 // Shared memory of the decode kernel with `boxes` boxes per block and `stages` blocks.
-static int latent_decode_smem(int boxes, int stages, int nh) { return boxes * stages * kLdBox + (boxes + 2) * nh * 128 + 512 + 12 * nh * 4 + 1024; }
+static int latent_decode_smem(int boxes, int stages, int nh) {
+  return boxes * stages * kLdBox + ((boxes > 2 ? boxes : 2) + 2) * nh * 128 + (7 + 2 * kLdMaxPairs) * 8 + 32 + 6 * nh * 4 + 1024;
+}
 
 struct LatentDecodeShape { int nh, boxes, stages; };
 
 // nh = 0: sizes the kernel is not built for.
 static LatentDecodeShape latent_decode_shape(int heads, int width, int rank) {
-  LatentDecodeShape s = {heads <= 16 ? 16 : 32, 2 * ((width + 127) / 128), 2};
-  if (s.boxes * s.stages > kLdMaxBoxes || latent_decode_smem(s.boxes, s.stages, s.nh) > 227 * 1024) s.stages = 1;
-  if (s.boxes > kLdMaxBoxes || latent_decode_smem(s.boxes, s.stages, s.nh) > 227 * 1024 || ((rank + 127) / 128 + 1) * s.nh > 256) s.nh = 0;
+  LatentDecodeShape s = {heads <= 16 ? 16 : 32, (width + 63) / 64, 4};
+  auto fits = [&]() { return (s.boxes + 1) / 2 * s.stages <= kLdMaxPairs && latent_decode_smem(s.boxes, s.stages, s.nh) <= 227 * 1024; };
+  while (s.stages > 1 && !fits()) --s.stages;
+  if (!fits() || ((rank + 127) / 128 + 2) * s.nh > 256) s.nh = 0;
   return s;
 }
 
@@ -549,7 +612,7 @@ GB_API int gb_latent_decode(const void* q, const void* cache, int ld_c, long num
   uint64_t dq[3] = {(uint64_t)ld_c, (uint64_t)m_rows, (uint64_t)heads}, sq[2] = {(uint64_t)ld_c * 2, (uint64_t)m_rows * ld_c * 2};
   uint32_t bq[3] = {64, 1, (uint32_t)sh.nh};
   if (make_tmap(&tmQ, q, TM_BF16, 3, dq, sq, bq, TM_SW_128)) return -1;
-  if (make_tmap_2d(&tmC, cache, TM_BF16, (uint64_t)ld_c, (uint64_t)num_slots, (uint64_t)ld_c * 2, 64, (uint32_t)page_size, TM_SW_128)) return -1;
+  if (make_tmap_2d(&tmC, cache, TM_BF16, (uint64_t)ld_c, (uint64_t)num_slots, (uint64_t)ld_c * 2, 64, (uint32_t)(page_size < kLdB ? page_size : kLdB), TM_SW_128)) return -1;
   LatentDecodeArgs a;
   a.tok_seq = tok_seq; a.tok_kv = tok_kv; a.kv_len = kv_len; a.block_table = block_table; a.max_pages = max_pages; a.page_size = page_size; a.tokens = tokens;
   a.heads = heads; a.head_tiles = (heads + sh.nh - 1) / sh.nh; a.splits = splits; a.width = width; a.rank = rank; a.boxes = sh.boxes; a.stages = sh.stages;

@@ -288,6 +288,9 @@ __device__ __forceinline__ uint64_t make_sdesc_sw128_mn(uint32_t smem_addr, uint
   d |= (uint64_t)2 << 61;
   return d;
 }
+// The descriptor of the operand `bytes` (a multiple of 16) further on: one add, where building it anew costs the issuing thread about eight dependent
+// instructions per MMA (shared memory ends below 2^18 bytes, so the address field does not carry over).
+__device__ __forceinline__ uint64_t sdesc_at(uint64_t d, uint32_t bytes) { return d + (bytes >> 4); }
 // Descriptor of an un-swizzled K-major block of 8-row x 16-byte core matrices laid out back to back:
 // used for the 32 x 16-byte scale-factor blocks copied with tcgen05.cp (4 core matrices of 128 bytes).
 __device__ __forceinline__ uint64_t make_sdesc_noswizzle(uint32_t smem_addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {

@@ -374,7 +374,60 @@ struct PartNormArgs {
   void* out; int ld_out; int n, parts; float eps; long items;
 };
 
-// G threads (a warp or a CTA) per (row, part).
+// G threads (a warp or a CTA) per (row, part), values in registers: parts of 4 G VPT columns at most, a multiple of 4; one weight per column of the row
+// or of the part.
+template <typename TG, typename TO, int G, int VPT>
+__global__ void __launch_bounds__(256)
+part_norm_vec_kernel(const PartNormArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[8];
+  const long item = (long)blockIdx.x * (256 / G) + threadIdx.x / G;
+  const bool live = item < a.items;
+  const long r = live ? item / a.parts : 0;
+  const int part = live ? (int)(item - r * a.parts) : 0, lane = threadIdx.x % G;
+  const int len = a.n / a.parts, c0 = part * len, nv = live ? len >> 2 : 0;
+  const float* o = a.o + (size_t)r * a.ld_o + c0;
+  const TG* g = (const TG*)a.gate + (size_t)r * a.ld_gate + c0;
+  float4 v[VPT], z[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = lane + i * G;
+    v[i] = z[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < nv) { v[i] = ld4(o + c * 4); if (a.gate != nullptr) z[i] = ld4(g + c * 4); }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = lane + i * G;
+    if (a.gate != nullptr && c < nv) {
+      for (int p = 1; p < a.n_part; ++p) {
+        const float4 q = ld4(g + (size_t)p * a.part_stride + c * 4);
+        z[i].x += q.x; z[i].y += q.y; z[i].z += q.z; z[i].w += q.w;
+      }
+      v[i].x *= z[i].x / (1.0f + expf(-z[i].x)); v[i].y *= z[i].y / (1.0f + expf(-z[i].y));
+      v[i].z *= z[i].z / (1.0f + expf(-z[i].z)); v[i].w *= z[i].w / (1.0f + expf(-z[i].w));
+    }
+    ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+  }
+  if constexpr (G == 32) ss = warp_sum(ss);
+  else ss = block_sum_256(ss, red);
+  if (!live) return;
+  const float inv = 1.0f / sqrtf(ss / (float)len + a.eps);
+  TO* out = (TO*)a.out + (size_t)r * a.ld_out;
+  const float* w = a.weight + (a.n_weight == a.n ? c0 : 0);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = lane + i * G;
+    if (c >= nv) continue;
+    const float4 q = ld4(w + c * 4);
+    st4(out + c0 + c * 4, make_float4(v[i].x * inv * q.x, v[i].y * inv * q.y, v[i].z * inv * q.z, v[i].w * inv * q.w));
+  }
+  if (part == a.parts - 1)
+    for (int c = a.n + lane; c < a.ld_out; c += G) st_f(out + c, 0.f);
+}
+
+// Any sizes.
 template <typename TG, typename TO, int G>
 __global__ void __launch_bounds__(256)
 part_norm_kernel(const PartNormArgs a) {
@@ -501,7 +554,17 @@ GB_API int gb_stream_dyt(float* x, const void* delta, int delta_f32, int n_part,
 
 template <typename TG, typename TO>
 static int part_norm_launch(const PartNormArgs& a, cudaStream_t stream) {
-  if (a.n / a.parts <= 512) launch_k(part_norm_kernel<TG, TO, 32>, (unsigned)((a.items + 7) / 8), 256, 0, stream, a);
+  const int len = a.n / a.parts;
+  const size_t eg = sizeof(TG) * 4, eo = sizeof(TO) * 4;
+  const bool vec = len % 4 == 0 && len <= 4096 && (a.n_weight == a.n || a.n_weight == len) && a.ld_o % 4 == 0 && a.ld_out % 4 == 0 && (uintptr_t)a.o % 16 == 0 &&
+                   (uintptr_t)a.weight % 16 == 0 && (uintptr_t)a.out % eo == 0 &&
+                   (a.gate == nullptr || (a.ld_gate % 4 == 0 && a.part_stride % 4 == 0 && (uintptr_t)a.gate % eg == 0));
+  const unsigned warps = (unsigned)((a.items + 7) / 8);
+  if (vec && len <= 128) launch_k(part_norm_vec_kernel<TG, TO, 32, 1>, warps, 256, 0, stream, a);
+  else if (vec && len <= 512) launch_k(part_norm_vec_kernel<TG, TO, 32, 4>, warps, 256, 0, stream, a);
+  else if (vec && len <= 1024) launch_k(part_norm_vec_kernel<TG, TO, 256, 1>, (unsigned)a.items, 256, 0, stream, a);
+  else if (vec) launch_k(part_norm_vec_kernel<TG, TO, 256, 4>, (unsigned)a.items, 256, 0, stream, a);
+  else if (len <= 512) launch_k(part_norm_kernel<TG, TO, 32>, (unsigned)((a.items + 7) / 8), 256, 0, stream, a);
   else launch_k(part_norm_kernel<TG, TO, 256>, (unsigned)a.items, 256, 0, stream, a);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
