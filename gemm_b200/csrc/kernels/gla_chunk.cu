@@ -24,8 +24,8 @@ namespace gb {
 
 constexpr int kGlB = 16;                   // tokens per block
 
-// Layout of a record (bytes), channels padded to DP: q c hi, lo; k r hi, lo (each DP / 64 tiles of 16 rows x 128 bytes, 128-byte swizzle); P (16 rows x
-// 128 bytes: 16 hi, 16 lo); b (f32).
+// Layout of a record (bytes), channels padded to DP: q c (DP / 64 tiles of 16 hi rows, then 16 lo rows, of 128 bytes); k r hi, then lo (each DP / 64
+// tiles of 16 rows x 128 bytes); P (16 rows x 128 bytes: 16 hi, 16 lo); b (f32).  128-byte swizzle.
 template <int DP> struct GlaRecord {
   static constexpr int kTile = DP / 64 * 2048;
   static constexpr int kQ = 0, kK = 2 * kTile, kP = 4 * kTile, kB = kP + 2048, kBytes = kB + DP * 4;
@@ -83,9 +83,9 @@ gla_prep_kernel(const GlaArgs a) {
       p0 *= f.x; p1 *= f.y;
       uint32_t hi, lo;
       split_bf16x2(q.x * p0, q.y * p1, hi, lo);
-      uint8_t* dst = rec + R::kQ + tile + i * 128 + ((chunk ^ (i & 7)) << 4) + in;
+      uint8_t* dst = rec + R::kQ + 2 * tile + i * 128 + ((chunk ^ (i & 7)) << 4) + in;
       *reinterpret_cast<uint32_t*>(dst) = hi;
-      *reinterpret_cast<uint32_t*>(dst + R::kTile) = lo;
+      *reinterpret_cast<uint32_t*>(dst + 2048) = lo;
     }
   } else if (role == 1) {
     float p0 = 1.f, p1 = 1.f;
@@ -141,17 +141,17 @@ gla_prep_kernel(const GlaArgs a) {
 constexpr int kGlStages = 8;
 template <int DP> constexpr int gla_stage() { return (4096 + GlaRecord<DP>::kBytes + 1023) / 1024 * 1024; }        // V (two tiles), record
 template <int DP> constexpr int gla_smem() { return kGlStages * gla_stage<DP>() + 512 + 1024; }
-template <int DP> constexpr int gla_threads() { return 32 * (6 + DP / 16); }
+template <int DP> constexpr int gla_threads() { return 32 * (8 + DP / 16); }      // producer, two MMA warps, one idle, 4 output, state warps
 
 template <int DP>
-__global__ void __launch_bounds__(32 * (6 + DP / 16), 1)
+__global__ void __launch_bounds__(32 * (8 + DP / 16), 1)
 gla_scan_kernel(const __grid_constant__ CUtensorMap tmV, const GlaArgs a) {
   using R = GlaRecord<DP>;
   constexpr int kStage = gla_stage<DP>(), kStateWarps = DP / 16;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
   uint64_t* full = (uint64_t*)(smem + kGlStages * kStage);
-  uint64_t* empty = full + kGlStages;      // the block's last product, and the state warps (b has been read)
+  uint64_t* empty = full + kGlStages;      // both products, and the state warps (b has been read)
   uint64_t* ds_full = empty + kGlStages;
   uint64_t* ds_free = ds_full + 1;         // state warps
   uint64_t* s_ready = ds_full + 2;         // 2, by block parity; state warps
@@ -162,7 +162,7 @@ gla_scan_kernel(const __grid_constant__ CUtensorMap tmV, const GlaArgs a) {
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
-    for (int i = 0; i < kGlStages; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 1 + kStateWarps); }
+    for (int i = 0; i < kGlStages; ++i) { mbar_init(&full[i], 1); mbar_init(&empty[i], 2 + kStateWarps); }
     mbar_init(ds_full, 1); mbar_init(ds_free, kStateWarps);
     for (int i = 0; i < 2; ++i) { mbar_init(&s_ready[i], kStateWarps); mbar_init(&o_full[i], 1); mbar_init(&o_free[i], 4); }
     *abort_flag = 0;
@@ -174,7 +174,7 @@ gla_scan_kernel(const __grid_constant__ CUtensorMap tmV, const GlaArgs a) {
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *tmem_slot;
-  const uint32_t t_ds = tmem, t_s = tmem + 128, t_o = tmem + 384;       // dS: DP columns; S: two buffers of (hi 64, lo 64); O: two of 16
+  const uint32_t t_ds = tmem, t_s = tmem + 128, t_o = tmem + 384;       // dS: DP columns; S: two buffers of (hi 64, lo 64); O: two of 32
   pdl_wait();
 
   const int h = blockIdx.x, e0 = blockIdx.y * 128, seq = blockIdx.z;
@@ -197,53 +197,57 @@ gla_scan_kernel(const __grid_constant__ CUtensorMap tmV, const GlaArgs a) {
       }
     }
   } else if (warp == 1) {
+    // dS is on the chain from block to block, O is not: two threads issue them
     if (lane == 0) {
-      constexpr uint32_t id_ds = make_idesc(128, DP, 1, 1, 1, 1), id_s = make_idesc(128, kGlB, 1, 1, 0, 0), id_p = make_idesc(128, kGlB, 1, 1, 1, 0);
-      const uint64_t d_k = make_sdesc_sw128(smem_u32(smem)), d_mn = make_sdesc_sw128_mn(smem_u32(smem), 2048);      // of stage 0's start
-      // vdim <= 64: rows 64 .. 127 of the products come from whatever the second V tile holds; nobody reads them
-      auto issue_ds = [&](int b) -> bool {
-        const int st = b % kGlStages;
-        if (!mbar_wait(&full[st], (uint32_t)(b / kGlStages) & 1, abort_flag, a.status, 910, b)) return false;
+      constexpr uint32_t id_ds = make_idesc(128, DP, 1, 1, 1, 1);
+      const uint64_t d_mn = make_sdesc_sw128_mn(smem_u32(smem), 2048);      // of stage 0's start
+      int st = 0; uint32_t ph = 0;
+      for (int b = 0; b < n_blk; ++b) {
+        if (!mbar_wait(&full[st], ph, abort_flag, a.status, 910, b)) break;
+        if (b > 0 && !mbar_wait(ds_free, (uint32_t)(b - 1) & 1, abort_flag, a.status, 911, b)) break;
         tc_fence_after();
+        // vdim <= 64: rows 64 .. 127 of the products come from whatever the second V tile holds; nobody reads them
         const uint64_t v = sdesc_at(d_mn, st * kStage), k = sdesc_at(v, 4096 + R::kK);
         mma_f16_ss(t_ds, v, k, id_ds, 0u);
         mma_f16_ss(t_ds, v, sdesc_at(k, R::kTile), id_ds, 1u);
         tc_commit(ds_full);
-        return true;
-      };
-      bool ok = n_blk == 0 || issue_ds(0);
-      for (int b = 0; b < n_blk && ok; ++b) {
-        // the state warps have taken dS of this block; S in front of it is in tensor memory (waited for before the next dS is issued, so that
-        // its barrier cannot complete another phase unseen)
-        if (!mbar_wait(ds_free, b & 1, abort_flag, a.status, 911, b)) break;
-        if (!mbar_wait(&s_ready[b & 1], (uint32_t)(b >> 1) & 1, abort_flag, a.status, 912, b)) break;
-        tc_fence_after();
-        if (b + 1 < n_blk && !issue_ds(b + 1)) break;
-        if (b >= 2 && !mbar_wait(&o_free[b & 1], ((uint32_t)(b >> 1) & 1) ^ 1, abort_flag, a.status, 913, b)) break;
-        tc_fence_after();
-        const int st = b % kGlStages;
-        const uint64_t v = sdesc_at(d_mn, st * kStage), q = sdesc_at(d_k, st * kStage + 4096 + R::kQ), p = sdesc_at(d_k, st * kStage + 4096 + R::kP);
-        const uint32_t s_hi = t_s + (b & 1) * 128, s_lo = s_hi + 64, o = t_o + (b & 1) * kGlB;
-        mma_f16_ss(o, v, p, id_p, 0u);
-        mma_f16_ss(o, v, sdesc_at(p, 32), id_p, 1u);
-#pragma unroll
-        for (int x = 0; x < 3; ++x)
-#pragma unroll
-          for (int ks = 0; ks < DP / 16; ++ks)
-            mma_f16_ts(o, (x == 1 ? s_lo : s_hi) + ks * 8, sdesc_at(q, (x == 2 ? R::kTile : 0) + (ks >> 2) * 2048 + (ks & 3) * 32), id_s, 1u);
-        tc_commit(&o_full[b & 1]);
         tc_commit(&empty[st]);
+        if (++st == kGlStages) { st = 0; ph ^= 1; }
       }
     }
-  } else if (warp < 6) {
+  } else if (warp == 2) {
+    if (lane == 0) {
+      // S_hi meets [q c hi; q c lo] in one product of 32 columns, which the output warps add
+      constexpr uint32_t id_hi = make_idesc(128, 2 * kGlB, 1, 1, 0, 0), id_lo = make_idesc(128, kGlB, 1, 1, 0, 0), id_p = make_idesc(128, kGlB, 1, 1, 1, 0);
+      const uint64_t d_k = make_sdesc_sw128(smem_u32(smem)), d_mn = make_sdesc_sw128_mn(smem_u32(smem), 2048);
+      int st = 0; uint32_t ph = 0;
+      for (int b = 0; b < n_blk; ++b) {
+        if (!mbar_wait(&full[st], ph, abort_flag, a.status, 915, b)) break;
+        if (!mbar_wait(&s_ready[b & 1], (uint32_t)(b >> 1) & 1, abort_flag, a.status, 912, b)) break;
+        if (b >= 2 && !mbar_wait(&o_free[b & 1], ((uint32_t)(b >> 1) & 1) ^ 1, abort_flag, a.status, 913, b)) break;
+        tc_fence_after();
+        const uint64_t v = sdesc_at(d_mn, st * kStage), q = sdesc_at(d_k, st * kStage + 4096 + R::kQ), p = sdesc_at(d_k, st * kStage + 4096 + R::kP);
+        const uint32_t s_hi = t_s + (b & 1) * 128, s_lo = s_hi + 64, o = t_o + (b & 1) * 2 * kGlB;
+#pragma unroll
+        for (int ks = 0; ks < DP / 16; ++ks) mma_f16_ts(o, s_hi + ks * 8, sdesc_at(q, (ks >> 2) * 4096 + (ks & 3) * 32), id_hi, ks > 0 ? 1u : 0u);
+#pragma unroll
+        for (int ks = 0; ks < DP / 16; ++ks) mma_f16_ts(o, s_lo + ks * 8, sdesc_at(q, (ks >> 2) * 4096 + (ks & 3) * 32), id_lo, 1u);
+        mma_f16_ss(o, v, p, id_p, 1u);
+        mma_f16_ss(o, v, sdesc_at(p, 32), id_p, 1u);
+        tc_commit(&o_full[b & 1]);
+        tc_commit(&empty[st]);
+        if (++st == kGlStages) { st = 0; ph ^= 1; }
+      }
+    }
+  } else if (warp >= 4 && warp < 8) {
     // ---------------------------------------------------------------- output: lane = value column
     const int q = warp & 3, v = e0 + q * 32 + lane;
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     for (int b = 0; b < n_blk; ++b) {
       if (!warp_wait(&o_full[b & 1], (uint32_t)(b >> 1) & 1, abort_flag, a.status, 920, b)) break;
       tc_fence_after();
-      float o[kGlB];
-      tmem_ld_x16(t_o + (b & 1) * kGlB + lane_off, reinterpret_cast<uint32_t*>(o));
+      float o[2 * kGlB];
+      tmem_ld_x32(t_o + (b & 1) * 2 * kGlB + lane_off, reinterpret_cast<uint32_t*>(o));
       tc_wait_ld();
       tc_fence_before();
       __syncwarp();
@@ -252,12 +256,12 @@ gla_scan_kernel(const __grid_constant__ CUtensorMap tmV, const GlaArgs a) {
       if (v < a.vdim) {
         float* dst = a.out + (size_t)t0 * a.ld_out + (size_t)h * a.vdim + v;
 #pragma unroll
-        for (int i = 0; i < kGlB; ++i) if (i < n) dst[(size_t)i * a.ld_out] = o[i];
+        for (int i = 0; i < kGlB; ++i) if (i < n) dst[(size_t)i * a.ld_out] = o[i] + o[kGlB + i];
       }
     }
-  } else {
+  } else if (warp >= 8) {
     // ---------------------------------------------------------------- state: lane = value column, 64 channels per warp
-    const int q = warp & 3, g = (warp - 6) >> 2, v = e0 + q * 32 + lane;
+    const int q = warp & 3, g = (warp - 8) >> 2, v = e0 + q * 32 + lane;
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     const bool live = v < a.vdim;
     float* st = a.state + ((size_t)(run ? slot : 0) * a.heads + h) * a.dim * a.vdim + (live ? v : 0);
@@ -305,7 +309,7 @@ gla_scan_kernel(const __grid_constant__ CUtensorMap tmV, const GlaArgs a) {
       __syncwarp();
       if (lane == 0) { mbar_arrive(ds_free); mbar_arrive(&empty[sg]); }
       if (b + 1 < n_blk) {
-        // the buffer held S in front of block b - 1: its output is done
+        // the buffer held S in front of block b - 1: its output is done (so a phase of s_ready cannot end unseen either)
         if (b >= 1 && !warp_wait(&o_full[(b - 1) & 1], (uint32_t)((b - 1) >> 1) & 1, abort_flag, a.status, 932, b)) { ok = false; break; }
         tc_fence_after();
         publish(b + 1);

@@ -20,7 +20,7 @@
 
 namespace gb {
 
-constexpr int kLdThreads = 192;
+constexpr int kLdThreads = 224;         // TMA warp, S warp, O warp, 4 softmax warps
 constexpr int kLdB = 64;                  // positions per block
 constexpr int kLdBox = 8192;              // 64 positions x 64 columns
 constexpr int kLdMaxPairs = 24;           // pairs of boxes in shared memory
@@ -62,8 +62,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   uint64_t* t_empty = t_full + kLdMaxPairs;
   uint32_t* tmem_slot = (uint32_t*)(t_empty + kLdMaxPairs);
   volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
-  float* red_max = (float*)(((uintptr_t)(tmem_slot + 2) + 15) & ~(uintptr_t)15);       // [2 (block parity)][2 warps][NH]
-  float* red_sum = red_max + 4 * NH;                                                   // [2][NH]
+  float* red_max = (float*)(((uintptr_t)(tmem_slot + 2) + 15) & ~(uintptr_t)15);       // [2 warps][NH]
+  float* red_sum = red_max + 2 * NH;                                                   // [2][NH]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
@@ -134,21 +134,21 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       }
     }
   } else if (warp == 1) {
+    // The products are issued by two threads: one thread needs longer to issue a block's 52 MMAs than its data take to arrive
     if (lane == 0 && n_blk > 0) {
       // S: the operand's rows 64 .. 127 are whatever lies behind the box; nobody reads their scores
       constexpr uint32_t id_s = make_idesc(128, NH, 1, 1, 0, 0);
-      constexpr uint32_t id_o = make_idesc(128, NH, 1, 1, 1, 0);      // A (latents by position) is MN-major
-      const uint64_t d_q = make_sdesc_sw128(smem_u32(sQ)), d_p = make_sdesc_sw128(smem_u32(sP)), d_c = make_sdesc_sw128(smem_u32(sC));
-      const uint64_t d_v = make_sdesc_sw128_mn(smem_u32(sC), kLdBox);
+      const uint64_t d_q = make_sdesc_sw128(smem_u32(sQ)), d_c = make_sdesc_sw128(smem_u32(sC));
       const int k_steps = (a.width + 15) >> 4;
       bool ok = mbar_wait(q_full, 0, abort_flag, a.status, 810);
-      int st_s = 0, st_o = 0; uint32_t ph_s = 0;
-      auto issue_s = [&](int j) -> bool {
+      int st = 0; uint32_t ph = 0;
+      for (int j = 0; j < n_blk && ok; ++j) {
+        // the scores of block j - 2 have been read
+        if (j >= 2 && !mbar_wait(&p_ready[j & 1], (uint32_t)((j - 2) >> 1) & 1, abort_flag, a.status, 813, j)) break;
         const uint32_t d = tmem_s + (j & 1) * NH;
-        uint64_t dc = sdesc_at(d_c, st_s * a.boxes * kLdBox), dq = d_q;
+        uint64_t dc = sdesc_at(d_c, st * a.boxes * kLdBox), dq = d_q;
         for (int b = 0; b < pairs; ++b) {
-          uint64_t* bar = &t_full[st_s * pairs + b];
-          if (!mbar_wait(bar, ph_s, abort_flag, a.status, 811, j)) return false;
+          if (!mbar_wait(&t_full[st * pairs + b], ph, abort_flag, a.status, 811, j)) { ok = false; break; }
           tc_fence_after();
           const uint32_t acc = b > 0 ? 1u : 0u;
           if (b * 8 + 8 <= k_steps) {
@@ -159,30 +159,34 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
             for (int x = 0; b * 8 + x < k_steps; ++x)
               mma_f16_ss(d, sdesc_at(dc, (x >> 2) * kLdBox + (x & 3) * 32), sdesc_at(dq, (x >> 2) * kQ + (x & 3) * 32), id_s, x > 0 ? 1u : acc);
           }
-          if (b >= m_tiles) tc_commit(&t_empty[st_s * pairs + b]);      // no values in these boxes
+          if (b >= m_tiles) tc_commit(&t_empty[st * pairs + b]);        // no values in these boxes
           dc = sdesc_at(dc, 2 * kLdBox); dq = sdesc_at(dq, 2 * kQ);
         }
+        if (!ok) break;
         tc_commit(&s_full[j & 1]);
-        if (++st_s == a.stages) { st_s = 0; ph_s ^= 1; }
-        return true;
-      };
-      if (ok) ok = issue_s(0);
-      for (int j = 0; j < n_blk && ok; ++j) {
-        if (a.stages > 1 && j + 1 < n_blk && !issue_s(j + 1)) { ok = false; break; }
-        if (!mbar_wait(&p_ready[j & 1], (uint32_t)(j >> 1) & 1, abort_flag, a.status, 812, j)) { ok = false; break; }
+        if (++st == a.stages) { st = 0; ph ^= 1; }
+      }
+    }
+  } else if (warp == 2) {
+    if (lane == 0 && n_blk > 0) {
+      constexpr uint32_t id_o = make_idesc(128, NH, 1, 1, 1, 0);      // A (latents by position) is MN-major
+      const uint64_t d_p = make_sdesc_sw128(smem_u32(sP)), d_v = make_sdesc_sw128_mn(smem_u32(sC), kLdBox);
+      int st = 0;
+      for (int j = 0; j < n_blk; ++j) {
+        // P follows from S, so the block's boxes have landed and S has read them
+        if (!mbar_wait(&p_ready[j & 1], (uint32_t)(j >> 1) & 1, abort_flag, a.status, 812, j)) break;
         tc_fence_after();
-        uint64_t dv = sdesc_at(d_v, st_o * a.boxes * kLdBox);
+        uint64_t dv = sdesc_at(d_v, st * a.boxes * kLdBox);
         const uint64_t dp = sdesc_at(d_p, (j & 1) * kQ);
         const uint32_t acc = j > 0 ? 1u : 0u;
         for (int m = 0; m < m_tiles; ++m) {
 #pragma unroll
           for (int ks = 0; ks < 4; ++ks) mma_f16_ss(tmem_o + m * NH, sdesc_at(dv, ks * 2048), sdesc_at(dp, ks * 32), id_o, ks > 0 ? 1u : acc);
-          tc_commit(&t_empty[st_o * pairs + m]);
+          tc_commit(&t_empty[st * pairs + m]);
           dv = sdesc_at(dv, 2 * kLdBox);
         }
         tc_commit(&o_ready[j & 1]);
-        if (++st_o == a.stages) st_o = 0;
-        if (a.stages == 1 && j + 1 < n_blk && !issue_s(j + 1)) { ok = false; break; }
+        if (++st == a.stages) st = 0;
       }
     }
   } else {
@@ -198,38 +202,39 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const bool got = warp_wait(&s_full[j & 1], (uint32_t)(j >> 1) & 1, abort_flag, a.status, 820, j);
       tc_fence_after();
       float sv[NH];
-      float* rm = red_max + (j & 1) * 2 * NH;
+      bool grow = false;
       if (q < 2) {
         tmem_ld_heads<NH>(tmem_s + (j & 1) * NH + lane_off, reinterpret_cast<uint32_t*>(sv));
         tc_wait_ld();
         const bool live = (blk0 + j) * kLdB + r < kv;
 #pragma unroll
-        for (int h = 0; h < NH; ++h) if (!live || h >= n_heads) sv[h] = -INFINITY;
-#pragma unroll
-        for (int x = 0; x < NH; x += 16) {
-          const float v = warp_reduce16_max(sv + x, lane);
-          if ((lane & 1) == 0) rm[q * NH + x + (lane >> 1)] = v;
+        for (int h = 0; h < NH; ++h) {
+          if (!live || h >= n_heads) sv[h] = -INFINITY;
+          grow |= sv[h] > m[h] + kTau;                   // also the first finite score
         }
       }
-      if (!bar128_and(got && !fail_o)) { ok = false; break; }       // all 128 threads leave together
-      bool need = false;
-#pragma unroll
-      for (int h = 0; h < NH; h += 4) {
-        const float4 x = *reinterpret_cast<const float4*>(rm + h), y = *reinterpret_cast<const float4*>(rm + NH + h);
-        need |= fmaxf(x.x, y.x) > m[h] + kTau || fmaxf(x.y, y.y) > m[h + 1] + kTau || fmaxf(x.z, y.z) > m[h + 2] + kTau || fmaxf(x.w, y.w) > m[h + 3] + kTau;
-      }
       bool got_o = true;
-      if (need) {                                        // the same for all 128 threads; also the first finite maximum
+      if (!bar128_and(got && !fail_o && !grow)) {        // rare: some score has outgrown its reference, or a wait ran out
+        if (!bar128_and(got && !fail_o)) { ok = false; break; }         // all 128 threads leave together
+        if (q < 2) {
+#pragma unroll
+          for (int x = 0; x < NH; x += 16) {
+            const float v = warp_reduce16_max(sv + x, lane);
+            if ((lane & 1) == 0) red_max[q * NH + x + (lane >> 1)] = v;
+          }
+        }
+        bar128_and(true);
         // every earlier product is in O before it is rescaled
         if (j > 0) got_o = warp_wait(&o_ready[(j - 1) & 1], (uint32_t)((j - 1) >> 1) & 1, abort_flag, a.status, 821, j);
         tc_fence_after();
         float al[NH];
 #pragma unroll
         for (int h = 0; h < NH; ++h) {
-          const float mn = fmaxf(m[h], fmaxf(rm[h], rm[NH + h]));
+          const float mn = fmaxf(m[h], fmaxf(red_max[h], red_max[NH + h]));
           al[h] = mn == -INFINITY ? 1.0f : fast_exp2(m[h] - mn);
           m[h] = mn; l[h] *= al[h];
         }
+        bar128_and(true);                                // red_max may be written again
         if (j > 0 && got_o)
           for (int t = 0; t < m_tiles; ++t) {
             uint32_t o[NH];
