@@ -4,10 +4,10 @@
 // token, a tile of NH heads and a range of its keys.  As in the decode kernel of flash_attn.cu the key POSITIONS are the MMA's M dimension:
 //   S^T[positions x NH]   = C_j[positions x width] Q^T       (A = rows as they are cached, K-major; B = the heads' queries)
 //   O^T[128 columns x NH] += C_j^T[128 x positions] P_j      (A = the same rows, MN-major, one product per 128 latent columns; B = P^T in shared memory)
-// so that every cached byte is fetched once for both products.  A block of 64 positions is a row of boxes of 64 columns (8 KB), each with its own
-// barriers: S starts with the first box that lands, and O's products free the boxes pair by pair.  Two blocks of 512 + 64 columns fit beside the
-// queries of 32 heads (with 128 positions it would be one, and loads would stop while a block is computed: measured 2.4 times slower), so S of a
-// block has only half of an MMA's rows.
+// so that every cached byte is fetched once for both products.  A block of 128 positions is a row of boxes of 64 columns (16 KB), a pair of boxes
+// sharing a barrier: S starts with the first pair that lands, and O's products free the pairs one by one for the next block.  With 512 + 64 columns
+// one block fills shared memory.  Two half-sized blocks in turn were measured 1.2 to 1.5 times slower: what bounds the loop is the chain load -> S ->
+// softmax -> O -> load, whose length hardly depends on the block's size.
 //
 // latent_prefill_kernel (expanded form): keys [expanded part | rotated part shared by the heads] and values of one head.  A CTA owns one head and
 // two tiles of 128 tokens, which take turns: while one tile's softmax runs, the tensor core works for the other.  K is double-buffered.
@@ -21,8 +21,8 @@
 namespace gb {
 
 constexpr int kLdThreads = 224;         // TMA warp, S warp, O warp, 4 softmax warps
-constexpr int kLdB = 64;                  // positions per block
-constexpr int kLdBox = 8192;              // 64 positions x 64 columns
+constexpr int kLdB = 128;                 // positions per block
+constexpr int kLdBox = 16384;             // 128 positions x 64 columns
 constexpr int kLdMaxPairs = 24;           // pairs of boxes in shared memory
 
 struct LatentDecodeArgs {
@@ -48,12 +48,12 @@ __global__ void __launch_bounds__(kLdThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmC, const LatentDecodeArgs a) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);
-  constexpr int kQ = NH * 128;            // bytes of a 64-column box of queries, and of P^T
+  constexpr int kQ = NH * 128;            // bytes of a 64-column box of queries, and of half of P^T
   const int pairs = (a.boxes + 1) >> 1;
   uint8_t* sC = smem;
   uint8_t* sP = sC + a.boxes * a.stages * kLdBox;      // two buffers
-  uint8_t* sQ = sP + 2 * kQ;              // (behind the last box at least 8 KB are queries and P: an operand of 128 rows may start in it)
-  uint64_t* bars = (uint64_t*)(sQ + max(a.boxes, 2) * kQ);
+  uint8_t* sQ = sP + 4 * kQ;              // (behind the last box at least 16 KB are P and queries: where the number of boxes is odd, O's operand goes on there)
+  uint64_t* bars = (uint64_t*)(sQ + max(a.boxes, 4) * kQ);
   uint64_t* q_full = bars;
   uint64_t* s_full = bars + 1;            // 2, by block parity
   uint64_t* p_ready = bars + 3;           // 2, 128 arrivals each (two for the reason given in flash_decode_kernel)
@@ -62,8 +62,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   uint64_t* t_empty = t_full + kLdMaxPairs;
   uint32_t* tmem_slot = (uint32_t*)(t_empty + kLdMaxPairs);
   volatile int* abort_flag = (volatile int*)(tmem_slot + 1);
-  float* red_max = (float*)(((uintptr_t)(tmem_slot + 2) + 15) & ~(uintptr_t)15);       // [2 warps][NH]
-  float* red_sum = red_max + 2 * NH;                                                   // [2][NH]
+  float* red_max = (float*)(((uintptr_t)(tmem_slot + 2) + 15) & ~(uintptr_t)15);       // [4 warps][NH]
+  float* red_sum = red_max + 4 * NH;                                                   // [4][NH]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   if (threadIdx.x == 0) {
@@ -99,19 +99,25 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       auto cache_row = [&](int pos) { return (bt[min(pos >> shift, last_page)] << shift) + (pos & (a.page_size - 1)); };
       bool ok = true;
       int st = 0; uint32_t ph = 1;
-      if (a.page_size >= kLdB) {                 // a block lies in one page; its row is looked up a block ahead
-        int next = cache_row(blk0 * kLdB);
+      if (2 * a.page_size >= kLdB) {             // a block lies in one or two pages; their rows are looked up a block ahead
+        const bool halves = a.page_size < kLdB;
+        const int half = kLdBox / 2;
+        int next0 = cache_row(blk0 * kLdB), next1 = halves ? cache_row(blk0 * kLdB + kLdB / 2) : 0;
         for (int j = 0; j < n_blk && ok; ++j) {
-          const int row = next;
-          if (j + 1 < n_blk) next = cache_row((blk0 + j + 1) * kLdB);
+          const int row0 = next0, row1 = next1;
+          if (j + 1 < n_blk) { next0 = cache_row((blk0 + j + 1) * kLdB); if (halves) next1 = cache_row((blk0 + j + 1) * kLdB + kLdB / 2); }
           uint8_t* dst = sC + st * a.boxes * kLdBox;
           for (int b = 0; b < a.boxes; b += 2, dst += 2 * kLdBox) {
             const int s = st * pairs + (b >> 1);
             if (!mbar_wait(&t_empty[s], ph, abort_flag, a.status, 800, j)) { ok = false; break; }
             const bool two = b + 1 < a.boxes;
             mbar_expect_tx(&t_full[s], two ? 2 * kLdBox : kLdBox);
-            tma_load_2d(dst, &tmC, &t_full[s], b * 64, row);
-            if (two) tma_load_2d(dst + kLdBox, &tmC, &t_full[s], b * 64 + 64, row);
+            tma_load_2d(dst, &tmC, &t_full[s], b * 64, row0);
+            if (two) tma_load_2d(dst + kLdBox, &tmC, &t_full[s], b * 64 + 64, row0);
+            if (halves) {
+              tma_load_2d(dst + half, &tmC, &t_full[s], b * 64, row1);
+              if (two) tma_load_2d(dst + kLdBox + half, &tmC, &t_full[s], b * 64 + 64, row1);
+            }
           }
           if (++st == a.stages) { st = 0; ph ^= 1; }
         }
@@ -134,9 +140,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       }
     }
   } else if (warp == 1) {
-    // The products are issued by two threads: one thread needs longer to issue a block's 52 MMAs than its data take to arrive
+    // the products are issued by two threads: one needs longer to issue a block's MMAs than its data take to arrive
     if (lane == 0 && n_blk > 0) {
-      // S: the operand's rows 64 .. 127 are whatever lies behind the box; nobody reads their scores
       constexpr uint32_t id_s = make_idesc(128, NH, 1, 1, 0, 0);
       const uint64_t d_q = make_sdesc_sw128(smem_u32(sQ)), d_c = make_sdesc_sw128(smem_u32(sC));
       const int k_steps = (a.width + 15) >> 4;
@@ -177,11 +182,11 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         if (!mbar_wait(&p_ready[j & 1], (uint32_t)(j >> 1) & 1, abort_flag, a.status, 812, j)) break;
         tc_fence_after();
         uint64_t dv = sdesc_at(d_v, st * a.boxes * kLdBox);
-        const uint64_t dp = sdesc_at(d_p, (j & 1) * kQ);
+        const uint64_t dp = sdesc_at(d_p, (j & 1) * 2 * kQ);
         const uint32_t acc = j > 0 ? 1u : 0u;
         for (int m = 0; m < m_tiles; ++m) {
 #pragma unroll
-          for (int ks = 0; ks < 4; ++ks) mma_f16_ss(tmem_o + m * NH, sdesc_at(dv, ks * 2048), sdesc_at(dp, ks * 32), id_o, ks > 0 ? 1u : acc);
+          for (int ks = 0; ks < 8; ++ks) mma_f16_ss(tmem_o + m * NH, sdesc_at(dv, ks * 2048), sdesc_at(dp, (ks >> 2) * kQ + (ks & 3) * 32), id_o, ks > 0 ? 1u : acc);
           tc_commit(&t_empty[st * pairs + m]);
           dv = sdesc_at(dv, 2 * kLdBox);
         }
@@ -190,7 +195,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       }
     }
   } else {
-    // thread r: position r of the block (r < 64), column r of each tile of O
+    // thread r: position r of the block, column r of each tile of O
     const int q = warp & 3, r = q * 32 + lane;
     const uint32_t lane_off = (uint32_t)(q * 32) << 16;
     float m[NH], l[NH];                                  // reference maximum; this thread's share of the sums
@@ -203,25 +208,21 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       tc_fence_after();
       float sv[NH];
       bool grow = false;
-      if (q < 2) {
-        tmem_ld_heads<NH>(tmem_s + (j & 1) * NH + lane_off, reinterpret_cast<uint32_t*>(sv));
-        tc_wait_ld();
-        const bool live = (blk0 + j) * kLdB + r < kv;
+      tmem_ld_heads<NH>(tmem_s + (j & 1) * NH + lane_off, reinterpret_cast<uint32_t*>(sv));
+      tc_wait_ld();
+      const bool live = (blk0 + j) * kLdB + r < kv;
 #pragma unroll
-        for (int h = 0; h < NH; ++h) {
-          if (!live || h >= n_heads) sv[h] = -INFINITY;
-          grow |= sv[h] > m[h] + kTau;                   // also the first finite score
-        }
+      for (int h = 0; h < NH; ++h) {
+        if (!live || h >= n_heads) sv[h] = -INFINITY;
+        grow |= sv[h] > m[h] + kTau;                     // also the first finite score
       }
       bool got_o = true;
       if (!bar128_and(got && !fail_o && !grow)) {        // rare: some score has outgrown its reference, or a wait ran out
         if (!bar128_and(got && !fail_o)) { ok = false; break; }         // all 128 threads leave together
-        if (q < 2) {
 #pragma unroll
-          for (int x = 0; x < NH; x += 16) {
-            const float v = warp_reduce16_max(sv + x, lane);
-            if ((lane & 1) == 0) red_max[q * NH + x + (lane >> 1)] = v;
-          }
+        for (int x = 0; x < NH; x += 16) {
+          const float v = warp_reduce16_max(sv + x, lane);
+          if ((lane & 1) == 0) red_max[q * NH + x + (lane >> 1)] = v;
         }
         bar128_and(true);
         // every earlier product is in O before it is rescaled
@@ -230,7 +231,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         float al[NH];
 #pragma unroll
         for (int h = 0; h < NH; ++h) {
-          const float mn = fmaxf(m[h], fmaxf(red_max[h], red_max[NH + h]));
+          const float mn = fmaxf(m[h], fmaxf(fmaxf(red_max[h], red_max[NH + h]), fmaxf(red_max[2 * NH + h], red_max[3 * NH + h])));
           al[h] = mn == -INFINITY ? 1.0f : fast_exp2(m[h] - mn);
           m[h] = mn; l[h] *= al[h];
         }
@@ -249,35 +250,31 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       // the P buffer of this parity was read by the product of block j - 2
       if (got_o && j >= 2) got_o = warp_wait(&o_ready[j & 1], (uint32_t)((j - 2) >> 1) & 1, abort_flag, a.status, 822, j);
       if (got_o) {
-        if (q < 2) {
-          uint8_t* pb = sP + (j & 1) * kQ + (r & 7) * 2;
-          const int chunk = r >> 3;
+        uint8_t* pb = sP + ((j & 1) * 2 + (r >> 6)) * kQ + (r & 7) * 2;
+        const int chunk = (r & 63) >> 3;
 #pragma unroll
-          for (int h = 0; h < NH; ++h) {
-            const float p = h < n_heads ? fast_exp2(sv[h] - m[h]) : 0.f;
-            l[h] += p;
-            *reinterpret_cast<__nv_bfloat16*>(pb + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16(p);
-          }
-          fence_proxy_async_smem();
+        for (int h = 0; h < NH; ++h) {
+          const float p = h < n_heads ? fast_exp2(sv[h] - m[h]) : 0.f;
+          l[h] += p;
+          *reinterpret_cast<__nv_bfloat16*>(pb + h * 128 + ((chunk ^ (h & 7)) << 4)) = __float2bfloat16(p);
         }
+        fence_proxy_async_smem();
         tc_fence_before();
         mbar_arrive(&p_ready[j & 1]);
       }
       fail_o |= !got_o;
     }
     if (ok && !fail_o && n_blk > 0) ok = warp_wait(&o_ready[(n_blk - 1) & 1], (uint32_t)((n_blk - 1) >> 1) & 1, abort_flag, a.status, 823, 0);
-    if (q < 2) {
 #pragma unroll
-      for (int x = 0; x < NH; x += 16) {
-        const float v = warp_reduce16_sum(l + x, lane);
-        if ((lane & 1) == 0) red_sum[q * NH + x + (lane >> 1)] = v;
-      }
+    for (int x = 0; x < NH; x += 16) {
+      const float v = warp_reduce16_sum(l + x, lane);
+      if ((lane & 1) == 0) red_sum[q * NH + x + (lane >> 1)] = v;
     }
     ok = bar128_and(ok && !fail_o);
     if (ok) {
       tc_fence_after();
 #pragma unroll
-      for (int h = 0; h < NH; ++h) l[h] = red_sum[h] + red_sum[NH + h];
+      for (int h = 0; h < NH; ++h) l[h] = red_sum[h] + red_sum[NH + h] + red_sum[2 * NH + h] + red_sum[3 * NH + h];
       float inv[NH];
 #pragma unroll
       for (int h = 0; h < NH; ++h) {
@@ -321,27 +318,35 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   if (warp == 1) { tc_fence_after(); tmem_dealloc(tmem_s, 256); }
 }
 
-// Merge of the key ranges, and the sink: out[h][tok] = sum_s 2^(lse_s) O_s / (sum_s 2^(lse_s) + 2^(sink)).  One CTA per (token, head).
+// Merge of the key ranges, and the sink: out[h][tok] = sum_s 2^(lse_s) O_s / (sum_s 2^(lse_s) + 2^(sink)).  One CTA per (token, head) and 128 columns.
+constexpr int kLdMaxSplits = 64;
 __global__ void __launch_bounds__(128)
 latent_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_lse, const float* __restrict__ sink, __nv_bfloat16* __restrict__ out, int splits,
                       int tokens, int heads, int rank, int m_rows, int ld_out) {
   pdl_wait();
   pdl_trigger();
-  const int h = blockIdx.x % heads, tok = blockIdx.x / heads;
+  __shared__ float w[kLdMaxSplits];
+  const int h = blockIdx.x % heads, tok = blockIdx.x / heads, c = blockIdx.y * 128 + threadIdx.x;
   const size_t row = (size_t)tok * heads + h, rows = (size_t)tokens * heads;
-  float mx = sink != nullptr ? sink[h] : -INFINITY;
-  for (int s = 0; s < splits; ++s) mx = fmaxf(mx, part_lse[s * rows + row]);
-  float den = sink != nullptr ? exp2f(sink[h] - mx) : 0.f;
-  for (int s = 0; s < splits; ++s) den += exp2f(part_lse[s * rows + row] - mx);
-  const float inv = 1.0f / den;
-  for (int c = threadIdx.x; c < rank; c += 128) {
-    float v = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float ls = part_lse[s * rows + row];
-      if (ls > -INFINITY) v = fmaf(exp2f(ls - mx), part_o[(s * rows + row) * rank + c], v);
-    }
-    out[((size_t)h * m_rows + tok) * ld_out + c] = __float2bfloat16(v * inv);
+  if (threadIdx.x < 32) {
+    const int lane = threadIdx.x;
+    const float sk = sink != nullptr ? sink[h] : -INFINITY;
+    float l[kLdMaxSplits / 32], mx = sk, den = 0.f;
+#pragma unroll
+    for (int i = 0; i < kLdMaxSplits / 32; ++i) { const int s = lane + 32 * i; l[i] = s < splits ? part_lse[s * rows + row] : -INFINITY; mx = fmaxf(mx, l[i]); }
+    mx = warp_max(mx);
+#pragma unroll
+    for (int i = 0; i < kLdMaxSplits / 32; ++i) { l[i] = l[i] > -INFINITY ? exp2f(l[i] - mx) : 0.f; den += l[i]; }
+    den = warp_sum(den) + (sk > -INFINITY ? exp2f(sk - mx) : 0.f);
+#pragma unroll
+    for (int i = 0; i < kLdMaxSplits / 32; ++i) w[lane + 32 * i] = den > 0.f ? l[i] / den : 0.f;
   }
+  __syncthreads();
+  if (c >= rank) return;
+  float v = 0.f;
+#pragma unroll 8
+  for (int s = 0; s < splits; ++s) v = fmaf(w[s], part_o[(s * rows + row) * rank + c], v);
+  out[((size_t)h * m_rows + tok) * ld_out + c] = __float2bfloat16(v);
 }
 
 // ------------------------------------------------------------------------------------------ expanded form
@@ -579,7 +584,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
 
 // Shared memory of the decode kernel with `boxes` boxes per block and `stages` blocks.
 static int latent_decode_smem(int boxes, int stages, int nh) {
-  return boxes * stages * kLdBox + ((boxes > 2 ? boxes : 2) + 2) * nh * 128 + (7 + 2 * kLdMaxPairs) * 8 + 32 + 6 * nh * 4 + 1024;
+  return boxes * stages * kLdBox + ((boxes > 4 ? boxes : 4) + 4) * nh * 128 + (7 + 2 * kLdMaxPairs) * 8 + 32 + 8 * nh * 4 + 1024;
 }
 
 struct LatentDecodeShape { int nh, boxes, stages; };
@@ -610,7 +615,7 @@ GB_API int gb_latent_decode(const void* q, const void* cache, int ld_c, long num
   if (tokens <= 0) return 0;
   if (gb_latent_decode_heads(heads, width, rank, page_size) == 0) return fail("latent_decode: unsupported sizes%s");
   if (ld_c % 8 || ld_c < width || ld_out < rank || m_rows < tokens || ((uintptr_t)q & 15) || ((uintptr_t)cache & 15)) return fail("latent_decode: bad rows%s");
-  if (splits < 1 || (splits > 1 && (part_o == nullptr || part_lse == nullptr))) return fail("latent_decode: bad splits%s");
+  if (splits < 1 || splits > kLdMaxSplits || (splits > 1 && (part_o == nullptr || part_lse == nullptr))) return fail("latent_decode: bad splits%s");
   if ((tok_seq == nullptr) != (tok_kv == nullptr)) return fail("latent_decode: tok_seq and tok_kv come together%s");
   const LatentDecodeShape sh = latent_decode_shape(heads, width, rank);
   CUtensorMap tmQ, tmC;
@@ -634,7 +639,7 @@ GB_API int gb_latent_decode(const void* q, const void* cache, int ld_c, long num
   else launch_k(latent_decode_kernel<32>, grid, kLdThreads, smem, stream, tmQ, tmC, a);
   GB_CUDA_OK(cudaGetLastError());
   if (splits > 1) {
-    launch_k(latent_combine_kernel, (unsigned)((long)tokens * heads), 128, 0, stream, (const float*)part_o, (const float*)part_lse, sink, (__nv_bfloat16*)out, splits, tokens,
+    launch_k(latent_combine_kernel, dim3((unsigned)((long)tokens * heads), (unsigned)((rank + 127) / 128)), 128, 0, stream, (const float*)part_o, (const float*)part_lse, sink, (__nv_bfloat16*)out, splits, tokens,
              heads, rank, m_rows, ld_out);
     GB_CUDA_OK(cudaGetLastError());
   }

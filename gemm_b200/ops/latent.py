@@ -72,7 +72,7 @@ class LatentPlan:
 def pick_latent_splits(n: int, max_kv: int, head_tiles: int, sm_count: int = 148) -> int:
     """Key ranges per token: enough work items to fill the GPU, at least two blocks of 128 keys each."""
     blocks = max(1, (max_kv + 127) // 128)
-    return max(1, min(sm_count // max(1, n * head_tiles), blocks // 2 if blocks >= 2 else 1, 32))
+    return max(1, min(sm_count // max(1, n * head_tiles), blocks // 2 if blocks >= 2 else 1, 64))
 
 
 def make_plan(q_lens: Sequence[int], kv_lens: Optional[Sequence[int]], max_kv: int, device, decode: bool, expand: bool, heads: Sequence[int]) -> LatentPlan:
