@@ -92,6 +92,7 @@ __device__ __forceinline__ void stage_slice(uint8_t* dst, uint32_t atom_bytes, c
   }
 }
 
+template <bool GROUPS>                 // routing limited to the best expert groups
 __global__ void __launch_bounds__(kPrepThreads, 1)
 moe_prep_kernel(const MoePrepArgs a) {
   static_assert(kPrepTok % (kPrepThreads / 32) == 0, "the gather phase gives every warp the same number of items");
@@ -189,7 +190,7 @@ moe_prep_kernel(const MoePrepArgs a) {
     for (int tl = warp; tl < TPC; tl += kPrepThreads / 32) {
       const int t = c * TPC + tl;
       if (t >= a.n_tok || !ok) continue;
-      const int id = route_row<4>(lg + tl * kPrepExp, a.bias, a.ids + (size_t)t * a.topk, a.weights + (size_t)t * a.topk, lane, a.n_exp, a.topk,
+      const int id = route_row<4, GROUPS>(lg + tl * kPrepExp, a.bias, a.ids + (size_t)t * a.topk, a.weights + (size_t)t * a.topk, lane, a.n_exp, a.topk,
                                   a.mode, a.renorm, a.routed_scale, a.groups, a.keep, a.id_shift, a.n_local);
       if (lane < a.topk)
         for (int d = 0; d < C; ++d) st_cluster_b32(mapa_u32(ids0 + (uint32_t)((t * kPrepIdsLd + lane) * 4), (uint32_t)d), (uint32_t)id);
@@ -338,12 +339,12 @@ GB_API int gb_moe_prep(const void* h, int ld_h, int n_tok, int hidden, const voi
   const int tpc = kPrepTok / C;
   const size_t smem = 1024 + (size_t)kPrepExp * kPrepKC * 2 + (size_t)kPrepTok * kPrepKC * 2 + (size_t)kPrepTok * kPrepExp * 4 +
                       (size_t)tpc * kPrepExp * 4 + (size_t)kPrepTok * kPrepIdsLd * 4 + kPrepExp * 8 + kPrepExp * 4 + 64 + 64;
-  auto kern = moe_prep_kernel;
-  static bool attr_set = false;
-  if (!attr_set) {
+  auto kern = keep < groups ? moe_prep_kernel<true> : moe_prep_kernel<false>;
+  static bool attr_set[2] = {false, false};
+  if (!attr_set[keep < groups]) {
     GB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
     GB_CUDA_OK(cudaFuncSetAttribute(kern, cudaFuncAttributeNonPortableClusterSizeAllowed, 1));
-    attr_set = true;
+    attr_set[keep < groups] = true;
   }
   GB_CUDA_OK(launch_k_cluster(kern, dim3((unsigned)C), kPrepThreads, smem, stream, (unsigned)C, a));
   GB_CUDA_OK(cudaGetLastError());

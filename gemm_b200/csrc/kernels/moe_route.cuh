@@ -13,9 +13,9 @@ constexpr int kMaxTopK = 16;
 constexpr int kMaxExpertGroups = 128;
 
 // Routing of token `w` by one warp (E <= 512): lane j < k ends with the j-th pick.  Returns the (possibly local) expert id.
-// groups > 1 (at most kMaxExpertGroups, dividing the experts): a group of neighbouring experts scores the sum of its two best, and only
+// GROUPS (an instance of its own: the code costs the others registers): `groups` (at most kMaxExpertGroups, dividing the experts): a group of neighbouring experts scores the sum of its two best, and only
 // experts of the `keep` best groups can be picked (ties: lower group).  renorm: 1 = weights over max(sum, 1e-20), 2 = over sum + 1e-20.
-template <int MAXV>
+template <int MAXV, bool GROUPS>
 __device__ __forceinline__ int route_row(const float* row, const float* __restrict__ bias, int* __restrict__ ids_row,
                                          float* __restrict__ weights_row, int lane, int n_exp, int k, int mode, int renorm,
                                          float routed_scale, int groups, int keep, int id_shift, int n_local) {
@@ -46,7 +46,7 @@ __device__ __forceinline__ int route_row(const float* row, const float* __restri
       sel[i] = (e < n_exp) ? p[i] + (bias != nullptr ? bias[e] : 0.f) : -FLT_MAX;
     }
   }
-  if (groups > 1 && keep < groups) {
+  if constexpr (GROUPS) {
     const int size = n_exp / groups;
     float gs[kMaxExpertGroups / 32];
     unsigned kept[kMaxExpertGroups / 32];
