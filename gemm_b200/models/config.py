@@ -350,7 +350,7 @@ def _famepel(pattern: str, hidden: int, vocab: int, moe: MoeSpec, hgrn, mamba, l
             own = i if c == "L" else own
             specs.append(LayerSpec("latent", heads, d, v, n_kv_heads=1, scale=(d + r) ** -0.5, kv_rank=kvr, q_rank=qr, rot_dim=r, rotary=rotary, sink=True,
                                    kv_from=own if c == "S" else -1, moe=moe))
-    return ModelConfig(arch="famepel", layer_specs=specs, hidden=hidden, n_heads=latent[0], n_kv_heads=1, head_dim=latent[1], ffn=moe.ffn, vocab=vocab,
+    return ModelConfig(arch="famepel", layer_specs=specs, hidden=hidden, n_heads=latent[0], n_kv_heads=latent[0], head_dim=latent[1], ffn=moe.ffn, vocab=vocab,
                        rms_eps=1e-5, norm_kind="dyt", post_norm=True, embed_scale=hidden ** 0.5, qk_norm=False)
 
 

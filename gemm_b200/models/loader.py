@@ -620,7 +620,7 @@ def _famepel_config(c: dict) -> ModelConfig:
     """config.json of Famepel: HGRN2, Mamba-2 and latent-attention mixers, grouped mixtures of experts, Dynamic-Tanh norms around every sublayer."""
     specs = [_famepel_layer(li, e, c["layers"]) for li, e in enumerate(c["layers"])]
     att = next((s for s in specs if s.mixer == "latent"), specs[0])
-    return ModelConfig(arch=LAYERED_ARCHS[c["architecture"]], layer_specs=specs, hidden=int(c["width"]), vocab=int(c["vocab"]), n_heads=att.n_heads, n_kv_heads=1,
+    return ModelConfig(arch=LAYERED_ARCHS[c["architecture"]], layer_specs=specs, hidden=int(c["width"]), vocab=int(c["vocab"]), n_heads=att.n_heads, n_kv_heads=att.n_heads,
                        head_dim=att.head_dim, ffn=max((s.moe.ffn for s in specs if s.moe), default=0), rms_eps=float(c["norm"]["eps"]), qk_norm=False,
                        norm_kind="dyt", post_norm=True, embed_scale=float(c["embedding"]["scale"]))
 

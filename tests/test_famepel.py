@@ -205,6 +205,25 @@ def test_greedy_generation_through_the_scheduler(folder, name, fmt, device):
 
 
 @pytest.mark.parametrize("device", DEVICES)
+def test_many_heads(tmp_path, device):
+    """More heads than an attention tile has rows, a latent too wide for the decode kernel, one expert group."""
+    name = "heads"
+    C.CASES[name] = (64, 50, 1.5, 1e-5, [C.latent(150, 8, 4, 8, 40, 24, 0.3, 1e3, C.moe(3, 2, 16, 1.1)), C.hgrn2(130, 8, 8, None),
+                                         C.latent(2, 8, 4, 16, 1000, 24, 0.3, 1e3, None), C.mamba2(132, 8, 8, 66, 2, 3, None)])
+    try:
+        model = C.make_model(name)
+    finally:
+        del C.CASES[name]
+    C.save_model(model, str(tmp_path))
+    toks = L.tokens(model, 90, 1)
+    ref = O.forward(model, toks)
+    for fmt in FORMATS:
+        llm = LLM(loader.load_safetensors(str(tmp_path), fmt, device), None, max_running=4, num_pages=4, page_size=PAGE)
+        assert_close(L.replay_one(Replay(llm), toks, [70, 1, 2, 17]), ref, fmt)
+    check_ok(device)
+
+
+@pytest.mark.parametrize("device", DEVICES)
 def test_sampling_is_served(folder, device):
     llm = make_llm(folder, "mixed", "bf16", device)
     sp = SamplingParams(max_new_tokens=6, temperature=0.8, top_k=20, top_p=0.9, seed=3)
