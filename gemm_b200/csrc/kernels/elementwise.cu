@@ -497,7 +497,7 @@ silu_mul_quant_kernel(const __nv_bfloat16* __restrict__ gate_up, const int* __re
 // split order; the result goes out as bf16 and / or as MXFP8 with scale atoms.  8 elements per thread, 4 threads share a scale.
 __global__ void __launch_bounds__(256)
 silu_mul_partials_kernel(const float* __restrict__ part, int n_part, long part_stride, __nv_bfloat16* __restrict__ out, uint8_t* __restrict__ out_q,
-                         uint8_t* __restrict__ out_sf, long rows, int inter, int sf32, int act) {
+                         uint8_t* __restrict__ out_sf, long rows, int inter, int sf32, int act, float cap) {
   pdl_wait();
   pdl_trigger();
   const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -519,7 +519,15 @@ silu_mul_partials_kernel(const float* __restrict__ part, int n_part, long part_s
       u[0] += u0.x; u[1] += u0.y; u[2] += u0.z; u[3] += u0.w; u[4] += u1.x; u[5] += u1.y; u[6] += u1.z; u[7] += u1.w;
     }
 #pragma unroll
-    for (int j = 0; j < 8; ++j) { const float z = act == 1 ? 1.5957691216057308f * (g[j] + 0.044715f * g[j] * g[j] * g[j]) : g[j]; y[j] = g[j] / (1.0f + __expf(-z)) * u[j]; amax = fmaxf(amax, fabsf(y[j])); }
+    for (int j = 0; j < 8; ++j) {
+      if (act == 2) {                                  // capped: g sigmoid(1.702 g) (u + 1)
+        g[j] = fminf(g[j], cap);
+        u[j] = fminf(fmaxf(u[j], -cap), cap) + 1.0f;
+      }
+      const float z = act == 2 ? 1.702f * g[j] : act == 1 ? 1.5957691216057308f * (g[j] + 0.044715f * g[j] * g[j] * g[j]) : g[j];
+      y[j] = g[j] / (1.0f + __expf(-z)) * u[j];
+      amax = fmaxf(amax, fabsf(y[j]));
+    }
     if (out != nullptr) store8(out + r * inter + vi * 8, y);
   }
   if (out_q == nullptr) return;
@@ -950,13 +958,13 @@ GB_API int gb_silu_mul_quant(const void* gate_up, const int* row_valid, void* ou
 }
 
 GB_API int gb_silu_mul_partials(const float* part, int n_part, long part_stride, void* out, void* out_q, void* out_sf, long rows, int inter,
-                                int sf32, int act, cudaStream_t stream) {
+                                int sf32, int act, float cap, cudaStream_t stream) {
   if (inter % 8 || (out_q != nullptr && inter % 128)) return fail("silu_mul_partials: inter must be a multiple of 8 (128 with MXFP8 output)%s");
   if (part_stride % 4 != 0 || ((uintptr_t)part & 15) != 0) return fail("silu_mul_partials: misaligned partials%s");
   const long n = rows * (inter / 8);
   if (n <= 0) return 0;
   launch_k(silu_mul_partials_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, part, n_part, part_stride, (__nv_bfloat16*)out, (uint8_t*)out_q,
-           (uint8_t*)out_sf, rows, inter, sf32, act);
+           (uint8_t*)out_sf, rows, inter, sf32, act, cap);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }

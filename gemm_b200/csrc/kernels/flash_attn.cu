@@ -54,6 +54,9 @@ struct FaArgs {
   int keep_first;           // positions below this stay visible behind the window
   const float* bias;        // [hq][ld_bias]: n_bias scores added at distances 0, 1, ... (the last one beyond), times log2 e; then, per
   int n_bias, ld_bias;      // distance n, the largest of the 128 from n on.  null = none
+  // forms 2 and 3
+  const float* sink;        // [hq] a score per head, times log2 e, that joins the sum of the weights; null = none
+  float cap;                // form 3: scores are cap * tanh(q . k), cap = softcap * log2 e (q carries scale / softcap)
 };
 
 // KV blocks of a query tile or decode token, in order: with a window and kept first positions, the blocks of the kept positions that lie
@@ -73,12 +76,13 @@ __device__ __forceinline__ FaBlocks fa_blocks(const FaArgs& a, int first_pos, in
 
 constexpr int kFaSmem = 32768 * 3 + 256 + 1024;
 
-// DK / DV: width of a key / value head in the cache (64 or 128 columns).  EXT: kept first positions and a distance bias.
-template <int DK, int DV, bool EXT>
-
+// DK / DV: width of a key / value head in the cache (64 or 128 columns).  FORM: 0 = plain, 1 = kept first positions and a distance bias, 2 = sinks,
+// 3 = capped scores (and sinks).
+template <int DK, int DV, int FORM>
 __global__ void __launch_bounds__(kFaThreads, 2)
 flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, const FaArgs a) {
+  constexpr bool EXT = FORM == 1, SINK = FORM >= 2, CAP = FORM == 3;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);      // an offset, so that accesses stay shared-memory ones
   uint8_t* sQ = smem;                       // 2 x [128 rows x 128 B]  (d halves)
@@ -222,6 +226,10 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     // than 2^kTau, so that O and l are rarely rescaled (P stays below 2^kTau, harmless in bf16 with fp32 sums).
     constexpr float kTau = 8.0f;
     float m = -INFINITY, l = 0.f;
+    if constexpr (SINK) {
+      // the sink is a key without a value: it is the first reference, and the first summand of the split that counts it
+      if (a.sink != nullptr && split == 0 && !bad_item) { m = a.sink[kvh * G + h_local]; l = 1.f; }
+    }
     bool ok = true;
     const float* bias_row = EXT && a.bias != nullptr ? a.bias + (size_t)(bad_item ? 0 : kvh * G) * a.ld_bias : nullptr;   // the group's first head
     float* s_bias = reinterpret_cast<float*>(smem + 32768 * 3 + 256);      // EXT: two windows of G x bias_w scores, by block parity
@@ -250,12 +258,16 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       const int keep = EXT ? a.keep_first : 0;
       const bool edge = (kv0 + kBN - 1 > hi || (kv0 < lo && !(EXT && kv0 + kBN <= keep)));
       // pass 1: row maximum (the scores are read again in pass 2 instead of being kept in 128 registers)
-      float mx = -INFINITY;
+      float mx = -INFINITY, far = 0.f;                   // far (CAP): the largest magnitude, masked or not
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         float sv[32];
         tmem_ld_x32(s_t + c * 32, reinterpret_cast<uint32_t*>(sv));
         tc_wait_ld();
+        if constexpr (CAP) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) far = fmaxf(far, fabsf(sv[i]));
+        }
         if (edge) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) { const int kp = kv0 + c * 32 + i; if (kp > hi || (kp < lo && !(EXT && kp < keep))) sv[i] = -INFINITY; }
@@ -271,6 +283,11 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
           bfar = *br;
           mx += br[a.n_bias];
         }
+      }
+      bool unit = false;                                 // CAP: every score of the warp's rows within +-1
+      if constexpr (CAP) {
+        unit = __all_sync(0xffffffffu, far <= 1.0f);
+        if (mx > -INFINITY) mx = a.cap * tanh_wide(mx);
       }
       float alpha = 1.0f;
       const bool grow = mx > m + kTau || (m == -INFINITY && mx > -INFINITY);
@@ -298,6 +315,15 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         float sv[32];
         tmem_ld_x32(s_t + c * 32, reinterpret_cast<uint32_t*>(sv));
         tc_wait_ld();
+        if constexpr (CAP) {
+          if (unit) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) sv[i] = tanh_unit(sv[i]);
+          } else {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) sv[i] = tanh_wide(sv[i]);
+          }
+        }
         if (edge) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) { const int kp = kv0 + c * 32 + i; if (kp > hi || (kp < lo && !(EXT && kp < keep))) sv[i] = -INFINITY; }
@@ -311,7 +337,7 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
         uint32_t pk[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-          const float p0 = fast_exp2(sv[2 * i] - m_far), p1 = fast_exp2(sv[2 * i + 1] - m_far);
+          const float p0 = fast_exp2(CAP ? fmaf(sv[2 * i], a.cap, -m_far) : sv[2 * i] - m_far), p1 = fast_exp2(CAP ? fmaf(sv[2 * i + 1], a.cap, -m_far) : sv[2 * i + 1] - m_far);
           rs += p0 + p1;
           pk[i] = pack_bf16x2(p0, p1);
         }
@@ -416,10 +442,11 @@ constexpr int kFdN = 16;                 // MMA N: query heads of one KV head, z
 constexpr int kFdThreads = 192;
 constexpr int kFdSmem = 4096 + 3 * 32768 + 8192 + 2048 + 1024;   // Q, tile ring, P x2, barriers + reductions, alignment
 
-template <int DK, int DV, bool EXT>
+template <int DK, int DV, int FORM>                 // FORM as in flash_attn_kernel
 __global__ void __launch_bounds__(kFdThreads, 2)
 flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const FaArgs a) {
+  constexpr bool EXT = FORM == 1, SINK = FORM >= 2, CAP = FORM == 3;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);      // an offset, so that accesses stay shared-memory ones
   uint8_t* sQ = smem;                          // 2 d-halves x [16 heads x 128 B]
@@ -556,6 +583,13 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
                                      // l: THIS thread's share of the row sums (its positions only); the threads' shares are added once, at the end
 #pragma unroll
     for (int h = 0; h < kFdN; ++h) { m[h] = -INFINITY; l[h] = 0.f; }
+    if constexpr (SINK) {
+      if (a.sink != nullptr && split == 0 && !bad_item) {
+#pragma unroll
+        for (int h = 0; h < kFdN; ++h)
+          if (h < G) { m[h] = a.sink[kvh * G + h]; l[h] = r == 0 ? 1.f : 0.f; }
+      }
+    }
     constexpr float kTau = 8.0f;     // O and l are only rescaled when a block raises a maximum by more than 2^kTau
     bool ok = true, fail_o = false;  // fail_o: a wait for the second MMA ran out; it is put to the vote at the next barrier
     for (int j = 0; j < n_blk && ok; ++j) {
@@ -582,6 +616,7 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
 #pragma unroll
       for (int h = 0; h < kFdN; ++h) {
         if constexpr (EXT) sv[h] += bv[h];
+        if constexpr (CAP) { if (h < G) sv[h] = a.cap * tanh_wide(sv[h]); }
         if (!live || h >= G) sv[h] = -INFINITY;
       }
       {
@@ -794,10 +829,10 @@ static int flash_attn_impl(const void* q, const void* k_cache, const void* v_cac
   const int smem = kFaSmem;
   static bool attr_set = false;
   if (!attr_set) {
-    GB_CUDA_OK(cudaFuncSetAttribute(flash_attn_kernel<128, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    GB_CUDA_OK(cudaFuncSetAttribute(flash_attn_kernel<128, 128, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     attr_set = true;
   }
-  launch_k(flash_attn_kernel<128, 128, false>, n_work, kFaThreads, smem, stream, tmQ, tmK, tmV, a);
+  launch_k(flash_attn_kernel<128, 128, 0>, n_work, kFaThreads, smem, stream, tmQ, tmK, tmV, a);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -854,10 +889,10 @@ static int flash_decode_impl(const void* q, const void* k_cache, const void* v_c
   a.out_q = out_q; a.out_sf = out_sf; a.out_sf32 = out_sf32;
   static bool attr_set = false;
   if (!attr_set) {
-    GB_CUDA_OK(cudaFuncSetAttribute(flash_decode_kernel<128, 128, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFdSmem));
+    GB_CUDA_OK(cudaFuncSetAttribute(flash_decode_kernel<128, 128, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFdSmem));
     attr_set = true;
   }
-  launch_k(flash_decode_kernel<128, 128, false>, n_work, kFdThreads, kFdSmem, stream, tmQ, tmK, tmV, a);
+  launch_k(flash_decode_kernel<128, 128, 0>, n_work, kFdThreads, kFdSmem, stream, tmQ, tmK, tmV, a);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -899,7 +934,7 @@ GB_API int gb_fa_combine_mx(const float* part_o, const float* part_lse, void* ou
 }
 
 // ------------------------------------------------------------------------------------------ masks, distance bias, 64- and 128-wide heads
-template <int DK, int DV>
+template <int DK, int DV, int FORM>
 static int flash_masked_launch(const void* q, const void* k_cache, const void* v_cache, const FaArgs& a, int n_work, long num_slots, int decode, cudaStream_t stream) {
   const int G = a.hq / a.hkv, tpt = 128 / G;
   CUtensorMap tmQ, tmK, tmV;
@@ -919,34 +954,37 @@ static int flash_masked_launch(const void* q, const void* k_cache, const void* v
   if (decode) {
     static bool attr_set = false;
     if (!attr_set) {
-      GB_CUDA_OK(cudaFuncSetAttribute(flash_decode_kernel<DK, DV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFdSmem));
+      GB_CUDA_OK(cudaFuncSetAttribute(flash_decode_kernel<DK, DV, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, kFdSmem));
       attr_set = true;
     }
-    launch_k(flash_decode_kernel<DK, DV, true>, n_work, kFdThreads, kFdSmem, stream, tmQ, tmK, tmV, a);
+    launch_k(flash_decode_kernel<DK, DV, FORM>, n_work, kFdThreads, kFdSmem, stream, tmQ, tmK, tmV, a);
   } else {
     const int smem = kFaSmem + (a.bias != nullptr ? 2 * G * (127 + tpt) * 4 : 0);
     static int attr_max = 0;
     if (smem > 227 * 1024) return fail("flash_masked: the bias windows of this group size do not fit shared memory%s");
     if (smem > attr_max) {
-      GB_CUDA_OK(cudaFuncSetAttribute(flash_attn_kernel<DK, DV, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+      GB_CUDA_OK(cudaFuncSetAttribute(flash_attn_kernel<DK, DV, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
       attr_max = smem;
     }
-    launch_k(flash_attn_kernel<DK, DV, true>, n_work, kFaThreads, smem, stream, tmQ, tmK, tmV, a);
+    launch_k(flash_attn_kernel<DK, DV, FORM>, n_work, kFaThreads, smem, stream, tmQ, tmK, tmV, a);
   }
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
 
 // gb_flash_attn / gb_flash_decode (decode != 0: one query token per sequence, Hq / Hkv <= 16) with keys of dk and values of dv columns (64 or
-// 128 each), a window that keeps the first `keep_first` positions, and a distance bias (see FaArgs).  q is [T, Hq, dk], out [T, Hq, dv].
+// 128 each), a window that keeps the first `keep_first` positions, and a distance bias, or with capped scores (softcap > 0) and sinks (see FaArgs).  q is
+// [T, Hq, dk], out [T, Hq, dv].
 GB_API int gb_flash_masked(const void* q, const void* k_cache, const void* v_cache, void* out, float* part_o, float* part_lse, const int* work, int n_work,
                            const int* cu_q, const int* kv_len, const int* block_table, int max_pages, int page_size, long num_slots, int total_tokens,
                            int hq, int hkv, int dk, int dv, int num_splits, int window, int keep_first, const float* bias, int n_bias, int ld_bias,
-                           int decode, void* status, cudaStream_t stream) {
+                           float softcap, const float* sink, int decode, void* status, cudaStream_t stream) {
   if ((dk != 64 && dk != 128) || (dv != 64 && dv != 128)) return fail("flash_masked: heads of 64 or 128 columns%s");
   if (hq < 1 || hkv < 1 || hq % hkv || hq / hkv > (decode ? kFdN : 128)) return fail("flash_masked: bad head counts%s");
   if (page_size < 8 || page_size > 128 || (128 % page_size) || (page_size % 8)) return fail("flash_masked: page_size must be 8..128, a multiple of 8 dividing 128%s");
   if (bias != nullptr && (n_bias < 1 || ld_bias < 2 * n_bias)) return fail("flash_masked: bad bias table%s");
+  const int form = softcap > 0.f ? 3 : sink != nullptr ? 2 : 1;
+  if (form > 1 && (bias != nullptr || keep_first > 0)) return fail("flash_masked: capped scores and sinks do not go with a bias or kept positions%s");
   if (window < 0 || keep_first < 0 || num_splits < 1) return fail("flash_masked: bad mask%s");
   if (n_work <= 0) return 0;
   if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return fail("flash_masked: num_splits > 1 needs partial buffers%s");
@@ -957,10 +995,19 @@ GB_API int gb_flash_masked(const void* q, const void* k_cache, const void* v_cac
   a.hq = hq; a.hkv = hkv; a.num_splits = num_splits; a.causal = 1; a.window = window; a.keep_first = window > 0 ? keep_first : 0; a.out = (__nv_bfloat16*)out;
   a.part_o = part_o; a.part_lse = part_lse; a.total_tokens = total_tokens; a.status = (KernelStatus*)status;
   a.bias = bias; a.n_bias = n_bias; a.ld_bias = ld_bias;
-  if (dk == 64) return dv == 64 ? flash_masked_launch<64, 64>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream)
-                                : flash_masked_launch<64, 128>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream);
-  return dv == 64 ? flash_masked_launch<128, 64>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream)
-                  : flash_masked_launch<128, 128>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream);
+  a.sink = sink; a.cap = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+#define GB_FORM(F)                                                                                                                                    \
+  if (form == F) {                                                                                                                                    \
+    if (dk == 64) return dv == 64 ? flash_masked_launch<64, 64, F>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream)                         \
+                                  : flash_masked_launch<64, 128, F>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream);                       \
+    return dv == 64 ? flash_masked_launch<128, 64, F>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream)                                      \
+                    : flash_masked_launch<128, 128, F>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream);                                    \
+  }
+  GB_FORM(1)
+  GB_FORM(2)
+  GB_FORM(3)
+#undef GB_FORM
+  return fail("flash_masked: unknown form%s");
 }
 
 // gb_fa_combine for heads of `head_dim` (64 or 128) features.

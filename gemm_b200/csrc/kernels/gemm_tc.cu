@@ -83,6 +83,7 @@ struct GemmArgs {
   int early_weights;  // != 0: a plain decode-sized launch requests its first weight tiles before the dependency wait
   int dual_raw;  // DUAL without the activation: the second accumulator is the row block up_row_offset further down the same matrix
   int w_tiled;
+  float act_cap; // DUAL with ACT = 2
   int silu_rows; // plain launches with ACT = 1: SiLU on the output features below this (the q / k / v part of a linear-attention projection)
 };
 
@@ -129,12 +130,20 @@ struct TileCursor {
 };
 
 __device__ __forceinline__ float silu_f(float x) { return x / (1.0f + __expf(-x)); }
-// Gate activation: 0 = SiLU, 1 = the tanh form of GELU, x (1 + tanh u) / 2 with u = sqrt(2 / pi) (x + 0.044715 x^3), which is
+// Gate activation of DUAL launches: 2 = "capped": g sigmoid(1.702 g) (u + 1), the gate at most cap, the up part within +-cap;  0 = SiLU, 1 = the tanh form of GELU, x (1 + tanh u) / 2 with u = sqrt(2 / pi) (x + 0.044715 x^3), which is
 // x / (1 + exp(-2 u)).
 template <int ACT>
 __device__ __forceinline__ float gate_act(float x) {
   if constexpr (ACT == 0) return silu_f(x);
   else return __fdividef(x, 1.0f + __expf(x * fmaf(-0.07135481627f, x * x, -1.5957691216057308f)));       // -2 sqrt(2 / pi) (x + 0.044715 x^3)
+}
+
+template <int ACT>
+__device__ __forceinline__ float gated(float g, float u, float cap) {
+  if constexpr (ACT == 2) {
+    g = fminf(g, cap);
+    return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (fminf(fmaxf(u, -cap), cap) + 1.0f);
+  } else return gate_act<ACT>(g) * u;
 }
 
 // E8M0 exponent for a block whose absolute maximum is `amax`: the smallest power of two s with
@@ -147,7 +156,7 @@ __device__ __forceinline__ int e8m0_from_amax(float amax) {
   return amax == 0.0f ? 127 : max(1, min(e, 254));   // an all-zero block gets scale 1
 }
 
-// ACT, DUAL: the gate's activation (gate_act); plain: 1 = SiLU on the output features below args.silu_rows, 2 = bf16 rows scattered by args.row_map.
+// ACT, DUAL: the gate's activation (gated); plain: 1 = SiLU on the output features below args.silu_rows, 2 = bf16 rows scattered by args.row_map.
 template <int TN, int MODE, bool DUAL, bool QUANT_OUT, int ACT = 0>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, const GemmArgs args) {
@@ -410,7 +419,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
         for (int j = 0; j < 16; ++j) {
           const int xr = c + j;
           float v = __uint_as_float(r0[j]);
-          if (DUAL) v = gate_act<ACT>(v) * __uint_as_float(r1[j]);
+          if (DUAL) v = gated<ACT>(v, __uint_as_float(r1[j]), args.act_cap);
           v += bias;
           if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
           const bool live = xr < t.valid;
@@ -637,7 +646,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               float v = __uint_as_float(r0[j]);
-              if (DUAL) v = gate_act<ACT>(v) * __uint_as_float(r1[j]);
+              if (DUAL) v = gated<ACT>(v, __uint_as_float(r1[j]), args.act_cap);
               v += bias;
               if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
               if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
@@ -647,7 +656,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               float v = __uint_as_float(r0[j]);
-              if (DUAL) v = gate_act<ACT>(v) * __uint_as_float(r1[j]);
+              if (DUAL) v = gated<ACT>(v, __uint_as_float(r1[j]), args.act_cap);
               v += bias;
               if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
               if (c + j < t.valid) {
@@ -764,10 +773,11 @@ struct GemmExtras {
   size_t sfa_bytes, sfb_bytes, out_bytes, out_sf_bytes;
   long partial_stride;       // > 0 with splits > 1: every K split stores its fp32 partial into its own slab of `out` (the consumer sums them)
   int silu_rows;             // SiLU on the output features below this (launches that are neither DUAL nor K-split)
+  float act_cap;             // GEMM_CAPPED: bound of gate and up part
 };
 
 // Flags of gb_gemm.
-enum { GEMM_MX = 1, GEMM_DUAL = 2, GEMM_QUANT_OUT = 4, GEMM_OUT_F32 = 8, GEMM_W_TILED = 16, GEMM_DUAL_RAW = 32, GEMM_GELU = 64 };
+enum { GEMM_MX = 1, GEMM_DUAL = 2, GEMM_QUANT_OUT = 4, GEMM_OUT_F32 = 8, GEMM_W_TILED = 16, GEMM_DUAL_RAW = 32, GEMM_GELU = 64, GEMM_CAPPED = 128 };
 
 // Linear layer on tensor cores.
 //   w        [w_rows, k] row-major (bf16, or e4m3 bytes when GEMM_MX), w_rows = groups * w_rows_per_group
@@ -823,7 +833,9 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
   }
   a.dual_raw = (flags & GEMM_DUAL_RAW) ? 1 : 0;
   const bool gelu = flags & GEMM_GELU;
-  if (gelu && (!dual || mx || qo)) return fail("gemm: GEMM_GELU needs a bf16 GEMM_DUAL launch%s");
+  const bool capped = flags & GEMM_CAPPED;
+  if ((gelu || capped) && (!dual || mx || qo || (gelu && capped))) return fail("gemm: GEMM_GELU / GEMM_CAPPED need a bf16 GEMM_DUAL launch%s");
+  if (capped && ex == nullptr) return fail("gemm: GEMM_CAPPED without a bound%s");
   if (a.dual_raw && (!dual || qo)) return fail("gemm: GEMM_DUAL_RAW needs GEMM_DUAL without GEMM_QUANT_OUT%s");
   a.out_sf = (uint8_t*)out_sf; a.bias = bias; a.row_map = row_map; a.row_scale = row_scale; a.status = (KernelStatus*)status;
   if (ex != nullptr) {
@@ -834,6 +846,7 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
     a.sfa_bytes = ex->sfa_bytes; a.sfb_bytes = ex->sfb_bytes; a.out_bytes = ex->out_bytes; a.out_sf_bytes = ex->out_sf_bytes;
     if (ex->silu_rows > 0 && (dual || mx || qo || ex->splits > 1 || tn < 128)) return fail("gemm: silu_rows needs a plain bf16 launch with a token tile of 128 or 256%s");
     a.silu_rows = ex->silu_rows;
+    a.act_cap = ex->act_cap;
     if (ex->splits > 1 && num_groups == 0 && ex->partial_stride > 0) {
       if (!(flags & GEMM_OUT_F32) || qo) return fail("gemm: split-K partials need a plain fp32 output%s");
       const int kb_elems = mx ? 128 : 64;
@@ -878,6 +891,7 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
   if (tn == TNV) {                                                                                            \
     if (!mx && !dual && !qo) return launch_gemm<TNV, 0, false, false>(tmW, tmX, a, max_tiles, stream);        \
     if (gelu) return launch_gemm<TNV, 0, true, false, 1>(tmW, tmX, a, max_tiles, stream);                     \
+    if (capped) return launch_gemm<TNV, 0, true, false, 2>(tmW, tmX, a, max_tiles, stream);                   \
     if (!mx && dual && !qo) return launch_gemm<TNV, 0, true, false>(tmW, tmX, a, max_tiles, stream);          \
   }
 #else
@@ -885,6 +899,7 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
   if (tn == TNV) {                                                                                            \
     if (!mx && !dual && !qo) return launch_gemm<TNV, 0, false, false>(tmW, tmX, a, max_tiles, stream);        \
     if (gelu) return launch_gemm<TNV, 0, true, false, 1>(tmW, tmX, a, max_tiles, stream);                     \
+    if (capped) return launch_gemm<TNV, 0, true, false, 2>(tmW, tmX, a, max_tiles, stream);                   \
     if (!mx && dual && !qo) return launch_gemm<TNV, 0, true, false>(tmW, tmX, a, max_tiles, stream);          \
     if (mx && !dual && !qo) return launch_gemm<TNV, 1, false, false>(tmW, tmX, a, max_tiles, stream);         \
     if (mx && dual && qo) return launch_gemm<TNV, 1, true, true>(tmW, tmX, a, max_tiles, stream);             \

@@ -1,10 +1,12 @@
-// Prefill scan of linear attention with a forget gate per key channel (HGRN2; the token-by-token form is in recurrent.cu), in two kernels:
+// Prefill scan of linear attention with a decay per key channel (HGRN2, RWKV; the token-by-token forms are in recurrent.cu), in two kernels:
 //
-//   S_t = diag(f_t) S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t,  k = 1 - f
+//   S_t = diag(f_t) S_{t-1} + k_t v_t^T,  o_t = S_t^T q_t,  k = 1 - f                    (HGRN2)
+//   S_t = diag(f_t) S_{t-1} + k_t v_t^T,  o_t = (S_{t-1} + diag(u) k_t v_t^T)^T q_t      (RWKV; f = exp(-exp(z)))
 //
 // Over a block of 16 tokens with the state S0 in front of it, c_i = f_0 ... f_i, r_j = f_{j+1} ... f_15 and b = c_15 (per channel):
 //   O_i   = (q_i c_i) S0 + sum_{j <= i} P_ij v_j,   P_ij = sum_d q_i k_j f_{j+1} ... f_i
 //   S_end = diag(b) S0 + sum_j (k_j r_j) v_j^T
+// RWKV's output reads the state in front of the token: c_i = f_0 ... f_{i-1}, P_ij = sum_d q_i k_j f_{j+1} ... f_{i-1} for j < i, P_ii = sum_d q_i u k_i.
 // All decays are products of gates, never quotients or differences of logarithms, so gates of any size (down to 0) are exact.
 //
 // gla_prep_kernel, parallel over blocks and heads: gates, q c, k r, P and b.  It writes a record per (block, head) that is the image of the scan's
@@ -35,7 +37,9 @@ template <int DP> struct GlaRecord {
 __device__ __forceinline__ int gla_first_block(int t0, int seq) { return t0 / kGlB + seq; }
 
 struct GlaArgs {
-  const __nv_bfloat16* qv; int ld;           // [tokens, ld]: q heads x dim (SiLU applied), v heads x vdim
+  const __nv_bfloat16* qv; int ld;           // [tokens, ld]: q heads x dim (HGRN2: SiLU applied)
+  const __nv_bfloat16* k;                    // RWKV: [tokens, ld]: k heads x dim
+  const float* u;                            // RWKV: [heads x dim]
   const float* gate; int g_part; long g_stride; int g_ld;      // forget gates before bias and sigmoid
   const float* gate_bias; const float* lower;
   float* state; int n_slots;
@@ -46,7 +50,7 @@ struct GlaArgs {
   KernelStatus* status;
 };
 
-template <int DP>
+template <int DP, bool RWKV>
 __global__ void __launch_bounds__(256)
 gla_prep_kernel(const GlaArgs a) {
   using R = GlaRecord<DP>;
@@ -66,7 +70,10 @@ gla_prep_kernel(const GlaArgs a) {
       const float* g = a.gate + (size_t)(t0 + i) * a.g_ld + col;
       float z = *g;
       for (int p = 1; p < a.g_part; ++p) z += g[(size_t)p * a.g_stride];
-      f = forget_gate(z + a.gate_bias[col], a.lower[col], k);
+      if constexpr (RWKV) {
+        f = expf(-expf(z + a.gate_bias[col]));
+        k = __bfloat162float(a.k[(size_t)(t0 + i) * a.ld + col]);
+      } else f = forget_gate(z + a.gate_bias[col], a.lower[col], k);
       q = __bfloat162float(a.qv[(size_t)(t0 + i) * a.ld + col]);
     }
     sf[i][c] = f; sk[i][c] = k; sq[i][c] = q;
@@ -80,9 +87,10 @@ gla_prep_kernel(const GlaArgs a) {
 #pragma unroll
     for (int i = 0; i < kGlB; ++i) {
       const float2 f = *reinterpret_cast<const float2*>(&sf[i][c2]), q = *reinterpret_cast<const float2*>(&sq[i][c2]);
-      p0 *= f.x; p1 *= f.y;
+      if constexpr (!RWKV) { p0 *= f.x; p1 *= f.y; }
       uint32_t hi, lo;
       split_bf16x2(q.x * p0, q.y * p1, hi, lo);
+      if constexpr (RWKV) { p0 *= f.x; p1 *= f.y; }
       uint8_t* dst = rec + R::kQ + 2 * tile + i * 128 + ((chunk ^ (i & 7)) << 4) + in;
       *reinterpret_cast<uint32_t*>(dst) = hi;
       *reinterpret_cast<uint32_t*>(dst + 2048) = lo;
@@ -105,9 +113,12 @@ gla_prep_kernel(const GlaArgs a) {
   {
     constexpr int CH = DP / 16;
     const int warp = tid >> 5, lane = tid & 31, j = lane & 15, c0 = warp * (DP / 8) + (lane >> 4) * CH;
-    float w[CH], k[CH];
+    float w[CH], k[CH], uk[RWKV ? CH : 1], fl[RWKV ? CH : 1];    // fl: the gates of the token in front
 #pragma unroll
-    for (int x = 0; x < CH; ++x) { w[x] = 0.f; k[x] = sk[j][c0 + x]; }
+    for (int x = 0; x < CH; ++x) {
+      w[x] = 0.f; k[x] = sk[j][c0 + x];
+      if constexpr (RWKV) { uk[x] = c0 + x < a.dim ? k[x] * a.u[h * a.dim + c0 + x] : 0.f; fl[x] = 1.f; }
+    }
 #pragma unroll
     for (int i = 0; i < kGlB; ++i) {
       float acc = 0.f;
@@ -117,8 +128,14 @@ gla_prep_kernel(const GlaArgs a) {
         const float fv[4] = {f.x, f.y, f.z, f.w}, qv[4] = {q.x, q.y, q.z, q.w};
 #pragma unroll
         for (int y = 0; y < 4; ++y) {
-          w[x + y] = i == j ? k[x + y] : w[x + y] * fv[y];
-          acc = fmaf(qv[y], w[x + y], acc);
+          if constexpr (RWKV) {
+            w[x + y] = i == j + 1 ? k[x + y] : w[x + y] * fl[x + y];
+            fl[x + y] = fv[y];
+            acc = fmaf(qv[y], i == j ? uk[x + y] : w[x + y], acc);
+          } else {
+            w[x + y] = i == j ? k[x + y] : w[x + y] * fv[y];
+            acc = fmaf(qv[y], w[x + y], acc);
+          }
         }
       }
       acc += __shfl_xor_sync(0xffffffffu, acc, 16);
@@ -331,14 +348,14 @@ gla_scan_kernel(const __grid_constant__ CUtensorMap tmV, const GlaArgs a) {
   if (warp == 1) { tc_fence_after(); tmem_dealloc(tmem, 512); }
 }
 
-template <int DP>
+template <int DP, bool RWKV>
 static int gla_chunk_launch(const CUtensorMap& tmV, const GlaArgs& a, int max_tokens, int n_seqs, cudaStream_t stream) {
   static bool attr_set = false;
   if (!attr_set) {
     GB_CUDA_OK(cudaFuncSetAttribute(gla_scan_kernel<DP>, cudaFuncAttributeMaxDynamicSharedMemorySize, gla_smem<DP>()));
     attr_set = true;
   }
-  launch_k(gla_prep_kernel<DP>, dim3((unsigned)((max_tokens + kGlB - 1) / kGlB), (unsigned)a.heads, (unsigned)n_seqs), 256, 0, stream, a);
+  launch_k(gla_prep_kernel<DP, RWKV>, dim3((unsigned)((max_tokens + kGlB - 1) / kGlB), (unsigned)a.heads, (unsigned)n_seqs), 256, 0, stream, a);
   GB_CUDA_OK(cudaGetLastError());
   launch_k(gla_scan_kernel<DP>, dim3((unsigned)a.heads, (unsigned)((a.vdim + 127) / 128), (unsigned)n_seqs), gla_threads<DP>(), gla_smem<DP>(), stream, tmV, a);
   GB_CUDA_OK(cudaGetLastError());
@@ -369,8 +386,33 @@ GB_API int gb_gla_chunk(const void* qv, int ld, int tokens, const float* gate, i
   uint64_t dv[3] = {(uint64_t)vdim, (uint64_t)heads, (uint64_t)tokens}, sv[2] = {(uint64_t)vdim * 2, (uint64_t)ld * 2};
   if (make_tmap(&tmV, (const __nv_bfloat16*)qv + (size_t)heads * dim, TM_BF16, 3, dv, sv, box, TM_SW_128)) return -1;
   GlaArgs a;
+  a.k = nullptr; a.u = nullptr;
   a.qv = (const __nv_bfloat16*)qv; a.ld = ld; a.gate = gate; a.g_part = g_part; a.g_stride = g_stride; a.g_ld = g_ld; a.gate_bias = gate_bias; a.lower = lower;
   a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out; a.ld_out = ld_out; a.heads = heads; a.dim = dim; a.vdim = vdim;
   a.ws = (uint8_t*)ws; a.status = (KernelStatus*)status;
-  return dim <= 64 ? gla_chunk_launch<64>(tmV, a, max_tokens, n_seqs, stream) : gla_chunk_launch<128>(tmV, a, max_tokens, n_seqs, stream);
+  return dim <= 64 ? gla_chunk_launch<64, false>(tmV, a, max_tokens, n_seqs, stream) : gla_chunk_launch<128, false>(tmV, a, max_tokens, n_seqs, stream);
+}
+
+// The RWKV form: rkv holds r, k and v as three blocks of bf16 rows [tokens, ld], `block_stride` elements apart; the other arguments as in gb_rwkv_step and
+// gb_gla_chunk.
+GB_API int gb_rwkv_chunk(const void* rkv, long block_stride, int ld, int tokens, const float* z, int z_part, long z_stride, int z_ld, const float* w0, const float* u,
+                         float* state, int n_slots, const int* cu_q, const int* seq_slots, float* out, int ld_out, int heads, int dim, int vdim, int max_tokens, int n_seqs,
+                         void* ws, long ws_bytes, void* status, cudaStream_t stream) {
+  if (n_seqs <= 0 || tokens <= 0 || max_tokens <= 0) return 0;
+  if (heads < 1 || dim < 8 || dim > 128 || dim % 8 || vdim < 8 || vdim % 8 || z_part < 1) return fail("rwkv_chunk: dim <= 128, dim and vdim multiples of 8%s");
+  if (ld % 8 || block_stride % 8 || ld < heads * dim || ld < heads * vdim || z_ld < heads * dim || ld_out < heads * vdim || ((uintptr_t)rkv & 15) || ((uintptr_t)ws & 15))
+    return fail("rwkv_chunk: bad rows%s");
+  if (ws_bytes < gb_gla_chunk_workspace(tokens, n_seqs, heads, dim)) return fail("rwkv_chunk: workspace too small%s");
+  if (n_seqs > 65535 || heads > 65535) return fail("rwkv_chunk: too many sequences%s");
+  const __nv_bfloat16* r = (const __nv_bfloat16*)rkv;
+  CUtensorMap tmV;
+  uint32_t box[3] = {64, 1, kGlB};
+  uint64_t dv[3] = {(uint64_t)vdim, (uint64_t)heads, (uint64_t)tokens}, sv[2] = {(uint64_t)vdim * 2, (uint64_t)ld * 2};
+  if (make_tmap(&tmV, r + 2 * block_stride, TM_BF16, 3, dv, sv, box, TM_SW_128)) return -1;
+  GlaArgs a;
+  memset(&a, 0, sizeof(a));
+  a.qv = r; a.k = r + block_stride; a.ld = ld; a.u = u; a.gate = z; a.g_part = z_part; a.g_stride = z_stride; a.g_ld = z_ld; a.gate_bias = w0;
+  a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out; a.ld_out = ld_out; a.heads = heads; a.dim = dim; a.vdim = vdim;
+  a.ws = (uint8_t*)ws; a.status = (KernelStatus*)status;
+  return dim <= 64 ? gla_chunk_launch<64, true>(tmV, a, max_tokens, n_seqs, stream) : gla_chunk_launch<128, true>(tmV, a, max_tokens, n_seqs, stream);
 }

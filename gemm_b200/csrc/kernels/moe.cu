@@ -21,31 +21,31 @@ namespace gb {
 template <int MAXV, bool GROUPS>
 __device__ __forceinline__ int route_token_n(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ ids,
                                            float* __restrict__ weights, int w, int lane, int n_exp, int k, int mode, int renorm,
-                                           float routed_scale, int groups, int keep, int ld, int id_shift, int n_local) {
+                                           float routed_scale, int groups, int keep, int group_best, int ld, int id_shift, int n_local) {
   return route_row<MAXV, GROUPS>(logits + (size_t)w * ld, bias, ids + (size_t)w * k, weights + (size_t)w * k, lane, n_exp, k, mode, renorm,
-                         routed_scale, groups, keep, id_shift, n_local);
+                         routed_scale, groups, keep, group_best, id_shift, n_local);
 }
 
 // The per-lane expert slots are sized to the expert count, so a 128-expert router runs a quarter of the 512-expert code.
 template <bool GROUPS>
 __device__ __forceinline__ int route_token(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ ids,
                                            float* __restrict__ weights, int w, int lane, int n_exp, int k, int mode, int renorm,
-                                           float routed_scale, int groups, int keep, int ld, int id_shift, int n_local) {
-  if (n_exp <= 128) return route_token_n<4, GROUPS>(logits, bias, ids, weights, w, lane, n_exp, k, mode, renorm, routed_scale, groups, keep, ld, id_shift, n_local);
-  if (n_exp <= 256) return route_token_n<8, GROUPS>(logits, bias, ids, weights, w, lane, n_exp, k, mode, renorm, routed_scale, groups, keep, ld, id_shift, n_local);
-  return route_token_n<16, GROUPS>(logits, bias, ids, weights, w, lane, n_exp, k, mode, renorm, routed_scale, groups, keep, ld, id_shift, n_local);
+                                           float routed_scale, int groups, int keep, int group_best, int ld, int id_shift, int n_local) {
+  if (n_exp <= 128) return route_token_n<4, GROUPS>(logits, bias, ids, weights, w, lane, n_exp, k, mode, renorm, routed_scale, groups, keep, group_best, ld, id_shift, n_local);
+  if (n_exp <= 256) return route_token_n<8, GROUPS>(logits, bias, ids, weights, w, lane, n_exp, k, mode, renorm, routed_scale, groups, keep, group_best, ld, id_shift, n_local);
+  return route_token_n<16, GROUPS>(logits, bias, ids, weights, w, lane, n_exp, k, mode, renorm, routed_scale, groups, keep, group_best, ld, id_shift, n_local);
 }
 
 // One warp per token.
 template <bool GROUPS>
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ ids, float* __restrict__ weights,
-                 int n_tok, int n_exp, int k, int mode, int renorm, float routed_scale, int groups, int keep, int ld, int id_shift, int n_local) {
+                 int n_tok, int n_exp, int k, int mode, int renorm, float routed_scale, int groups, int keep, int group_best, int ld, int id_shift, int n_local) {
   pdl_wait();
   pdl_trigger();
   const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
   if (w >= n_tok) return;
-  route_token<GROUPS>(logits, bias, ids, weights, w, threadIdx.x & 31, n_exp, k, mode, renorm, routed_scale, groups, keep, ld, id_shift, n_local);
+  route_token<GROUPS>(logits, bias, ids, weights, w, threadIdx.x & 31, n_exp, k, mode, renorm, routed_scale, groups, keep, group_best, ld, id_shift, n_local);
 }
 
 // Router logits for decode-sized batches on the CUDA cores: out[m, n] = sum_k x[m, k] * w[n, k] (bf16 in, fp32 out).
@@ -183,7 +183,7 @@ router_route_kernel(const __nv_bfloat16* __restrict__ x, const __nv_bfloat16* __
   const int tok = m0 + warp;                         // 8 warps, 8 tokens
   if (tok >= m) return;
   route_row<4, false>(&lg[warp][0], bias, ids + (size_t)tok * topk, weights + (size_t)tok * topk, lane, n, topk, mode, renorm, routed_scale,
-               1, 1, id_shift, n_local);
+               1, 1, 2, id_shift, n_local);
 }
 
 constexpr int kPlanBlock = 256;
@@ -282,7 +282,7 @@ moe_plan_small_kernel(const int* __restrict__ ids, int* __restrict__ seg_start, 
                       int* __restrict__ region_rows_used, int* __restrict__ pair_row, int* __restrict__ row_token, int n_pairs,
                       int n_exp, int k, int experts_per_region, int region_rows, int align, int capacity, unsigned* epoch_ctr,
                       const float* __restrict__ logits, const float* __restrict__ bias, int* __restrict__ ids_out,
-                      float* __restrict__ weights_out, int n_route_exp, int mode, int renorm, float routed_scale, int groups, int keep, int ld, int id_shift,
+                      float* __restrict__ weights_out, int n_route_exp, int mode, int renorm, float routed_scale, int groups, int keep, int group_best, int ld, int id_shift,
                       int n_local) {
   pdl_wait();
   pdl_trigger();
@@ -297,7 +297,7 @@ moe_plan_small_kernel(const int* __restrict__ ids, int* __restrict__ seg_start, 
     // routing fused in: a warp per token picks the top-k and leaves the ids in shared memory for the plan
     const int lane = t & 31, n_tok = n_pairs / k;
     for (int w = t >> 5; w < n_tok; w += (int)(blockDim.x >> 5)) {
-      int e = route_token<GROUPS>(logits, bias, ids_out, weights_out, w, lane, n_route_exp, k, mode, renorm, routed_scale, groups, keep, ld, id_shift, n_local);
+      int e = route_token<GROUPS>(logits, bias, ids_out, weights_out, w, lane, n_route_exp, k, mode, renorm, routed_scale, groups, keep, group_best, ld, id_shift, n_local);
       if (lane < k) {
         if (e < 0 || e >= n_exp) e = -1;
         se[w * k + lane] = e;
@@ -489,11 +489,11 @@ GB_API int gb_small_linear(const void* x, const void* w, float* out, int m, int 
 }
 
 GB_API int gb_moe_route(const float* logits, const float* bias, int* ids, float* weights, int n_tok, int n_exp, int k, int mode,
-                        int renorm, float routed_scale, int groups, int keep, int ld, int id_shift, int n_local, cudaStream_t stream) {
+                        int renorm, float routed_scale, int groups, int keep, int group_best, int ld, int id_shift, int n_local, cudaStream_t stream) {
   if (n_exp > 512 || k > kMaxTopK || k > n_exp) return fail("moe_route: need n_exp <= 512 and k <= 16%s");
-  if (groups < 1 || groups > kMaxExpertGroups || n_exp % groups || keep < 1 || keep > groups) return fail("moe_route: bad expert groups%s");
+  if (groups < 1 || groups > kMaxExpertGroups || n_exp % groups || keep < 1 || keep > groups || group_best < 1 || group_best > 2) return fail("moe_route: bad expert groups%s");
   if (n_tok <= 0) return 0;
-  launch_k(keep < groups ? moe_route_kernel<true> : moe_route_kernel<false>, (n_tok + 7) / 8, 256, 0, stream, logits, bias, ids, weights, n_tok, n_exp, k, mode, renorm, routed_scale, groups, keep, ld, id_shift, n_local);
+  launch_k(keep < groups ? moe_route_kernel<true> : moe_route_kernel<false>, (n_tok + 7) / 8, 256, 0, stream, logits, bias, ids, weights, n_tok, n_exp, k, mode, renorm, routed_scale, groups, keep, group_best, ld, id_shift, n_local);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
@@ -507,7 +507,7 @@ GB_API int gb_moe_plan(const int* ids, int* workspace, int* seg_start, int* seg_
   if (n_pairs <= kSmallPairs && capacity < (1l << 30)) {
     launch_k(moe_plan_small_kernel<false>, 1, 1024, 0, stream, ids, seg_start, seg_count, region_rows_used, pair_row, row_token, (int)n_pairs,
              n_exp, k, experts_per_region, region_rows, align, (int)capacity, (unsigned*)epoch_ctr, (const float*)nullptr,
-             (const float*)nullptr, (int*)nullptr, (float*)nullptr, 0, 0, 0, 1.0f, 1, 1, 0, 0, 0);
+             (const float*)nullptr, (int*)nullptr, (float*)nullptr, 0, 0, 0, 1.0f, 1, 1, 2, 0, 0, 0);
     GB_CUDA_OK(cudaGetLastError());
     return 0;
   }
@@ -524,16 +524,16 @@ GB_API int gb_moe_plan(const int* ids, int* workspace, int* seg_start, int* seg_
 // Routing and plan in one launch for decode-sized batches (n_tok * k <= 2048): logits f32 [n_tok, n_route_exp] -> ids / weights
 // [n_tok, k] plus every output of gb_moe_plan over `n_exp` plan experts (= n_local when the ids are made local, else n_route_exp).
 GB_API int gb_moe_route_plan(const float* logits, const float* bias, int* ids, float* weights, int n_tok, int n_route_exp, int k, int mode,
-                             int renorm, float routed_scale, int groups, int keep, int ld, int id_shift, int n_local, int* seg_start, int* seg_count,
+                             int renorm, float routed_scale, int groups, int keep, int group_best, int ld, int id_shift, int n_local, int* seg_start, int* seg_count,
                              int* region_rows_used, int* pair_row, int* row_token, int n_exp, int experts_per_region, int region_rows,
                              int align, long capacity, void* epoch_ctr, cudaStream_t stream) {
   if (n_route_exp > 512 || n_exp > 512 || k > kMaxTopK || k > n_route_exp) return fail("moe_route_plan: need n_exp <= 512 and k <= 16%s");
-  if (groups < 1 || groups > kMaxExpertGroups || n_route_exp % groups || keep < 1 || keep > groups) return fail("moe_route_plan: bad expert groups%s");
+  if (groups < 1 || groups > kMaxExpertGroups || n_route_exp % groups || keep < 1 || keep > groups || group_best < 1 || group_best > 2) return fail("moe_route_plan: bad expert groups%s");
   if ((long)n_tok * k > kSmallPairs || n_tok <= 0) return fail("moe_route_plan: batch too large for the single-kernel path%s");
   if (n_exp % experts_per_region) return fail("moe_route_plan: n_exp %% experts_per_region != 0%s");
   launch_k(keep < groups ? moe_plan_small_kernel<true> : moe_plan_small_kernel<false>, 1, 1024, 0, stream, (const int*)nullptr, seg_start, seg_count, region_rows_used, pair_row, row_token,
            n_tok * k, n_exp, k, experts_per_region, region_rows, align, (int)capacity, (unsigned*)epoch_ctr, logits, bias, ids, weights,
-           n_route_exp, mode, renorm, routed_scale, groups, keep, ld, id_shift, n_local);
+           n_route_exp, mode, renorm, routed_scale, groups, keep, group_best, ld, id_shift, n_local);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }

@@ -44,7 +44,7 @@ constexpr int kPrepIdsLd = 16;        // ids per token in the shared id table (>
 struct MoePrepArgs {
   const __nv_bfloat16* h; int ld_h; int n_tok; int hidden;
   const __nv_bfloat16* w; int ld_w; int n_exp;
-  const float* bias; int topk; int mode; int renorm; float routed_scale; int groups; int keep; int id_shift; int n_local;
+  const float* bias; int topk; int mode; int renorm; float routed_scale; int groups; int keep; int group_best; int id_shift; int n_local;
   int plan_exp;                 // experts the plan covers: n_local when the ids are made local, else n_exp
   int align; int capacity;      // segment alignment (rows) and rows of the expert-sorted buffer
   int* ids; float* weights;     // [n_tok, topk]
@@ -191,7 +191,7 @@ moe_prep_kernel(const MoePrepArgs a) {
       const int t = c * TPC + tl;
       if (t >= a.n_tok || !ok) continue;
       const int id = route_row<4, GROUPS>(lg + tl * kPrepExp, a.bias, a.ids + (size_t)t * a.topk, a.weights + (size_t)t * a.topk, lane, a.n_exp, a.topk,
-                                  a.mode, a.renorm, a.routed_scale, a.groups, a.keep, a.id_shift, a.n_local);
+                                  a.mode, a.renorm, a.routed_scale, a.groups, a.keep, a.group_best, a.id_shift, a.n_local);
       if (lane < a.topk)
         for (int d = 0; d < C; ++d) st_cluster_b32(mapa_u32(ids0 + (uint32_t)((t * kPrepIdsLd + lane) * 4), (uint32_t)d), (uint32_t)id);
     }
@@ -319,19 +319,19 @@ GB_API int gb_moe_prep_supported(int n_tok, int hidden, int n_exp, int topk) {
 // the layout of `align`-row tiles: sf32 != 0 for 32-row atoms) or, with xq == NULL, as bf16 (xs [capacity, hidden]).
 // id_shift / n_local as in gb_moe_route; plan_exp = n_local when n_local > 0, else n_exp.  Segments start at multiples of `align`.
 GB_API int gb_moe_prep(const void* h, int ld_h, int n_tok, int hidden, const void* w, int ld_w, int n_exp, const float* bias, int topk,
-                       int mode, int renorm, float routed_scale, int groups, int keep, int id_shift, int n_local, int align, int capacity, int* ids,
+                       int mode, int renorm, float routed_scale, int groups, int keep, int group_best, int id_shift, int n_local, int align, int capacity, int* ids,
                        float* weights, int* seg_start, int* seg_count, int* pair_row, int* row_token, void* xq, void* xsf, int sf32,
                        void* xs, const void* wait_flags, int wait_n, const void* epoch_ptr, void* status, cudaStream_t stream) {
   if (!gb_moe_prep_supported(n_tok, hidden, n_exp, topk)) return fail("moe_prep: unsupported shape%s (tokens %ld, hidden %ld)", "", n_tok, hidden);
   if (ld_h % 8 || ld_w % 8 || ((uintptr_t)h & 15) || ((uintptr_t)w & 15)) return fail("moe_prep: rows must be 16-byte aligned%s");
-  if (groups < 1 || groups > kMaxExpertGroups || n_exp % groups || keep < 1 || keep > groups) return fail("moe_prep: bad expert groups%s");
+  if (groups < 1 || groups > kMaxExpertGroups || n_exp % groups || keep < 1 || keep > groups || group_best < 1 || group_best > 2) return fail("moe_prep: bad expert groups%s");
   if (align < 1 || capacity < 1) return fail("moe_prep: bad plan geometry%s");
   if (xq == nullptr && xs == nullptr) return fail("moe_prep: no output buffer for the gathered rows%s");
   const int C = prep_cluster(hidden);
   MoePrepArgs a;
   memset(&a, 0, sizeof(a));
   a.h = (const __nv_bfloat16*)h; a.ld_h = ld_h; a.n_tok = n_tok; a.hidden = hidden; a.w = (const __nv_bfloat16*)w; a.ld_w = ld_w; a.n_exp = n_exp;
-  a.bias = bias; a.topk = topk; a.mode = mode; a.renorm = renorm; a.routed_scale = routed_scale; a.groups = groups; a.keep = keep; a.id_shift = id_shift; a.n_local = n_local;
+  a.bias = bias; a.topk = topk; a.mode = mode; a.renorm = renorm; a.routed_scale = routed_scale; a.groups = groups; a.keep = keep; a.group_best = group_best; a.id_shift = id_shift; a.n_local = n_local;
   a.plan_exp = n_local > 0 ? n_local : n_exp; a.align = align; a.capacity = capacity; a.ids = ids; a.weights = weights;
   a.seg_start = seg_start; a.seg_count = seg_count; a.pair_row = pair_row; a.row_token = row_token;
   a.xq = (uint8_t*)xq; a.xsf = (uint8_t*)xsf; a.sf32 = sf32; a.xs = (__nv_bfloat16*)xs;

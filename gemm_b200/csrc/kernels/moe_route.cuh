@@ -13,12 +13,12 @@ constexpr int kMaxTopK = 16;
 constexpr int kMaxExpertGroups = 128;
 
 // Routing of token `w` by one warp (E <= 512): lane j < k ends with the j-th pick.  Returns the (possibly local) expert id.
-// GROUPS (an instance of its own: the code costs the others registers): `groups` (at most kMaxExpertGroups, dividing the experts): a group of neighbouring experts scores the sum of its two best, and only
+// GROUPS (an instance of its own: the code costs the others registers): `groups` (at most kMaxExpertGroups, dividing the experts): a group of neighbouring experts scores the sum of its `group_best` (1 or 2) best, and only
 // experts of the `keep` best groups can be picked (ties: lower group).  renorm: 1 = weights over max(sum, 1e-20), 2 = over sum + 1e-20.
 template <int MAXV, bool GROUPS>
 __device__ __forceinline__ int route_row(const float* row, const float* __restrict__ bias, int* __restrict__ ids_row,
                                          float* __restrict__ weights_row, int lane, int n_exp, int k, int mode, int renorm,
-                                         float routed_scale, int groups, int keep, int id_shift, int n_local) {
+                                         float routed_scale, int groups, int keep, int group_best, int id_shift, int n_local) {
   float p[MAXV], sel[MAXV];
   float mx = -FLT_MAX;
 #pragma unroll
@@ -63,7 +63,7 @@ __device__ __forceinline__ int route_row(const float* row, const float* __restri
         v = mode == 0 ? expf(v - mx) : 1.0f / (1.0f + expf(-v)) + (bias != nullptr ? bias[g * size + x] : 0.f);
         if (v > b1) { b2 = b1; b1 = v; } else if (v > b2) b2 = v;
       }
-      gs[i] = size > 1 ? b1 + b2 : b1;
+      gs[i] = size > 1 && group_best > 1 ? b1 + b2 : b1;
     }
     for (int j = 0; j < keep; ++j) {
       float best = -FLT_MAX; int bi = 0x7fffffff;

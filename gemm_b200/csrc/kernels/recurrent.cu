@@ -2,8 +2,11 @@
 //   causal_conv   depthwise causal convolution with bias + SiLU over packed tokens, the last taps - 1 inputs carried per sequence
 //   ssd           Mamba-2:  S_t = exp(a dt_t) S_{t-1} + dt_t B_t x_t^T,  y_t = S_t^T C_t + D x_t, one scalar decay per head and token
 //   gla           HGRN2:    S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T,  o_t = S_t^T q_t, one decay per key channel
+//   rwkv          o_t = (S_{t-1} + diag(u) k_t v_t^T)^T r_t,  S_t = diag(w_t) S_{t-1} + k_t v_t^T, w = exp(-exp(z)) per key channel
+//   token_shift   mixes of a token's row and the one in front of it, the last row carried per sequence
+//   tanh_rows     tanh of a projection's result (the middle of a low-rank projection)
 // The state S [dim, vdim] is f32 and lives in a slot per sequence.  The chunked forms for prompts are in lightning_chunk.cu (Mamba-2) and
-// gla_chunk.cu (HGRN2).
+// gla_chunk.cu (HGRN2, RWKV).
 //
 // The step kernel has the layout of lightning.cu: one CTA per (sequence, head, slice of value columns); a lane owns VEC value columns, the eight
 // warps split the key rows, and a decode step is one pass over the state with all of a thread's loads in flight at once.
@@ -107,11 +110,12 @@ causal_conv_kernel(const CausalConvArgs a) {
 struct RecurrentArgs {
   // ssd: activated channels of the convolution [tokens, ld]: [x heads x vdim | B groups x dim | C groups x dim] (one slab)
   // gla: input projection [n_part][tokens, ld]: q heads x dim from column 0, v heads x vdim behind it
+  // rwkv: r, k, v as three blocks of rows [tokens, ld], `part_stride` elements apart (one slab)
   const void* in; int n_part; long part_stride; int ld;
   // the gate's pre-activations, [g_part][tokens, g_ld] f32: dt (heads columns) or f (heads x dim columns)
   const float* gate; int g_part; long g_stride; int g_ld;
-  const float* gate_bias;       // ssd: dt_bias [heads]; gla: [heads * dim]
-  const float* par;             // ssd: a [heads], negative; gla: lower bound [heads * dim]
+  const float* gate_bias;       // ssd: dt_bias [heads]; gla, rwkv: [heads * dim]
+  const float* par;             // ssd: a [heads], negative; gla: lower bound [heads * dim]; rwkv: u [heads * dim]
   const float* d_skip;          // ssd: [heads]
   float* state; int n_slots;    // [slots, heads, dim, vdim]
   const int* cu_q; const int* seq_slots;
@@ -121,7 +125,7 @@ struct RecurrentArgs {
 };
 
 template <typename TI>
-__device__ __forceinline__ float in_col(const RecurrentArgs& a, size_t tok, int col) {
+__device__ __forceinline__ float in_col(const RecurrentArgs& a, size_t tok, long col) {
   const TI* p = (const TI*)a.in + tok * a.ld + col;
   float s = ldv(p);
   for (int i = 1; i < a.n_part; ++i) s += ldv(p + (size_t)i * a.part_stride);
@@ -134,10 +138,13 @@ __device__ __forceinline__ float gate_col(const RecurrentArgs& a, size_t tok, in
   return s;
 }
 
-template <typename TI, bool GLA, int VEC, int R>   // dim <= 8 * R
+enum RecurrentKind { kSsd = 0, kGla = 1, kRwkv = 2 };
+
+template <typename TI, int KIND, int VEC, int R>   // dim <= 8 * R
 __global__ void __launch_bounds__(256)
 recurrent_step_kernel(const RecurrentArgs a) {
-  __shared__ float sq[8 * R], sk[8 * R], sf[GLA ? 8 * R : 1];
+  constexpr bool GLA = KIND == kGla, RWKV = KIND == kRwkv, CHAN = GLA || RWKV;       // CHAN: a decay per key channel
+  __shared__ float sq[8 * R], sk[8 * R], sf[CHAN ? 8 * R : 1], su[RWKV ? 8 * R : 1];
   __shared__ float red[8][32 * VEC];
   __shared__ float s_dec;
   pdl_wait();
@@ -158,12 +165,12 @@ recurrent_step_kernel(const RecurrentArgs a) {
     if (live && d < a.dim) load_cols<VEC>(st + (size_t)d * a.vdim, S[r]);
   }
   const int nv = a.heads * a.vdim, grp = h / (a.heads / a.groups);
-  const int q_col = GLA ? h * a.dim : nv + (a.groups + grp) * a.dim, k_col = nv + grp * a.dim;
-  const int v_col = (GLA ? a.heads * a.dim : 0) + h * a.vdim + e0;
-  const float a_h = GLA ? 0.f : a.par[h], bias_h = GLA ? 0.f : a.gate_bias[h], skip = GLA ? 0.f : a.d_skip[h];
+  const long q_col = CHAN ? h * a.dim : nv + (a.groups + grp) * a.dim, k_col = RWKV ? a.part_stride + h * a.dim : nv + grp * a.dim;
+  const long v_col = (RWKV ? 2 * a.part_stride : GLA ? a.heads * a.dim : 0) + h * a.vdim + e0;
+  const float a_h = CHAN ? 0.f : a.par[h], bias_h = CHAN ? 0.f : a.gate_bias[h], skip = CHAN ? 0.f : a.d_skip[h];
   for (int t = t0; t < t1; ++t) {
     float dt = 0.f;
-    if constexpr (!GLA) {
+    if constexpr (!CHAN) {
       dt = softplus_exact(gate_col(a, t, h) + bias_h);
       if (threadIdx.x == 0) s_dec = expf(a_h * dt);
     }
@@ -178,6 +185,13 @@ recurrent_step_kernel(const RecurrentArgs a) {
           const float q = in_col<TI>(a, t, q_col + c);
           sq[c] = a.q_raw ? q / (1.0f + expf(-q)) : q;
         }
+      } else if constexpr (RWKV) {
+        if (isk) {
+          const float k = in_col<TI>(a, t, k_col + c);
+          sk[c] = k;
+          su[c] = k * a.par[h * a.dim + c];
+          sf[c] = expf(-expf(gate_col(a, t, h * a.dim + c) + a.gate_bias[h * a.dim + c]));
+        } else sq[c] = in_col<TI>(a, t, q_col + c);
       } else {
         if (isk) sk[c] = in_col<TI>(a, t, k_col + c) * dt; else sq[c] = in_col<TI>(a, t, q_col + c);
       }
@@ -189,17 +203,23 @@ recurrent_step_kernel(const RecurrentArgs a) {
     float o[VEC];
 #pragma unroll
     for (int j = 0; j < VEC; ++j) o[j] = 0.f;
-    const float dec = GLA ? 0.f : s_dec;
+    const float dec = CHAN ? 0.f : s_dec;
 #pragma unroll
     for (int r = 0; r < R; ++r) {
       const int d = warp + 8 * r;
       if (d < a.dim) {
-        const float kd = sk[d], qd = sq[d], f = GLA ? sf[GLA ? d : 0] : dec;
+        const float kd = sk[d], qd = sq[d], f = CHAN ? sf[CHAN ? d : 0] : dec;
+        if constexpr (RWKV) {                      // the output reads the state in front of the token
+          const float ud = su[d];
+#pragma unroll
+          for (int j = 0; j < VEC; ++j) { o[j] = fmaf(fmaf(ud, v[j], S[r][j]), qd, o[j]); S[r][j] = fmaf(f, S[r][j], kd * v[j]); }
+          continue;
+        }
 #pragma unroll
         for (int j = 0; j < VEC; ++j) { S[r][j] = fmaf(f, S[r][j], kd * v[j]); o[j] = fmaf(S[r][j], qd, o[j]); }
       }
     }
-    if (!GLA && warp == 0) {
+    if (!CHAN && warp == 0) {
 #pragma unroll
       for (int j = 0; j < VEC; ++j) o[j] = fmaf(skip, v[j], o[j]);
     }
@@ -224,12 +244,12 @@ recurrent_step_kernel(const RecurrentArgs a) {
   }
 }
 
-template <typename TI, bool GLA>
+template <typename TI, int KIND>
 static int recurrent_step_launch(const RecurrentArgs& a, int n_seqs, cudaStream_t stream) {
   const bool vec = a.vdim % 4 == 0 && a.vdim > 32 && a.dim <= 256 && ((uintptr_t)a.state & 15) == 0;
   const int cols = vec ? 128 : 32;
   const dim3 grid((unsigned)a.heads, (unsigned)((a.vdim + cols - 1) / cols), (unsigned)n_seqs);
-#define GB_RS(VECV, RV) launch_k(recurrent_step_kernel<TI, GLA, VECV, RV>, grid, 256, 0, stream, a)
+#define GB_RS(VECV, RV) launch_k(recurrent_step_kernel<TI, KIND, VECV, RV>, grid, 256, 0, stream, a)
   if (vec) {
     if (a.dim <= 32) GB_RS(4, 4); else if (a.dim <= 64) GB_RS(4, 8); else if (a.dim <= 128) GB_RS(4, 16); else GB_RS(4, 32);
   } else {
@@ -238,6 +258,91 @@ static int recurrent_step_launch(const RecurrentArgs& a, int n_seqs, cudaStream_
 #undef GB_RS
   GB_CUDA_OK(cudaGetLastError());
   return 0;
+}
+
+// ------------------------------------------------------------------------------------------ mixes with the token in front
+struct TokenShiftArgs {
+  const void* h; int ld;                                      // [tokens, ld], `width` columns
+  const float* mu; int n;                                     // [n, width]
+  float* state; int n_slots;                                  // [slots, width]: the row in front of a sequence's next token
+  const int* cu_q; const int* seq_slots;
+  void* out; long mix_stride; int ld_out;                     // [n][.., ld_out], zero behind `width`
+  int width;
+};
+
+constexpr int kShiftTile = 8;                                 // tokens per CTA
+
+// V neighbouring columns per thread.  Only a sequence's first tile reads the state, and the same threads write it.
+template <typename T, int V>
+__global__ void __launch_bounds__(128)
+token_shift_kernel(const TokenShiftArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const int c = (blockIdx.x * 128 + threadIdx.x) * V, s = blockIdx.z;
+  const int t0 = a.cu_q[s], t1 = a.cu_q[s + 1];
+  const int tb = t0 + blockIdx.y * kShiftTile, te = min(t1, tb + kShiftTile);
+  const int slot = a.seq_slots[s];
+  if (c >= a.ld_out || tb >= t1 || slot < 0 || slot >= a.n_slots) return;
+  const bool live = c < a.width;                              // V > 1: width % V == 0
+  const T* h = (const T*)a.h + c;
+  float prev[V], cur[V];
+#pragma unroll
+  for (int i = 0; i < V; ++i) prev[i] = cur[i] = 0.f;
+  if (live) {
+    float* st = a.state + (size_t)slot * a.width + c;
+    if (blockIdx.y == 0) {
+      float last[V];
+      load_cols<V>(st, prev);
+      load_cols<V>(h + (size_t)(t1 - 1) * a.ld, last);
+      store_cols<V>(st, last);
+    } else load_cols<V>(h + (size_t)(tb - 1) * a.ld, prev);
+  }
+  for (int t = tb; t < te; ++t) {
+    if (live) load_cols<V>(h + (size_t)t * a.ld, cur);
+    for (int x = 0; x < a.n; ++x) {
+      float m[V];
+#pragma unroll
+      for (int i = 0; i < V; ++i) m[i] = 0.f;
+      if (live) {
+        load_cols<V>(a.mu + (size_t)x * a.width + c, m);
+#pragma unroll
+        for (int i = 0; i < V; ++i) m[i] = fmaf(prev[i] - cur[i], m[i], cur[i]);
+      }
+      store_cols<V>((T*)a.out + (size_t)x * a.mix_stride + (size_t)t * a.ld_out + c, m);
+    }
+#pragma unroll
+    for (int i = 0; i < V; ++i) prev[i] = cur[i];
+  }
+}
+
+template <typename T>
+static int token_shift_launch(const TokenShiftArgs& a, int max_tokens, int n_seqs, cudaStream_t stream) {
+  const size_t es = 4 * sizeof(T);
+  const bool vec = a.width % 4 == 0 && a.ld % 4 == 0 && a.ld_out % 4 == 0 && a.mix_stride % 4 == 0 && (uintptr_t)a.h % es == 0 && (uintptr_t)a.out % es == 0 &&
+                   ((uintptr_t)a.state & 15) == 0 && ((uintptr_t)a.mu & 15) == 0;
+  const int cols = vec ? 512 : 128;
+  const dim3 grid((unsigned)((a.ld_out + cols - 1) / cols), (unsigned)((max_tokens + kShiftTile - 1) / kShiftTile), (unsigned)n_seqs);
+  if (vec) launch_k(token_shift_kernel<T, 4>, grid, 128, 0, stream, a);
+  else launch_k(token_shift_kernel<T, 1>, grid, 128, 0, stream, a);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+template <typename TI, typename TO>
+__global__ void __launch_bounds__(256)
+tanh_rows_kernel(const TI* __restrict__ z, int n_part, long part_stride, int ld, TO* __restrict__ out, int ld_out, long total, int n) {
+  pdl_wait();
+  pdl_trigger();
+  const long i = (long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= total) return;
+  const long r = i / ld_out;
+  const int c = (int)(i - r * ld_out);
+  float v = 0.f;
+  if (c < n) {
+    for (int q = 0; q < n_part; ++q) v += ldv(z + (size_t)q * part_stride + (size_t)r * ld + c);
+    v = tanhf(v);
+  }
+  stv(out + i, v);
 }
 
 template <typename TI, typename TO>
@@ -286,6 +391,50 @@ GB_API int gb_recurrent_step(int gla, const void* in, int in_f32, int n_part, lo
   a.in = in; a.n_part = n_part; a.part_stride = part_stride; a.ld = ld; a.gate = gate; a.g_part = g_part; a.g_stride = g_stride; a.g_ld = g_ld;
   a.gate_bias = gate_bias; a.par = par; a.d_skip = d_skip; a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out;
   a.ld_out = ld_out; a.heads = heads; a.groups = groups; a.dim = dim; a.vdim = vdim; a.q_raw = q_raw;
-  if (gla) return in_f32 ? recurrent_step_launch<float, true>(a, n_seqs, stream) : recurrent_step_launch<__nv_bfloat16, true>(a, n_seqs, stream);
-  return in_f32 ? recurrent_step_launch<float, false>(a, n_seqs, stream) : recurrent_step_launch<__nv_bfloat16, false>(a, n_seqs, stream);
+  if (gla) return in_f32 ? recurrent_step_launch<float, kGla>(a, n_seqs, stream) : recurrent_step_launch<__nv_bfloat16, kGla>(a, n_seqs, stream);
+  return in_f32 ? recurrent_step_launch<float, kSsd>(a, n_seqs, stream) : recurrent_step_launch<__nv_bfloat16, kSsd>(a, n_seqs, stream);
+}
+
+// r, k, v: three blocks [tokens, ld] of one element type, `block_stride` elements apart; z [z_part][tokens, z_ld]: w = exp(-exp(z + w0)); u, w0 [heads * dim].  See
+// RecurrentArgs for the rest.
+GB_API int gb_rwkv_step(const void* rkv, int in_f32, long block_stride, int ld, const float* z, int z_part, long z_stride, int z_ld, const float* w0, const float* u,
+                        float* state, int n_slots, const int* cu_q, const int* seq_slots, float* out, int ld_out, int heads, int dim, int vdim, int n_seqs, cudaStream_t stream) {
+  if (n_seqs <= 0) return 0;
+  if (heads < 1 || dim < 1 || vdim < 1 || z_part < 1 || ld_out < heads * vdim || ld < heads * dim || ld < heads * vdim || z_ld < heads * dim) return fail("rwkv: bad sizes%s");
+  if (dim > 512) return fail("rwkv: a key dimension of at most 512%s");
+  if (n_seqs > 65535) return fail("rwkv: too many sequences%s");
+  RecurrentArgs a;
+  memset(&a, 0, sizeof(a));
+  a.in = rkv; a.n_part = 1; a.part_stride = block_stride; a.ld = ld; a.gate = z; a.g_part = z_part; a.g_stride = z_stride; a.g_ld = z_ld; a.gate_bias = w0; a.par = u;
+  a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out; a.ld_out = ld_out; a.heads = heads; a.groups = 1; a.dim = dim; a.vdim = vdim;
+  return in_f32 ? recurrent_step_launch<float, kRwkv>(a, n_seqs, stream) : recurrent_step_launch<__nv_bfloat16, kRwkv>(a, n_seqs, stream);
+}
+
+// See TokenShiftArgs.  max_tokens: of the longest sequence.
+GB_API int gb_token_shift(const void* h, int h_f32, int ld, int width, const float* mu, int n, float* state, int n_slots, const int* cu_q, const int* seq_slots, void* out,
+                          long mix_stride, int ld_out, int max_tokens, int n_seqs, cudaStream_t stream) {
+  if (n_seqs <= 0 || max_tokens <= 0) return 0;
+  if (width < 1 || n < 1 || ld < width || ld_out < width) return fail("token_shift: bad sizes%s");
+  if (n_seqs > 65535 || (max_tokens + kShiftTile - 1) / kShiftTile > 65535) return fail("token_shift: too many tokens%s");
+  TokenShiftArgs a;
+  a.h = h; a.ld = ld; a.mu = mu; a.n = n; a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out; a.mix_stride = mix_stride;
+  a.ld_out = ld_out; a.width = width;
+  return h_f32 ? token_shift_launch<float>(a, max_tokens, n_seqs, stream) : token_shift_launch<__nv_bfloat16>(a, max_tokens, n_seqs, stream);
+}
+
+// out [rows, ld_out] = tanh of the first n columns of z [n_part][rows, ld], zero behind.
+GB_API int gb_tanh_rows(const void* z, int z_f32, int n_part, long part_stride, int ld, void* out, int out_f32, int ld_out, int rows, int n, cudaStream_t stream) {
+  const long total = (long)rows * ld_out;
+  if (total <= 0) return 0;
+  if (n < 1 || n_part < 1 || ld < n || ld_out < n) return fail("tanh_rows: bad sizes%s");
+  const unsigned grid = (unsigned)((total + 255) / 256);
+  if (z_f32) {
+    if (out_f32) launch_k(tanh_rows_kernel<float, float>, grid, 256, 0, stream, (const float*)z, n_part, part_stride, ld, (float*)out, ld_out, total, n);
+    else launch_k(tanh_rows_kernel<float, __nv_bfloat16>, grid, 256, 0, stream, (const float*)z, n_part, part_stride, ld, (__nv_bfloat16*)out, ld_out, total, n);
+  } else {
+    if (out_f32) return fail("tanh_rows: 32-bit results take 32-bit rows%s");
+    launch_k(tanh_rows_kernel<__nv_bfloat16, __nv_bfloat16>, grid, 256, 0, stream, (const __nv_bfloat16*)z, n_part, part_stride, ld, (__nv_bfloat16*)out, ld_out, total, n);
+  }
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
 }

@@ -4,10 +4,14 @@
 //                       every row], then RMSNorm of the row with an f32 weight -> bf16 or f32 rows for the next projection
 //   stream_dyt          the same with Dynamic Tanh, tanh(alpha x) w + b, in place of the norm, and one of its own over the update, which
 //                       may also be the router-weighted sum of expert outputs (formed here)
+//   stream_rms2         stream_norm for an update with an RMSNorm of its own, a row added per token, and a second set of normalised rows
+//   stream_join         stream += factor * result, for up to three pending results; a copy of the rows for a projection of the stream itself
 //   qk_unit_store       fused Q | K | V rows -> Q / K divided by their root mean square per head (no weight), K / V into their
 //                       cache slots, Q scaled and laid out for the attention kernels
 //   gated_norm          RMSNorm over all heads' outputs together, times sigmoid(gate): the tail of a linear-attention mixer
-//   part_norm           RMSNorm of equal parts of a row, after SiLU(gate) if there is one: the tail of Mamba-2 and HGRN2 mixers
+//   part_norm           RMSNorm of equal parts of a row, after (or before) SiLU(gate) if there is one: the tail of Mamba-2, HGRN2 and RWKV mixers
+//   sigmoid_gate        the heads' outputs of an attention, times sigmoid(gate)
+//   token_gate          GELU(z) times a row of a table, by token
 //   act_mul             act(gate) * up of f32 rows (the 32-bit path; the bf16 path has it in the GEMM epilogue)
 // One pass over HBM each; sizes are arbitrary (vector paths when they divide).  Output rows may be wider than the data (padding to
 // the 16-byte row pitch the TMA descriptors of the next GEMM need); the padding is written as zero.
@@ -147,6 +151,261 @@ stream_norm_any_kernel(const StreamNormArgs a) {
   TO* o = (TO*)a.out + r * a.ld_out;
   for (int c = threadIdx.x; c < a.width; c += 256) st_f(o + c, (in_place ? x[c] : value(c)) * inv * a.weight[c]);
   for (int c = a.width + threadIdx.x; c < a.ld_out; c += 256) st_f(o + c, 0.f);
+}
+
+// ------------------------------------------------------------------------------------------ stream norm, normed update, two outputs
+struct StreamRms2Args {
+  float* x;                     // stream [rows, width]
+  const void* delta; int n_part; long part_stride; int ld_delta;   // as in StreamNormArgs
+  const float* post_w; float post_eps;                             // the update is divided by its root mean square and multiplied by this (null: added as it is)
+  const float* add;             // [rows, width], added after the update; null = none
+  const float* w[2];            // weights of the two outputs
+  const long long* rows;        // as in StreamNormArgs
+  void* out[2]; int ld_out;     // out[1] null = one output
+  int width; float eps;
+};
+
+template <typename TD, typename TO, int VPT>       // VPT float4 per thread, width <= 1024 * VPT and width % 4 == 0
+__global__ void __launch_bounds__(256)
+stream_rms2_vec_kernel(const StreamRms2Args a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[2][8];
+  const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
+  float* x = a.x + src * a.width;
+  const int nv = a.width >> 2;
+  float4 v[VPT], u[VPT];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * 256;
+    v[i] = u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < nv) v[i] = ld4(x + c * 4);
+  }
+  if (a.delta != nullptr) {
+    const TD* d = (const TD*)a.delta + src * a.ld_delta;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * 256;
+      if (c >= nv) continue;
+      u[i] = ld4(d + c * 4);
+      for (int p = 1; p < a.n_part; ++p) {
+        const float4 q = ld4(d + (size_t)p * a.part_stride + c * 4);
+        u[i].x += q.x; u[i].y += q.y; u[i].z += q.z; u[i].w += q.w;
+      }
+      ss += u[i].x * u[i].x + u[i].y * u[i].y + u[i].z * u[i].z + u[i].w * u[i].w;
+    }
+    const bool post = a.post_w != nullptr;
+    const float inv = post ? 1.0f / sqrtf(block_sum_256(ss, red[0]) / (float)a.width + a.post_eps) : 1.0f;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * 256;
+      if (c >= nv) continue;
+      const float4 w = post ? ld4(a.post_w + c * 4) : make_float4(1.f, 1.f, 1.f, 1.f);
+      v[i].x += u[i].x * inv * w.x; v[i].y += u[i].y * inv * w.y; v[i].z += u[i].z * inv * w.z; v[i].w += u[i].w * inv * w.w;
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = threadIdx.x + i * 256;
+    if (c >= nv) continue;
+    if (a.add != nullptr) {
+      const float4 q = ld4(a.add + src * a.width + c * 4);
+      v[i].x += q.x; v[i].y += q.y; v[i].z += q.z; v[i].w += q.w;
+    }
+    if (a.rows == nullptr && (a.delta != nullptr || a.add != nullptr)) st4(x + c * 4, v[i]);
+    ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+  }
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red[1]) / (float)a.width + a.eps);
+#pragma unroll
+  for (int y = 0; y < 2; ++y) {
+    if (a.out[y] == nullptr) continue;
+    TO* o = (TO*)a.out[y] + r * a.ld_out;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = threadIdx.x + i * 256;
+      if (c >= nv) continue;
+      const float4 w = ld4(a.w[y] + c * 4);
+      st4(o + c * 4, make_float4(v[i].x * inv * w.x, v[i].y * inv * w.y, v[i].z * inv * w.z, v[i].w * inv * w.w));
+    }
+    for (int c = a.width + threadIdx.x; c < a.ld_out; c += 256) st_f(o + c, 0.f);
+  }
+}
+
+template <typename TD, typename TO>                // any width
+__global__ void __launch_bounds__(256)
+stream_rms2_any_kernel(const StreamRms2Args a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[2][8];
+  const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
+  float* x = a.x + src * a.width;
+  const TD* d = a.delta != nullptr ? (const TD*)a.delta + src * a.ld_delta : nullptr;
+  auto update = [&](int c) {
+    float s = ld_f(d + c);
+    for (int p = 1; p < a.n_part; ++p) s += ld_f(d + (size_t)p * a.part_stride + c);
+    return s;
+  };
+  float ud = 1.0f;
+  if (d != nullptr && a.post_w != nullptr) {
+    float ss = 0.f;
+    for (int c = threadIdx.x; c < a.width; c += 256) { const float u = update(c); ss += u * u; }
+    ud = 1.0f / sqrtf(block_sum_256(ss, red[0]) / (float)a.width + a.post_eps);
+  }
+  auto value = [&](int c) {
+    float v = x[c];
+    if (d != nullptr) v += update(c) * ud * (a.post_w != nullptr ? a.post_w[c] : 1.0f);
+    if (a.add != nullptr) v += a.add[src * a.width + c];
+    return v;
+  };
+  const bool in_place = a.rows == nullptr;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < a.width; c += 256) {
+    const float v = value(c);
+    if (in_place) x[c] = v;
+    ss += v * v;
+  }
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red[1]) / (float)a.width + a.eps);
+  for (int c = threadIdx.x; c < a.ld_out; c += 256) {
+    const float v = c < a.width ? (in_place ? x[c] : value(c)) * inv : 0.f;
+    for (int y = 0; y < 2; ++y)
+      if (a.out[y] != nullptr) st_f((TO*)a.out[y] + r * a.ld_out + c, c < a.width ? v * a.w[y][c] : 0.f);
+  }
+}
+
+// ------------------------------------------------------------------------------------------ several pending results into the stream
+struct JoinPart {               // mirrored by ops/stream.py
+  const void* p;                // f32 / bf16 [n_part][rows, ld], or expert outputs [*, ld] when pair_row is set
+  const int* pair_row; const float* weights;         // as in DytArgs
+  long stride;
+  int f32, n_part, ld, k;
+  float scale;
+};
+struct JoinArgs {
+  float* x;
+  JoinPart part[3]; int n;
+  void* out; int ld_out;        // copy of the new rows (null = none), zero behind `width`
+  int width;
+};
+
+template <typename TO, int V>                      // V neighbouring columns per thread
+__global__ void __launch_bounds__(256)
+stream_join_kernel(const JoinArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const size_t r = blockIdx.x;
+  const int c = (blockIdx.y * 256 + threadIdx.x) * V;
+  if (c >= a.width) {                              // padding (V == 4: width % 4 == 0)
+    if (a.out != nullptr) {
+#pragma unroll
+      for (int i = 0; i < V; ++i) if (c + i < a.ld_out) st_f((TO*)a.out + r * a.ld_out + c + i, 0.f);
+    }
+    return;
+  }
+  float x[V];
+  auto load = [&](const auto* p, float* v) {
+    if constexpr (V == 4) { const float4 q = ld4(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+    else v[0] = ld_f(p);
+  };
+  load(a.x + r * a.width + c, x);
+#pragma unroll
+  for (int i = 0; i < 3; ++i) {
+    if (i >= a.n) break;
+    const JoinPart& d = a.part[i];
+    float u[V];
+#pragma unroll
+    for (int j = 0; j < V; ++j) u[j] = 0.f;
+    auto add = [&](size_t off, float w) {
+      float q[V];
+      if (d.f32) load((const float*)d.p + off + c, q); else load((const __nv_bfloat16*)d.p + off + c, q);
+#pragma unroll
+      for (int j = 0; j < V; ++j) u[j] = fmaf(w, q[j], u[j]);
+    };
+    if (d.pair_row != nullptr) {
+      for (int e = 0; e < d.k; ++e) {
+        const int row = d.pair_row[r * d.k + e];
+        if (row >= 0) add((size_t)row * d.ld, d.weights[r * d.k + e]);
+      }
+    } else {
+      for (int p = 0; p < d.n_part; ++p) add((size_t)p * d.stride + r * d.ld, 1.0f);
+    }
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[j] = fmaf(d.scale, u[j], x[j]);
+  }
+  if constexpr (V == 4) {
+    const float4 y = make_float4(x[0], x[1], x[2], x[3]);
+    st4(a.x + r * a.width + c, y);
+    if (a.out != nullptr) st4((TO*)a.out + r * a.ld_out + c, y);
+  } else {
+    a.x[r * a.width + c] = x[0];
+    if (a.out != nullptr) st_f((TO*)a.out + r * a.ld_out + c, x[0]);
+  }
+}
+
+// ------------------------------------------------------------------------------------------ gates
+struct HeadGateArgs {
+  void* a;                      // [rows, heads, dvp], in place
+  const void* gate; int n_part; long part_stride; int ld_gate;     // pre-activations [n_part][rows, ld_gate]: heads x dv columns
+  long n; int heads, dv, dvp;
+};
+
+template <typename TA, typename TG, int V>         // V neighbouring values of a head per thread
+__global__ void __launch_bounds__(256)
+sigmoid_gate_kernel(const HeadGateArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const long i = (long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= a.n) return;
+  const int per = a.dv / V;
+  const long rh = i / per;                         // row * heads + head
+  const int c = (int)(i - rh * per) * V;
+  const long r = rh / a.heads;
+  const int h = (int)(rh - r * a.heads);
+  TA* p = (TA*)a.a + (size_t)rh * a.dvp + c;
+  const TG* g = (const TG*)a.gate + (size_t)r * a.ld_gate + (size_t)h * a.dv + c;
+  if constexpr (V == 4) {
+    float4 z = ld4(g);
+    for (int q = 1; q < a.n_part; ++q) {
+      const float4 y = ld4(g + (size_t)q * a.part_stride);
+      z.x += y.x; z.y += y.y; z.z += y.z; z.w += y.w;
+    }
+    const float4 v = ld4(p);
+    st4(p, make_float4(v.x / (1.0f + expf(-z.x)), v.y / (1.0f + expf(-z.y)), v.z / (1.0f + expf(-z.z)), v.w / (1.0f + expf(-z.w))));
+  } else {
+    float z = ld_f(g);
+    for (int q = 1; q < a.n_part; ++q) z += ld_f(g + (size_t)q * a.part_stride);
+    st_f(p, ld_f(p) / (1.0f + expf(-z)));
+  }
+}
+
+struct TokenGateArgs {
+  const void* z; int n_part; long part_stride; int ld_z;           // [n_part][rows, ld_z]
+  const int* ids; const void* table; int table_f32, ld_t, col, vocab;
+  void* out; int ld_out; long total; int n;
+};
+
+template <typename TZ, typename TO>
+__global__ void __launch_bounds__(256)
+token_gate_kernel(const TokenGateArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  const long i = (long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= a.total) return;
+  const long r = i / a.ld_out;
+  const int c = (int)(i - r * a.ld_out);
+  float y = 0.f;
+  if (c < a.n) {
+    const TZ* p = (const TZ*)a.z + (size_t)r * a.ld_z + c;
+    float z = ld_f(p);
+    for (int q = 1; q < a.n_part; ++q) z += ld_f(p + (size_t)q * a.part_stride);
+    int id = a.ids[r];
+    if (id < 0 || id >= a.vocab) id = 0;
+    const size_t off = (size_t)id * a.ld_t + a.col + c;
+    const float e = a.table_f32 ? ((const float*)a.table)[off] : __bfloat162float(((const __nv_bfloat16*)a.table)[off]);
+    y = 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))) * e;
+  }
+  st_f((TO*)a.out + i, y);
 }
 
 // ------------------------------------------------------------------------------------------ stream with Dynamic Tanh
@@ -370,6 +629,7 @@ gated_norm_any_kernel(const GatedNormArgs a) {
 struct PartNormArgs {
   const float* o; int ld_o;     // [rows, n] f32
   const void* gate; int n_part; long part_stride; int ld_gate;     // gate pre-activations (null = none)
+  int gate_after;               // the gate multiplies the normalised values instead of the values
   const float* weight; int n_weight;   // f32, column c uses weight[c % n_weight]
   void* out; int ld_out; int n, parts; float eps; long items;
 };
@@ -405,8 +665,9 @@ part_norm_vec_kernel(const PartNormArgs a) {
         const float4 q = ld4(g + (size_t)p * a.part_stride + c * 4);
         z[i].x += q.x; z[i].y += q.y; z[i].z += q.z; z[i].w += q.w;
       }
-      v[i].x *= z[i].x / (1.0f + expf(-z[i].x)); v[i].y *= z[i].y / (1.0f + expf(-z[i].y));
-      v[i].z *= z[i].z / (1.0f + expf(-z[i].z)); v[i].w *= z[i].w / (1.0f + expf(-z[i].w));
+      z[i].x /= 1.0f + expf(-z[i].x); z[i].y /= 1.0f + expf(-z[i].y);
+      z[i].z /= 1.0f + expf(-z[i].z); z[i].w /= 1.0f + expf(-z[i].w);
+      if (!a.gate_after) { v[i].x *= z[i].x; v[i].y *= z[i].y; v[i].z *= z[i].z; v[i].w *= z[i].w; }
     }
     ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
   }
@@ -420,7 +681,8 @@ part_norm_vec_kernel(const PartNormArgs a) {
   for (int i = 0; i < VPT; ++i) {
     const int c = lane + i * G;
     if (c >= nv) continue;
-    const float4 q = ld4(w + c * 4);
+    float4 q = ld4(w + c * 4);
+    if (a.gate_after) { q.x *= z[i].x; q.y *= z[i].y; q.z *= z[i].z; q.w *= z[i].w; }
     st4(out + c0 + c * 4, make_float4(v[i].x * inv * q.x, v[i].y * inv * q.y, v[i].z * inv * q.z, v[i].w * inv * q.w));
   }
   if (part == a.parts - 1)
@@ -442,15 +704,12 @@ part_norm_kernel(const PartNormArgs a) {
   const int len = a.n / a.parts, c0 = part * len;
   const float* o = a.o + (size_t)r * a.ld_o + c0;
   const TG* g = a.gate != nullptr ? (const TG*)a.gate + (size_t)r * a.ld_gate + c0 : nullptr;
-  auto value = [&](int c) {
-    float v = o[c];
-    if (g != nullptr) {
-      float z = ld_f(g + c);
-      for (int p = 1; p < a.n_part; ++p) z += ld_f(g + (size_t)p * a.part_stride + c);
-      v *= z / (1.0f + expf(-z));
-    }
-    return v;
+  auto gate = [&](int c) {
+    float z = ld_f(g + c);
+    for (int p = 1; p < a.n_part; ++p) z += ld_f(g + (size_t)p * a.part_stride + c);
+    return z / (1.0f + expf(-z));
   };
+  auto value = [&](int c) { return g != nullptr && !a.gate_after ? o[c] * gate(c) : o[c]; };
   float keep[kKeep];
   float ss = 0.f;
   if (live) {
@@ -463,7 +722,7 @@ part_norm_kernel(const PartNormArgs a) {
   if (!live) return;
   const float inv = 1.0f / sqrtf(ss / (float)len + a.eps);
   TO* out = (TO*)a.out + (size_t)r * a.ld_out;
-  auto w = [&](int c) { return a.weight[(c0 + c) % a.n_weight]; };
+  auto w = [&](int c) { return a.weight[(c0 + c) % a.n_weight] * (a.gate_after ? gate(c) : 1.0f); };
 #pragma unroll
   for (int i = 0; i < kKeep; ++i) { const int c = lane + i * G; if (c < len) st_f(out + c0 + c, keep[i] * inv * w(c)); }
   for (int c = lane + kKeep * G; c < len; c += G) st_f(out + c0 + c, value(c) * inv * w(c));
@@ -472,14 +731,19 @@ part_norm_kernel(const PartNormArgs a) {
 }
 
 // ------------------------------------------------------------------------------------------ act(gate) * up, f32
-__global__ void act_mul_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, long n, int inter, int ld, int act) {
+__global__ void act_mul_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, long n, int inter, int ld, int act, float cap) {
   pdl_wait();
   pdl_trigger();
   const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n) return;
   const long r = i / inter;
   const int c = (int)(i - r * inter);
-  const float g = gu[r * ld + c], u = gu[r * ld + inter + c];
+  float g = gu[r * ld + c], u = gu[r * ld + inter + c];
+  if (act == 2) {
+    g = fminf(g, cap);
+    out[r * inter + c] = g / (1.0f + expf(-1.702f * g)) * (fminf(fmaxf(u, -cap), cap) + 1.0f);
+    return;
+  }
   const float y = act == 1 ? 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) : g / (1.0f + expf(-g));
   out[r * inter + c] = y * u;
 }
@@ -571,12 +835,13 @@ static int part_norm_launch(const PartNormArgs& a, cudaStream_t stream) {
 }
 
 GB_API int gb_part_norm(const float* o, int ld_o, const void* gate, int gate_f32, int n_part, long part_stride, int ld_gate, const float* weight, int n_weight,
-                        void* out, int out_f32, int ld_out, int rows, int n, int parts, float eps, cudaStream_t stream) {
+                        void* out, int out_f32, int ld_out, int rows, int n, int parts, float eps, int gate_after, cudaStream_t stream) {
   if (rows <= 0) return 0;
+  if (gate_after && gate == nullptr) return fail("part_norm: no gate%s");
   if (n < 1 || parts < 1 || n % parts || n_weight < 1 || n % n_weight || ld_o < n || ld_out < n || n_part < 1) return fail("part_norm: bad sizes%s");
   PartNormArgs a;
   a.o = o; a.ld_o = ld_o; a.gate = gate; a.n_part = n_part; a.part_stride = part_stride; a.ld_gate = ld_gate; a.weight = weight; a.n_weight = n_weight;
-  a.out = out; a.ld_out = ld_out; a.n = n; a.parts = parts; a.eps = eps; a.items = (long)rows * parts;
+  a.out = out; a.ld_out = ld_out; a.n = n; a.parts = parts; a.eps = eps; a.items = (long)rows * parts; a.gate_after = gate_after;
   if (gate_f32) return out_f32 ? part_norm_launch<float, float>(a, stream) : part_norm_launch<float, __nv_bfloat16>(a, stream);
   return out_f32 ? part_norm_launch<__nv_bfloat16, float>(a, stream) : part_norm_launch<__nv_bfloat16, __nv_bfloat16>(a, stream);
 }
@@ -625,11 +890,104 @@ GB_API int gb_gated_norm(const float* o, int ld_o, const void* gate, int gate_f3
   return out_f32 ? gated_norm_launch<__nv_bfloat16, float>(a, rows, stream) : gated_norm_launch<__nv_bfloat16, __nv_bfloat16>(a, rows, stream);
 }
 
-// act(gate) * up over f32 rows [gate | up]; act 0 = SiLU, 1 = the tanh form of GELU.
-GB_API int gb_act_mul_f32(const float* gate_up, float* out, long rows, int inter, int ld, int act, cudaStream_t stream) {
+// act(gate) * up over f32 rows [gate | up]; act 0 = SiLU, 1 = the tanh form of GELU, 2 = g sigmoid(1.702 g) (u + 1), bounded by cap.
+GB_API int gb_act_mul_f32(const float* gate_up, float* out, long rows, int inter, int ld, int act, float cap, cudaStream_t stream) {
   const long n = rows * inter;
   if (n <= 0) return 0;
-  launch_k(act_mul_f32_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, gate_up, out, n, inter, ld, act);
+  launch_k(act_mul_f32_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, gate_up, out, n, inter, ld, act, cap);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+template <typename TD, typename TO>
+static int stream_rms2_launch(const StreamRms2Args& a, int n_rows, cudaStream_t stream) {
+  const size_t ed = sizeof(TD) * 4, eo = sizeof(TO) * 4;
+  const auto ok16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  const bool vec = a.width % 4 == 0 && a.width <= 16384 && (a.delta == nullptr || (a.ld_delta % 4 == 0 && a.part_stride % 4 == 0 && (uintptr_t)a.delta % ed == 0)) &&
+                   a.ld_out % 4 == 0 && (uintptr_t)a.out[0] % eo == 0 && (uintptr_t)a.out[1] % eo == 0 && ok16(a.x) && ok16(a.w[0]) && ok16(a.w[1]) && ok16(a.post_w) && ok16(a.add);
+  if (!vec) launch_k(stream_rms2_any_kernel<TD, TO>, (unsigned)n_rows, 256, 0, stream, a);
+  else if (a.width <= 1024) launch_k(stream_rms2_vec_kernel<TD, TO, 1>, (unsigned)n_rows, 256, 0, stream, a);
+  else if (a.width <= 2048) launch_k(stream_rms2_vec_kernel<TD, TO, 2>, (unsigned)n_rows, 256, 0, stream, a);
+  else if (a.width <= 4096) launch_k(stream_rms2_vec_kernel<TD, TO, 4>, (unsigned)n_rows, 256, 0, stream, a);
+  else launch_k(stream_rms2_vec_kernel<TD, TO, 16>, (unsigned)n_rows, 256, 0, stream, a);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// See StreamRms2Args.
+GB_API int gb_stream_rms2(float* x, const void* delta, int delta_f32, int n_part, long part_stride, int ld_delta, const float* post_w, float post_eps, const float* add,
+                          const float* w0, const float* w1, const long long* rows, void* out0, void* out1, int out_f32, int ld_out, int n_rows, int width, float eps,
+                          cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (width <= 0 || out0 == nullptr || w0 == nullptr || (out1 != nullptr && w1 == nullptr) || ld_out < width || (delta != nullptr && (ld_delta < width || n_part < 1)))
+    return fail("stream_rms2: bad arguments%s");
+  StreamRms2Args a;
+  a.x = x; a.delta = delta; a.n_part = n_part; a.part_stride = part_stride; a.ld_delta = ld_delta; a.post_w = post_w; a.post_eps = post_eps; a.add = add;
+  a.w[0] = w0; a.w[1] = w1; a.rows = rows; a.out[0] = out0; a.out[1] = out1; a.ld_out = ld_out; a.width = width; a.eps = eps;
+  if (delta_f32) return out_f32 ? stream_rms2_launch<float, float>(a, n_rows, stream) : stream_rms2_launch<float, __nv_bfloat16>(a, n_rows, stream);
+  return out_f32 ? stream_rms2_launch<__nv_bfloat16, float>(a, n_rows, stream) : stream_rms2_launch<__nv_bfloat16, __nv_bfloat16>(a, n_rows, stream);
+}
+
+// x [n_rows, width] += sum of parts[0 .. n - 1] (host array of three); out: see JoinArgs.
+GB_API int gb_stream_join(float* x, const JoinPart* parts, int n, void* out, int out_f32, int ld_out, int n_rows, int width, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (width <= 0 || n < 1 || n > 3 || (out != nullptr && ld_out < width)) return fail("stream_join: bad sizes%s");
+  JoinArgs a;
+  bool vec = width % 4 == 0 && ((uintptr_t)x & 15) == 0 && (out == nullptr || (ld_out % 4 == 0 && (uintptr_t)out % (out_f32 ? 16 : 8) == 0));
+  for (int i = 0; i < 3; ++i) {
+    a.part[i] = parts[i];
+    if (i >= n) continue;
+    const JoinPart& d = parts[i];
+    if (d.p == nullptr || d.ld < width || d.n_part < 1 || (d.pair_row != nullptr && (d.weights == nullptr || d.k < 1))) return fail("stream_join: bad part%s");
+    vec = vec && d.ld % 4 == 0 && d.stride % 4 == 0 && (uintptr_t)d.p % (d.f32 ? 16 : 8) == 0;
+  }
+  a.x = x; a.n = n; a.out = out; a.ld_out = ld_out; a.width = width;
+  const int cols = out != nullptr ? ld_out : width;
+  const dim3 grid((unsigned)n_rows, (unsigned)((cols + (vec ? 1023 : 255)) / (vec ? 1024 : 256)));
+  if (out_f32) { if (vec) launch_k(stream_join_kernel<float, 4>, grid, 256, 0, stream, a); else launch_k(stream_join_kernel<float, 1>, grid, 256, 0, stream, a); }
+  else { if (vec) launch_k(stream_join_kernel<__nv_bfloat16, 4>, grid, 256, 0, stream, a); else launch_k(stream_join_kernel<__nv_bfloat16, 1>, grid, 256, 0, stream, a); }
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+template <typename TA, typename TG>
+static int sigmoid_gate_launch(HeadGateArgs a, long rows, cudaStream_t stream) {
+  const bool vec = a.dv % 4 == 0 && a.dvp % 4 == 0 && a.ld_gate % 4 == 0 && a.part_stride % 4 == 0 && (uintptr_t)a.a % (4 * sizeof(TA)) == 0 && (uintptr_t)a.gate % (4 * sizeof(TG)) == 0;
+  a.n = rows * a.heads * (a.dv / (vec ? 4 : 1));
+  const unsigned grid = (unsigned)((a.n + 255) / 256);
+  if (vec) launch_k(sigmoid_gate_kernel<TA, TG, 4>, grid, 256, 0, stream, a);
+  else launch_k(sigmoid_gate_kernel<TA, TG, 1>, grid, 256, 0, stream, a);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// See HeadGateArgs.
+GB_API int gb_sigmoid_gate(void* a_, int a_f32, const void* gate, int gate_f32, int n_part, long part_stride, int ld_gate, int rows, int heads, int dv, int dvp,
+                           cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (heads < 1 || dv < 1 || dvp < dv || n_part < 1 || ld_gate < heads * dv) return fail("sigmoid_gate: bad sizes%s");
+  HeadGateArgs a;
+  a.a = a_; a.gate = gate; a.n_part = n_part; a.part_stride = part_stride; a.ld_gate = ld_gate; a.heads = heads; a.dv = dv; a.dvp = dvp; a.n = 0;
+  if (a_f32) return gate_f32 ? sigmoid_gate_launch<float, float>(a, rows, stream) : sigmoid_gate_launch<float, __nv_bfloat16>(a, rows, stream);
+  return gate_f32 ? sigmoid_gate_launch<__nv_bfloat16, float>(a, rows, stream) : sigmoid_gate_launch<__nv_bfloat16, __nv_bfloat16>(a, rows, stream);
+}
+
+// out [rows, ld_out] = gelu(z) * table[ids[row], col ...], zero behind n columns.
+GB_API int gb_token_gate(const void* z, int z_f32, int n_part, long part_stride, int ld_z, const int* ids, const void* table, int table_f32, int ld_t, int col, int vocab,
+                         void* out, int out_f32, int ld_out, int rows, int n, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (n < 1 || ld_out < n || ld_z < n || n_part < 1 || col < 0 || col + n > ld_t || vocab < 1) return fail("token_gate: bad sizes%s");
+  TokenGateArgs a;
+  a.z = z; a.n_part = n_part; a.part_stride = part_stride; a.ld_z = ld_z; a.ids = ids; a.table = table; a.table_f32 = table_f32; a.ld_t = ld_t; a.col = col; a.vocab = vocab;
+  a.out = out; a.ld_out = ld_out; a.n = n; a.total = (long)rows * ld_out;
+  const unsigned grid = (unsigned)((a.total + 255) / 256);
+  if (z_f32) {
+    if (out_f32) launch_k(token_gate_kernel<float, float>, grid, 256, 0, stream, a);
+    else launch_k(token_gate_kernel<float, __nv_bfloat16>, grid, 256, 0, stream, a);
+  } else {
+    if (out_f32) launch_k(token_gate_kernel<__nv_bfloat16, float>, grid, 256, 0, stream, a);
+    else launch_k(token_gate_kernel<__nv_bfloat16, __nv_bfloat16>, grid, 256, 0, stream, a);
+  }
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }

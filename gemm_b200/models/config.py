@@ -14,7 +14,7 @@ from dataclasses import asdict, dataclass, field, replace
 from typing import Dict, List, Optional
 
 # Architectures described layer by layer (``ModelConfig.layer_specs``): name in config.json -> arch
-LAYERED_ARCHS = {"Zogavik": "zogavik", "Famepel": "famepel"}
+LAYERED_ARCHS = {"Zogavik": "zogavik", "Famepel": "famepel", "Fidolix": "fidolix"}
 
 ARCHS = ("qwen2", "qwen2vl", "qwen3", "qwen3vl", "qwen3moe", "qwen3vlmoe", "qwen35", "qwen35moe")
 
@@ -52,7 +52,7 @@ class RotarySpec:
 @dataclass
 class MoeSpec:
     """A mixture of experts: gated feed-forwards of width ``ffn``, ``top`` of ``n_experts`` per token.  ``groups`` > 1: the experts form groups of
-    neighbours, a group scores the sum of its two best experts, and only the best ``groups_kept`` groups can be chosen from."""
+    neighbours, a group scores the sum of its ``group_best`` (1 or 2) best experts, and only the best ``groups_kept`` groups can be chosen from."""
     n_experts: int
     top: int
     ffn: int
@@ -61,12 +61,13 @@ class MoeSpec:
     scale: float = 1.0
     groups: int = 1
     groups_kept: int = 1
+    group_best: int = 2
 
 
 @dataclass
 class LayerSpec:
     """One layer of a model described layer by layer: its mixer with the mixer's own sizes, and its feed-forward."""
-    mixer: str                              # "attention" | "lightning" | "mamba2" | "hgrn2" | "latent"
+    mixer: str                              # "attention" | "lightning" | "mamba2" | "hgrn2" | "latent" | "rwkv" | "parallel"
     n_heads: int
     head_dim: int                           # query / key size per head (mamba2: the state size; latent: without the rotated part)
     v_dim: int                              # value size per head
@@ -79,12 +80,23 @@ class LayerSpec:
     keep_first: int = 0                     # ... or j < keep_first
     rel_buckets: int = 0                    # rows of the learned distance-bias table (0 = none)
     rel_max: float = 0                      # distance from which the last bucket holds
+    qk_norm_rows: bool = False              # RMS norm with weights over all of q, and over all of k
+    softcap: float = 0.0                    # scores become softcap * tanh(score / softcap) (0 = as they are)
+    out_gate: bool = False                  # the heads' outputs are multiplied by the sigmoid of a projection
+    v_from_k: bool = False                  # the values are the keys before their rotation
     # lightning attention
     decay: Optional[List[float]] = None     # per head
     # mamba2
     state_groups: int = 1                   # heads share B and C by groups
-    conv_taps: int = 0                      # causal convolution in front of the recurrence
+    conv_taps: int = 0                      # causal convolution in front of the recurrence (attention: of q and k, in front of the rotation)
     norm_parts: int = 1                     # the output norm's equal parts
+    # rwkv: a decay per key channel through a low-rank projection of the input
+    decay_rank: int = 0
+    # parallel: two mixers side by side over the same input, left_scale * left + right_scale * right
+    left: Optional["LayerSpec"] = None
+    right: Optional["LayerSpec"] = None
+    left_scale: float = 1.0
+    right_scale: float = 1.0
     # latent attention: keys and values are projections of a cached latent, next to one rotated key part for all heads
     kv_rank: int = 0
     q_rank: int = 0
@@ -94,7 +106,8 @@ class LayerSpec:
     kv_from: int = -1                       # layer whose cache this one reads (-1: its own)
     # feed-forward: act(gate) * up -> down; 0 = none
     ffn: int = 0
-    act: str = "silu"                       # or "gelu_tanh"
+    act: str = "silu"                       # or "gelu_tanh", "capped" (x sigmoid(1.702 x) of min(gate, cap), times 1 + up within +-cap)
+    act_cap: float = 0.0
     moe: Optional[MoeSpec] = None           # in place of the dense feed-forward
 
     def __post_init__(self):
@@ -102,6 +115,15 @@ class LayerSpec:
             self.rotary = RotarySpec(**self.rotary)
         if isinstance(self.moe, dict):
             self.moe = MoeSpec(**self.moe)
+        if isinstance(self.left, dict):
+            self.left = LayerSpec(**self.left)
+        if isinstance(self.right, dict):
+            self.right = LayerSpec(**self.right)
+
+    @property
+    def mixers(self) -> List["LayerSpec"]:
+        """The mixer itself, or the two of a parallel one."""
+        return [self.left, self.right] if self.mixer == "parallel" else [self]
 
     @property
     def q_dim(self) -> int:
@@ -113,12 +135,19 @@ class LayerSpec:
 
     @property
     def has_state(self) -> bool:
-        """Whether the mixer carries recurrent state (in place of cache pages)."""
-        return self.mixer in ("lightning", "mamba2", "hgrn2")
+        """Whether the mixer carries state of a fixed size per sequence, which cannot drop positions."""
+        return any(x.mixer in ("lightning", "mamba2", "hgrn2", "rwkv") or x.conv_taps > 1 for x in self.mixers)
+
+    @property
+    def paged(self) -> Optional["LayerSpec"]:
+        """The mixer that keeps keys and values in cache pages."""
+        return next((x for x in self.mixers if x.mixer in ("attention", "latent")), None)
 
     @property
     def conv_channels(self) -> int:
-        """Channels of the convolution: [x heads x v_dim | B groups x head_dim | C groups x head_dim]."""
+        """Channels of the convolution: [x heads x v_dim | B groups x head_dim | C groups x head_dim], attention: [q heads | k heads]."""
+        if self.mixer == "attention":
+            return (self.n_heads + self.n_kv_heads) * self.head_dim
         return self.n_heads * self.v_dim + 2 * self.state_groups * self.head_dim
 
     @property
@@ -129,19 +158,21 @@ class LayerSpec:
 
 @dataclass
 class LoopSpec:
-    """Layers ``start .. stop - 1`` run ``times`` times in a row with the same weights; every pass has its own cache or state, and
-    a learned vector is added to the stream in front of each pass."""
+    """Layers ``start .. stop - 1`` run ``times`` times in a row with the same weights; every pass has its own cache or state.  ``add`` "step": a
+    learned vector is added to the stream in front of each pass; "embedding": the embedding output, in front of each but the first."""
     start: int
     stop: int
     times: int
+    add: str = "step"
 
 
 @dataclass(frozen=True)
 class LayerRun:
     """One execution of a layer: ``layer`` is its index in the weights, ``step`` the row of the step-vector table added in front of it
-    (-1 = none).  The position of the run in ``ModelConfig.layer_runs`` is the index of its cache."""
+    (-1 = none), ``again`` whether the embedding output is.  The position of the run in ``ModelConfig.layer_runs`` is the index of its cache."""
     layer: int
     step: int = -1
+    again: bool = False
 
 
 @dataclass
@@ -188,6 +219,8 @@ class ModelConfig:
     norm_kind: str = "rms"                  # or "dyt": tanh(alpha x) w + b
     post_norm: bool = False                 # every sublayer's result passes a norm of its own and a per-channel scale
     embed_scale: float = 1.0
+    parallel_ffn: bool = False              # mixer and feed-forward read the same stream, each through a norm of its own
+    side_dim: int = 0                       # per-layer token input of this size (a table of the token's vectors for all layers), 0 = none
 
     def __post_init__(self):
         if self.layer_specs is not None:
@@ -209,12 +242,13 @@ class ModelConfig:
             raise ValueError(f"bad layer loop {lp} for {n} layers")
         runs = [LayerRun(i) for i in range(lp.start)]
         for t in range(lp.times):
-            runs += [LayerRun(i, t if i == lp.start else -1) for i in range(lp.start, lp.stop)]
+            emb, first = lp.add == "embedding", lp.start
+            runs += [LayerRun(i, t if i == first and not emb else -1, emb and i == first and t > 0) for i in range(lp.start, lp.stop)]
         return runs + [LayerRun(i) for i in range(lp.stop, n)]
 
     @property
     def has_recurrent_state(self) -> bool:
-        """Whether a sequence carries state that cannot drop positions (Delta-Net, lightning, Mamba-2 or HGRN2 layers)."""
+        """Whether a sequence carries state that cannot drop positions (Delta-Net, lightning, Mamba-2, HGRN2 or RWKV layers, convolutions)."""
         return self.is_hybrid or (self.is_layered and any(x.has_state for x in self.layer_specs))
 
     @property
@@ -248,11 +282,13 @@ class ModelConfig:
 
     def param_count(self) -> int:
         if self.is_layered:
-            tot = self.vocab * self.hidden * (1 if self.tie_embeddings else 2)
+            tot = self.vocab * self.hidden * (1 if self.tie_embeddings else 2) + self.vocab * self.n_layers * self.side_dim
             for x in self.layer_specs:
-                nv = x.n_heads * x.v_dim
                 if x.moe is not None:
                     tot += x.moe.n_experts * self.hidden * (3 * x.moe.ffn + 1)
+                tot += 3 * self.hidden * x.ffn + 2 * self.hidden * self.side_dim
+            for x in (m for sp in self.layer_specs for m in sp.mixers):
+                nv = x.n_heads * x.v_dim
                 if x.mixer == "lightning":
                     tot += self.hidden * (2 * x.q_dim + 3 * nv)
                 elif x.mixer == "hgrn2":
@@ -262,9 +298,10 @@ class ModelConfig:
                 elif x.mixer == "latent":
                     own = 0 if x.kv_from >= 0 else x.kv_rank + x.rot_dim
                     tot += self.hidden * (x.q_rank + own + nv) + x.q_rank * x.n_heads * (x.head_dim + x.rot_dim) + x.kv_rank * (x.q_dim + nv)
+                elif x.mixer == "rwkv":
+                    tot += self.hidden * (2 * x.q_dim + 3 * nv + x.decay_rank) + x.q_dim * x.decay_rank
                 else:
-                    tot += self.hidden * (x.q_dim + x.n_kv_heads * (x.head_dim + x.v_dim) + x.n_heads * x.v_dim)
-                tot += 3 * self.hidden * x.ffn
+                    tot += self.hidden * (x.q_dim + x.n_kv_heads * (x.head_dim + (0 if x.v_from_k else x.v_dim)) + (2 if x.out_gate else 1) * nv)
             return tot
         per_layer = self.hidden * (self.q_dim + 2 * self.kv_dim) + self.q_dim * self.hidden
         if self.is_moe:
@@ -359,6 +396,32 @@ PRESETS["tiny-famepel"] = _famepel("MHLMS", 192, 300, MoeSpec(10, 3, 48, "sigmoi
 # layers of the sizes of a 30-billion-parameter mixture of experts (128 experts, 8 per token)
 PRESETS["famepel-30b-a3b"] = _famepel("HMLHMMHMS" * 5, 2048, 151936, MoeSpec(128, 8, 768, "sigmoid", True, 2.5, 8, 4), (16, 128, 128), (64, 128, 64, 8, 4, 8),
                                       (32, 128, 64, 128, 512, 1536), RotarySpec(64, 500000.0, 8.0, 4096, 32.0, 1.0))
+
+
+def _fidolix(pattern: str, hidden: int, vocab: int, side_dim: int, att, left, right, rotary: RotarySpec, window: int, taps: int, cap: float, dense: int, act_cap: float, moe: MoeSpec,
+             embed_scale: float, scales=(1.0, 1.0), loop: Optional[LoopSpec] = None) -> ModelConfig:
+    """``pattern``: one letter per layer, A = attention, P = windowed attention beside an RWKV recurrence, with a mixture of experts; a, p = with a dense
+    feed-forward.  ``att`` (heads, KV heads, dim, vdim), ``left`` (heads, KV heads, dim), ``right`` (heads, dim, decay rank)."""
+    specs: List[LayerSpec] = []
+    for c in pattern:
+        ff = dict(ffn=dense, act="capped", act_cap=act_cap) if c.islower() else dict(moe=moe)
+        if c in "Aa":
+            hd, g, d, v = att
+            specs.append(LayerSpec("attention", hd, d, v, n_kv_heads=g, scale=d ** -0.5, qkv_bias=True, qk_norm_rows=True, softcap=cap, out_gate=True, **ff))
+        else:
+            hd, g, d = left
+            lt = LayerSpec("attention", hd, d, d, n_kv_heads=g, scale=d ** -0.5, qkv_bias=True, v_from_k=True, conv_taps=taps, rotary=rotary, window=window, sink=True)
+            rt = LayerSpec("rwkv", right[0], right[1], right[1], decay_rank=right[2])
+            specs.append(LayerSpec("parallel", hd, d, d, n_kv_heads=g, left=lt, right=rt, left_scale=scales[0], right_scale=scales[1], **ff))
+    return ModelConfig(arch="fidolix", layer_specs=specs, hidden=hidden, n_heads=att[0], n_kv_heads=att[1], head_dim=att[2], ffn=dense, vocab=vocab, rms_eps=1e-5,
+                       embed_scale=embed_scale, parallel_ffn=True, side_dim=side_dim, qk_norm=False, loop=loop)
+
+
+PRESETS["tiny-fidolix"] = _fidolix("pAPa", 192, 300, 20, (4, 2, 40, 24), (6, 3, 32), (3, 24, 12), RotarySpec(24, 10000.0, 4.0, 64, 32.0, 1.0), 50, 4, 20.0, 320, 1.5,
+                                   MoeSpec(12, 3, 48, renorm=True, groups=4, groups_kept=2, group_best=1), 3.0, (0.7, 1.2), LoopSpec(1, 3, 2, "embedding"))
+# layers of the sizes of a 30-billion-parameter mixture of experts (128 experts, 8 per token), every third one attention without a window
+PRESETS["fidolix-30b-a3b"] = _fidolix("pPA" + "PPA" * 14, 2048, 151936, 128, (32, 4, 128, 128), (16, 2, 128), (16, 128, 64), RotarySpec(64, 500000.0, 8.0, 4096, 32.0, 1.0),
+                                      1024, 4, 30.0, 6144, 7.0, MoeSpec(128, 8, 768, renorm=True, groups=8, groups_kept=4, group_best=1), 2048 ** 0.5)
 
 
 def get_config(name: str) -> ModelConfig:

@@ -520,8 +520,9 @@ def _qwen35_config_from_hf(c: dict) -> ModelConfig:
 
 
 class LayeredSource(SafetensorsSource):
-    """Checkpoints of models described layer by layer: tensors ``l<i>.norm1``, ``l<i>.mix.*``, ``l<i>.norm2``, ``l<i>.mlp.*``, ``embed``,
-    ``final.norm``, ``loop.step``, served under the names the model builder asks for."""
+    """Checkpoints of models described layer by layer: tensors ``l<i>.norm1``, ``l<i>.mix.*`` (``l<i>.mix.left.*`` and ``l<i>.mix.right.*`` for two mixers side
+    by side), ``l<i>.norm2``, ``l<i>.mlp.*``, ``l<i>.side.*``, ``embed``, ``side.embed``, ``final.norm``, ``loop.step``, served under the names the model
+    builder asks for."""
 
     _LAYER = {"attn_q.weight": "mix.q", "attn_k.weight": "mix.k", "attn_v.weight": "mix.v",
               "attn_q.bias": "mix.q.b", "attn_k.bias": "mix.k.b", "attn_v.bias": "mix.v.b", "attn_output.weight": "mix.o", "attn_rel.weight": "mix.rel",
@@ -533,11 +534,16 @@ class LayeredSource(SafetensorsSource):
               "gla_q.weight": "mix.q", "gla_f.weight": "mix.f", "gla_f.bias": "mix.f.b", "gla_lower": "mix.lower", "gla_v.weight": "mix.v", "gla_norm.weight": "mix.norm",
               "gla_out.weight": "mix.o",
               "attn_q_a.weight": "mix.dq", "attn_q_a_norm.weight": "mix.dq.norm", "attn_q_b.weight": "mix.uq", "attn_kv_a.weight": "mix.dkv",
-              "attn_kv_a_norm.weight": "mix.dkv.norm", "attn_k_b.weight": "mix.uk", "attn_v_b.weight": "mix.uv", "attn_sink": "mix.sink"}
+              "attn_kv_a_norm.weight": "mix.dkv.norm", "attn_k_b.weight": "mix.uk", "attn_v_b.weight": "mix.uv", "attn_sink": "mix.sink",
+              "attn_q.conv": "mix.q.conv", "attn_k.conv": "mix.k.conv", "attn_q_rows.norm": "mix.q.norm", "attn_k_rows.norm": "mix.k.norm", "attn_gate.weight": "mix.g",
+              "rwkv_r.weight": "mix.r", "rwkv_k.weight": "mix.k", "rwkv_v.weight": "mix.v", "rwkv_g.weight": "mix.g", "rwkv_mu_r": "mix.mu.r", "rwkv_mu_k": "mix.mu.k",
+              "rwkv_mu_v": "mix.mu.v", "rwkv_mu_g": "mix.mu.g", "rwkv_mu_w": "mix.mu.w", "rwkv_w1.weight": "mix.w1", "rwkv_w2.weight": "mix.w2", "rwkv_w0": "mix.w0",
+              "rwkv_u": "mix.u", "rwkv_norm.weight": "mix.norm", "rwkv_out.weight": "mix.o",
+              "side_gate.weight": "side.gate", "side_proj.weight": "side.proj", "side_norm.weight": "side.norm"}
     _NORM = {"attn_norm": "norm1", "attn_post_norm": "norm1b", "ffn_norm": "norm2", "ffn_post_norm": "norm2b", "output_norm": "final.norm"}
     _PART = {"weight": "", "bias": ".b", "alpha": ".alpha"}
     _EXPERT = {"ffn_gate_exps.weight": "gate", "ffn_up_exps.weight": "up", "ffn_down_exps.weight": "down"}
-    _TOP = {"token_embd.weight": "embed", "loop_step.weight": "loop.step", "output.weight": "head"}
+    _TOP = {"token_embd.weight": "embed", "loop_step.weight": "loop.step", "output.weight": "head", "side_embd.weight": "side.embed"}
 
     @classmethod
     def file_name(cls, name: str) -> str:
@@ -553,6 +559,9 @@ class LayeredSource(SafetensorsSource):
         if rest.partition("#")[0] in cls._EXPERT:              # "<name>#<expert>"
             rest, _, e = rest.partition("#")
             return f"{pre}mlp.e{e}.{cls._EXPERT[rest]}"
+        for part in ("left.", "right."):
+            if rest.startswith(part):
+                return pre + cls._LAYER[rest[len(part):]].replace("mix.", "mix." + part, 1)
         return pre + cls._LAYER[rest]
 
     def get_expert(self, name: str, e: int, shape) -> torch.Tensor:
@@ -575,10 +584,10 @@ class LayeredSource(SafetensorsSource):
         return t
 
 
-def _moe_spec(mlp: dict) -> MoeSpec:
+def _moe_spec(mlp: dict, **rule) -> MoeSpec:
+    """``rule``: what the design fixes of the routing."""
     r, g = mlp["router"], mlp["router"].get("groups") or {"count": 1, "keep": 1}
-    spec = MoeSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), router="sigmoid", renorm=True, scale=float(r["scale"]), groups=int(g["count"]),
-                   groups_kept=int(g["keep"]))
+    spec = MoeSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), renorm=True, groups=int(g["count"]), groups_kept=int(g["keep"]), **rule)
     if spec.groups < 1 or spec.n_experts % spec.groups or not 1 <= spec.groups_kept <= spec.groups:
         raise ValueError(f"router groups: {spec.n_experts} experts in {spec.groups} groups, {spec.groups_kept} kept")
     if not 1 <= spec.top <= spec.n_experts // spec.groups * spec.groups_kept:
@@ -586,11 +595,16 @@ def _moe_spec(mlp: dict) -> MoeSpec:
     return spec
 
 
+def _rotary_spec(r: dict) -> RotarySpec:
+    sc = r.get("scaling")
+    return RotarySpec(int(r["dims"]), float(r["base"]), *((float(sc[k]) for k in ("factor", "original", "fast", "slow")) if sc else ()))
+
+
 def _famepel_layer(li: int, e: dict, layers: list) -> LayerSpec:
     m, mlp = e["mixer"], e.get("mlp")
     if mlp is not None and mlp.get("kind") != "moe":
         raise ValueError(f"layer {li}: feed-forward kind {mlp.get('kind')!r} is not supported")
-    moe = _moe_spec(mlp) if mlp is not None else None
+    moe = _moe_spec(mlp, router="sigmoid", scale=float(mlp["router"]["scale"])) if mlp is not None else None
     heads, v = int(m["heads"]), int(m["vdim"])
     if e["type"] == "hgrn2":
         return LayerSpec("hgrn2", heads, int(m["dim"]), v, moe=moe)
@@ -600,9 +614,7 @@ def _famepel_layer(li: int, e: dict, layers: list) -> LayerSpec:
             raise ValueError(f"layer {li}: {heads} heads in {g} groups, norm over {parts} parts of {heads * v}")
         return LayerSpec("mamba2", heads, int(m["state"]), v, state_groups=g, conv_taps=int(m["conv"]), norm_parts=parts, moe=moe)
     if e["type"] == "latent_attention":
-        r = m["rot"]
-        sc = r.get("scaling")
-        rot = RotarySpec(int(r["dims"]), float(r["base"]), *((float(sc[k]) for k in ("factor", "original", "fast", "slow")) if sc else ()))
+        rot = _rotary_spec(m["rot"])
         if rot.dims != int(m["rot_dim"]):
             raise ValueError(f"layer {li}: rotation over {rot.dims} of {m['rot_dim']} dimensions is not supported")
         src = m.get("kv_from")
@@ -625,9 +637,56 @@ def _famepel_config(c: dict) -> ModelConfig:
                        norm_kind="dyt", post_norm=True, embed_scale=float(c["embedding"]["scale"]))
 
 
+def _loop_spec(c: dict, add: str) -> Optional[LoopSpec]:
+    lp = c.get("loop")
+    return LoopSpec(int(lp["start"]), int(lp["stop"]), int(lp["times"]), add) if lp else None
+
+
+def _fidolix_layer(li: int, e: dict, src: "LayeredSource") -> LayerSpec:
+    m, mlp = e["mixer"], e.get("mlp")
+    ff = {}
+    if mlp is not None:
+        if mlp.get("kind") == "dense":
+            ff = dict(ffn=int(mlp["ff"]), act="capped", act_cap=float(mlp["limit"]))
+        elif mlp.get("kind") == "moe":
+            ff = dict(moe=_moe_spec(mlp, router="softmax", group_best=1))
+        else:
+            raise ValueError(f"layer {li}: feed-forward kind {mlp.get('kind')!r} is not supported")
+    att = m["left"] if e["type"] == "parallel" else m
+    if e["type"] not in ("attention", "parallel"):
+        raise ValueError(f"layer {li}: mixer {e['type']!r} is not supported")
+    heads, g, d, v = (int(att[k]) for k in ("heads", "kv_heads", "dim", "vdim"))
+    if g < 1 or heads % g:
+        raise ValueError(f"layer {li}: {heads} query heads over kv_heads {g}")
+    if e["type"] == "attention":
+        return LayerSpec("attention", heads, d, v, n_kv_heads=g, scale=float(m["scale"]), qkv_bias=True, qk_norm_rows=True, softcap=float(m["softcap"]), out_gate=True, **ff)
+    rot, mask, r = _rotary_spec(att["rot"]), att.get("mask") or {}, m["right"]
+    if v != d:
+        raise ValueError(f"layer {li}: the values are the keys, but vdim is {v} and dim {d}")
+    if rot.dims % 2 or not 0 < rot.dims <= d:
+        raise ValueError(f"layer {li}: rotation over {rot.dims} of {d} dimensions")
+    left = LayerSpec("attention", heads, d, d, n_kv_heads=g, scale=float(att["scale"]), qkv_bias=True, v_from_k=True, conv_taps=int(att["conv"]), rotary=rot,
+                     window=int(mask.get("size") or 0), sink=True)
+    right = LayerSpec("rwkv", int(r["heads"]), int(r["dim"]), int(r["dim"]), decay_rank=int(src.shape(f"blk.{li}.right.rwkv_w1.weight")[0]))
+    return LayerSpec("parallel", heads, d, d, n_kv_heads=g, left=left, right=right, left_scale=float(m["left_scale"]), right_scale=float(m["right_scale"]), **ff)
+
+
+def _fidolix_config(c: dict, path: str) -> ModelConfig:
+    """config.json of Fidolix: gated attention with capped scores, windowed attention with sinks beside an RWKV recurrence, dense or mixture-of-experts
+    feed-forwards next to the mixer, a token input per layer, a looped range of layers that sees the embedding again."""
+    src = LayeredSource(path)
+    specs = [_fidolix_layer(li, e, src) for li, e in enumerate(c["layers"])]
+    att = next((s for s in specs if s.mixer == "attention"), specs[0])
+    return ModelConfig(arch=LAYERED_ARCHS[c["architecture"]], layer_specs=specs, hidden=int(c["width"]), vocab=int(c["vocab"]), n_heads=att.n_heads, n_kv_heads=att.n_kv_heads,
+                       head_dim=att.head_dim, ffn=max(s.ffn for s in specs), rms_eps=float(c["norm"]["eps"]), qk_norm=False, embed_scale=float(c["embedding"]["scale"]),
+                       parallel_ffn=True, side_dim=int(c["token_side"]["dim"]), loop=_loop_spec(c, "embedding"))
+
+
 def _layered_config(c: dict, path: str) -> ModelConfig:
     if c["architecture"] == "Famepel":
         return _famepel_config(c)
+    if c["architecture"] == "Fidolix":
+        return _fidolix_config(c, path)
     return _zogavik_config(c, path)
 
 
@@ -655,12 +714,11 @@ def _zogavik_config(c: dict, path: str) -> ModelConfig:
                                    rel_buckets=int(src.shape(f"blk.{li}.attn_rel.weight")[0]), rel_max=float(m["bias_max"]), ffn=ff, act="gelu_tanh"))
         else:
             raise ValueError(f"layer {li}: mixer {e['type']!r} is not supported")
-    lp = c.get("loop")
     att = next((s for s in specs if s.mixer == "attention"), specs[0])
     return ModelConfig(arch=LAYERED_ARCHS[c["architecture"]], layer_specs=specs, hidden=int(c["width"]), vocab=int(c["vocab"]), n_heads=att.n_heads,
                        n_kv_heads=max(1, att.n_kv_heads), head_dim=att.head_dim, ffn=max(s.ffn for s in specs), rms_eps=float(c["norm"]["eps"]),
                        tie_embeddings=True, qk_norm=False, qkv_bias=True, norm_offset=1.0, logit_scale=float(c.get("logit_scale", 1.0)),
-                       loop=LoopSpec(int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else None)
+                       loop=_loop_spec(c, "step"))
 
 
 def config_from_hf(path: str) -> ModelConfig:
@@ -779,8 +837,10 @@ def _save_layered(cfg: ModelConfig, src, path: str) -> None:
     put_norm("output_norm")
     if not cfg.tie_embeddings:
         put("output.weight", (cfg.vocab, h))
-    if cfg.loop is not None:
+    if cfg.loop is not None and cfg.loop.add == "step":
         put("loop_step.weight", (cfg.loop.times, h))
+    if cfg.side_dim:
+        put("side_embd.weight", (cfg.vocab, cfg.n_layers * cfg.side_dim))
     layers = []
     for li, sp in enumerate(cfg.layer_specs):
         p = f"blk.{li}."
@@ -790,8 +850,11 @@ def _save_layered(cfg: ModelConfig, src, path: str) -> None:
                 if cfg.post_norm:
                     put_norm(p + nm + "_post_norm")
                     put(p + nm + "_post_scale.weight", (h,))
-        for nm, shp in mixer_tensors(sp, h):
-            put(p + nm, shp)
+        for part, mx in zip(("left.", "right.") if sp.mixer == "parallel" else ("",), sp.mixers):
+            for nm, shp in mixer_tensors(mx, h):
+                put(p + part + nm, shp)
+        if cfg.side_dim:
+            put(p + "side_gate.weight", (cfg.side_dim, h)); put(p + "side_proj.weight", (h, cfg.side_dim)); put(p + "side_norm.weight", (h,))
         if sp.ffn:
             put(p + "ffn_gate.weight", (sp.ffn, h)); put(p + "ffn_up.weight", (sp.ffn, h)); put(p + "ffn_down.weight", (h, sp.ffn))
         if sp.moe is not None:
@@ -804,11 +867,14 @@ def _save_layered(cfg: ModelConfig, src, path: str) -> None:
     save_safetensors(out, os.path.join(path, "model.safetensors"))
     name = {v: k for k, v in LAYERED_ARCHS.items()}[cfg.arch]
     c = {"architecture": name, "layers": layers, "vocab": cfg.vocab, "width": h, "norm": {"eps": cfg.rms_eps}}
-    if cfg.arch == "famepel":
+    if cfg.arch in ("famepel", "fidolix"):
         c["embedding"] = {"scale": cfg.embed_scale}
-    else:
+    if cfg.arch == "zogavik":
         c["logit_scale"] = cfg.logit_scale
+    if cfg.arch in ("zogavik", "fidolix"):
         c["loop"] = {"start": cfg.loop.start, "stop": cfg.loop.stop, "times": cfg.loop.times} if cfg.loop else None
+    if cfg.side_dim:
+        c["token_side"] = {"dim": cfg.side_dim}
     with open(os.path.join(path, "config.json"), "w") as fh:
         json.dump(c, fh)
 
@@ -831,10 +897,24 @@ def mixer_tensors(sp: LayerSpec, h: int):
         return own + [("attn_q_a.weight", (sp.q_rank, h)), ("attn_q_a_norm.weight", (sp.q_rank,)),
                       ("attn_q_b.weight", (sp.n_heads * (sp.head_dim + sp.rot_dim), sp.q_rank)), ("attn_k_b.weight", (nq, sp.kv_rank)),
                       ("attn_v_b.weight", (nv, sp.kv_rank)), ("attn_sink", (sp.n_heads,)), ("attn_output.weight", (h, nv))]
-    own = []
-    for c, n in (("q", nq), ("k", sp.n_kv_heads * sp.head_dim), ("v", sp.n_kv_heads * sp.v_dim)):
+    if sp.mixer == "rwkv":
+        own = [(f"rwkv_{c}.weight", (nq if c in "rk" else nv, h)) for c in "rkvg"] + [(f"rwkv_mu_{c}", (h,)) for c in "rkvgw"]
+        return own + [("rwkv_w1.weight", (sp.decay_rank, h)), ("rwkv_w2.weight", (nq, sp.decay_rank)), ("rwkv_w0", (nq,)), ("rwkv_u", (sp.n_heads, sp.head_dim)),
+                      ("rwkv_norm.weight", (nv,)), ("rwkv_out.weight", (h, nv))]
+    own, nk = [], sp.n_kv_heads * sp.head_dim
+    for c, n in (("q", nq), ("k", nk)) + ((() if sp.v_from_k else (("v", sp.n_kv_heads * sp.v_dim),))):
         own += [(f"attn_{c}.weight", (n, h)), (f"attn_{c}.bias", (n,))]
-    return own + [("attn_rel.weight", (sp.rel_buckets, sp.n_heads)), ("attn_output.weight", (h, nv))]
+    if sp.conv_taps:
+        own += [("attn_q.conv", (nq, sp.conv_taps)), ("attn_k.conv", (nk, sp.conv_taps))]
+    if sp.qk_norm_rows:
+        own += [("attn_q_rows.norm", (nq,)), ("attn_k_rows.norm", (nk,))]
+    if sp.out_gate:
+        own.append(("attn_gate.weight", (nv, h)))
+    if sp.sink:
+        own.append(("attn_sink", (sp.n_heads,)))
+    if sp.rel_buckets:
+        own.append(("attn_rel.weight", (sp.rel_buckets, sp.n_heads)))
+    return own + [("attn_output.weight", (h, nv))]
 
 
 def _mixer_config(sp: LayerSpec) -> dict:
@@ -846,19 +926,34 @@ def _mixer_config(sp: LayerSpec) -> dict:
     if sp.mixer == "mamba2":
         return {**m, "state": sp.head_dim, "groups": sp.state_groups, "conv": sp.conv_taps, "norm_groups": sp.norm_parts}
     if sp.mixer == "latent":
-        r = sp.rotary
-        rot = {"dims": r.dims, "base": r.base}
-        if r.factor > 0:
-            rot["scaling"] = {"factor": r.factor, "original": r.original, "fast": r.fast, "slow": r.slow}
-        m = {**m, "dim": sp.head_dim, "rot_dim": sp.rot_dim, "kv_rank": sp.kv_rank, "q_rank": sp.q_rank, "scale": sp.scale, "rot": rot}
+        m = {**m, "dim": sp.head_dim, "rot_dim": sp.rot_dim, "kv_rank": sp.kv_rank, "q_rank": sp.q_rank, "scale": sp.scale, "rot": _rotary_config(sp.rotary)}
         return {**m, "kv_from": sp.kv_from} if sp.kv_from >= 0 else m
-    return {**m, "kv_heads": sp.n_kv_heads, "dim": sp.head_dim, "scale": sp.scale, "bias_max": sp.rel_max,
-            "mask": {"size": sp.window, "keep_first": sp.keep_first} if sp.window else None}
+    if sp.mixer == "parallel":
+        return {"left": _mixer_config(sp.left), "right": _mixer_config(sp.right), "left_scale": sp.left_scale, "right_scale": sp.right_scale}
+    if sp.mixer == "rwkv":
+        return {"heads": sp.n_heads, "dim": sp.head_dim}
+    m = {**m, "kv_heads": sp.n_kv_heads, "dim": sp.head_dim, "scale": sp.scale}
+    if sp.softcap:
+        return {**m, "softcap": sp.softcap}
+    if sp.conv_taps:
+        return {**m, "conv": sp.conv_taps, "rot": _rotary_config(sp.rotary), "mask": {"size": sp.window} if sp.window else None}
+    return {**m, "bias_max": sp.rel_max, "mask": {"size": sp.window, "keep_first": sp.keep_first} if sp.window else None}
+
+
+def _rotary_config(r: RotarySpec) -> dict:
+    rot = {"dims": r.dims, "base": r.base}
+    if r.factor > 0:
+        rot["scaling"] = {"factor": r.factor, "original": r.original, "fast": r.fast, "slow": r.slow}
+    return rot
 
 
 def _ffn_config(sp: LayerSpec):
     if sp.moe is not None:
         r = sp.moe
-        return {"kind": "moe", "expert": {"ff": r.ffn}, "router": {"experts": r.n_experts, "top": r.top, "scale": r.scale,
-                                                                  "groups": {"count": r.groups, "keep": r.groups_kept}}}
-    return {"kind": "dense", "ff": sp.ffn} if sp.ffn else None
+        rt = {"experts": r.n_experts, "top": r.top, "groups": {"count": r.groups, "keep": r.groups_kept}}
+        if r.router == "sigmoid":
+            rt["scale"] = r.scale
+        return {"kind": "moe", "expert": {"ff": r.ffn}, "router": rt}
+    if not sp.ffn:
+        return None
+    return {"kind": "dense", "ff": sp.ffn, "limit": sp.act_cap} if sp.act == "capped" else {"kind": "dense", "ff": sp.ffn}

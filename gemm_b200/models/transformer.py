@@ -12,10 +12,10 @@ Layer recipe (reference: common/transformer.h:3550-4174):
                   MoE  : softmax router -> top-k -> renormalise; x += sum_k w_k FFN_k(h)  [EP dispatch / combine]
   logits = RMSNorm(x) Whead^T on the last token of every sequence.
 
-Models described layer by layer (``ModelConfig.layer_specs``) run through the same loop: every layer names its mixer (windowed
-attention with kept first tokens and a distance bias, latent attention, lightning attention, HGRN2 or Mamba-2) and its feed-forward (dense or
-a mixture of experts) with sizes of its own, layers may be looped (every run has its own cache: ``KvCache`` is indexed by run), and the
-residual stream is f32.
+Models described layer by layer (``ModelConfig.layer_specs``) run through the same loop: every layer names its mixer (attention with a window, kept
+first tokens, a distance bias, capped scores or sinks, latent attention, lightning attention, HGRN2, Mamba-2, RWKV, or two of them side by side)
+and its feed-forward (dense or a mixture of experts) with sizes of its own, layers may be looped (every run has its own cache: ``KvCache`` is
+indexed by run), and the residual stream is f32.  The feed-forward follows the mixer, or reads the same stream beside it (``parallel_ffn``).
 """
 from __future__ import annotations
 
@@ -45,9 +45,11 @@ class KvCache:
     page_size: int
     num_pages: int
     # Delta-Net layers of the hybrid models keep a fixed-size state per sequence slot instead of K/V pages:
-    # conv[l] f32 [slots, conv_k - 1, qkv_dim], rec[l] f32 [slots, heads_v, d, d] (None for attention layers)
+    # conv[l] f32 [slots, conv_k - 1, qkv_dim], rec[l] f32 [slots, heads_v, d, d] (None for attention layers); shift[l] f32 [slots, 1, hidden]: the
+    # row of the token in front (mixers that shift tokens)
     conv: Optional[List[Optional[torch.Tensor]]] = None
     rec: Optional[List[Optional[torch.Tensor]]] = None
+    shift: Optional[List[Optional[torch.Tensor]]] = None
     # INT8 mode (``kv_dtype="int8"``): the pages live in ``kq`` / ``vq`` (int8 ``[slots, Hkv, D]``) with one f32 scale per slot and
     # head in ``ks`` / ``vs`` (the format of ops.attention.kv_store_q8), read directly by the INT8 decode attention kernel.  ``k`` /
     # ``v`` then name ONE bf16 staging buffer shared by all layers: the QK-norm + RoPE kernel writes a step's new rows there, the
@@ -100,38 +102,41 @@ class KvCache:
     @staticmethod
     def _allocate_layered(cfg: ModelConfig, num_pages: int, page_size: int, device, n_seq_slots: int, kv_dtype: str) -> "KvCache":
         """One entry per layer RUN: K / V pages with the layer's own head sizes (attention); pages of latents and rotated key parts in ``k`` (latent
-        attention; nothing for a layer that reads another's); or ``rec`` f32 ``[slots, heads, dim, vdim]``, for Mamba-2 also ``conv`` f32 ``[slots,
-        taps - 1, channels]`` (recurrent layers)."""
+        attention; nothing for a layer that reads another's); ``rec`` f32 ``[slots, heads, dim, vdim]`` (recurrent mixers); ``conv`` f32 ``[slots, taps - 1,
+        channels]`` (Mamba-2, attention behind a convolution); ``shift`` f32 ``[slots, 1, hidden]`` (RWKV)."""
         dtypes = {"bf16": torch.bfloat16, "f32": torch.float32}
         if kv_dtype not in dtypes:
             raise ValueError(f"models described layer by layer keep a bf16 or f32 KV cache, not {kv_dtype!r}")
         dt = dtypes[kv_dtype]
         kv = KvCache([], [], page_size, num_pages)
-        kv.rec, kv.conv = [], []
+        kv.rec, kv.conv, kv.shift = [], [], []
+        f32 = dict(dtype=torch.float32, device=device)
         for run in cfg.layer_runs():
-            sp = cfg.layer_specs[run.layer]
-            dkp, dvp = att.cache_head_dims(sp.head_dim, sp.v_dim, dt)
-            rows, heads = (0, 1) if sp.has_state else (num_pages * page_size, sp.n_kv_heads)
-            if sp.mixer == "latent":
-                rows, dkp, dvp = (rows if sp.kv_from < 0 else 0), stream.row_width(sp.kv_rank + sp.rot_dim, dt), 0
+            spec = cfg.layer_specs[run.layer]
+            sp, rows, heads, dkp, dvp = spec.paged, 0, 1, 0, 0
+            if sp is not None and sp.mixer == "latent":
+                rows, dkp = (num_pages * page_size if sp.kv_from < 0 else 0), stream.row_width(sp.kv_rank + sp.rot_dim, dt)
+            elif sp is not None:
+                rows, heads, (dkp, dvp) = num_pages * page_size, sp.n_kv_heads, att.cache_head_dims(sp.head_dim, sp.v_dim, dt)
             kv.k.append(torch.zeros(rows, heads, dkp, dtype=dt, device=device))
             kv.v.append(torch.zeros(rows, heads, dvp, dtype=dt, device=device))
-            f32 = dict(dtype=torch.float32, device=device)
-            kv.rec.append(torch.zeros(n_seq_slots, sp.n_heads, sp.head_dim, sp.v_dim, **f32) if sp.has_state else None)
-            kv.conv.append(torch.zeros(n_seq_slots, sp.conv_taps - 1, sp.conv_channels, **f32) if sp.mixer == "mamba2" else None)
-        if not any(r is not None for r in kv.rec):
-            kv.rec = None
-        if not any(r is not None for r in kv.conv):
-            kv.conv = None
+            rec = next((x for x in spec.mixers if x.mixer in ("lightning", "mamba2", "hgrn2", "rwkv")), None)
+            conv = next((x for x in spec.mixers if x.conv_taps), None)
+            kv.rec.append(torch.zeros(n_seq_slots, rec.n_heads, rec.head_dim, rec.v_dim, **f32) if rec is not None else None)
+            kv.conv.append(torch.zeros(n_seq_slots, conv.conv_taps - 1, conv.conv_channels, **f32) if conv is not None else None)
+            kv.shift.append(torch.zeros(n_seq_slots, 1, cfg.hidden, **f32) if rec is not None and rec.mixer == "rwkv" else None)
+        for name in ("rec", "conv", "shift"):
+            if not any(t is not None for t in getattr(kv, name)):
+                setattr(kv, name, None)
         return kv
 
     def recurrent(self, li: int) -> List[torch.Tensor]:
         """The per-slot state tensors of entry ``li`` (empty for attention layers)."""
-        return [t[li] for t in (self.conv, self.rec) if t is not None and t[li] is not None]
+        return [t[li] for t in (self.conv, self.rec, self.shift) if t is not None and t[li] is not None]
 
     def reset_slots(self, slots) -> None:
         """Zero the recurrent state of the given sequence slots (a new sequence starts from an empty state)."""
-        if self.rec is None:
+        if self.rec is None and self.conv is None:
             return
         idx = torch.as_tensor(list(slots), dtype=torch.long, device=self.k[0].device)
         for li in range(len(self.k)):
@@ -394,7 +399,7 @@ class Transformer:
         self.rope_table = ew.rope_table(min(max(cfg.max_seq_len, 4096), 65536), rd, cfg.rope_theta, weights.embed.device) \
             if weights.embed.is_cuda and not cfg.is_layered else None
         self.mixer_blocks = {"attention": self.masked_attention_block, "lightning": self.lightning_block, "mamba2": self.mamba2_block, "hgrn2": self.hgrn2_block,
-                             "latent": self.latent_block}
+                             "latent": self.latent_block, "rwkv": self.rwkv_block}
         self.snapshots = {}            # layer -> hidden rows captured after that layer (debug / DeepStack)
         self.snapshot_layers: Sequence[int] = ()
 
@@ -496,26 +501,101 @@ class Transformer:
         plans = {}
         if any(sp.mixer == "latent" for sp in (self.cfg.layer_specs or ())):
             plans["latent"] = self.latent_plan(q_lens, [max_kv] * len(q_lens), max_kv, device, decode)
-        for sp in (self.cfg.layer_specs or ()):
+        for sp in (x for spec in (self.cfg.layer_specs or ()) for x in spec.mixers):
             if sp.mixer == "attention" and (sp.n_heads, sp.n_kv_heads, sp.span) not in plans:
                 plans[(sp.n_heads, sp.n_kv_heads, sp.span)] = attention_plan(q_lens, max_kv, sp.n_heads, sp.n_kv_heads, sp.span, device, decode)
+            if sp.mixer == "rwkv" and "shift" not in plans:
+                plans["shift"] = self.shift_plan(sum(q_lens), device)
         return plans
 
+    @staticmethod
+    def shift_plan(t: int, device):
+        """(rows per mix, segment starts, segment counts) of the grouped product over four mixes of ``t`` tokens."""
+        pad = recurrent.shift_pad(t)
+        return pad, torch.arange(4, dtype=torch.int32, device=device) * pad, torch.full((4,), t, dtype=torch.int32, device=device)
+
     def masked_attention_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
-        """Attention of a layer described by ``LayerSpec``: biased projection -> Q / K unit norm + cache store -> windowed attention with
-        kept first tokens and distance bias -> output projection.  ``li`` is the run, which has its own cache."""
-        kc, vc = self.kv.k[li], self.kv.v[li]
+        """Attention of a layer described by ``LayerSpec``: biased projection -> norm of Q and K (per head or over all of them) or convolution and rotation, cache
+        store -> attention with a window, kept first tokens and distance bias, capped scores, a sink -> gate -> output projection.  ``li`` is the
+        run, which has its own cache."""
+        kc, vc, eps = self.kv.k[li], self.kv.v[li], self.cfg.rms_eps
         qkv, _ = apply_linear_mixer(lw.wqkv, h)
-        q = stream.qk_unit(qkv, fb.slots, kc, vc, sp.n_heads, sp.n_kv_heads, sp.head_dim, sp.v_dim, self.cfg.rms_eps,
-                           (sp.scale or sp.head_dim ** -0.5) * att.LOG2E, unit=sp.qk_unit)
-        key = (sp.n_heads, sp.n_kv_heads, sp.span)
+        hq, hkv, d, dv = sp.n_heads, sp.n_kv_heads, sp.head_dim, sp.v_dim
+        # capped scores: the queries carry scale / cap, and the kernels multiply by cap * log2 e behind the tanh
+        scale = (sp.scale or d ** -0.5) * (1.0 / sp.softcap if sp.softcap else att.LOG2E)
+        if sp.rotary is not None:
+            q = stream.conv_rotary(qkv, self.rotary_table(lw, sp, fb), fb.slots, lw.conv_w, self.kv.conv[li], fb.cu_q, fb.seq_slots, kc, vc, hq, hkv, d, scale, self.most_tokens(fb))
+        elif sp.qk_norm_rows:
+            q = stream.qk_rows(qkv, fb.slots, lw.q_norm, lw.k_norm, kc, vc, hq, hkv, d, dv, eps, scale)
+        else:
+            q = stream.qk_unit(qkv, fb.slots, kc, vc, hq, hkv, d, dv, eps, scale, unit=sp.qk_unit)
+        key = (hq, hkv, sp.span)
         if fb.plans is None:
             fb.plans = {}
         if key not in fb.plans and q.is_cuda:
             fb.plans[key] = attention_plan(fb.q_lens, max(fb.kv_lens), *key, q.device, fb.is_decode)
         a = att.attention_masked(q, kc, vc, fb.cu_q, fb.kv_len, fb.block_table, self.kv.page_size, window=sp.window, keep_first=sp.keep_first,
-                                 bias=lw.rel_bias, plan=fb.plans.get(key), decode=fb.is_decode)
+                                 bias=lw.rel_bias, plan=fb.plans.get(key), decode=fb.is_decode, softcap=sp.softcap, sink=lw.sink)
+        if sp.out_gate:
+            a = stream.sigmoid_gate(a, qkv, sp.q_dim + hkv * (d + dv), dv)
         return apply_linear_stream(lw.wo, a.reshape(a.shape[0], -1))
+
+    @staticmethod
+    def most_tokens(fb: ForwardBatch) -> int:
+        """Tokens of the batch's longest sequence."""
+        return max(fb.q_lens) if fb.q_lens else 1
+
+    def rotary_table(self, lw, sp: LayerSpec, fb: ForwardBatch) -> torch.Tensor:
+        """cos and sin of the step's positions, formed once per forward pass and kind of rotation."""
+        key = tuple(vars(sp.rotary).values())
+        if key not in self._rotary:
+            self._rotary[key] = stream.rotary_table(fb.positions, lw.rot_freq, sp.rotary.magnitude)
+        return self._rotary[key]
+
+    def rwkv_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
+        """RWKV-style time mixing: five mixes with the token in front -> four projections as one grouped product, low-rank decay (f32) -> recurrence with a bonus
+        for the current token -> RMSNorm per head * SiLU(gate) -> output projection."""
+        w, t, most, n = lw.rwkv, h.shape[0], self.most_tokens(fb), sp.q_dim
+        if fb.plans is None:
+            fb.plans = {}
+        if "shift" not in fb.plans:
+            fb.plans["shift"] = self.shift_plan(t, h.device)
+        pad, seg, cnt = fb.plans["shift"]
+        mix = recurrent.token_shift(h, self.cfg.hidden, w.mu, self.kv.shift[li], fb.cu_q, fb.seq_slots, pad, most)
+        ld = stream.row_width(n, self.act_dtype)
+        if w.w_in.fmt == "f32":
+            rkvg = torch.empty(4, pad, ld, dtype=torch.float32, device=h.device)
+            gemm.batched_linear_f32(mix[:4], w.w_in.w.view(4, n, -1), rkvg)
+        else:
+            # decode-sized batches keep the projections in f32
+            rkvg = torch.empty(4, pad, ld, dtype=torch.float32 if t <= 64 else torch.bfloat16, device=h.device)
+            gemm.grouped_linear(mix[:4].view(4 * pad, -1), w.w_in.w.view(4, w.w_in.rows_per_group, -1), seg, cnt, min(pad, 128), out=rkvg.view(4 * pad, ld), n_out=n,
+                                w_tiled=w.w_in.tiled)
+        z = apply_linear_stream(w.w2, recurrent.tanh_rows(apply_linear_stream(w.w1, mix[4, :t]), sp.decay_rank, self.act_dtype))
+        o = recurrent.rwkv(rkvg, z, w.w0, w.u, self.kv.rec[li], fb.cu_q, fb.seq_slots, sp.n_heads, sp.head_dim, sp.v_dim, t, most)
+        y = stream.part_norm(o, w.norm, sp.n_heads, self.cfg.rms_eps, rkvg[3, :t], 0, self.act_dtype, gate_after=True)
+        return apply_linear_stream(w.w_out, y)
+
+    def mixer_parts(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
+        """(result, factor) of the mixer, or of each of the two side by side."""
+        if sp.mixer != "parallel":
+            return [(self.mixer_blocks[sp.mixer](li, lw, sp, h, fb), 1.0)]
+        return [(self.mixer_blocks[m.mixer](li, lw, m, h, fb), f) for m, f in ((sp.left, sp.left_scale), (sp.right, sp.right_scale))]
+
+    def parallel_layer(self, li: int, lw, sp: LayerSpec, x: torch.Tensor, delta, first: Optional[torch.Tensor], fb: ForwardBatch):
+        """A layer whose mixer and feed-forward read the same stream, with the token input behind them; returns the pending update of the token input."""
+        cfg, layer = self.cfg, self.runs[li].layer
+        hs = stream.norm2(x, lw.attn_norm, cfg.rms_eps, delta, add=first if self.runs[li].again else None, weight2=lw.ffn_norm, out_dtype=self.act_dtype)
+        with profiler.region(sp.mixer, "block", "attention", li):
+            parts = self.mixer_parts(li, lw, sp, hs[0], fb)
+        if sp.has_ffn:
+            with profiler.region("ffn", "block", "ffn", li):
+                parts.append((self.stream_ffn(lw, sp, hs[1]), 1.0))
+        rows = stream.join(x, parts, self.act_dtype if lw.side is not None else None)
+        if lw.side is None:
+            return None
+        g = stream.token_gate(apply_linear_stream(lw.side.gate, rows), fb.ids, self.w.side_embed, layer * cfg.side_dim, cfg.side_dim, self.act_dtype)
+        return stream.RmsPosted(apply_linear_stream(lw.side.proj, g), lw.side.norm, cfg.rms_eps)
 
     def lightning_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
         """Lightning attention: projection -> SiLU + decayed recurrence -> RMSNorm over all heads * sigmoid(gate) -> output projection."""
@@ -599,7 +679,7 @@ class Transformer:
 
     def stream_moe(self, lw, m: MoeSpec, h: torch.Tensor):
         """Mixture of experts of a layer described by ``LayerSpec``; the weighted sum stays pending for the stream's norm."""
-        rt = dict(mode=m.router, renorm=2 if m.renorm else 0, routed_scale=m.scale, groups=(m.groups, m.groups_kept))
+        rt = dict(mode=m.router, renorm=2 if m.renorm else 0, routed_scale=m.scale, groups=(m.groups, m.groups_kept, m.group_best))
         if lw.w13.fmt != "f32":
             return self.moe_local(lw, h, spec=m, rt=rt)
         ids, wts, pl = moe.route_plan(gemm.linear_f32(h, lw.router), m.top, m.n_experts, 64, **rt)
@@ -612,13 +692,13 @@ class Transformer:
             return self.stream_moe(lw, sp.moe, h)
         gu = lw.w_gate_up
         if gu.fmt == "f32":
-            return apply_linear_stream(lw.w_down, stream.act_mul(gemm.linear_f32(h, gu.w), sp.act))
+            return apply_linear_stream(lw.w_down, stream.act_mul(gemm.linear_f32(h, gu.w), sp.act, sp.act_cap))
         inter = gu.n // 2
         split = gemm.pick_partials_dual(inter, h.shape[0], (gu.k + 63) // 64 * 64, False) if SPLIT_PROJ and h.is_cuda else 1
         if split > 1:
-            act = ew.silu_mul_partials(gemm.swiglu_partials(h, gu.w, split, w_tiled=gu.tiled), act=sp.act)
+            act = ew.silu_mul_partials(gemm.swiglu_partials(h, gu.w, split, w_tiled=gu.tiled), act=sp.act, cap=sp.act_cap)
         else:
-            act = gemm.linear_swiglu(h, gu.w, w_tiled=gu.tiled, act=sp.act)
+            act = gemm.linear_swiglu(h, gu.w, w_tiled=gu.tiled, act=sp.act, cap=sp.act_cap)
         return apply_linear_stream(lw.w_down, act)
 
     def shared_expert(self, lw, h: torch.Tensor) -> torch.Tensor:
@@ -708,6 +788,8 @@ class Transformer:
         elif x is None:
             x = fb.embeds if fb.embeds is not None else ew.embed(fb.ids, w.embed)
         delta = None
+        first = x.clone() if any(r.again for r in self.runs) else None       # the embedding output, for later passes of a loop
+        self._rotary = {}
         if hasattr(self.par, "_sp_ok"):
             # the fused tensor-parallel prefill path keeps the residual stream sharded by rows between the layers' GEMMs: only for
             # plain dense stacks (nothing reads the whole stream or the normalised rows outside a GEMM in between)
@@ -715,6 +797,11 @@ class Transformer:
                                    any(l.ssm is not None for l in w.layers[first_layer:last_layer]))
         for li in range(first_layer, last_layer):           # li: the layer RUN, index of its cache (looped layers run several times)
             lw = w.layers[self.runs[li].layer]
+            if cfg.parallel_ffn:
+                delta = self.parallel_layer(li, lw, cfg.layer_specs[self.runs[li].layer], x, delta, first, fb)
+                if li in self.snapshot_layers:
+                    self.snapshots[li] = x + stream.whole(delta)[:, : x.shape[1]] if delta is not None else x.clone()
+                continue
             if self.stream_f32:
                 sp, step = cfg.layer_specs[self.runs[li].layer], self.runs[li].step
                 h = stream.norm(x, lw.attn_norm, cfg.rms_eps, delta, add=w.loop_step[step] if step >= 0 else None, out_dtype=self.act_dtype)

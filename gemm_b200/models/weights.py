@@ -285,6 +285,34 @@ class LatentWeights:
 
 
 @dataclass
+class RwkvWeights:
+    """An RWKV-style mixer.  ``w_in``: the receptance, key, value and gate projections as four groups of rows, each over a mix of its own of the
+    token's row and the one before it; ``w1`` / ``w2``: the decay's low-rank projection."""
+    mu: torch.Tensor              # f32 [5, H]: r, k, v, g, decay
+    w_in: LinearWeight
+    w1: LinearWeight              # [rank, H]
+    w2: LinearWeight              # [heads * dim, rank]
+    w0: torch.Tensor              # f32 [heads * dim]
+    u: torch.Tensor               # f32 [heads * dim]: weight of the current token
+    norm: torch.Tensor            # f32 [heads * v_dim]
+    w_out: LinearWeight
+
+    def to(self, device) -> "RwkvWeights":
+        return RwkvWeights(*(t.to(device) for t in (self.mu, self.w_in, self.w1, self.w2, self.w0, self.u, self.norm, self.w_out)))
+
+
+@dataclass
+class SideWeights:
+    """The token input of a layer: a gate on the stream, a projection back into it, a norm of the result."""
+    gate: LinearWeight            # [dim, H]
+    proj: LinearWeight            # [H, dim]
+    norm: torch.Tensor            # f32 [H]
+
+    def to(self, device) -> "SideWeights":
+        return SideWeights(self.gate.to(device), self.proj.to(device), self.norm.to(device))
+
+
+@dataclass
 class LayerWeights:
     attn_norm: torch.Tensor                       # or DynTanh
     wqkv: Optional[LinearWeight]                  # rows [Q ; K ; V] (+ [gate] after V when the attention output is gated); None in SSM layers
@@ -309,6 +337,11 @@ class LayerWeights:
     mamba: Optional[Mamba2Weights] = None
     gla: Optional[GlaWeights] = None
     latent: Optional[LatentWeights] = None        # (the output projection is wo)
+    sink: Optional[torch.Tensor] = None           # f32 [heads], times log2 e: joins the softmax's sum (attention)
+    conv_w: Optional[torch.Tensor] = None         # f32 [q and k channels, taps]: convolution of the projected q and k
+    rot_freq: Optional[torch.Tensor] = None       # f64 [dims / 2] rotary frequencies
+    rwkv: Optional[RwkvWeights] = None
+    side: Optional[SideWeights] = None
 
     def linears(self) -> List[LinearWeight]:
         """Every projection matrix of the layer."""
@@ -316,6 +349,10 @@ class LayerWeights:
         for part in (self.ssm, self.lin, self.mamba, self.gla):
             if part is not None:
                 own += [part.w_in, part.w_out]
+        if self.rwkv is not None:
+            own += [self.rwkv.w_in, self.rwkv.w1, self.rwkv.w2, self.rwkv.w_out]
+        if self.side is not None:
+            own += [self.side.gate, self.side.proj]
         if self.latent is not None:
             own += [self.latent.w_a, self.latent.w_qb, self.latent.w_kv, self.latent.w_uk, self.latent.w_uv]
         return [lw for lw in own if lw is not None]
@@ -335,6 +372,7 @@ class ModelWeights:
     ep_size: int = 1
     vocab_start: int = 0                          # first vocabulary id of the LM-head shard
     loop_step: Optional[torch.Tensor] = None      # f32 [times, H]: vectors added in front of the passes of a layer loop
+    side_embed: Optional[torch.Tensor] = None     # bf16 (f32) [V, layers * side_dim]: token inputs of the layers
 
     @property
     def kv_dtype(self) -> str:
@@ -348,10 +386,11 @@ class ModelWeights:
                                k_norm=mv(l.k_norm), w_gate_up=mv(l.w_gate_up), w_down=mv(l.w_down), router=mv(l.router),
                                router_bias=mv(l.router_bias), w13=mv(l.w13), w2=mv(l.w2), ssm=mv(l.ssm), sh_gate_up=mv(l.sh_gate_up),
                                sh_down=mv(l.sh_down), sh_gate=mv(l.sh_gate), lin=mv(l.lin), rel_bias=mv(l.rel_bias), attn_post=mv(l.attn_post),
-                               ffn_post=mv(l.ffn_post), mamba=mv(l.mamba), gla=mv(l.gla), latent=mv(l.latent)) for l in self.layers]
+                               ffn_post=mv(l.ffn_post), mamba=mv(l.mamba), gla=mv(l.gla), latent=mv(l.latent), sink=mv(l.sink), conv_w=mv(l.conv_w),
+                               rot_freq=mv(l.rot_freq), rwkv=mv(l.rwkv), side=mv(l.side)) for l in self.layers]
         return ModelWeights(cfg=self.cfg, embed=mv(self.embed), layers=layers, final_norm=mv(self.final_norm), lm_head=mv(self.lm_head),
                             fmt=self.fmt, tp_rank=self.tp_rank, tp_size=self.tp_size, ep_rank=self.ep_rank, ep_size=self.ep_size,
-                            vocab_start=self.vocab_start, loop_step=mv(self.loop_step))
+                            vocab_start=self.vocab_start, loop_step=mv(self.loop_step), side_embed=mv(self.side_embed))
 
     def tile_(self) -> "ModelWeights":
         """Put every projection matrix into the tiled weight layout (in place).  An LM head that shares its storage with
@@ -416,6 +455,14 @@ class RandomSource:
             return (self._randn(name, shape).float() * 25 - 3.0).to(torch.bfloat16)
         if name.endswith("gla_lower"):
             return (self._randn(name, shape).float() * 5 + 0.5).clamp(0.0, 0.95).to(torch.bfloat16)
+        if "rwkv_mu_" in name:
+            return (self._randn(name, shape).float() * 10 + 0.5).clamp(0.0, 1.0).to(torch.bfloat16)
+        if name.endswith("rwkv_w0"):                     # decays of about exp(-exp(-3))
+            return (self._randn(name, shape).float() * 50 - 3.0).to(torch.bfloat16)
+        if name.endswith("rwkv_u") or name.endswith(".conv"):
+            return (self._randn(name, shape).float() * 25).to(torch.bfloat16)
+        if name.endswith("_rows.norm"):
+            return torch.ones(tuple(shape), dtype=torch.bfloat16, device=self.device)
         if name.endswith("norm.weight") and not name.endswith("lin_norm.weight") and self.cfg.norm_offset:
             return torch.full(tuple(shape), 1.0 - self.cfg.norm_offset, dtype=torch.bfloat16, device=self.device)
         if name.endswith("norm.weight"):
@@ -673,11 +720,21 @@ class _LayeredBuilder:
     def attention(self, pre, sp, lw):
         h, nv = self.h, sp.n_heads * sp.v_dim
         nk, nkv = sp.n_kv_heads * sp.head_dim, sp.n_kv_heads * sp.v_dim
-        w = torch.cat([self.get(pre + "attn_q.weight", sp.q_dim, h), self.get(pre + "attn_k.weight", nk, h), self.get(pre + "attn_v.weight", nkv, h)])
+        rows = [("q", sp.q_dim), ("k", nk)] + ([] if sp.v_from_k else [("v", nkv)])
         bias = None
         if sp.qkv_bias:
-            bias = torch.cat([self.get(pre + f"attn_{c}.bias", n).float() for c, n in (("q", sp.q_dim), ("k", nk), ("v", nkv))]).contiguous().to(self.dev)
+            bias = [self.get(pre + f"attn_{c}.bias", n).float() for c, n in rows]
+            bias = torch.cat(bias + ([bias[0].new_zeros(nv)] if sp.out_gate else [])).contiguous().to(self.dev)
+        w = torch.cat([self.get(pre + f"attn_{c}.weight", n, h) for c, n in rows + ([("gate", nv)] if sp.out_gate else [])])
         lw.wqkv = self.linear(w, bias=bias)
+        if sp.qk_norm_rows:
+            lw.q_norm, lw.k_norm = self.f32(pre + "attn_q_rows.norm", sp.q_dim), self.f32(pre + "attn_k_rows.norm", nk)
+        if sp.conv_taps:
+            lw.conv_w = torch.cat([self.f32(pre + "attn_q.conv", sp.q_dim, sp.conv_taps), self.f32(pre + "attn_k.conv", nk, sp.conv_taps)]).contiguous()
+        if sp.rotary is not None:
+            lw.rot_freq = torch.tensor(sp.rotary.frequencies(), dtype=torch.float64, device=self.dev)
+        if sp.sink:
+            lw.sink = (self.get(pre + "attn_sink", sp.n_heads).double() * LOG2E).float().contiguous().to(self.dev)
         # the attention kernels emit heads of the cache's (padded) value width: the output projection has zero columns there
         wo = self.get(pre + "attn_output.weight", h, nv)
         dvp = cache_head_dims(sp.head_dim, sp.v_dim, torch.float32 if self.exact else torch.bfloat16)[1]
@@ -685,6 +742,26 @@ class _LayeredBuilder:
         lw.wo = self.linear(wo)
         if sp.rel_buckets:
             lw.rel_bias = distance_bias_table(self.get(pre + "attn_rel.weight", sp.rel_buckets, sp.n_heads).float().cpu(), sp.rel_max).to(self.dev)
+
+    def rwkv(self, pre, sp, lw):
+        h, nq, nv = self.h, sp.q_dim, sp.n_heads * sp.v_dim
+        assert nq == nv, "the four projections of the mixes share a size"
+        np_ = nq if self.exact else (nq + 127) // 128 * 128              # whole 128-row tiles per group
+        w = [torch.nn.functional.pad(self.get(pre + f"rwkv_{c}.weight", nq, h), (0, 0, 0, np_ - nq)) for c in "rkvg"]
+        lw.rwkv = RwkvWeights(mu=torch.stack([self.f32(pre + f"rwkv_mu_{c}", h) for c in "rkvgw"]).contiguous(), w_in=self.linear(torch.cat(w), groups=4),
+                              w1=self.linear(self.get(pre + "rwkv_w1.weight", sp.decay_rank, h)), w2=self.linear(self.get(pre + "rwkv_w2.weight", nq, sp.decay_rank)),
+                              w0=self.f32(pre + "rwkv_w0", nq), u=self.f32(pre + "rwkv_u", sp.n_heads, sp.head_dim).reshape(-1), norm=self.f32(pre + "rwkv_norm.weight", nv),
+                              w_out=self.linear(self.get(pre + "rwkv_out.weight", h, nv)))
+
+    def parallel(self, pre, sp, lw):
+        """Both mixers' weights are parts of one layer's: they have no name in common."""
+        for part, mx in (("left.", sp.left), ("right.", sp.right)):
+            getattr(self, mx.mixer)(pre + part, mx, lw)
+
+    def side(self, pre, lw):
+        h, d = self.h, self.cfg.side_dim
+        lw.side = SideWeights(gate=self.linear(self.get(pre + "side_gate.weight", d, h)), proj=self.linear(self.get(pre + "side_proj.weight", h, d)),
+                              norm=self.f32(pre + "side_norm.weight", h))
 
     def dense_ffn(self, pre, sp, lw):
         h = self.h
@@ -722,18 +799,22 @@ class _LayeredBuilder:
             self.dense_ffn(pre, sp, lw)
         elif sp.moe is not None:
             self.moe_ffn(pre, sp, lw)
+        if self.cfg.side_dim:
+            self.side(pre, lw)
         return lw
 
     def model(self) -> ModelWeights:
         cfg, h, src = self.cfg, self.h, self.src
         layers = [self.layer(li, sp) for li, sp in enumerate(cfg.layer_specs)]
-        embed = self.get("token_embd.weight", cfg.vocab, h).to(torch.float32 if self.exact else torch.bfloat16).contiguous().to(self.dev)
+        dt = torch.float32 if self.exact else torch.bfloat16
+        embed = self.get("token_embd.weight", cfg.vocab, h).to(dt).contiguous().to(self.dev)
+        side = self.get("side_embd.weight", cfg.vocab, cfg.n_layers * cfg.side_dim).to(dt).contiguous().to(self.dev) if cfg.side_dim else None
         head = embed if (cfg.tie_embeddings or not src.has("output.weight")) else self.get("output.weight", cfg.vocab, h)
-        step = self.f32("loop_step.weight", cfg.loop.times, h) if cfg.loop is not None else None
+        step = self.f32("loop_step.weight", cfg.loop.times, h) if cfg.loop is not None and cfg.loop.add == "step" else None
         final = self.norm("output_norm")
         if cfg.norm_kind == "rms":
             final = final * cfg.logit_scale
-        return ModelWeights(cfg=cfg, embed=embed, layers=layers, final_norm=final, lm_head=self.linear(head), fmt=self.fmt, loop_step=step)
+        return ModelWeights(cfg=cfg, embed=embed, layers=layers, final_norm=final, lm_head=self.linear(head), fmt=self.fmt, loop_step=step, side_embed=side)
 
 
 def _build_layered(cfg: ModelConfig, src, fmt: str, dev, tile: Optional[bool]) -> ModelWeights:

@@ -17,7 +17,7 @@ import torch
 
 from .. import _native
 
-_c, _i, _l = ctypes.c_void_p, ctypes.c_int, ctypes.c_long
+_c, _i, _f, _l = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_long
 
 
 def _p(t):
@@ -359,7 +359,7 @@ def cache_head_dims(dk: int, dv: int, dtype: torch.dtype):
     return flash_head_dims(dk, dv) or ((dk + 7) // 8 * 8, (dv + 7) // 8 * 8)
 
 
-def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window=0, keep_first=0, bias=None) -> torch.Tensor:
+def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window=0, keep_first=0, bias=None, softcap=0.0, sink=None) -> torch.Tensor:
     t, hq, d = q.shape
     g = hq // k_cache.shape[1]
     out = torch.zeros(t, hq, v_cache.shape[2], dtype=torch.float32)
@@ -374,6 +374,8 @@ def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_si
         k = k_cache[slots].float().repeat_interleave(g, dim=1)
         v = v_cache[slots].float().repeat_interleave(g, dim=1)
         sc = torch.einsum("qhd,khd->hqk", q[q0:q1].float(), k)
+        if softcap > 0:
+            sc = softcap * LOG2E * torch.tanh(sc)
         dist = torch.arange(kl - ql, kl).unsqueeze(1) - torch.arange(kl).unsqueeze(0)
         if bias is not None:
             n = bias.shape[1] // 2
@@ -381,22 +383,28 @@ def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_si
         see = dist >= 0
         if window > 0:
             see &= (dist < window) | (torch.arange(kl).unsqueeze(0) < keep_first)
-        p = torch.softmax((sc * math.log(2.0)).masked_fill(~see.unsqueeze(0), float("-inf")), dim=-1)
+        sc = (sc * math.log(2.0)).masked_fill(~see.unsqueeze(0), float("-inf"))
+        if sink is not None:                # a column of its own that has no value
+            sc = torch.cat([sc, (sink * math.log(2.0)).reshape(hq, 1, 1).expand(hq, ql, 1)], dim=-1)
+        p = torch.softmax(sc, dim=-1)[..., :kl]
         out[q0:q1] = torch.einsum("hqk,khd->qhd", p, v)
     return out.to(k_cache.dtype)
 
 
 def attention_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
                      block_table: torch.Tensor, page_size: int, window: int = 0, keep_first: int = 0, bias: Optional[torch.Tensor] = None,
-                     plan=None, decode: bool = False) -> torch.Tensor:
+                     plan=None, decode: bool = False, softcap: float = 0.0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention in which position i sees j <= i with ``i - j < window`` (0: no limit) or ``j < keep_first``, with an optional distance
     bias (``distance_bias_table``) added to the scores.  Key and value widths may differ (``k_cache [slots, Hkv, dk]``, ``v_cache [slots, Hkv,
-    dv]``, ``q [T, Hq, dk]`` times scale * log2(e)).  Returns ``[T, Hq, dv]`` in the cache's dtype.  ``plan``: ``(work list, KV splits)`` for
+    dv]``, ``q [T, Hq, dk]`` times scale * log2(e)).  ``softcap`` > 0: the scores are softcap * tanh(score / softcap), and ``q`` comes times scale /
+    softcap.  ``sink`` (f32 ``[Hq]``, times log2(e)): a score per head that joins the sum of the weights (neither goes with a bias or kept positions).  Returns ``[T, Hq, dv]`` in the cache's dtype.  ``plan``: ``(work list, KV splits)`` for
     the tcgen05 kernels; without one, or for an f32 cache or wider heads, the any-size kernel runs."""
     t, hq, dk = q.shape
     hkv, dv = k_cache.shape[1], v_cache.shape[2]
     if not q.is_cuda:
-        return attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window, keep_first, bias)
+        return attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window, keep_first, bias, softcap, sink)
+    if (softcap > 0 or sink is not None) and (bias is not None or keep_first):
+        raise ValueError("capped scores and sinks do not go with a distance bias or kept positions")
     out = torch.empty(t, hq, dv, dtype=k_cache.dtype, device=q.device)
     n_bias, ld_bias = (bias.shape[1] // 2, bias.stride(0)) if bias is not None else (0, 0)
     lib, stream = _native.cuda(), _c(torch.cuda.current_stream().cuda_stream)
@@ -409,14 +417,14 @@ def attention_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             part_lse = torch.empty(splits, t, hq, dtype=torch.float32, device=q.device)
         rc = lib.gb_flash_masked(_p(q), _p(k_cache), _p(v_cache), _p(out), _p(part_o), _p(part_lse), _p(work), _i(work.shape[0]), _p(cu_q), _p(kv_len),
                                  _p(block_table), _i(block_table.shape[1]), _i(page_size), _l(k_cache.shape[0]), _i(t), _i(hq), _i(hkv), _i(dk), _i(dv),
-                                 _i(splits), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), _i(int(decode and hq // hkv <= 16)),
-                                 _c(_native.status_ptr()), stream)
+                                 _i(splits), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), _f(softcap), _p(sink),
+                                 _i(int(decode and hq // hkv <= 16)), _c(_native.status_ptr()), stream)
         _native.check(rc, "gb_flash_masked")
         if splits > 1:
             _native.check(lib.gb_fa_combine_dim(_p(part_o), _p(part_lse), _p(out), _i(splits), _l(t * hq), _i(dv), stream), "gb_fa_combine_dim")
         return out
     rc = lib.gb_attn_any(_p(q), _p(k_cache), _p(v_cache), _p(out), _i(int(k_cache.dtype == torch.float32)), _p(cu_q), _p(kv_len),
                          _p(block_table), _i(block_table.shape[1]), _i(page_size), _i(cu_q.numel() - 1), _l(k_cache.shape[0]), _i(t), _i(hq),
-                         _i(hkv), _i(dk), _i(dv), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), stream)
+                         _i(hkv), _i(dk), _i(dv), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), _f(softcap), _p(sink), stream)
     _native.check(rc, "gb_attn_any")
     return out

@@ -16,8 +16,9 @@ from .. import _native
 from . import mxfp8
 from .mxfp8 import MxTensor
 
-GEMM_MX, GEMM_DUAL, GEMM_QUANT_OUT, GEMM_OUT_F32, GEMM_W_TILED, GEMM_DUAL_RAW, GEMM_GELU = 1, 2, 4, 8, 16, 32, 64
-GATE_ACTS = ("silu", "gelu_tanh")         # activations of a gated feed-forward, by the code the kernels use
+GEMM_MX, GEMM_DUAL, GEMM_QUANT_OUT, GEMM_OUT_F32, GEMM_W_TILED, GEMM_DUAL_RAW, GEMM_GELU, GEMM_CAPPED = 1, 2, 4, 8, 16, 32, 64, 128
+GATE_ACTS = ("silu", "gelu_tanh", "capped")         # activations of a gated feed-forward, by the code the kernels use
+GATE_ACT_CODE = {a: i for i, a in enumerate(GATE_ACTS)}
 
 
 class GemmExtras(ctypes.Structure):
@@ -29,7 +30,7 @@ class GemmExtras(ctypes.Structure):
                 ("sk_ws", ctypes.c_void_p), ("sk_ctr", ctypes.c_void_p), ("amax_val", ctypes.c_void_p), ("amax_idx", ctypes.c_void_p),
                 ("sk_ws_bytes", ctypes.c_long), ("sk_ctr_count", ctypes.c_long), ("peer_bcast", ctypes.c_int), ("epoch_self_tick", ctypes.c_int),
                 ("sfa_bytes", ctypes.c_size_t), ("sfb_bytes", ctypes.c_size_t), ("out_bytes", ctypes.c_size_t), ("out_sf_bytes", ctypes.c_size_t),
-                ("partial_stride", ctypes.c_long), ("silu_rows", ctypes.c_int)]
+                ("partial_stride", ctypes.c_long), ("silu_rows", ctypes.c_int), ("act_cap", ctypes.c_float)]
 
 
 _SK_WS_BYTES = 64 << 20
@@ -180,10 +181,14 @@ def linear_argmax(x: torch.Tensor, w: torch.Tensor, idx_offset: int = 0, want_va
     return (out, val) if want_value else out
 
 
-def gate_act_ref(g: torch.Tensor, act: str) -> torch.Tensor:
+def gated_act_ref(g: torch.Tensor, u: torch.Tensor, act: str, cap: float = 0.0) -> torch.Tensor:
+    """``act(g) * u``; "capped": ``g sigmoid(1.702 g) (u + 1)`` of g at most ``cap`` and u within ``+-cap``."""
     if act == "gelu_tanh":
-        return torch.nn.functional.gelu(g, approximate="tanh")
-    return torch.nn.functional.silu(g)
+        return torch.nn.functional.gelu(g, approximate="tanh") * u
+    if act == "capped":
+        g = g.clamp(max=cap)
+        return g * torch.sigmoid(1.702 * g) * (u.clamp(-cap, cap) + 1.0)
+    return torch.nn.functional.silu(g) * u
 
 
 def linear_f32(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -233,17 +238,18 @@ def grouped_linear_f32(x: torch.Tensor, w: torch.Tensor, seg_start: torch.Tensor
 
 
 def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: Optional[torch.Tensor] = None,
-                  tn: Optional[int] = None, w_tiled: bool = False, act: str = "silu") -> torch.Tensor:
-    """``act(x @ Wg^T) * (x @ Wu^T)`` with ``w_gate_up = [Wg; Wu]`` stacked along rows ([2I, K]); ``act`` is one of ``GATE_ACTS``."""
+                  tn: Optional[int] = None, w_tiled: bool = False, act: str = "silu", cap: float = 0.0) -> torch.Tensor:
+    """``act(x @ Wg^T) * (x @ Wu^T)`` with ``w_gate_up = [Wg; Wu]`` stacked along rows ([2I, K]); ``act`` is one of ``GATE_ACTS`` (see ``gated_act_ref``)."""
     m, k = x.shape
     inter = w_gate_up.shape[0] // 2
     if not x.is_cuda:
         y = x.float() @ (mxfp8.untile_weight(w_gate_up) if w_tiled else w_gate_up).float().t()
-        return (gate_act_ref(y[:, :inter], act) * y[:, inter:]).to(torch.bfloat16)
+        return gated_act_ref(y[:, :inter], y[:, inter:], act, cap).to(torch.bfloat16)
     if out is None:
         out = torch.empty(m, inter, dtype=torch.bfloat16, device=x.device)
     _launch(w_gate_up, x, out, inter, k, m, w_gate_up.stride(0), x.stride(0), out.stride(0),
-            GEMM_DUAL | (GEMM_W_TILED if w_tiled else 0) | (GEMM_GELU if act == "gelu_tanh" else 0), tn or pick_tn(m, dual=True), up_row_offset=inter)
+            GEMM_DUAL | (GEMM_W_TILED if w_tiled else 0) | {"silu": 0, "gelu_tanh": GEMM_GELU, "capped": GEMM_CAPPED}[act], tn or pick_tn(m, dual=True), up_row_offset=inter,
+            extras=GemmExtras(act_cap=cap) if act == "capped" else None)
     return out
 
 

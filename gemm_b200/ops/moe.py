@@ -43,8 +43,13 @@ def router_logits(h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
     return gemm.linear(h, w, out_dtype=torch.float32)
 
 
+def _group_best(groups) -> int:
+    """How many of its best scores a group is ranked by."""
+    return groups[2] if len(groups) > 2 else 2
+
+
 def route_ref(logits: torch.Tensor, k: int, mode: str = "softmax", bias: Optional[torch.Tensor] = None,
-              renorm=True, routed_scale: float = 1.0, groups: Tuple[int, int] = (1, 1)):
+              renorm=True, routed_scale: float = 1.0, groups: Tuple[int, ...] = (1, 1)):
     lf = torch.nan_to_num(logits.float(), nan=-3.4e38)
     if mode == "softmax":
         p = torch.softmax(lf, dim=-1)
@@ -54,8 +59,8 @@ def route_ref(logits: torch.Tensor, k: int, mode: str = "softmax", bias: Optiona
         sel = p + (bias.float() if bias is not None else 0.0)
     if groups[0] > 1:
         t, e = sel.shape
-        best2 = sel.reshape(t, groups[0], e // groups[0]).topk(min(2, e // groups[0]), dim=-1).values.sum(-1)
-        kept = torch.sort(best2, dim=-1, descending=True, stable=True).indices[:, : groups[1]]
+        best = sel.reshape(t, groups[0], e // groups[0]).topk(min(_group_best(groups), e // groups[0]), dim=-1).values.sum(-1)
+        kept = torch.sort(best, dim=-1, descending=True, stable=True).indices[:, : groups[1]]
         ok = torch.zeros(t, groups[0], dtype=torch.bool, device=sel.device).scatter_(1, kept, True)
         sel = sel.masked_fill(~ok.repeat_interleave(e // groups[0], dim=1), -3.4e38)
     # ties -> lower index: stable descending sort
@@ -67,11 +72,12 @@ def route_ref(logits: torch.Tensor, k: int, mode: str = "softmax", bias: Optiona
 
 
 def route(logits: torch.Tensor, k: int, mode: str = "softmax", bias: Optional[torch.Tensor] = None, renorm=True,
-          routed_scale: float = 1.0, local_range: Optional[Tuple[int, int]] = None, groups: Tuple[int, int] = (1, 1)) -> Tuple[torch.Tensor, torch.Tensor]:
+          routed_scale: float = 1.0, local_range: Optional[Tuple[int, int]] = None, groups: Tuple[int, ...] = (1, 1)) -> Tuple[torch.Tensor, torch.Tensor]:
     """``logits`` f32 [T, E] -> (ids int32 [T, k], weights f32 [T, k]).  ``local_range = (first, count)`` turns the ids into
     indices of this rank's experts (``id - first``) and marks the picks that belong to other ranks with -1; the weights are
     still those of the full top-k.  ``renorm``: False, True (scores over their sum, at least 1e-20) or 2 (over the sum + 1e-20).  ``groups = (n, keep)``:
-    the experts form ``n`` groups of neighbours; only experts of the ``keep`` groups with the largest sums of their two best scores are picked."""
+    the experts form ``n`` groups of neighbours; only experts of the ``keep`` groups with the largest sums of their two best scores are picked
+    (``(n, keep, 1)``: with the largest scores)."""
     if not logits.is_cuda:
         ids, w = route_ref(logits, k, mode, bias, renorm, routed_scale, groups)
         if local_range is not None:
@@ -82,7 +88,7 @@ def route(logits: torch.Tensor, k: int, mode: str = "softmax", bias: Optional[to
     ids = torch.empty(t, k, dtype=torch.int32, device=logits.device)
     w = torch.empty(t, k, dtype=torch.float32, device=logits.device)
     rc = _native.cuda().gb_moe_route(_p(logits), _p(bias), _p(ids), _p(w), _i(t), _i(e), _i(k), _i(0 if mode == "softmax" else 1),
-                                     _i(int(renorm)), _f(routed_scale), _i(groups[0]), _i(groups[1]), _i(logits.stride(0)),
+                                     _i(int(renorm)), _f(routed_scale), _i(groups[0]), _i(groups[1]), _i(_group_best(groups)), _i(logits.stride(0)),
                                      _i(local_range[0] if local_range else 0), _i(local_range[1] if local_range else 0), _s())
     _native.check(rc, "gb_moe_route")
     return ids, w
@@ -120,7 +126,7 @@ def route_hidden(h: torch.Tensor, w: torch.Tensor, k: int, mode: str = "softmax"
 def route_plan_hidden(h: torch.Tensor, w: torch.Tensor, k: int, n_exp: int, align: int, mode: str = "softmax",
                       bias: Optional[torch.Tensor] = None, renorm=True, routed_scale: float = 1.0,
                       local_range: Optional[Tuple[int, int]] = None, regions: int = 1, epoch_ctr: int = 0, region_rows: Optional[int] = None,
-                      groups: Tuple[int, int] = (1, 1)):
+                      groups: Tuple[int, ...] = (1, 1)):
     """Router projection, routing and plan from the hidden rows: ``(ids, weights, MoePlan)`` (see ``route_plan``)."""
     if groups[0] == 1 and can_route_hidden(h, w, k) and h.shape[0] * k > FUSED_ROUTE_PAIRS:
         ids, wt = route_hidden(h, w, k, mode, bias, renorm, routed_scale, local_range)
@@ -144,7 +150,7 @@ def can_prep(h: torch.Tensor, w: torch.Tensor, k: int) -> bool:
 
 def prep_hidden(h: torch.Tensor, w: torch.Tensor, k: int, n_exp: int, align: int, mode: str = "softmax", bias: Optional[torch.Tensor] = None,
                 renorm=True, routed_scale: float = 1.0, local_range: Optional[Tuple[int, int]] = None, quantize: bool = True,
-                wait_flags: int = 0, wait_n: int = 0, epoch_ptr: int = 0, groups: Tuple[int, int] = (1, 1)):
+                wait_flags: int = 0, wait_n: int = 0, epoch_ptr: int = 0, groups: Tuple[int, ...] = (1, 1)):
     """Router projection, routing, plan AND the gather of the token rows into expert order in one launch.
 
     Returns ``(ids, weights, MoePlan, rows)``; ``rows`` is an ``MxTensor`` (MXFP8 with scale atoms in the ``align``-row layout,
@@ -171,7 +177,7 @@ def prep_hidden(h: torch.Tensor, w: torch.Tensor, k: int, n_exp: int, align: int
     else:
         xs = torch.empty(capacity, hid, dtype=torch.bfloat16, device=dev)
     rc = _native.cuda().gb_moe_prep(_p(h), _i(h.stride(0)), _i(t), _i(hid), _p(w), _i(w.stride(0)), _i(w.shape[0]), _p(bias), _i(k),
-                                    _i(0 if mode == "softmax" else 1), _i(int(renorm)), _f(routed_scale), _i(groups[0]), _i(groups[1]),
+                                    _i(0 if mode == "softmax" else 1), _i(int(renorm)), _f(routed_scale), _i(groups[0]), _i(groups[1]), _i(_group_best(groups)),
                                     _i(local_range[0] if local_range else 0), _i(local_range[1] if local_range else 0), _i(align),
                                     _i(capacity), _p(ids), _p(wt), _p(seg_start), _p(seg_count), _p(pair_row), _p(row_token), _p(xq), _p(xsf),
                                     _i(1 if align == 32 else 0), _p(xs), _c(wait_flags), _i(wait_n), _c(epoch_ptr),
@@ -316,7 +322,7 @@ FUSED_ROUTE_PAIRS = int(os.environ.get("GB_FUSED_ROUTE_PAIRS", "256"))
 
 def route_plan(logits: torch.Tensor, k: int, n_exp: int, align: int, mode: str = "softmax", bias: Optional[torch.Tensor] = None,
                renorm=True, routed_scale: float = 1.0, local_range: Optional[Tuple[int, int]] = None, regions: int = 1,
-               epoch_ctr: int = 0, region_rows: Optional[int] = None, groups: Tuple[int, int] = (1, 1)):
+               epoch_ctr: int = 0, region_rows: Optional[int] = None, groups: Tuple[int, ...] = (1, 1)):
     """``route`` followed by ``plan``; decode-sized batches (T * k <= ``FUSED_ROUTE_PAIRS``) do both in ONE kernel.  ``n_exp`` is the number of
     experts the plan is built over (the local count when ``local_range`` is given).  Returns ``(ids, weights, MoePlan)``."""
     t, e_all = logits.shape
@@ -339,7 +345,7 @@ def route_plan(logits: torch.Tensor, k: int, n_exp: int, align: int, mode: str =
     pair_row = torch.empty(n_pairs, dtype=torch.int32, device=dev)
     row_token = torch.empty(capacity, dtype=torch.int32, device=dev)
     rc = _native.cuda().gb_moe_route_plan(_p(logits), _p(bias), _p(ids), _p(w), _i(t), _i(e_all), _i(k), _i(0 if mode == "softmax" else 1),
-                                          _i(int(renorm)), _f(routed_scale), _i(groups[0]), _i(groups[1]), _i(logits.stride(0)),
+                                          _i(int(renorm)), _f(routed_scale), _i(groups[0]), _i(groups[1]), _i(_group_best(groups)), _i(logits.stride(0)),
                                           _i(local_range[0] if local_range else 0), _i(local_range[1] if local_range else 0),
                                           _p(seg_start), _p(seg_count), _p(region_used), _p(pair_row), _p(row_token), _i(n_exp),
                                           _i(n_exp // regions), _i(region_rows), _i(align), _l(capacity), _c(epoch_ctr), _s())

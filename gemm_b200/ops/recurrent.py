@@ -3,6 +3,8 @@
 ``causal_conv``  depthwise causal convolution + SiLU, the last inputs carried per sequence (Mamba-2)
 ``ssd``          Mamba-2:  S_t = exp(a dt_t) S_{t-1} + dt_t B_t x_t^T,  y_t = S_t^T C_t + D x_t
 ``gla``          HGRN2:    S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T,  o_t = S_t^T q_t
+``rwkv``         RWKV:     o_t = (S_{t-1} + diag(u) k_t v_t^T)^T r_t,  S_t = diag(w_t) S_{t-1} + k_t v_t^T,  w = exp(-exp(z))
+``token_shift``  mixes of a token's row and the one before it, for the projections of ``rwkv``
 
 State tensors: ``conv_state`` f32 ``[slots, taps - 1, channels]`` (oldest row first), ``state`` f32 ``[slots, heads, dim, vdim]``; one slot per
 sequence, updated in place.
@@ -15,6 +17,7 @@ import os
 import torch
 
 from .. import _native
+from . import gemm
 from .stream import row_width, split_rows, whole
 
 _c, _i, _f, _l = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_long
@@ -162,4 +165,89 @@ def gla(qv, gate, gate_col: int, f_bias: torch.Tensor, lower: torch.Tensor, stat
                                           _c(0), _p(state), _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(nv), _i(heads), _i(1), _i(dim), _i(vdim),
                                           _i(int(not activated)), _i(cu_q.numel() - 1), _s())
     _native.check(rc, "gb_recurrent_step")
+    return out
+
+
+def shift_pad(t: int) -> int:
+    """Rows per mix of ``token_shift`` for ``t`` tokens: whole token tiles of the grouped product that follows."""
+    tn = gemm.pick_tn(t) if t < 128 else 128
+    return (t + tn - 1) // tn * tn
+
+
+def token_shift(h: torch.Tensor, width: int, mu: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, seq_slots: torch.Tensor, pad: int, max_tokens: int) -> torch.Tensor:
+    """Rows ``h [T, ld]`` -> ``[n, pad, ld]``: mix i of token t is ``h + (h' - h) * mu[i]`` with the row h' in front of it (``mu`` f32 ``[n, width]``).  The row in front
+    of a sequence's first token comes from ``state`` f32 ``[slots, 1, width]``, its last one goes there.  Rows behind T are undefined."""
+    t, ld = h.shape
+    n = mu.shape[0]
+    if not h.is_cuda:
+        out, cu = torch.zeros(n, pad, ld, dtype=h.dtype), cu_q.tolist()
+        x = h[:, :width].float()
+        for s in range(len(cu) - 1):
+            if cu[s + 1] > cu[s]:
+                cur, slot = x[cu[s]: cu[s + 1]], int(seq_slots[s])
+                prev = torch.cat([state[slot], cur[:-1]])
+                out[:, cu[s]: cu[s + 1], :width] = (cur + (prev - cur) * mu.unsqueeze(1)).to(h.dtype)
+                state[slot] = cur[-1:]
+        return out
+    assert h.stride(1) == 1 and state.is_contiguous() and state.dtype == torch.float32
+    out = torch.empty(n, pad, ld, dtype=h.dtype, device=h.device)
+    rc = _native.cuda().gb_token_shift(_p(h), _i(int(h.dtype == torch.float32)), _i(h.stride(0)), _i(width), _p(mu), _i(n), _p(state), _i(state.shape[0]), _p(cu_q), _p(seq_slots),
+                                       _p(out), _l(pad * ld), _i(ld), _i(max_tokens), _i(cu_q.numel() - 1), _s())
+    _native.check(rc, "gb_token_shift")
+    return out
+
+
+def tanh_rows(z, n: int, out_dtype=torch.bfloat16) -> torch.Tensor:
+    """tanh of the first ``n`` columns of a projection result -> rows ``[T, row_width(n)]``."""
+    base, f32, parts, stride, ld = split_rows(z)
+    t = _n_rows(z)
+    out = torch.empty(t, row_width(n, out_dtype), dtype=out_dtype, device=base.device)
+    if not base.is_cuda:
+        out.zero_()
+        out[:, :n] = torch.tanh(whole(z)[:, :n]).to(out_dtype)
+        return out
+    rc = _native.cuda().gb_tanh_rows(_p(base), _i(f32), _i(parts), _l(stride), _i(ld), _p(out), _i(int(out_dtype == torch.float32)), _i(out.shape[1]), _i(t), _i(n), _s())
+    _native.check(rc, "gb_tanh_rows")
+    return out
+
+
+def rwkv_ref(r, k, v, z, u, state, cu_q, seq_slots, heads, dim, vdim):
+    t = r.shape[0]
+    r, k, v = r.reshape(t, heads, dim), k.reshape(t, heads, dim), v.reshape(t, heads, vdim)
+    w = torch.exp(-torch.exp(z)).reshape(t, heads, dim)
+    bonus = (r * u.reshape(heads, dim) * k).sum(-1, keepdim=True)
+    out = torch.zeros(t, heads * vdim)
+    cu = cu_q.tolist()
+    for s in range(len(cu) - 1):
+        st = state[int(seq_slots[s])] if cu[s + 1] > cu[s] else None
+        for i in range(cu[s], cu[s + 1]):
+            out[i] = (torch.einsum("hde,hd->he", st, r[i]) + bonus[i] * v[i]).reshape(-1)
+            st.mul_(w[i].unsqueeze(-1)).add_(k[i].unsqueeze(-1) * v[i].unsqueeze(1))
+    return out
+
+
+def rwkv(rkv: torch.Tensor, z, w0: torch.Tensor, u: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, seq_slots: torch.Tensor, heads: int, dim: int, vdim: int,
+         tokens: int, max_tokens: int = 1) -> torch.Tensor:
+    """``rkv [>= 3, pad, ld]``: receptances, keys and values of ``tokens`` tokens; ``z``: projection result (f32 or partial sums) whose columns, plus ``w0``, are the
+    decay exponents (w = exp(-exp(z + w0))); ``u`` f32 ``[heads * dim]``.  Returns f32 ``[tokens, heads * vdim]``."""
+    gb, gf32, gparts, gstride, gld = split_rows(z)
+    nq, nv = heads * dim, heads * vdim
+    if not rkv.is_cuda:
+        x = rkv[:, :tokens].float()
+        return rwkv_ref(x[0, :, :nq], x[1, :, :nq], x[2, :, :nv], whole(z)[:, :nq] + w0, u, state, cu_q, seq_slots, heads, dim, vdim)
+    assert gf32 and state.is_contiguous() and state.dtype == torch.float32 and rkv.stride(2) == 1
+    out = torch.empty(tokens, nv, dtype=torch.float32, device=rkv.device)
+    ld, gs = rkv.stride(1), rkv.stride(0)
+    if CHUNKED and max_tokens >= CHUNKED_MIN_TOKENS and can_chunk(rkv[0], dim, vdim) and gs % 8 == 0:
+        lib, n_seqs = _native.cuda(), cu_q.numel() - 1
+        lib.gb_gla_chunk_workspace.restype = _l
+        nb = int(lib.gb_gla_chunk_workspace(_l(tokens), _i(n_seqs), _i(heads), _i(dim)))
+        ws = torch.empty(nb, dtype=torch.uint8, device=rkv.device)
+        rc = lib.gb_rwkv_chunk(_p(rkv), _l(gs), _i(ld), _i(tokens), _p(gb), _i(gparts), _l(gstride), _i(gld), _p(w0), _p(u), _p(state), _i(state.shape[0]), _p(cu_q),
+                               _p(seq_slots), _p(out), _i(nv), _i(heads), _i(dim), _i(vdim), _i(max_tokens), _i(n_seqs), _p(ws), _l(nb), _c(_native.status_ptr()), _s())
+        _native.check(rc, "gb_rwkv_chunk", n=2)
+        return out
+    rc = _native.cuda().gb_rwkv_step(_p(rkv), _i(int(rkv.dtype == torch.float32)), _l(gs), _i(ld), _p(gb), _i(gparts), _l(gstride), _i(gld), _p(w0), _p(u), _p(state),
+                                     _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(nv), _i(heads), _i(dim), _i(vdim), _i(cu_q.numel() - 1), _s())
+    _native.check(rc, "gb_rwkv_step")
     return out

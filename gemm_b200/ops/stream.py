@@ -3,9 +3,14 @@
 ``embed``        embedding rows (times a factor) as an f32 stream
 ``norm``         stream += pending update (+ a vector), then RMSNorm or Dynamic Tanh -> rows for the next projection; the update may have a
                  norm of its own (``PostNormed``)
+``join``         stream += a weighted sum of several pending results; a copy of the rows for a projection of the stream itself
+``qk_rows``      Q and K normed over all their heads at once, K / V to the cache, Q scaled for the attention kernels
+``conv_rotary``  short causal convolution of Q and K, rotation, the rotated K and the K before it (as V) to the cache
+``sigmoid_gate`` the heads' outputs times sigmoid(gate)
+``token_gate``   GELU(z) times a row of a table, by token
 ``qk_unit``      Q / K divided by their root mean square per head, K / V to the cache, Q scaled for the attention kernels
 ``gated_norm``   RMSNorm over all heads' outputs times sigmoid(gate)
-``part_norm``    RMSNorm of equal parts of a row, after multiplying by SiLU(gate) if there is one
+``part_norm``    RMSNorm of equal parts of a row, after (or before) multiplying by SiLU(gate) if there is one
 ``act_mul``      act(gate) * up of f32 rows
 
 The rows that feed a projection have the width ``row_width(n, dtype)``: bf16 rows are padded with zeros to a multiple of 8 elements
@@ -17,12 +22,12 @@ from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from typing import Optional
+from typing import List, Optional, Tuple
 
 import torch
 
 from .. import _native
-from .gemm import gate_act_ref
+from .gemm import GATE_ACT_CODE, gated_act_ref
 
 _c, _i, _f, _l = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_long
 
@@ -68,10 +73,21 @@ class PostNormed:
     post: DynTanh
 
 
+@dataclass
+class RmsPosted:
+    """A result that is divided by its root mean square and multiplied by ``weight`` (f32 ``[W]``) before it joins the stream."""
+    delta: object
+    weight: torch.Tensor
+    eps: float
+
+
 def whole(y) -> torch.Tensor:
     """f32 copy of a projection result or of a pending update (CPU references, captured layers)."""
     if isinstance(y, PostNormed):
         return y.post(whole(y.delta)[:, : y.post.weight.numel()])
+    if isinstance(y, RmsPosted):
+        u = whole(y.delta)[:, : y.weight.numel()]
+        return u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + y.eps) * y.weight
     if hasattr(y, "pair_row"):
         rows = y.pair_row.reshape(y.n_tok, y.k).long()
         g = y.y.float()[rows.clamp_min(0)] * (rows >= 0).unsqueeze(-1)
@@ -88,11 +104,85 @@ def embed(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0) -> torch.T
     return out
 
 
+def _rms2_ref(x, weight, weight2, eps, delta, add, rows, out_dtype):
+    w = x.shape[1]
+    y = x
+    if delta is not None:
+        y = y + whole(delta)[:, :w]
+    if add is not None:
+        y = y + add
+    if rows is None:
+        x.copy_(y)
+    else:
+        y = y[rows]
+    unit = y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+    outs = []
+    for wt in (weight, weight2):
+        if wt is not None:
+            o = torch.zeros(y.shape[0], row_width(w, out_dtype), dtype=out_dtype)
+            o[:, :w] = (unit * wt).to(out_dtype)
+            outs.append(o)
+    return outs
+
+
+def norm2(x: torch.Tensor, weight: torch.Tensor, eps: float, delta: Optional[RmsPosted] = None, add: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+          weight2: Optional[torch.Tensor] = None, out_dtype=torch.bfloat16) -> List[torch.Tensor]:
+    """``norm`` for an update with a norm of its own (``RmsPosted``), for ``add`` one row per token (f32 ``[T, W]``), and with the rows under a second weight as
+    well: one list entry per weight."""
+    t, w = x.shape
+    n = t if rows is None else rows.numel()
+    if not x.is_cuda:
+        return _rms2_ref(x, weight, weight2, eps, delta, add, rows, out_dtype)
+    d = delta.delta if delta is not None else None
+    base, f32, parts, stride, ld = split_rows(d) if d is not None else (None, 1, 1, 0, w)
+    outs = [torch.empty(n, row_width(w, out_dtype), dtype=out_dtype, device=x.device) for wt in (weight, weight2) if wt is not None]
+    rc = _native.cuda().gb_stream_rms2(_p(x), _p(base), _i(f32), _i(parts), _l(stride), _i(ld), _p(delta.weight if delta is not None else None),
+                                       _f(delta.eps if delta is not None else 0.0), _p(add), _p(weight), _p(weight2), _p(rows), _p(outs[0]),
+                                       _p(outs[1] if weight2 is not None else None), _i(int(out_dtype == torch.float32)), _i(outs[0].shape[1]), _i(n), _i(w), _f(eps), _s())
+    _native.check(rc, "gb_stream_rms2")
+    return outs
+
+
+class _JoinPart(ctypes.Structure):
+    """``struct JoinPart`` of csrc/kernels/stream_ops.cu."""
+    _fields_ = [("p", ctypes.c_void_p), ("pair_row", ctypes.c_void_p), ("weights", ctypes.c_void_p), ("stride", ctypes.c_long), ("f32", ctypes.c_int),
+                ("n_part", ctypes.c_int), ("ld", ctypes.c_int), ("k", ctypes.c_int), ("scale", ctypes.c_float)]
+
+
+def join(x: torch.Tensor, parts: List[Tuple[object, float]], out_dtype=None) -> Optional[torch.Tensor]:
+    """``x += sum of factor * result`` in place (at most three (result, factor) pairs: tensors, partial sums or pending expert sums); returns the new rows in
+    ``out_dtype`` (None: nothing), of width ``row_width(W)``."""
+    t, w = x.shape
+    if not x.is_cuda:
+        x.add_(sum(whole(d)[:, :w] * f for d, f in parts))
+        if out_dtype is None:
+            return None
+        o = torch.zeros(t, row_width(w, out_dtype), dtype=out_dtype)
+        o[:, :w] = x.to(out_dtype)
+        return o
+    arr = (_JoinPart * 3)()
+    for a, (d, f) in zip(arr, parts):
+        a.scale = f
+        if hasattr(d, "pair_row"):
+            a.p, a.f32, a.n_part, a.ld = d.y.data_ptr(), int(d.y.dtype == torch.float32), 1, d.y.stride(0)
+            a.pair_row, a.weights, a.k = d.pair_row.data_ptr(), d.weights.data_ptr(), d.k
+        else:
+            base, a.f32, a.n_part, a.stride, a.ld = split_rows(d)
+            a.p = base.data_ptr()
+    out = torch.empty(t, row_width(w, out_dtype), dtype=out_dtype, device=x.device) if out_dtype is not None else None
+    rc = _native.cuda().gb_stream_join(_p(x), ctypes.byref(arr), _i(len(parts)), _p(out), _i(int(out_dtype == torch.float32)), _i(out.shape[1] if out is not None else 0), _i(t),
+                                       _i(w), _s())
+    _native.check(rc, "gb_stream_join")
+    return out
+
+
 def norm(x: torch.Tensor, weight, eps: float, delta=None, add: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
          out_dtype=torch.bfloat16) -> Optional[torch.Tensor]:
     """``x += delta + add`` in place (``x`` f32 ``[T, W]``; both optional), then ``x / rms(x) * weight`` (f32 ``[W]``), or ``weight(x)`` if it is a
     ``DynTanh``, as ``out_dtype`` rows of width ``row_width(W)``.  With ``rows`` (int64): only those stream rows are normalised, and the stream is left as it is.  ``weight``
     None: only the update."""
+    if isinstance(delta, RmsPosted):
+        return norm2(x, weight, eps, delta, add, rows, out_dtype=out_dtype)[0]
     t, w = x.shape
     n = t if rows is None else rows.numel()
     if not x.is_cuda:
@@ -156,6 +246,105 @@ def qk_unit(qkv, slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     return q
 
 
+def qk_rows(qkv, slots: torch.Tensor, q_norm: torch.Tensor, k_norm: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, hq: int, hkv: int, dk: int, dv: int,
+            eps: float, q_scale: float) -> torch.Tensor:
+    """As ``qk_unit``, with one RMS norm over all of Q and one over all of K (weights f32 ``[hq * dk]`` and ``[hkv * dk]``).  Columns behind V are not read."""
+    base, f32, parts, stride, ld = split_rows(qkv)
+    t = qkv.rows if hasattr(qkv, "buf") else qkv.shape[0]
+    nq, nk, dkp, dvp = hq * dk, hkv * dk, k_cache.shape[2], v_cache.shape[2]
+    if not base.is_cuda:
+        y = whole(qkv)
+        n = lambda z, w: z / torch.sqrt(z.pow(2).mean(-1, keepdim=True) + eps) * w
+        q, k, v = n(y[:, :nq], q_norm), n(y[:, nq: nq + nk], k_norm), y[:, nq + nk: nq + nk + hkv * dv]
+        pad = torch.nn.functional.pad
+        ok = slots >= 0
+        k_cache[slots[ok].long()] = pad(k.reshape(t, hkv, dk), (0, dkp - dk))[ok].to(k_cache.dtype)
+        v_cache[slots[ok].long()] = pad(v.reshape(t, hkv, dv), (0, dvp - dv))[ok].to(v_cache.dtype)
+        return pad(q.reshape(t, hq, dk) * q_scale, (0, dkp - dk)).to(k_cache.dtype)
+    q = torch.empty(t, hq, dkp, dtype=k_cache.dtype, device=base.device)
+    rc = _native.cuda().gb_qk_rows_store(_p(base), _i(f32), _i(parts), _l(stride), _i(ld), _p(slots), _p(q_norm), _p(k_norm), _p(q), _p(k_cache), _p(v_cache),
+                                         _i(int(k_cache.dtype == torch.float32)), _l(k_cache.shape[0]), _i(t), _i(hq), _i(hkv), _i(dk), _i(dv), _i(dkp), _i(dvp), _f(eps),
+                                         _f(q_scale), _s())
+    _native.check(rc, "gb_qk_rows_store")
+    return q
+
+
+def rotary_table(positions: torch.Tensor, freq: torch.Tensor, mag: float) -> torch.Tensor:
+    """f32 ``[T, pairs, 2]``: cos and sin of position * freq (f64 ``[pairs]``), times ``mag``."""
+    if not positions.is_cuda:
+        a = positions.double().unsqueeze(1) * freq
+        return torch.stack([torch.cos(a) * mag, torch.sin(a) * mag], dim=-1).float()
+    out = torch.empty(positions.numel(), freq.numel(), 2, dtype=torch.float32, device=positions.device)
+    _native.check(_native.cuda().gb_rotary_table(_p(positions), _p(freq), _f(mag), _p(out), _i(positions.numel()), _i(freq.numel()), _s()), "gb_rotary_table")
+    return out
+
+
+def conv_rotary(qk, table: torch.Tensor, slots: torch.Tensor, conv_w: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, seq_slots: torch.Tensor,
+                k_cache: torch.Tensor, v_cache: torch.Tensor, hq: int, hkv: int, d: int, q_scale: float, max_tokens: int) -> torch.Tensor:
+    """Rows ``[Q heads | K heads]`` through a causal convolution over time (``conv_w`` f32 ``[channels, taps]``, the last tap meets the current token; the last
+    ``taps - 1`` rows of a sequence are kept in ``state`` f32 ``[slots, taps - 1, channels]``), then neighbours (2i, 2i + 1) of each head turned by ``table``
+    (``rotary_table``; dimensions behind its pairs pass).  Returns ``q [T, hq, dkp]`` times ``q_scale``; the rotated K and the K before the rotation (as V) go to
+    cache slot ``slots[t]``.  ``max_tokens``: of the longest sequence."""
+    base, f32, parts, stride, ld = split_rows(qk)
+    t = qk.rows if hasattr(qk, "buf") else qk.shape[0]
+    ch, taps = conv_w.shape
+    dkp, dvp, dims = k_cache.shape[2], v_cache.shape[2], 2 * table.shape[1]
+    if not base.is_cuda:
+        x, y, cu = whole(qk)[:, :ch], torch.zeros(t, ch), cu_q.tolist()
+        for s in range(len(cu) - 1):
+            n = cu[s + 1] - cu[s]
+            if n:
+                rows = torch.cat([state[int(seq_slots[s])], x[cu[s]: cu[s + 1]]])
+                y[cu[s]: cu[s + 1]] = sum(conv_w[:, j] * rows[j: j + n] for j in range(taps))
+                state[int(seq_slots[s])] = rows[n:]
+        h = y.reshape(t, hq + hkv, d)
+        r = h.clone()
+        c, sn = table[:, :, 0].unsqueeze(1), table[:, :, 1].unsqueeze(1)
+        r[..., 0:dims:2], r[..., 1:dims:2] = h[..., 0:dims:2] * c - h[..., 1:dims:2] * sn, h[..., 1:dims:2] * c + h[..., 0:dims:2] * sn
+        pad = torch.nn.functional.pad
+        ok = slots >= 0
+        k_cache[slots[ok].long()] = pad(r[:, hq:], (0, dkp - d))[ok].to(k_cache.dtype)
+        v_cache[slots[ok].long()] = pad(h[:, hq:], (0, dvp - d))[ok].to(v_cache.dtype)
+        return pad(r[:, :hq] * q_scale, (0, dkp - d)).to(k_cache.dtype)
+    assert state.is_contiguous() and state.dtype == torch.float32
+    q = torch.empty(t, hq, dkp, dtype=k_cache.dtype, device=base.device)
+    rc = _native.cuda().gb_conv_rotary_store(_p(base), _i(f32), _i(parts), _l(stride), _i(ld), _p(table), _i(dims), _p(slots), _p(conv_w), _i(taps), _p(state),
+                                             _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(q), _p(k_cache), _p(v_cache), _i(int(k_cache.dtype == torch.float32)),
+                                             _l(k_cache.shape[0]), _i(hq), _i(hkv), _i(d), _i(dkp), _i(dvp), _f(q_scale), _i(max_tokens), _i(cu_q.numel() - 1), _s())
+    _native.check(rc, "gb_conv_rotary_store")
+    return q
+
+
+def sigmoid_gate(a: torch.Tensor, proj, col: int, dv: int) -> torch.Tensor:
+    """``a [T, H, dvp] *= sigmoid(gate)`` in place on the first ``dv`` columns of each head: the gate is columns ``col ...`` (head by head, ``dv`` each) of the
+    projection result ``proj``."""
+    t, hd, dvp = a.shape
+    base, f32, parts, stride, ld = split_rows(proj)
+    if not a.is_cuda:
+        g = torch.sigmoid(whole(proj)[:, col: col + hd * dv]).reshape(t, hd, dv)
+        a[:, :, :dv] = (a[:, :, :dv].float() * g).to(a.dtype)
+        return a
+    rc = _native.cuda().gb_sigmoid_gate(_p(a), _i(int(a.dtype == torch.float32)), _c(base.data_ptr() + col * base.element_size()), _i(f32), _i(parts), _l(stride), _i(ld),
+                                        _i(t), _i(hd), _i(dv), _i(dvp), _s())
+    _native.check(rc, "gb_sigmoid_gate")
+    return a
+
+
+def token_gate(z, ids: torch.Tensor, table: torch.Tensor, col: int, n: int, out_dtype=torch.bfloat16) -> torch.Tensor:
+    """``gelu(z) * table[id, col : col + n]`` (the tanh form of GELU) -> rows ``[T, row_width(n)]``; ``z`` is a projection result of ``n`` columns."""
+    base, f32, parts, stride, ld = split_rows(z)
+    t = z.rows if hasattr(z, "buf") else z.shape[0]
+    out = torch.empty(t, row_width(n, out_dtype), dtype=out_dtype, device=base.device)
+    if not base.is_cuda:
+        out.zero_()
+        out[:, :n] = (torch.nn.functional.gelu(whole(z)[:, :n], approximate="tanh") * table[ids.long(), col: col + n].float()).to(out_dtype)
+        return out
+    rc = _native.cuda().gb_token_gate(_p(base), _i(f32), _i(parts), _l(stride), _i(ld), _p(ids), _p(table), _i(int(table.dtype == torch.float32)), _i(table.shape[1]), _i(col),
+                                      _i(table.shape[0]), _p(out), _i(int(out_dtype == torch.float32)), _i(out.shape[1]), _i(t), _i(n), _s())
+    _native.check(rc, "gb_token_gate")
+    return out
+
+
 def gated_norm(o: torch.Tensor, proj, gate_col: int, weight: torch.Tensor, eps: float, out_dtype=torch.bfloat16) -> torch.Tensor:
     """``rms_norm(o) * weight * sigmoid(gate)``: ``o`` f32 ``[T, N]`` (all heads side by side), the gate is columns ``gate_col ...`` of the
     projection result ``proj``."""
@@ -175,17 +364,18 @@ def gated_norm(o: torch.Tensor, proj, gate_col: int, weight: torch.Tensor, eps: 
     return out
 
 
-def part_norm(o: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, gate=None, gate_col: int = 0, out_dtype=torch.bfloat16) -> torch.Tensor:
+def part_norm(o: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, gate=None, gate_col: int = 0, out_dtype=torch.bfloat16,
+              gate_after: bool = False) -> torch.Tensor:
     """``o`` f32 ``[T, N]`` times SiLU(gate) (columns ``gate_col ...`` of the projection result ``gate``, if given), then every one of ``parts`` equal
-    parts divided by its root mean square and multiplied by ``weight`` (f32 ``[N]``, or shorter and repeated)."""
+    parts divided by its root mean square and multiplied by ``weight`` (f32 ``[N]``, or shorter and repeated).  ``gate_after``: the gate multiplies the result."""
     t, n = o.shape
     ldo = row_width(n, out_dtype)
     if not o.is_cuda:
-        y = o
-        if gate is not None:
-            y = y * torch.nn.functional.silu(whole(gate)[:, gate_col: gate_col + n])
-        y = y.reshape(t, parts, n // parts)
+        g = torch.nn.functional.silu(whole(gate)[:, gate_col: gate_col + n]) if gate is not None else 1.0
+        y = (o if gate_after else o * g).reshape(t, parts, n // parts)
         y = (y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps)).reshape(t, n) * weight.repeat(n // weight.numel())
+        if gate_after:
+            y = y * g
         out = torch.zeros(t, ldo, dtype=out_dtype)
         out[:, :n] = y.to(out_dtype)
         return out
@@ -193,18 +383,18 @@ def part_norm(o: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, gat
     out = torch.empty(t, ldo, dtype=out_dtype, device=o.device)
     g = _c(base.data_ptr() + gate_col * base.element_size()) if gate is not None else _c(0)
     rc = _native.cuda().gb_part_norm(_p(o), _i(o.stride(0)), g, _i(f32), _i(np_), _l(stride), _i(ld), _p(weight), _i(weight.numel()), _p(out),
-                                     _i(int(out_dtype == torch.float32)), _i(ldo), _i(t), _i(n), _i(parts), _f(eps), _s())
+                                     _i(int(out_dtype == torch.float32)), _i(ldo), _i(t), _i(n), _i(parts), _f(eps), _i(int(gate_after)), _s())
     _native.check(rc, "gb_part_norm")
     return out
 
 
-def act_mul(gate_up: torch.Tensor, act: str) -> torch.Tensor:
-    """``act(gate) * up`` of f32 rows ``[gate | up]``."""
+def act_mul(gate_up: torch.Tensor, act: str, cap: float = 0.0) -> torch.Tensor:
+    """``act(gate) * up`` of f32 rows ``[gate | up]`` (``ops.gemm.gated_act_ref``)."""
     rows, two_i = gate_up.shape
     inter = two_i // 2
     if not gate_up.is_cuda:
-        return gate_act_ref(gate_up[:, :inter], act) * gate_up[:, inter:]
+        return gated_act_ref(gate_up[:, :inter], gate_up[:, inter:], act, cap)
     out = torch.empty(rows, inter, dtype=torch.float32, device=gate_up.device)
-    _native.check(_native.cuda().gb_act_mul_f32(_p(gate_up), _p(out), _l(rows), _i(inter), _i(gate_up.stride(0)), _i(1 if act == "gelu_tanh" else 0), _s()),
+    _native.check(_native.cuda().gb_act_mul_f32(_p(gate_up), _p(out), _l(rows), _i(inter), _i(gate_up.stride(0)), _i(GATE_ACT_CODE[act]), _f(cap), _s()),
                   "gb_act_mul_f32")
     return out

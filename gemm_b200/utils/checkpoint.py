@@ -3,11 +3,11 @@ later — e.g. to skip a long prefill when sweeping decode settings.
 
 Counterpart of the reference's 'TPCP' files (a64fx/llm/tp_runner.c:155-563: magic + version, model and TP geometry,
 cache position, next token, then per-layer K / V buffers; every header field is validated on load,
-tp_cache_matches_model :356-387).  Our file: magic ``GBKV1\\n``, a JSON header line (geometry, sequences), then for every layer
+tp_cache_matches_model :356-387).  Our file: magic ``GBKV1\\n``, a JSON header line (geometry, sequences), then for every layer its recurrent state, if it has one, and
 the K and V rows of the used cache slots in sequence order: bf16, or with ``kv_format="q8"`` int8 rows followed by one f32 scale per
-(slot, KV head) (``ops.kvquant``: about half the size, the reference's INT8 KV rule).  Layers of the hybrid models that keep a recurrent state
-instead of K/V (gated Delta-Net) write, per live sequence, the f32 conv history and the f32 recurrent matrix of its state slot
-(the reference stores conv state and recurrent state per layer as well, tp_runner.c:155-563).  A truncated or mismatching file
+(slot, KV head) (``ops.kvquant``: about half the size, the reference's INT8 KV rule).  Layers that keep a recurrent state, instead of K/V (gated
+Delta-Net) or beside it, write, per live sequence, the f32 tensors of its state slot (convolution history, recurrent matrix, row of the token in front;
+the reference stores conv state and recurrent state per layer as well, tp_runner.c:155-563).  A truncated or mismatching file
 is rejected.
 """
 from __future__ import annotations
@@ -58,10 +58,10 @@ def save_state(engine, path: str, next_tokens=None, kv_format: str = "bf16") -> 
         f.write(hb)
         n_seq = len(engine.seq_len)
         for li in range(len(engine.kv.k)):
+            # recurrent state: the slots of the live sequences (slot s belongs to sequence s in a static-batch engine)
+            for t in engine.kv.recurrent(li):
+                f.write(t[:n_seq].contiguous().cpu().numpy().tobytes())
             if engine.kv.k[li].shape[0] == 0:
-                # recurrent layer: the state slots of the live sequences (slot s belongs to sequence s in a static-batch engine)
-                for t in engine.kv.recurrent(li):
-                    f.write(t[:n_seq].contiguous().cpu().numpy().tobytes())
                 continue
             for t in (engine.kv.k[li], engine.kv.v[li]):
                 if t.shape[2] == 0:
@@ -111,15 +111,15 @@ def load_state(engine, path: str) -> torch.Tensor:
         idx = torch.tensor(slots, dtype=torch.long, device=engine.device)
         n_seq = len(header["seq_len"])
         for li in range(len(engine.kv.k)):
+            for t in engine.kv.recurrent(li):
+                nb = n_seq * t[0].numel() * 4
+                if nb == 0:
+                    continue
+                buf = f.read(nb)
+                if len(buf) != nb:
+                    raise ValueError("truncated KV state file")
+                t[:n_seq] = torch.frombuffer(bytearray(buf), dtype=torch.float32).reshape(n_seq, *t.shape[1:]).to(engine.device)
             if engine.kv.k[li].shape[0] == 0:
-                for t in engine.kv.recurrent(li):
-                    nb = n_seq * t[0].numel() * 4
-                    if nb == 0:
-                        continue
-                    buf = f.read(nb)
-                    if len(buf) != nb:
-                        raise ValueError("truncated KV state file")
-                    t[:n_seq] = torch.frombuffer(bytearray(buf), dtype=torch.float32).reshape(n_seq, *t.shape[1:]).to(engine.device)
                 continue
             for t in (engine.kv.k[li], engine.kv.v[li]):
                 if t.shape[2] == 0:
