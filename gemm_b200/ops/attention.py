@@ -32,6 +32,8 @@ def build_work(q_lens: Sequence[int], hq: int, hkv: int, num_splits: int = 1) ->
     the heads of one tile adjacent (their K/V blocks hit in L2)."""
     g = hq // hkv
     tpt = 128 // g
+    if tpt == 0:                          # more query heads per KV head than a tile has rows: no work for the tcgen05 kernels
+        return torch.zeros(0, 4, dtype=torch.int32)
     items: List[List[int]] = []
     for s, ql in enumerate(q_lens):
         n_tiles = (ql + tpt - 1) // tpt

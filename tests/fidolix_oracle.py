@@ -96,7 +96,8 @@ def left_mixer(h, t, pre, m):
     n, hd, g = h.shape[0], m["heads"], m["kv_heads"]
     q, k = (short_conv(h @ t[pre + c].t() + t[pre + c + ".b"], t[pre + c + ".conv"]) for c in "qk")
     q, k = q.reshape(n, hd, -1), k.reshape(n, g, -1)
-    o = attend(rotate(q, m["rot"]), rotate(k, m["rot"]), k, m["scale"], window=m["mask"]["size"], sink=t[pre + "sink"])
+    window = m["mask"]["size"] if m.get("mask") else None
+    o = attend(rotate(q, m["rot"]), rotate(k, m["rot"]), k, m["scale"], window=window, sink=t[pre + "sink"])
     return o.reshape(n, -1) @ t[pre + "o"].t()
 
 
