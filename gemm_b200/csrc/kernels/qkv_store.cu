@@ -32,7 +32,7 @@ struct QkRowsArgs {
   float eps, q_scale;
 };
 
-constexpr int kQkThreads = 512, kQkKeep = 4;                   // kQkKeep vectors of a thread stay in registers between the two passes
+constexpr int kQkThreads = 256, kQkKeep = 8;                   // kQkKeep vectors of a thread stay in registers between the two passes
 
 template <typename TI, typename TC, int V>                     // V neighbouring columns of a head (dk % V == 0, dv % V == 0)
 __global__ void __launch_bounds__(kQkThreads)

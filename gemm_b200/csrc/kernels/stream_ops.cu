@@ -323,11 +323,13 @@ stream_join_kernel(const JoinArgs a) {
       for (int j = 0; j < V; ++j) u[j] = fmaf(w, q[j], u[j]);
     };
     if (d.pair_row != nullptr) {
+#pragma unroll 4
       for (int e = 0; e < d.k; ++e) {
         const int row = d.pair_row[r * d.k + e];
         if (row >= 0) add((size_t)row * d.ld, d.weights[r * d.k + e]);
       }
     } else {
+#pragma unroll 4
       for (int p = 0; p < d.n_part; ++p) add((size_t)p * d.stride + r * d.ld, 1.0f);
     }
 #pragma unroll

@@ -266,6 +266,10 @@ SPLIT_PROJ = os.environ.get("GB_SPLIT_PROJ", "1") != "0"
 FUSE_ATTN_QUANT = os.environ.get("GB_FUSE_ATTN_QUANT", "1") != "0"
 
 
+# mixers and feed-forward that read the same stream as branches of a captured decode step (GB_BRANCHES=0: one after the other)
+BRANCHES = os.environ.get("GB_BRANCHES", "1") != "0"
+
+
 PAIR_DOWN = os.environ.get("GB_PAIR_DOWN", "1") != "0"
 
 
@@ -400,6 +404,7 @@ class Transformer:
             if weights.embed.is_cuda and not cfg.is_layered else None
         self.mixer_blocks = {"attention": self.masked_attention_block, "lightning": self.lightning_block, "mamba2": self.mamba2_block, "hgrn2": self.hgrn2_block,
                              "latent": self.latent_block, "rwkv": self.rwkv_block}
+        self._branches: List = []      # streams of a captured step's branches
         self.snapshots = {}            # layer -> hidden rows captured after that layer (debug / DeepStack)
         self.snapshot_layers: Sequence[int] = ()
 
@@ -569,32 +574,60 @@ class Transformer:
         else:
             # decode-sized batches keep the projections in f32
             rkvg = torch.empty(4, pad, ld, dtype=torch.float32 if t <= 64 else torch.bfloat16, device=h.device)
-            gemm.grouped_linear(mix[:4].view(4 * pad, -1), w.w_in.w.view(4, w.w_in.rows_per_group, -1), seg, cnt, min(pad, 128), out=rkvg.view(4 * pad, ld), n_out=n,
-                                w_tiled=w.w_in.tiled)
-        z = apply_linear_stream(w.w2, recurrent.tanh_rows(apply_linear_stream(w.w1, mix[4, :t]), sp.decay_rank, self.act_dtype))
-        o = recurrent.rwkv(rkvg, z, w.w0, w.u, self.kv.rec[li], fb.cu_q, fb.seq_slots, sp.n_heads, sp.head_dim, sp.v_dim, t, most)
+            gemm.grouped_linear(mix[:4].view(4 * pad, -1), w.w_in.w.view(4, w.w_in.rows_per_group, -1), seg, cnt, 256 if pad >= 512 else min(pad, 128), out=rkvg.view(4 * pad, ld),
+                                n_out=n, w_tiled=w.w_in.tiled)
+        z, w2 = apply_linear_stream(w.w1, mix[4, :t]), None
+        if w.w2_rows is not None and recurrent.can_fuse_decay(t, most, sp.decay_rank):
+            w2 = w.w2_rows
+        else:
+            z = apply_linear_stream(w.w2, recurrent.tanh_rows(z, sp.decay_rank, self.act_dtype))
+        o = recurrent.rwkv(rkvg, z, w.w0, w.u, self.kv.rec[li], fb.cu_q, fb.seq_slots, sp.n_heads, sp.head_dim, sp.v_dim, t, most, w2)
         y = stream.part_norm(o, w.norm, sp.n_heads, self.cfg.rms_eps, rkvg[3, :t], 0, self.act_dtype, gate_after=True)
         return apply_linear_stream(w.w_out, y)
+
+    def branch(self, i: int, x: torch.Tensor, fn):
+        """``fn()`` as branch ``i`` of the graph while a decode step is captured, beside what the current stream does until ``join_branch(i)``; at once otherwise.
+        What the branch reads must stay alive until then: memory is handed out again in the order of the stream that asked for it."""
+        if not (BRANCHES and x.is_cuda and torch.cuda.is_current_stream_capturing()):
+            return fn()
+        while len(self._branches) <= i:
+            self._branches.append(torch.cuda.Stream(x.device))
+        side = self._branches[i]
+        side.wait_stream(torch.cuda.current_stream())
+        with torch.cuda.stream(side):
+            return fn()
+
+    def join_branch(self, i: int, x: torch.Tensor) -> None:
+        if BRANCHES and x.is_cuda and torch.cuda.is_current_stream_capturing():
+            torch.cuda.current_stream().wait_stream(self._branches[i])
 
     def mixer_parts(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
         """(result, factor) of the mixer, or of each of the two side by side."""
         if sp.mixer != "parallel":
             return [(self.mixer_blocks[sp.mixer](li, lw, sp, h, fb), 1.0)]
-        return [(self.mixer_blocks[m.mixer](li, lw, m, h, fb), f) for m, f in ((sp.left, sp.left_scale), (sp.right, sp.right_scale))]
+        right = self.branch(1, h, lambda: self.mixer_blocks[sp.right.mixer](li, lw, sp.right, h, fb))
+        left = self.mixer_blocks[sp.left.mixer](li, lw, sp.left, h, fb)
+        self.join_branch(1, h)
+        return [(left, sp.left_scale), (right, sp.right_scale)]
 
     def parallel_layer(self, li: int, lw, sp: LayerSpec, x: torch.Tensor, delta, first: Optional[torch.Tensor], fb: ForwardBatch):
         """A layer whose mixer and feed-forward read the same stream, with the token input behind them; returns the pending update of the token input."""
         cfg, layer = self.cfg, self.runs[li].layer
         hs = stream.norm2(x, lw.attn_norm, cfg.rms_eps, delta, add=first if self.runs[li].again else None, weight2=lw.ffn_norm, out_dtype=self.act_dtype)
+        ffn = None
+        if sp.has_ffn:
+            with profiler.region("ffn", "block", "ffn", li):
+                ffn = self.branch(0, x, lambda: self.stream_ffn(lw, sp, hs[1]))
         with profiler.region(sp.mixer, "block", "attention", li):
             parts = self.mixer_parts(li, lw, sp, hs[0], fb)
         if sp.has_ffn:
-            with profiler.region("ffn", "block", "ffn", li):
-                parts.append((self.stream_ffn(lw, sp, hs[1]), 1.0))
+            self.join_branch(0, x)
+            parts.append((ffn, 1.0))
         rows = stream.join(x, parts, self.act_dtype if lw.side is not None else None)
         if lw.side is None:
             return None
-        g = stream.token_gate(apply_linear_stream(lw.side.gate, rows), fb.ids, self.w.side_embed, layer * cfg.side_dim, cfg.side_dim, self.act_dtype)
+        z = apply_linear_stream(lw.side.gate, rows)
+        g = stream.token_gate(z, fb.ids, self.w.side_embed, layer * cfg.side_dim, cfg.side_dim, self.act_dtype)
         return stream.RmsPosted(apply_linear_stream(lw.side.proj, g), lw.side.norm, cfg.rms_eps)
 
     def lightning_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):

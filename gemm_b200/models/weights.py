@@ -292,13 +292,15 @@ class RwkvWeights:
     w_in: LinearWeight
     w1: LinearWeight              # [rank, H]
     w2: LinearWeight              # [heads * dim, rank]
+    w2_rows: Optional[torch.Tensor]   # bf16, the same row by row, for the step kernel (None in 32-bit)
     w0: torch.Tensor              # f32 [heads * dim]
     u: torch.Tensor               # f32 [heads * dim]: weight of the current token
     norm: torch.Tensor            # f32 [heads * v_dim]
     w_out: LinearWeight
 
     def to(self, device) -> "RwkvWeights":
-        return RwkvWeights(*(t.to(device) for t in (self.mu, self.w_in, self.w1, self.w2, self.w0, self.u, self.norm, self.w_out)))
+        return RwkvWeights(*(t.to(device) for t in (self.mu, self.w_in, self.w1, self.w2)), self.w2_rows.to(device) if self.w2_rows is not None else None,
+                           *(t.to(device) for t in (self.w0, self.u, self.norm, self.w_out)))
 
 
 @dataclass
@@ -748,8 +750,9 @@ class _LayeredBuilder:
         assert nq == nv, "the four projections of the mixes share a size"
         np_ = nq if self.exact else (nq + 127) // 128 * 128              # whole 128-row tiles per group
         w = [torch.nn.functional.pad(self.get(pre + f"rwkv_{c}.weight", nq, h), (0, 0, 0, np_ - nq)) for c in "rkvg"]
+        w2 = self.get(pre + "rwkv_w2.weight", nq, sp.decay_rank)
         lw.rwkv = RwkvWeights(mu=torch.stack([self.f32(pre + f"rwkv_mu_{c}", h) for c in "rkvgw"]).contiguous(), w_in=self.linear(torch.cat(w), groups=4),
-                              w1=self.linear(self.get(pre + "rwkv_w1.weight", sp.decay_rank, h)), w2=self.linear(self.get(pre + "rwkv_w2.weight", nq, sp.decay_rank)),
+                              w1=self.linear(self.get(pre + "rwkv_w1.weight", sp.decay_rank, h)), w2=self.linear(w2), w2_rows=None if self.exact else w2.to(torch.bfloat16).contiguous().to(self.dev, copy=True),
                               w0=self.f32(pre + "rwkv_w0", nq), u=self.f32(pre + "rwkv_u", sp.n_heads, sp.head_dim).reshape(-1), norm=self.f32(pre + "rwkv_norm.weight", nv),
                               w_out=self.linear(self.get(pre + "rwkv_out.weight", h, nv)))
 

@@ -13,6 +13,7 @@ from __future__ import annotations
 
 import ctypes
 import os
+from typing import Optional
 
 import torch
 
@@ -226,19 +227,28 @@ def rwkv_ref(r, k, v, z, u, state, cu_q, seq_slots, heads, dim, vdim):
     return out
 
 
+def can_fuse_decay(tokens: int, max_tokens: int, rank: int) -> bool:
+    """Whether ``rwkv`` forms the decays from the middle of their low-rank projection: short portions of a few tokens (each sequence and
+    head reads its part of the matrix), ranks up to 256."""
+    return tokens <= 32 and max_tokens < CHUNKED_MIN_TOKENS and rank <= 256
+
+
 def rwkv(rkv: torch.Tensor, z, w0: torch.Tensor, u: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, seq_slots: torch.Tensor, heads: int, dim: int, vdim: int,
-         tokens: int, max_tokens: int = 1) -> torch.Tensor:
+         tokens: int, max_tokens: int = 1, w2: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``rkv [>= 3, pad, ld]``: receptances, keys and values of ``tokens`` tokens; ``z``: projection result (f32 or partial sums) whose columns, plus ``w0``, are the
-    decay exponents (w = exp(-exp(z + w0))); ``u`` f32 ``[heads * dim]``.  Returns f32 ``[tokens, heads * vdim]``."""
+    decay exponents (w = exp(-exp(z + w0))); ``u`` f32 ``[heads * dim]``.  ``w2`` (bf16 ``[heads * dim, rank]``, see ``can_fuse_decay``): ``z`` is the middle of a
+    low-rank projection, and the exponents are ``w2 tanh(z) + w0``.  Returns f32 ``[tokens, heads * vdim]``."""
     gb, gf32, gparts, gstride, gld = split_rows(z)
     nq, nv = heads * dim, heads * vdim
     if not rkv.is_cuda:
-        x = rkv[:, :tokens].float()
-        return rwkv_ref(x[0, :, :nq], x[1, :, :nq], x[2, :, :nv], whole(z)[:, :nq] + w0, u, state, cu_q, seq_slots, heads, dim, vdim)
+        x, e = rkv[:, :tokens].float(), whole(z)
+        if w2 is not None:
+            e = torch.tanh(e[:, : w2.shape[1]]) @ w2.float().t()
+        return rwkv_ref(x[0, :, :nq], x[1, :, :nq], x[2, :, :nv], e[:, :nq] + w0, u, state, cu_q, seq_slots, heads, dim, vdim)
     assert gf32 and state.is_contiguous() and state.dtype == torch.float32 and rkv.stride(2) == 1
     out = torch.empty(tokens, nv, dtype=torch.float32, device=rkv.device)
     ld, gs = rkv.stride(1), rkv.stride(0)
-    if CHUNKED and max_tokens >= CHUNKED_MIN_TOKENS and can_chunk(rkv[0], dim, vdim) and gs % 8 == 0:
+    if w2 is None and CHUNKED and max_tokens >= CHUNKED_MIN_TOKENS and can_chunk(rkv[0], dim, vdim) and gs % 8 == 0:
         lib, n_seqs = _native.cuda(), cu_q.numel() - 1
         lib.gb_gla_chunk_workspace.restype = _l
         nb = int(lib.gb_gla_chunk_workspace(_l(tokens), _i(n_seqs), _i(heads), _i(dim)))
@@ -247,7 +257,8 @@ def rwkv(rkv: torch.Tensor, z, w0: torch.Tensor, u: torch.Tensor, state: torch.T
                                _p(seq_slots), _p(out), _i(nv), _i(heads), _i(dim), _i(vdim), _i(max_tokens), _i(n_seqs), _p(ws), _l(nb), _c(_native.status_ptr()), _s())
         _native.check(rc, "gb_rwkv_chunk", n=2)
         return out
-    rc = _native.cuda().gb_rwkv_step(_p(rkv), _i(int(rkv.dtype == torch.float32)), _l(gs), _i(ld), _p(gb), _i(gparts), _l(gstride), _i(gld), _p(w0), _p(u), _p(state),
-                                     _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(nv), _i(heads), _i(dim), _i(vdim), _i(cu_q.numel() - 1), _s())
+    rc = _native.cuda().gb_rwkv_step(_p(rkv), _i(int(rkv.dtype == torch.float32)), _l(gs), _i(ld), _p(gb), _i(gparts), _l(gstride), _i(gld), _p(w2),
+                                     _i(w2.shape[1] if w2 is not None else 0), _p(w0), _p(u), _p(state), _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(nv), _i(heads),
+                                     _i(dim), _i(vdim), _i(cu_q.numel() - 1), _s())
     _native.check(rc, "gb_rwkv_step")
     return out

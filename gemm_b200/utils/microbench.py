@@ -22,6 +22,8 @@ Cases
                plain causal kernels; the f32-stream norm, Q / K unit norm and gated norm and their bf16-stream counterparts
   famepel      the kernels of Famepel at the sizes of ``famepel-30b-a3b`` beside the like kernels of the other models: Mamba-2 and HGRN2
                scans and Delta-Net; latent attention and plain attention; Dynamic-Tanh stream and RMSNorm, part norm, convolution, routing
+  fidolix      the kernels of Fidolix at the sizes of ``fidolix-30b-a3b`` beside the like kernels of the other models: RWKV (HGRN2), token shift,
+               convolution and rotation, norms of Q and K, capped scores and sinks (plain attention), the stream's norms and sums
   spec_verify  whole-model step over 1, 2, 3 and 5 positions per sequence (speculative verification against plain decode);
                builds the full Qwen3-30B-A3B shape, not part of ``all``
 
@@ -552,10 +554,125 @@ def case_famepel(args):
         _run(f"qk_norm_rope_{t}", lambda: ew.qk_norm_rope(qkv, pos, pos, qw, qw, kc, vc, hd, 4, 128, 1e6, 1e-6, 1.0, table=tab), 0.0, t * (hd + 8) * 128 * 4, args)
 
 
+def case_fidolix(args):
+    from ..models.config import get_config
+    from ..ops import recurrent, stream
+    dev, page = "cuda", 128
+    cfg = get_config("fidolix-30b-a3b")
+    spec = {sp.mixer: sp for sp in cfg.layer_specs}
+    at, lf, rw, h = spec["attention"], spec["parallel"].left, spec["parallel"].right, cfg.hidden
+    f32 = dict(device=dev, dtype=torch.float32)
+    for name, lens in (("decode_1", [1]), ("decode_64", [1] * 64), ("prefill_1x8192", [8192]), ("prefill_8x2048", [2048] * 8)):
+        t, b, dec = sum(lens), len(lens), len(lens) == sum(lens)
+        cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        sl = torch.arange(b, dtype=torch.int32, device=dev)
+        n, hd, d = rw.q_dim, rw.n_heads, rw.head_dim
+        dt = torch.float32 if dec else torch.bfloat16
+        es = 4 if dec else 2
+        # recurrence, beside HGRN2 of the same sizes
+        pad = recurrent.shift_pad(t)
+        rkvg, z = torch.randn(4, pad, n, device=dev).to(dt), torch.randn(t, n, device=dev) - 3
+        st = torch.randn(b, hd, d, d, device=dev) * 0.1
+        w0, u, low = torch.zeros(n, device=dev), torch.randn(n, device=dev), torch.full((n,), 0.3, device=dev)
+        _run(f"rwkv_{name}", lambda: recurrent.rwkv(rkvg, z, w0, u, st, cu, sl, hd, d, d, t, max(lens)), 4.0 * t * hd * d * d, 2 * st.numel() * 4 + t * (3 * n * es + n * 4 + n * 4), args)
+        qv = torch.randn(t, 2 * n, device=dev).to(dt)
+        _run(f"gla_{name}", lambda: recurrent.gla(qv, z, 0, w0, low, st, cu, sl, hd, d, d, not dec, max(lens)), 4.0 * t * hd * d * d,
+             2 * st.numel() * 4 + t * (2 * n * es + n * 4 + n * 4), args)
+        del st, qv
+        x = torch.randn(t, h, device=dev).bfloat16()
+        mu, sh = torch.rand(5, h, device=dev), torch.zeros(b, 1, h, **f32)
+        _run(f"token_shift_{name}", lambda: recurrent.token_shift(x, h, mu, sh, cu, sl, pad, max(lens)), 0.0, t * h * 12, args)
+        lr = torch.randn(t, rw.decay_rank, device=dev)
+        _run(f"tanh_rows_{name}", lambda: recurrent.tanh_rows(lr, rw.decay_rank), 0.0, lr.numel() * 6, args)
+        o, nw = torch.randn(t, n, device=dev), torch.ones(n, device=dev)
+        gate = rkvg[3, :t]
+        _run(f"part_norm_gate_after_{name}", lambda: stream.part_norm(o, nw, hd, 1e-5, gate, gate_after=True), 0.0, t * n * (4 + es + 2), args)
+        _run(f"part_norm_gated_{name}", lambda: stream.part_norm(o, nw, hd, 1e-5, gate), 0.0, t * n * (4 + es + 2), args)
+        wg = (torch.randn(4, n, h, device=dev) * 0.02).bfloat16()
+        seg, cnt = torch.arange(4, dtype=torch.int32, device=dev) * pad, torch.full((4,), t, dtype=torch.int32, device=dev)
+        mix = torch.randn(4 * pad, h, device=dev).bfloat16()
+        wt = mxfp8.tile_weight(wg.view(4 * n, h)).view(4, n, h)
+        _run(f"grouped_rkvg_{name}", lambda: gemm.grouped_linear(mix, wt, seg, cnt, min(pad, 128), out=rkvg.view(4 * pad, n), w_tiled=True), 8.0 * t * n * h,
+             4 * n * h * 2 + 4 * t * h * 2 + 4 * t * n * es, args)
+        _run(f"gemm_same_size_{name}", lambda: gemm.linear(x, wt.view(4 * n, h), w_tiled=True, out_dtype=dt), 8.0 * t * n * h, 4 * n * h * 2 + t * h * 2 + 4 * t * n * es, args)
+        del rkvg, mix, o, z
+        # from projection to attention
+        ch = lf.conv_channels
+        rows, cw, cst = torch.randn(t, ch, device=dev).to(dt), torch.randn(ch, lf.conv_taps, device=dev), torch.zeros(b, lf.conv_taps - 1, ch, **f32)
+        pos = torch.arange(t, device=dev, dtype=torch.int32)
+        freq = torch.tensor(lf.rotary.frequencies(), dtype=torch.float64, device=dev)
+        tab = stream.rotary_table(pos, freq, 1.1)
+        kc, vc = (torch.empty(t, lf.n_kv_heads, lf.head_dim, device=dev, dtype=torch.bfloat16) for _ in range(2))
+        nk = lf.n_kv_heads * lf.head_dim
+        _run(f"rotary_table_{name}", lambda: stream.rotary_table(pos, freq, 1.1), 0.0, tab.numel() * 4, args)
+        _run(f"conv_rotary_{name}", lambda: stream.conv_rotary(rows, tab, pos, cw, cst, cu, sl, kc, vc, lf.n_heads, lf.n_kv_heads, lf.head_dim, 0.1, max(lens)), 0.0,
+             t * (ch * (es + 2) + nk * 2 + tab.shape[1] * 8) + 2 * cst.numel() * 4, args)
+        cb = torch.zeros(ch, device=dev)
+        _run(f"causal_conv_{name}", lambda: recurrent.causal_conv(rows, 0, cw, cb, cst, cu, sl, max(lens)), 0.0, t * ch * (es + 2) + 2 * cst.numel() * 4, args)
+        nq, nk, nv = at.q_dim, at.n_kv_heads * at.head_dim, at.n_heads * at.v_dim
+        rows = torch.randn(t, nq + 2 * nk + nv, device=dev).to(dt)
+        qn, kn = torch.ones(nq, device=dev), torch.ones(nk, device=dev)
+        kc, vc = (torch.empty(t, at.n_kv_heads, at.head_dim, device=dev, dtype=torch.bfloat16) for _ in range(2))
+        by = t * (nq + 2 * nk) * (es + 2)
+        _run(f"qk_rows_{name}", lambda: stream.qk_rows(rows, pos, qn, kn, kc, vc, at.n_heads, at.n_kv_heads, at.head_dim, at.v_dim, 1e-5, 0.1), 0.0, by, args)
+        _run(f"qk_unit_{name}", lambda: stream.qk_unit(rows, pos, kc, vc, at.n_heads, at.n_kv_heads, at.head_dim, at.v_dim, 1e-5, 0.1), 0.0, by, args)
+        a = torch.randn(t, at.n_heads, at.v_dim, device=dev).bfloat16()
+        _run(f"sigmoid_gate_{name}", lambda: stream.sigmoid_gate(a, rows, nq + 2 * nk, at.v_dim), 0.0, t * nv * (4 + es), args)
+        del rows, a
+    # attention: capped scores over everything, sinks over a window, and the plain and biased forms of the same sizes
+    for name, b, q_len, ctx in (("decode_1x32768", 1, 1, 32767), ("decode_64x2048", 64, 1, 2047), ("decode_64x8192", 64, 1, 8191), ("prefill_1x8192", 1, 8192, 0), ("prefill_8x2048", 8, 2048, 0)):
+        for sp, win in ((at, 0), (lf, lf.window)):
+            hq, hkv, d = sp.n_heads, sp.n_kv_heads, sp.head_dim
+            kv, dec = ctx + q_len, q_len == 1
+            pages = (kv + page - 1) // page
+            k, v = ((torch.randn((b * pages + 1) * page, hkv, d, device=dev) * 0.5).bfloat16() for _ in range(2))
+            bt = torch.arange(b * pages, device=dev, dtype=torch.int32).reshape(b, pages) + 1
+            cu, kvl = torch.tensor([i * q_len for i in range(b + 1)], device=dev, dtype=torch.int32), torch.full((b,), kv, device=dev, dtype=torch.int32)
+            seen = float(sum(min(i + 1, win or kv) for i in range(ctx, kv)) * b)
+            by = b * min(kv, (win or kv) + q_len) * hkv * d * 4 + b * q_len * hq * d * 4
+            splits = att.pick_splits(b, hkv, min(kv, win + 128) if win else kv) if dec else 1
+            plan = (att.build_work([q_len] * b, hq, hkv, splits).to(dev), splits)
+            sink = torch.zeros(hq, device=dev)
+            q = (torch.randn(b * q_len, hq, d, device=dev) * 0.5 * d ** -0.5).bfloat16()
+            run = lambda nm, qq, **kw: _run(f"attn_{nm}_{name}", lambda: att.attention_masked(qq, k, v, cu, kvl, bt, page, win, plan=plan, decode=dec, **kw), 4.0 * seen * hq * d, by, args,
+                                            splits=splits)
+            if win:
+                run("window_sink", q * att.LOG2E, sink=sink)
+                _run(f"attn_window_{name}", lambda: att.attention(q, k, v, cu, kvl, bt, page, plan[0], num_splits=splits, window=win, decode=dec), 4.0 * seen * hq * d, by, args, splits=splits)
+            else:
+                run("capped", (q / at.softcap).bfloat16(), softcap=at.softcap)                                   # scores well within the cap
+                run("capped_wide", (q * 40.0 / at.softcap).bfloat16(), softcap=at.softcap)                       # ... and around it
+                _run(f"attn_{name}", lambda: att.attention(q, k, v, cu, kvl, bt, page, plan[0], num_splits=splits, decode=dec), 4.0 * seen * hq * d, by, args, splits=splits)
+            del k, v
+    for t in (1, 64, 8192):
+        x, u = torch.randn(t, h, device=dev), torch.randn(t, h, device=dev)
+        w1, w2, w3 = (torch.ones(h, device=dev) for _ in range(3))
+        _run(f"stream_rms2_{t}x{h}", lambda: stream.norm2(x, w1, 1e-5, stream.RmsPosted(u, w3, 1e-5), weight2=w2), 0.0, t * h * 16, args)
+        _run(f"stream_norm_{t}x{h}", lambda: stream.norm(x, w1, 1e-5, u), 0.0, t * h * 14, args)
+        k, e = 8, 128
+        y = torch.randn(t * k, h, device=dev).bfloat16()
+        pend = moe.PendingCombine(y, torch.randperm(t * k, device=dev).to(torch.int32), torch.rand(t, k, device=dev), t, k)
+        u2 = torch.randn(t, h, device=dev)
+        _run(f"stream_join_moe_{t}x{h}", lambda: stream.join(x, [(u, 1.0), (u2, 1.0), (pend, 1.0)], torch.bfloat16), 0.0, t * h * (18 + 2 * k), args)
+        xb = x.bfloat16()
+        _run(f"rmsnorm_moe_{t}x{h}", lambda: ew.rmsnorm(pend, w1.bfloat16(), 1e-5, residual=xb), 0.0, t * h * (6 + 2 * k), args)
+        z, sd = torch.randn(t, cfg.side_dim, device=dev), cfg.side_dim
+        table, ids = torch.randn(4096, 45 * sd, device=dev).bfloat16(), torch.randint(0, 4096, (t,), device=dev, dtype=torch.int32)
+        _run(f"token_gate_{t}", lambda: stream.token_gate(z, ids, table, 3 * sd, sd), 0.0, t * sd * 8, args)
+        z = torch.randn(t, e, device=dev)
+        for best in (1, 2):
+            _run(f"route_8_groups_best{best}_{t}", lambda: moe.route(z, k, "softmax", None, 2, 1.0, None, (8, 4, best)), 0.0, t * (e * 4 + k * 8), args)
+        ff = 6144
+        wg = mxfp8.tile_weight((torch.randn(2 * ff, h, device=dev) * 0.02).bfloat16())
+        for act in ("silu", "capped"):
+            _run(f"gate_up_{act}_{t}", lambda: gemm.linear_swiglu(xb, wg, w_tiled=True, act=act, cap=7.0), 4.0 * t * ff * h, 2 * ff * h * 2 + t * h * 2 + t * ff * 2, args)
+        del wg
+
+
 MODEL_CASES = {"spec_verify": case_spec_verify}      # build the whole benchmark model: not part of --case all
 CASES = {"gemm": case_gemm, "moe_decode": case_moe_decode, "moe_prefill": case_moe_prefill, "attn_decode": case_attn_decode,
          "attn_prefill": case_attn_prefill, "lm_head": case_lm_head, "quant": case_quant, "small": case_small, "layered": case_layered,
-         "famepel": case_famepel}
+         "famepel": case_famepel, "fidolix": case_fidolix}
 
 
 def main(argv=None):

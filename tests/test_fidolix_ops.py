@@ -375,7 +375,7 @@ def test_decay_projection_and_head_norm(device):
 
 
 @pytest.mark.parametrize("device", DEVICES)
-@pytest.mark.parametrize("t", [1, 5, 16, 70, 200])
+@pytest.mark.parametrize("t", [1, 5, 16, 70, 200, 600])
 def test_projections_of_the_mixes(t, device):
     """One grouped product for four mixes: f32 and 16-bit results, feature counts off and on the tiles, rows behind the tokens left over."""
     g = gen(t)
@@ -389,8 +389,10 @@ def test_projections_of_the_mixes(t, device):
         ref = torch.bmm(x[:, :t].double(), w[:, :n].double().transpose(1, 2))
         for dtype, tol in ((torch.float32, 1e-5), (torch.bfloat16, 5e-3)):
             out = torch.zeros(4, pad, n + 8, dtype=dtype, device=device)
-            gemm.grouped_linear(x.to(device).view(4 * pad, k), w.to(device), seg, cnt, min(pad, 128), out=out.view(4 * pad, n + 8), n_out=n)
-            assert rel(out[:, :t, :n], ref) < tol and not out[:, :, n:].any()
+            for tn in {min(pad, 128), 256 if pad >= 256 else min(pad, 128)}:
+                gemm.grouped_linear(x.to(device).view(4 * pad, k), w.to(device), seg, cnt, tn, out=out.view(4 * pad, n + 8), n_out=n)
+                assert rel(out[:, :t, :n], ref) < tol and not out[:, :, n:].any()
+                out.zero_()
     check_status(device)
 
 
@@ -528,3 +530,29 @@ def test_token_gate(n, device):
         got = stream.token_gate(z.to(device), ids.to(device), table.bfloat16().to(device), col, n)
         ref = O.gelu_tanh(z[:, :n].double()) * table.bfloat16().double()[ids.long(), col: col + n]
         assert got.shape[1] == stream.row_width(n, torch.bfloat16) and rel(got[:, :n], ref) < 8e-3 and not got[:, n:].any()
+
+
+# ------------------------------------------------------------------------------------------ fused steps of decoding
+@pytest.mark.parametrize("device", DEVICES)
+@pytest.mark.parametrize("heads,dim,rank", [(2, 128, 64), (3, 24, 12), (1, 8, 1), (2, 136, 32), (4, 40, 256), (5, 9, 48)])
+def test_rwkv_with_its_low_rank_decay(heads, dim, rank, device):
+    """The step forms the decays itself: single tokens and short portions."""
+    for lens in ([1] * 9, [1], [3, 1, 15, 2]):
+        g = gen(rank + len(lens))
+        t, n = sum(lens), heads * dim
+        r, k, v = (rnd(g, t, n) for _ in range(3))
+        w0, u, w2, z = rnd(g, n) - 2.0, rnd(g, n), rnd(g, n, rank, s=1.5 * rank ** -0.5).bfloat16(), rnd(g, t, rank, s=2.0)
+        cu, slots = batch(lens, device)
+        state = torch.zeros(len(lens) + 3, heads, dim, dim, device=device)
+        s0 = rnd(g, len(lens), heads, dim, dim)
+        state[slots.long()] = s0.to(device)
+        assert recurrent.can_fuse_decay(t, max(lens), rank)
+        got = recurrent.rwkv(torch.stack([r, k, v]).to(device), halves(z, device), w0.to(device), u.to(device), state, cu, slots, heads, dim, dim, t, max(lens), w2.to(device)).cpu()
+        w = torch.exp(-torch.exp(torch.tanh(z.double()) @ w2.double().t() + w0.double()))
+        for i, m in enumerate(lens):
+            s = slice(int(cu[i]), int(cu[i]) + m)
+            sh = lambda x: x[s].double().reshape(m, heads, dim)
+            ref = O.time_recurrence(sh(r), sh(k), sh(v), sh(w), u.double().reshape(heads, dim))
+            decay = torch.cumprod(torch.cat([torch.ones(1, heads, dim, dtype=torch.float64), sh(w)[:-1]]), 0)
+            ref = ref + torch.einsum("hde,thd->the", s0[i].double(), decay * sh(r))                # what the state in front of the portion adds
+            assert rel(got[s], ref.reshape(m, n)) < 1e-4
