@@ -32,21 +32,20 @@ struct QkRowsArgs {
   float eps, q_scale;
 };
 
-constexpr int kQkThreads = 256, kQkKeep = 8;                   // kQkKeep vectors of a thread stay in registers between the two passes
-
-template <typename TI, typename TC, int V>                     // V neighbouring columns of a head (dk % V == 0, dv % V == 0)
-__global__ void __launch_bounds__(kQkThreads)
+// V neighbouring columns of a head (dk % V == 0, dv % V == 0); NT threads, of which each keeps KEEP vectors in registers between the two passes.
+template <typename TI, typename TC, int V, int NT, int KEEP>
+__global__ void __launch_bounds__(NT)
 qk_rows_store_kernel(const QkRowsArgs a) {
   pdl_wait();
   pdl_trigger();
-  __shared__ float red[2][kQkThreads / 32];
+  __shared__ float red[2][NT / 32];
   const int t = blockIdx.x, tid = threadIdx.x;
   const TI* row = (const TI*)a.qkv + (size_t)t * a.ld;
   const int nq = a.hq * a.dk / V, nk = a.hkv * a.dk / V, nv = a.hkv * a.dv / V;     // vectors: Q, then K, then V, as the columns lie
   const int slot = a.slots[t];
   const bool store = slot >= 0 && slot < a.num_slots;
   const int n = store ? nq + nk + nv : nq;
-  float keep[kQkKeep][V], sq = 0.f, sk = 0.f;
+  float keep[KEEP][V], sq = 0.f, sk = 0.f;
   auto square = [&](int x, const float* v) {
     float s = 0.f;
 #pragma unroll
@@ -54,13 +53,13 @@ qk_rows_store_kernel(const QkRowsArgs a) {
     if (x < nq) sq += s; else sk += s;
   };
 #pragma unroll
-  for (int i = 0; i < kQkKeep; ++i) {
-    const int x = tid + i * kQkThreads;
+  for (int i = 0; i < KEEP; ++i) {
+    const int x = tid + i * NT;
     if (x >= n) continue;
     load_sum<TI, V>(row + (size_t)x * V, a.n_part, a.part_stride, keep[i]);
     if (x < nq + nk) square(x, keep[i]);
   }
-  for (int x = tid + kQkKeep * kQkThreads; x < min(n, nq + nk); x += kQkThreads) {
+  for (int x = tid + KEEP * NT; x < min(n, nq + nk); x += NT) {
     float v[V];
     load_sum<TI, V>(row + (size_t)x * V, a.n_part, a.part_stride, v);
     square(x, v);
@@ -70,7 +69,7 @@ qk_rows_store_kernel(const QkRowsArgs a) {
   __syncthreads();
   sq = sk = 0.f;
 #pragma unroll
-  for (int i = 0; i < kQkThreads / 32; ++i) { sq += red[0][i]; sk += red[1][i]; }
+  for (int i = 0; i < NT / 32; ++i) { sq += red[0][i]; sk += red[1][i]; }
   const float iq = a.q_scale / sqrtf(sq / (float)(a.hq * a.dk) + a.eps), ik = 1.0f / sqrtf(sk / (float)(a.hkv * a.dk) + a.eps);
   auto put = [&](int x, float* v) {
     TC* dst;
@@ -91,8 +90,8 @@ qk_rows_store_kernel(const QkRowsArgs a) {
     store_cols<V>(dst, v);
   };
 #pragma unroll
-  for (int i = 0; i < kQkKeep; ++i) { const int x = tid + i * kQkThreads; if (x < n) put(x, keep[i]); }
-  for (int x = tid + kQkKeep * kQkThreads; x < n; x += kQkThreads) {
+  for (int i = 0; i < KEEP; ++i) { const int x = tid + i * NT; if (x < n) put(x, keep[i]); }
+  for (int x = tid + KEEP * NT; x < n; x += NT) {
     float v[V];
     load_sum<TI, V>(row + (size_t)x * V, a.n_part, a.part_stride, v);
     put(x, v);
@@ -100,22 +99,24 @@ qk_rows_store_kernel(const QkRowsArgs a) {
   // padding of the heads
   if (a.dkp > a.dk) {
     const int pad = a.dkp - a.dk;
-    for (int x = tid; x < (a.hq + (store ? a.hkv : 0)) * pad; x += kQkThreads) {
+    for (int x = tid; x < (a.hq + (store ? a.hkv : 0)) * pad; x += NT) {
       const int h = x / pad, c = a.dk + x % pad;
       stv(h < a.hq ? (TC*)a.q_out + ((size_t)t * a.hq + h) * a.dkp + c : (TC*)a.k_cache + ((size_t)slot * a.hkv + h - a.hq) * a.dkp + c, 0.f);
     }
   }
   if (store && a.dvp > a.dv) {
     const int pad = a.dvp - a.dv;
-    for (int x = tid; x < a.hkv * pad; x += kQkThreads) stv((TC*)a.v_cache + ((size_t)slot * a.hkv + x / pad) * a.dvp + a.dv + x % pad, 0.f);
+    for (int x = tid; x < a.hkv * pad; x += NT) stv((TC*)a.v_cache + ((size_t)slot * a.hkv + x / pad) * a.dvp + a.dv + x % pad, 0.f);
   }
 }
 
 template <typename TI, typename TC>
 static int qk_rows_launch(const QkRowsArgs& a, int tokens, cudaStream_t stream) {
   const bool vec = a.dk % 4 == 0 && a.dv % 4 == 0 && a.dkp % 4 == 0 && a.dvp % 4 == 0 && a.ld % 4 == 0 && a.part_stride % 4 == 0 && (uintptr_t)a.qkv % (4 * sizeof(TI)) == 0;
-  if (vec) launch_k(qk_rows_store_kernel<TI, TC, 4>, (unsigned)tokens, kQkThreads, 0, stream, a);
-  else launch_k(qk_rows_store_kernel<TI, TC, 1>, (unsigned)tokens, kQkThreads, 0, stream, a);
+  // few tokens: more threads per token; many: more loads in flight per thread
+  if (vec && tokens <= 64) launch_k(qk_rows_store_kernel<TI, TC, 4, 512, 4>, (unsigned)tokens, 512, 0, stream, a);
+  else if (vec) launch_k(qk_rows_store_kernel<TI, TC, 4, 256, 8>, (unsigned)tokens, 256, 0, stream, a);
+  else launch_k(qk_rows_store_kernel<TI, TC, 1, 256, 8>, (unsigned)tokens, 256, 0, stream, a);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
