@@ -122,7 +122,7 @@ struct RecurrentArgs {
   float* out; int ld_out;       // [tokens, heads * vdim]
   int heads, groups, dim, vdim;
   int q_raw;                    // gla: != 0: q has no SiLU yet
-  // rwkv: != 0: gate holds the middle of a low-rank projection, [g_part][tokens, g_ld] with `rank` columns, before its tanh; its second matrix
+  // kRwkvLow: gate holds the middle of a low-rank projection, [g_part][tokens, g_ld] with `rank` columns, before its tanh; its second matrix
   int rank; const __nv_bfloat16* w2;    // is w2 [heads * dim, rank]
 };
 
@@ -142,14 +142,14 @@ __device__ __forceinline__ float gate_col(const RecurrentArgs& a, size_t tok, in
   return s;
 }
 
-enum RecurrentKind { kSsd = 0, kGla = 1, kRwkv = 2 };
+enum RecurrentKind { kSsd = 0, kGla = 1, kRwkv = 2, kRwkvLow = 3 };       // kRwkvLow: forms the decays from the middle of their low-rank projection
 
 template <typename TI, int KIND, int VEC, int R>   // dim <= 8 * R
 __global__ void __launch_bounds__(256)
 recurrent_step_kernel(const RecurrentArgs a) {
-  constexpr bool GLA = KIND == kGla, RWKV = KIND == kRwkv, CHAN = GLA || RWKV;       // CHAN: a decay per key channel
+  constexpr bool GLA = KIND == kGla, RWKV = KIND >= kRwkv, LOW = KIND == kRwkvLow, CHAN = GLA || RWKV;       // CHAN: a decay per key channel
   __shared__ float sq[8 * R], sk[8 * R], sf[CHAN ? 8 * R : 1], su[RWKV ? 8 * R : 1];
-  __shared__ float s_low[RWKV ? kMaxRank : 1];
+  __shared__ float s_low[LOW ? kMaxRank : 1];
   __shared__ float red[8][32 * VEC];
   __shared__ float s_dec;
   pdl_wait();
@@ -179,33 +179,31 @@ recurrent_step_kernel(const RecurrentArgs a) {
       dt = softplus_exact(gate_col(a, t, h) + bias_h);
       if (threadIdx.x == 0) s_dec = expf(a_h * dt);
     }
-    if constexpr (RWKV) {
-      if (a.rank > 0) {
-        for (int i = threadIdx.x; i < a.rank; i += 256) s_low[i] = tanhf(gate_col(a, t, i));
-        __syncthreads();
-        for (int c0 = 0; c0 < a.dim; c0 += 128) {             // two threads per channel
-          const int c = c0 + (threadIdx.x >> 1);
-          float z = 0.f;
-          if (c < a.dim) {
-            const __nv_bfloat16* w = a.w2 + (size_t)(h * a.dim + c) * a.rank;
-            if (a.rank % 16 == 0) {
-              for (int x = (threadIdx.x & 1) * 8; x < a.rank; x += 16) {
-                const uint4 q = *reinterpret_cast<const uint4*>(w + x);
-                const uint32_t u[4] = {q.x, q.y, q.z, q.w};
+    if constexpr (LOW) {
+      for (int i = threadIdx.x; i < a.rank; i += 256) s_low[i] = tanhf(gate_col(a, t, i));
+      __syncthreads();
+      for (int c0 = 0; c0 < a.dim; c0 += 128) {             // two threads per channel
+        const int c = c0 + (threadIdx.x >> 1);
+        float z = 0.f;
+        if (c < a.dim) {
+          const __nv_bfloat16* w = a.w2 + (size_t)(h * a.dim + c) * a.rank;
+          if (a.rank % 16 == 0) {
+            for (int x = (threadIdx.x & 1) * 8; x < a.rank; x += 16) {
+              const uint4 q = *reinterpret_cast<const uint4*>(w + x);
+              const uint32_t u[4] = {q.x, q.y, q.z, q.w};
 #pragma unroll
-                for (int y = 0; y < 4; ++y) {
-                  const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u[y]));
-                  z = fmaf(f.x, s_low[x + 2 * y], z);
-                  z = fmaf(f.y, s_low[x + 2 * y + 1], z);
-                }
+              for (int y = 0; y < 4; ++y) {
+                const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u[y]));
+                z = fmaf(f.x, s_low[x + 2 * y], z);
+                z = fmaf(f.y, s_low[x + 2 * y + 1], z);
               }
-            } else {
-              for (int x = threadIdx.x & 1; x < a.rank; x += 2) z = fmaf(__bfloat162float(w[x]), s_low[x], z);
             }
+          } else {
+            for (int x = threadIdx.x & 1; x < a.rank; x += 2) z = fmaf(__bfloat162float(w[x]), s_low[x], z);
           }
-          z += __shfl_xor_sync(0xffffffffu, z, 1);
-          if (c < a.dim && (threadIdx.x & 1) == 0) sf[c] = expf(-expf(z + a.gate_bias[h * a.dim + c]));
         }
+        z += __shfl_xor_sync(0xffffffffu, z, 1);
+        if (c < a.dim && (threadIdx.x & 1) == 0) sf[c] = expf(-expf(z + a.gate_bias[h * a.dim + c]));
       }
     }
     for (int i = threadIdx.x; i < 2 * a.dim; i += 256) {
@@ -224,7 +222,7 @@ recurrent_step_kernel(const RecurrentArgs a) {
           const float k = in_col<TI>(a, t, k_col + c);
           sk[c] = k;
           su[c] = k * a.par[h * a.dim + c];
-          if (a.rank == 0) sf[c] = expf(-expf(gate_col(a, t, h * a.dim + c) + a.gate_bias[h * a.dim + c]));
+          if constexpr (!LOW) sf[c] = expf(-expf(gate_col(a, t, h * a.dim + c) + a.gate_bias[h * a.dim + c]));
         } else sq[c] = in_col<TI>(a, t, q_col + c);
       } else {
         if (isk) sk[c] = in_col<TI>(a, t, k_col + c) * dt; else sq[c] = in_col<TI>(a, t, q_col + c);
@@ -442,6 +440,7 @@ GB_API int gb_rwkv_step(const void* rkv, int in_f32, long block_stride, int ld, 
   memset(&a, 0, sizeof(a));
   a.in = rkv; a.n_part = 1; a.part_stride = block_stride; a.ld = ld; a.gate = z; a.g_part = z_part; a.g_stride = z_stride; a.g_ld = z_ld; a.gate_bias = w0; a.par = u;
   a.state = state; a.n_slots = n_slots; a.cu_q = cu_q; a.seq_slots = seq_slots; a.out = out; a.ld_out = ld_out; a.heads = heads; a.groups = 1; a.dim = dim; a.vdim = vdim; a.rank = rank; a.w2 = (const __nv_bfloat16*)w2;
+  if (rank > 0) return in_f32 ? recurrent_step_launch<float, kRwkvLow>(a, n_seqs, stream) : recurrent_step_launch<__nv_bfloat16, kRwkvLow>(a, n_seqs, stream);
   return in_f32 ? recurrent_step_launch<float, kRwkv>(a, n_seqs, stream) : recurrent_step_launch<__nv_bfloat16, kRwkv>(a, n_seqs, stream);
 }
 

@@ -574,7 +574,7 @@ class Transformer:
         else:
             # decode-sized batches keep the projections in f32
             rkvg = torch.empty(4, pad, ld, dtype=torch.float32 if t <= 64 else torch.bfloat16, device=h.device)
-            gemm.grouped_linear(mix[:4].view(4 * pad, -1), w.w_in.w.view(4, w.w_in.rows_per_group, -1), seg, cnt, 256 if pad >= 512 else min(pad, 128), out=rkvg.view(4 * pad, ld),
+            gemm.grouped_linear(mix[:4].view(4 * pad, -1), w.w_in.w.view(4, w.w_in.rows_per_group, -1), seg, cnt, recurrent.shift_tile(pad), out=rkvg.view(4 * pad, ld),
                                 n_out=n, w_tiled=w.w_in.tiled)
         z, w2 = apply_linear_stream(w.w1, mix[4, :t]), None
         if w.w2_rows is not None and recurrent.can_fuse_decay(t, most, sp.decay_rank):

@@ -175,6 +175,11 @@ def shift_pad(t: int) -> int:
     return (t + tn - 1) // tn * tn
 
 
+def shift_tile(pad: int) -> int:
+    """Token tile of that product."""
+    return 256 if pad >= 512 else min(pad, 128)
+
+
 def token_shift(h: torch.Tensor, width: int, mu: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, seq_slots: torch.Tensor, pad: int, max_tokens: int) -> torch.Tensor:
     """Rows ``h [T, ld]`` -> ``[n, pad, ld]``: mix i of token t is ``h + (h' - h) * mu[i]`` with the row h' in front of it (``mu`` f32 ``[n, width]``).  The row in front
     of a sequence's first token comes from ``state`` f32 ``[slots, 1, width]``, its last one goes there.  Rows behind T are undefined."""

@@ -592,7 +592,7 @@ def case_fidolix(args):
         seg, cnt = torch.arange(4, dtype=torch.int32, device=dev) * pad, torch.full((4,), t, dtype=torch.int32, device=dev)
         mix = torch.randn(4 * pad, h, device=dev).bfloat16()
         wt = mxfp8.tile_weight(wg.view(4 * n, h)).view(4, n, h)
-        _run(f"grouped_rkvg_{name}", lambda: gemm.grouped_linear(mix, wt, seg, cnt, min(pad, 128), out=rkvg.view(4 * pad, n), w_tiled=True), 8.0 * t * n * h,
+        _run(f"grouped_rkvg_{name}", lambda: gemm.grouped_linear(mix, wt, seg, cnt, recurrent.shift_tile(pad), out=rkvg.view(4 * pad, n), w_tiled=True), 8.0 * t * n * h,
              4 * n * h * 2 + 4 * t * h * 2 + 4 * t * n * es, args)
         _run(f"gemm_same_size_{name}", lambda: gemm.linear(x, wt.view(4 * n, h), w_tiled=True, out_dtype=dt), 8.0 * t * n * h, 4 * n * h * 2 + t * h * 2 + 4 * t * n * es, args)
         del rkvg, mix, o, z
