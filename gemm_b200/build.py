@@ -89,7 +89,7 @@ SHARED_HEADER = CSRC / "kernels" / "geometry.cuh"      # inline code the host li
 # name -> (CUDA sources, extra nvcc flags, host sources)
 SUBSETS = {
     "layered": (["runtime", "elementwise", "gemm_tc", "gemm_f32", "flash_attn", "attn_any", "stream_ops", "qkv_store", "lightning", "lightning_chunk", "sampler",
-                 "recurrent", "gla_chunk", "latent", "latent_attn", "moe", "moe_prep"],
+                 "recurrent", "gla_chunk", "mingru", "latent", "latent_attn", "moe", "moe_prep"],
                 ["-DGB_GEMM_BF16_ONLY"], ["common", "runtime", "safetensors"]),
 }
 

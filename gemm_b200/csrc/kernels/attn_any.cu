@@ -1,7 +1,7 @@
 // Paged attention for any head sizes and element types, one warp per (token, query head): the path of the "f32" weight format and
 // of head sizes the tcgen05 kernels (flash_attn.cu) are not built for.  Keys and values may differ in size.  A query at position i
 // sees j <= i with i - j < window (0 = no limit) or j < keep_first; an optional table adds bias[h][min(i - j, n_bias - 1)] to the
-// score, a cap c > 0 makes it c tanh(score / c) (q then arrives multiplied by scale / c), and a learned score per head (a sink) may join the sum of the weights.  Q arrives multiplied by scale * log2(e), bias table and sinks by log2(e);
+// score, or r1[h] ln(1 + r2[h] (i - j)) is taken off it, a cap c > 0 makes it c tanh(score / c) (q then arrives multiplied by scale / c), and a learned score per head (a sink) may join the sum of the weights.  Q arrives multiplied by scale * log2(e), bias table and sinks by log2(e);
 // scores, weights and sums are f32.  Latent attention runs here as one key / value head whose values are the first columns of the keys.
 #include "sm100.cuh"
 #include "host_common.h"
@@ -18,6 +18,7 @@ struct AttnAnyArgs {
   int tokens, hq, hkv, dk, dv, window, keep_first;
   const float* bias; int n_bias, ld_bias;
   float cap;                                                   // softcap * log2(e); 0 = none
+  const float* log_bias;                                       // [2][hq]: r1, r2; null = none
 };
 
 __device__ __forceinline__ float lda(const float* p) { return *p; }
@@ -52,6 +53,7 @@ attn_any_kernel(const AttnAnyArgs a) {
   const int n_keep = min(a.keep_first, first);
   const int n = n_keep + (i - first + 1);           // visible keys: [0, n_keep) and [first, i]
   const int* bt = a.block_table + (size_t)seq * a.max_pages;
+  const float r1 = a.log_bias != nullptr ? a.log_bias[h] : 0.f, r2 = a.log_bias != nullptr ? a.log_bias[a.hq + h] : 0.f;
   float m = -INFINITY, l = 0.f, acc[NV];
 #pragma unroll
   for (int c = 0; c < NV; ++c) acc[c] = 0.f;
@@ -69,6 +71,7 @@ attn_any_kernel(const AttnAnyArgs a) {
       for (int c = 0; c < a.dk; ++c) s = fmaf(q[c], lda(kr + c), s);
       if (a.cap > 0.f) s = a.cap * tanhf(s);
       if (a.bias != nullptr) s += a.bias[(size_t)h * a.ld_bias + min(i - j, a.n_bias - 1)];
+      if (a.log_bias != nullptr) s = fmaf(-r1, log2f(fmaf(r2, (float)(i - j), 1.0f)), s);
       sc = s;
     }
     const float mn = fmaxf(m, warp_max(sc));
@@ -117,7 +120,7 @@ using namespace gb;
 
 GB_API int gb_attn_any(const void* q, const void* k, const void* v, void* out, int f32, const int* cu_q, const int* kv_len, const int* block_table,
                        int max_pages, int page_size, int n_seqs, long num_slots, int tokens, int hq, int hkv, int dk, int dv, int window, int keep_first,
-                       const float* bias, int n_bias, int ld_bias, float softcap, const float* sink, cudaStream_t stream) {
+                       const float* bias, int n_bias, int ld_bias, float softcap, const float* sink, const float* log_bias, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (hq < 1 || hkv < 1 || hq % hkv || dk < 1 || dv < 1 || n_seqs < 1 || page_size < 1) return fail("attn_any: bad sizes%s");
   if (dk > 2048 || dv > 1024) return fail("attn_any: keys of at most 2048 and values of at most 1024 features%s");
@@ -128,6 +131,7 @@ GB_API int gb_attn_any(const void* q, const void* k, const void* v, void* out, i
   a.bias = bias; a.n_bias = n_bias; a.ld_bias = ld_bias;
   a.q_hs = dk; a.q_ts = (long)hq * dk; a.k_hs = dk; a.k_ss = (long)hkv * dk; a.v_hs = dv; a.v_ss = (long)hkv * dv; a.o_hs = dv; a.o_ts = (long)hq * dv;
   a.tok_seq = nullptr; a.tok_kv = nullptr; a.sink = sink; a.cap = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+  a.log_bias = log_bias;
   return f32 ? attn_any_launch<float>(a, stream) : attn_any_launch<__nv_bfloat16>(a, stream);
 }
 

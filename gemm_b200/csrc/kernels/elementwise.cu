@@ -497,7 +497,7 @@ silu_mul_quant_kernel(const __nv_bfloat16* __restrict__ gate_up, const int* __re
 // split order; the result goes out as bf16 and / or as MXFP8 with scale atoms.  8 elements per thread, 4 threads share a scale.
 __global__ void __launch_bounds__(256)
 silu_mul_partials_kernel(const float* __restrict__ part, int n_part, long part_stride, __nv_bfloat16* __restrict__ out, uint8_t* __restrict__ out_q,
-                         uint8_t* __restrict__ out_sf, long rows, int inter, int sf32, int act, float cap) {
+                         uint8_t* __restrict__ out_sf, long rows, int inter, int sf32, int act, float cap, const float* __restrict__ bias) {
   pdl_wait();
   pdl_trigger();
   const long idx = (long)blockIdx.x * blockDim.x + threadIdx.x;
@@ -510,7 +510,7 @@ silu_mul_partials_kernel(const float* __restrict__ part, int n_part, long part_s
   if (live) {
     float g[8], u[8];
 #pragma unroll
-    for (int j = 0; j < 8; ++j) { g[j] = 0.f; u[j] = 0.f; }
+    for (int j = 0; j < 8; ++j) { g[j] = bias != nullptr ? bias[vi * 8 + j] : 0.f; u[j] = bias != nullptr ? bias[inter + vi * 8 + j] : 0.f; }
     const float* pp = part + r * (2L * inter) + vi * 8;
     for (int p = 0; p < n_part; ++p, pp += part_stride) {
       const float4 g0 = *reinterpret_cast<const float4*>(pp), g1 = *reinterpret_cast<const float4*>(pp + 4);
@@ -958,13 +958,13 @@ GB_API int gb_silu_mul_quant(const void* gate_up, const int* row_valid, void* ou
 }
 
 GB_API int gb_silu_mul_partials(const float* part, int n_part, long part_stride, void* out, void* out_q, void* out_sf, long rows, int inter,
-                                int sf32, int act, float cap, cudaStream_t stream) {
+                                int sf32, int act, float cap, const float* bias, cudaStream_t stream) {
   if (inter % 8 || (out_q != nullptr && inter % 128)) return fail("silu_mul_partials: inter must be a multiple of 8 (128 with MXFP8 output)%s");
   if (part_stride % 4 != 0 || ((uintptr_t)part & 15) != 0) return fail("silu_mul_partials: misaligned partials%s");
   const long n = rows * (inter / 8);
   if (n <= 0) return 0;
   launch_k(silu_mul_partials_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, part, n_part, part_stride, (__nv_bfloat16*)out, (uint8_t*)out_q,
-           (uint8_t*)out_sf, rows, inter, sf32, act, cap);
+           (uint8_t*)out_sf, rows, inter, sf32, act, cap, bias);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }

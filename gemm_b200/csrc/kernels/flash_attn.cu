@@ -57,6 +57,7 @@ struct FaArgs {
   // forms 2 and 3
   const float* sink;        // [hq] a score per head, times log2 e, that joins the sum of the weights; null = none
   float cap;                // form 3: scores are cap * tanh(q . k), cap = softcap * log2 e (q carries scale / softcap)
+  const float* log_bias;    // form 4: [2][hq]: r1[h] log2(1 + r2[h] * distance) is taken off the scores
 };
 
 // KV blocks of a query tile or decode token, in order: with a window and kept first positions, the blocks of the kept positions that lie
@@ -77,12 +78,21 @@ __device__ __forceinline__ FaBlocks fa_blocks(const FaArgs& a, int first_pos, in
 constexpr int kFaSmem = 32768 * 3 + 256 + 1024;
 
 // DK / DV: width of a key / value head in the cache (64 or 128 columns).  FORM: 0 = plain, 1 = kept first positions and a distance bias, 2 = sinks,
-// 3 = capped scores (and sinks).
+// 3 = capped scores (and sinks), 4 = as 1 with a logarithmic distance bias that is formed here.
+__device__ __forceinline__ float log_dist(float r1, float r2, int dist) { return -r1 * __log2f(fmaf(r2, (float)max(dist, 0), 1.0f)); }
+
+// Columns of a head's window of biases in shared memory: 127 + tokens per tile, padded so that the rows of a warp (32 / G tokens of G heads) lie in
+// different banks when G is a power of two.
+__host__ __device__ inline int bias_width(int g) {
+  const int n = 127 + 128 / g, want = g <= 32 && (g & (g - 1)) == 0 ? 32 / g % 32 : n % 32;
+  return n + (want - n % 32 + 32) % 32;
+}
+
 template <int DK, int DV, int FORM>
 __global__ void __launch_bounds__(kFaThreads, 2)
 flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                   const __grid_constant__ CUtensorMap tmV, const FaArgs a) {
-  constexpr bool EXT = FORM == 1, SINK = FORM >= 2, CAP = FORM == 3;
+  constexpr bool LOGB = FORM == 4, EXT = FORM == 1 || LOGB, SINK = FORM == 2 || FORM == 3, CAP = FORM == 3;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);      // an offset, so that accesses stay shared-memory ones
   uint8_t* sQ = smem;                       // 2 x [128 rows x 128 B]  (d halves)
@@ -233,18 +243,26 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
     bool ok = true;
     const float* bias_row = EXT && a.bias != nullptr ? a.bias + (size_t)(bad_item ? 0 : kvh * G) * a.ld_bias : nullptr;   // the group's first head
     float* s_bias = reinterpret_cast<float*>(smem + 32768 * 3 + 256);      // EXT: two windows of G x bias_w scores, by block parity
-    const int bias_w = 127 + tpt;
+    const int bias_w = bias_width(G);
+    float lb1 = 0.f, lb2 = 0.f;                            // LOGB: the row's head's numbers
+    const float* lb = LOGB ? a.log_bias + (bad_item ? 0 : kvh * G) : nullptr;
+    if constexpr (LOGB) { lb1 = lb[min(h_local, G - 1)]; lb2 = lb[a.hq + min(h_local, G - 1)]; }
     for (int j = 0; j < n_blk && ok; ++j) {
       const int kv0 = blocks.at(blk_lo + j) * kBN;
       // distance of the tile's first token to the block's last key: a row's distances are dmin + t_local + 127 - (column)
       const int dmin = pos0 - kv0 - (kBN - 1);
-      const bool near = EXT && bias_row != nullptr && dmin < a.n_bias - 1;       // else one score for the whole block
+      const bool near = LOGB || (EXT && bias_row != nullptr && dmin < a.n_bias - 1);       // else one score for the whole block
       float* win = s_bias + (size_t)(j & 1) * G * bias_w;
       bool got = true;
-      if constexpr (EXT) {
+      if constexpr (LOGB) {
+        for (int h = 0; h < G; ++h) {
+          const float r1 = lb[h], r2 = lb[a.hq + h];
+          for (int x = q * 32 + lane; x < 127 + tpt; x += 128) win[h * bias_w + x] = log_dist(r1, r2, dmin + x);
+        }
+      } else if constexpr (EXT) {
         if (near)
           for (int h = 0; h < G; ++h)
-            for (int x = q * 32 + lane; x < bias_w; x += 128)
+            for (int x = q * 32 + lane; x < 127 + tpt; x += 128)
               win[h * bias_w + x] = bias_row[(size_t)h * a.ld_bias + max(0, min(dmin + x, a.n_bias - 1))];
       }
       got = mbar_wait(s_full, j & 1, abort_flag, a.status, 600, j);
@@ -277,7 +295,10 @@ flash_attn_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant
       }
       // with a bias the reference is an upper bound: the largest raw score plus the largest bias of the row's 128 distances
       float bfar = 0.f;
-      if constexpr (EXT) {
+      if constexpr (LOGB) {
+        // monotone in the distance: the larger of the two ends of the row's 128
+        mx += fmaxf(log_dist(lb1, lb2, qpos - kv0 - (kBN - 1)), log_dist(lb1, lb2, qpos - kv0));
+      } else if constexpr (EXT) {
         if (bias_row != nullptr) {
           const float* br = bias_row + (size_t)h_local * a.ld_bias + max(0, min(qpos - kv0 - (kBN - 1), a.n_bias - 1));
           bfar = *br;
@@ -446,7 +467,7 @@ template <int DK, int DV, int FORM>                 // FORM as in flash_attn_ker
 __global__ void __launch_bounds__(kFdThreads, 2)
 flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmV, const FaArgs a) {
-  constexpr bool EXT = FORM == 1, SINK = FORM >= 2, CAP = FORM == 3;
+  constexpr bool LOGB = FORM == 4, EXT = FORM == 1 || LOGB, SINK = FORM == 2 || FORM == 3, CAP = FORM == 3;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = smem_raw + ((1024u - (smem_u32(smem_raw) & 1023u)) & 1023u);      // an offset, so that accesses stay shared-memory ones
   uint8_t* sQ = smem;                          // 2 d-halves x [16 heads x 128 B]
@@ -596,7 +617,10 @@ flash_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const int s = j & 1;
       const int kp = blocks.at(blk_lo + j) * kBN + r;
       float bv[kFdN];                                    // the position's distance bias, requested before the wait for the scores
-      if constexpr (EXT) {
+      if constexpr (LOGB) {
+#pragma unroll
+        for (int h = 0; h < kFdN; ++h) bv[h] = h < G && !bad_item ? log_dist(a.log_bias[kvh * G + h], a.log_bias[a.hq + kvh * G + h], qpos - kp) : 0.f;
+      } else if constexpr (EXT) {
         if (a.bias != nullptr && !bad_item) {
           const float* br = a.bias + (size_t)kvh * G * a.ld_bias + max(0, min(qpos - kp, a.n_bias - 1));
 #pragma unroll
@@ -959,7 +983,7 @@ static int flash_masked_launch(const void* q, const void* k_cache, const void* v
     }
     launch_k(flash_decode_kernel<DK, DV, FORM>, n_work, kFdThreads, kFdSmem, stream, tmQ, tmK, tmV, a);
   } else {
-    const int smem = kFaSmem + (a.bias != nullptr ? 2 * G * (127 + tpt) * 4 : 0);
+    const int smem = kFaSmem + (a.bias != nullptr || FORM == 4 ? 2 * G * bias_width(G) * 4 : 0);
     static int attr_max = 0;
     if (smem > 227 * 1024) return fail("flash_masked: the bias windows of this group size do not fit shared memory%s");
     if (smem > attr_max) {
@@ -973,18 +997,19 @@ static int flash_masked_launch(const void* q, const void* k_cache, const void* v
 }
 
 // gb_flash_attn / gb_flash_decode (decode != 0: one query token per sequence, Hq / Hkv <= 16) with keys of dk and values of dv columns (64 or
-// 128 each), a window that keeps the first `keep_first` positions, and a distance bias, or with capped scores (softcap > 0) and sinks (see FaArgs).  q is
+// 128 each), a window that keeps the first `keep_first` positions, and a distance bias (a table, or logarithmic), or with capped scores (softcap > 0) and sinks (see FaArgs).  q is
 // [T, Hq, dk], out [T, Hq, dv].
 GB_API int gb_flash_masked(const void* q, const void* k_cache, const void* v_cache, void* out, float* part_o, float* part_lse, const int* work, int n_work,
                            const int* cu_q, const int* kv_len, const int* block_table, int max_pages, int page_size, long num_slots, int total_tokens,
                            int hq, int hkv, int dk, int dv, int num_splits, int window, int keep_first, const float* bias, int n_bias, int ld_bias,
-                           float softcap, const float* sink, int decode, void* status, cudaStream_t stream) {
+                           float softcap, const float* sink, const float* log_bias, int decode, void* status, cudaStream_t stream) {
   if ((dk != 64 && dk != 128) || (dv != 64 && dv != 128)) return fail("flash_masked: heads of 64 or 128 columns%s");
   if (hq < 1 || hkv < 1 || hq % hkv || hq / hkv > (decode ? kFdN : 128)) return fail("flash_masked: bad head counts%s");
   if (page_size < 8 || page_size > 128 || (128 % page_size) || (page_size % 8)) return fail("flash_masked: page_size must be 8..128, a multiple of 8 dividing 128%s");
   if (bias != nullptr && (n_bias < 1 || ld_bias < 2 * n_bias)) return fail("flash_masked: bad bias table%s");
-  const int form = softcap > 0.f ? 3 : sink != nullptr ? 2 : 1;
-  if (form > 1 && (bias != nullptr || keep_first > 0)) return fail("flash_masked: capped scores and sinks do not go with a bias or kept positions%s");
+  const int form = softcap > 0.f ? 3 : sink != nullptr ? 2 : log_bias != nullptr ? 4 : 1;
+  if (log_bias != nullptr && (form != 4 || bias != nullptr)) return fail("flash_masked: a logarithmic distance bias does not go with another bias, capped scores or sinks%s");
+  if ((form == 2 || form == 3) && (bias != nullptr || keep_first > 0)) return fail("flash_masked: capped scores and sinks do not go with a bias or kept positions%s");
   if (window < 0 || keep_first < 0 || num_splits < 1) return fail("flash_masked: bad mask%s");
   if (n_work <= 0) return 0;
   if (num_splits > 1 && (part_o == nullptr || part_lse == nullptr)) return fail("flash_masked: num_splits > 1 needs partial buffers%s");
@@ -995,7 +1020,7 @@ GB_API int gb_flash_masked(const void* q, const void* k_cache, const void* v_cac
   a.hq = hq; a.hkv = hkv; a.num_splits = num_splits; a.causal = 1; a.window = window; a.keep_first = window > 0 ? keep_first : 0; a.out = (__nv_bfloat16*)out;
   a.part_o = part_o; a.part_lse = part_lse; a.total_tokens = total_tokens; a.status = (KernelStatus*)status;
   a.bias = bias; a.n_bias = n_bias; a.ld_bias = ld_bias;
-  a.sink = sink; a.cap = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
+  a.log_bias = log_bias; a.sink = sink; a.cap = softcap > 0.f ? softcap * 1.4426950408889634f : 0.f;
 #define GB_FORM(F)                                                                                                                                    \
   if (form == F) {                                                                                                                                    \
     if (dk == 64) return dv == 64 ? flash_masked_launch<64, 64, F>(q, k_cache, v_cache, a, n_work, num_slots, decode, stream)                         \
@@ -1006,6 +1031,7 @@ GB_API int gb_flash_masked(const void* q, const void* k_cache, const void* v_cac
   GB_FORM(1)
   GB_FORM(2)
   GB_FORM(3)
+  GB_FORM(4)
 #undef GB_FORM
   return fail("flash_masked: unknown form%s");
 }

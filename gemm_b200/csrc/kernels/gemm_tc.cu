@@ -45,7 +45,7 @@ struct GemmArgs {
   int ldo;
   int out_f32;
   uint8_t* out_sf;      // quantising epilogue: scale atoms [x_row/128][n/128]
-  const float* bias;    // optional [n_out] (plain, per group not supported)
+  const float* bias;    // optional [n_out] (per group not supported); DUAL with ACT = 3: [up_row_offset + n_out]
   const int* row_map;   // optional: output row of X row r (negative = drop)
   const float* row_scale; // optional: multiply row r of the result
   int stages;
@@ -156,7 +156,10 @@ __device__ __forceinline__ int e8m0_from_amax(float amax) {
   return amax == 0.0f ? 127 : max(1, min(e, 254));   // an all-zero block gets scale 1
 }
 
-// ACT, DUAL: the gate's activation (gated); plain: 1 = SiLU on the output features below args.silu_rows, 2 = bf16 rows scattered by args.row_map.
+__device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f)); }
+
+// ACT, DUAL: the gate's activation (gated), 3 = the tanh form of GELU with a bias on either product; plain: 1 = SiLU on the output features below args.silu_rows, 2 = bf16
+// rows scattered by args.row_map, 3 = the exact GELU on every feature.
 template <int TN, int MODE, bool DUAL, bool QUANT_OUT, int ACT = 0>
 __global__ void __launch_bounds__(kGemmThreads, 1)
 gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmX, const GemmArgs args) {
@@ -413,15 +416,22 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
       const bool n_ok = n < args.n_out;
       const bool row_act = !DUAL && ACT == 1 && n < args.silu_rows;
       const float bias = (args.bias != nullptr && n_ok && (args.partial_stride == 0 || t.ks == 0)) ? args.bias[n] : 0.0f;
+      const float bias_up = (DUAL && ACT == 3 && n_ok) ? args.bias[args.up_row_offset + n] : 0.0f;
+      auto value = [&](uint32_t r0, uint32_t r1) {         // bias and activation of one result (or of a gate / up pair)
+        float v = __uint_as_float(r0);
+        if constexpr (DUAL && ACT == 3) return gated<ACT>(v + bias, __uint_as_float(r1) + bias_up, args.act_cap);
+        if (DUAL) v = gated<ACT>(v, __uint_as_float(r1), args.act_cap);
+        v += bias;
+        if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
+        if (!DUAL && ACT == 3) v = gelu_erf(v);
+        return v;
+      };
       // Everything after the accumulators are in registers: activation, bias, then one of the store forms.
       auto finish_chunk = [&](int c, const uint32_t* r0, const uint32_t* r1) {
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
           const int xr = c + j;
-          float v = __uint_as_float(r0[j]);
-          if (DUAL) v = gated<ACT>(v, __uint_as_float(r1[j]), args.act_cap);
-          v += bias;
-          if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
+          float v = value(r0[j], r1[j]);
           const bool live = xr < t.valid;
           const int x_row = t.x_row0 + xr;
           if (QUANT_OUT) {
@@ -645,20 +655,14 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
           if (c + 16 <= t.valid) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
-              float v = __uint_as_float(r0[j]);
-              if (DUAL) v = gated<ACT>(v, __uint_as_float(r1[j]), args.act_cap);
-              v += bias;
-              if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
+              const float v = value(r0[j], r1[j]);
               if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
               else o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v);
             }
           } else {
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
-              float v = __uint_as_float(r0[j]);
-              if (DUAL) v = gated<ACT>(v, __uint_as_float(r1[j]), args.act_cap);
-              v += bias;
-              if (!DUAL && ACT == 1 && row_act) v = __fdividef(v, 1.0f + __expf(-v));
+              const float v = value(r0[j], r1[j]);
               if (c + j < t.valid) {
                 if (args.out_f32) o32[(size_t)(c + j) * args.ldo] = v;
                 else o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v);
@@ -777,7 +781,7 @@ struct GemmExtras {
 };
 
 // Flags of gb_gemm.
-enum { GEMM_MX = 1, GEMM_DUAL = 2, GEMM_QUANT_OUT = 4, GEMM_OUT_F32 = 8, GEMM_W_TILED = 16, GEMM_DUAL_RAW = 32, GEMM_GELU = 64, GEMM_CAPPED = 128 };
+enum { GEMM_MX = 1, GEMM_DUAL = 2, GEMM_QUANT_OUT = 4, GEMM_OUT_F32 = 8, GEMM_W_TILED = 16, GEMM_DUAL_RAW = 32, GEMM_GELU = 64, GEMM_CAPPED = 128, GEMM_GELU_ERF = 256 };
 
 // Linear layer on tensor cores.
 //   w        [w_rows, k] row-major (bf16, or e4m3 bytes when GEMM_MX), w_rows = groups * w_rows_per_group
@@ -835,6 +839,10 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
   const bool gelu = flags & GEMM_GELU;
   const bool capped = flags & GEMM_CAPPED;
   if ((gelu || capped) && (!dual || mx || qo || (gelu && capped))) return fail("gemm: GEMM_GELU / GEMM_CAPPED need a bf16 GEMM_DUAL launch%s");
+  const bool gelu_all = flags & GEMM_GELU_ERF;
+  if (gelu_all && (dual || mx || qo || (flags & GEMM_OUT_F32) || (ex != nullptr && (ex->splits > 1 || ex->silu_rows > 0)) || row_map != nullptr))
+    return fail("gemm: GEMM_GELU_ERF needs a plain bf16 launch%s");
+  if (dual && bias != nullptr && (!gelu || num_groups > 0 || (ex != nullptr && ex->splits > 1))) return fail("gemm: biases of a gate / up pair go with GEMM_GELU%s");
   if (capped && ex == nullptr) return fail("gemm: GEMM_CAPPED without a bound%s");
   if (a.dual_raw && (!dual || qo)) return fail("gemm: GEMM_DUAL_RAW needs GEMM_DUAL without GEMM_QUANT_OUT%s");
   a.out_sf = (uint8_t*)out_sf; a.bias = bias; a.row_map = row_map; a.row_scale = row_scale; a.status = (KernelStatus*)status;
@@ -879,6 +887,13 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
     if (tn == 128) return launch_gemm<128, 0, false, false, 1>(tmW, tmX, a, max_tiles, stream);
     if (tn == 256) return launch_gemm<256, 0, false, false, 1>(tmW, tmX, a, max_tiles, stream);
   }
+  if (gelu_all) {
+    if (tn == 16) return launch_gemm<16, 0, false, false, 3>(tmW, tmX, a, max_tiles, stream);
+    if (tn == 32) return launch_gemm<32, 0, false, false, 3>(tmW, tmX, a, max_tiles, stream);
+    if (tn == 64) return launch_gemm<64, 0, false, false, 3>(tmW, tmX, a, max_tiles, stream);
+    if (tn == 128) return launch_gemm<128, 0, false, false, 3>(tmW, tmX, a, max_tiles, stream);
+    if (tn == 256) return launch_gemm<256, 0, false, false, 3>(tmW, tmX, a, max_tiles, stream);
+  }
   if (row_map != nullptr && !mx && !dual && !qo && row_scale == nullptr && a.amax_val == nullptr && !a.out_f32 && a.splits <= 1 && a.peer_bcast == 0 && a.peer_region_rows == 0) {
     if (tn == 16) return launch_gemm<16, 0, false, false, 2>(tmW, tmX, a, max_tiles, stream);
     if (tn == 32) return launch_gemm<32, 0, false, false, 2>(tmW, tmX, a, max_tiles, stream);
@@ -890,6 +905,7 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
 #define GB_DISPATCH(TNV)                                                                                      \
   if (tn == TNV) {                                                                                            \
     if (!mx && !dual && !qo) return launch_gemm<TNV, 0, false, false>(tmW, tmX, a, max_tiles, stream);        \
+    if (gelu && bias != nullptr) return launch_gemm<TNV, 0, true, false, 3>(tmW, tmX, a, max_tiles, stream);  \
     if (gelu) return launch_gemm<TNV, 0, true, false, 1>(tmW, tmX, a, max_tiles, stream);                     \
     if (capped) return launch_gemm<TNV, 0, true, false, 2>(tmW, tmX, a, max_tiles, stream);                   \
     if (!mx && dual && !qo) return launch_gemm<TNV, 0, true, false>(tmW, tmX, a, max_tiles, stream);          \
@@ -898,6 +914,7 @@ GB_API int gb_gemm(const void* w, const void* x, void* out, int n_out, int k, in
 #define GB_DISPATCH(TNV)                                                                                      \
   if (tn == TNV) {                                                                                            \
     if (!mx && !dual && !qo) return launch_gemm<TNV, 0, false, false>(tmW, tmX, a, max_tiles, stream);        \
+    if (gelu && bias != nullptr) return launch_gemm<TNV, 0, true, false, 3>(tmW, tmX, a, max_tiles, stream);  \
     if (gelu) return launch_gemm<TNV, 0, true, false, 1>(tmW, tmX, a, max_tiles, stream);                     \
     if (capped) return launch_gemm<TNV, 0, true, false, 2>(tmW, tmX, a, max_tiles, stream);                   \
     if (!mx && dual && !qo) return launch_gemm<TNV, 0, true, false>(tmW, tmX, a, max_tiles, stream);          \

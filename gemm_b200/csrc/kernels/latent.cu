@@ -23,7 +23,7 @@ __device__ __forceinline__ void rotation(int pos, double freq, float mag, float&
 struct LatentStoreArgs {
   const void* a; int n_part; long part_stride; int ld;         // [n_part][tokens, ld]: q latent, kv latent, rotated key part
   const int* positions; const int* slots;
-  const float* q_norm; const float* kv_norm;                   // kv_norm null: only the q latent
+  const float* q_norm; const float* kv_norm;                   // kv_norm null: only the q latent; q_rank 0: none
   const double* freq; float mag;
   void* q_out; int ld_q;                                       // [tokens, ld_q], zero behind q_rank
   void* cache; long num_slots; int ld_c;                       // [slots, ld_c], zero behind rank + rot_dim
@@ -81,7 +81,7 @@ latent_store_kernel(const LatentStoreArgs a) {
   sq = sk = 0.f;
 #pragma unroll
   for (int i = 0; i < 8; ++i) { sq += red[0][i]; sk += red[1][i]; }
-  const float iq = 1.0f / sqrtf(sq / (float)a.q_rank + a.eps), ik = 1.0f / sqrtf(sk / (float)a.rank + a.eps);
+  const float iq = a.q_rank > 0 ? 1.0f / sqrtf(sq / (float)a.q_rank + a.eps) : 0.f, ik = 1.0f / sqrtf(sk / (float)a.rank + a.eps);
   TO* qo = (TO*)a.q_out + (size_t)t * a.ld_q;
 #pragma unroll
   for (int i = 0; i < N; ++i) {
@@ -179,7 +179,7 @@ GB_API int gb_latent_store(const void* rows, int in_f32, int n_part, long part_s
                            const float* kv_norm, const double* freq, float mag, void* q_out, int ld_q, void* cache, int out_f32, long num_slots, int ld_c, int tokens,
                            int q_rank, int rank, int rot_dim, float eps, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (q_rank < 1 || rank < 1 || rot_dim < 0 || rot_dim % 2 || n_part < 1 || ld_q < q_rank || (kv_norm != nullptr && ld_c < rank + rot_dim) ||
+  if (q_rank < 0 || (q_rank == 0 ? kv_norm == nullptr || ld_q != 0 : q_out == nullptr) || rank < 1 || rot_dim < 0 || rot_dim % 2 || n_part < 1 || ld_q < q_rank || (kv_norm != nullptr && ld_c < rank + rot_dim) ||
       ld < q_rank + (kv_norm != nullptr ? rank + rot_dim : 0)) return fail("latent_store: bad sizes%s");
   if (ld_q > 256 * kLatKeep || rank > 256 * kLatKeep) return fail("latent_store: ranks of at most 2048%s");
   LatentStoreArgs a;

@@ -6,12 +6,15 @@
 //                       may also be the router-weighted sum of expert outputs (formed here)
 //   stream_rms2         stream_norm for an update with an RMSNorm of its own, a row added per token, and a second set of normalised rows
 //   stream_join         stream += factor * result, for up to three pending results; a copy of the rows for a projection of the stream itself
+//   stream_depth        stream += results as in stream_join; the new stream is kept, and a weighted sum of it and of earlier kept ones goes on, RMSNormed
+//   depth_base          the part of later sums that is known already, for several of them in one pass
 //   qk_unit_store       fused Q | K | V rows -> Q / K divided by their root mean square per head (no weight), K / V into their
-//                       cache slots, Q scaled and laid out for the attention kernels
+//                       cache slots, Q scaled (by a function of the position, too) and laid out for the attention kernels
 //   gated_norm          RMSNorm over all heads' outputs together, times sigmoid(gate): the tail of a linear-attention mixer
 //   part_norm           RMSNorm of equal parts of a row, after (or before) SiLU(gate) if there is one: the tail of Mamba-2, HGRN2 and RWKV mixers
 //   sigmoid_gate        the heads' outputs of an attention, times sigmoid(gate)
 //   token_gate          GELU(z) times a row of a table, by token
+//   gelu_f32            the exact GELU of f32 values (the 32-bit path)
 //   act_mul             act(gate) * up of f32 rows (the 32-bit path; the bf16 path has it in the GEMM epilogue)
 // One pass over HBM each; sizes are arbitrary (vector paths when they divide).  Output rows may be wider than the data (padding to
 // the 16-byte row pitch the TMA descriptors of the next GEMM need); the padding is written as zero.
@@ -68,8 +71,10 @@ struct StreamNormArgs {
   const void* delta;            // pending update: f32 / bf16 [n_part][rows, ld_delta]; null = none
   int n_part; long part_stride; // K-split partial sums: slabs `part_stride` elements apart, added in order
   int ld_delta;
+  float factor;                 // of the update
   const float* add;             // vector added to every row after the update; null = none
   const float* weight;          // f32 [width]
+  const float* dot; float* gate;   // gate[r] = sigmoid(sum of x / rms(x) * dot) of output row r; null = none
   const long long* rows;        // output row r comes from stream row rows[r] (then the stream is not written); null = all rows in place
   void* out; int ld_out;        // normalised rows, ld_out >= width, the columns behind `width` are zeroed; null = only update the stream
   int width; float eps;
@@ -80,13 +85,13 @@ __global__ void __launch_bounds__(256)
 stream_norm_vec_kernel(const StreamNormArgs a) {
   pdl_wait();
   pdl_trigger();
-  __shared__ float red[8];
+  __shared__ float red[2][8];
   const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
   float* x = a.x + src * a.width;
   const TD* d = a.delta != nullptr ? (const TD*)a.delta + src * a.ld_delta : nullptr;
   const int nv = a.width >> 2;
   float4 v[VPT];
-  float ss = 0.f;
+  float ss = 0.f, sd = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = threadIdx.x + i * 256;
@@ -98,7 +103,7 @@ stream_norm_vec_kernel(const StreamNormArgs a) {
         const float4 q = ld4(d + (size_t)p * a.part_stride + c * 4);
         s.x += q.x; s.y += q.y; s.z += q.z; s.w += q.w;
       }
-      v[i].x += s.x; v[i].y += s.y; v[i].z += s.z; v[i].w += s.w;
+      v[i].x = fmaf(a.factor, s.x, v[i].x); v[i].y = fmaf(a.factor, s.y, v[i].y); v[i].z = fmaf(a.factor, s.z, v[i].z); v[i].w = fmaf(a.factor, s.w, v[i].w);
     }
     if (a.add != nullptr) {
       const float4 q = ld4(a.add + c * 4);
@@ -106,9 +111,17 @@ stream_norm_vec_kernel(const StreamNormArgs a) {
     }
     if (a.rows == nullptr && (d != nullptr || a.add != nullptr)) st4(x + c * 4, v[i]);
     ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+    if (a.dot != nullptr) {
+      const float4 q = ld4(a.dot + c * 4);
+      sd += v[i].x * q.x + v[i].y * q.y + v[i].z * q.z + v[i].w * q.w;
+    }
   }
   if (a.out == nullptr) return;
-  const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.width + a.eps);
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red[0]) / (float)a.width + a.eps);
+  if (a.dot != nullptr) {
+    const float g = block_sum_256(sd, red[1]) * inv;
+    if (threadIdx.x == 0) a.gate[r] = 1.0f / (1.0f + expf(-g));
+  }
   TO* o = (TO*)a.out + r * a.ld_out;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
@@ -125,7 +138,7 @@ __global__ void __launch_bounds__(256)
 stream_norm_any_kernel(const StreamNormArgs a) {
   pdl_wait();
   pdl_trigger();
-  __shared__ float red[8];
+  __shared__ float red[2][8];
   const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
   float* x = a.x + src * a.width;
   const TD* d = a.delta != nullptr ? (const TD*)a.delta + src * a.ld_delta : nullptr;
@@ -134,20 +147,25 @@ stream_norm_any_kernel(const StreamNormArgs a) {
     if (d != nullptr) {
       float s = ld_f(d + c);
       for (int p = 1; p < a.n_part; ++p) s += ld_f(d + (size_t)p * a.part_stride + c);
-      v += s;
+      v = fmaf(a.factor, s, v);
     }
     if (a.add != nullptr) v += a.add[c];
     return v;
   };
   const bool in_place = a.rows == nullptr;
-  float ss = 0.f;
+  float ss = 0.f, sd = 0.f;
   for (int c = threadIdx.x; c < a.width; c += 256) {
     const float v = value(c);
     if (in_place) x[c] = v;
     ss += v * v;
+    if (a.dot != nullptr) sd += v * a.dot[c];
   }
   if (a.out == nullptr) return;
-  const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.width + a.eps);
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red[0]) / (float)a.width + a.eps);
+  if (a.dot != nullptr) {
+    const float g = block_sum_256(sd, red[1]) * inv;
+    if (threadIdx.x == 0) a.gate[r] = 1.0f / (1.0f + expf(-g));
+  }
   TO* o = (TO*)a.out + r * a.ld_out;
   for (int c = threadIdx.x; c < a.width; c += 256) st_f(o + c, (in_place ? x[c] : value(c)) * inv * a.weight[c]);
   for (int c = a.width + threadIdx.x; c < a.ld_out; c += 256) st_f(o + c, 0.f);
@@ -281,7 +299,40 @@ struct JoinPart {               // mirrored by ops/stream.py
   long stride;
   int f32, n_part, ld, k;
   float scale;
+  const float* row_scale;       // one more factor per row (null = none)
 };
+
+// x[0 .. V - 1] (columns c ... of row r) += the part's result
+template <int V>
+__device__ __forceinline__ void add_part(const JoinPart& d, size_t r, int c, float* x) {
+  float u[V];
+#pragma unroll
+  for (int j = 0; j < V; ++j) u[j] = 0.f;
+  auto load = [&](const auto* p, float* v) {
+    if constexpr (V == 4) { const float4 q = ld4(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+    else v[0] = ld_f(p);
+  };
+  auto add = [&](size_t off, float w) {
+    float q[V];
+    if (d.f32) load((const float*)d.p + off + c, q); else load((const __nv_bfloat16*)d.p + off + c, q);
+#pragma unroll
+    for (int j = 0; j < V; ++j) u[j] = fmaf(w, q[j], u[j]);
+  };
+  if (d.pair_row != nullptr) {
+#pragma unroll 4
+    for (int e = 0; e < d.k; ++e) {
+      const int row = d.pair_row[r * d.k + e];
+      if (row >= 0) add((size_t)row * d.ld, d.weights[r * d.k + e]);
+    }
+  } else {
+#pragma unroll 4
+    for (int p = 0; p < d.n_part; ++p) add((size_t)p * d.stride + r * d.ld, 1.0f);
+  }
+  const float f = d.row_scale != nullptr ? d.scale * d.row_scale[r] : d.scale;
+#pragma unroll
+  for (int j = 0; j < V; ++j) x[j] = fmaf(f, u[j], x[j]);
+}
+
 struct JoinArgs {
   float* x;
   JoinPart part[3]; int n;
@@ -312,28 +363,7 @@ stream_join_kernel(const JoinArgs a) {
 #pragma unroll
   for (int i = 0; i < 3; ++i) {
     if (i >= a.n) break;
-    const JoinPart& d = a.part[i];
-    float u[V];
-#pragma unroll
-    for (int j = 0; j < V; ++j) u[j] = 0.f;
-    auto add = [&](size_t off, float w) {
-      float q[V];
-      if (d.f32) load((const float*)d.p + off + c, q); else load((const __nv_bfloat16*)d.p + off + c, q);
-#pragma unroll
-      for (int j = 0; j < V; ++j) u[j] = fmaf(w, q[j], u[j]);
-    };
-    if (d.pair_row != nullptr) {
-#pragma unroll 4
-      for (int e = 0; e < d.k; ++e) {
-        const int row = d.pair_row[r * d.k + e];
-        if (row >= 0) add((size_t)row * d.ld, d.weights[r * d.k + e]);
-      }
-    } else {
-#pragma unroll 4
-      for (int p = 0; p < d.n_part; ++p) add((size_t)p * d.stride + r * d.ld, 1.0f);
-    }
-#pragma unroll
-    for (int j = 0; j < V; ++j) x[j] = fmaf(d.scale, u[j], x[j]);
+    add_part<V>(a.part[i], r, c, x);
   }
   if constexpr (V == 4) {
     const float4 y = make_float4(x[0], x[1], x[2], x[3]);
@@ -343,6 +373,131 @@ stream_join_kernel(const JoinArgs a) {
     a.x[r * a.width + c] = x[0];
     if (a.out != nullptr) st_f((TO*)a.out + r * a.ld_out + c, x[0]);
   }
+}
+
+// ------------------------------------------------------------------------------------------ averages over the stream at earlier places
+struct DepthArgs {
+  float* x;                     // stream [rows, width]; becomes the average
+  JoinPart part[3]; int n;
+  float* hist; long stride;     // [places][rows, width], `stride` elements apart: the streams kept so far; the new one goes to place `at`
+  const float* base; int first; // the sum over the places below `first` [rows, width] (null: first = 0)
+  int at; const float* w;       // the average is the sum of w[j] * place j, j = 0 .. at
+  const float* weight;          // f32 [width], of the norm
+  const long long* rows;        // output row r comes from stream row rows[r] (then neither stream nor history is written); null = all rows in place
+  void* out; int ld_out;        // normalised rows, zero behind `width`; null = only the average
+  int width; float eps;
+};
+
+template <typename TO, int V, int VPT>             // V columns at a time, VPT times: width <= 256 * V * VPT, a multiple of V
+__global__ void __launch_bounds__(256)
+stream_depth_kernel(const DepthArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[8];
+  const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
+  auto load = [&](const float* p, float* v) {
+    if constexpr (V == 4) { const float4 q = ld4(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
+    else v[0] = *p;
+  };
+  auto store = [&](auto* p, const float* v) {
+    if constexpr (V == 4) st4(p, make_float4(v[0], v[1], v[2], v[3]));
+    else st_f(p, v[0]);
+  };
+  float x[VPT][V];
+  const float w_at = a.w[a.at];
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * 256) * V;
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[i][j] = 0.f;
+    if (c >= a.width) continue;
+    load(a.x + src * a.width + c, x[i]);
+#pragma unroll
+    for (int p = 0; p < 3; ++p) if (p < a.n) add_part<V>(a.part[p], src, c, x[i]);
+    if (a.rows == nullptr) store(a.hist + (size_t)a.at * a.stride + src * a.width + c, x[i]);
+#pragma unroll
+    for (int j = 0; j < V; ++j) x[i][j] *= w_at;
+    if (a.base != nullptr) {
+      float q[V];
+      load(a.base + src * a.width + c, q);
+#pragma unroll
+      for (int j = 0; j < V; ++j) x[i][j] += q[j];
+    }
+  }
+#pragma unroll 4
+  for (int j = a.first; j < a.at; ++j) {
+    const float w = a.w[j];
+    const float* h = a.hist + (size_t)j * a.stride + src * a.width;
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (threadIdx.x + i * 256) * V;
+      if (c >= a.width) continue;
+      float q[V];
+      load(h + c, q);
+#pragma unroll
+      for (int y = 0; y < V; ++y) x[i][y] = fmaf(w, q[y], x[i][y]);
+    }
+  }
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * 256) * V;
+#pragma unroll
+    for (int j = 0; j < V; ++j) ss += x[i][j] * x[i][j];
+    if (c < a.width && a.rows == nullptr) store(a.x + src * a.width + c, x[i]);
+  }
+  if (a.out == nullptr) return;
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.width + a.eps);
+  TO* o = (TO*)a.out + r * a.ld_out;
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (threadIdx.x + i * 256) * V;
+    if (c >= a.width) continue;
+    float w[V], y[V];
+    load(a.weight + c, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) y[j] = x[i][j] * inv * w[j];
+    store(o + c, y);
+  }
+  for (int c = a.width + threadIdx.x; c < a.ld_out; c += 256) st_f(o + c, 0.f);
+}
+
+// base[k] = sum of w[k][j] * place j over j < places, for k < K: every place is read once.
+constexpr int kDepthBlock = 8;
+struct DepthBaseArgs { const float* hist; long stride; int places; const float* w[kDepthBlock]; float* base; long n; };
+
+template <int V>
+__global__ void __launch_bounds__(256)
+depth_base_kernel(const DepthBaseArgs a, int k_n) {
+  pdl_wait();
+  pdl_trigger();
+  const long i = ((long)blockIdx.x * 256 + threadIdx.x) * V;
+  if (i >= a.n) return;
+  float acc[kDepthBlock][V];
+#pragma unroll
+  for (int k = 0; k < kDepthBlock; ++k)
+#pragma unroll
+    for (int y = 0; y < V; ++y) acc[k][y] = 0.f;
+#pragma unroll 4
+  for (int j = 0; j < a.places; ++j) {
+    float q[V];
+    const float* p = a.hist + (size_t)j * a.stride + i;
+    if constexpr (V == 4) { const float4 f = ld4(p); q[0] = f.x; q[1] = f.y; q[2] = f.z; q[3] = f.w; }
+    else q[0] = *p;
+#pragma unroll
+    for (int k = 0; k < kDepthBlock; ++k) {
+      const float w = k < k_n ? a.w[k][j] : 0.f;
+#pragma unroll
+      for (int y = 0; y < V; ++y) acc[k][y] = fmaf(w, q[y], acc[k][y]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < kDepthBlock; ++k)
+    if (k < k_n) {
+      float* p = a.base + (size_t)k * a.n + i;
+      if constexpr (V == 4) st4(p, make_float4(acc[k][0], acc[k][1], acc[k][2], acc[k][3]));
+      else *p = acc[k][0];
+    }
 }
 
 // ------------------------------------------------------------------------------------------ gates
@@ -507,6 +662,7 @@ struct QkUnitArgs {
   int hq, hkv, dk, dv, dkp, dvp;
   float eps, q_scale;
   int unit;                     // 0: no normalisation
+  const int* positions; float temp; double every;    // Q times 1 + temp ln(floor((position + 1) / every) + 1); null = not
 };
 
 // One warp per (token, head): heads 0 .. hq-1 are queries, then hkv keys, then hkv values.
@@ -539,6 +695,7 @@ qk_unit_store_kernel(const QkUnitArgs a, long n_items) {
     return s;
   };
   const bool norm = a.unit && (is_q || is_k);
+  const float q_scale = is_q && a.positions != nullptr ? a.q_scale * fmaf(a.temp, logf((float)floor((double)(a.positions[t] + 1) / a.every) + 1.0f), 1.0f) : a.q_scale;
   if (d <= 128) {               // the head's values stay in registers
     float v[4];
     float ss = 0.f;
@@ -546,7 +703,7 @@ qk_unit_store_kernel(const QkUnitArgs a, long n_items) {
     for (int i = 0; i < 4; ++i) { const int c = lane + 32 * i; v[i] = c < d ? value(c) : 0.f; ss += v[i] * v[i]; }
     float sc = 1.0f;
     if (norm) sc = 1.0f / sqrtf(warp_sum(ss) / (float)d + a.eps);
-    if (is_q) sc *= a.q_scale;
+    if (is_q) sc *= q_scale;
 #pragma unroll
     for (int i = 0; i < 4; ++i) { const int c = lane + 32 * i; if (c < dp) st_f(dst + c, v[i] * sc); }
     return;
@@ -557,7 +714,7 @@ qk_unit_store_kernel(const QkUnitArgs a, long n_items) {
     for (int c = lane; c < d; c += 32) { const float v = value(c); ss += v * v; }
     sc = 1.0f / sqrtf(warp_sum(ss) / (float)d + a.eps);
   }
-  if (is_q) sc *= a.q_scale;
+  if (is_q) sc *= q_scale;
   for (int c = lane; c < dp; c += 32) st_f(dst + c, c < d ? value(c) * sc : 0.f);
 }
 
@@ -732,7 +889,14 @@ part_norm_kernel(const PartNormArgs a) {
     for (int c = a.n + lane; c < a.ld_out; c += G) st_f(out + c, 0.f);
 }
 
-// ------------------------------------------------------------------------------------------ act(gate) * up, f32
+// ------------------------------------------------------------------------------------------ activations, f32
+__global__ void gelu_f32_kernel(const float* __restrict__ x, float* __restrict__ out, long n) {
+  pdl_wait();
+  pdl_trigger();
+  const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i < n) out[i] = 0.5f * x[i] * (1.0f + erff(x[i] * 0.70710678118654752f));
+}
+
 __global__ void act_mul_f32_kernel(const float* __restrict__ gu, float* __restrict__ out, long n, int inter, int ld, int act, float cap) {
   pdl_wait();
   pdl_trigger();
@@ -768,7 +932,7 @@ static int stream_norm_launch(const StreamNormArgs& a, int n_rows, cudaStream_t 
   const size_t ed = sizeof(TD) * 4, eo = sizeof(TO) * 4;
   const bool vec = a.width % 4 == 0 && a.width <= 16384 && (a.delta == nullptr || (a.ld_delta % 4 == 0 && a.part_stride % 4 == 0 && (uintptr_t)a.delta % ed == 0)) &&
                    (a.out == nullptr || (a.ld_out % 4 == 0 && (uintptr_t)a.out % eo == 0)) && (uintptr_t)a.x % 16 == 0 && (uintptr_t)a.weight % 16 == 0 &&
-                   (uintptr_t)a.add % 16 == 0;
+                   (uintptr_t)a.add % 16 == 0 && (uintptr_t)a.dot % 16 == 0;
   if (!vec) launch_k(stream_norm_any_kernel<TD, TO>, (unsigned)n_rows, 256, 0, stream, a);
   else if (a.width <= 1024) launch_k(stream_norm_vec_kernel<TD, TO, 1>, (unsigned)n_rows, 256, 0, stream, a);
   else if (a.width <= 4096) launch_k(stream_norm_vec_kernel<TD, TO, 4>, (unsigned)n_rows, 256, 0, stream, a);
@@ -778,13 +942,15 @@ static int stream_norm_launch(const StreamNormArgs& a, int n_rows, cudaStream_t 
 }
 
 // See StreamNormArgs.  delta_f32 / out_f32 give the element types; `rows` (int64, device) selects stream rows.
-GB_API int gb_stream_norm(float* x, const void* delta, int delta_f32, int n_part, long part_stride, int ld_delta, const float* add, const float* weight,
-                          const long long* rows, void* out, int out_f32, int ld_out, int n_rows, int width, float eps, cudaStream_t stream) {
+GB_API int gb_stream_norm(float* x, const void* delta, int delta_f32, int n_part, long part_stride, int ld_delta, float factor, const float* add, const float* weight,
+                          const float* dot, float* gate, const long long* rows, void* out, int out_f32, int ld_out, int n_rows, int width, float eps, cudaStream_t stream) {
   if (n_rows <= 0) return 0;
   if (width <= 0 || (out != nullptr && (ld_out < width || weight == nullptr)) || (delta != nullptr && (ld_delta < width || n_part < 1)))
     return fail("stream_norm: bad widths%s");
   StreamNormArgs a;
+  if (dot != nullptr && (gate == nullptr || rows != nullptr || out == nullptr)) return fail("stream_norm: a gate goes with all rows%s");
   a.x = x; a.delta = delta; a.n_part = n_part; a.part_stride = part_stride; a.ld_delta = ld_delta; a.add = add; a.weight = weight; a.rows = rows;
+  a.factor = factor; a.dot = dot; a.gate = gate;
   a.out = out; a.ld_out = ld_out; a.width = width; a.eps = eps;
   if (delta_f32) return out_f32 ? stream_norm_launch<float, float>(a, n_rows, stream) : stream_norm_launch<float, __nv_bfloat16>(a, n_rows, stream);
   return out_f32 ? stream_norm_launch<__nv_bfloat16, float>(a, n_rows, stream) : stream_norm_launch<__nv_bfloat16, __nv_bfloat16>(a, n_rows, stream);
@@ -851,13 +1017,15 @@ GB_API int gb_part_norm(const float* o, int ld_o, const void* gate, int gate_f32
 // See QkUnitArgs.  in_f32: element type of qkv; cache_f32: element type of q_out and the caches.
 GB_API int gb_qk_unit_store(const void* qkv, int in_f32, int n_part, long part_stride, int ld, const int* slots, void* q_out, void* k_cache, void* v_cache,
                             int cache_f32, long num_slots, int tokens, int hq, int hkv, int dk, int dv, int dkp, int dvp, float eps, float q_scale,
-                            int unit, cudaStream_t stream) {
+                            int unit, const int* positions, float temp, double every, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (hq < 1 || hkv < 1 || hq % hkv || dk < 1 || dv < 1 || dkp < dk || dvp < dv || n_part < 1) return fail("qk_unit_store: bad sizes%s");
   if ((dk <= 128 && dkp > 128) || (dv <= 128 && dvp > 128)) return fail("qk_unit_store: padding beyond 128%s");
   QkUnitArgs a;
   a.qkv = qkv; a.n_part = n_part; a.part_stride = part_stride; a.ld = ld; a.slots = slots; a.q_out = q_out; a.k_cache = k_cache; a.v_cache = v_cache;
   a.num_slots = num_slots; a.hq = hq; a.hkv = hkv; a.dk = dk; a.dv = dv; a.dkp = dkp; a.dvp = dvp; a.eps = eps; a.q_scale = q_scale; a.unit = unit;
+  if (positions != nullptr && !(every > 0.0)) return fail("qk_unit_store: bad temperature%s");
+  a.positions = positions; a.temp = temp; a.every = every;
   const long n = (long)tokens * (hq + 2 * hkv);
   const unsigned grid = (unsigned)((n + 7) / 8);
   if (in_f32 && cache_f32) launch_k(qk_unit_store_kernel<float, float>, grid, 256, 0, stream, a, n);
@@ -948,6 +1116,62 @@ GB_API int gb_stream_join(float* x, const JoinPart* parts, int n, void* out, int
   const dim3 grid((unsigned)n_rows, (unsigned)((cols + (vec ? 1023 : 255)) / (vec ? 1024 : 256)));
   if (out_f32) { if (vec) launch_k(stream_join_kernel<float, 4>, grid, 256, 0, stream, a); else launch_k(stream_join_kernel<float, 1>, grid, 256, 0, stream, a); }
   else { if (vec) launch_k(stream_join_kernel<__nv_bfloat16, 4>, grid, 256, 0, stream, a); else launch_k(stream_join_kernel<__nv_bfloat16, 1>, grid, 256, 0, stream, a); }
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+template <typename TO>
+static int stream_depth_launch(const DepthArgs& a, bool vec, int n_rows, cudaStream_t stream) {
+  const unsigned g = (unsigned)n_rows;
+  if (vec && a.width <= 1024) launch_k(stream_depth_kernel<TO, 4, 1>, g, 256, 0, stream, a);
+  else if (vec && a.width <= 2048) launch_k(stream_depth_kernel<TO, 4, 2>, g, 256, 0, stream, a);
+  else if (vec && a.width <= 4096) launch_k(stream_depth_kernel<TO, 4, 4>, g, 256, 0, stream, a);
+  else if (vec && a.width <= 16384) launch_k(stream_depth_kernel<TO, 4, 16>, g, 256, 0, stream, a);
+  else if (a.width <= 1024) launch_k(stream_depth_kernel<TO, 1, 4>, g, 256, 0, stream, a);
+  else if (a.width <= 16384) launch_k(stream_depth_kernel<TO, 1, 64>, g, 256, 0, stream, a);
+  else return fail("stream_depth: rows of at most 16384 columns%s");
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+// See DepthArgs; parts: host array of three.
+GB_API int gb_stream_depth(float* x, const JoinPart* parts, int n, float* hist, long stride, const float* base, int first, int at, const float* w, const float* weight,
+                           const long long* rows, void* out, int out_f32, int ld_out, int n_rows, int width, float eps, cudaStream_t stream) {
+  if (n_rows <= 0) return 0;
+  if (width <= 0 || n < 1 || n > 3 || at < 1 || first < 0 || first > at || (base == nullptr) != (first == 0) || (out != nullptr && (ld_out < width || weight == nullptr)))
+    return fail("stream_depth: bad arguments%s");
+  DepthArgs a;
+  const auto ok16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  bool vec = width % 4 == 0 && stride % 4 == 0 && ok16(x) && ok16(hist) && ok16(base) && ok16(weight) && (out == nullptr || (ld_out % 4 == 0 && (uintptr_t)out % (out_f32 ? 16 : 8) == 0));
+  for (int i = 0; i < 3; ++i) {
+    a.part[i] = parts[i];
+    if (i >= n) continue;
+    const JoinPart& d = parts[i];
+    if (d.p == nullptr || d.ld < width || d.n_part < 1 || (d.pair_row != nullptr && (d.weights == nullptr || d.k < 1))) return fail("stream_depth: bad part%s");
+    vec = vec && d.ld % 4 == 0 && d.stride % 4 == 0 && (uintptr_t)d.p % (d.f32 ? 16 : 8) == 0;
+  }
+  a.x = x; a.n = n; a.hist = hist; a.stride = stride; a.base = base; a.first = first; a.at = at; a.w = w; a.weight = weight; a.rows = rows; a.out = out; a.ld_out = ld_out;
+  a.width = width; a.eps = eps;
+  return out_f32 ? stream_depth_launch<float>(a, vec, n_rows, stream) : stream_depth_launch<__nv_bfloat16>(a, vec, n_rows, stream);
+}
+
+// base [k_n][n] from `places` blocks of n elements, `stride` apart; w: host array of k_n device pointers to at least `places` weights.
+GB_API int gb_depth_base(const float* hist, long stride, int places, const float* const* w, int k_n, float* base, long n, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  if (places < 1 || k_n < 1 || k_n > kDepthBlock) return fail("depth_base: bad sizes%s");
+  DepthBaseArgs a;
+  for (int k = 0; k < kDepthBlock; ++k) a.w[k] = k < k_n ? w[k] : nullptr;
+  a.hist = hist; a.stride = stride; a.places = places; a.base = base; a.n = n;
+  const bool vec = n % 4 == 0 && stride % 4 == 0 && ((uintptr_t)hist & 15) == 0 && ((uintptr_t)base & 15) == 0;
+  if (vec) launch_k(depth_base_kernel<4>, (unsigned)((n / 4 + 255) / 256), 256, 0, stream, a, k_n);
+  else launch_k(depth_base_kernel<1>, (unsigned)((n + 255) / 256), 256, 0, stream, a, k_n);
+  GB_CUDA_OK(cudaGetLastError());
+  return 0;
+}
+
+GB_API int gb_gelu_f32(const float* x, float* out, long n, cudaStream_t stream) {
+  if (n <= 0) return 0;
+  launch_k(gelu_f32_kernel, (unsigned)((n + 255) / 256), 256, 0, stream, x, out, n);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }

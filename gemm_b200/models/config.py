@@ -14,21 +14,28 @@ from dataclasses import asdict, dataclass, field, replace
 from typing import Dict, List, Optional
 
 # Architectures described layer by layer (``ModelConfig.layer_specs``): name in config.json -> arch
-LAYERED_ARCHS = {"Zogavik": "zogavik", "Famepel": "famepel", "Fidolix": "fidolix"}
+LAYERED_ARCHS = {"Zogavik": "zogavik", "Famepel": "famepel", "Fidolix": "fidolix", "Zedirax": "zedirax"}
 
 ARCHS = ("qwen2", "qwen2vl", "qwen3", "qwen3vl", "qwen3moe", "qwen3vlmoe", "qwen35", "qwen35moe")
 
 
 @dataclass
 class RotarySpec:
-    """Rotary positions of neighbouring pairs (2i, 2i + 1).  ``factor`` > 0: YaRN, with the pairs between ``fast`` and ``slow`` turns over
-    ``original`` positions blended from the plain to the divided frequency."""
+    """Rotary positions of neighbouring pairs (2i, 2i + 1), or (``halves``) of the pairs (i, i + dims / 2).  ``factor`` > 0: YaRN, with the pairs between
+    ``fast`` and ``slow`` turns over ``original`` positions blended from the plain to the divided frequency."""
     dims: int
     base: float
     factor: float = 0.0
     original: float = 0.0
     fast: float = 0.0
     slow: float = 0.0
+    halves: bool = False
+
+    def pair_order(self) -> List[int]:
+        """The rotated dimensions with the members of a pair side by side: a projection whose rows are in this order makes neighbouring pairs of any
+        layout (scores do not depend on the order, as long as queries and keys share it)."""
+        n = self.dims // 2
+        return [j for i in range(n) for j in (i, i + n)] if self.halves else list(range(self.dims))
 
     def frequencies(self) -> List[float]:
         f = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
@@ -51,8 +58,9 @@ class RotarySpec:
 
 @dataclass
 class MoeSpec:
-    """A mixture of experts: gated feed-forwards of width ``ffn``, ``top`` of ``n_experts`` per token.  ``groups`` > 1: the experts form groups of
-    neighbours, a group scores the sum of its ``group_best`` (1 or 2) best experts, and only the best ``groups_kept`` groups can be chosen from."""
+    """A mixture of experts: feed-forwards of width ``ffn``, ``top`` of ``n_experts`` per token, SiLU-gated or (``act`` "gelu") plain.  ``groups`` > 1: the experts
+    form groups of neighbours, a group scores the sum of its ``group_best`` (1 or 2) best experts, and only the best ``groups_kept`` groups can be chosen from.
+    ``shared`` > 0: one more expert of that width sees every token, times the sigmoid of a projection of the token to one number."""
     n_experts: int
     top: int
     ffn: int
@@ -62,15 +70,25 @@ class MoeSpec:
     groups: int = 1
     groups_kept: int = 1
     group_best: int = 2
+    act: str = "silu"                       # act(gate) * up -> down; "gelu": the exact GELU of up alone -> down
+    shared: int = 0
+
+    @property
+    def gated(self) -> bool:
+        return self.act != "gelu"
+
+
+# mixers with a state of a fixed size per sequence
+RECURRENT = ("lightning", "mamba2", "hgrn2", "rwkv", "mingru")
 
 
 @dataclass
 class LayerSpec:
     """One layer of a model described layer by layer: its mixer with the mixer's own sizes, and its feed-forward."""
-    mixer: str                              # "attention" | "lightning" | "mamba2" | "hgrn2" | "latent" | "rwkv" | "parallel"
+    mixer: str                              # "attention" | "lightning" | "mamba2" | "hgrn2" | "latent" | "rwkv" | "mingru" | "parallel"
     n_heads: int
     head_dim: int                           # query / key size per head (mamba2: the state size; latent: without the rotated part)
-    v_dim: int                              # value size per head
+    v_dim: int                              # value size per head (mingru: the state, one head of one row)
     n_kv_heads: int = 0                     # attention only
     # attention
     scale: float = 0.0                      # factor of q . k (0 = 1 / sqrt(head_dim))
@@ -84,6 +102,9 @@ class LayerSpec:
     softcap: float = 0.0                    # scores become softcap * tanh(score / softcap) (0 = as they are)
     out_gate: bool = False                  # the heads' outputs are multiplied by the sigmoid of a projection
     v_from_k: bool = False                  # the values are the keys before their rotation
+    log_bias: bool = False                  # r1 ln(1 + r2 distance) is taken off the scores, two learned numbers per head
+    temp_coef: float = 0.0                  # queries at position p are multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)
+    temp_every: float = 1.0
     # lightning attention
     decay: Optional[List[float]] = None     # per head
     # mamba2
@@ -99,7 +120,7 @@ class LayerSpec:
     right_scale: float = 1.0
     # latent attention: keys and values are projections of a cached latent, next to one rotated key part for all heads
     kv_rank: int = 0
-    q_rank: int = 0
+    q_rank: int = 0                         # queries through a normed latent of their own (0: projected at once)
     rot_dim: int = 0
     rotary: Optional[RotarySpec] = None
     sink: bool = False                      # a learned score per head joins the softmax's sum
@@ -108,6 +129,7 @@ class LayerSpec:
     ffn: int = 0
     act: str = "silu"                       # or "gelu_tanh", "capped" (x sigmoid(1.702 x) of min(gate, cap), times 1 + up within +-cap)
     act_cap: float = 0.0
+    ffn_bias: bool = False                  # all three projections of the dense feed-forward have biases
     moe: Optional[MoeSpec] = None           # in place of the dense feed-forward
 
     def __post_init__(self):
@@ -136,7 +158,7 @@ class LayerSpec:
     @property
     def has_state(self) -> bool:
         """Whether the mixer carries state of a fixed size per sequence, which cannot drop positions."""
-        return any(x.mixer in ("lightning", "mamba2", "hgrn2", "rwkv") or x.conv_taps > 1 for x in self.mixers)
+        return any(x.mixer in RECURRENT or x.conv_taps > 1 for x in self.mixers)
 
     @property
     def paged(self) -> Optional["LayerSpec"]:
@@ -221,6 +243,8 @@ class ModelConfig:
     embed_scale: float = 1.0
     parallel_ffn: bool = False              # mixer and feed-forward read the same stream, each through a norm of its own
     side_dim: int = 0                       # per-layer token input of this size (a table of the token's vectors for all layers), 0 = none
+    residual_mult: float = 1.0              # factor of every sublayer's result
+    depth_average: bool = False             # a layer hands on a learned weighted sum of the embedding output and all layers' results so far
 
     def __post_init__(self):
         if self.layer_specs is not None:
@@ -248,7 +272,7 @@ class ModelConfig:
 
     @property
     def has_recurrent_state(self) -> bool:
-        """Whether a sequence carries state that cannot drop positions (Delta-Net, lightning, Mamba-2, HGRN2 or RWKV layers, convolutions)."""
+        """Whether a sequence carries state that cannot drop positions (Delta-Net, lightning, Mamba-2, HGRN2, RWKV or minGRU layers, convolutions)."""
         return self.is_hybrid or (self.is_layered and any(x.has_state for x in self.layer_specs))
 
     @property
@@ -285,7 +309,8 @@ class ModelConfig:
             tot = self.vocab * self.hidden * (1 if self.tie_embeddings else 2) + self.vocab * self.n_layers * self.side_dim
             for x in self.layer_specs:
                 if x.moe is not None:
-                    tot += x.moe.n_experts * self.hidden * (3 * x.moe.ffn + 1)
+                    per = 3 if x.moe.gated else 2
+                    tot += x.moe.n_experts * self.hidden * (per * x.moe.ffn + 1) + (self.hidden * (per * x.moe.shared + 1) if x.moe.shared else 0)
                 tot += 3 * self.hidden * x.ffn + 2 * self.hidden * self.side_dim
             for x in (m for sp in self.layer_specs for m in sp.mixers):
                 nv = x.n_heads * x.v_dim
@@ -297,7 +322,9 @@ class ModelConfig:
                     tot += self.hidden * (2 * nv + x.conv_channels + x.n_heads) + x.conv_channels * x.conv_taps
                 elif x.mixer == "latent":
                     own = 0 if x.kv_from >= 0 else x.kv_rank + x.rot_dim
-                    tot += self.hidden * (x.q_rank + own + nv) + x.q_rank * x.n_heads * (x.head_dim + x.rot_dim) + x.kv_rank * (x.q_dim + nv)
+                    tot += self.hidden * (x.q_rank + own + (2 if x.out_gate else 1) * nv) + (x.q_rank or self.hidden) * x.n_heads * (x.head_dim + x.rot_dim) + x.kv_rank * (x.q_dim + nv)
+                elif x.mixer == "mingru":
+                    tot += 4 * self.hidden * nv
                 elif x.mixer == "rwkv":
                     tot += self.hidden * (2 * x.q_dim + 3 * nv + x.decay_rank) + x.q_dim * x.decay_rank
                 else:
@@ -422,6 +449,31 @@ PRESETS["tiny-fidolix"] = _fidolix("pAPa", 192, 300, 20, (4, 2, 40, 24), (6, 3, 
 # layers of the sizes of a 30-billion-parameter mixture of experts (128 experts, 8 per token), every third one attention without a window
 PRESETS["fidolix-30b-a3b"] = _fidolix("pPA" + "PPA" * 14, 2048, 151936, 128, (32, 4, 128, 128), (16, 2, 128), (16, 128, 64), RotarySpec(64, 500000.0, 8.0, 4096, 32.0, 1.0),
                                       1024, 4, 30.0, 6144, 7.0, MoeSpec(128, 8, 768, renorm=True, groups=8, groups_kept=4, group_best=1), 2048 ** 0.5)
+
+
+def _zedirax(pattern: str, hidden: int, vocab: int, width: int, latent, att, temp, rotary: RotarySpec, dense: int, moe: MoeSpec, mult: float) -> ModelConfig:
+    """``pattern``: one letter per layer, G = minGRU, L = latent attention, A = attention, with a mixture of experts; g, l, a = with a dense feed-forward.  ``latent``
+    (heads, dim, rot_dim, vdim, kv_rank), ``att`` (heads, KV heads, dim, vdim), ``temp`` (coefficient, every)."""
+    specs: List[LayerSpec] = []
+    for c in pattern:
+        ff = dict(ffn=dense, act="gelu_tanh", ffn_bias=True) if c.islower() else dict(moe=moe)
+        if c in "Gg":
+            specs.append(LayerSpec("mingru", 1, 1, width, **ff))
+        elif c in "Ll":
+            hd, d, r, v, kvr = latent
+            specs.append(LayerSpec("latent", hd, d, v, n_kv_heads=1, scale=(d + r) ** -0.5, kv_rank=kvr, rot_dim=r, rotary=rotary, out_gate=True, **ff))
+        else:
+            hd, g, d, v = att
+            specs.append(LayerSpec("attention", hd, d, v, n_kv_heads=g, scale=d ** -0.5, log_bias=True, temp_coef=temp[0], temp_every=temp[1], **ff))
+    return ModelConfig(arch="zedirax", layer_specs=specs, hidden=hidden, n_heads=att[0], n_kv_heads=att[1], head_dim=att[2], ffn=dense, vocab=vocab, rms_eps=1e-5, norm_offset=1.0,
+                       residual_mult=mult, depth_average=True, qk_norm=False)
+
+
+PRESETS["tiny-zedirax"] = _zedirax("gLAgl", 192, 300, 136, (3, 24, 8, 40, 72), (4, 2, 40, 24), (0.25, 50), RotarySpec(8, 10000.0, halves=True), 320,
+                                   MoeSpec(10, 3, 56, act="gelu", shared=88), 0.6)
+# layers of the sizes of a 30-billion-parameter mixture of experts (128 experts, 8 per token; a plain expert of 1152 has the size of a gated one of 768)
+PRESETS["zedirax-30b-a3b"] = _zedirax("gGLGGAGGL" + "GGLGGAGGL" * 4, 2048, 151936, 4096, (32, 128, 64, 128, 512), (32, 4, 128, 128), (0.1, 8192), RotarySpec(64, 500000.0, halves=True),
+                                      6144, MoeSpec(128, 8, 1152, act="gelu", shared=1152), 0.5)
 
 
 def get_config(name: str) -> ModelConfig:

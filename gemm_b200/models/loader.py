@@ -521,7 +521,7 @@ def _qwen35_config_from_hf(c: dict) -> ModelConfig:
 
 class LayeredSource(SafetensorsSource):
     """Checkpoints of models described layer by layer: tensors ``l<i>.norm1``, ``l<i>.mix.*`` (``l<i>.mix.left.*`` and ``l<i>.mix.right.*`` for two mixers side
-    by side), ``l<i>.norm2``, ``l<i>.mlp.*``, ``l<i>.side.*``, ``embed``, ``side.embed``, ``final.norm``, ``loop.step``, served under the names the model
+    by side), ``l<i>.norm2``, ``l<i>.mlp.*``, ``l<i>.side.*``, ``l<i>.dwa``, ``embed``, ``side.embed``, ``final.norm``, ``loop.step``, served under the names the model
     builder asks for."""
 
     _LAYER = {"attn_q.weight": "mix.q", "attn_k.weight": "mix.k", "attn_v.weight": "mix.v",
@@ -539,6 +539,10 @@ class LayeredSource(SafetensorsSource):
               "rwkv_r.weight": "mix.r", "rwkv_k.weight": "mix.k", "rwkv_v.weight": "mix.v", "rwkv_g.weight": "mix.g", "rwkv_mu_r": "mix.mu.r", "rwkv_mu_k": "mix.mu.k",
               "rwkv_mu_v": "mix.mu.v", "rwkv_mu_g": "mix.mu.g", "rwkv_mu_w": "mix.mu.w", "rwkv_w1.weight": "mix.w1", "rwkv_w2.weight": "mix.w2", "rwkv_w0": "mix.w0",
               "rwkv_u": "mix.u", "rwkv_norm.weight": "mix.norm", "rwkv_out.weight": "mix.o",
+              "attn_q_direct.weight": "mix.q", "attn_r1": "mix.r1", "attn_r2": "mix.r2",
+              "gru_z.weight": "mix.z", "gru_z.bias": "mix.z.b", "gru_x.weight": "mix.x", "gru_x.bias": "mix.x.b", "gru_gate.weight": "mix.g", "gru_out.weight": "mix.o",
+              "ffn_gate.bias": "mlp.gate.b", "ffn_up.bias": "mlp.up.b", "ffn_down.bias": "mlp.down.b",
+              "ffn_up_shexp.weight": "mlp.shared.up", "ffn_down_shexp.weight": "mlp.shared.down", "ffn_gate_inp_shexp.weight": "mlp.shared.sg", "depth_weights": "dwa",
               "side_gate.weight": "side.gate", "side_proj.weight": "side.proj", "side_norm.weight": "side.norm"}
     _NORM = {"attn_norm": "norm1", "attn_post_norm": "norm1b", "ffn_norm": "norm2", "ffn_post_norm": "norm2b", "output_norm": "final.norm"}
     _PART = {"weight": "", "bias": ".b", "alpha": ".alpha"}
@@ -595,9 +599,9 @@ def _moe_spec(mlp: dict, **rule) -> MoeSpec:
     return spec
 
 
-def _rotary_spec(r: dict) -> RotarySpec:
+def _rotary_spec(r: dict, halves: bool = False) -> RotarySpec:
     sc = r.get("scaling")
-    return RotarySpec(int(r["dims"]), float(r["base"]), *((float(sc[k]) for k in ("factor", "original", "fast", "slow")) if sc else ()))
+    return RotarySpec(int(r["dims"]), float(r["base"]), *((float(sc[k]) for k in ("factor", "original", "fast", "slow")) if sc else ()), halves=halves)
 
 
 def _famepel_layer(li: int, e: dict, layers: list) -> LayerSpec:
@@ -682,7 +686,46 @@ def _fidolix_config(c: dict, path: str) -> ModelConfig:
                        parallel_ffn=True, side_dim=int(c["token_side"]["dim"]), loop=_loop_spec(c, "embedding"))
 
 
+def _zedirax_layer(li: int, e: dict) -> LayerSpec:
+    m, mlp, kind = e["mixer"], e.get("mlp"), e["type"]
+    ff = {}
+    if mlp is not None:
+        if mlp.get("kind") == "dense":
+            ff = dict(ffn=int(mlp["ff"]), act="gelu_tanh", ffn_bias=True)
+        elif mlp.get("kind") == "moe":
+            ff = dict(moe=_moe_spec(mlp, router="softmax", act="gelu", shared=int((mlp.get("shared") or {}).get("ff", 0))))
+        else:
+            raise ValueError(f"layer {li}: feed-forward kind {mlp.get('kind')!r} is not supported")
+    if kind == "mingru":
+        return LayerSpec("mingru", 1, 1, int(m["width"]), **ff)
+    if kind == "latent_attention":
+        rot = _rotary_spec(m["rot"], halves=True)
+        if rot.dims != int(m["rot_dim"]) or rot.dims % 2:
+            raise ValueError(f"layer {li}: rotation over {rot.dims} of {m['rot_dim']} dimensions is not supported")
+        return LayerSpec("latent", int(m["heads"]), int(m["dim"]), int(m["vdim"]), n_kv_heads=1, scale=float(m["scale"]), kv_rank=int(m["kv_rank"]), rot_dim=rot.dims, rotary=rot,
+                         out_gate=True, **ff)
+    if kind == "attention":
+        heads, g, temp = int(m["heads"]), int(m["kv_heads"]), m.get("q_temp") or {}
+        if g < 1 or heads % g:
+            raise ValueError(f"layer {li}: {heads} query heads over kv_heads {g}")
+        return LayerSpec("attention", heads, int(m["dim"]), int(m["vdim"]), n_kv_heads=g, scale=float(m["scale"]), log_bias=True, temp_coef=float(temp.get("coef", 0.0)),
+                         temp_every=float(temp.get("every", 1.0)), **ff)
+    raise ValueError(f"layer {li}: mixer {kind!r} is not supported")
+
+
+def _zedirax_config(c: dict, path: str) -> ModelConfig:
+    """config.json of Zedirax: minGRU, latent attention with a gate on its heads, attention with a logarithmic distance bias and a query temperature, dense or
+    mixture-of-experts feed-forwards, an average over all earlier layers behind every layer."""
+    specs = [_zedirax_layer(li, e) for li, e in enumerate(c["layers"])]
+    att = next((s for s in specs if s.mixer == "attention"), specs[0])
+    return ModelConfig(arch=LAYERED_ARCHS[c["architecture"]], layer_specs=specs, hidden=int(c["width"]), vocab=int(c["vocab"]), n_heads=att.n_heads,
+                       n_kv_heads=max(1, att.n_kv_heads), head_dim=att.head_dim, ffn=max(s.ffn for s in specs), rms_eps=float(c["norm"]["eps"]), qk_norm=False, norm_offset=1.0,
+                       residual_mult=float(c["residual_mult"]), depth_average=True)
+
+
 def _layered_config(c: dict, path: str) -> ModelConfig:
+    if c["architecture"] == "Zedirax":
+        return _zedirax_config(c, path)
     if c["architecture"] == "Famepel":
         return _famepel_config(c)
     if c["architecture"] == "Fidolix":
@@ -855,14 +898,20 @@ def _save_layered(cfg: ModelConfig, src, path: str) -> None:
                 put(p + part + nm, shp)
         if cfg.side_dim:
             put(p + "side_gate.weight", (cfg.side_dim, h)); put(p + "side_proj.weight", (h, cfg.side_dim)); put(p + "side_norm.weight", (h,))
+        if cfg.depth_average:
+            put(p + "depth_weights", (li + 2,))
         if sp.ffn:
             put(p + "ffn_gate.weight", (sp.ffn, h)); put(p + "ffn_up.weight", (sp.ffn, h)); put(p + "ffn_down.weight", (h, sp.ffn))
+        if sp.ffn_bias:
+            put(p + "ffn_gate.bias", (sp.ffn,)); put(p + "ffn_up.bias", (sp.ffn,)); put(p + "ffn_down.bias", (h,))
         if sp.moe is not None:
             put(p + "ffn_gate_inp.weight", (sp.moe.n_experts, h))
             for e in range(sp.moe.n_experts):
-                for nm, shp in (("gate", (sp.moe.ffn, h)), ("up", (sp.moe.ffn, h)), ("down", (h, sp.moe.ffn))):
+                for nm, shp in (("gate", (sp.moe.ffn, h)), ("up", (sp.moe.ffn, h)), ("down", (h, sp.moe.ffn)))[0 if sp.moe.gated else 1:]:
                     name = f"ffn_{nm}_exps.weight"
                     out[LayeredSource.file_name(f"{p}{name}#{e}")] = src.get_expert(p + name, e, shp).to(torch.bfloat16)
+            if sp.moe.shared:
+                put(p + "ffn_up_shexp.weight", (sp.moe.shared, h)); put(p + "ffn_down_shexp.weight", (h, sp.moe.shared)); put(p + "ffn_gate_inp_shexp.weight", (1, h))
         layers.append({"type": {"latent": "latent_attention"}.get(sp.mixer, sp.mixer), "mixer": _mixer_config(sp), "mlp": _ffn_config(sp)})
     save_safetensors(out, os.path.join(path, "model.safetensors"))
     name = {v: k for k, v in LAYERED_ARCHS.items()}[cfg.arch]
@@ -875,6 +924,8 @@ def _save_layered(cfg: ModelConfig, src, path: str) -> None:
         c["loop"] = {"start": cfg.loop.start, "stop": cfg.loop.stop, "times": cfg.loop.times} if cfg.loop else None
     if cfg.side_dim:
         c["token_side"] = {"dim": cfg.side_dim}
+    if cfg.arch == "zedirax":
+        c["residual_mult"] = cfg.residual_mult
     with open(os.path.join(path, "config.json"), "w") as fh:
         json.dump(c, fh)
 
@@ -894,16 +945,21 @@ def mixer_tensors(sp: LayerSpec, h: int):
                 ("ssm_a_log", hd), ("ssm_d", hd), ("ssm_norm.weight", (nv,)), ("ssm_out.weight", (h, nv))]
     if sp.mixer == "latent":
         own = [] if sp.kv_from >= 0 else [("attn_kv_a.weight", (sp.kv_rank + sp.rot_dim, h)), ("attn_kv_a_norm.weight", (sp.kv_rank,))]
-        return own + [("attn_q_a.weight", (sp.q_rank, h)), ("attn_q_a_norm.weight", (sp.q_rank,)),
-                      ("attn_q_b.weight", (sp.n_heads * (sp.head_dim + sp.rot_dim), sp.q_rank)), ("attn_k_b.weight", (nq, sp.kv_rank)),
-                      ("attn_v_b.weight", (nv, sp.kv_rank)), ("attn_sink", (sp.n_heads,)), ("attn_output.weight", (h, nv))]
+        n = sp.n_heads * (sp.head_dim + sp.rot_dim)
+        own += [("attn_q_a.weight", (sp.q_rank, h)), ("attn_q_a_norm.weight", (sp.q_rank,)), ("attn_q_b.weight", (n, sp.q_rank))] if sp.q_rank else [("attn_q_direct.weight", (n, h))]
+        own += ([("attn_gate.weight", (nv, h))] if sp.out_gate else []) + ([("attn_sink", (sp.n_heads,))] if sp.sink else [])
+        return own + [("attn_k_b.weight", (nq, sp.kv_rank)), ("attn_v_b.weight", (nv, sp.kv_rank)), ("attn_output.weight", (h, nv))]
+    if sp.mixer == "mingru":
+        return [("gru_z.weight", (nv, h)), ("gru_z.bias", (nv,)), ("gru_x.weight", (nv, h)), ("gru_x.bias", (nv,)), ("gru_gate.weight", (nv, h)), ("gru_out.weight", (h, nv))]
     if sp.mixer == "rwkv":
         own = [(f"rwkv_{c}.weight", (nq if c in "rk" else nv, h)) for c in "rkvg"] + [(f"rwkv_mu_{c}", (h,)) for c in "rkvgw"]
         return own + [("rwkv_w1.weight", (sp.decay_rank, h)), ("rwkv_w2.weight", (nq, sp.decay_rank)), ("rwkv_w0", (nq,)), ("rwkv_u", (sp.n_heads, sp.head_dim)),
                       ("rwkv_norm.weight", (nv,)), ("rwkv_out.weight", (h, nv))]
     own, nk = [], sp.n_kv_heads * sp.head_dim
     for c, n in (("q", nq), ("k", nk)) + ((() if sp.v_from_k else (("v", sp.n_kv_heads * sp.v_dim),))):
-        own += [(f"attn_{c}.weight", (n, h)), (f"attn_{c}.bias", (n,))]
+        own += [(f"attn_{c}.weight", (n, h))] + ([(f"attn_{c}.bias", (n,))] if sp.qkv_bias else [])
+    if sp.log_bias:
+        own += [("attn_r1", (sp.n_heads,)), ("attn_r2", (sp.n_heads,))]
     if sp.conv_taps:
         own += [("attn_q.conv", (nq, sp.conv_taps)), ("attn_k.conv", (nk, sp.conv_taps))]
     if sp.qk_norm_rows:
@@ -918,6 +974,8 @@ def mixer_tensors(sp: LayerSpec, h: int):
 
 
 def _mixer_config(sp: LayerSpec) -> dict:
+    if sp.mixer == "mingru":
+        return {"width": sp.v_dim}
     m = {"heads": sp.n_heads, "vdim": sp.v_dim}
     if sp.mixer == "lightning":
         return {**m, "dim": sp.head_dim, "decay": list(sp.decay)}
@@ -926,7 +984,9 @@ def _mixer_config(sp: LayerSpec) -> dict:
     if sp.mixer == "mamba2":
         return {**m, "state": sp.head_dim, "groups": sp.state_groups, "conv": sp.conv_taps, "norm_groups": sp.norm_parts}
     if sp.mixer == "latent":
-        m = {**m, "dim": sp.head_dim, "rot_dim": sp.rot_dim, "kv_rank": sp.kv_rank, "q_rank": sp.q_rank, "scale": sp.scale, "rot": _rotary_config(sp.rotary)}
+        m = {**m, "dim": sp.head_dim, "rot_dim": sp.rot_dim, "kv_rank": sp.kv_rank, "scale": sp.scale, "rot": _rotary_config(sp.rotary)}
+        if sp.q_rank:
+            m["q_rank"] = sp.q_rank
         return {**m, "kv_from": sp.kv_from} if sp.kv_from >= 0 else m
     if sp.mixer == "parallel":
         return {"left": _mixer_config(sp.left), "right": _mixer_config(sp.right), "left_scale": sp.left_scale, "right_scale": sp.right_scale}
@@ -935,6 +995,8 @@ def _mixer_config(sp: LayerSpec) -> dict:
     m = {**m, "kv_heads": sp.n_kv_heads, "dim": sp.head_dim, "scale": sp.scale}
     if sp.softcap:
         return {**m, "softcap": sp.softcap}
+    if sp.log_bias:
+        return {**m, "q_temp": {"coef": sp.temp_coef, "every": sp.temp_every}}
     if sp.conv_taps:
         return {**m, "conv": sp.conv_taps, "rot": _rotary_config(sp.rotary), "mask": {"size": sp.window} if sp.window else None}
     return {**m, "bias_max": sp.rel_max, "mask": {"size": sp.window, "keep_first": sp.keep_first} if sp.window else None}
@@ -950,7 +1012,10 @@ def _rotary_config(r: RotarySpec) -> dict:
 def _ffn_config(sp: LayerSpec):
     if sp.moe is not None:
         r = sp.moe
-        rt = {"experts": r.n_experts, "top": r.top, "groups": {"count": r.groups, "keep": r.groups_kept}}
+        rt = {"experts": r.n_experts, "top": r.top}
+        if not r.gated:
+            return {"kind": "moe", "expert": {"ff": r.ffn}, "router": rt, **({"shared": {"ff": r.shared}} if r.shared else {})}
+        rt["groups"] = {"count": r.groups, "keep": r.groups_kept}
         if r.router == "sigmoid":
             rt["scale"] = r.scale
         return {"kind": "moe", "expert": {"ff": r.ffn}, "router": rt}

@@ -13,9 +13,10 @@ Layer recipe (reference: common/transformer.h:3550-4174):
   logits = RMSNorm(x) Whead^T on the last token of every sequence.
 
 Models described layer by layer (``ModelConfig.layer_specs``) run through the same loop: every layer names its mixer (attention with a window, kept
-first tokens, a distance bias, capped scores or sinks, latent attention, lightning attention, HGRN2, Mamba-2, RWKV, or two of them side by side)
+first tokens, a distance bias, capped scores or sinks, latent attention, lightning attention, HGRN2, Mamba-2, RWKV, minGRU, or two of them side by side)
 and its feed-forward (dense or a mixture of experts) with sizes of its own, layers may be looped (every run has its own cache: ``KvCache`` is
 indexed by run), and the residual stream is f32.  The feed-forward follows the mixer, or reads the same stream beside it (``parallel_ffn``).
+A layer may hand on a weighted sum of all the streams so far (``depth_average``).
 """
 from __future__ import annotations
 
@@ -32,7 +33,7 @@ from ..ops import elementwise as ew
 from ..ops import deltanet as dn
 from ..ops import gemm, latent, lightning, moe, qlinear, recurrent, sampling, stream
 from ..ops.mxfp8 import MxTensor
-from .config import LayerRun, LayerSpec, ModelConfig, MoeSpec
+from .config import RECURRENT, LayerRun, LayerSpec, ModelConfig, MoeSpec
 from .weights import LinearWeight, ModelWeights
 from ..utils import profiler
 
@@ -120,7 +121,7 @@ class KvCache:
                 rows, heads, (dkp, dvp) = num_pages * page_size, sp.n_kv_heads, att.cache_head_dims(sp.head_dim, sp.v_dim, dt)
             kv.k.append(torch.zeros(rows, heads, dkp, dtype=dt, device=device))
             kv.v.append(torch.zeros(rows, heads, dvp, dtype=dt, device=device))
-            rec = next((x for x in spec.mixers if x.mixer in ("lightning", "mamba2", "hgrn2", "rwkv")), None)
+            rec = next((x for x in spec.mixers if x.mixer in RECURRENT), None)
             conv = next((x for x in spec.mixers if x.conv_taps), None)
             kv.rec.append(torch.zeros(n_seq_slots, rec.n_heads, rec.head_dim, rec.v_dim, **f32) if rec is not None else None)
             kv.conv.append(torch.zeros(n_seq_slots, conv.conv_taps - 1, conv.conv_channels, **f32) if conv is not None else None)
@@ -403,7 +404,7 @@ class Transformer:
         self.rope_table = ew.rope_table(min(max(cfg.max_seq_len, 4096), 65536), rd, cfg.rope_theta, weights.embed.device) \
             if weights.embed.is_cuda and not cfg.is_layered else None
         self.mixer_blocks = {"attention": self.masked_attention_block, "lightning": self.lightning_block, "mamba2": self.mamba2_block, "hgrn2": self.hgrn2_block,
-                             "latent": self.latent_block, "rwkv": self.rwkv_block}
+                             "latent": self.latent_block, "rwkv": self.rwkv_block, "mingru": self.mingru_block}
         self._branches: List = []      # streams of a captured step's branches
         self.snapshots = {}            # layer -> hidden rows captured after that layer (debug / DeepStack)
         self.snapshot_layers: Sequence[int] = ()
@@ -533,14 +534,14 @@ class Transformer:
         elif sp.qk_norm_rows:
             q = stream.qk_rows(qkv, fb.slots, lw.q_norm, lw.k_norm, kc, vc, hq, hkv, d, dv, eps, scale)
         else:
-            q = stream.qk_unit(qkv, fb.slots, kc, vc, hq, hkv, d, dv, eps, scale, unit=sp.qk_unit)
+            q = stream.qk_unit(qkv, fb.slots, kc, vc, hq, hkv, d, dv, eps, scale, unit=sp.qk_unit, positions=fb.positions, temp=(sp.temp_coef, sp.temp_every))
         key = (hq, hkv, sp.span)
         if fb.plans is None:
             fb.plans = {}
         if key not in fb.plans and q.is_cuda:
             fb.plans[key] = attention_plan(fb.q_lens, max(fb.kv_lens), *key, q.device, fb.is_decode)
         a = att.attention_masked(q, kc, vc, fb.cu_q, fb.kv_len, fb.block_table, self.kv.page_size, window=sp.window, keep_first=sp.keep_first,
-                                 bias=lw.rel_bias, plan=fb.plans.get(key), decode=fb.is_decode, softcap=sp.softcap, sink=lw.sink)
+                                 bias=lw.rel_bias, plan=fb.plans.get(key), decode=fb.is_decode, softcap=sp.softcap, sink=lw.sink, log_bias=lw.log_bias)
         if sp.out_gate:
             a = stream.sigmoid_gate(a, qkv, sp.q_dim + hkv * (d + dv), dv)
         return apply_linear_stream(lw.wo, a.reshape(a.shape[0], -1))
@@ -630,6 +631,26 @@ class Transformer:
         g = stream.token_gate(z, fb.ids, self.w.side_embed, layer * cfg.side_dim, cfg.side_dim, self.act_dtype)
         return stream.RmsPosted(apply_linear_stream(lw.side.proj, g), lw.side.norm, cfg.rms_eps)
 
+    def weighted_tail(self, li: int, lw, sp: LayerSpec, x: torch.Tensor, delta: stream.Update, hist: Optional[torch.Tensor]) -> stream.Update:
+        """The feed-forward of a layer whose results join the stream with a factor; returns the pending update with the average behind it, if there is one."""
+        eps = self.cfg.rms_eps
+        if sp.has_ffn:
+            gate = None
+            if lw.sh_dot is not None:
+                h, gate = stream.norm_gate(x, lw.ffn_norm, eps, delta, lw.sh_dot, self.act_dtype)
+            else:
+                h = stream.norm(x, lw.ffn_norm, eps, delta, out_dtype=self.act_dtype)
+            with profiler.region("ffn", "block", "ffn", li):
+                delta = stream.Update(self.ffn_parts(lw, sp, h, gate))
+        if hist is not None:
+            # every DEPTH_BLOCK places, the sums over the places so far are formed for the layers until the next time: each place is read once for all of them
+            at, n = li + 1, stream.DEPTH_BLOCK
+            if at > 1 and (at - 1) % n == 0:
+                self._depth = (at, stream.depth_base(hist, at, [self.w.layers[r.layer].depth_w for r in self.runs[li: li + n]]))
+            first, base = self._depth if at > n else (0, None)
+            delta.depth = stream.Depth(hist, at, lw.depth_w, base[at - first] if base is not None else None, first)
+        return delta
+
     def lightning_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
         """Lightning attention: projection -> SiLU + decayed recurrence -> RMSNorm over all heads * sigmoid(gate) -> output projection."""
         proj, activated = apply_linear_mixer(lw.lin.w_in, h, silu_rows=2 * sp.q_dim + sp.n_heads * sp.v_dim)
@@ -637,6 +658,13 @@ class Transformer:
                                 max(fb.q_lens) if fb.q_lens else 1)
         y = stream.gated_norm(o, proj, 2 * sp.q_dim + sp.n_heads * sp.v_dim, lw.lin.norm, self.cfg.rms_eps, self.act_dtype)
         return apply_linear_stream(lw.lin.w_out, y)
+
+    def mingru_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
+        """minGRU: projection -> recurrence per channel (gates and candidates f32) * SiLU(output gate) -> output projection."""
+        w = lw.gru
+        xg, z, col = self._mixer_rows(w.w_in, h, w.z_row)
+        y = recurrent.mingru(xg, z, col, w.x_bias, w.z_bias, self.kv.rec[li], fb.cu_q, fb.seq_slots, sp.v_dim, self.most_tokens(fb), self.act_dtype)
+        return apply_linear_stream(w.w_out, y)
 
     def mamba2_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
         """Mamba-2: projection -> causal convolution + SiLU -> recurrence -> norm of y * SiLU(z) -> output projection.  The step sizes stay f32."""
@@ -670,8 +698,8 @@ class Transformer:
         return latent.make_plan(q_lens, kv_lens, max_kv, device, decode, expand, sorted({sp.n_heads for sp in specs}))
 
     def latent_block(self, li: int, lw, sp: LayerSpec, h: torch.Tensor, fb: ForwardBatch):
-        """Latent attention: q and kv latents -> norms, cache store -> query heads -> attention over the cached latents (absorbed) or over keys and values
-        expanded from them -> output projection.  A layer with ``kv_from`` reads the cache of that layer."""
+        """Latent attention: q and kv latents -> norms, cache store -> query heads (without a q latent: part of the first projection) -> attention over the cached
+        latents (absorbed) or over keys and values expanded from them -> gate -> output projection.  A layer with ``kv_from`` reads the cache of that layer."""
         w, dt, dev = lw.latent, self.act_dtype, h.device
         hd, d, rd, r = sp.n_heads, sp.head_dim, sp.rot_dim, sp.kv_rank
         cache = self.kv.k[li if sp.kv_from < 0 else sp.kv_from]
@@ -681,8 +709,12 @@ class Transformer:
         if plan is None:
             plan = fb.plans["latent"] = self.latent_plan(fb.q_lens, fb.kv_lens, max(fb.kv_lens), dev, fb.is_decode)
         mag = sp.rotary.magnitude
-        cq = latent.latent_store(apply_linear_rows(w.w_a, h), fb.positions, fb.slots, w.q_norm, w.kv_norm, w.freq, mag, cache, sp.q_rank, r, rd, self.cfg.rms_eps, dt)
-        q = apply_linear_rows(w.w_qb, cq)
+        rows_a = apply_linear_rows(w.w_a, h)
+        cq = None
+        if sp.q_rank or w.kv_norm is not None:
+            cq = latent.latent_store(rows_a, fb.positions, fb.slots, w.q_norm, w.kv_norm, w.freq, mag, cache, sp.q_rank, r, rd, self.cfg.rms_eps, dt,
+                                     0 if sp.q_rank else w.cols["kv"])
+        q = apply_linear_rows(w.w_qb, cq) if sp.q_rank else rows_a
         dp, vp, rp = (stream.row_width(n, dt) for n in (d, sp.v_dim, rd))
         a = torch.empty(h.shape[0], hd * vp, dtype=dt, device=dev)
         qa = qn = en = er = None
@@ -708,30 +740,47 @@ class Transformer:
             rows_kv = latent.gather_latents(cache, plan, fb.block_table, self.kv.page_size)
             kvx = gemm.linear(rows_kv[:, : w.w_kv.k], w.w_kv.w, w_tiled=w.w_kv.tiled)
             latent.attend_expanded(en, er, kvx, rows_kv, r, plan, w.sink, a.view(-1, hd, vp))
+        if sp.out_gate:
+            stream.sigmoid_gate(a.view(-1, hd, vp), rows_a, w.cols["gate"], sp.v_dim)
         return apply_linear_stream(lw.wo, a)
 
     def stream_moe(self, lw, m: MoeSpec, h: torch.Tensor):
         """Mixture of experts of a layer described by ``LayerSpec``; the weighted sum stays pending for the stream's norm."""
-        rt = dict(mode=m.router, renorm=2 if m.renorm else 0, routed_scale=m.scale, groups=(m.groups, m.groups_kept, m.group_best))
+        rt = dict(mode=m.router, renorm=(2 if m.gated else 1) if m.renorm else 0, routed_scale=m.scale, groups=(m.groups, m.groups_kept, m.group_best))
         if lw.w13.fmt != "f32":
             return self.moe_local(lw, h, spec=m, rt=rt)
         ids, wts, pl = moe.route_plan(gemm.linear_f32(h, lw.router), m.top, m.n_experts, 64, **rt)
         gu = gemm.grouped_linear_f32(h, lw.w13.w.view(m.n_experts, -1, h.shape[1]), pl.seg_start, pl.seg_count, pl.capacity, pl.row_token)
-        y = gemm.grouped_linear_f32(stream.act_mul(gu, "silu"), lw.w2.w.view(m.n_experts, -1, lw.w2.k), pl.seg_start, pl.seg_count, pl.capacity)
+        y = gemm.grouped_linear_f32(stream.act_mul(gu, "silu") if m.gated else stream.gelu_rows(gu), lw.w2.w.view(m.n_experts, -1, lw.w2.k), pl.seg_start, pl.seg_count, pl.capacity)
         return moe.PendingCombine(y, pl.pair_row, wts, h.shape[0], m.top)
+
+    def plain_ffn(self, up: LinearWeight, down: LinearWeight, h: torch.Tensor):
+        """down(gelu(up(h))), the exact GELU."""
+        a = stream.gelu_rows(gemm.linear_f32(h, up.w)) if up.fmt == "f32" else gemm.linear(h, up.w, w_tiled=up.tiled, gelu=True)
+        return apply_linear_stream(down, a)
+
+    def ffn_parts(self, lw, sp: LayerSpec, h: torch.Tensor, gate: Optional[torch.Tensor]):
+        """The feed-forward's results as parts of an ``Update``: with a shared expert two of them, its own times the tokens' ``gate``."""
+        m = self.cfg.residual_mult
+        if gate is None:
+            return [(self.stream_ffn(lw, sp, h), m, None)]
+        shared = self.branch(0, h, lambda: self.plain_ffn(lw.sh_up, lw.sh_down, h))
+        y = self.stream_ffn(lw, sp, h)
+        self.join_branch(0, h)
+        return [(y, m, None), (shared, m, gate)]
 
     def stream_ffn(self, lw, sp: LayerSpec, h: torch.Tensor):
         if sp.moe is not None:
             return self.stream_moe(lw, sp.moe, h)
         gu = lw.w_gate_up
         if gu.fmt == "f32":
-            return apply_linear_stream(lw.w_down, stream.act_mul(gemm.linear_f32(h, gu.w), sp.act, sp.act_cap))
+            return apply_linear_stream(lw.w_down, stream.act_mul(gemm.linear_f32(h, gu.w, gu.bias), sp.act, sp.act_cap))
         inter = gu.n // 2
         split = gemm.pick_partials_dual(inter, h.shape[0], (gu.k + 63) // 64 * 64, False) if SPLIT_PROJ and h.is_cuda else 1
         if split > 1:
-            act = ew.silu_mul_partials(gemm.swiglu_partials(h, gu.w, split, w_tiled=gu.tiled), act=sp.act, cap=sp.act_cap)
+            act = ew.silu_mul_partials(gemm.swiglu_partials(h, gu.w, split, w_tiled=gu.tiled), act=sp.act, cap=sp.act_cap, bias=gu.bias)
         else:
-            act = gemm.linear_swiglu(h, gu.w, w_tiled=gu.tiled, act=sp.act, cap=sp.act_cap)
+            act = gemm.linear_swiglu(h, gu.w, w_tiled=gu.tiled, act=sp.act, cap=sp.act_cap, bias=gu.bias)
         return apply_linear_stream(lw.w_down, act)
 
     def shared_expert(self, lw, h: torch.Tensor) -> torch.Tensor:
@@ -776,8 +825,9 @@ class Transformer:
         t = h.shape[0]
         e, k, inter, hid = (local_range[1] if local_range else cfg.n_experts), cfg.n_experts_used, cfg.expert_ffn, cfg.hidden
         n_exp = cfg.n_experts
+        gated = True
         if spec is not None:
-            e, n_exp, k, inter, hid = spec.n_experts, spec.n_experts, spec.top, lw.w2.k, lw.w13.k
+            e, n_exp, k, inter, hid, gated = spec.n_experts, spec.n_experts, spec.top, lw.w2.k, lw.w13.k, spec.gated
         rt = rt or dict(mode=cfg.router, bias=lw.router_bias, renorm=cfg.norm_topk, routed_scale=cfg.routed_scale, local_range=local_range)
         if self.mx:
             # token tile (= scale-atom layout) by the expected rows per expert: 32 for decode-sized batches
@@ -806,7 +856,7 @@ class Transformer:
             else:
                 ids, wts, pl = moe.route_plan_hidden(h, lw.router, k, e, tn, **rt)
                 xs = moe.gather_rows(h, pl.row_token)
-            act = gemm.grouped_linear(xs, lw.w13.w.view(e, 2 * inter, hid), pl.seg_start, pl.seg_count, tn, dual=True, w_tiled=lw.w13.tiled)
+            act = gemm.grouped_linear(xs, lw.w13.w.view(e, -1, hid), pl.seg_start, pl.seg_count, tn, dual=gated, gelu=not gated, w_tiled=lw.w13.tiled)
             y = gemm.grouped_linear(act, lw.w2.w.view(e, -1, inter), pl.seg_start, pl.seg_count, tn, w_tiled=lw.w2.tiled)
         return moe.PendingCombine(y, pl.pair_row, wts, t, k)
 
@@ -822,6 +872,9 @@ class Transformer:
             x = fb.embeds if fb.embeds is not None else ew.embed(fb.ids, w.embed)
         delta = None
         first = x.clone() if any(r.again for r in self.runs) else None       # the embedding output, for later passes of a loop
+        hist = torch.empty(last_layer, *x.shape, dtype=x.dtype, device=x.device) if cfg.depth_average else None      # it, and all layers' results but the last
+        if hist is not None:
+            hist[0].copy_(x)
         self._rotary = {}
         if hasattr(self.par, "_sp_ok"):
             # the fused tensor-parallel prefill path keeps the residual stream sharded by rows between the layers' GEMMs: only for
@@ -833,23 +886,26 @@ class Transformer:
             if cfg.parallel_ffn:
                 delta = self.parallel_layer(li, lw, cfg.layer_specs[self.runs[li].layer], x, delta, first, fb)
                 if li in self.snapshot_layers:
-                    self.snapshots[li] = x + stream.whole(delta)[:, : x.shape[1]] if delta is not None else x.clone()
+                    self.snapshots[li] = stream.settled(x, delta)
                 continue
             if self.stream_f32:
                 sp, step = cfg.layer_specs[self.runs[li].layer], self.runs[li].step
                 h = stream.norm(x, lw.attn_norm, cfg.rms_eps, delta, add=w.loop_step[step] if step >= 0 else None, out_dtype=self.act_dtype)
                 with profiler.region(sp.mixer, "block", "attention", li):
                     delta = self.mixer_blocks[sp.mixer](li, lw, sp, h, fb)
-                if lw.attn_post is not None:
-                    delta = stream.PostNormed(delta, lw.attn_post)
-                if sp.has_ffn:
-                    h = stream.norm(x, lw.ffn_norm, cfg.rms_eps, delta, out_dtype=self.act_dtype)
-                    with profiler.region("ffn", "block", "ffn", li):
-                        delta = self.stream_ffn(lw, sp, h)
-                    if lw.ffn_post is not None:
-                        delta = stream.PostNormed(delta, lw.ffn_post)
+                if cfg.depth_average or cfg.residual_mult != 1.0:
+                    delta = self.weighted_tail(li, lw, sp, x, stream.Update([(delta, cfg.residual_mult, None)]), hist)
+                else:
+                    if lw.attn_post is not None:
+                        delta = stream.PostNormed(delta, lw.attn_post)
+                    if sp.has_ffn:
+                        h = stream.norm(x, lw.ffn_norm, cfg.rms_eps, delta, out_dtype=self.act_dtype)
+                        with profiler.region("ffn", "block", "ffn", li):
+                            delta = self.stream_ffn(lw, sp, h)
+                        if lw.ffn_post is not None:
+                            delta = stream.PostNormed(delta, lw.ffn_post)
                 if li in self.snapshot_layers:
-                    self.snapshots[li] = x + stream.whole(delta)[:, : x.shape[1]]
+                    self.snapshots[li] = stream.settled(x, delta)
                 continue
             lay = 32 if x.shape[0] <= 32 else 128
             par = self.par
@@ -929,7 +985,7 @@ class Transformer:
         if self._last_delta is None:
             return x
         if self.stream_f32:
-            return x + stream.whole(self._last_delta)[:, : x.shape[1]]
+            return stream.settled(x, self._last_delta)
         return (x.float() + self._last_delta.float()).to(torch.bfloat16)
 
 

@@ -266,22 +266,37 @@ class GlaWeights:
 
 @dataclass
 class LatentWeights:
-    """A latent-attention mixer.  ``w_kv`` expands cached latents to all heads' keys and values (prompts); ``w_uk`` / ``w_uv`` are the same matrices
+    """A latent-attention mixer.  ``w_a`` without a query latent: rows [q heads | kv latent | rotated key part | gate], each part starting at the column that
+    ``cols`` names (multiples of 8).  ``w_kv`` expands cached latents to all heads' keys and values (prompts); ``w_uk`` / ``w_uv`` are the same matrices
     head by head, for attention over the latents themselves (decoding)."""
     w_a: LinearWeight             # rows [q latent | kv latent | rotated key part], or [q latent] alone
-    q_norm: torch.Tensor          # f32 [q_rank]
+    q_norm: Optional[torch.Tensor]    # f32 [q_rank]
     kv_norm: Optional[torch.Tensor]   # f32 [kv_rank]
-    w_qb: LinearWeight            # [heads * (dim + rot_dim), q_rank]
+    w_qb: Optional[LinearWeight]  # [heads * (dim + rot_dim), q_rank]
     w_kv: Optional[LinearWeight]  # rows [heads * dim ; heads * v_dim], each head padded to 8 rows (bf16 only)
     w_uk: LinearWeight            # per head [rank, dim]
     w_uv: LinearWeight            # per head [v_dim, rank]
-    sink: torch.Tensor            # f32 [heads], times log2 e
+    sink: Optional[torch.Tensor]  # f32 [heads], times log2 e
     freq: torch.Tensor            # f64 [rot_dim / 2] rotary frequencies
+    cols: Optional[Dict[str, int]] = None     # first columns of "kv" and "gate"
 
     def to(self, device) -> "LatentWeights":
         mv = lambda t: t.to(device) if t is not None else None
-        return LatentWeights(self.w_a.to(device), mv(self.q_norm), mv(self.kv_norm), self.w_qb.to(device), mv(self.w_kv), self.w_uk.to(device), self.w_uv.to(device),
-                             mv(self.sink), mv(self.freq))
+        return LatentWeights(self.w_a.to(device), mv(self.q_norm), mv(self.kv_norm), mv(self.w_qb), mv(self.w_kv), self.w_uk.to(device), self.w_uv.to(device),
+                             mv(self.sink), mv(self.freq), self.cols)
+
+
+@dataclass
+class MinGruWeights:
+    """A minGRU mixer.  ``w_in`` rows: [x | output gate], padding up to ``z_row`` (a multiple of 128), [z]."""
+    w_in: LinearWeight
+    z_row: int
+    z_bias: torch.Tensor          # f32 [width]
+    x_bias: torch.Tensor          # f32 [width]
+    w_out: LinearWeight
+
+    def to(self, device) -> "MinGruWeights":
+        return MinGruWeights(self.w_in.to(device), self.z_row, self.z_bias.to(device), self.x_bias.to(device), self.w_out.to(device))
 
 
 @dataclass
@@ -344,11 +359,16 @@ class LayerWeights:
     rot_freq: Optional[torch.Tensor] = None       # f64 [dims / 2] rotary frequencies
     rwkv: Optional[RwkvWeights] = None
     side: Optional[SideWeights] = None
+    gru: Optional[MinGruWeights] = None
+    log_bias: Optional[torch.Tensor] = None       # f32 [2, heads]: r1 and r2 of the logarithmic distance bias
+    sh_up: Optional[LinearWeight] = None          # plain shared expert (its down projection is sh_down)
+    sh_dot: Optional[torch.Tensor] = None         # f32 [H]: row that gates the shared expert, times the weight of the norm in front of the feed-forward
+    depth_w: Optional[torch.Tensor] = None        # f32 [layer + 2]: weights of the embedding output and of every layer's result so far
 
     def linears(self) -> List[LinearWeight]:
         """Every projection matrix of the layer."""
-        own = [self.wqkv, self.wo, self.w_gate_up, self.w_down, self.w13, self.w2, self.sh_gate_up, self.sh_down]
-        for part in (self.ssm, self.lin, self.mamba, self.gla):
+        own = [self.wqkv, self.wo, self.w_gate_up, self.w_down, self.w13, self.w2, self.sh_gate_up, self.sh_down, self.sh_up]
+        for part in (self.ssm, self.lin, self.mamba, self.gla, self.gru):
             if part is not None:
                 own += [part.w_in, part.w_out]
         if self.rwkv is not None:
@@ -389,7 +409,7 @@ class ModelWeights:
                                router_bias=mv(l.router_bias), w13=mv(l.w13), w2=mv(l.w2), ssm=mv(l.ssm), sh_gate_up=mv(l.sh_gate_up),
                                sh_down=mv(l.sh_down), sh_gate=mv(l.sh_gate), lin=mv(l.lin), rel_bias=mv(l.rel_bias), attn_post=mv(l.attn_post),
                                ffn_post=mv(l.ffn_post), mamba=mv(l.mamba), gla=mv(l.gla), latent=mv(l.latent), sink=mv(l.sink), conv_w=mv(l.conv_w),
-                               rot_freq=mv(l.rot_freq), rwkv=mv(l.rwkv), side=mv(l.side)) for l in self.layers]
+                               rot_freq=mv(l.rot_freq), rwkv=mv(l.rwkv), side=mv(l.side), gru=mv(l.gru), log_bias=mv(l.log_bias), sh_up=mv(l.sh_up), sh_dot=mv(l.sh_dot), depth_w=mv(l.depth_w)) for l in self.layers]
         return ModelWeights(cfg=self.cfg, embed=mv(self.embed), layers=layers, final_norm=mv(self.final_norm), lm_head=mv(self.lm_head),
                             fmt=self.fmt, tp_rank=self.tp_rank, tp_size=self.tp_size, ep_rank=self.ep_rank, ep_size=self.ep_size,
                             vocab_start=self.vocab_start, loop_step=mv(self.loop_step), side_embed=mv(self.side_embed))
@@ -463,9 +483,17 @@ class RandomSource:
             return (self._randn(name, shape).float() * 50 - 3.0).to(torch.bfloat16)
         if name.endswith("rwkv_u") or name.endswith(".conv"):
             return (self._randn(name, shape).float() * 25).to(torch.bfloat16)
+        if name.endswith("depth_weights"):               # mostly the layer's own result
+            w = self._randn(name, shape).float()
+            w[-1] += 1.0
+            return w.to(torch.bfloat16)
+        if name.endswith("attn_r1") or name.endswith("attn_r2"):
+            return (self._randn(name, shape).float().abs() * 10 + 0.1).to(torch.bfloat16)
+        if name.endswith("gru_z.bias"):                  # states that hold for some ten to a hundred tokens
+            return (self._randn(name, shape).float() * 50 - 3.0).to(torch.bfloat16)
         if name.endswith("_rows.norm"):
             return torch.ones(tuple(shape), dtype=torch.bfloat16, device=self.device)
-        if name.endswith("norm.weight") and not name.endswith("lin_norm.weight") and self.cfg.norm_offset:
+        if name.endswith("norm.weight") and not name.endswith(("lin_norm.weight", "attn_kv_a_norm.weight")) and self.cfg.norm_offset:
             return torch.full(tuple(shape), 1.0 - self.cfg.norm_offset, dtype=torch.bfloat16, device=self.device)
         if name.endswith("norm.weight"):
             return torch.ones(tuple(shape), dtype=torch.bfloat16, device=self.device)
@@ -645,6 +673,17 @@ def _stack_at_128(a: torch.Tensor, b: torch.Tensor):
     return out, at
 
 
+def _stack_at_8(parts: Dict[str, Optional[torch.Tensor]]):
+    """Rows of the parts one behind the other, each starting at a multiple of 8 (zero rows in between).  Returns (stack, first row of each part)."""
+    rows, at, n = [], {}, 0
+    for name, t in parts.items():
+        if t is not None:
+            at[name] = n
+            rows += [t] + ([t.new_zeros(-t.shape[0] % 8, t.shape[1])] if t.shape[0] % 8 else [])
+            n += (t.shape[0] + 7) // 8 * 8
+    return torch.cat(rows), at
+
+
 class _LayeredBuilder:
     """Weights of a model described layer by layer.  Norm weights become f32 ``offset + w``; the factor of the logits is folded into the
     final norm's weight, the per-channel scale behind a post norm into that norm."""
@@ -697,11 +736,19 @@ class _LayeredBuilder:
 
     def latent(self, pre, sp, lw):
         h, hd, d, v, r, qr = self.h, sp.n_heads, sp.head_dim, sp.v_dim, sp.kv_rank, sp.q_rank
-        w_a = self.get(pre + "attn_q_a.weight", qr, h)
-        kv_norm = None
-        if sp.kv_from < 0:
-            w_a = torch.cat([w_a, self.get(pre + "attn_kv_a.weight", r + sp.rot_dim, h)])
-            kv_norm = self.f32(pre + "attn_kv_a_norm.weight", r)
+        order = torch.tensor(sp.rotary.pair_order())                     # pairs side by side, as the kernels rotate them
+        turn = lambda w, at: torch.cat([w[..., :at, :], w[..., at + order.to(w.device), :]], -2)
+        q_of = lambda w: turn(w.reshape(hd, d + sp.rot_dim, -1), d).reshape(w.shape)
+        kv_a = turn(self.get(pre + "attn_kv_a.weight", r + sp.rot_dim, h), r) if sp.kv_from < 0 else None
+        kv_norm = self.f32(pre + "attn_kv_a_norm.weight", r) if sp.kv_from < 0 else None
+        w_qb = cols = None
+        if qr:
+            w_a = self.get(pre + "attn_q_a.weight", qr, h)
+            w_a = torch.cat([w_a, kv_a]) if kv_a is not None else w_a
+            w_qb = self.linear(q_of(self.get(pre + "attn_q_b.weight", hd * (d + sp.rot_dim), qr)))
+        else:
+            w_a, cols = _stack_at_8({"q": q_of(self.get(pre + "attn_q_direct.weight", hd * (d + sp.rot_dim), h)), "kv": kv_a,
+                                     "gate": self.get(pre + "attn_gate.weight", hd * v, h) if sp.out_gate else None})
         uk, uv = self.get(pre + "attn_k_b.weight", hd * d, r).reshape(hd, d, r), self.get(pre + "attn_v_b.weight", hd * v, r).reshape(hd, v, r)
         w_kv, pad = None, torch.nn.functional.pad
         rows_k, v8 = r, v
@@ -711,8 +758,7 @@ class _LayeredBuilder:
             w_kv = self.linear(torch.cat([pad(uk, (0, 0, 0, d8 - d)).reshape(hd * d8, r), uv.reshape(hd * v8, r)]))
             rows_k = (r + 127) // 128 * 128          # whole 128-row tiles per head
         lw.latent = LatentWeights(
-            w_a=self.linear(w_a), q_norm=self.f32(pre + "attn_q_a_norm.weight", qr), kv_norm=kv_norm,
-            w_qb=self.linear(self.get(pre + "attn_q_b.weight", hd * (d + sp.rot_dim), qr)), w_kv=w_kv,
+            w_a=self.linear(w_a), q_norm=self.f32(pre + "attn_q_a_norm.weight", qr) if qr else None, kv_norm=kv_norm, w_qb=w_qb, w_kv=w_kv, cols=cols,
             w_uk=self.linear(pad(uk.transpose(1, 2), (0, 0, 0, rows_k - r)).reshape(hd * rows_k, d), groups=hd),
             w_uv=self.linear(uv.reshape(hd * v8, r), groups=hd),
             sink=(self.get(pre + "attn_sink", hd).double() * LOG2E).float().contiguous().to(self.dev) if sp.sink else None,
@@ -737,6 +783,8 @@ class _LayeredBuilder:
             lw.rot_freq = torch.tensor(sp.rotary.frequencies(), dtype=torch.float64, device=self.dev)
         if sp.sink:
             lw.sink = (self.get(pre + "attn_sink", sp.n_heads).double() * LOG2E).float().contiguous().to(self.dev)
+        if sp.log_bias:
+            lw.log_bias = torch.stack([self.f32(pre + "attn_r1", sp.n_heads), self.f32(pre + "attn_r2", sp.n_heads)]).contiguous()
         # the attention kernels emit heads of the cache's (padded) value width: the output projection has zero columns there
         wo = self.get(pre + "attn_output.weight", h, nv)
         dvp = cache_head_dims(sp.head_dim, sp.v_dim, torch.float32 if self.exact else torch.bfloat16)[1]
@@ -744,6 +792,12 @@ class _LayeredBuilder:
         lw.wo = self.linear(wo)
         if sp.rel_buckets:
             lw.rel_bias = distance_bias_table(self.get(pre + "attn_rel.weight", sp.rel_buckets, sp.n_heads).float().cpu(), sp.rel_max).to(self.dev)
+
+    def mingru(self, pre, sp, lw):
+        h, n = self.h, sp.v_dim
+        w_in, at = _stack_at_128(torch.cat([self.get(pre + "gru_x.weight", n, h), self.get(pre + "gru_gate.weight", n, h)]), self.get(pre + "gru_z.weight", n, h))
+        lw.gru = MinGruWeights(w_in=self.linear(w_in), z_row=at, z_bias=self.f32(pre + "gru_z.bias", n), x_bias=self.f32(pre + "gru_x.bias", n),
+                               w_out=self.linear(self.get(pre + "gru_out.weight", h, n)))
 
     def rwkv(self, pre, sp, lw):
         h, nq, nv = self.h, sp.q_dim, sp.n_heads * sp.v_dim
@@ -772,24 +826,34 @@ class _LayeredBuilder:
         wd = self.get(pre + "ffn_down.weight", h, sp.ffn)
         fp = sp.ffn if self.exact else (sp.ffn + 127) // 128 * 128       # the gate / up GEMM works on whole 128-row tiles
         pad = torch.nn.functional.pad
-        lw.w_gate_up = self.linear(torch.cat([pad(wg, (0, 0, 0, fp - sp.ffn)), pad(wu, (0, 0, 0, fp - sp.ffn))]))
-        lw.w_down = self.linear(pad(wd, (0, fp - sp.ffn)))
+        bias = down_bias = None
+        if sp.ffn_bias:
+            bias = torch.cat([pad(self.f32(pre + f"ffn_{c}.bias", sp.ffn), (0, fp - sp.ffn)) for c in ("gate", "up")]).contiguous()
+            down_bias = self.f32(pre + "ffn_down.bias", h)
+        lw.w_gate_up = self.linear(torch.cat([pad(wg, (0, 0, 0, fp - sp.ffn)), pad(wu, (0, 0, 0, fp - sp.ffn))]), bias=bias)
+        lw.w_down = self.linear(pad(wd, (0, fp - sp.ffn)), bias=down_bias)
 
     def moe_ffn(self, pre, sp, lw):
         """Expert weights with the expert width and, per expert, the rows of the down projection padded to whole 128-row tiles (bf16)."""
         h, m = self.h, sp.moe
         dt = torch.float32 if self.exact else torch.bfloat16
         up = lambda n: n if self.exact else (n + 127) // 128 * 128
-        k, ip, hp = row_width(h, dt), up(m.ffn), up(h)
+        k, ip, hp, n_in = row_width(h, dt), up(m.ffn), up(h), 2 if m.gated else 1
         lw.router = torch.nn.functional.pad(self.get(pre + "ffn_gate_inp.weight", m.n_experts, h).to(dt), (0, k - h)).contiguous().to(self.dev)
-        w13 = torch.zeros(m.n_experts, 2, ip, k, dtype=dt, device=self.dev)
+        w13 = torch.zeros(m.n_experts, n_in, ip, k, dtype=dt, device=self.dev)
         w2 = torch.zeros(m.n_experts, hp, ip, dtype=dt, device=self.dev)
         for e in range(m.n_experts):
-            w13[e, 0, : m.ffn, :h] = self.src.get_expert(pre + "ffn_gate_exps.weight", e, (m.ffn, h)).to(self.dev)
-            w13[e, 1, : m.ffn, :h] = self.src.get_expert(pre + "ffn_up_exps.weight", e, (m.ffn, h)).to(self.dev)
+            if m.gated:
+                w13[e, 0, : m.ffn, :h] = self.src.get_expert(pre + "ffn_gate_exps.weight", e, (m.ffn, h)).to(self.dev)
+            w13[e, n_in - 1, : m.ffn, :h] = self.src.get_expert(pre + "ffn_up_exps.weight", e, (m.ffn, h)).to(self.dev)
             w2[e, :h, : m.ffn] = self.src.get_expert(pre + "ffn_down_exps.weight", e, (h, m.ffn)).to(self.dev)
         lw.w13 = make_linear(w13.reshape(-1, k), self.fmt, groups=m.n_experts)
         lw.w2 = make_linear(w2.reshape(-1, ip), self.fmt, groups=m.n_experts)
+        if m.shared:
+            pad, sp_ = torch.nn.functional.pad, up(m.shared)
+            lw.sh_up = self.linear(pad(self.get(pre + "ffn_up_shexp.weight", m.shared, h), (0, 0, 0, sp_ - m.shared)))
+            lw.sh_down = self.linear(pad(self.get(pre + "ffn_down_shexp.weight", h, m.shared), (0, sp_ - m.shared)))
+            lw.sh_dot = (self.f32(pre + "ffn_gate_inp_shexp.weight", 1, h)[0] * lw.ffn_norm).contiguous()
 
     def layer(self, li: int, sp) -> LayerWeights:
         pre, post = f"blk.{li}.", self.cfg.post_norm
@@ -804,6 +868,8 @@ class _LayeredBuilder:
             self.moe_ffn(pre, sp, lw)
         if self.cfg.side_dim:
             self.side(pre, lw)
+        if self.cfg.depth_average:
+            lw.depth_w = self.f32(pre + "depth_weights", li + 2)
         return lw
 
     def model(self) -> ModelWeights:

@@ -361,7 +361,7 @@ def cache_head_dims(dk: int, dv: int, dtype: torch.dtype):
     return flash_head_dims(dk, dv) or ((dk + 7) // 8 * 8, (dv + 7) // 8 * 8)
 
 
-def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window=0, keep_first=0, bias=None, softcap=0.0, sink=None) -> torch.Tensor:
+def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window=0, keep_first=0, bias=None, softcap=0.0, sink=None, log_bias=None) -> torch.Tensor:
     t, hq, d = q.shape
     g = hq // k_cache.shape[1]
     out = torch.zeros(t, hq, v_cache.shape[2], dtype=torch.float32)
@@ -382,6 +382,9 @@ def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_si
         if bias is not None:
             n = bias.shape[1] // 2
             sc = sc + bias[:, dist.clamp(0, n - 1)]
+        if log_bias is not None:
+            r1, r2 = (r.reshape(hq, 1, 1) for r in log_bias)
+            sc = sc - r1 * torch.log2(1.0 + r2 * dist.clamp_min(0))
         see = dist >= 0
         if window > 0:
             see &= (dist < window) | (torch.arange(kl).unsqueeze(0) < keep_first)
@@ -395,16 +398,20 @@ def attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_si
 
 def attention_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, cu_q: torch.Tensor, kv_len: torch.Tensor,
                      block_table: torch.Tensor, page_size: int, window: int = 0, keep_first: int = 0, bias: Optional[torch.Tensor] = None,
-                     plan=None, decode: bool = False, softcap: float = 0.0, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                     plan=None, decode: bool = False, softcap: float = 0.0, sink: Optional[torch.Tensor] = None,
+                     log_bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Causal attention in which position i sees j <= i with ``i - j < window`` (0: no limit) or ``j < keep_first``, with an optional distance
     bias (``distance_bias_table``) added to the scores.  Key and value widths may differ (``k_cache [slots, Hkv, dk]``, ``v_cache [slots, Hkv,
     dv]``, ``q [T, Hq, dk]`` times scale * log2(e)).  ``softcap`` > 0: the scores are softcap * tanh(score / softcap), and ``q`` comes times scale /
-    softcap.  ``sink`` (f32 ``[Hq]``, times log2(e)): a score per head that joins the sum of the weights (neither goes with a bias or kept positions).  Returns ``[T, Hq, dv]`` in the cache's dtype.  ``plan``: ``(work list, KV splits)`` for
+    softcap.  ``sink`` (f32 ``[Hq]``, times log2(e)): a score per head that joins the sum of the weights (neither goes with a bias or kept positions).
+    ``log_bias`` f32 ``[2, Hq]``: r1 ln(1 + r2 (i - j)) is taken off the scores (not with another bias, a cap or a sink).  Returns ``[T, Hq, dv]`` in the cache's dtype.  ``plan``: ``(work list, KV splits)`` for
     the tcgen05 kernels; without one, or for an f32 cache or wider heads, the any-size kernel runs."""
     t, hq, dk = q.shape
     hkv, dv = k_cache.shape[1], v_cache.shape[2]
     if not q.is_cuda:
-        return attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window, keep_first, bias, softcap, sink)
+        return attention_masked_ref(q, k_cache, v_cache, cu_q, kv_len, block_table, page_size, window, keep_first, bias, softcap, sink, log_bias)
+    if log_bias is not None and (bias is not None or softcap > 0 or sink is not None):
+        raise ValueError("a logarithmic distance bias does not go with another bias, capped scores or sinks")
     if (softcap > 0 or sink is not None) and (bias is not None or keep_first):
         raise ValueError("capped scores and sinks do not go with a distance bias or kept positions")
     out = torch.empty(t, hq, dv, dtype=k_cache.dtype, device=q.device)
@@ -419,7 +426,7 @@ def attention_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
             part_lse = torch.empty(splits, t, hq, dtype=torch.float32, device=q.device)
         rc = lib.gb_flash_masked(_p(q), _p(k_cache), _p(v_cache), _p(out), _p(part_o), _p(part_lse), _p(work), _i(work.shape[0]), _p(cu_q), _p(kv_len),
                                  _p(block_table), _i(block_table.shape[1]), _i(page_size), _l(k_cache.shape[0]), _i(t), _i(hq), _i(hkv), _i(dk), _i(dv),
-                                 _i(splits), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), _f(softcap), _p(sink),
+                                 _i(splits), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), _f(softcap), _p(sink), _p(log_bias),
                                  _i(int(decode and hq // hkv <= 16)), _c(_native.status_ptr()), stream)
         _native.check(rc, "gb_flash_masked")
         if splits > 1:
@@ -427,6 +434,6 @@ def attention_masked(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         return out
     rc = lib.gb_attn_any(_p(q), _p(k_cache), _p(v_cache), _p(out), _i(int(k_cache.dtype == torch.float32)), _p(cu_q), _p(kv_len),
                          _p(block_table), _i(block_table.shape[1]), _i(page_size), _i(cu_q.numel() - 1), _l(k_cache.shape[0]), _i(t), _i(hq),
-                         _i(hkv), _i(dk), _i(dv), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), _f(softcap), _p(sink), stream)
+                         _i(hkv), _i(dk), _i(dv), _i(window), _i(keep_first), _p(bias), _i(n_bias), _i(ld_bias), _f(softcap), _p(sink), _p(log_bias), stream)
     _native.check(rc, "gb_attn_any")
     return out

@@ -266,13 +266,15 @@ def silu_mul(gate_up: torch.Tensor) -> torch.Tensor:
     return out
 
 
-def silu_mul_partials(pend, quantize: bool = False, sf_layout: int = 128, act: str = "silu", cap: float = 0.0):
+def silu_mul_partials(pend, quantize: bool = False, sf_layout: int = 128, act: str = "silu", cap: float = 0.0, bias: Optional[torch.Tensor] = None):
     """act(gate) * up (``ops.gemm.gated_act_ref``) from the K-split partial sums of ``ops.gemm.swiglu_partials`` (``pend.buf`` f32
-    ``[S, M, 2I]``): bf16 ``[M, I]``, or an ``MxTensor`` when ``quantize``."""
+    ``[S, M, 2I]``, plus ``bias`` f32 ``[2I]``): bf16 ``[M, I]``, or an ``MxTensor`` when ``quantize``."""
     s_, m, two_i = pend.buf.shape
     inter = two_i // 2
     if not pend.buf.is_cuda:
         y = pend.buf.sum(0)
+        if bias is not None:
+            y = y + bias
         from .gemm import gated_act_ref
         h = gated_act_ref(y[:, :inter], y[:, inter:], act, cap)
         return mxfp8.quantize(h, sf_layout=sf_layout) if quantize else h.to(torch.bfloat16)
@@ -285,7 +287,7 @@ def silu_mul_partials(pend, quantize: bool = False, sf_layout: int = 128, act: s
     else:
         out = torch.empty(m, inter, dtype=torch.bfloat16, device=dev)
     rc = _native.cuda().gb_silu_mul_partials(_p(pend.buf), _i(s_), _l(m * two_i), _p(out), _p(q), _p(sf), _l(m), _i(inter),
-                                             _i(1 if sf_layout == 32 else 0), _i({"silu": 0, "gelu_tanh": 1, "capped": 2}[act]), _f(cap), _s())
+                                             _i(1 if sf_layout == 32 else 0), _i({"silu": 0, "gelu_tanh": 1, "capped": 2}[act]), _f(cap), _p(bias), _s())
     _native.check(rc, "gb_silu_mul_partials")
     return MxTensor(q, sf, m, inter, sf_layout) if quantize else out
 

@@ -16,7 +16,7 @@ from .. import _native
 from . import mxfp8
 from .mxfp8 import MxTensor
 
-GEMM_MX, GEMM_DUAL, GEMM_QUANT_OUT, GEMM_OUT_F32, GEMM_W_TILED, GEMM_DUAL_RAW, GEMM_GELU, GEMM_CAPPED = 1, 2, 4, 8, 16, 32, 64, 128
+GEMM_MX, GEMM_DUAL, GEMM_QUANT_OUT, GEMM_OUT_F32, GEMM_W_TILED, GEMM_DUAL_RAW, GEMM_GELU, GEMM_CAPPED, GEMM_GELU_ERF = 1, 2, 4, 8, 16, 32, 64, 128, 256
 GATE_ACTS = ("silu", "gelu_tanh", "capped")         # activations of a gated feed-forward, by the code the kernels use
 GATE_ACT_CODE = {a: i for i, a in enumerate(GATE_ACTS)}
 
@@ -134,9 +134,9 @@ def _launch(w, x, out, n_out, k, m_tok, ldw, ldx, ldo, flags, tn, num_groups=0, 
 # --------------------------------------------------------------------------------------------- bf16
 def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None,
            out_dtype=torch.bfloat16, tn: Optional[int] = None, split_k: bool = False, w_tiled: bool = False,
-           silu_rows: int = 0) -> torch.Tensor:
+           silu_rows: int = 0, gelu: bool = False) -> torch.Tensor:
     """``x [M, K] @ w[N, K]^T`` (bf16 operands, fp32 accumulate).  ``w_tiled``: ``w`` is in ``mxfp8.tile_weight`` layout.  ``silu_rows``: SiLU on
-    that many leading output features, in the epilogue."""
+    that many leading output features, in the epilogue; ``gelu``: the exact GELU on all of them (bf16 results)."""
     m, k = x.shape
     n = w.shape[0]
     if not x.is_cuda:
@@ -145,13 +145,13 @@ def linear(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = None
             y = y + bias.float()
         if silu_rows:
             y = torch.cat([torch.nn.functional.silu(y[:, :silu_rows]), y[:, silu_rows:]], dim=1)
-        return y.to(out_dtype)
+        return (torch.nn.functional.gelu(y) if gelu else y).to(out_dtype)
     assert x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and x.stride(1) == 1 and w.stride(1) == 1
     if out is None:
         out = torch.empty(m, n, dtype=out_dtype, device=x.device)
-    flags = (GEMM_OUT_F32 if out.dtype == torch.float32 else 0) | (GEMM_W_TILED if w_tiled else 0)
+    flags = (GEMM_OUT_F32 if out.dtype == torch.float32 else 0) | (GEMM_W_TILED if w_tiled else 0) | (GEMM_GELU_ERF if gelu else 0)
     tn = tn or (max(128, pick_tn(m)) if silu_rows else pick_tn(m))
-    ex = _splitk_extras(n, m, k, tn, False, x.device, split_k) if not silu_rows else GemmExtras()
+    ex = _splitk_extras(n, m, k, tn, False, x.device, split_k) if not (silu_rows or gelu) else GemmExtras()
     if silu_rows:
         ex.silu_rows = silu_rows
     _launch(w, x, out, n, k, m, w.stride(0), x.stride(0), out.stride(0), flags, tn, bias=bias, extras=ex)
@@ -238,18 +238,21 @@ def grouped_linear_f32(x: torch.Tensor, w: torch.Tensor, seg_start: torch.Tensor
 
 
 def linear_swiglu(x: torch.Tensor, w_gate_up: torch.Tensor, out: Optional[torch.Tensor] = None,
-                  tn: Optional[int] = None, w_tiled: bool = False, act: str = "silu", cap: float = 0.0) -> torch.Tensor:
-    """``act(x @ Wg^T) * (x @ Wu^T)`` with ``w_gate_up = [Wg; Wu]`` stacked along rows ([2I, K]); ``act`` is one of ``GATE_ACTS`` (see ``gated_act_ref``)."""
+                  tn: Optional[int] = None, w_tiled: bool = False, act: str = "silu", cap: float = 0.0, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``act(x @ Wg^T) * (x @ Wu^T)`` with ``w_gate_up = [Wg; Wu]`` stacked along rows ([2I, K]); ``act`` is one of ``GATE_ACTS`` (see ``gated_act_ref``).  ``bias`` f32
+    ``[2I]``: added to both products in front of the activation ("gelu_tanh" only)."""
     m, k = x.shape
     inter = w_gate_up.shape[0] // 2
     if not x.is_cuda:
         y = x.float() @ (mxfp8.untile_weight(w_gate_up) if w_tiled else w_gate_up).float().t()
+        if bias is not None:
+            y = y + bias
         return gated_act_ref(y[:, :inter], y[:, inter:], act, cap).to(torch.bfloat16)
     if out is None:
         out = torch.empty(m, inter, dtype=torch.bfloat16, device=x.device)
     _launch(w_gate_up, x, out, inter, k, m, w_gate_up.stride(0), x.stride(0), out.stride(0),
             GEMM_DUAL | (GEMM_W_TILED if w_tiled else 0) | {"silu": 0, "gelu_tanh": GEMM_GELU, "capped": GEMM_CAPPED}[act], tn or pick_tn(m, dual=True), up_row_offset=inter,
-            extras=GemmExtras(act_cap=cap) if act == "capped" else None)
+            bias=bias, extras=GemmExtras(act_cap=cap) if act == "capped" else None)
     return out
 
 
@@ -388,27 +391,28 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, seg_start: torch.Tensor, se
                    out: Optional[torch.Tensor] = None, dual: bool = False, row_map: Optional[torch.Tensor] = None,
                    row_scale: Optional[torch.Tensor] = None, sfa=None, sfb=None, quant_out: bool = False,
                    out_sf: Optional[torch.Tensor] = None, extras=None, w_groups: Optional[int] = None,
-                   w_tiled: bool = False, pair_rows: bool = False, n_out: Optional[int] = None) -> torch.Tensor:
+                   w_tiled: bool = False, pair_rows: bool = False, n_out: Optional[int] = None, gelu: bool = False) -> torch.Tensor:
     """One GEMM per group over row segments of ``x``.
 
     ``w`` is ``[G, R, K]`` (R = 2I stacked gate/up rows when ``dual``); group g multiplies the rows
     ``seg_start[g] : seg_start[g] + seg_count[g]`` of ``x``.  ``seg_start`` entries must be multiples of
     ``min(tn, 128)``.  With ``sfa``/``sfb`` the operands are e4m3 bytes with scale atoms (MXFP8); that mode
     needs ``tn`` 32 or 128, segments aligned to ``tn`` and activation scales in the matching atom layout.
+    ``gelu``: the exact GELU of every result, in the epilogue (bf16, plain).
     """
     g, r, k = w.shape
     if w_groups is not None:
         g = w_groups                      # more row groups than weight groups (expert parallel: group = (source, expert))
     # ``pair_rows``: a tile takes row blocks n and R/2 + n of the SAME projection (two accumulators, plain stores): half the tiles
     # and token-tile loads for projections with a short K, such as the expert down projection of a decode step
-    pair = bool(pair_rows and not dual and not quant_out and row_map is None and row_scale is None and x.is_cuda and r % 256 == 0)
+    pair = bool(pair_rows and not gelu and not dual and not quant_out and row_map is None and row_scale is None and x.is_cuda and r % 256 == 0)
     n_out = r // 2 if (dual or pair) else n_out or r          # ``n_out``: leading features of each group (bf16, plain)
     mx = sfa is not None
     if not x.is_cuda:
         if w_tiled:
             w = mxfp8.untile_weight(w.reshape(-1, k)).reshape(w.shape)
-        return _grouped_reference(x, w if dual else w[:, :n_out], seg_start, seg_count, dual, row_map, row_scale, sfa, sfb, quant_out, out, out_sf)
-    flags = (GEMM_MX if mx else 0) | (GEMM_DUAL if dual else 0) | (GEMM_QUANT_OUT if quant_out else 0) | (GEMM_W_TILED if w_tiled else 0)
+        return _grouped_reference(x, w if dual else w[:, :n_out], seg_start, seg_count, dual, row_map, row_scale, sfa, sfb, quant_out, out, out_sf, gelu)
+    flags = (GEMM_GELU_ERF if gelu else 0) | (GEMM_MX if mx else 0) | (GEMM_DUAL if dual else 0) | (GEMM_QUANT_OUT if quant_out else 0) | (GEMM_W_TILED if w_tiled else 0)
     if pair:
         flags |= GEMM_DUAL | GEMM_DUAL_RAW
     if out is None:
@@ -427,7 +431,7 @@ def grouped_linear(x: torch.Tensor, w: torch.Tensor, seg_start: torch.Tensor, se
     return out
 
 
-def _grouped_reference(x, w, seg_start, seg_count, dual, row_map, row_scale, sfa, sfb, quant_out, out, out_sf=None):
+def _grouped_reference(x, w, seg_start, seg_count, dual, row_map, row_scale, sfa, sfb, quant_out, out, out_sf=None, gelu=False):
     g, r, k = w.shape
     n_out = r // 2 if dual else r
     if sfa is not None:
@@ -444,7 +448,7 @@ def _grouped_reference(x, w, seg_start, seg_count, dual, row_map, row_scale, sfa
         y = xf[s:s + c] @ wf[gi].t()
         if dual:
             y = torch.nn.functional.silu(y[:, :n_out]) * y[:, n_out:]
-        res[s:s + c] = y
+        res[s:s + c] = torch.nn.functional.gelu(y) if gelu else y
     if quant_out:
         q = mxfp8.quantize(res, sf_layout=(32 if (out_sf is not None and out_sf.shape[0] * 32 == res.shape[0]) else 128))
         if out is not None:

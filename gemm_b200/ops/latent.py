@@ -119,25 +119,28 @@ def rotate_ref(x: torch.Tensor, positions: torch.Tensor, freq: torch.Tensor, mag
     return torch.stack([u * c - v * s, v * c + u * s], dim=-1).reshape(x.shape)
 
 
-def latent_store(rows, positions, slots, q_norm, kv_norm, freq, mag: float, cache: torch.Tensor, q_rank: int, rank: int, rot_dim: int, eps: float, dtype) -> torch.Tensor:
-    """Projection rows ``[q latent | kv latent | rotated key part]`` -> normalised q latents ``[T, row_width(q_rank)]``; the normalised kv latent and the
-    rotated key part go to cache slot ``slots[t]`` (``kv_norm`` None: the rows hold a q latent only)."""
+def latent_store(rows, positions, slots, q_norm, kv_norm, freq, mag: float, cache: torch.Tensor, q_rank: int, rank: int, rot_dim: int, eps: float, dtype,
+                 col: int = 0) -> Optional[torch.Tensor]:
+    """Projection rows ``[q latent | kv latent | rotated key part]`` (from column ``col`` on) -> normalised q latents ``[T, row_width(q_rank)]``; the normalised kv
+    latent and the rotated key part go to cache slot ``slots[t]``.  ``kv_norm`` None: the rows hold a q latent only; ``q_rank`` 0: they hold none."""
     base, f32, parts, stride, ld = split_rows(rows)
     t = rows.rows if hasattr(rows, "buf") else rows.shape[0]
     ldq = row_width(q_rank, dtype)
     if not base.is_cuda:
-        y = whole(rows)
+        y = whole(rows)[:, col:]
         n = lambda z: z / torch.sqrt(z.pow(2).mean(-1, keepdim=True) + eps)
-        out = torch.zeros(t, ldq, dtype=dtype)
-        out[:, :q_rank] = (n(y[:, :q_rank]) * q_norm).to(dtype)
+        out = None
+        if q_rank:
+            out = torch.zeros(t, ldq, dtype=dtype)
+            out[:, :q_rank] = (n(y[:, :q_rank]) * q_norm).to(dtype)
         if kv_norm is not None:
             c = n(y[:, q_rank: q_rank + rank]) * kv_norm
             r = rotate_ref(y[:, q_rank + rank: q_rank + rank + rot_dim], positions, freq, mag)
             ok = slots >= 0
             cache[slots[ok].long(), 0, : rank + rot_dim] = torch.cat([c, r], -1)[ok].to(cache.dtype)
         return out
-    out = torch.empty(t, ldq, dtype=dtype, device=base.device)
-    rc = _native.cuda().gb_latent_store(_p(base), _i(f32), _i(parts), _l(stride), _i(ld), _p(positions), _p(slots), _p(q_norm), _p(kv_norm), _p(freq), _f(mag), _p(out),
+    out = torch.empty(t, ldq, dtype=dtype, device=base.device) if q_rank else None
+    rc = _native.cuda().gb_latent_store(_c(base.data_ptr() + col * base.element_size()), _i(f32), _i(parts), _l(stride), _i(ld), _p(positions), _p(slots), _p(q_norm), _p(kv_norm), _p(freq), _f(mag), _p(out),
                                         _i(ldq), _p(cache), _i(int(dtype == torch.float32)), _l(cache.shape[0]), _i(cache.shape[2]), _i(t), _i(q_rank), _i(rank),
                                         _i(rot_dim), _f(eps), _s())
     _native.check(rc, "gb_latent_store")

@@ -4,6 +4,7 @@
 ``ssd``          Mamba-2:  S_t = exp(a dt_t) S_{t-1} + dt_t B_t x_t^T,  y_t = S_t^T C_t + D x_t
 ``gla``          HGRN2:    S_t = diag(f_t) S_{t-1} + (1 - f_t) v_t^T,  o_t = S_t^T q_t
 ``rwkv``         RWKV:     o_t = (S_{t-1} + diag(u) k_t v_t^T)^T r_t,  S_t = diag(w_t) S_{t-1} + k_t v_t^T,  w = exp(-exp(z))
+``mingru``       s_t = (1 - z_t) s_{t-1} + z_t c_t per channel, the gate z and the candidate c from the current token alone
 ``token_shift``  mixes of a token's row and the one before it, for the projections of ``rwkv``
 
 State tensors: ``conv_state`` f32 ``[slots, taps - 1, channels]`` (oldest row first), ``state`` f32 ``[slots, heads, dim, vdim]``; one slot per
@@ -166,6 +167,39 @@ def gla(qv, gate, gate_col: int, f_bias: torch.Tensor, lower: torch.Tensor, stat
                                           _c(0), _p(state), _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(nv), _i(heads), _i(1), _i(dim), _i(vdim),
                                           _i(int(not activated)), _i(cu_q.numel() - 1), _s())
     _native.check(rc, "gb_recurrent_step")
+    return out
+
+
+def mingru_ref(x, g, z, x_bias, z_bias, state, cu_q, seq_slots, out_dtype):
+    t, n = x.shape
+    u, z = x + x_bias, z + z_bias
+    keep, cand = torch.sigmoid(-z), torch.sigmoid(z) * torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
+    out, cu = torch.zeros(t, row_width(n, out_dtype), dtype=out_dtype), cu_q.tolist()
+    for s in range(len(cu) - 1):
+        st = state[int(seq_slots[s])].reshape(-1) if cu[s + 1] > cu[s] else None
+        for i in range(cu[s], cu[s + 1]):
+            st.mul_(keep[i]).add_(cand[i])
+            out[i, :n] = (st * F.silu(g[i])).to(out_dtype)
+    return out
+
+
+def mingru(xg, z, z_col: int, x_bias: torch.Tensor, z_bias: torch.Tensor, state: torch.Tensor, cu_q: torch.Tensor, seq_slots: torch.Tensor, n: int, max_tokens: int = 1,
+           out_dtype=torch.bfloat16) -> torch.Tensor:
+    """``xg``: projection result with columns ``[x | output gate]``, ``n`` each; ``z``: projection result (f32 or partial sums) whose columns ``z_col ...`` are the
+    gate's logits.  With u = x + x_bias the candidate is u + 1/2 (u >= 0) or sigmoid(u); ``state`` f32 ``[slots, 1, 1, n]``.  Returns the rows
+    ``s_t * silu(output gate)``, ``[T, row_width(n)]``."""
+    zb, zf32, zparts, zstride, zld = split_rows(z)
+    if not zb.is_cuda:
+        y = whole(xg)
+        return mingru_ref(y[:, :n], y[:, n: 2 * n], whole(z)[:, z_col: z_col + n], x_bias, z_bias, state, cu_q, seq_slots, out_dtype)
+    base, f32, parts, stride, ld = split_rows(xg)
+    t = _n_rows(xg)
+    assert zf32 and state.is_contiguous() and state.dtype == torch.float32
+    out = torch.empty(t, row_width(n, out_dtype), dtype=out_dtype, device=base.device)
+    rc = _native.cuda().gb_mingru(_p(base), _i(f32), _i(parts), _l(stride), _i(ld), _at(zb, z_col), _i(zparts), _l(zstride), _i(zld), _p(x_bias), _p(z_bias), _p(state),
+                                  _i(state.shape[0]), _p(cu_q), _p(seq_slots), _p(out), _i(int(out_dtype == torch.float32)), _i(out.shape[1]), _i(n), _i(max_tokens),
+                                  _i(cu_q.numel() - 1), _i(int(CHUNKED and max_tokens >= CHUNKED_MIN_TOKENS)), _s())
+    _native.check(rc, "gb_mingru")
     return out
 
 

@@ -12,11 +12,13 @@
 ``gated_norm``   RMSNorm over all heads' outputs times sigmoid(gate)
 ``part_norm``    RMSNorm of equal parts of a row, after (or before) multiplying by SiLU(gate) if there is one
 ``act_mul``      act(gate) * up of f32 rows
+``gelu_rows``    the exact GELU of f32 rows
 
 The rows that feed a projection have the width ``row_width(n, dtype)``: bf16 rows are padded with zeros to a multiple of 8 elements
 (the 16-byte row pitch of a TMA tile); f32 rows are not padded.  A projection's result comes in as a tensor (bf16 or f32) or as
 ``ops.gemm.PendingPartials`` (K-split fp32 partial sums, added here in split order); the stream's update may also be ``ops.moe.PendingCombine``
-(expert outputs whose weighted sum is formed here).
+(expert outputs whose weighted sum is formed here).  ``Update`` is a sum of results with factors, some times a number per token, and may end in an average
+over the stream at earlier places (``Depth``).
 """
 from __future__ import annotations
 
@@ -79,6 +81,56 @@ class RmsPosted:
     delta: object
     weight: torch.Tensor
     eps: float
+
+
+@dataclass
+class Depth:
+    """Average behind an update: the stream with the update is kept as row block ``at`` of ``hist`` (f32 ``[places, T, W]``), and goes on as the sum of
+    ``weights[j] * hist[j]`` over the places up to it (``weights`` f32 ``[at + 1]``).  ``base`` f32 ``[T, W]``: that sum over the places below ``first``."""
+    hist: torch.Tensor
+    at: int
+    weights: torch.Tensor
+    base: Optional[torch.Tensor] = None
+    first: int = 0
+
+
+DEPTH_BLOCK = 8
+
+
+def depth_base(hist: torch.Tensor, places: int, weights: List[torch.Tensor]) -> torch.Tensor:
+    """f32 ``[K, T, W]``: for each of the K (at most ``DEPTH_BLOCK``) coming averages the sum of ``weights[k][j] * hist[j]`` over the ``places`` kept so far."""
+    if not hist.is_cuda:
+        return torch.stack([sum(hist[j] * w[j] for j in range(places)) for w in weights])
+    assert hist.is_contiguous() and len(weights) <= DEPTH_BLOCK and all(w.numel() >= places for w in weights)
+    out = torch.empty(len(weights), *hist.shape[1:], dtype=torch.float32, device=hist.device)
+    ptr = (ctypes.c_void_p * len(weights))(*(w.data_ptr() for w in weights))
+    _native.check(_native.cuda().gb_depth_base(_p(hist), _l(hist.stride(0)), _i(places), ptr, _i(len(weights)), _p(out), _l(hist[0].numel()), _s()), "gb_depth_base")
+    return out
+
+
+@dataclass
+class Update:
+    """``parts``: (result, factor, number per token or None); at most three."""
+    parts: List[Tuple[object, float, Optional[torch.Tensor]]]
+    depth: Optional[Depth] = None
+
+
+def settled(x: torch.Tensor, delta) -> torch.Tensor:
+    """The stream with a pending update, as a new tensor (captured layers, CPU references)."""
+    w = x.shape[1]
+    if delta is None:
+        return x.clone()
+    if not isinstance(delta, Update):
+        return x + whole(delta)[:, :w]
+    y = x.clone()
+    for d, f, g in delta.parts:
+        y += whole(d)[:, :w] * (f if g is None else f * g.unsqueeze(1))
+    if delta.depth is not None:
+        d = delta.depth
+        y = y * d.weights[d.at] + sum(d.hist[j] * d.weights[j] for j in range(d.first, d.at))
+        if d.base is not None:
+            y = y + d.base
+    return y
 
 
 def whole(y) -> torch.Tensor:
@@ -146,29 +198,36 @@ def norm2(x: torch.Tensor, weight: torch.Tensor, eps: float, delta: Optional[Rms
 class _JoinPart(ctypes.Structure):
     """``struct JoinPart`` of csrc/kernels/stream_ops.cu."""
     _fields_ = [("p", ctypes.c_void_p), ("pair_row", ctypes.c_void_p), ("weights", ctypes.c_void_p), ("stride", ctypes.c_long), ("f32", ctypes.c_int),
-                ("n_part", ctypes.c_int), ("ld", ctypes.c_int), ("k", ctypes.c_int), ("scale", ctypes.c_float)]
+                ("n_part", ctypes.c_int), ("ld", ctypes.c_int), ("k", ctypes.c_int), ("scale", ctypes.c_float), ("row_scale", ctypes.c_void_p)]
 
 
-def join(x: torch.Tensor, parts: List[Tuple[object, float]], out_dtype=None) -> Optional[torch.Tensor]:
-    """``x += sum of factor * result`` in place (at most three (result, factor) pairs: tensors, partial sums or pending expert sums); returns the new rows in
-    ``out_dtype`` (None: nothing), of width ``row_width(W)``."""
-    t, w = x.shape
-    if not x.is_cuda:
-        x.add_(sum(whole(d)[:, :w] * f for d, f in parts))
-        if out_dtype is None:
-            return None
-        o = torch.zeros(t, row_width(w, out_dtype), dtype=out_dtype)
-        o[:, :w] = x.to(out_dtype)
-        return o
+def _join_parts(parts):
     arr = (_JoinPart * 3)()
-    for a, (d, f) in zip(arr, parts):
+    for a, (d, f, g) in zip(arr, parts):
         a.scale = f
+        a.row_scale = g.data_ptr() if g is not None else None
         if hasattr(d, "pair_row"):
             a.p, a.f32, a.n_part, a.ld = d.y.data_ptr(), int(d.y.dtype == torch.float32), 1, d.y.stride(0)
             a.pair_row, a.weights, a.k = d.pair_row.data_ptr(), d.weights.data_ptr(), d.k
         else:
             base, a.f32, a.n_part, a.stride, a.ld = split_rows(d)
             a.p = base.data_ptr()
+    return arr
+
+
+def join(x: torch.Tensor, parts: List[Tuple], out_dtype=None) -> Optional[torch.Tensor]:
+    """``x += sum of factor * result`` in place (at most three (result, factor) pairs, or (result, factor, f32 number per token or None): tensors, partial sums
+    or pending expert sums); returns the new rows in ``out_dtype`` (None: nothing), of width ``row_width(W)``."""
+    t, w = x.shape
+    parts = [p if len(p) == 3 else (*p, None) for p in parts]
+    if not x.is_cuda:
+        x.copy_(settled(x, Update(parts)))
+        if out_dtype is None:
+            return None
+        o = torch.zeros(t, row_width(w, out_dtype), dtype=out_dtype)
+        o[:, :w] = x.to(out_dtype)
+        return o
+    arr = _join_parts(parts)
     out = torch.empty(t, row_width(w, out_dtype), dtype=out_dtype, device=x.device) if out_dtype is not None else None
     rc = _native.cuda().gb_stream_join(_p(x), ctypes.byref(arr), _i(len(parts)), _p(out), _i(int(out_dtype == torch.float32)), _i(out.shape[1] if out is not None else 0), _i(t),
                                        _i(w), _s())
@@ -176,19 +235,61 @@ def join(x: torch.Tensor, parts: List[Tuple[object, float]], out_dtype=None) -> 
     return out
 
 
+def depth_norm(x: torch.Tensor, weight: Optional[torch.Tensor], eps: float, delta: Update, rows: Optional[torch.Tensor] = None, out_dtype=torch.bfloat16) -> Optional[torch.Tensor]:
+    """``norm`` for an update that ends in an average (``Depth``): the stream with the update goes to its place in ``hist``, the average becomes the stream."""
+    d = delta.depth
+    t, w = x.shape
+    n = t if rows is None else rows.numel()
+    if not x.is_cuda:
+        y = settled(x, delta)
+        if rows is None:
+            d.hist[d.at] = settled(x, Update(delta.parts))
+            x.copy_(y)
+        else:
+            y = y[rows]
+        if weight is None:
+            return None
+        o = torch.zeros(n, row_width(w, out_dtype), dtype=out_dtype)
+        o[:, :w] = (y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps) * weight).to(out_dtype)
+        return o
+    assert d.hist.is_contiguous() and d.hist.shape[1:] == x.shape and d.at < d.hist.shape[0] + int(rows is not None) and d.weights.numel() == d.at + 1
+    out = torch.empty(n, row_width(w, out_dtype), dtype=out_dtype, device=x.device) if weight is not None else None
+    rc = _native.cuda().gb_stream_depth(_p(x), ctypes.byref(_join_parts(delta.parts)), _i(len(delta.parts)), _p(d.hist), _l(d.hist.stride(0)), _p(d.base), _i(d.first), _i(d.at), _p(d.weights), _p(weight),
+                                        _p(rows), _p(out), _i(int(out_dtype == torch.float32)), _i(out.shape[1] if out is not None else 0), _i(n), _i(w), _f(eps), _s())
+    _native.check(rc, "gb_stream_depth")
+    return out
+
+
+def norm_gate(x: torch.Tensor, weight: torch.Tensor, eps: float, delta, dot: torch.Tensor, out_dtype=torch.bfloat16) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``norm``, and for every token the sigmoid of the product of its normalised row with one more row: ``dot`` f32 ``[W]`` is that row times ``weight``."""
+    gate = torch.empty(x.shape[0], dtype=torch.float32, device=x.device)
+    return norm(x, weight, eps, delta, out_dtype=out_dtype, dot=dot, gate=gate), gate
+
+
 def norm(x: torch.Tensor, weight, eps: float, delta=None, add: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
-         out_dtype=torch.bfloat16) -> Optional[torch.Tensor]:
+         out_dtype=torch.bfloat16, dot: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
     """``x += delta + add`` in place (``x`` f32 ``[T, W]``; both optional), then ``x / rms(x) * weight`` (f32 ``[W]``), or ``weight(x)`` if it is a
     ``DynTanh``, as ``out_dtype`` rows of width ``row_width(W)``.  With ``rows`` (int64): only those stream rows are normalised, and the stream is left as it is.  ``weight``
     None: only the update."""
     if isinstance(delta, RmsPosted):
         return norm2(x, weight, eps, delta, add, rows, out_dtype=out_dtype)[0]
+    factor = 1.0
+    if isinstance(delta, Update):
+        if delta.depth is not None:
+            assert add is None and dot is None
+            return depth_norm(x, weight, eps, delta, rows, out_dtype)
+        (d, f, g), *more = delta.parts
+        if more or g is not None or hasattr(d, "pair_row"):
+            join(x, delta.parts)
+            delta = None
+        else:
+            delta, factor = d, f
     t, w = x.shape
     n = t if rows is None else rows.numel()
     if not x.is_cuda:
         y = x
         if delta is not None:
-            y = y + whole(delta)[:, :w]
+            y = y + (whole(delta)[:, :w] * factor if factor != 1.0 else whole(delta)[:, :w])
         if add is not None:
             y = y + add
         if rows is None:
@@ -199,10 +300,12 @@ def norm(x: torch.Tensor, weight, eps: float, delta=None, add: Optional[torch.Te
             return None
         o = torch.zeros(n, row_width(w, out_dtype), dtype=out_dtype)
         o[:, :w] = (weight(y) if isinstance(weight, DynTanh) else y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps) * weight).to(out_dtype)
+        if dot is not None:
+            gate.copy_(torch.sigmoid((y / torch.sqrt(y.pow(2).mean(-1, keepdim=True) + eps) * dot).sum(-1)))
         return o
     out = torch.empty(n, row_width(w, out_dtype), dtype=out_dtype, device=x.device) if weight is not None else None
     if isinstance(weight, DynTanh) or isinstance(delta, PostNormed):
-        assert add is None and (weight is None or isinstance(weight, DynTanh))
+        assert add is None and dot is None and factor == 1.0 and (weight is None or isinstance(weight, DynTanh))
         post, d = (delta.post, delta.delta) if isinstance(delta, PostNormed) else (None, delta)
         moe = hasattr(d, "pair_row")
         base, f32, parts, stride, ld = (d.y, int(d.y.dtype == torch.float32), 1, 0, d.y.stride(0)) if moe else split_rows(d) if d is not None else (None, 0, 1, 0, w)
@@ -213,17 +316,18 @@ def norm(x: torch.Tensor, weight, eps: float, delta=None, add: Optional[torch.Te
         _native.check(rc, "gb_stream_dyt")
         return out
     base, f32, parts, stride, ld = split_rows(delta) if delta is not None else (None, 0, 1, 0, w)
-    rc = _native.cuda().gb_stream_norm(_p(x), _p(base), _i(f32), _i(parts), _l(stride), _i(ld), _p(add), _p(weight), _p(rows), _p(out),
+    rc = _native.cuda().gb_stream_norm(_p(x), _p(base), _i(f32), _i(parts), _l(stride), _i(ld), _f(factor), _p(add), _p(weight), _p(dot), _p(gate), _p(rows), _p(out),
                                        _i(int(out_dtype == torch.float32)), _i(out.shape[1] if out is not None else 0), _i(n), _i(w), _f(eps), _s())
     _native.check(rc, "gb_stream_norm")
     return out
 
 
 def qk_unit(qkv, slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, hq: int, hkv: int, dk: int, dv: int, eps: float, q_scale: float,
-            unit: bool = True) -> torch.Tensor:
+            unit: bool = True, positions: Optional[torch.Tensor] = None, temp: Tuple[float, float] = (0.0, 1.0)) -> torch.Tensor:
     """Rows ``[Q heads | K heads | V heads]`` -> ``q [T, hq, dkp]`` (times ``q_scale``) in the cache's dtype; K / V of token ``t`` go to cache slot
     ``slots[t]`` (-1: not stored).  ``k_cache [slots, hkv, dkp]`` and ``v_cache [slots, hkv, dvp]`` may be wider than the heads (zero padding).
-    ``unit``: Q and K are divided by their root mean square over the head."""
+    ``unit``: Q and K are divided by their root mean square over the head.  ``temp`` = (coef, every), with a coefficient: Q at position p is also multiplied by
+    1 + coef ln(floor((p + 1) / every) + 1)."""
     base, f32, parts, stride, ld = split_rows(qkv)
     t = qkv.rows if hasattr(qkv, "buf") else qkv.shape[0]
     dkp, dvp = k_cache.shape[2], v_cache.shape[2]
@@ -233,6 +337,8 @@ def qk_unit(qkv, slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
         if unit:
             q = q / torch.sqrt(q.pow(2).mean(-1, keepdim=True) + eps)
             k = k / torch.sqrt(k.pow(2).mean(-1, keepdim=True) + eps)
+        if temp[0]:
+            q = q * (1.0 + temp[0] * torch.log(torch.floor((positions.double() + 1) / temp[1]) + 1)).float().reshape(t, 1, 1)
         pad = torch.nn.functional.pad
         ok = slots >= 0
         k_cache[slots[ok].long()] = pad(k, (0, dkp - dk))[ok].to(k_cache.dtype)
@@ -241,7 +347,7 @@ def qk_unit(qkv, slots: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     q = torch.empty(t, hq, dkp, dtype=k_cache.dtype, device=base.device)
     rc = _native.cuda().gb_qk_unit_store(_p(base), _i(f32), _i(parts), _l(stride), _i(ld), _p(slots), _p(q), _p(k_cache), _p(v_cache),
                                          _i(int(k_cache.dtype == torch.float32)), _l(k_cache.shape[0]), _i(t), _i(hq), _i(hkv), _i(dk), _i(dv), _i(dkp),
-                                         _i(dvp), _f(eps), _f(q_scale), _i(int(unit)), _s())
+                                         _i(dvp), _f(eps), _f(q_scale), _i(int(unit)), _p(positions if temp[0] else None), _f(temp[0]), ctypes.c_double(temp[1]), _s())
     _native.check(rc, "gb_qk_unit_store")
     return q
 
@@ -385,6 +491,16 @@ def part_norm(o: torch.Tensor, weight: torch.Tensor, parts: int, eps: float, gat
     rc = _native.cuda().gb_part_norm(_p(o), _i(o.stride(0)), g, _i(f32), _i(np_), _l(stride), _i(ld), _p(weight), _i(weight.numel()), _p(out),
                                      _i(int(out_dtype == torch.float32)), _i(ldo), _i(t), _i(n), _i(parts), _f(eps), _i(int(gate_after)), _s())
     _native.check(rc, "gb_part_norm")
+    return out
+
+
+def gelu_rows(x: torch.Tensor) -> torch.Tensor:
+    """The exact GELU, ``x (1 + erf(x / sqrt 2)) / 2``, of contiguous f32 rows."""
+    if not x.is_cuda:
+        return torch.nn.functional.gelu(x)
+    assert x.is_contiguous() and x.dtype == torch.float32
+    out = torch.empty_like(x)
+    _native.check(_native.cuda().gb_gelu_f32(_p(x), _p(out), _l(x.numel()), _s()), "gb_gelu_f32")
     return out
 
 
