@@ -53,7 +53,7 @@ def parse_args():
                          "batch replicated (dense models); tp+ep = attention sharded by heads and experts spread over the same ranks, "
                          "batch replicated (the layout of the largest MoE models, e.g. --model qwen3-235b-a22b); auto picks by model")
     ap.add_argument("--moe-path", default="fused", choices=["fused", "nccl"], help="multi-GPU expert exchange: fused peer-memory kernels or the NCCL baseline")
-    ap.add_argument("--design", default="", choices=["", "zogavik", "famepel", "fidolix"],
+    ap.add_argument("--design", default="", choices=["", "zogavik", "famepel", "fidolix", "zedirax"],
                     help="instead of the default workload: prefill and decode throughput of a model described layer by layer, at several sizes, beside the "
                          "closest other model at equal size (random weights, bf16, one GPU); one JSON line per measurement")
     return ap.parse_args()
@@ -310,6 +310,8 @@ def design_arm(args):
         models = [("famepel-30b-a3b", get_config("famepel-30b-a3b")), ("qwen35moe-hybrid, 45 layers of the same sizes", hybrid_moe(45))]
     elif args.design == "fidolix":
         models = [(n, get_config(n)) for n in ("fidolix-30b-a3b", "famepel-30b-a3b")]
+    elif args.design == "zedirax":
+        models = [(n, get_config(n)) for n in ("zedirax-30b-a3b", "famepel-30b-a3b")]
     else:
         models = [("zogavik-8b", get_config("zogavik-8b")), ("qwen35-hybrid, 36 layers of the same sizes", hybrid(36)), ("zogavik-4b-loop2", get_config("zogavik-4b-loop2"))]
     sampler = ClockSampler(0)

@@ -4,12 +4,6 @@
 
 namespace gb {
 
-__device__ __forceinline__ float fast_exp2(float x) {
-  float y;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-
 // tanh(x), absolute error below 3e-7: 1 - 2 / (1 + e^2x).
 __device__ __forceinline__ float tanh_wide(float x) {
   return 1.0f - __fdividef(2.0f, 1.0f + fast_exp2(2.885390081777927f * x));

@@ -156,7 +156,18 @@ __device__ __forceinline__ int e8m0_from_amax(float amax) {
   return amax == 0.0f ? 127 : max(1, min(e, 254));   // an all-zero block gets scale 1
 }
 
-__device__ __forceinline__ float gelu_erf(float x) { return 0.5f * x * (1.0f + erff(x * 0.70710678118654752f)); }
+// x (1 + erf(x / sqrt 2)) / 2 with erf(y) = 1 - (a1 t + ... + a5 t^5) exp(-y^2), t = 1 / (1 + p y), y >= 0 (Abramowitz and Stegun, Handbook of Mathematical
+// Functions, 7.1.26; |error| <= 1.5e-7); the negative side is x (1 - erf) / 2, without cancellation.
+__device__ __forceinline__ float gelu_erf(float x) {
+  constexpr float kRoot = 0.70710678118654752f;
+  const float t = fast_rcp(fmaf(0.3275911f * kRoot, fabsf(x), 1.0f));
+  float p = fmaf(0.5f * 1.061405429f, t, 0.5f * -1.453152027f);
+  p = fmaf(p, t, 0.5f * 1.421413741f);
+  p = fmaf(p, t, 0.5f * -0.284496736f);
+  p = fmaf(p, t, 0.5f * 0.254829592f);
+  const float w = x * (p * t * fast_exp2(x * x * -0.72134752044448170f));      // x (1 - erf(|x| / sqrt 2)) / 2
+  return x >= 0.f ? x - w : w;
+}
 
 // ACT, DUAL: the gate's activation (gated), 3 = the tanh form of GELU with a bias on either product; plain: 1 = SiLU on the output features below args.silu_rows, 2 = bf16
 // rows scattered by args.row_map, 3 = the exact GELU on every feature.
@@ -652,7 +663,19 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ 
               }
             continue;
           }
-          if (c + 16 <= t.valid) {
+          if constexpr (DUAL || ACT != 0) {              // the activations of all sixteen first, then the stores
+            float v[16];
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = value(r0[j], r1[j]);
+            const int n_live = min(16, t.valid - c);
+            if (args.out_f32) {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) if (j < n_live) o32[(size_t)(c + j) * args.ldo] = v[j];
+            } else {
+#pragma unroll
+              for (int j = 0; j < 16; ++j) if (j < n_live) o16[(size_t)(c + j) * args.ldo] = __float2bfloat16(v[j]);
+            }
+          } else if (c + 16 <= t.valid) {
 #pragma unroll
             for (int j = 0; j < 16; ++j) {
               const float v = value(r0[j], r1[j]);

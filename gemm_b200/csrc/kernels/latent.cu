@@ -30,14 +30,14 @@ struct LatentStoreArgs {
   int q_rank, rank, rot_dim; float eps;
 };
 
-constexpr int kLatKeep = 8;                                    // values per thread kept in registers (ranks up to 256 * kLatKeep)
+constexpr int kLatKeep = 8;                                    // values per thread kept in registers (ranks up to threads * kLatKeep)
 
-template <typename TI, typename TO, int V>                     // V columns at a time
-__global__ void __launch_bounds__(256)
+template <typename TI, typename TO, int V, int NT>             // V columns at a time, NT threads per token
+__global__ void __launch_bounds__(NT)
 latent_store_kernel(const LatentStoreArgs a) {
   pdl_wait();
   pdl_trigger();
-  __shared__ float red[2][8];
+  __shared__ float red[2][NT / 32];
   constexpr int N = kLatKeep / V;
   const int t = blockIdx.x, tid = threadIdx.x, warp = tid >> 5;
   const TI* src = (const TI*)a.a + (size_t)t * a.ld;
@@ -55,7 +55,7 @@ latent_store_kernel(const LatentStoreArgs a) {
   float q[N][V], k[N][V], sq = 0.f, sk = 0.f;
 #pragma unroll
   for (int i = 0; i < N; ++i) {
-    const int c = (tid + i * 256) * V;
+    const int c = (tid + i * NT) * V;
 #pragma unroll
     for (int x = 0; x < V; ++x) q[i][x] = k[i][x] = 0.f;
     if (c < a.q_rank) values(c, q[i]);
@@ -67,7 +67,7 @@ latent_store_kernel(const LatentStoreArgs a) {
   if ((tid & 31) == 0) { red[0][warp] = sq; red[1][warp] = sk; }
   TO* co = (TO*)a.cache + (size_t)(kv ? slot : 0) * a.ld_c;
   if (kv) {
-    for (int i = 255 - tid; i < a.rot_dim / 2; i += 256) {     // (the last warps: the first hold the ends of the ranks)
+    for (int i = NT - 1 - tid; i < a.rot_dim / 2; i += NT) {     // (the last warps: the first hold the ends of the ranks)
       float c, s, u = 0.f, v = 0.f;
       rotation(a.positions[t], a.freq[i], a.mag, c, s);
       const TI* p0 = src + a.q_rank + a.rank + 2 * i;
@@ -75,17 +75,17 @@ latent_store_kernel(const LatentStoreArgs a) {
       stv(co + a.rank + 2 * i, u * c - v * s);
       stv(co + a.rank + 2 * i + 1, v * c + u * s);
     }
-    for (int c = a.rank + a.rot_dim + tid; c < a.ld_c; c += 256) stv(co + c, 0.f);
+    for (int c = a.rank + a.rot_dim + tid; c < a.ld_c; c += NT) stv(co + c, 0.f);
   }
   __syncthreads();
   sq = sk = 0.f;
 #pragma unroll
-  for (int i = 0; i < 8; ++i) { sq += red[0][i]; sk += red[1][i]; }
+  for (int i = 0; i < NT / 32; ++i) { sq += red[0][i]; sk += red[1][i]; }
   const float iq = a.q_rank > 0 ? 1.0f / sqrtf(sq / (float)a.q_rank + a.eps) : 0.f, ik = 1.0f / sqrtf(sk / (float)a.rank + a.eps);
   TO* qo = (TO*)a.q_out + (size_t)t * a.ld_q;
 #pragma unroll
   for (int i = 0; i < N; ++i) {
-    const int c = (tid + i * 256) * V;
+    const int c = (tid + i * NT) * V;
     if (c < a.ld_q) {                                          // zero behind q_rank
       float w[V];
 #pragma unroll
@@ -191,7 +191,11 @@ GB_API int gb_latent_store(const void* rows, int in_f32, int n_part, long part_s
   const bool vec = q_rank % 4 == 0 && rank % 4 == 0 && ld % 4 == 0 && part_stride % 4 == 0 && ld_q % 4 == 0 && ld_c % 4 == 0 && al(rows, ei) && al(q_out, eo) && al(cache, eo) &&
                    al(q_norm, 16) && al(kv_norm, 16);
   if (!in_f32 && out_f32) return fail("latent_store: a 32-bit cache takes 32-bit rows%s");
-#define GB_LAT(TI, TO) (vec ? launch_k(latent_store_kernel<TI, TO, 4>, (unsigned)tokens, 256, 0, stream, a) : launch_k(latent_store_kernel<TI, TO, 1>, (unsigned)tokens, 256, 0, stream, a))
+  const bool narrow = vec && ld_q <= 64 * kLatKeep && rank <= 64 * kLatKeep;     // short rows: more tokens per SM
+#define GB_LAT(TI, TO)                                                                                                                    \
+  (narrow ? launch_k(latent_store_kernel<TI, TO, 4, 64>, (unsigned)tokens, 64, 0, stream, a)                                               \
+   : vec  ? launch_k(latent_store_kernel<TI, TO, 4, 256>, (unsigned)tokens, 256, 0, stream, a)                                             \
+          : launch_k(latent_store_kernel<TI, TO, 1, 256>, (unsigned)tokens, 256, 0, stream, a))
   if (in_f32 && out_f32) GB_LAT(float, float);
   else if (in_f32) GB_LAT(float, __nv_bfloat16);
   else GB_LAT(__nv_bfloat16, __nv_bfloat16);

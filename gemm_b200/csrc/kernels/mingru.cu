@@ -28,15 +28,23 @@ struct MinGruArgs {
   int n;
 };
 
-// keep = 1 - z and add = z * candidate; sigmoid of either sign without cancellation
-__device__ __forceinline__ void gru_gate(float z, float u, float& keep, float& add) {
-  const float ez = __expf(-fabsf(z)), big = __fdividef(1.0f, 1.0f + ez), small = ez * big;     // sigmoid(|z|), sigmoid(-|z|)
-  keep = z >= 0.f ? small : big;
-  const float eu = __expf(fminf(u, 0.f));
-  const float cand = u >= 0.f ? u + 0.5f : __fdividef(eu, 1.0f + eu);
-  add = (z >= 0.f ? big : small) * cand;
+__device__ __forceinline__ float2 pair(float x) { return make_float2(x, x); }
+
+// keep = 1 - z and add = z * candidate of two channels, from the gate's logits and u.  The bound on the logit
+// keeps its exponential finite; the candidate is max(u, 0) + sigmoid(min(u, 0)); one reciprocal serves both sigmoids.
+__device__ __forceinline__ void gru_gate2(float2 z, float2 u, float2& keep, float2& add) {
+  constexpr float kLog2e = 1.4426950408889634f;
+  const float2 zs = __fmul2_rn(z, pair(kLog2e)), us = __fmul2_rn(u, pair(kLog2e));
+  const float2 ez = make_float2(fast_exp2(fminf(zs.x, 115.f)), fast_exp2(fminf(zs.y, 115.f)));
+  const float2 eu = make_float2(fast_exp2(fminf(us.x, 0.f)), fast_exp2(fminf(us.y, 0.f)));
+  const float2 nz = __fadd2_rn(ez, pair(1.0f)), nu = __fadd2_rn(eu, pair(1.0f)), d = __fmul2_rn(nz, nu);
+  const float2 r = make_float2(fast_rcp(d.x), fast_rcp(d.y));
+  const float2 gate = __fmul2_rn(ez, __fmul2_rn(r, nu));
+  keep = __ffma2_rn(gate, pair(-1.0f), pair(1.0f));            // exactly 1 behind a gate that is shut: a state may have to hold for very long
+  const float2 cand = __ffma2_rn(eu, __fmul2_rn(r, nz), make_float2(fmaxf(u.x, 0.f), fmaxf(u.y, 0.f)));
+  add = __fmul2_rn(gate, cand);
 }
-// The same with the full-precision functions (32-bit format).
+// One channel, with the full-precision functions (steps).
 __device__ __forceinline__ void gru_gate_exact(float z, float u, float& keep, float& add) {
   const float ez = expf(-fabsf(z)), big = 1.0f / (1.0f + ez), small = ez * big;
   keep = z >= 0.f ? small : big;
@@ -96,9 +104,8 @@ constexpr int kGruWarps = 16, kGruRun = 8;                     // tokens of a CT
 constexpr int kGruTile = kGruWarps * kGruRun, kGruCols = 64;   // a lane owns two neighbouring channels
 constexpr int kGruMaxCluster = 8;
 
-struct GruLoads { float2 z[kGruRun]; __nv_bfloat162 x[kGruRun], g[kGruRun]; };
-
-__global__ void __launch_bounds__(kGruWarps * 32)
+// Two CTAs share an SM: one's loads travel under the other's arithmetic.
+__global__ void __launch_bounds__(kGruWarps * 32, 2)
 mingru_scan_kernel(const MinGruArgs a, int cluster) {
   __shared__ float2 s_a[kGruWarps][32], s_b[kGruWarps][32];    // the warps' pairs
   __shared__ float2 s_ca[2][kGruMaxCluster][32], s_cb[2][kGruMaxCluster][32];     // the cluster's CTAs' pairs, by parity of the tile
@@ -121,49 +128,51 @@ mingru_scan_kernel(const MinGruArgs a, int cluster) {
   const __nv_bfloat16* xg = (const __nv_bfloat16*)a.xg;
   __nv_bfloat16* out = (__nv_bfloat16*)a.out;
   const int step = kGruTile * cluster;                         // tokens per round of the cluster
-  GruLoads ld;
-  auto fetch = [&](int base) {                                 // this warp's tokens of the round that starts at `base`
-#pragma unroll
-    for (int i = 0; i < kGruRun; ++i) {
-      const int t = base + rank * kGruTile + warp * kGruRun + i;
-      if (live && t < t1) {
-        ld.z[i] = *reinterpret_cast<const float2*>(a.z + (size_t)t * a.z_ld + c);
-        ld.x[i] = *reinterpret_cast<const __nv_bfloat162*>(xg + (size_t)t * a.ld + c);
-        ld.g[i] = *reinterpret_cast<const __nv_bfloat162*>(xg + (size_t)t * a.ld + a.n + c);
-      }
-    }
-  };
-  fetch(t0);
   for (int base = t0, round = 0; base < t1; base += step, ++round) {
     float2 keep[kGruRun], add[kGruRun];
-    __nv_bfloat162 g[kGruRun];
-    float2 pa = make_float2(1.f, 1.f), pb = make_float2(0.f, 0.f);
+    uint32_t g[kGruRun];
+    float2 pa = pair(1.f), pb = pair(0.f);
     const int first = base + rank * kGruTile + warp * kGruRun;
+    const int n_tok = live ? max(0, min(kGruRun, t1 - first)) : 0;
+    const float* zp = a.z + (size_t)first * a.z_ld + c;
+    const __nv_bfloat16* xp = xg + (size_t)first * a.ld + c;
+    // all loads in flight at once; keep holds the logits and add holds x for now
+    auto fetch = [&](int i) {
+      keep[i] = *reinterpret_cast<const float2*>(zp + (size_t)i * a.z_ld);
+      add[i].x = __uint_as_float(*reinterpret_cast<const uint32_t*>(xp + (size_t)i * a.ld));
+      g[i] = *reinterpret_cast<const uint32_t*>(xp + (size_t)i * a.ld + a.n);
+    };
+    auto form = [&](int i) {
+      const uint32_t u = __float_as_uint(add[i].x);
+      gru_gate2(__fadd2_rn(keep[i], zb), __fadd2_rn(make_float2(__uint_as_float(u << 16), __uint_as_float(u & 0xffff0000u)), xb), keep[i], add[i]);
+      pa = __fmul2_rn(pa, keep[i]);
+      pb = __ffma2_rn(keep[i], pb, add[i]);
+    };
+    if (n_tok == kGruRun) {
 #pragma unroll
-    for (int i = 0; i < kGruRun; ++i) {
-      keep[i] = make_float2(1.f, 1.f); add[i] = make_float2(0.f, 0.f);     // no token: the state stays
-      if (live && first + i < t1) {
-        const float2 x = __bfloat1622float2(ld.x[i]);
-        gru_gate(ld.z[i].x + zb.x, x.x + xb.x, keep[i].x, add[i].x);
-        gru_gate(ld.z[i].y + zb.y, x.y + xb.y, keep[i].y, add[i].y);
-      }
-      g[i] = ld.g[i];
-      pa.x *= keep[i].x; pa.y *= keep[i].y;
-      pb.x = fmaf(keep[i].x, pb.x, add[i].x); pb.y = fmaf(keep[i].y, pb.y, add[i].y);
+      for (int i = 0; i < kGruRun; ++i) fetch(i);
+#pragma unroll
+      for (int i = 0; i < kGruRun; ++i) form(i);
+    } else {
+#pragma unroll
+      for (int i = 0; i < kGruRun; ++i) { keep[i] = pair(1.f); add[i] = pair(0.f); g[i] = 0; }       // no token: the state stays
+#pragma unroll
+      for (int i = 0; i < kGruRun; ++i) if (i < n_tok) fetch(i);
+#pragma unroll
+      for (int i = 0; i < kGruRun; ++i) if (i < n_tok) form(i);
     }
-    if (base + step < t1) fetch(base + step);                  // the next round's rows travel while this one's pairs are exchanged
     s_a[warp][lane] = pa; s_b[warp][lane] = pb;
     __syncthreads();
     // the state in front of this CTA, and behind the whole round
     float2 cur = st, end;
     if (cluster > 1) {
       if (warp < cluster) {                                    // warp w hands the CTA's pair to CTA w of the cluster
-        float2 ta = make_float2(1.f, 1.f), tb = make_float2(0.f, 0.f);
+        float2 ta = pair(1.f), tb = pair(0.f);
 #pragma unroll
         for (int w = 0; w < kGruWarps; ++w) {
-          const float2 wa = s_a[w][lane], wb = s_b[w][lane];
-          ta.x *= wa.x; ta.y *= wa.y;
-          tb.x = fmaf(wa.x, tb.x, wb.x); tb.y = fmaf(wa.y, tb.y, wb.y);
+          const float2 wa = s_a[w][lane];
+          ta = __fmul2_rn(ta, wa);
+          tb = __ffma2_rn(wa, tb, s_b[w][lane]);
         }
         *cl.map_shared_rank(&s_ca[round & 1][rank][lane], warp) = ta;
         *cl.map_shared_rank(&s_cb[round & 1][rank][lane], warp) = tb;
@@ -172,34 +181,38 @@ mingru_scan_kernel(const MinGruArgs a, int cluster) {
       end = st;
       for (int r = 0; r < cluster; ++r) {
         if (r == rank) cur = end;
-        const float2 ra = s_ca[round & 1][r][lane], rb = s_cb[round & 1][r][lane];
-        end.x = fmaf(ra.x, end.x, rb.x); end.y = fmaf(ra.y, end.y, rb.y);
+        end = __ffma2_rn(s_ca[round & 1][r][lane], end, s_cb[round & 1][r][lane]);
       }
     }
     float2 mine = cur;                                         // in front of this warp
     if (cluster > 1) {
-      for (int w = 0; w < warp; ++w) {
-        const float2 wa = s_a[w][lane], wb = s_b[w][lane];
-        mine.x = fmaf(wa.x, mine.x, wb.x); mine.y = fmaf(wa.y, mine.y, wb.y);
-      }
+      for (int w = 0; w < warp; ++w) mine = __ffma2_rn(s_a[w][lane], mine, s_b[w][lane]);
     } else {
       end = cur;
 #pragma unroll
       for (int w = 0; w < kGruWarps; ++w) {
         if (w == warp) mine = end;
-        const float2 wa = s_a[w][lane], wb = s_b[w][lane];
-        end.x = fmaf(wa.x, end.x, wb.x); end.y = fmaf(wa.y, end.y, wb.y);
+        end = __ffma2_rn(s_a[w][lane], end, s_b[w][lane]);
       }
     }
     st = end;
+    __nv_bfloat16* op = out + (size_t)first * a.ld_out + c;
+    auto emit = [&](int i) {
+      mine = __ffma2_rn(keep[i], mine, add[i]);
+      const float2 y = make_float2(__uint_as_float(g[i] << 16), __uint_as_float(g[i] & 0xffff0000u)), e = __fmul2_rn(y, pair(-1.4426950408889634f));
+      const float2 d = __fadd2_rn(make_float2(fast_exp2(fminf(e.x, 115.f)), fast_exp2(fminf(e.y, 115.f))), pair(1.0f));
+      const float2 o = __fmul2_rn(__fmul2_rn(mine, y), make_float2(fast_rcp(d.x), fast_rcp(d.y)));
+      *reinterpret_cast<uint32_t*>(op + (size_t)i * a.ld_out) = pack_bf16x2(o.x, o.y);
+    };
+    if (n_tok == kGruRun) {
 #pragma unroll
-    for (int i = 0; i < kGruRun; ++i) {
-      mine.x = fmaf(keep[i].x, mine.x, add[i].x); mine.y = fmaf(keep[i].y, mine.y, add[i].y);
-      if (live && first + i < t1) {
-        const float2 y = __bfloat1622float2(g[i]);
-        *reinterpret_cast<uint32_t*>(out + (size_t)(first + i) * a.ld_out + c) =
-            pack_bf16x2(mine.x * __fdividef(y.x, 1.0f + __expf(-y.x)), mine.y * __fdividef(y.y, 1.0f + __expf(-y.y)));
-      } else if (c < a.ld_out && first + i < t1) *reinterpret_cast<uint32_t*>(out + (size_t)(first + i) * a.ld_out + c) = 0u;
+      for (int i = 0; i < kGruRun; ++i) emit(i);
+    } else {
+#pragma unroll
+      for (int i = 0; i < kGruRun; ++i) {
+        if (i < n_tok) emit(i);
+        else if (!live && c < a.ld_out && first + i < t1) *reinterpret_cast<uint32_t*>(op + (size_t)i * a.ld_out) = 0u;     // padding
+      }
     }
     __syncthreads();                                           // s_a, s_b are read
   }
@@ -225,8 +238,8 @@ GB_API int gb_mingru(const void* xg, int in_f32, int n_part, long part_stride, i
   if (parallel && !in_f32 && !out_f32 && n_part == 1 && z_part == 1 && n % 2 == 0 && ld % 2 == 0 && z_ld % 2 == 0 && ld_out % 2 == 0 && al(xg, 4) && al(z, 8) &&
       al(x_bias, 8) && al(z_bias, 8) && al(state, 8) && al(out, 4)) {
     const int blocks = (ld_out + kGruCols - 1) / kGruCols;
-    int cluster = 1;                                           // CTAs along the time axis: until the GPU is full or a round holds the longest sequence
-    while (cluster < kGruMaxCluster && (long)blocks * n_seqs * cluster < 2L * sm_count() && cluster * kGruTile < max_tokens) cluster *= 2;
+    int cluster = 1;                                           // CTAs along the time axis: while they fit the GPU at once and a round is shorter than the longest sequence
+    while (cluster < kGruMaxCluster && (long)blocks * n_seqs * cluster * 2 <= 2L * sm_count() && cluster * kGruTile < max_tokens) cluster *= 2;
     const dim3 grid((unsigned)(blocks * cluster), (unsigned)n_seqs);
     GB_CUDA_OK(launch_k_cluster(mingru_scan_kernel, grid, kGruWarps * 32, 0, stream, (unsigned)cluster, a, cluster));
     return 0;

@@ -850,14 +850,16 @@ class Transformer:
                 y = gemm.grouped_linear(hq, lw.w2.mx.data.view(e, hid, inter), pl.seg_start, pl.seg_count, tn, sfa=lw.w2.mx.sf, sfb=hsf,
                                         w_tiled=lw.w2.mx.tiled, pair_rows=(tn == 32 and PAIR_DOWN))
         else:
-            tn = gemm.pick_tn(max(1, (t * k + n_exp - 1) // n_exp), dual=True)
+            per = max(1, (t * k + n_exp - 1) // n_exp)       # expected rows per expert
+            tn = gemm.pick_tn(per, dual=True)
+            wide = 256 if per >= 96 and tn == 128 else tn     # token tile of the products with one accumulator
             if moe.can_prep(h, lw.router, k):
                 ids, wts, pl, xs = moe.prep_hidden(h, lw.router, k, e, tn, quantize=False, **rt)
             else:
                 ids, wts, pl = moe.route_plan_hidden(h, lw.router, k, e, tn, **rt)
                 xs = moe.gather_rows(h, pl.row_token)
-            act = gemm.grouped_linear(xs, lw.w13.w.view(e, -1, hid), pl.seg_start, pl.seg_count, tn, dual=gated, gelu=not gated, w_tiled=lw.w13.tiled)
-            y = gemm.grouped_linear(act, lw.w2.w.view(e, -1, inter), pl.seg_start, pl.seg_count, tn, w_tiled=lw.w2.tiled)
+            act = gemm.grouped_linear(xs, lw.w13.w.view(e, -1, hid), pl.seg_start, pl.seg_count, tn if gated else wide, dual=gated, gelu=not gated, w_tiled=lw.w13.tiled)
+            y = gemm.grouped_linear(act, lw.w2.w.view(e, -1, inter), pl.seg_start, pl.seg_count, wide, w_tiled=lw.w2.tiled)
         return moe.PendingCombine(y, pl.pair_row, wts, t, k)
 
     # ------------------------------------------------------------------------------------------------

@@ -24,6 +24,8 @@ Cases
                scans and Delta-Net; latent attention and plain attention; Dynamic-Tanh stream and RMSNorm, part norm, convolution, routing
   fidolix      the kernels of Fidolix at the sizes of ``fidolix-30b-a3b`` beside the like kernels of the other models: RWKV (HGRN2), token shift,
                convolution and rotation, norms of Q and K, capped scores and sinks (plain attention), the stream's norms and sums
+  zedirax      the kernels of Zedirax at the sizes of ``zedirax-30b-a3b`` beside the like kernels of the other models: minGRU (HGRN2), logarithmic distance
+               bias (a table of biases, plain attention), the average over earlier layers (the stream's norms and sums), GELU epilogues
   spec_verify  whole-model step over 1, 2, 3 and 5 positions per sequence (speculative verification against plain decode);
                builds the full Qwen3-30B-A3B shape, not part of ``all``
 
@@ -669,10 +671,109 @@ def case_fidolix(args):
         del wg
 
 
+def case_zedirax(args):
+    from ..models.config import get_config
+    from ..ops import latent, recurrent, stream
+    dev, page = "cuda", 128
+    cfg = get_config("zedirax-30b-a3b")
+    spec = {sp.mixer: sp for sp in cfg.layer_specs}
+    gr, at, la, h = spec["mingru"], spec["attention"], spec["latent"], cfg.hidden
+    for name, lens in (("decode_1", [1]), ("decode_64", [1] * 64), ("prefill_1x1024", [1024]), ("prefill_1x8192", [8192]), ("prefill_8x2048", [2048] * 8)):
+        t, b, dec = sum(lens), len(lens), len(lens) == sum(lens)
+        cu = torch.tensor([0] + list(torch.tensor(lens).cumsum(0)), dtype=torch.int32, device=dev)
+        sl = torch.arange(b, dtype=torch.int32, device=dev)
+        pos = torch.arange(t, device=dev, dtype=torch.int32)
+        n, dt = gr.v_dim, torch.float32 if dec else torch.bfloat16
+        es = 4 if dec else 2
+        xg, z = torch.randn(t, 2 * n, device=dev).to(dt), torch.randn(t, n, device=dev) - 3
+        zero, st = torch.zeros(n, device=dev), torch.zeros(b, 1, 1, n, device=dev)
+        _run(f"mingru_{name}", lambda: recurrent.mingru(xg, z, 0, zero, zero, st, cu, sl, n, max(lens)), 0.0, t * n * (2 * es + 4 + 2) + 2 * st.numel() * 4, args)
+        hd, d = 16, 128
+        n2 = hd * d
+        qv, f, s2 = xg[:, : 2 * n2].contiguous(), z[:, :n2].contiguous(), torch.zeros(b, hd, d, d, device=dev)
+        low = torch.full((n2,), 0.3, device=dev)
+        _run(f"gla_{name}", lambda: recurrent.gla(qv, f, 0, zero[:n2], low, s2, cu, sl, hd, d, d, not dec, max(lens)), 4.0 * t * hd * d * d,
+             2 * s2.numel() * 4 + t * (2 * n2 * es + n2 * 4 + n2 * 4), args)
+        del xg, z, qv, f
+        nq, nk = at.q_dim, at.n_kv_heads * at.head_dim
+        rows = torch.randn(t, nq + 2 * nk, device=dev).to(dt)
+        kc, vc = (torch.empty(t, at.n_kv_heads, at.head_dim, device=dev, dtype=torch.bfloat16) for _ in range(2))
+        by = t * (nq + 2 * nk) * (es + 2)
+        for nm, kw in (("temperature", dict(unit=False, positions=pos, temp=(0.1, 8192.0))), ("unit", {})):
+            _run(f"qk_{nm}_{name}", lambda: stream.qk_unit(rows, pos, kc, vc, at.n_heads, at.n_kv_heads, at.head_dim, at.v_dim, 1e-5, 0.1, **kw), 0.0, by, args)
+        del rows
+        r, rd, qn = la.kv_rank, la.rot_dim, la.n_heads * (la.head_dim + la.rot_dim)
+        rows = torch.randn(t, qn + r + rd + la.n_heads * la.v_dim, device=dev).to(dt)
+        cache, freq = torch.empty(t, 1, r + rd, device=dev, dtype=torch.bfloat16), torch.tensor(la.rotary.frequencies(), dtype=torch.float64, device=dev)
+        one = torch.ones(1536, device=dev)
+        _run(f"latent_store_alone_{name}", lambda: latent.latent_store(rows, pos, pos, None, one[:r], freq, 1.0, cache, 0, r, rd, 1e-5, torch.bfloat16, qn), 0.0, t * (r + rd) * (es + 2), args)
+        _run(f"latent_store_with_q_{name}", lambda: latent.latent_store(rows, pos, pos, one, one[:r], freq, 1.0, cache, 1536, r, rd, 1e-5, torch.bfloat16), 0.0, t * (1536 + r + rd) * (es + 2), args)
+        a = torch.randn(t, la.n_heads, la.v_dim, device=dev).bfloat16()
+        _run(f"sigmoid_gate_{name}", lambda: stream.sigmoid_gate(a, rows, qn + r + rd, la.v_dim), 0.0, a.numel() * (4 + es), args)
+        del rows, a
+    for name, b, q_len, ctx in (("decode_1x32768", 1, 1, 32767), ("decode_64x2048", 64, 1, 2047), ("decode_64x8192", 64, 1, 8191), ("prefill_1x8192", 1, 8192, 0), ("prefill_8x2048", 8, 2048, 0)):
+        hq, hkv, d = at.n_heads, at.n_kv_heads, at.head_dim
+        kv, dec = ctx + q_len, q_len == 1
+        pages = (kv + page - 1) // page
+        k, v = ((torch.randn((b * pages + 1) * page, hkv, d, device=dev) * 0.5).bfloat16() for _ in range(2))
+        bt = torch.arange(b * pages, device=dev, dtype=torch.int32).reshape(b, pages) + 1
+        cu, kvl = torch.tensor([i * q_len for i in range(b + 1)], device=dev, dtype=torch.int32), torch.full((b,), kv, device=dev, dtype=torch.int32)
+        seen = float(sum(i + 1 for i in range(ctx, kv)) * b)
+        by = b * kv * hkv * d * 4 + b * q_len * hq * d * 4
+        splits = att.pick_splits(b, hkv, kv) if dec else 1
+        plan = (att.build_work([q_len] * b, hq, hkv, splits).to(dev), splits)
+        q = (torch.randn(b * q_len, hq, d, device=dev) * 0.5 * d ** -0.5 * att.LOG2E).bfloat16()
+        table = att.distance_bias_table(torch.randn(32, hq), 8192).to(dev)
+        lb = torch.rand(2, hq, device=dev)
+        run = lambda nm, **kw: _run(f"attn_{nm}_{name}", lambda: att.attention_masked(q, k, v, cu, kvl, bt, page, plan=plan, decode=dec, **kw), 4.0 * seen * hq * d, by, args, splits=splits)
+        run("log_bias", log_bias=lb)
+        run("table_bias", bias=table)
+        _run(f"attn_{name}", lambda: att.attention(q, k, v, cu, kvl, bt, page, plan[0], num_splits=splits, decode=dec), 4.0 * seen * hq * d, by, args, splits=splits)
+        del k, v
+    for t in (1, 64, 8192):
+        x, u = torch.randn(t, h, device=dev), torch.randn(t, h, device=dev)
+        w1 = torch.ones(h, device=dev)
+        _run(f"stream_norm_gate_{t}x{h}", lambda: stream.norm_gate(x, w1, 1e-5, stream.Update([(u, 0.5, None)]), w1), 0.0, t * h * 14, args)
+        _run(f"stream_norm_{t}x{h}", lambda: stream.norm(x, w1, 1e-5, u), 0.0, t * h * 14, args)
+        k, places = 8, 46
+        y = torch.randn(t * k, h, device=dev).bfloat16()
+        pend = moe.PendingCombine(y, torch.randperm(t * k, device=dev).to(torch.int32), torch.rand(t, k, device=dev), t, k)
+        hist, gate = torch.randn(places, t, h, device=dev), torch.rand(t, device=dev)
+        coef = [torch.full((p + 1,), 0.02, device=dev) for p in range(places)]
+        bs = stream.depth_base(hist, 41, coef[41:46])
+        for nm, p, base, first in (("1_place", 1, None, 0), ("8_places", 8, None, 0), ("41_and_4_places", 45, bs[4], 41)):
+            _run(f"stream_depth_moe_{nm}_{t}x{h}", lambda: stream.norm(x, w1, 1e-5, stream.Update([(pend, 0.5, None), (u, 0.5, gate)], stream.Depth(hist, p, coef[p], base, first))), 0.0,
+                 t * h * (4 * (4 + p - first + (base is not None)) + 2 * k + 2), args)
+        ones = [torch.full((46,), 0.02, device=dev) for _ in range(8)]
+        _run(f"depth_base_41_places_{t}x{h}", lambda: stream.depth_base(hist, 41, ones), 0.0, t * h * 4 * (41 + 8), args)
+        _run(f"stream_join_moe_{t}x{h}", lambda: stream.join(x, [(u, 1.0), (pend, 1.0)], torch.bfloat16), 0.0, t * h * (14 + 2 * k), args)
+        xb = x.bfloat16()
+        _run(f"rmsnorm_moe_{t}x{h}", lambda: ew.rmsnorm(pend, w1.bfloat16(), 1e-5, residual=xb), 0.0, t * h * (6 + 2 * k), args)
+        del hist, y, pend
+        ff = 6144
+        wg = mxfp8.tile_weight((torch.randn(2 * ff, h, device=dev) * 0.02).bfloat16())
+        bias = torch.randn(2 * ff, device=dev)
+        for nm, kw in (("gelu_biased", dict(bias=bias)), ("gelu", {})):
+            _run(f"gate_up_{nm}_{t}", lambda: gemm.linear_swiglu(xb, wg, w_tiled=True, act="gelu_tanh", **kw), 4.0 * t * ff * h, 2 * ff * h * 2 + t * h * 2 + t * ff * 2, args)
+        for nm, kw in (("gelu_erf", dict(gelu=True)), ("plain", {})):
+            _run(f"gemm_{nm}_{t}", lambda: gemm.linear(xb, wg, w_tiled=True, **kw), 4.0 * t * ff * h, 2 * ff * h * 2 + t * h * 2 + 2 * t * ff * 2, args)
+        del wg
+        # experts: plain ones of 1152, gated ones of 768
+        e, mo = 128, la.moe
+        tn = gemm.pick_tn(max(1, (t * k + e - 1) // e), dual=True)
+        _, _, pl = moe.route_plan(torch.randn(t, e, device=dev), k, e, tn)
+        xs = moe.gather_rows(xb, pl.row_token)
+        used = min(t * k, e)
+        for nm, rows, kw in (("plain_gelu", mo.ffn, dict(gelu=True)), ("plain", mo.ffn, {}), ("gated_silu", 2 * 768, dict(dual=True))):
+            we = mxfp8.tile_weight((torch.randn(e * rows, h, device=dev) * 0.02).bfloat16()).view(e, rows, h)
+            _run(f"experts_up_{nm}_{t}", lambda: gemm.grouped_linear(xs, we, pl.seg_start, pl.seg_count, tn, w_tiled=True, **kw), 2.0 * t * k * rows * h, used * rows * h * 2 + t * k * (h + rows) * 2, args)
+            del we
+
+
 MODEL_CASES = {"spec_verify": case_spec_verify}      # build the whole benchmark model: not part of --case all
 CASES = {"gemm": case_gemm, "moe_decode": case_moe_decode, "moe_prefill": case_moe_prefill, "attn_decode": case_attn_decode,
          "attn_prefill": case_attn_prefill, "lm_head": case_lm_head, "quant": case_quant, "small": case_small, "layered": case_layered,
-         "famepel": case_famepel, "fidolix": case_fidolix}
+         "famepel": case_famepel, "fidolix": case_fidolix, "zedirax": case_zedirax}
 
 
 def main(argv=None):
