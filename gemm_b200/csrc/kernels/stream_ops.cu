@@ -388,40 +388,31 @@ struct DepthArgs {
   int width; float eps;
 };
 
-template <typename TO, int V, int VPT>             // V columns at a time, VPT times: width <= 256 * V * VPT, a multiple of V
+template <typename TO, int VPT>                    // VPT float4 per thread, width <= 1024 * VPT and width % 4 == 0
 __global__ void __launch_bounds__(256)
-stream_depth_kernel(const DepthArgs a) {
+stream_depth_vec_kernel(const DepthArgs a) {
   pdl_wait();
   pdl_trigger();
   __shared__ float red[8];
   const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
-  auto load = [&](const float* p, float* v) {
-    if constexpr (V == 4) { const float4 q = ld4(p); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
-    else v[0] = *p;
-  };
-  auto store = [&](auto* p, const float* v) {
-    if constexpr (V == 4) st4(p, make_float4(v[0], v[1], v[2], v[3]));
-    else st_f(p, v[0]);
-  };
-  float x[VPT][V];
+  const int nv = a.width >> 2;
   const float w_at = a.w[a.at];
+  float4 x[VPT];
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
-    const int c = (threadIdx.x + i * 256) * V;
+    const int c = threadIdx.x + i * 256;
+    x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c >= nv) continue;
+    float v[4];
+    *reinterpret_cast<float4*>(v) = ld4(a.x + src * a.width + c * 4);
 #pragma unroll
-    for (int j = 0; j < V; ++j) x[i][j] = 0.f;
-    if (c >= a.width) continue;
-    load(a.x + src * a.width + c, x[i]);
-#pragma unroll
-    for (int p = 0; p < 3; ++p) if (p < a.n) add_part<V>(a.part[p], src, c, x[i]);
-    if (a.rows == nullptr) store(a.hist + (size_t)a.at * a.stride + src * a.width + c, x[i]);
-#pragma unroll
-    for (int j = 0; j < V; ++j) x[i][j] *= w_at;
+    for (int p = 0; p < 3; ++p) if (p < a.n) add_part<4>(a.part[p], src, c * 4, v);
+    x[i] = make_float4(v[0], v[1], v[2], v[3]);
+    if (a.rows == nullptr) st4(a.hist + (size_t)a.at * a.stride + src * a.width + c * 4, x[i]);
+    x[i].x *= w_at; x[i].y *= w_at; x[i].z *= w_at; x[i].w *= w_at;
     if (a.base != nullptr) {
-      float q[V];
-      load(a.base + src * a.width + c, q);
-#pragma unroll
-      for (int j = 0; j < V; ++j) x[i][j] += q[j];
+      const float4 q = ld4(a.base + src * a.width + c * 4);
+      x[i].x += q.x; x[i].y += q.y; x[i].z += q.z; x[i].w += q.w;
     }
   }
 #pragma unroll 4
@@ -430,35 +421,60 @@ stream_depth_kernel(const DepthArgs a) {
     const float* h = a.hist + (size_t)j * a.stride + src * a.width;
 #pragma unroll
     for (int i = 0; i < VPT; ++i) {
-      const int c = (threadIdx.x + i * 256) * V;
-      if (c >= a.width) continue;
-      float q[V];
-      load(h + c, q);
-#pragma unroll
-      for (int y = 0; y < V; ++y) x[i][y] = fmaf(w, q[y], x[i][y]);
+      const int c = threadIdx.x + i * 256;
+      if (c >= nv) continue;
+      const float4 q = ld4(h + c * 4);
+      x[i].x = fmaf(w, q.x, x[i].x); x[i].y = fmaf(w, q.y, x[i].y); x[i].z = fmaf(w, q.z, x[i].z); x[i].w = fmaf(w, q.w, x[i].w);
     }
   }
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
-    const int c = (threadIdx.x + i * 256) * V;
-#pragma unroll
-    for (int j = 0; j < V; ++j) ss += x[i][j] * x[i][j];
-    if (c < a.width && a.rows == nullptr) store(a.x + src * a.width + c, x[i]);
+    const int c = threadIdx.x + i * 256;
+    ss += x[i].x * x[i].x + x[i].y * x[i].y + x[i].z * x[i].z + x[i].w * x[i].w;
+    if (c < nv && a.rows == nullptr) st4(a.x + src * a.width + c * 4, x[i]);
   }
   if (a.out == nullptr) return;
   const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.width + a.eps);
   TO* o = (TO*)a.out + r * a.ld_out;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
-    const int c = (threadIdx.x + i * 256) * V;
-    if (c >= a.width) continue;
-    float w[V], y[V];
-    load(a.weight + c, w);
-#pragma unroll
-    for (int j = 0; j < V; ++j) y[j] = x[i][j] * inv * w[j];
-    store(o + c, y);
+    const int c = threadIdx.x + i * 256;
+    if (c >= nv) continue;
+    const float4 w = ld4(a.weight + c * 4);
+    st4(o + c * 4, make_float4(x[i].x * inv * w.x, x[i].y * inv * w.y, x[i].z * inv * w.z, x[i].w * inv * w.w));
   }
+  for (int c = a.width + threadIdx.x; c < a.ld_out; c += 256) st_f(o + c, 0.f);
+}
+
+template <typename TO>                             // any width
+__global__ void __launch_bounds__(256)
+stream_depth_any_kernel(const DepthArgs a) {
+  pdl_wait();
+  pdl_trigger();
+  __shared__ float red[8];
+  const size_t r = blockIdx.x, src = a.rows != nullptr ? (size_t)a.rows[r] : r;
+  const size_t at = src * a.width;
+  const bool in_place = a.rows == nullptr;
+  auto average = [&](int c) {
+    float x = a.x[at + c];
+    for (int p = 0; p < a.n; ++p) add_part<1>(a.part[p], src, c, &x);
+    if (in_place) a.hist[(size_t)a.at * a.stride + at + c] = x;
+    float s = x * a.w[a.at];
+    if (a.base != nullptr) s += a.base[at + c];
+    for (int j = a.first; j < a.at; ++j) s = fmaf(a.w[j], a.hist[(size_t)j * a.stride + at + c], s);
+    return s;
+  };
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < a.width; c += 256) {
+    const float v = average(c);
+    if (in_place) a.x[at + c] = v;
+    ss += v * v;
+  }
+  if (a.out == nullptr) return;
+  const float inv = 1.0f / sqrtf(block_sum_256(ss, red) / (float)a.width + a.eps);
+  TO* o = (TO*)a.out + r * a.ld_out;
+  for (int c = threadIdx.x; c < a.width; c += 256) st_f(o + c, (in_place ? a.x[at + c] : average(c)) * inv * a.weight[c]);
   for (int c = a.width + threadIdx.x; c < a.ld_out; c += 256) st_f(o + c, 0.f);
 }
 
@@ -1123,13 +1139,11 @@ GB_API int gb_stream_join(float* x, const JoinPart* parts, int n, void* out, int
 template <typename TO>
 static int stream_depth_launch(const DepthArgs& a, bool vec, int n_rows, cudaStream_t stream) {
   const unsigned g = (unsigned)n_rows;
-  if (vec && a.width <= 1024) launch_k(stream_depth_kernel<TO, 4, 1>, g, 256, 0, stream, a);
-  else if (vec && a.width <= 2048) launch_k(stream_depth_kernel<TO, 4, 2>, g, 256, 0, stream, a);
-  else if (vec && a.width <= 4096) launch_k(stream_depth_kernel<TO, 4, 4>, g, 256, 0, stream, a);
-  else if (vec && a.width <= 16384) launch_k(stream_depth_kernel<TO, 4, 16>, g, 256, 0, stream, a);
-  else if (a.width <= 1024) launch_k(stream_depth_kernel<TO, 1, 4>, g, 256, 0, stream, a);
-  else if (a.width <= 16384) launch_k(stream_depth_kernel<TO, 1, 64>, g, 256, 0, stream, a);
-  else return fail("stream_depth: rows of at most 16384 columns%s");
+  if (vec && a.width <= 1024) launch_k(stream_depth_vec_kernel<TO, 1>, g, 256, 0, stream, a);
+  else if (vec && a.width <= 2048) launch_k(stream_depth_vec_kernel<TO, 2>, g, 256, 0, stream, a);
+  else if (vec && a.width <= 4096) launch_k(stream_depth_vec_kernel<TO, 4>, g, 256, 0, stream, a);
+  else if (vec && a.width <= 16384) launch_k(stream_depth_vec_kernel<TO, 16>, g, 256, 0, stream, a);
+  else launch_k(stream_depth_any_kernel<TO>, g, 256, 0, stream, a);
   GB_CUDA_OK(cudaGetLastError());
   return 0;
 }
